@@ -38,7 +38,7 @@
 extern "C" {
 #endif
 
-#define B200_ABI_VERSION 9
+#define B200_ABI_VERSION 10
 
 #define B200_DTYPE_F32 0
 #define B200_DTYPE_BF16 1
@@ -470,6 +470,77 @@ size_t b200_lm_head_argmax_workspace_bytes(int32_t num_rows, int32_t vocab_size)
 int b200_lm_head_argmax(const void* hidden, const void* w, const void* bias, int64_t* tokens, int32_t num_rows,
                         int32_t vocab_size, int32_t k_dim, void* workspace, size_t workspace_bytes,
                         int32_t dtype, int32_t* status, void* stream);
+
+/* ---------------------------------------------------------------------------------------------
+ * Mechanisms of decoders with hyper-connected residual streams, talking-heads attention and a gated linear
+ * recurrence (the Nabalix family; the reference has no counterpart).  All constants are parameters.
+ * ------------------------------------------------------------------------------------------- */
+
+/* store_kvcache for a pool whose key and value rows differ in width: k_cache [num_slots, k_width],
+ * v_cache [num_slots, v_width]; strides in elements, slots < 0 are skipped. */
+int b200_store_kv_rows(const void* k, const void* v, int64_t k_token_stride, int64_t v_token_stride, void* k_cache,
+                       void* v_cache, const int64_t* slot_mapping, int32_t num_tokens, int32_t k_width,
+                       int32_t v_width, int64_t num_slots, int32_t dtype, int32_t* status, void* stream);
+
+/* One sublayer boundary of a decoder with `streams` (1..8) fp32 residual streams x [rows, streams, dim], in place:
+ *   y     = y0, or (rms(y0) join_w0 + rms(y1) join_w1) / 2 with y1 (eps join_eps); times layer_scale [dim] if given
+ *   x'[t] = sum_s mix[s, t] x[s] + out_w[t] y          (mix [streams, streams] from-to; y0 == NULL: x' = x)
+ *   u     = sum_t in_w[t] x'[t]                        (in_w == NULL: the plain sum)
+ *   h     = u / sqrt(mean(u^2) + eps) * (norm_w + (norm_plus_one ? 1 : 0))     in `dtype`; h == NULL: not formed
+ * With `embed` [vocab, dim] (dtype) and tokens int64 [rows] every stream starts as the token's row (no update).
+ * y0, y1 [rows, dim] in dtype; all other vectors fp32.  A token id outside the table reads row 0 and reports
+ * B200_ERR_BOUNDS. */
+int b200_stream_update(float* x, const int64_t* tokens, const void* embed, int64_t vocab, const void* y0, const void* y1,
+                       const float* join_w0, const float* join_w1, float join_eps, const float* layer_scale,
+                       const float* mix, const float* out_w, const float* in_w, const float* norm_w,
+                       int32_t norm_plus_one, float eps, void* h, int64_t rows, int32_t streams, int32_t dim,
+                       int32_t dtype, int32_t* status, void* stream);
+
+/* act [rows, d_ff] = g sigmoid(slope g) (u + 1) for h [rows, 2 d_ff] = [gate | up], g = min(gate, limit),
+ * u = clamp(up, -limit, limit); fp32 arithmetic, one rounding. */
+int b200_clamped_glu(const void* h, void* act, int64_t rows, int32_t d_ff, float limit, float slope, int32_t dtype,
+                     void* stream);
+
+/* Causal attention over a paged pool with heads mixed before the softmax; for a query at position i
+ *   s[g, j] = softcap tanh(scale q[g].k[j] / softcap) - r1[g] ln(1 + r2[g] (i - j))   (softcap <= 0: no cap)
+ *   m[h, j] = sum_g talk[h, g] s[g, j],  softmax over 0 <= i - j < window (window <= 0: all earlier keys),
+ *   out[h]  = sum_j softmax(m[h])_j v[j] * sigmoid(gate[h])                            (gate == NULL: no gate)
+ * Query head h reads key / value head h / (num_heads / num_kv_heads).  q [rows, num_heads * dim_k], gate
+ * [rows, num_heads * dim_v] with free row strides; out [rows, num_heads, dim_v]; caches [num_blocks, block_size,
+ * num_kv_heads, dim].  The rows of sequence s are cu_seqlens_q[s] .. cu_seqlens_q[s+1]-1, its context (which the
+ * pool already holds, the new rows included) is cu_seqlens_k[s+1]-cu_seqlens_k[s] long; with cu_seqlens_q ==
+ * NULL row i is the last token of sequence i and context_lens[i] its length (0: padding row, nothing written).
+ * Rows beyond the last sequence are padding.  max_seqlen_q: host bound on rows per sequence.
+ * r1, r2 [num_heads] and talk [num_heads, num_heads] fp32 (device); bias_table [bias_len, num_heads] fp32 or
+ * NULL: r1 ln(1 + r2 distance) for distances 0 .. bias_len - 1; talk_host: the same matrix on the host (may be
+ * NULL: general kernel).  Workspace: b200_talking_attention_workspace_bytes(). */
+size_t b200_talking_attention_workspace_bytes(int32_t num_seqs, int32_t num_heads, int32_t dim_v, int32_t window,
+                                              int32_t decode, int32_t dtype);
+int b200_talking_attention(const void* q, int64_t q_stride, const void* gate, int64_t gate_stride, const void* k_cache,
+                           const void* v_cache, void* out, const int32_t* block_tables, int64_t bt_stride,
+                           int32_t block_size, int64_t num_blocks, const int32_t* cu_seqlens_q,
+                           const int32_t* cu_seqlens_k, const int64_t* context_lens, int32_t num_seqs, int64_t rows,
+                           int32_t max_seqlen_q, int32_t num_heads, int32_t num_kv_heads, int32_t dim_k, int32_t dim_v,
+                           float scale, float softcap, const float* r1, const float* r2, const float* talk,
+                           const float* talk_host, const float* bias_table, int32_t bias_len, int32_t window,
+                           void* workspace, size_t workspace_bytes, int32_t dtype, int32_t* status, void* stream);
+
+/* Gated linear recurrence (HGRN2) over per-sequence states: per head
+ *   q = silu(q_in), f = lower + (1 - lower) sigmoid(f_in + f_bias), S <- diag(f) S + (1 - f) v^T, o = S^T q,
+ *   out = o / sqrt(mean(o^2) + eps) * norm_w
+ * q, f [tokens, heads * dim_k], v [tokens, heads * dim_v] with one token stride (views of one projection);
+ * f_bias, lower [heads, dim_k], norm_w [dim_v] fp32; state fp32 [num_slots, heads, dim_k, dim_v], slot of
+ * sequence s = state_slots[s] (< 0: skipped).  Sequence ranges as in b200_talking_attention; a sequence whose
+ * first token of the call is at position 0 starts from the zero state.  out [tokens, heads, dim_v] in dtype.
+ * max_seqlen_q, total_tokens: host bounds (workspace: b200_gated_recurrence_workspace_bytes()). */
+size_t b200_gated_recurrence_workspace_bytes(int32_t num_seqs, int64_t total_tokens, int32_t max_seqlen_q,
+                                             int32_t num_heads, int32_t dim_k, int32_t dim_v);
+int b200_gated_recurrence(const void* q, const void* f, const void* v, int64_t token_stride, const float* f_bias,
+                          const float* lower, const float* norm_w, float eps, float* state, int64_t num_slots,
+                          const int64_t* state_slots, const int32_t* cu_seqlens_q, const int32_t* cu_seqlens_k,
+                          const int64_t* context_lens, int32_t num_seqs, int64_t total_tokens, int32_t max_seqlen_q,
+                          int32_t num_heads, int32_t dim_k, int32_t dim_v, void* out, void* workspace,
+                          size_t workspace_bytes, int32_t dtype, int32_t* status, void* stream);
 
 /* ---------------------------------------------------------------------------------------------
  * Diagnostic (no counterpart in the reference, which has no device code): runs the give-up path of the

@@ -6,6 +6,7 @@ cross-compiles without a GPU.  Run ``python -m llm_from_scratch_b200._build`` or
 """
 from __future__ import annotations
 
+import fcntl
 import os
 import shutil
 import subprocess
@@ -42,12 +43,44 @@ def _stale(target: Path, deps: list[Path]) -> bool:
     return any(d.stat().st_mtime > t for d in deps)
 
 
-def build(force: bool = False, verbose: bool = False) -> Path:
-    """Compile every kernel source and link ``libb200llm.so``; returns its path."""
-    nvcc = _nvcc()
-    OBJ_DIR.mkdir(exist_ok=True)
-    headers = sorted(CSRC.glob("*.cuh")) + sorted(INCLUDE.glob("*.h")) + [Path(__file__)]
+# Sources a model family runs on, where that is not the whole library: ``ensure`` builds a library of just these
+# when the full one is absent.  "api" and "host_path" are the parts every engine uses.
+FAMILY_SOURCES = {
+    "Nabalix": ("api", "host_path", "decode_advance", "sampler", "moe_gemm", "moe_gemm_rows", "store_kvcache", "streams",
+                "talking_attention", "gated_recurrence"),
+}
+
+
+def _headers() -> list[Path]:
+    return sorted(CSRC.glob("*.cuh")) + sorted(INCLUDE.glob("*.h")) + [Path(__file__)]
+
+
+def ensure(family: str | None = None) -> Path:
+    """A library that can run ``family`` (an ``architecture`` name), built if need be: the full library when it
+    is there and current, else one of the family's sources only.  Sets ``B200LLM_LIBRARY`` for ``_lib``."""
     sources = sorted(CSRC.glob("*.cu"))
+    if not _stale(LIB_PATH, sources + _headers()) or family not in FAMILY_SOURCES:
+        path = build()
+    else:
+        names = FAMILY_SOURCES[family]
+        path = build(sources=[CSRC / f"{n}.cu" for n in names], target=PKG / f"libb200llm_{family.lower()}.so")
+    os.environ["B200LLM_LIBRARY"] = str(path)
+    return path
+
+
+def build(force: bool = False, verbose: bool = False, sources: list[Path] | None = None,
+          target: Path | None = None) -> Path:
+    """Compile every kernel source and link ``libb200llm.so`` (or the given sources into ``target``); returns its
+    path.  Builds of one checkout take turns."""
+    OBJ_DIR.mkdir(exist_ok=True)
+    with open(OBJ_DIR / "lock", "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        return _build_locked(force, verbose, sources or sorted(CSRC.glob("*.cu")), target or LIB_PATH)
+
+
+def _build_locked(force: bool, verbose: bool, sources: list[Path], target: Path) -> Path:
+    nvcc = _nvcc()
+    headers = _headers()
     jobs = []
     for src in sources:
         obj = OBJ_DIR / (src.stem + ".o")
@@ -70,13 +103,13 @@ def build(force: bool = False, verbose: bool = False) -> Path:
         with ThreadPoolExecutor(max_workers=min(8, len(jobs))) as ex:
             list(ex.map(compile_one, jobs))
     objs = [OBJ_DIR / (s.stem + ".o") for s in sources]
-    if force or jobs or _stale(LIB_PATH, objs):
+    if force or jobs or _stale(target, objs):
         cmd = [nvcc, "-shared", "-gencode", "arch=compute_100a,code=sm_100a",
-               "-o", str(LIB_PATH), *map(str, objs)]
+               "-o", str(target), *map(str, objs)]
         r = subprocess.run(cmd, capture_output=True, text=True)
         if r.returncode != 0:
             raise RuntimeError(f"link failed:\n{r.stdout}\n{r.stderr}")
-    return LIB_PATH
+    return target
 
 
 if __name__ == "__main__":

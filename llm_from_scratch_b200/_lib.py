@@ -5,9 +5,11 @@ There is no fallback: if the library has not been built, importing this module r
 from __future__ import annotations
 
 import ctypes as C
+import os
 from pathlib import Path
 
-LIB_PATH = Path(__file__).resolve().parent / "libb200llm.so"
+# B200LLM_LIBRARY: a library built from one model family's sources (``_build.ensure``) instead of the full one
+LIB_PATH = Path(os.environ.get("B200LLM_LIBRARY") or Path(__file__).resolve().parent / "libb200llm.so")
 
 DTYPE_F32 = 0
 DTYPE_BF16 = 1
@@ -67,6 +69,17 @@ SIGNATURES = {
     "b200_decode_advance": (_i32, [_vp, _vp, _vp, _vp, _vp, _i64, _i32, _i64, _i32, _vp, _vp, _vp]),
     "b200_block_table_patch": (_i32, [_vp, _i32, _vp, _i64, _i32, _vp, _vp]),
     "b200_sample": (_i32, [_vp, _i64, _vp, _i64, _i32, _u64, _u64, _vp, _i32, _vp]),
+    "b200_store_kv_rows": (_i32, [_vp, _vp, _i64, _i64, _vp, _vp, _vp, _i32, _i32, _i32, _i64, _i32, _vp, _vp]),
+    "b200_stream_update": (_i32, [_vp, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _f32, _vp, _vp, _vp, _vp, _vp, _i32, _f32,
+                                  _vp, _i64, _i32, _i32, _i32, _vp, _vp]),
+    "b200_clamped_glu": (_i32, [_vp, _vp, _i64, _i32, _f32, _f32, _i32, _vp]),
+    "b200_talking_attention_workspace_bytes": (_sz, [_i32, _i32, _i32, _i32, _i32, _i32]),
+    "b200_talking_attention": (_i32, [_vp, _i64, _vp, _i64, _vp, _vp, _vp, _vp, _i64, _i32, _i64, _vp, _vp, _vp, _i32,
+                                      _i64, _i32, _i32, _i32, _i32, _i32, _f32, _f32, _vp, _vp, _vp, _vp, _vp, _i32,
+                                      _i32, _vp, _sz, _i32, _vp, _vp]),
+    "b200_gated_recurrence_workspace_bytes": (_sz, [_i32, _i64, _i32, _i32, _i32, _i32]),
+    "b200_gated_recurrence": (_i32, [_vp, _vp, _vp, _i64, _vp, _vp, _vp, _f32, _vp, _i64, _vp, _vp, _vp, _vp, _i32,
+                                     _i64, _i32, _i32, _i32, _i32, _vp, _vp, _sz, _i32, _vp, _vp]),
     "b200_moe_combine": (_i32, [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i32, _i32, _i32, _vp]),
     "b200_selftest_bounded_wait": (_i32, [_i32, _vp, _vp, _vp]),
     "b200_lm_head_argmax_workspace_bytes": (_sz, [_i32, _i32]),
@@ -83,7 +96,10 @@ def load() -> C.CDLL:
             f"{LIB_PATH} is missing: build the CUDA library first "
             "(python -m llm_from_scratch_b200._build); there is no CPU fallback")
     lib = C.CDLL(str(LIB_PATH))
+    whole = LIB_PATH.name == "libb200llm.so"
     for name, (res, args) in SIGNATURES.items():
+        if not whole and not hasattr(lib, name):
+            continue      # another family's kernel: calling it raises AttributeError
         fn = getattr(lib, name)
         fn.restype = res
         fn.argtypes = args

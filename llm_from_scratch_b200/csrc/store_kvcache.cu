@@ -78,8 +78,65 @@ store_kvcache_scalar(const T* __restrict__ k, const T* __restrict__ v, int64_t k
   }
 }
 
+// Key and value rows of different widths (a pool whose heads have value size != key size): one launch, a unit
+// is one U of one row, the key row's units first.
+template <typename U>
+__global__ void __launch_bounds__(kThreads)
+store_kv_rows_kernel(const U* __restrict__ k, const U* __restrict__ v, int64_t k_stride, int64_t v_stride,
+                     U* __restrict__ kc, U* __restrict__ vc, const int64_t* __restrict__ slots, int64_t total, int ku,
+                     int vu, int64_t num_slots, int32_t* status) {
+  const int64_t step = static_cast<int64_t>(gridDim.x) * kThreads;
+  const int row = ku + vu;
+  for (int64_t i = static_cast<int64_t>(blockIdx.x) * kThreads + threadIdx.x; i < total; i += step) {
+    const int64_t t = i / row;
+    const int c = static_cast<int>(i - t * row);
+    const int64_t slot = __ldg(slots + t);
+    if (slot < 0) continue;
+    if (slot >= num_slots) {
+      report(status, B200_ERR_BOUNDS);
+      continue;
+    }
+    if (c < ku) kc[slot * ku + c] = k[t * k_stride + c];
+    else vc[slot * vu + c - ku] = v[t * v_stride + c - ku];
+  }
+}
+
 }  // namespace
 }  // namespace b200
+
+extern "C" int b200_store_kv_rows(const void* k, const void* v, int64_t k_token_stride, int64_t v_token_stride,
+                                  void* k_cache, void* v_cache, const int64_t* slot_mapping, int32_t num_tokens,
+                                  int32_t k_width, int32_t v_width, int64_t num_slots, int32_t dtype,
+                                  int32_t* status, void* stream) {
+  using namespace b200;
+  if (num_tokens < 0 || k_width <= 0 || v_width <= 0 || num_slots < 0) return B200_ERR_ARG;
+  if (dtype != B200_DTYPE_F32 && dtype != B200_DTYPE_BF16) return B200_ERR_UNSUPPORTED;
+  if (num_tokens == 0) return B200_OK;
+  if (!k || !v || !k_cache || !v_cache || !slot_mapping) return B200_ERR_ARG;
+  if (k_token_stride < k_width || v_token_stride < v_width) return B200_ERR_ARG;
+  const int sms = sm_count_cached();
+  if (sms <= 0) return B200_ERR_NO_DEVICE;
+  const int es = dtype == B200_DTYPE_F32 ? 4 : 2;
+  const bool vec = (int64_t(k_width) * es) % 16 == 0 && (int64_t(v_width) * es) % 16 == 0 &&
+                   (k_token_stride * es) % 16 == 0 && (v_token_stride * es) % 16 == 0 && aligned16(k) && aligned16(v) &&
+                   aligned16(k_cache) && aligned16(v_cache);
+  const int div = vec ? 16 / es : 1;
+  const int ku = k_width / div, vu = v_width / div;
+  const int64_t total = static_cast<int64_t>(num_tokens) * (ku + vu), cap = int64_t(sms) * kCtasPerSm;
+  const int64_t want = (total + kThreads - 1) / kThreads;
+  const unsigned grid = static_cast<unsigned>(want < cap ? want : cap);
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  auto go = [&](auto unit) {
+    using U = decltype(unit);
+    store_kv_rows_kernel<U><<<grid, kThreads, 0, s>>>(
+        static_cast<const U*>(k), static_cast<const U*>(v), k_token_stride / div, v_token_stride / div,
+        static_cast<U*>(k_cache), static_cast<U*>(v_cache), slot_mapping, total, ku, vu, num_slots, status);
+  };
+  if (vec) go(uint4{});
+  else if (es == 4) go(uint32_t{});
+  else go(uint16_t{});
+  return launch_result();
+}
 
 extern "C" int b200_store_kvcache(const void* k, const void* v, int64_t k_token_stride,
                                   int64_t v_token_stride, void* k_cache, void* v_cache,

@@ -255,13 +255,16 @@ class NativeBlockManager:
 
     reference_exact = False
 
-    def __init__(self, num_blocks: int, block_size: int):
+    def __init__(self, num_blocks: int, block_size: int, prefix_caching: bool = True):
+        """``prefix_caching=False``: blocks are never sealed with a hash and so never shared between sequences
+        (a model with recurrent state cannot resume behind somebody else's prefix)."""
         import ctypes
         import numpy as np
         from .._lib import lib
         self._np, self._ct, self._lib = np, ctypes, lib
         self.block_size = block_size
         self.num_blocks = num_blocks
+        self.prefix_caching = prefix_caching
         self._h = lib.b200_pool_create(num_blocks, block_size)
         if not self._h:
             raise MemoryError("could not create the native block pool")
@@ -317,6 +320,8 @@ class NativeBlockManager:
         return self.num_free_blocks >= seq.num_blocks
 
     def allocate(self, seq: Sequence) -> None:
+        if not self.prefix_caching:
+            return self.grow(seq, seq.num_tokens)
         np = self._np
         ids = np.asarray(seq.token_ids, dtype=np.int32)
         table = np.empty(seq.num_blocks, dtype=np.int32)
@@ -342,6 +347,8 @@ class NativeBlockManager:
         return (self._ct.c_int32 * self.block_size)(*token_ids)
 
     def append(self, seq: Sequence) -> None:
+        if not self.prefix_caching:
+            return self.grow(seq, seq.num_tokens)
         n = len(seq)
         rem = n % self.block_size
         if rem > 1:
@@ -354,6 +361,16 @@ class NativeBlockManager:
         elif b < -1:
             raise IndexError("KV block pool exhausted")
 
+    # ------------------------------------------------------------------ growth by any number of tokens
+    def blocks_to_grow(self, seq: Sequence, num_tokens: int) -> int:
+        """Blocks that ``grow`` would open."""
+        return max((num_tokens + self.block_size - 1) // self.block_size - len(seq.block_table), 0)
+
+    def grow(self, seq: Sequence, num_tokens: int) -> None:
+        """Opens blocks until the table of ``seq`` covers ``num_tokens`` tokens (a portion of a prompt)."""
+        for _ in range(self.blocks_to_grow(seq, num_tokens)):
+            self.open_block(seq)
+
     def open_block(self, seq: Sequence) -> None:
         b = self._lib.b200_pool_open_block(self._h)
         if b < 0:
@@ -361,6 +378,8 @@ class NativeBlockManager:
         seq.block_table.append(b)
 
     def seal_block(self, seq: Sequence, index: int) -> None:
+        if not self.prefix_caching:
+            return
         table, bs = seq.block_table, self.block_size
         toks = self._tokens(seq.token_ids[index * bs:(index + 1) * bs])
         if self._lib.b200_pool_seal_block(self._h, table[index], table[index - 1] if index > 0 else -1, toks) != 0:

@@ -12,7 +12,7 @@ import time
 
 from .model_runner import ModelRunner, _cfg
 from .sampling_params import SamplingParams
-from .scheduler import Scheduler
+from .scheduler import MixedScheduler, Scheduler
 from .sequence import Sequence
 
 
@@ -24,13 +24,17 @@ class LLMEngine:
         # ``runner`` lets a caller supply its own executor (anything with ``run(seqs, is_prefill)``,
         # ``num_kv_blocks`` and ``exit()``); by default the GPU model runner is built here
         self.model_runner = runner if runner is not None else ModelRunner(config, model)
-        self.scheduler = Scheduler(
+        limits = dict(
             max_num_sequences=_cfg(config, "max_num_sequences", "max_num_seqs", default=16),
             max_num_batched_tokens=_cfg(config, "max_num_batched_tokens", "max_num_batch_tokens", default=1024),
             max_cached_blocks=self.model_runner.num_kv_blocks,
             block_size=block_size,
             eos=_cfg(config, "eos", default=50256),
         )
+        if getattr(self.model_runner, "mixed_batches", False):
+            self.scheduler = MixedScheduler(**limits, num_state_slots=self.model_runner.num_state_slots)
+        else:
+            self.scheduler = Scheduler(**limits)
         # decode steps the engine may run per scheduling decision (1 = the reference's step-by-step loop);
         # larger values keep the GPU busy while the host schedules, at the price of admitting waiting
         # requests and retiring finished ones up to decode_window - 1 steps later
@@ -68,6 +72,7 @@ class LLMEngine:
         if not seqs:
             return [], 0, is_prefill
         runner = self.model_runner
+        processed = self.scheduler.step_tokens(seqs, is_prefill)
         window = 1
         if not is_prefill and self.decode_window > 1 and getattr(runner, "can_run_window", None) \
                 and runner.can_run_window(seqs):
@@ -88,7 +93,6 @@ class LLMEngine:
             self.timing[f"run_{kind}_s"] += t2 - t1
             self.timing[f"{kind}_steps"] += 1
             self.scheduler.postprocess(seqs, token_ids)
-            processed = sum(len(s) for s in seqs) if is_prefill else len(seqs)
         self.timing["postprocess_s"] += time.perf_counter() - t2
         if not is_prefill:
             self.timing["decode_seq_steps"] = getattr(runner, "decode_seq_steps", 0)

@@ -29,6 +29,7 @@ class StepMetadata:
     context_lens: Optional[np.ndarray] = None   # int64 [n]
     block_tables: Optional[np.ndarray] = None   # int32 [n, maxb]
     last_token_index: Optional[np.ndarray] = None  # int64 [n]  row of each sequence's last token
+    state_slots: Optional[np.ndarray] = None    # int64 [n]  recurrent-state slot of every sequence
 
 
 def block_table_array(s: Sequence) -> np.ndarray:
@@ -70,15 +71,20 @@ def _flat_tables(seqs: list[Sequence]):
     return offsets, np.ascontiguousarray(flat, dtype=np.int32)
 
 
-def prepare_prefill(seqs: list[Sequence], block_size: int) -> StepMetadata:
-    """Packs the non-cached suffix of every sequence (model_runner.py:202-249): cu_seqlens, positions and the slot
+def state_slot_array(seqs: list[Sequence]) -> np.ndarray:
+    return np.fromiter((s.state_slot for s in seqs), dtype=np.int64, count=len(seqs))
+
+
+def prepare_prefill(seqs: list[Sequence], block_size: int, tables_always: bool = False) -> StepMetadata:
+    """Packs the tokens every sequence computes this step — its non-cached suffix, up to ``step_end`` where the
+    scheduler set one (model_runner.py:202-249): cu_seqlens, positions and the slot
     mapping come from the library's native builder (``b200_prepare_prefill``); ``prepare_prefill_py`` is the
     same thing in numpy, kept as the definition and for the reference-exact mode."""
     if Sequence.reference_exact or any(not s.block_table for s in seqs):
         return prepare_prefill_py(seqs, block_size)
     from .._lib import lib
     n = len(seqs)
-    num_tokens = np.fromiter((s.num_tokens for s in seqs), dtype=np.int64, count=n)
+    num_tokens = np.fromiter((s.num_tokens if s.step_end is None else s.step_end for s in seqs), dtype=np.int64, count=n)
     cached = np.fromiter((s.num_cached_tokens for s in seqs), dtype=np.int64, count=n)
     offsets, flat = _flat_tables(seqs)
     total = int((num_tokens - cached).sum())
@@ -90,13 +96,13 @@ def prepare_prefill(seqs: list[Sequence], block_size: int) -> StepMetadata:
                                    slots.ctypes.data, total, mx.ctypes.data)
     if got != total:
         raise RuntimeError(f"prepare_prefill: the native builder returned {got} for {total} tokens")
-    ids = [np.asarray(s.token_ids[s.num_cached_tokens:], dtype=np.int64) for s in seqs]
+    ids = [np.asarray(s.token_ids[s.num_cached_tokens:s.step_end], dtype=np.int64) for s in seqs]
     return StepMetadata(
         is_prefill=True, input_ids=np.concatenate(ids) if ids else np.zeros(0, dtype=np.int64),
         slot_mapping=slots, positions=positions, cu_seqlens_q=cu_q, cu_seqlens_k=cu_k,
         max_seqlen_q=int(mx[0]), max_seqlen_k=int(mx[1]),
-        block_tables=pad_block_tables(seqs) if cu_q[-1] < cu_k[-1] else None,
-        last_token_index=(cu_q[1:] - 1).astype(np.int64))
+        block_tables=pad_block_tables(seqs) if tables_always or cu_q[-1] < cu_k[-1] else None,
+        last_token_index=(cu_q[1:] - 1).astype(np.int64), state_slots=state_slot_array(seqs))
 
 
 def prepare_prefill_py(seqs: list[Sequence], block_size: int) -> StepMetadata:
@@ -158,7 +164,7 @@ def prepare_decode(seqs: list[Sequence], block_size: int, tables_out: np.ndarray
     return StepMetadata(
         is_prefill=False, input_ids=np.fromiter((s.last_token for s in seqs), dtype=np.int64, count=n),
         slot_mapping=slots, positions=lens - 1, context_lens=lens, block_tables=tables,
-        last_token_index=np.arange(n, dtype=np.int64))
+        last_token_index=np.arange(n, dtype=np.int64), state_slots=state_slot_array(seqs))
 
 
 def prepare_decode_py(seqs: list[Sequence], block_size: int, tables_out: np.ndarray | None = None) -> StepMetadata:

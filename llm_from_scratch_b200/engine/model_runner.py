@@ -18,10 +18,11 @@ import numpy as np
 import torch
 
 from .. import ops
-from ..model import EngineTransformerLM, ModelConfig, init_reference_order
+from ..model import EngineTransformerLM, build_model, init_weights, resolve_config
 from ..utils.context import get_context, reset_context, set_context
 from ..utils.sampler import Sampler
 from . import metadata as md
+from .cache_pool import LayeredCache
 from .sequence import Sequence
 
 
@@ -82,19 +83,28 @@ class ModelRunner:
         dtype = _cfg(config, "dtype", default=torch.float32)
         self.dtype = getattr(torch, dtype) if isinstance(dtype, str) else dtype
         if model is None:
-            mc = config["model"]
-            mc = mc if isinstance(mc, ModelConfig) else ModelConfig.from_dict(mc)
-            weights = _cfg(config, "weights", "model_path", default=None)
+            mc, weights = config["model"], _cfg(config, "weights", "model_path", default=None)
+            if isinstance(mc, str) or hasattr(mc, "__fspath__"):
+                from ..utils.loader import load_model_dir   # a folder with config.json and weights
+                mc, stored = load_model_dir(str(mc))
+                weights = stored if weights is None else weights
+            mc = resolve_config(mc)                         # the family is the configuration's architecture
             if isinstance(weights, (str, bytes)) or hasattr(weights, "__fspath__"):
                 from ..utils.loader import load_weights     # a checkpoint in one of the reference's formats
                 weights = load_weights(str(weights))
             if weights is None:
-                weights = init_reference_order(mc, _cfg(config, "seed", default=0))
-            model = EngineTransformerLM(mc, weights, self.device, self.dtype)
+                weights = init_weights(mc, _cfg(config, "seed", default=0))
+            model = build_model(mc, weights, self.device, self.dtype)
         self.model = model
         self.model_config = model.cfg
-        if self.max_model_length is None:
-            self.max_model_length = self.model_config.context_length
+        # models with recurrent state hold a slot per live sequence; models with mixed batches take portions of
+        # prompts beside decoded tokens and read every key from the pool
+        self.recurrent_state, self.mixed_batches = model.recurrent_state, model.mixed_batches
+        self.num_state_slots = self.max_num_seqs if self.recurrent_state else 0
+        if self.mixed_batches:      # their matrix products accumulate in fp32 from end to end
+            torch.backends.cuda.matmul.allow_bf16_reduced_precision_reduction = False
+        if self.dtype == torch.float32:
+            torch.backends.cuda.matmul.allow_tf32 = False
         self.sampler = Sampler()
         self.staging = _Staging(self.device)
         self.graphs: dict[int, torch.cuda.CUDAGraph] = {}
@@ -105,14 +115,10 @@ class ModelRunner:
         # (what the decode kernels had to read), for throughput and memory-roofline reports
         self.decode_seq_steps = 0
         self.decode_ctx_tokens = 0
-        c = self.model_config
-        if c.attention_type == "MLA":    # prefill runs the expanded form: 192-wide keys, 128-wide values
-            self.prefill_tile_rows = ops.prefill_tile_rows(c.num_heads, c.num_heads, c.head_dim + c.rope_dim,
-                                                           c.head_dim, self.dtype)
-        else:
-            self.prefill_tile_rows = ops.prefill_tile_rows(c.num_heads, c.num_kv_heads, c.head_dim, c.head_dim,
-                                                           self.dtype)
+        self.prefill_tile_rows = model.prefill_tile_rows()
         self.allocate_kv_cache()
+        if self.max_model_length is None:
+            self.max_model_length = self.model_config.context_length or min(self.num_kv_blocks * self.block_size, 1 << 17)
         if not self.enforce_eager:
             self.capture_cudagraph()
             if self.prefill_tile_rows and _cfg(config, "prefill_graphs", default=True):
@@ -120,6 +126,8 @@ class ModelRunner:
 
     # ------------------------------------------------------------------ KV pool
     def kv_block_bytes(self) -> int:
+        if self.layered_cache is not None:
+            return self.layered_cache.block_bytes()
         c = self.model_config
         itemsize = torch.empty(0, dtype=self.dtype).element_size()
         if c.attention_type == "MLA":
@@ -129,15 +137,22 @@ class ModelRunner:
     def allocate_kv_cache(self) -> None:
         """One pool for all layers; per-layer views injected into the attention modules."""
         c = self.model_config
+        self.layered_cache = None
+        if hasattr(self.model, "cache_owners"):
+            self.layered_cache = LayeredCache(self.model, self.block_size, self.dtype, self.device)
         num_blocks = _cfg(self.config, "max_cached_blocks", "num_kv_blocks", default=None)
         if num_blocks is None:
             free, _total = torch.cuda.mem_get_info(self.device)
             util = _cfg(self.config, "gpu_memory_utilization", default=0.5)
+            if self.layered_cache is not None:
+                free -= self.num_state_slots * self.layered_cache.slot_bytes()
             num_blocks = int(free * util) // self.kv_block_bytes()
         if num_blocks < 1:
             raise RuntimeError("not enough device memory for a single KV block")
         self.num_kv_blocks = int(num_blocks)
-        if c.attention_type == "MLA":
+        if self.layered_cache is not None:
+            self.layered_cache.allocate(self.num_kv_blocks, self.num_state_slots)
+        elif c.attention_type == "MLA":
             self.kv_cache = torch.zeros(c.num_layers, num_blocks, self.block_size, c.kv_lora_rank + c.rope_dim,
                                         dtype=self.dtype, device=self.device)
             for i, att in enumerate(self.model.attention_layers):
@@ -155,7 +170,8 @@ class ModelRunner:
     # ------------------------------------------------------------------ metadata -> device
     def _publish(self, m: md.StepMetadata) -> torch.Tensor:
         arrays = {"input_ids": m.input_ids, "slot_mapping": m.slot_mapping, "positions": m.positions}
-        for name in ("cu_seqlens_q", "cu_seqlens_k", "context_lens", "block_tables"):
+        for name in ("cu_seqlens_q", "cu_seqlens_k", "context_lens", "block_tables") \
+                + (("state_slots",) if self.recurrent_state else ()):
             a = getattr(m, name)
             if a is not None:
                 arrays[name] = a
@@ -174,11 +190,12 @@ class ModelRunner:
             # one tile list per step, shared by the attention calls of all layers
             plan = ops.prefill_plan(t["cu_seqlens_q"], len(arrays["input_ids"]), m.max_seqlen_q, self.prefill_tile_rows)
         set_context(m.is_prefill, t.get("cu_seqlens_q"), t.get("cu_seqlens_k"), m.max_seqlen_q, m.max_seqlen_k,
-                    t["slot_mapping"], t.get("context_lens"), t.get("block_tables"), t["positions"], plan)
+                    t["slot_mapping"], t.get("context_lens"), t.get("block_tables"), t["positions"], plan,
+                    t.get("state_slots"))
         return t["input_ids"]
 
     def prepare_prefill(self, seqs: list[Sequence]) -> torch.Tensor:
-        return self._publish(md.prepare_prefill(seqs, self.block_size))
+        return self._publish(md.prepare_prefill(seqs, self.block_size, tables_always=self.mixed_batches))
 
     def prepare_decode(self, seqs: list[Sequence]) -> torch.Tensor:
         return self._publish(md.prepare_decode(seqs, self.block_size))
@@ -204,26 +221,35 @@ class ModelRunner:
         v["context_lens"][:bucket].zero_()
         v["context_lens"][:bs].copy_(ctx.context_lens)
         v["block_tables"][:bs, :ctx.block_tables.size(1)].copy_(ctx.block_tables)
+        if ctx.state_slots is not None:
+            v["state_slots"][:bucket].fill_(-1)
+            v["state_slots"][:bs].copy_(ctx.state_slots)
         self.graphs[bucket].replay()
         return self.model.compute_logits(v["outputs"][:bs])
 
+    def _uses_decode_graph(self, seqs: list[Sequence], is_prefill: bool) -> bool:
+        return not is_prefill and bool(self.graphs) and not self.enforce_eager and len(seqs) <= max(self.graphs)
+
+    @torch.inference_mode()
+    def _hidden(self, seqs: list[Sequence], is_prefill: bool) -> torch.Tensor:
+        """Final hidden states of a scheduled batch (the context is left set for the head)."""
+        if self._uses_decode_graph(seqs, is_prefill):
+            return self._replay_decode(seqs)
+        if is_prefill and self.prefill_graphs and (hidden := self._replay_prefill(seqs)) is not None:
+            self.decode_builder.invalidate(seqs)
+            return hidden
+        if is_prefill and self.decode_builder is not None:
+            self.decode_builder.invalidate(seqs)
+        return self.model(self.prepare_prefill(seqs) if is_prefill else self.prepare_decode(seqs))
+
     def run(self, seqs: list[Sequence], is_prefill: bool) -> list[int]:
         greedy = not any(s.temperature for s in seqs)
-        if not is_prefill and self.graphs and not self.enforce_eager and len(seqs) <= max(self.graphs):
-            hidden = self._replay_decode(seqs)
-            if greedy:
-                # the fused head (projection + argmax) was part of the graph; reading it is the step's only sync
-                token_ids = self.graph_vars["greedy"][:len(seqs)].tolist()
-                reset_context()
-                return token_ids
-        elif is_prefill and self.prefill_graphs and (hidden := self._replay_prefill(seqs)) is not None:
-            self.decode_builder.invalidate(seqs)
-        else:
-            if is_prefill and self.decode_builder is not None:
-                self.decode_builder.invalidate(seqs)
-            input_ids = self.prepare_prefill(seqs) if is_prefill else self.prepare_decode(seqs)
-            with torch.inference_mode():
-                hidden = self.model(input_ids)
+        hidden = self._hidden(seqs, is_prefill)
+        if greedy and self._uses_decode_graph(seqs, is_prefill):
+            # the fused head (projection + argmax) was part of the graph; reading it is the step's only sync
+            token_ids = self.graph_vars["greedy"][:len(seqs)].tolist()
+            reset_context()
+            return token_ids
         with torch.inference_mode():
             if greedy:
                 token_ids = self.model.greedy_tokens(hidden).tolist()
@@ -247,6 +273,9 @@ class ModelRunner:
                                             h["block_tables"], patches=h["patches"])
         h["slot_mapping"][n:bucket] = -1
         h["context_lens"][n:bucket] = 0
+        if self.recurrent_state:
+            h["state_slots"][:n] = md.state_slot_array(seqs)
+            h["state_slots"][n:bucket] = -1
         self.decode_seq_steps += n
         self.decode_ctx_tokens += int(h["context_lens"][:n].sum())
         if patched >= 0:
@@ -298,6 +327,21 @@ class ModelRunner:
         """Like ``run`` but returns the last-token logits [num_seqs, vocab] (used by parity tests)."""
         input_ids = self.prepare_prefill(seqs) if is_prefill else self.prepare_decode(seqs)
         logits = self.run_model(input_ids, is_prefill).float().clone()
+        reset_context()
+        return logits
+
+    @torch.inference_mode()
+    def run_wanted(self, seqs: list[Sequence], is_prefill: bool, want: list[list[int]]) -> torch.Tensor:
+        """The step ``run`` would execute, but instead of sampling: fp32 logits [total wanted, vocab] at the
+        places ``want[i]`` among the tokens sequence i computes in this step."""
+        lens = [(s.num_tokens if s.step_end is None else s.step_end) - s.num_cached_tokens for s in seqs] if is_prefill \
+            else [1] * len(seqs)
+        starts = np.concatenate([[0], np.cumsum(lens)])
+        rows = [int(starts[i]) + w for i, places in enumerate(want) for w in places]
+        hidden = self._hidden(seqs, is_prefill)
+        get_context().logit_rows = torch.tensor(rows, dtype=torch.int64, device=self.device)
+        logits = self.model.compute_logits(hidden).float() if rows else \
+            torch.empty(0, self.model_config.vocab_size, device=self.device)
         reset_context()
         return logits
 
@@ -398,6 +442,7 @@ class ModelRunner:
         # step copies only the prefix its batch bucket uses)
         fields = (("input_ids", np.int64, torch.int64, (max_bs,)), ("slot_mapping", np.int64, torch.int64, (max_bs,)),
                   ("context_lens", np.int64, torch.int64, (max_bs,)),
+                  ("state_slots", np.int64, torch.int64, (max_bs,)),
                   ("patches", np.int32, torch.int32, (8 * max_bs, 3)),
                   ("block_tables", np.int32, torch.int32, (max_bs, max_blocks)))
         offsets, total = {}, 0
@@ -414,8 +459,9 @@ class ModelRunner:
             nbytes = int(np.prod(shape)) * np.dtype(npdt).itemsize
             v[name] = self.graph_dev[offsets[name]:offsets[name] + nbytes].view(tdt).view(*shape)
             self.graph_host_np[name] = host_bytes[offsets[name]:offsets[name] + nbytes].view(npdt).reshape(shape)
-        v["slot_mapping"].fill_(-1)
-        self.graph_host_np["slot_mapping"][:] = -1
+        for name in ("slot_mapping", "state_slots"):
+            v[name].fill_(-1)
+            self.graph_host_np[name][:] = -1
         self.decode_builder = md.DecodeBatchBuilder(self.block_size, max_blocks, rows=4 * max_bs, device_rows=max_bs)
         v["outputs"] = torch.zeros(max_bs, self.model_config.d_model, dtype=self.dtype, device=dev)
         # the graph also holds the greedy head (lm_head projection fused with the argmax), so a greedy step
@@ -429,7 +475,7 @@ class ModelRunner:
         for b in reversed(buckets):
             # a padded row decodes position 0 of an empty context: its output row is never read
             set_context(False, slot_mapping=v["slot_mapping"][:b], context_lens=v["context_lens"][:b],
-                        block_tables=v["block_tables"][:b])
+                        block_tables=v["block_tables"][:b], state_slots=v["state_slots"][:b])
             positions = (v["context_lens"][:b] - 1).clamp_min(0)
             v["outputs"][:b] = self.model(v["input_ids"][:b], positions)       # warm-up, allocates workspaces
             self.model.greedy_tokens(v["outputs"][:b], out=v["greedy"][:b])

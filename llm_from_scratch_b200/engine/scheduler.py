@@ -33,6 +33,7 @@ class Scheduler:
             self.block_manager = BlockManager(max_cached_blocks, block_size, reference_exact)
         else:
             self.block_manager = NativeBlockManager(max_cached_blocks, block_size)
+        self.state_slots = None       # StateSlots of a model with recurrent state (MixedScheduler)
         self.waiting: deque[Sequence] = deque()
         self.running: deque[Sequence] = deque()
 
@@ -188,6 +189,10 @@ class Scheduler:
         seq.status = SequenceStatus.WAITING
         self.waiting.appendleft(seq)
 
+    def step_tokens(self, seqs: list[Sequence], is_prefill: bool) -> int:
+        """Tokens a scheduled step is counted with (a prefill: its sequences once they hold the sampled token)."""
+        return sum(len(s) + 1 for s in seqs) if is_prefill else len(seqs)
+
     # ------------------------------------------------------------------ after the model ran
     def postprocess(self, seqs: list[Sequence], token_ids: list[int]) -> None:
         eos = self.eos
@@ -203,3 +208,167 @@ class Scheduler:
                 seq.status = SequenceStatus.FINISHED
                 self.block_manager.deallocate(seq)
                 self.running.remove(seq)
+
+
+class StateSlots:
+    """Slots of the recurrent-state pool: one per live sequence, first in first out like the KV blocks."""
+
+    def __init__(self, num_slots: int):
+        self.num_slots = num_slots
+        self.free: deque[int] = deque(range(num_slots))
+
+    def take(self, seq: Sequence) -> None:
+        if seq.state_slot < 0:
+            if not self.free:
+                raise IndexError("recurrent-state slots exhausted")
+            seq.state_slot = self.free.popleft()
+
+    def give_back(self, seq: Sequence) -> None:
+        if seq.state_slot >= 0:
+            self.free.append(seq.state_slot)
+            seq.state_slot = -1
+
+
+class MixedScheduler(Scheduler):
+    """Continuous batching for models that take portions of prompts beside decoded tokens in one step.
+
+    A step serves the running sequences first, oldest first, then admits waiting ones, until the token budget is
+    spent; a prompt that does not fit is cut and continues on the next step.  ``seq.num_cached_tokens`` counts the
+    tokens whose keys (and state) exist, ``seq.step_end`` what it will be after the scheduled step.  Blocks are
+    opened as a sequence grows and never shared (no prefix caching); a model with recurrent state also holds one
+    slot of ``state_slots`` per live sequence.  When the pool runs dry the newest running sequence is preempted
+    and recomputed later.
+
+    ``schedule()`` returns ``(sequences, is_prefill)``: sequences with a single token first, and ``is_prefill``
+    False when every sequence just decodes its last token."""
+
+    def __init__(self, max_num_sequences: int, max_num_batched_tokens: int, max_cached_blocks: int, block_size: int,
+                 eos: int, num_state_slots: int = 0):
+        super().__init__(max_num_sequences, max_num_batched_tokens, max_cached_blocks, block_size, eos)
+        self.block_manager = NativeBlockManager(max_cached_blocks, block_size, prefix_caching=False)
+        self.state_slots = StateSlots(num_state_slots) if num_state_slots else None
+
+    # ------------------------------------------------------------------ what a sequence holds
+    def _admit(self, seq: Sequence) -> None:
+        if self.state_slots is not None:
+            self.state_slots.take(seq)
+        seq.status = SequenceStatus.RUNNING
+        self.running.append(seq)
+
+    def _release(self, seq: Sequence) -> None:
+        self.block_manager.deallocate(seq)
+        seq.step_end = None
+        if self.state_slots is not None:
+            self.state_slots.give_back(seq)
+
+    def preempt(self, seq: Sequence) -> None:
+        self._release(seq)
+        seq.status = SequenceStatus.WAITING
+        self.waiting.appendleft(seq)
+
+    # ------------------------------------------------------------------ one step
+    def schedule(self) -> tuple[list[Sequence], bool]:
+        bm, batch, budget, dry = self.block_manager, [], self.max_num_batched_tokens, False
+        for seq in list(self.running):
+            if budget <= 0 or len(batch) >= self.max_num_sequences:
+                break
+            if seq.status is not SequenceStatus.RUNNING:       # preempted earlier in this loop
+                continue
+            end = seq.num_cached_tokens + min(seq.num_tokens - seq.num_cached_tokens, budget)
+            while bm.blocks_to_grow(seq, end) > bm.num_free_blocks:
+                victim, dry = self.running.pop(), True         # newest; it comes later in this loop or is seq
+                self.preempt(victim)
+                if victim is seq:
+                    break
+            if seq.status is not SequenceStatus.RUNNING:
+                break
+            bm.grow(seq, end)
+            seq.step_end = end
+            budget -= end - seq.num_cached_tokens
+            batch.append(seq)
+        while self.waiting and not dry and budget > 0 and len(batch) < self.max_num_sequences \
+                and len(self.running) < self.max_num_sequences:
+            seq = self.waiting[0]
+            if self.state_slots is not None and not self.state_slots.free:
+                break
+            # room for the whole prompt, also when only a portion of it runs now; a sequence that was preempted
+            # in the middle of its output also needs its next token's place
+            if bm.blocks_to_grow(seq, seq.num_tokens + (seq.num_completion_tokens > 0)) > bm.num_free_blocks:
+                break
+            end = min(seq.num_tokens, budget)
+            self.waiting.popleft()
+            self._admit(seq)
+            bm.grow(seq, end)
+            seq.step_end = end
+            budget -= end
+            batch.append(seq)
+        return self._order(batch)
+
+    @staticmethod
+    def _order(batch: list[Sequence]) -> tuple[list[Sequence], bool]:
+        batch.sort(key=lambda s: s.step_end - s.num_cached_tokens != 1)
+        decode = all(s.step_end - s.num_cached_tokens == 1 and s.step_end == s.num_tokens for s in batch)
+        return batch, not decode
+
+    def step_tokens(self, seqs: list[Sequence], is_prefill: bool) -> int:
+        return sum(s.step_end - s.num_cached_tokens for s in seqs)
+
+    def plan_decode_window(self, seqs, max_steps, max_positions) -> int:
+        # every running sequence must be in the window's batch, or one that is not would fall behind by the window
+        if len(seqs) < len(self.running):
+            return 1
+        return super().plan_decode_window(seqs, max_steps, max_positions)
+
+    # ------------------------------------------------------------------ after the model ran
+    def postprocess(self, seqs: list[Sequence], token_ids: list[int]) -> None:
+        """Sequences whose step reached their last token take the sampled token; the others (a prompt still being
+        read in portions) only advance."""
+        done_s, done_t = [], []
+        for seq, token_id in zip(seqs, token_ids):
+            seq.num_cached_tokens, end = seq.step_end, seq.step_end
+            seq.step_end = None
+            if end == seq.num_tokens:
+                done_s.append(seq)
+                done_t.append(token_id)
+        super().postprocess(done_s, done_t)
+        self._retire(done_s)
+
+    def postprocess_window(self, seqs: list[Sequence], steps: list[list[int]]) -> int:
+        kept = super().postprocess_window(seqs, steps)
+        for seq in seqs:
+            seq.step_end = None
+            if not seq.is_finished:
+                seq.num_cached_tokens = seq.num_tokens - 1
+        self._retire(seqs)
+        return kept
+
+    def _retire(self, seqs: list[Sequence]) -> None:
+        if self.state_slots is not None:
+            for seq in seqs:
+                if seq.is_finished:
+                    self.state_slots.give_back(seq)
+
+    # ------------------------------------------------------------------ tokens supplied from outside
+    def feed(self, batch: list[tuple[Sequence, list[int]]]) -> tuple[list[Sequence], bool]:
+        """Schedules exactly the given tokens as one step: every sequence (new or running) gets its tokens appended
+        and all of them computed.  The caller ends a sequence with ``drop``."""
+        for seq, tokens in batch:
+            if seq.status is not SequenceStatus.RUNNING:
+                self._admit(seq)
+            seq.token_ids.extend(tokens)
+            seq.num_tokens = seq.step_end = len(seq.token_ids)
+            seq.last_token = seq.token_ids[-1]
+            self.block_manager.grow(seq, seq.num_tokens)
+        return self._order([seq for seq, _ in batch])
+
+    def fed(self, seqs: list[Sequence]) -> None:
+        """The fed step has run."""
+        for seq in seqs:
+            seq.num_cached_tokens = seq.step_end
+            seq.step_end = None
+
+    def drop(self, seq: Sequence) -> None:
+        """Ends a fed sequence and gives back what it holds."""
+        seq.status = SequenceStatus.FINISHED
+        self._release(seq)
+        self.running.remove(seq)

@@ -32,7 +32,7 @@ class Sequence:
 
     __slots__ = ("seq_id", "status", "token_ids", "last_token", "num_tokens", "num_prompt_tokens",
                  "num_cached_tokens", "block_table", "temperature", "max_tokens", "ignore_eos",
-                 "max_model_length", "_bt_cache", "_row")
+                 "max_model_length", "state_slot", "step_end", "_bt_cache", "_row")
 
     def __init__(self, token_ids, sampling_params: SamplingParams | None = None):
         sp = sampling_params if sampling_params is not None else SamplingParams()
@@ -43,6 +43,8 @@ class Sequence:
         self.num_tokens = self.num_prompt_tokens = len(self.token_ids)
         self.num_cached_tokens = 0
         self.block_table: list[int] = []
+        self.state_slot = -1      # slot of the recurrent state (models that have one), -1 = none held
+        self.step_end = None      # mixed scheduling: tokens computed once the scheduled step has run; None = all
         self._bt_cache = None     # [list object, int32 buffer, entries valid]: see metadata.block_table_array
         self._row = None          # row of this sequence in a metadata.DecodeBatchBuilder table
         self.temperature = sp.temperature
@@ -109,6 +111,7 @@ class Sequence:
 
     def __setstate__(self, state):
         self.num_tokens, self.num_prompt_tokens, self.num_cached_tokens, self.block_table, payload = state
+        self.state_slot, self.step_end = -1, None
         self._bt_cache = None
         self._row = None
         self.token_ids = payload if self.num_tokens == self.num_prompt_tokens else [payload]

@@ -431,7 +431,44 @@ class DecoderLayer(nn.Module):
         return self.ffn(h), residual
 
 
-class EngineTransformerLM(nn.Module):
+class TokenHead:
+    """Language-model head shared by the engine's models: logits and greedy tokens of a step's hidden states.
+    The model supplies ``w_head`` [vocab, d], ``b_head`` (or None) and ``dtype``."""
+
+    @staticmethod
+    def logit_rows(hidden: torch.Tensor) -> torch.Tensor:
+        """The rows of a step's hidden states whose logits are read: the rows the context names, or the last row
+        of every sequence."""
+        ctx = get_context()
+        if ctx.logit_rows is not None:
+            return hidden[ctx.logit_rows]
+        if ctx.is_prefill:
+            return hidden[ctx.cu_seqlens_q[1:].long() - 1]
+        return hidden
+
+    def compute_logits(self, hidden: torch.Tensor) -> torch.Tensor:
+        return F.linear(self.logit_rows(hidden).to(self.dtype), self.w_head, self.b_head)
+
+    fused_head_max_rows = 64     # rows up to which the fused head (weights as the MMA M side) beats GEMM + argmax
+
+    def greedy_tokens(self, hidden: torch.Tensor, out: torch.Tensor | None = None) -> torch.Tensor:
+        """argmax of ``compute_logits(hidden)`` per sequence (first maximum), int64 [num_seqs].  In bf16, up to 64
+        rows, the head projection and the argmax are one fused pass over the head matrix
+        (``ops.lm_head_argmax``: the logits are never written; 20-22 us against 24-27 us on B200).  Larger batches
+        take the library GEMM followed by the argmax kernel of ``ops.sample`` (the fused kernel keeps the tokens
+        on the narrow side of the MMA and takes 41 us at 256 rows against 27 us)."""
+        hidden = self.logit_rows(hidden).to(self.dtype)
+        if hidden.shape[0] <= self.fused_head_max_rows and ops.lm_head_argmax_supported(hidden, self.w_head):
+            return ops.lm_head_argmax(hidden.contiguous(), self.w_head, self.b_head, out)
+        logits = F.linear(hidden, self.w_head, self.b_head)
+        if logits.is_cuda and logits.dtype in (torch.float32, torch.bfloat16) and logits.shape[0] > 0:
+            return ops.sample(logits, None, 0, 0, out=out)   # no temperatures: greedy rows, first maximum
+        if out is None:
+            return torch.argmax(logits, dim=-1)
+        return torch.argmax(logits, dim=-1, out=out)
+
+
+class EngineTransformerLM(TokenHead, nn.Module):
     """``model(input_ids)`` -> hidden states [T, d]; ``compute_logits(hidden)`` -> [num_seqs, vocab]."""
 
     def __init__(self, cfg: ModelConfig, weights: dict, device, dtype=torch.float32):
@@ -444,9 +481,19 @@ class EngineTransformerLM(nn.Module):
         self.final_norm = p.f32("final_norm.weight")
         self.w_head, self.b_head = p.lin("lm_head")
 
+    recurrent_state = False
+    mixed_batches = False
+
     @property
     def attention_layers(self):
         return [layer.att for layer in self.layers]
+
+    def prefill_tile_rows(self) -> int:
+        """Query rows per tile of the prefill kernel that serves this model (0: no tile list)."""
+        c = self.cfg
+        if c.attention_type == "MLA":    # prefill runs the expanded form: 192-wide keys, 128-wide values
+            return ops.prefill_tile_rows(c.num_heads, c.num_heads, c.head_dim + c.rope_dim, c.head_dim, self.dtype)
+        return ops.prefill_tile_rows(c.num_heads, c.num_kv_heads, c.head_dim, c.head_dim, self.dtype)
 
     def forward(self, input_ids: torch.Tensor, positions: torch.Tensor | None = None) -> torch.Tensor:
         ctx = get_context()
@@ -465,30 +512,3 @@ class EngineTransformerLM(nn.Module):
             x, residual = layer(x, residual, ctx, positions, attn_out)
         h, _ = rms_norm(x, self.final_norm, self.cfg.rms_eps, residual)
         return h
-
-    def compute_logits(self, hidden: torch.Tensor) -> torch.Tensor:
-        ctx = get_context()
-        if ctx.is_prefill:
-            hidden = hidden[ctx.cu_seqlens_q[1:].long() - 1]
-        return F.linear(hidden.to(self.dtype), self.w_head, self.b_head)
-
-    fused_head_max_rows = 64     # rows up to which the fused head (weights as the MMA M side) beats GEMM + argmax
-
-    def greedy_tokens(self, hidden: torch.Tensor, out: torch.Tensor | None = None) -> torch.Tensor:
-        """argmax of ``compute_logits(hidden)`` per sequence (first maximum), int64 [num_seqs].  In bf16, up to 64
-        rows, the head projection and the argmax are one fused pass over the head matrix
-        (``ops.lm_head_argmax``: the logits are never written; 20-22 us against 24-27 us on B200).  Larger batches
-        take the library GEMM followed by the argmax kernel of ``ops.sample`` (the fused kernel keeps the tokens
-        on the narrow side of the MMA and takes 41 us at 256 rows against 27 us)."""
-        ctx = get_context()
-        if ctx.is_prefill:
-            hidden = hidden[ctx.cu_seqlens_q[1:].long() - 1]
-        hidden = hidden.to(self.dtype)
-        if hidden.shape[0] <= self.fused_head_max_rows and ops.lm_head_argmax_supported(hidden, self.w_head):
-            return ops.lm_head_argmax(hidden.contiguous(), self.w_head, self.b_head, out)
-        logits = F.linear(hidden, self.w_head, self.b_head)
-        if logits.is_cuda and logits.dtype in (torch.float32, torch.bfloat16) and logits.shape[0] > 0:
-            return ops.sample(logits, None, 0, 0, out=out)   # no temperatures: greedy rows, first maximum
-        if out is None:
-            return torch.argmax(logits, dim=-1)
-        return torch.argmax(logits, dim=-1, out=out)

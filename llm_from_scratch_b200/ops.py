@@ -716,3 +716,183 @@ def sample(logits: torch.Tensor, temperatures: torch.Tensor | None, seed: int, o
                           else None, B, V, seed & 0xFFFFFFFFFFFFFFFF, offset & 0xFFFFFFFFFFFFFFFF, out.data_ptr(),
                           _dt(logits), _stream()), "sample")
     return out
+
+
+# ------------------------------------------------------------------------------------------------
+# residual streams, talking-heads attention, gated recurrence
+# ------------------------------------------------------------------------------------------------
+def _ptr(t: torch.Tensor | None):
+    return t.data_ptr() if t is not None else None
+
+
+def _f32vec(name: str, t: torch.Tensor | None, n: int) -> None:
+    if t is not None and (t.dtype != torch.float32 or t.numel() != n or not t.is_contiguous()):
+        raise ValueError(f"{name} must be a contiguous fp32 tensor of {n} elements")
+
+
+def store_kv_rows(k: torch.Tensor, v: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
+                  slot_mapping: torch.Tensor) -> None:
+    """``store_kvcache`` for pools whose key and value rows differ in width: k [T, Wk], v [T, Wv] (row stride
+    free) into caches [num_blocks, block_size, heads, dim] with heads * dim == W; slots < 0 are skipped."""
+    dev = _cuda(k, v, k_cache, v_cache, slot_mapping)
+    T, wk = k.shape
+    wv = v.shape[1]
+    if v.shape[0] != T or k.stride(1) != 1 or v.stride(1) != 1:
+        raise ValueError("k and v must be [T, width] with contiguous rows")
+    if slot_mapping.dtype != torch.int64 or slot_mapping.numel() != T or not slot_mapping.is_contiguous():
+        raise ValueError("slot_mapping must be a contiguous int64 tensor with one entry per token")
+    slots = k_cache.shape[0] * k_cache.shape[1]
+    if k_cache.numel() != slots * wk or v_cache.numel() != slots * wv or not k_cache.is_contiguous() \
+            or not v_cache.is_contiguous() or any(t.dtype != k.dtype for t in (v, k_cache, v_cache)):
+        raise ValueError("caches must be contiguous, of k's dtype, with the same slots and rows as wide as k / v")
+    check(lib.b200_store_kv_rows(k.data_ptr(), v.data_ptr(), k.stride(0), v.stride(0), k_cache.data_ptr(),
+                                 v_cache.data_ptr(), slot_mapping.data_ptr(), T, wk, wv, slots, _dt(k),
+                                 status_word(dev).data_ptr(), _stream()), "store_kv_rows")
+
+
+def stream_update(x: torch.Tensor, norm_w: torch.Tensor, eps: float, dtype: torch.dtype, *,
+                  tokens: torch.Tensor | None = None, embed: torch.Tensor | None = None,
+                  y: torch.Tensor | None = None, y1: torch.Tensor | None = None,
+                  join_w: tuple[torch.Tensor, torch.Tensor] | None = None, join_eps: float = 0.0,
+                  layer_scale: torch.Tensor | None = None, mix: torch.Tensor | None = None,
+                  out_w: torch.Tensor | None = None, in_w: torch.Tensor | None = None, plus_one: bool = True):
+    """One sublayer boundary of a decoder with fp32 residual streams x [T, S, d], in place
+    (``b200_stream_update``): write the sublayer result ``y`` (or the join of ``y`` and ``y1``) back into the
+    streams, read the next sublayer's input from them and return its norm [T, d] in ``dtype``.  With
+    ``embed`` / ``tokens`` the streams start from the embedding rows instead of an update."""
+    dev = _cuda(x, norm_w, tokens, embed, y, y1, layer_scale, mix, out_w, in_w)
+    T, S, d = x.shape
+    if x.dtype != torch.float32 or not x.is_contiguous():
+        raise ValueError("x must be a contiguous fp32 [T, streams, d] tensor")
+    for name, t, n in (("norm_w", norm_w, d), ("layer_scale", layer_scale, d), ("mix", mix, S * S), ("out_w", out_w, S),
+                       ("in_w", in_w, S)) + ((("join_w", join_w[0], d), ("join_w", join_w[1], d)) if join_w else ()):
+        _f32vec(name, t, n)
+    for t in (y, y1):
+        if t is not None and (t.shape != (T, d) or t.dtype != dtype or not t.is_contiguous()):
+            raise ValueError("y must be contiguous [T, d] in the activation dtype")
+    if embed is not None and (embed.shape[1] != d or embed.dtype != dtype or not embed.is_contiguous()
+                              or tokens is None or tokens.dtype != torch.int64 or tokens.numel() != T):
+        raise ValueError("embed must be contiguous [vocab, d] in the activation dtype, tokens int64 [T]")
+    h = torch.empty(T, d, dtype=dtype, device=x.device)
+    check(lib.b200_stream_update(
+        x.data_ptr(), _ptr(tokens) if embed is not None else None, _ptr(embed), embed.shape[0] if embed is not None else 0,
+        _ptr(y), _ptr(y1), _ptr(join_w[0]) if join_w else None, _ptr(join_w[1]) if join_w else None, float(join_eps),
+        _ptr(layer_scale), _ptr(mix), _ptr(out_w), _ptr(in_w), norm_w.data_ptr(), 1 if plus_one else 0, float(eps),
+        h.data_ptr(), T, S, d, _dt(h), status_word(dev).data_ptr(), _stream()), "stream_update")
+    return h
+
+
+def clamped_glu(h: torch.Tensor, limit: float, slope: float) -> torch.Tensor:
+    """g sigmoid(slope g) (u + 1) for h = [gate | up] [rows, 2F], g = min(gate, limit), u = clamp(up, +-limit)."""
+    _cuda(h)
+    rows, F2 = h.shape
+    if not h.is_contiguous() or F2 % 2:
+        raise ValueError("h must be contiguous [rows, 2*d_ff]")
+    act = torch.empty(rows, F2 // 2, dtype=h.dtype, device=h.device)
+    check(lib.b200_clamped_glu(h.data_ptr(), act.data_ptr(), rows, F2 // 2, float(limit), float(slope), _dt(h),
+                               _stream()), "clamped_glu")
+    return act
+
+
+class TalkingHeads:
+    """Constants of a talking-heads attention layer on the device: the score scale and cap, the distance bias
+    (r1, r2 [H]), the head mix ``talk`` [H, H] (out, in) and the window (0: none).  The bias of every distance
+    inside the window is tabulated once."""
+
+    max_table = 1 << 16
+
+    def __init__(self, scale: float, softcap: float, r1: torch.Tensor, r2: torch.Tensor, talk: torch.Tensor, window: int,
+                 device):
+        H = talk.shape[0]
+        self.scale, self.softcap, self.window, self.H = float(scale), float(softcap), int(window), H
+        host = talk.detach().float().cpu().contiguous()
+        self.talk_host = host
+        self.talk = host.to(device)
+        self.r1 = r1.detach().float().to(device).contiguous()
+        self.r2 = r2.detach().float().to(device).contiguous()
+        for name, t, n in (("r1", self.r1, H), ("r2", self.r2, H), ("talk", self.talk, H * H)):
+            _f32vec(name, t, n)
+        self.table = None
+        if 0 < self.window <= self.max_table:
+            dist = torch.arange(self.window, dtype=torch.float64)[:, None]
+            t = r1.detach().double().cpu() * torch.log1p(r2.detach().double().cpu() * dist)
+            self.table = t.float().to(device).contiguous()       # [window, H]
+
+
+def talking_attention(q: torch.Tensor, gate: torch.Tensor | None, k_cache: torch.Tensor, v_cache: torch.Tensor,
+                      block_tables: torch.Tensor, c: TalkingHeads, *, cu_seqlens_q: torch.Tensor | None = None,
+                      cu_seqlens_k: torch.Tensor | None = None, context_lens: torch.Tensor | None = None,
+                      max_seqlen_q: int = 1, out: torch.Tensor | None = None, general: bool = False) -> torch.Tensor:
+    """Attention of ``b200_talking_attention`` over the paged pool: q [rows, H * dk], gate [rows, H * dv] (row
+    strides free), caches [num_blocks, block_size, Hkv, d*].  Rows are ragged (``cu_seqlens_*``) or one per sequence
+    (``context_lens``).  ``general`` forces the general kernel.  Returns [rows, H, dv]."""
+    dev = _cuda(q, gate, k_cache, v_cache, block_tables, cu_seqlens_q, cu_seqlens_k, context_lens, out)
+    rows, H = q.shape[0], c.H
+    nb, bs, Hkv, dk = k_cache.shape
+    dv = v_cache.shape[3]
+    if v_cache.shape[:3] != (nb, bs, Hkv) or not k_cache.is_contiguous() or not v_cache.is_contiguous() \
+            or k_cache.dtype != q.dtype or v_cache.dtype != q.dtype:
+        raise ValueError("caches must be contiguous [num_blocks, block_size, Hkv, d] of q's dtype")
+    if q.shape[1] != H * dk or q.stride(1) != 1 or (gate is not None and (gate.shape != (rows, H * dv)
+                                                    or gate.stride(1) != 1 or gate.dtype != q.dtype)):
+        raise ValueError("q must be [rows, H * dk] and gate [rows, H * dv] with contiguous rows")
+    if cu_seqlens_q is not None:
+        n = cu_seqlens_q.numel() - 1
+        if cu_seqlens_q.dtype != torch.int32 or cu_seqlens_k is None or cu_seqlens_k.dtype != torch.int32 \
+                or cu_seqlens_k.numel() != n + 1:
+            raise ValueError("cu_seqlens must be int32 tensors of the same length")
+    else:
+        n = rows
+        if context_lens is None or context_lens.dtype != torch.int64 or context_lens.numel() < rows:
+            raise ValueError("context_lens must be int64 with one entry per row")
+    if block_tables.dtype != torch.int32 or block_tables.shape[0] < n or block_tables.stride(1) != 1:
+        raise ValueError("block_tables must be int32 [num_seqs, max_blocks]")
+    if out is None:
+        out = torch.empty(rows, H, dv, dtype=q.dtype, device=q.device)
+    elif out.shape != (rows, H, dv) or out.dtype != q.dtype or not out.is_contiguous():
+        raise ValueError("out must be a contiguous [rows, H, dv] tensor")
+    need = int(lib.b200_talking_attention_workspace_bytes(n, H, dv, c.window, 0 if cu_seqlens_q is not None else 1, _dt(q)))
+    ws = workspace(dev, need, "talking") if need else None
+    check(lib.b200_talking_attention(
+        q.data_ptr(), q.stride(0), _ptr(gate), gate.stride(0) if gate is not None else 0, k_cache.data_ptr(),
+        v_cache.data_ptr(), out.data_ptr(), block_tables.data_ptr(), block_tables.stride(0), bs, nb, _ptr(cu_seqlens_q),
+        _ptr(cu_seqlens_k), _ptr(context_lens), n, rows, int(max_seqlen_q), H, Hkv, dk, dv, c.scale, c.softcap,
+        c.r1.data_ptr(), c.r2.data_ptr(), c.talk.data_ptr(), None if general else c.talk_host.data_ptr(), _ptr(c.table),
+        c.table.shape[0] if c.table is not None else 0, c.window, _ptr(ws), ws.numel() if ws is not None else 0, _dt(q),
+        status_word(dev).data_ptr(), _stream()), "talking_attention")
+    return out
+
+
+def gated_recurrence(q: torch.Tensor, f: torch.Tensor, v: torch.Tensor, f_bias: torch.Tensor, lower: torch.Tensor,
+                     norm_w: torch.Tensor, eps: float, state: torch.Tensor, state_slots: torch.Tensor, *,
+                     cu_seqlens_q: torch.Tensor | None = None, cu_seqlens_k: torch.Tensor | None = None,
+                     context_lens: torch.Tensor | None = None, max_seqlen_q: int = 1) -> torch.Tensor:
+    """Gated linear recurrence of ``b200_gated_recurrence``: q, f [T, heads * dk], v [T, heads * dv] (views of one
+    projection), state fp32 [slots, heads, dk, dv] updated in place.  Returns the normed heads [T, heads * dv]."""
+    dev = _cuda(q, f, v, f_bias, lower, norm_w, state, state_slots, cu_seqlens_q, cu_seqlens_k, context_lens)
+    slots, H, dk, dv = state.shape
+    T = q.shape[0]
+    if q.shape != (T, H * dk) or f.shape != (T, H * dk) or v.shape != (T, H * dv) or any(
+            t.stride(1) != 1 or t.stride(0) != q.stride(0) or t.dtype != q.dtype for t in (q, f, v)):
+        raise ValueError("q, f [T, H * dk] and v [T, H * dv] must share dtype and row stride")
+    if state.dtype != torch.float32 or not state.is_contiguous():
+        raise ValueError("state must be contiguous fp32 [slots, H, dk, dv]")
+    for name, t, n in (("f_bias", f_bias, H * dk), ("lower", lower, H * dk), ("norm_w", norm_w, dv)):
+        _f32vec(name, t, n)
+    n = cu_seqlens_q.numel() - 1 if cu_seqlens_q is not None else T
+    if state_slots.dtype != torch.int64 or state_slots.numel() < n or not state_slots.is_contiguous():
+        raise ValueError("state_slots must be contiguous int64 with one entry per sequence")
+    if cu_seqlens_q is not None:
+        if cu_seqlens_q.dtype != torch.int32 or cu_seqlens_k is None or cu_seqlens_k.dtype != torch.int32:
+            raise ValueError("cu_seqlens must be int32")
+    elif context_lens is None or context_lens.dtype != torch.int64 or context_lens.numel() < n:
+        raise ValueError("context_lens must be int64 with one entry per row")
+    out = torch.empty(T, H * dv, dtype=q.dtype, device=q.device)
+    need = int(lib.b200_gated_recurrence_workspace_bytes(n, T, int(max_seqlen_q), H, dk, dv))
+    ws = workspace(dev, need, "recurrence") if need else None
+    check(lib.b200_gated_recurrence(
+        q.data_ptr(), f.data_ptr(), v.data_ptr(), q.stride(0), f_bias.data_ptr(), lower.data_ptr(), norm_w.data_ptr(),
+        float(eps), state.data_ptr(), slots, state_slots.data_ptr(), _ptr(cu_seqlens_q), _ptr(cu_seqlens_k),
+        _ptr(context_lens), n, T, int(max_seqlen_q), H, dk, dv, out.data_ptr(), _ptr(ws),
+        ws.numel() if ws is not None else 0, _dt(q), status_word(dev).data_ptr(), _stream()), "gated_recurrence")
+    return out

@@ -24,6 +24,8 @@ class Context:
     # not in the reference (its runner builds no positions although the model needs them for RoPE):
     positions: Optional[torch.Tensor] = None      # int64 [num_tokens]; None in decode = context_lens - 1
     prefill_plan: object = None                   # ops.PrefillPlan of this step's cu_seqlens_q, or None
+    state_slots: Optional[torch.Tensor] = None    # int64 [num_seqs] slot of every sequence's recurrent state, -1 = none
+    logit_rows: Optional[torch.Tensor] = None     # int64 rows whose logits are wanted; None = each sequence's last
 
 
 _current = Context()
@@ -35,10 +37,11 @@ def get_context() -> Context:
 
 def set_context(is_prefill, cu_seqlens_q=None, cu_seqlens_k=None, max_seqlen_q=0, max_seqlen_k=0,
                 slot_mapping=None, context_lens=None, block_tables=None, positions=None,
-                prefill_plan=None) -> None:
+                prefill_plan=None, state_slots=None, logit_rows=None) -> None:
     global _current
     _current = Context(is_prefill, cu_seqlens_q, cu_seqlens_k, max_seqlen_q, max_seqlen_k,
-                       slot_mapping, context_lens, block_tables, positions, prefill_plan)
+                       slot_mapping, context_lens, block_tables, positions, prefill_plan,
+                       state_slots, logit_rows)
 
 
 def reset_context() -> None:

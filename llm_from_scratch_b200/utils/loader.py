@@ -14,6 +14,7 @@ loaders return that dict.  Accepted inputs, with the reference's resolution rule
 """
 from __future__ import annotations
 
+import json
 import os
 from glob import glob
 
@@ -102,3 +103,10 @@ def check_names(state: dict, expected: dict, strict: bool = True) -> tuple[list[
     if strict and missing:
         raise KeyError(f"checkpoint lacks {len(missing)} parameters, first: {missing[0]}")
     return missing, unexpected
+
+
+def load_model_dir(path: str) -> tuple[dict, dict]:
+    """(configuration dict, weights) of a folder with ``config.json`` and ``*.safetensors`` / ``.pt`` weights."""
+    with open(os.path.join(path, "config.json")) as f:
+        config = json.load(f)
+    return config, load_weights(path)
