@@ -511,9 +511,9 @@ int b200_clamped_glu(const void* h, void* act, int64_t rows, int32_t d_ff, float
  * pool already holds, the new rows included) is cu_seqlens_k[s+1]-cu_seqlens_k[s] long; with cu_seqlens_q ==
  * NULL row i is the last token of sequence i and context_lens[i] its length (0: padding row, nothing written).
  * Rows beyond the last sequence are padding.  max_seqlen_q: host bound on rows per sequence.
- * r1, r2 [num_heads] and talk [num_heads, num_heads] fp32 (device); bias_table [bias_len, num_heads] fp32 or
- * NULL: r1 ln(1 + r2 distance) for distances 0 .. bias_len - 1; talk_host: the same matrix on the host (may be
- * NULL: general kernel).  Workspace: b200_talking_attention_workspace_bytes(). */
+ * r1, r2 [num_heads] and talk [num_heads, num_heads] fp32 (device); bias_table [num_heads, bias_len] fp32
+ * or NULL: r1 ln(1 + r2 distance) for distances 0 .. bias_len - 1, bias_len >= window if given; consts_host: talk,
+ * r1, r2 one after the other on the host (NULL: the general kernel runs).  Workspace: b200_talking_attention_workspace_bytes(). */
 size_t b200_talking_attention_workspace_bytes(int32_t num_seqs, int32_t num_heads, int32_t dim_v, int32_t window,
                                               int32_t decode, int32_t dtype);
 int b200_talking_attention(const void* q, int64_t q_stride, const void* gate, int64_t gate_stride, const void* k_cache,
@@ -522,7 +522,7 @@ int b200_talking_attention(const void* q, int64_t q_stride, const void* gate, in
                            const int32_t* cu_seqlens_k, const int64_t* context_lens, int32_t num_seqs, int64_t rows,
                            int32_t max_seqlen_q, int32_t num_heads, int32_t num_kv_heads, int32_t dim_k, int32_t dim_v,
                            float scale, float softcap, const float* r1, const float* r2, const float* talk,
-                           const float* talk_host, const float* bias_table, int32_t bias_len, int32_t window,
+                           const float* consts_host, const float* bias_table, int32_t bias_len, int32_t window,
                            void* workspace, size_t workspace_bytes, int32_t dtype, int32_t* status, void* stream);
 
 /* Gated linear recurrence (HGRN2) over per-sequence states: per head

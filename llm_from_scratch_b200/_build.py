@@ -47,7 +47,7 @@ def _stale(target: Path, deps: list[Path]) -> bool:
 # when the full one is absent.  "api" and "host_path" are the parts every engine uses.
 FAMILY_SOURCES = {
     "Nabalix": ("api", "host_path", "decode_advance", "sampler", "moe_gemm", "moe_gemm_rows", "store_kvcache", "streams",
-                "talking_attention", "gated_recurrence"),
+                "talking_attention", "talking_attention_mma", "talking_decode_mma", "gated_recurrence"),
 }
 
 

@@ -8,7 +8,17 @@
 // the call is at position 0 starts from zero whatever its slot holds, so slots need no clearing when they
 // change hands.
 //
-// recurrence_step_kernel   one CTA per (sequence, head), tokens in order: decode, and short portions.
+// recurrence_step_kernel   one CTA per (sequence, head), tokens in order: decode, and sizes the scan does not take.
+//
+// recurrence_scan_kernel   prompts and portions, cut into segments of seg_len tokens that run in parallel.  A segment
+//                          maps its entry state to D * S + P (D: product of its forget gates, P: its own writes), so
+//   pass 1 (scan, LOCAL)   P and D of every segment but the last of its sequence, from the zero state
+//   pass 2 (chain)         the entry state of every segment, segment after segment
+//   pass 3 (scan)          the outputs from the entry states; the last segment leaves the state in the pool
+//                          A sequence of one segment needs pass 3 only.  A thread keeps R key channels x C value
+//                          columns of the state in registers and walks the tokens; q / f / k / v of 16 tokens at a
+//                          time sit in shared memory as fp32, the 16 threads of a column reduce their part of o by
+//                          shuffles, and 16 tokens of outputs are normed together.
 #include "common.cuh"
 
 namespace b200 {
@@ -172,12 +182,319 @@ int launch_step(const RecArgs& a, int n, bool vec, cudaStream_t s) {
   return launch_result();
 }
 
+// ---------------------------------------------------------------------------------------------
+// Segmented scan
+// ---------------------------------------------------------------------------------------------
+constexpr int kRowGroups = 16;       // threads that share a column group
+constexpr int kBlockTokens = 16;     // tokens staged at a time
+
+struct ScanArgs {
+  float* seg_state;          // [segments, H, dk, dv]  pass 1: P, after pass 2: entry state
+  float* seg_decay;          // [segments, H, dk]      pass 1: D
+  int n, seg_len;
+};
+
+using f32x2 = unsigned long long;
+__device__ __forceinline__ f32x2 pack2(float lo, float hi) {
+  f32x2 r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
+  return r;
+}
+__device__ __forceinline__ float2 unpack2(f32x2 v) {
+  float2 r;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+  return r;
+}
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
+  f32x2 r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
+  f32x2 r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+
+// segment number -> (sequence, index within it, first segment number of the sequence); every thread calls it
+__device__ __forceinline__ bool find_segment(const RecArgs& a, const ScanArgs& c, int number, int* seq, int* index) {
+  __shared__ int found[2];
+  if (threadIdx.x < 32) {
+    const int lane = threadIdx.x;
+    int left = number, hit_seq = -1, hit_idx = 0;
+    for (int base = 0; base < c.n && hit_seq < 0; base += 32) {
+      const int s = base + lane;
+      const int t = s < c.n ? (a.cu_q[s + 1] - a.cu_q[s] + c.seg_len - 1) / c.seg_len : 0;
+      int incl = t;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const int y = __shfl_up_sync(0xffffffffu, incl, o);
+        if (lane >= o) incl += y;
+      }
+      const unsigned hit = __ballot_sync(0xffffffffu, left < incl);
+      if (hit) {
+        const int src = __ffs(hit) - 1;
+        hit_seq = base + src;
+        hit_idx = left - __shfl_sync(0xffffffffu, incl - t, src);
+      } else {
+        left -= __shfl_sync(0xffffffffu, incl, 31);
+      }
+    }
+    if (lane == 0) {
+      found[0] = hit_seq;
+      found[1] = hit_idx;
+    }
+  }
+  __syncthreads();
+  *seq = found[0];
+  *index = found[1];
+  return found[0] >= 0;
+}
+
+template <typename T, int R, int C, bool LOCAL>
+__global__ void __launch_bounds__(512, 1) recurrence_scan_kernel(const RecArgs a, const ScanArgs sc) {
+  constexpr int DK = R * kRowGroups, P = R / 2;
+  extern __shared__ __align__(16) float sm[];
+  const int dk = a.dk, dv = a.dv, head = blockIdx.y, number = blockIdx.x;
+  int seq, index;
+  if (!find_segment(a, sc, number, &seq, &index)) return;
+  SeqInfo info;
+  if (!sequence_info(a, seq, &info)) return;
+  const int segments = (info.len + sc.seg_len - 1) / sc.seg_len;
+  const bool last = index == segments - 1;
+  if (LOCAL && last) return;                       // its own map is never needed
+  const int tok_lo = index * sc.seg_len, ntok = min(sc.seg_len, info.len - tok_lo);
+
+  float* sf = sm;                                  // [kBlockTokens, DK]
+  float* sk = sf + kBlockTokens * DK;
+  float* sq = sk + kBlockTokens * DK;              // outputs only
+  float* sv = sq + (LOCAL ? 0 : kBlockTokens * DK);
+  float* so = sv + kBlockTokens * dv;              // [kBlockTokens, dv], outputs only
+  const int tid = threadIdx.x, threads = blockDim.x, rg = tid & (kRowGroups - 1), c0 = (tid / kRowGroups) * C;
+  const bool cols = c0 < dv;                       // dv is a multiple of 4: a float4 is in or out as a whole
+
+  // pair p of this thread: rows row(p), row(p) + 1
+  auto row = [&](int p) { return (p >> 1) * 64 + rg * 4 + (p & 1) * 2; };
+  f32x2 S[P][C], D[P];
+  const int64_t head_state = static_cast<int64_t>(dk) * dv;
+  float* pool = a.state + (info.slot * a.H + head) * head_state;
+  float* mine = sc.seg_state + (static_cast<int64_t>(number) * a.H + head) * head_state;
+  const float* from = LOCAL ? nullptr : segments > 1 ? mine : info.fresh ? nullptr : pool;
+#pragma unroll
+  for (int p = 0; p < P; ++p) {
+    D[p] = pack2(1.f, 1.f);
+#pragma unroll
+    for (int c = 0; c < C; c += 4) {
+      float4 x0 = make_float4(0.f, 0.f, 0.f, 0.f), x1 = x0;
+      if (from != nullptr && c0 + c < dv) {
+        if (row(p) < dk) x0 = *reinterpret_cast<const float4*>(from + static_cast<int64_t>(row(p)) * dv + c0 + c);
+        if (row(p) + 1 < dk) x1 = *reinterpret_cast<const float4*>(from + static_cast<int64_t>(row(p) + 1) * dv + c0 + c);
+      }
+      S[p][c] = pack2(x0.x, x1.x);
+      S[p][c + 1] = pack2(x0.y, x1.y);
+      S[p][c + 2] = pack2(x0.z, x1.z);
+      S[p][c + 3] = pack2(x0.w, x1.w);
+    }
+  }
+
+  for (int b = 0; b < ntok; b += kBlockTokens) {
+    const int nb = min(kBlockTokens, ntok - b);
+    const int64_t tok = info.tok0 + tok_lo + b;
+    __syncthreads();
+    for (int i = tid; i < nb * DK; i += threads) {
+      const int t = i / DK, d = i % DK;
+      float f = 1.f, k = 0.f, q = 0.f;
+      if (d < dk) {
+        const int64_t off = (tok + t) * a.stride + head * dk + d;
+        gates(to_float<T>(static_cast<const T*>(a.f)[off]) + a.f_bias[head * dk + d], a.lower[head * dk + d], &f, &k);
+        if (!LOCAL) {
+          q = to_float<T>(static_cast<const T*>(a.q)[off]);
+          q *= sigmoid_f(q);
+        }
+      }
+      sf[i] = f;
+      sk[i] = k;
+      if (!LOCAL) sq[i] = q;
+    }
+    for (int i = tid; i < nb * dv; i += threads) {
+      const int t = i / dv, d = i - t * dv;
+      sv[i] = to_float<T>(static_cast<const T*>(a.v)[(tok + t) * a.stride + head * dv + d]);
+    }
+    __syncthreads();
+    for (int t = 0; t < nb; ++t) {
+      f32x2 f[P], k[P], q[P], v[C];
+#pragma unroll
+      for (int i = 0; i < P; i += 2) {
+        const int at = t * DK + (i >> 1) * 64 + rg * 4;
+        const ulonglong2 fx = *reinterpret_cast<const ulonglong2*>(sf + at), kx = *reinterpret_cast<const ulonglong2*>(sk + at);
+        f[i] = fx.x, f[i + 1] = fx.y, k[i] = kx.x, k[i + 1] = kx.y;
+        if (!LOCAL) {
+          const ulonglong2 qx = *reinterpret_cast<const ulonglong2*>(sq + at);
+          q[i] = qx.x, q[i + 1] = qx.y;
+        }
+      }
+#pragma unroll
+      for (int c = 0; c < C; c += 4) {
+        const float4 x = c0 + c < dv ? *reinterpret_cast<const float4*>(sv + t * dv + c0 + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        v[c] = pack2(x.x, x.x);
+        v[c + 1] = pack2(x.y, x.y);
+        v[c + 2] = pack2(x.z, x.z);
+        v[c + 3] = pack2(x.w, x.w);
+      }
+      float o[C];
+#pragma unroll
+      for (int c = 0; c < C; ++c) {
+        f32x2 acc = 0;
+#pragma unroll
+        for (int p = 0; p < P; ++p) {
+          S[p][c] = fma2(f[p], S[p][c], mul2(k[p], v[c]));
+          if (!LOCAL) acc = fma2(q[p], S[p][c], acc);
+        }
+        const float2 h = unpack2(acc);
+        o[c] = h.x + h.y;
+      }
+      if constexpr (LOCAL) {
+#pragma unroll
+        for (int p = 0; p < P; ++p) D[p] = mul2(D[p], f[p]);
+      } else {
+        // sum over the 16 row groups; every step a lane keeps half of the columns it still has
+        int col = 0;
+#pragma unroll
+        for (int half = C / 2, step = 8; half >= 1; half >>= 1, step >>= 1) {
+          const bool up = rg & step;
+#pragma unroll
+          for (int c = 0; c < half; ++c) {
+            const float send = up ? o[c] : o[c + half], keep = up ? o[c + half] : o[c];
+            o[c] = keep + __shfl_xor_sync(0xffffffffu, send, step);
+          }
+          if (up) col += half;
+        }
+        constexpr int kLeft = kRowGroups / C;        // lanes that still share one column
+#pragma unroll
+        for (int step = kLeft / 2; step >= 1; step >>= 1) o[0] += __shfl_xor_sync(0xffffffffu, o[0], step);
+        if (cols && (rg & (kLeft - 1)) == 0) so[t * dv + c0 + col] = o[0];
+      }
+    }
+    if constexpr (!LOCAL) {
+      __syncthreads();
+      const int lane = tid & 31;
+      for (int t = tid >> 5; t < nb; t += threads >> 5) {
+        float ss = 0.f;
+        for (int d = lane; d < dv; d += 32) ss += so[t * dv + d] * so[t * dv + d];
+        const float inv = rsqrtf(warp_sum(ss) / static_cast<float>(dv) + a.eps);
+        T* op = static_cast<T*>(a.out) + ((tok + t) * a.H + head) * dv;
+        for (int d = lane; d < dv; d += 32) op[d] = from_float<T>(so[t * dv + d] * inv * a.norm_w[d]);
+      }
+    }
+  }
+  if (LOCAL && tid < kRowGroups) {
+    float* dec = sc.seg_decay + (static_cast<int64_t>(number) * a.H + head) * dk;
+#pragma unroll
+    for (int p = 0; p < P; ++p) {
+      const float2 x = unpack2(D[p]);
+      if (row(p) < dk) dec[row(p)] = x.x;
+      if (row(p) + 1 < dk) dec[row(p) + 1] = x.y;
+    }
+  }
+  float* to = LOCAL ? mine : last ? pool : nullptr;
+  if (to != nullptr) {
+#pragma unroll
+    for (int p = 0; p < P; ++p)
+#pragma unroll
+      for (int c = 0; c < C; c += 4) {
+        if (c0 + c >= dv) continue;
+        const float2 x0 = unpack2(S[p][c]), x1 = unpack2(S[p][c + 1]), x2 = unpack2(S[p][c + 2]), x3 = unpack2(S[p][c + 3]);
+        float* at = to + static_cast<int64_t>(row(p)) * dv + c0 + c;
+        if (row(p) < dk) *reinterpret_cast<float4*>(at) = make_float4(x0.x, x1.x, x2.x, x3.x);
+        if (row(p) + 1 < dk) *reinterpret_cast<float4*>(at + dv) = make_float4(x0.y, x1.y, x2.y, x3.y);
+      }
+  }
+}
+
+// Entry states: one thread carries four consecutive state elements of one (sequence, head) through its segments.
+__global__ void __launch_bounds__(256) recurrence_chain_kernel(const RecArgs a, const ScanArgs sc) {
+  __shared__ int s_first;
+  const int seq = blockIdx.z, head = blockIdx.y;
+  SeqInfo info;
+  if (!sequence_info(a, seq, &info)) return;
+  const int segments = (info.len + sc.seg_len - 1) / sc.seg_len;
+  if (segments <= 1) return;
+  if (threadIdx.x < 32) {                            // number of the sequence's first segment
+    int sum = 0;
+    for (int s = threadIdx.x; s < seq; s += 32) sum += (a.cu_q[s + 1] - a.cu_q[s] + sc.seg_len - 1) / sc.seg_len;
+    for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+    if (threadIdx.x == 0) s_first = sum;
+  }
+  __syncthreads();
+  const int64_t per_head = static_cast<int64_t>(a.dk) * a.dv;
+  const int64_t e = (static_cast<int64_t>(blockIdx.x) * blockDim.x + threadIdx.x) * 4;
+  if (e >= per_head) return;
+  const int r = static_cast<int>(e / a.dv);
+  float4 S = info.fresh ? make_float4(0.f, 0.f, 0.f, 0.f)
+                        : *reinterpret_cast<const float4*>(a.state + (info.slot * a.H + head) * per_head + e);
+  float* st = sc.seg_state + (static_cast<int64_t>(s_first) * a.H + head) * per_head + e;
+  const float* dec = sc.seg_decay + (static_cast<int64_t>(s_first) * a.H + head) * a.dk + r;
+#pragma unroll 4
+  for (int i = 0; i < segments - 1; ++i, st += a.H * per_head, dec += static_cast<int64_t>(a.H) * a.dk) {
+    const float4 p = *reinterpret_cast<const float4*>(st);
+    const float d = *dec;
+    *reinterpret_cast<float4*>(st) = S;
+    S.x = fmaf(d, S.x, p.x);
+    S.y = fmaf(d, S.y, p.y);
+    S.z = fmaf(d, S.z, p.z);
+    S.w = fmaf(d, S.w, p.w);
+  }
+  *reinterpret_cast<float4*>(st) = S;
+}
+
+// sizes the scan takes: columns of all threads of a CTA, rows in registers
+inline bool scan_shape(int dk, int dv) { return dv % 4 == 0 && ((dk <= 128 && dv <= 256) || (dk <= 256 && dv <= 128)); }
+
+inline int scan_seg_len(int64_t tokens, int H) {
+  // long enough to amortise the passes over the states, short enough for two waves of CTAs
+  const int64_t want = tokens * H / 600;
+  return want >= 128 ? 128 : want >= 64 ? 64 : 32;
+}
+
+template <typename T, int R, int C>
+int launch_scan(const RecArgs& a, const ScanArgs& sc, int64_t segments, bool chained, cudaStream_t s) {
+  const int groups = (a.dv + C - 1) / C, threads = (groups * kRowGroups + 31) / 32 * 32;
+  auto local = recurrence_scan_kernel<T, R, C, true>;
+  auto full = recurrence_scan_kernel<T, R, C, false>;
+  const size_t one = size_t(kBlockTokens) * R * kRowGroups * sizeof(float), v = size_t(kBlockTokens) * a.dv * sizeof(float);
+  const size_t smem_local = 2 * one + 2 * v, smem_full = 3 * one + 2 * v;
+  if (smem_full > 48 * 1024 &&
+      (cudaFuncSetAttribute(local, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem_local)) != cudaSuccess ||
+       cudaFuncSetAttribute(full, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem_full)) != cudaSuccess))
+    return B200_ERR_LAUNCH;
+  const dim3 grid(static_cast<unsigned>(segments), a.H);
+  if (chained) {
+    local<<<grid, threads, smem_local, s>>>(a, sc);
+    const int64_t units = static_cast<int64_t>(a.dk) * a.dv / 4;
+    recurrence_chain_kernel<<<dim3(static_cast<unsigned>((units + 255) / 256), a.H, sc.n), 256, 0, s>>>(a, sc);
+  }
+  full<<<grid, threads, smem_full, s>>>(a, sc);
+  return launch_result();
+}
+
+template <typename T>
+int dispatch_scan(const RecArgs& a, const ScanArgs& sc, int64_t segments, bool chained, cudaStream_t s) {
+  if (a.dk <= 64) return launch_scan<T, 4, 8>(a, sc, segments, chained, s);
+  if (a.dk <= 128) return launch_scan<T, 8, 8>(a, sc, segments, chained, s);
+  return launch_scan<T, 16, 4>(a, sc, segments, chained, s);
+}
+
 }  // namespace
 }  // namespace b200
 
 extern "C" size_t b200_gated_recurrence_workspace_bytes(int32_t num_seqs, int64_t total_tokens, int32_t max_seqlen_q,
                                                         int32_t num_heads, int32_t dim_k, int32_t dim_v) {
-  return 0;
+  using namespace b200;
+  if (num_seqs <= 0 || total_tokens <= 0 || max_seqlen_q <= 1 || num_heads <= 0 || !scan_shape(dim_k, dim_v)) return 0;
+  const int seg = scan_seg_len(total_tokens, num_heads);
+  if (max_seqlen_q <= seg) return 0;                      // every sequence is one segment
+  const size_t segments = static_cast<size_t>(total_tokens / seg + num_seqs);
+  return segments * num_heads * (static_cast<size_t>(dim_k) * dim_v + dim_k) * sizeof(float);
 }
 
 extern "C" int b200_gated_recurrence(const void* q, const void* f, const void* v, int64_t token_stride,
@@ -199,6 +516,22 @@ extern "C" int b200_gated_recurrence(const void* q, const void* f, const void* v
             cu_seqlens_k, context_lens, out, num_heads, dim_k, dim_v, status};
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   const bool vec = dim_v % 4 == 0 && aligned16(state);
+  if (cu_seqlens_q && vec && max_seqlen_q > 1 && scan_shape(dim_k, dim_v)) {
+    ScanArgs sc{};
+    sc.n = num_seqs;
+    sc.seg_len = scan_seg_len(total_tokens, num_heads);
+    const int64_t segments = total_tokens / sc.seg_len + num_seqs;
+    const bool chained = max_seqlen_q > sc.seg_len;
+    if (chained) {
+      if (!workspace || workspace_bytes < b200_gated_recurrence_workspace_bytes(num_seqs, total_tokens, max_seqlen_q,
+                                                                               num_heads, dim_k, dim_v))
+        return B200_ERR_WORKSPACE;
+      sc.seg_state = static_cast<float*>(workspace);
+      sc.seg_decay = sc.seg_state + static_cast<size_t>(segments) * num_heads * dim_k * dim_v;
+    }
+    return dtype == B200_DTYPE_F32 ? dispatch_scan<float>(a, sc, segments, chained, s)
+                                   : dispatch_scan<__nv_bfloat16>(a, sc, segments, chained, s);
+  }
   return dtype == B200_DTYPE_F32 ? launch_step<float>(a, num_seqs, vec, s)
                                  : launch_step<__nv_bfloat16>(a, num_seqs, vec, s);
 }

@@ -150,7 +150,9 @@ int launch_simple(const TalkArgs& a, cudaStream_t s) {
 
 extern "C" size_t b200_talking_attention_workspace_bytes(int32_t num_seqs, int32_t num_heads, int32_t dim_v,
                                                          int32_t window, int32_t decode, int32_t dtype) {
-  return 0;
+  using namespace b200;
+  if (!decode || dtype != B200_DTYPE_BF16 || num_seqs <= 0 || num_heads <= 0 || dim_v <= 0) return 0;
+  return talking_decode_workspace_bytes(num_seqs, num_heads, dim_v, window);
 }
 
 extern "C" int b200_talking_attention(const void* q, int64_t q_stride, const void* gate, int64_t gate_stride,
@@ -160,7 +162,7 @@ extern "C" int b200_talking_attention(const void* q, int64_t q_stride, const voi
                                       const int64_t* context_lens, int32_t num_seqs, int64_t rows, int32_t max_seqlen_q,
                                       int32_t num_heads, int32_t num_kv_heads, int32_t dim_k, int32_t dim_v,
                                       float scale, float softcap, const float* r1, const float* r2, const float* talk,
-                                      const float* talk_host, const float* bias_table, int32_t bias_len,
+                                      const float* consts_host, const float* bias_table, int32_t bias_len,
                                       int32_t window, void* workspace, size_t workspace_bytes, int32_t dtype,
                                       int32_t* status, void* stream) {
   using namespace b200;
@@ -200,12 +202,16 @@ extern "C" int b200_talking_attention(const void* q, int64_t q_stride, const voi
   a.talk = talk;
   a.window = window;
   a.max_q = max_seqlen_q;
-  a.talk_host = talk_host;
+  a.talk_host = consts_host;
+  a.r1_host = consts_host ? consts_host + static_cast<size_t>(num_heads) * num_heads : nullptr;
+  a.r2_host = consts_host ? a.r1_host + num_heads : nullptr;
   a.bias_table = bias_table;
   a.bias_len = bias_table ? bias_len : 0;
   a.workspace = workspace;
   a.workspace_bytes = workspace_bytes;
   a.status = status;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  return dtype == B200_DTYPE_F32 ? launch_simple<float>(a, s) : launch_simple<__nv_bfloat16>(a, s);
+  if (dtype == B200_DTYPE_F32) return launch_simple<float>(a, s);
+  const int rc = a.cu_q ? talking_prefill_mma_launch(a, s) : talking_decode_mma_launch(a, s);
+  return rc != B200_ERR_UNSUPPORTED ? rc : launch_simple<__nv_bfloat16>(a, s);
 }

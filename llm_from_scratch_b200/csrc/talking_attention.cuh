@@ -30,11 +30,18 @@ struct TalkArgs {
   int window;                // <= 0: none
   int max_q;                 // bound on rows per sequence
   const float* talk_host;    // talk on the host, or null
-  const float* bias_table;   // [bias_len, H] r1 ln(1 + r2 distance), or null
+  const float* r1_host;      // r1, r2 on the host with talk_host
+  const float* r2_host;
+  const float* bias_table;   // [H, bias_len] r1 ln(1 + r2 distance), or null
   int bias_len;
   void* workspace;
   size_t workspace_bytes;
   int32_t* status;
 };
+
+// bf16 tensor-core paths; B200_ERR_UNSUPPORTED = sizes or alignments they do not take
+int talking_prefill_mma_launch(const TalkArgs& a, cudaStream_t s);
+int talking_decode_mma_launch(const TalkArgs& a, cudaStream_t s);
+size_t talking_decode_workspace_bytes(int n, int H, int dv, int window);
 
 }  // namespace b200

@@ -1,0 +1,423 @@
+// Talking-heads attention, bf16 tensor-core path for ragged prompts and portions (mathematics: talking_attention.cu).
+//
+// The head mix couples all heads of a (query, key) pair, so one CTA owns 16 query rows of one sequence with ALL
+// heads and walks the visible keys in tiles of 32:
+//
+//   QK   warp w holds heads w*HPW ..: S = Q K^T on mma.sync m16n8k16, fp32 scores to shared memory
+//   mix  warp w owns query rows w and w + 8, lane = key: soft cap, distance bias, the H x H mix with the matrix
+//        as constant-bank operands (it is a kernel parameter), mask, exp2 -> bf16 weights, which overwrite the
+//        scores of the same row
+//   PV   warp w again holds its heads: O += P V, fp32 accumulators in registers; row sums from the same fragments
+//
+// The three phases are separated by CTA barriers; K of the next tile arrives (cp.async) during mix and PV, V during
+// QK and mix.  Scores are fp32 from the accumulator to the exponential.  The running maximum is lazy: a row keeps
+// the reference maximum of an earlier tile until a score exceeds it by 2^kSlack, so the ordinary tile needs no
+// reduction over lanes; the exact maximum only has to keep the exponentials in range.
+#include <string.h>
+
+#include "talking_attention.cuh"
+
+namespace b200 {
+namespace {
+
+constexpr int BQ = 16;
+constexpr int BK = 32;
+constexpr int kWarps = 8;
+constexpr int kThreads = kWarps * 32;
+constexpr int kSRow = 40;            // floats per score row: 32 keys + padding against bank conflicts
+constexpr float kSlack = 30.f;       // log2 of how far a score may exceed the row's reference
+
+constexpr float kLog2e = 1.4426950408889634f;
+
+template <int HP>
+struct MixParam {
+  float t[HP * HP];                  // talk * log2(e), [out][in], zero-padded
+  float r1[HP], r2[HP];
+};
+
+__device__ __forceinline__ float rcp_approx(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+// cap tanh(x scale / cap) - bias; k = 2 log2(e) scale / cap
+__device__ __forceinline__ float capped(float x, float k, float cap, float two_cap, float bias) {
+  return (cap - bias) - two_cap * rcp_approx(1.f + fast_exp2(x * k));
+}
+
+template <int HP, int MAXC, int MINB>
+__global__ void __launch_bounds__(kThreads, MINB)
+talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp) {
+  constexpr int HPW = HP / kWarps;
+  extern __shared__ __align__(128) uint8_t smem[];
+  __shared__ float s_ref[HP * BQ];     // reference maximum (log2 domain) per (head, row)
+  __shared__ float s_cor[HP * BQ];     // factor of this tile for accumulators and sums
+  __shared__ int s_flag, s_seq, s_tile;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
+  const int H = a.H, G = a.Hkv, Gs = H / G, dk = a.dk;
+  const int dvc = a.dv / gridDim.y, dv0 = blockIdx.y * dvc, nc = dvc / 16;
+
+  // ---- which (sequence, tile): tiles are numbered sequence by sequence ----
+  if (warp == 0) {
+    int left = blockIdx.x, seq = -1, tile = 0;
+    for (int base = 0; base < a.n && seq < 0; base += 32) {
+      const int s = base + lane;
+      const int t = s < a.n ? (a.cu_q[s + 1] - a.cu_q[s] + BQ - 1) / BQ : 0;
+      int incl = t;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const int y = __shfl_up_sync(0xffffffffu, incl, o);
+        if (lane >= o) incl += y;
+      }
+      const unsigned hit = __ballot_sync(0xffffffffu, left < incl);
+      if (hit) {
+        const int src = __ffs(hit) - 1;
+        seq = base + src;
+        tile = left - __shfl_sync(0xffffffffu, incl - t, src);
+      } else {
+        left -= __shfl_sync(0xffffffffu, incl, 31);
+      }
+    }
+    if (lane == 0) {
+      s_seq = seq;
+      s_tile = tile;
+    }
+  }
+  __syncthreads();
+  const int seq = s_seq;
+  if (seq < 0) return;
+  const int q0 = a.cu_q[seq], q_len = a.cu_q[seq + 1] - q0;
+  const int k_len = a.cu_k[seq + 1] - a.cu_k[seq];
+  const int m0 = s_tile * BQ, rows = min(BQ, q_len - m0);
+  const int pos0 = k_len - q_len + m0;                 // position of row 0
+  const int klo = a.window > 0 ? max(0, pos0 - a.window + 1) : 0;
+  const int khi = pos0 + rows;                         // one past the last visible key
+  const int ntiles = (khi - klo + BK - 1) / BK;
+
+  const int strQ = dk + 8, strK = G * dk + 8, strV = G * dvc + 8;      // elements; odd multiples of 16 bytes
+  const uint32_t sQ = smem_u32(smem);
+  const uint32_t sS = sQ + H * BQ * strQ * 2;
+  const uint32_t sK = sS + H * BQ * kSRow * 4;
+  const uint32_t sV = sK + BK * strK * 2;
+  float* S = reinterpret_cast<float*>(smem + (sS - sQ));
+
+  // ---- loads ----
+  auto pool_row = [&](int j) -> int64_t {
+    const int blk = j / a.bs;
+    const int id = blk < a.bt_stride ? __ldg(a.bt + static_cast<int64_t>(seq) * a.bt_stride + blk) : -1;
+    if (id < 0 || id >= a.num_blocks) {
+      report(a.status, B200_ERR_BOUNDS);
+      return -1;
+    }
+    return static_cast<int64_t>(id) * a.bs + j % a.bs;
+  };
+  auto load_rows = [&](int t, const void* cache, int d, int d0, int width, uint32_t dst, int stride) {
+    // 32 rows x G heads x width columns (from column d0 of d) of the pool; 8 threads per row
+    const int r = tid >> 3, j = klo + t * BK + r;
+    const int64_t row = j < khi ? pool_row(j) : -1;
+    const int cpw = width / 8, total = G * cpw;
+    const __nv_bfloat16* src = static_cast<const __nv_bfloat16*>(cache) + (row < 0 ? 0 : row) * G * d + d0;
+    const int bytes = row >= 0 ? 16 : 0;
+    if (width == d) {
+      for (int c = tid & 7; c < total; c += 8) cp_async16(dst + (r * stride + c * 8) * 2, src + c * 8, bytes);
+    } else {
+      for (int c = tid & 7; c < total; c += 8) {
+        const int hd = c / cpw, cc = c - hd * cpw;
+        cp_async16(dst + (r * stride + c * 8) * 2, src + hd * d + cc * 8, bytes);
+      }
+    }
+  };
+  {
+    const int cpr = dk / 8, per_row = H * cpr;
+    for (int i = tid; i < BQ * per_row; i += kThreads) {
+      const int r = i / per_row, c = i - r * per_row, h = c / cpr, cc = c - h * cpr;
+      const __nv_bfloat16* src = static_cast<const __nv_bfloat16*>(a.q) +
+                                 static_cast<int64_t>(q0 + m0 + (r < rows ? r : 0)) * a.q_stride + h * dk + cc * 8;
+      cp_async16(sQ + ((h * BQ + r) * strQ + cc * 8) * 2, src, r < rows ? 16 : 0);
+    }
+  }
+  load_rows(0, a.kc, dk, 0, dk, sK, strK);
+  cp_async_commit();
+  load_rows(0, a.vc, a.dv, dv0, dvc, sV, strV);
+  cp_async_commit();
+  for (int i = tid; i < HP * BQ; i += kThreads) {
+    s_ref[i] = -INFINITY;
+    s_cor[i] = 1.f;
+  }
+  if (tid == 0) s_flag = 0;
+
+  float o[HPW][2 * MAXC][4], l[HPW][2];
+#pragma unroll
+  for (int hh = 0; hh < HPW; ++hh) {
+    l[hh][0] = l[hh][1] = 0.f;
+#pragma unroll
+    for (int c = 0; c < 2 * MAXC; ++c) o[hh][c][0] = o[hh][c][1] = o[hh][c][2] = o[hh][c][3] = 0.f;
+  }
+  const float kx = a.cap > 0.f ? 2.f * kLog2e * a.scale / a.cap : 0.f;
+  const float cap = a.cap, two_cap = 2.f * a.cap;
+  cp_async_wait<1>();
+  __syncthreads();
+
+  for (int t = 0; t < ntiles; ++t) {
+    // ---- QK ----
+    {
+      const int ar = (lane & 7) + ((lane >> 3) & 1) * 8, ac = lane >> 4;
+      const int br = (lane & 7) + (lane >> 4) * 8, bc = (lane >> 3) & 1;
+#pragma unroll
+      for (int h0 = 0; h0 < HPW; h0 += 2) {            // two heads at a time share the key fragments of their group
+        constexpr int HS = HPW < 2 ? 1 : 2;
+        float s[HS][4][4];
+#pragma unroll
+        for (int hh = 0; hh < HS; ++hh)
+#pragma unroll
+          for (int n = 0; n < 4; ++n) s[hh][n][0] = s[hh][n][1] = s[hh][n][2] = s[hh][n][3] = 0.f;
+        const int hbase = warp * HPW + h0;
+        if (hbase < H) {
+          for (int ks = 0; ks < dk / 16; ++ks) {
+            uint32_t b0[4], b1[4];
+            int cur = -1;
+#pragma unroll
+            for (int hh = 0; hh < HS; ++hh) {
+              const int h = hbase + hh;
+              if (h < H) {
+                if (h / Gs != cur) {
+                  cur = h / Gs;
+                  ldmatrix_x4(b0, sK + (br * strK + cur * dk + (2 * ks + bc) * 8) * 2);
+                  ldmatrix_x4(b1, sK + ((br + 16) * strK + cur * dk + (2 * ks + bc) * 8) * 2);
+                }
+                uint32_t af[4];
+                ldmatrix_x4(af, sQ + ((h * BQ + ar) * strQ + (2 * ks + ac) * 8) * 2);
+                const uint32_t f0[2] = {b0[0], b0[1]}, f1[2] = {b0[2], b0[3]}, f2[2] = {b1[0], b1[1]},
+                               f3[2] = {b1[2], b1[3]};
+                mma_bf16_16816(s[hh][0], af, f0);
+                mma_bf16_16816(s[hh][1], af, f1);
+                mma_bf16_16816(s[hh][2], af, f2);
+                mma_bf16_16816(s[hh][3], af, f3);
+              }
+            }
+          }
+#pragma unroll
+          for (int hh = 0; hh < HS; ++hh) {
+            const int h = hbase + hh;
+            if (h < H) {
+              float* row = S + (h * BQ + g) * kSRow + tq * 2;
+#pragma unroll
+              for (int n = 0; n < 4; ++n) {
+                *reinterpret_cast<float2*>(row + n * 8) = make_float2(s[hh][n][0], s[hh][n][1]);
+                *reinterpret_cast<float2*>(row + 8 * kSRow + n * 8) = make_float2(s[hh][n][2], s[hh][n][3]);
+              }
+            }
+          }
+        }
+      }
+      for (int i = tid; i < H * BQ; i += kThreads) s_cor[i] = 1.f;
+      if (tid == 0) s_flag = 0;
+    }
+    __syncthreads();
+    if (t + 1 < ntiles) load_rows(t + 1, a.kc, dk, 0, dk, sK, strK);
+    cp_async_commit();
+
+    // ---- mix ----
+#pragma unroll 1
+    for (int r = warp; r < rows; r += kWarps) {
+      const int dist = pos0 + r - (klo + t * BK + lane);
+      const bool seen = dist >= 0 && (a.window <= 0 || dist < a.window);
+      const int dc = seen ? dist : 0;
+      float* Sr = S + r * kSRow + lane;
+      float s[HP];
+#pragma unroll
+      for (int h = 0; h < HP; ++h) {
+        s[h] = 0.f;
+        if (h < H) {
+          const float bias = a.bias_len > 0 ? __ldg(a.bias_table + h * a.bias_len + dc)
+                                            : mp.r1[h] * logf(1.f + mp.r2[h] * static_cast<float>(dc));
+          const float x = Sr[h * BQ * kSRow];
+          s[h] = cap > 0.f ? capped(x, kx, cap, two_cap, bias) : x * a.scale - bias;
+        }
+      }
+      __nv_bfloat16* Pr = reinterpret_cast<__nv_bfloat16*>(S + r * kSRow) + lane;
+      __syncwarp();                            // every lane has read its scores of the row
+      // eight mixed heads at a time: few registers stay live beside the accumulators
+#pragma unroll
+      for (int hb = 0; hb < HP; hb += 8) {
+        float m[8];
+        bool up = false;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+          float acc = 0.f;
+#pragma unroll
+          for (int k = 0; k < HP; ++k) acc = fmaf(mp.t[(hb + i) * HP + k], s[k], acc);
+          m[i] = seen ? acc : -INFINITY;
+          up |= hb + i < H && m[i] > s_ref[(hb + i) * BQ + r] + kSlack;
+        }
+        if (__any_sync(0xffffffffu, up)) {     // some head of this row needs a new reference
+#pragma unroll
+          for (int i = 0; i < 8; ++i)
+            if (hb + i < H) {
+              const float mx = warp_max(m[i]), ref = s_ref[(hb + i) * BQ + r];
+              __syncwarp();
+              if (mx > ref + kSlack && lane == 0) {
+                s_ref[(hb + i) * BQ + r] = mx;
+                s_cor[(hb + i) * BQ + r] = fast_exp2(ref - mx);   // ref = -inf: nothing accumulated yet
+                s_flag = 1;
+              }
+            }
+          __syncwarp();
+        }
+#pragma unroll
+        for (int i = 0; i < 8; ++i)
+          if (hb + i < H)
+            Pr[(hb + i) * BQ * kSRow * 2] =
+                __float2bfloat16_rn(seen ? fast_exp2(m[i] - s_ref[(hb + i) * BQ + r]) : 0.f);
+      }
+    }
+    cp_async_wait<1>();
+    __syncthreads();
+
+    // ---- PV ----
+    {
+      const int ar = (lane & 7) + ((lane >> 3) & 1) * 8, ac = lane >> 4;
+      uint32_t pf[HPW][2][4];
+      const bool rescale = s_flag != 0;
+#pragma unroll
+      for (int hh = 0; hh < HPW; ++hh) {
+        const int h = warp * HPW + hh;
+        if (h < H) {
+          if (rescale) {
+            const float c0 = s_cor[h * BQ + g], c1 = s_cor[h * BQ + g + 8];
+            l[hh][0] *= c0;
+            l[hh][1] *= c1;
+#pragma unroll
+            for (int c = 0; c < 2 * MAXC; ++c) {
+              o[hh][c][0] *= c0;
+              o[hh][c][1] *= c0;
+              o[hh][c][2] *= c1;
+              o[hh][c][3] *= c1;
+            }
+          }
+#pragma unroll
+          for (int kk = 0; kk < 2; ++kk) {
+            ldmatrix_x4(pf[hh][kk], sS + ((h * BQ + ar) * kSRow) * 4 + (2 * kk + ac) * 16);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+              const float2 p = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&pf[hh][kk][e]));
+              l[hh][e & 1] += p.x + p.y;
+            }
+          }
+        }
+      }
+#pragma unroll
+      for (int kk = 0; kk < 2; ++kk) {
+#pragma unroll
+        for (int c = 0; c < MAXC; ++c) {
+          if (c < nc) {
+            uint32_t bf[4];
+            int cur = -1;
+#pragma unroll
+            for (int hh = 0; hh < HPW; ++hh) {
+              const int h = warp * HPW + hh;
+              if (h < H) {
+                if (h / Gs != cur) {
+                  cur = h / Gs;
+                  ldmatrix_x4_trans(bf, sV + ((kk * 16 + ar) * strV + cur * dvc + (2 * c + ac) * 8) * 2);
+                }
+                const uint32_t b0[2] = {bf[0], bf[1]}, b1[2] = {bf[2], bf[3]};
+                mma_bf16_16816(o[hh][2 * c], pf[hh][kk], b0);
+                mma_bf16_16816(o[hh][2 * c + 1], pf[hh][kk], b1);
+              }
+            }
+          }
+        }
+      }
+    }
+    cp_async_wait<0>();
+    __syncthreads();
+    if (t + 1 < ntiles) load_rows(t + 1, a.vc, a.dv, dv0, dvc, sV, strV);
+    cp_async_commit();
+  }
+  cp_async_wait<0>();
+
+  // ---- normalise, gate, store ----
+#pragma unroll
+  for (int hh = 0; hh < HPW; ++hh) {
+    const int h = warp * HPW + hh;
+    if (h >= H) continue;
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      float sum = l[hh][e];
+      sum += __shfl_xor_sync(0xffffffffu, sum, 1);
+      sum += __shfl_xor_sync(0xffffffffu, sum, 2);
+      const int r = g + e * 8;
+      if (r >= rows) continue;
+      const float inv = sum > 0.f ? 1.f / sum : 0.f;
+      const int64_t row = q0 + m0 + r;
+      __nv_bfloat16* op = static_cast<__nv_bfloat16*>(a.out) + (row * H + h) * a.dv + dv0 + tq * 2;
+      const __nv_bfloat16* gp =
+          a.gate ? static_cast<const __nv_bfloat16*>(a.gate) + row * a.gate_stride + h * a.dv + dv0 + tq * 2 : nullptr;
+#pragma unroll
+      for (int c = 0; c < 2 * MAXC; ++c) {
+        if (c < 2 * nc) {
+          float x = o[hh][c][e * 2] * inv, y = o[hh][c][e * 2 + 1] * inv;
+          if (gp) {
+            const float2 gv = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gp + c * 8));
+            x = x / (1.f + __expf(-gv.x));
+            y = y / (1.f + __expf(-gv.y));
+          }
+          *reinterpret_cast<uint32_t*>(op + c * 8) = pack_bf16x2(x, y);
+        }
+      }
+    }
+  }
+}
+
+template <int HP, int MAXC, int MINB>
+int launch_prefill(const TalkArgs& a, int chunks, size_t smem, cudaStream_t s) {
+  MixParam<HP> mp;
+  memset(&mp, 0, sizeof(mp));
+  for (int h = 0; h < a.H; ++h)
+    for (int k = 0; k < a.H; ++k) mp.t[h * HP + k] = a.talk_host[h * a.H + k] * kLog2e;
+  for (int h = 0; h < a.H; ++h) {
+    mp.r1[h] = a.r1_host[h];
+    mp.r2[h] = a.r2_host[h];
+  }
+  auto kern = talking_prefill_kernel<HP, MAXC, MINB>;
+  static size_t configured[64] = {};
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (dev < 0 || dev >= 64 || configured[dev] < smem) {
+    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)) != cudaSuccess)
+      return B200_ERR_LAUNCH;
+    if (dev >= 0 && dev < 64) configured[dev] = smem;
+  }
+  const int64_t tiles = a.rows / BQ + a.n;          // sum over sequences of ceil(q_len / 16) is at most this
+  kern<<<dim3(static_cast<unsigned>(tiles), chunks), kThreads, smem, s>>>(a, mp);
+  return launch_result();
+}
+
+}  // namespace
+
+int talking_prefill_mma_launch(const TalkArgs& a, cudaStream_t s) {
+  if (!a.talk_host || !a.r1_host || !a.r2_host || !a.cu_q || a.H > 32 || a.dk % 16 || a.dv % 16 || a.dk > 256)
+    return B200_ERR_UNSUPPORTED;
+  if (a.q_stride % 8 || (a.gate && a.gate_stride % 2) || !aligned16(a.q) || !aligned16(a.kc) || !aligned16(a.vc) ||
+      !aligned16(a.out) || (reinterpret_cast<uintptr_t>(a.gate) & 3))
+    return B200_ERR_UNSUPPORTED;
+  // value columns per CTA: what the accumulators of a warp's heads hold, and what shared memory leaves room for
+  const int max_c = a.H <= 8 ? 16 : a.H <= 16 ? 8 : 4;     // units of 16 columns
+  for (int chunks = 1; chunks <= a.dv / 16; ++chunks) {
+    if (a.dv % (16 * chunks)) continue;
+    const int dvc = a.dv / chunks;
+    if (dvc / 16 > max_c) continue;
+    const size_t smem = size_t(a.H) * BQ * (a.dk + 8) * 2 + size_t(a.H) * BQ * kSRow * 4 +
+                        size_t(BK) * (a.Hkv * a.dk + 8) * 2 + size_t(BK) * (a.Hkv * dvc + 8) * 2;
+    if (smem > 220 * 1024) continue;
+    const bool two = smem <= 108 * 1024 && dvc / 16 <= max_c / 2;     // two CTAs per SM: half the registers each
+    if (a.H <= 8) return two ? launch_prefill<8, 8, 2>(a, chunks, smem, s) : launch_prefill<8, 16, 1>(a, chunks, smem, s);
+    if (a.H <= 16) return two ? launch_prefill<16, 4, 2>(a, chunks, smem, s) : launch_prefill<16, 8, 1>(a, chunks, smem, s);
+    return launch_prefill<32, 4, 1>(a, chunks, smem, s);
+  }
+  return B200_ERR_UNSUPPORTED;
+}
+
+}  // namespace b200

@@ -806,17 +806,17 @@ class TalkingHeads:
         H = talk.shape[0]
         self.scale, self.softcap, self.window, self.H = float(scale), float(softcap), int(window), H
         host = talk.detach().float().cpu().contiguous()
-        self.talk_host = host
         self.talk = host.to(device)
         self.r1 = r1.detach().float().to(device).contiguous()
         self.r2 = r2.detach().float().to(device).contiguous()
         for name, t, n in (("r1", self.r1, H), ("r2", self.r2, H), ("talk", self.talk, H * H)):
             _f32vec(name, t, n)
+        self.consts_host = torch.cat([host.reshape(-1), r1.detach().float().cpu(), r2.detach().float().cpu()]).contiguous()
         self.table = None
         if 0 < self.window <= self.max_table:
-            dist = torch.arange(self.window, dtype=torch.float64)[:, None]
-            t = r1.detach().double().cpu() * torch.log1p(r2.detach().double().cpu() * dist)
-            self.table = t.float().to(device).contiguous()       # [window, H]
+            dist = torch.arange(self.window, dtype=torch.float64)[None, :]
+            t = r1.detach().double().cpu()[:, None] * torch.log1p(r2.detach().double().cpu()[:, None] * dist)
+            self.table = t.float().to(device).contiguous()       # [H, window]
 
 
 def talking_attention(q: torch.Tensor, gate: torch.Tensor | None, k_cache: torch.Tensor, v_cache: torch.Tensor,
@@ -857,8 +857,8 @@ def talking_attention(q: torch.Tensor, gate: torch.Tensor | None, k_cache: torch
         q.data_ptr(), q.stride(0), _ptr(gate), gate.stride(0) if gate is not None else 0, k_cache.data_ptr(),
         v_cache.data_ptr(), out.data_ptr(), block_tables.data_ptr(), block_tables.stride(0), bs, nb, _ptr(cu_seqlens_q),
         _ptr(cu_seqlens_k), _ptr(context_lens), n, rows, int(max_seqlen_q), H, Hkv, dk, dv, c.scale, c.softcap,
-        c.r1.data_ptr(), c.r2.data_ptr(), c.talk.data_ptr(), None if general else c.talk_host.data_ptr(), _ptr(c.table),
-        c.table.shape[0] if c.table is not None else 0, c.window, _ptr(ws), ws.numel() if ws is not None else 0, _dt(q),
+        c.r1.data_ptr(), c.r2.data_ptr(), c.talk.data_ptr(), None if general else c.consts_host.data_ptr(), _ptr(c.table),
+        c.table.shape[1] if c.table is not None else 0, c.window, _ptr(ws), ws.numel() if ws is not None else 0, _dt(q),
         status_word(dev).data_ptr(), _stream()), "talking_attention")
     return out
 
