@@ -282,7 +282,8 @@ def main():
     ap.add_argument("--no-e2e", action="store_true", help="skip the host-input leg (profiling runs)")
     ap.add_argument("--no-secondary", action="store_true", help="skip the secondary kernels (profiling runs)")
     ap.add_argument("--no-engine", action="store_true", help="skip the engine job (profiling runs)")
-    ap.add_argument("--workload", default="decode", choices=["decode", "mla_decode", "prefill", "prefill64", "mla_prefill", "store", "moe_experts", "lm_head", "engine", "engine_mla", "engine_step"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "mla_decode", "prefill", "prefill64", "mla_prefill", "store", "moe_experts", "lm_head", "engine", "engine_mla", "engine_step",
+                                                                 "nabalix", "nabalix_kernels"],
                     help="decode = the benchmark (paged GQA decode); the others time a secondary kernel on "
                          "its benchmark shape and print a short JSON line (single GPU, no reference arm)")
     ap.add_argument("--rate", type=float, default=0.0, help="engine workload: Poisson arrival rate (req/s); 0 = offline")
@@ -297,7 +298,12 @@ def main():
     if args.workload != "decode":
         from llm_from_scratch_b200 import microbench
         torch.cuda.set_device(int(os.environ.get("LOCAL_RANK", "0")))
-        fn = getattr(microbench, args.workload)
+        if args.workload.startswith("nabalix"):
+            from llm_from_scratch_b200 import microbench_nabalix
+            fn = microbench_nabalix.kernels if args.workload == "nabalix_kernels" else microbench_nabalix.throughput
+            args.steps = min(args.steps, 50)
+        else:
+            fn = getattr(microbench, args.workload)
         kw = dict(steps=args.steps, warmup=args.warmup)
         if args.workload == "engine" and args.rate > 0:
             kw["rate"] = args.rate
@@ -306,7 +312,7 @@ def main():
         if args.batch != BATCH:   # profiling cases: fewer sequences / tokens
             key = {"mla_decode": "batch", "engine": "batch", "prefill": "total", "store": "tokens",
                    "moe_experts": "tokens", "engine_mla": "batch", "mla_prefill": "seqs", "engine_step": "batch",
-                   "prefill64": "seqs", "lm_head": "rows"}[args.workload]
+                   "prefill64": "seqs", "lm_head": "rows", "nabalix": "batch"}[args.workload]
             kw[key] = args.batch
         res = fn(**kw)
         if not res:       # a non-zero rank of a multi-replica engine run
