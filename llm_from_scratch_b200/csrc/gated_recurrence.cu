@@ -44,14 +44,31 @@ struct RecArgs {
   int32_t* status;
 };
 
-__device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
+__device__ __forceinline__ float rcp_approx(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
 
-// forget gate and write gate of one channel; 1 - f is formed from sigmoid(-z) so that it keeps its relative
-// accuracy when the gate is almost closed
+// sigmoid(z) and sigmoid(-z) from one exponential of -|z|, so that the small one keeps its relative accuracy
+__device__ __forceinline__ void sigmoids(float z, float* s, float* s_neg) {
+  const float t = expf(-fabsf(z)), big = rcp_approx(1.f + t), small = t * big;
+  *s = z >= 0.f ? big : small;
+  *s_neg = z >= 0.f ? small : big;
+}
+__device__ __forceinline__ float silu_f(float x) {
+  float s, n;
+  sigmoids(x, &s, &n);
+  return x * s;
+}
+
+// forget gate and write gate of one channel
 __device__ __forceinline__ void gates(float z, float lower, float* f, float* k) {
   const float open = 1.f - lower;
-  *f = lower + open * sigmoid_f(z);
-  *k = open * sigmoid_f(-z);
+  float s, n;
+  sigmoids(z, &s, &n);
+  *f = lower + open * s;
+  *k = open * n;
 }
 
 // The sequence's token range, first position and state slot; false = nothing to do.
@@ -106,7 +123,7 @@ __global__ void __launch_bounds__(kStepThreads) recurrence_step_kernel(const Rec
     const bool zero = info.fresh && t == 0;
     for (int i = threadIdx.x; i < dk; i += kStepThreads) {
       const float qv = to_float<T>(qp[i]);
-      sq[i] = qv * sigmoid_f(qv);
+      sq[i] = silu_f(qv);
       gates(to_float<T>(fp[i]) + a.f_bias[head * dk + i], a.lower[head * dk + i], &sf[i], &sk[i]);
     }
     __syncthreads();
@@ -175,7 +192,7 @@ int launch_step(const RecArgs& a, int n, bool vec, cudaStream_t s) {
   while (CL < units && CL < kStepThreads) CL *= 2;
   const size_t smem = (3 * static_cast<size_t>(a.dk) + a.dv + kStepThreads * V + 8) * sizeof(float);
   auto kern = vec ? recurrence_step_kernel<T, 4> : recurrence_step_kernel<T, 1>;
-  if (smem > 48 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize,
+  if (smem > 40 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                                static_cast<int>(smem)) != cudaSuccess)
     return B200_ERR_LAUNCH;
   kern<<<dim3(a.H, n), kStepThreads, smem, s>>>(a, CL);
@@ -269,7 +286,7 @@ __global__ void __launch_bounds__(512, 1) recurrence_scan_kernel(const RecArgs a
   float* sk = sf + kBlockTokens * DK;
   float* sq = sk + kBlockTokens * DK;              // outputs only
   float* sv = sq + (LOCAL ? 0 : kBlockTokens * DK);
-  float* so = sv + kBlockTokens * dv;              // [kBlockTokens, dv], outputs only
+  float* so = sv + 2 * kBlockTokens * dv;          // [kBlockTokens, dv], outputs only
   const int tid = threadIdx.x, threads = blockDim.x, rg = tid & (kRowGroups - 1), c0 = (tid / kRowGroups) * C;
   const bool cols = c0 < dv;                       // dv is a multiple of 4: a float4 is in or out as a whole
 
@@ -308,8 +325,7 @@ __global__ void __launch_bounds__(512, 1) recurrence_scan_kernel(const RecArgs a
         const int64_t off = (tok + t) * a.stride + head * dk + d;
         gates(to_float<T>(static_cast<const T*>(a.f)[off]) + a.f_bias[head * dk + d], a.lower[head * dk + d], &f, &k);
         if (!LOCAL) {
-          q = to_float<T>(static_cast<const T*>(a.q)[off]);
-          q *= sigmoid_f(q);
+          q = silu_f(to_float<T>(static_cast<const T*>(a.q)[off]));
         }
       }
       sf[i] = f;
@@ -318,9 +334,11 @@ __global__ void __launch_bounds__(512, 1) recurrence_scan_kernel(const RecArgs a
     }
     for (int i = tid; i < nb * dv; i += threads) {
       const int t = i / dv, d = i - t * dv;
-      sv[i] = to_float<T>(static_cast<const T*>(a.v)[(tok + t) * a.stride + head * dv + d]);
+      const float x = to_float<T>(static_cast<const T*>(a.v)[(tok + t) * a.stride + head * dv + d]);
+      *reinterpret_cast<float2*>(sv + 2 * i) = make_float2(x, x);       // both halves of a packed operand
     }
     __syncthreads();
+#pragma unroll 2
     for (int t = 0; t < nb; ++t) {
       f32x2 f[P], k[P], q[P], v[C];
 #pragma unroll
@@ -334,12 +352,11 @@ __global__ void __launch_bounds__(512, 1) recurrence_scan_kernel(const RecArgs a
         }
       }
 #pragma unroll
-      for (int c = 0; c < C; c += 4) {
-        const float4 x = c0 + c < dv ? *reinterpret_cast<const float4*>(sv + t * dv + c0 + c) : make_float4(0.f, 0.f, 0.f, 0.f);
-        v[c] = pack2(x.x, x.x);
-        v[c + 1] = pack2(x.y, x.y);
-        v[c + 2] = pack2(x.z, x.z);
-        v[c + 3] = pack2(x.w, x.w);
+      for (int c = 0; c < C; c += 2) {
+        // columns past the last one (dv not a multiple of C) repeat column 0: never stored
+        const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(sv + 2 * (t * dv + (c0 + c < dv ? c0 + c : 0)));
+        v[c] = x.x;
+        v[c + 1] = x.y;
       }
       float o[C];
 #pragma unroll
@@ -434,15 +451,28 @@ __global__ void __launch_bounds__(256) recurrence_chain_kernel(const RecArgs a, 
                         : *reinterpret_cast<const float4*>(a.state + (info.slot * a.H + head) * per_head + e);
   float* st = sc.seg_state + (static_cast<int64_t>(s_first) * a.H + head) * per_head + e;
   const float* dec = sc.seg_decay + (static_cast<int64_t>(s_first) * a.H + head) * a.dk + r;
-#pragma unroll 4
-  for (int i = 0; i < segments - 1; ++i, st += a.H * per_head, dec += static_cast<int64_t>(a.H) * a.dk) {
-    const float4 p = *reinterpret_cast<const float4*>(st);
-    const float d = *dec;
-    *reinterpret_cast<float4*>(st) = S;
-    S.x = fmaf(d, S.x, p.x);
-    S.y = fmaf(d, S.y, p.y);
-    S.z = fmaf(d, S.z, p.z);
-    S.w = fmaf(d, S.w, p.w);
+  const int64_t st_step = a.H * per_head, dec_step = static_cast<int64_t>(a.H) * a.dk;
+  constexpr int U = 8;                               // loads in flight
+  for (int i = 0; i < segments - 1; i += U) {
+    float4 p[U];
+    float d[U];
+#pragma unroll
+    for (int u = 0; u < U; ++u)
+      if (i + u < segments - 1) {
+        p[u] = *reinterpret_cast<const float4*>(st + u * st_step);
+        d[u] = dec[u * dec_step];
+      }
+#pragma unroll
+    for (int u = 0; u < U; ++u)
+      if (i + u < segments - 1) {
+        *reinterpret_cast<float4*>(st) = S;
+        S.x = fmaf(d[u], S.x, p[u].x);
+        S.y = fmaf(d[u], S.y, p[u].y);
+        S.z = fmaf(d[u], S.z, p[u].z);
+        S.w = fmaf(d[u], S.w, p[u].w);
+        st += st_step;
+        dec += dec_step;
+      }
   }
   *reinterpret_cast<float4*>(st) = S;
 }
@@ -462,8 +492,8 @@ int launch_scan(const RecArgs& a, const ScanArgs& sc, int64_t segments, bool cha
   auto local = recurrence_scan_kernel<T, R, C, true>;
   auto full = recurrence_scan_kernel<T, R, C, false>;
   const size_t one = size_t(kBlockTokens) * R * kRowGroups * sizeof(float), v = size_t(kBlockTokens) * a.dv * sizeof(float);
-  const size_t smem_local = 2 * one + 2 * v, smem_full = 3 * one + 2 * v;
-  if (smem_full > 48 * 1024 &&
+  const size_t smem_local = 2 * one + 2 * v, smem_full = 3 * one + 3 * v;
+  if (smem_full > 40 * 1024 &&
       (cudaFuncSetAttribute(local, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem_local)) != cudaSuccess ||
        cudaFuncSetAttribute(full, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem_full)) != cudaSuccess))
     return B200_ERR_LAUNCH;

@@ -231,7 +231,7 @@ int launch_streams(const StreamArgs& a, int64_t rows, cudaStream_t s) {
     case 4: kern = stream_update_kernel<T, V, 4>; break;
     default: break;
   }
-  if (smem > 48 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize,
+  if (smem > 40 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                                static_cast<int>(smem)) != cudaSuccess)
     return B200_ERR_LAUNCH;
   kern<<<static_cast<unsigned>(rows), threads, smem, s>>>(a);

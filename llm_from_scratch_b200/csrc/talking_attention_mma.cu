@@ -22,11 +22,10 @@ namespace {
 
 constexpr int BQ = 16;
 constexpr int BK = 32;
-constexpr int kWarps = 8;
-constexpr int kThreads = kWarps * 32;
 constexpr int kSRow = 40;            // floats per score row: 32 keys + padding against bank conflicts
 constexpr float kSlack = 30.f;       // log2 of how far a score may exceed the row's reference
 
+constexpr float kNoRef = -3.0e38f;   // reference of a row that has seen no key
 constexpr float kLog2e = 1.4426950408889634f;
 
 template <int HP>
@@ -46,13 +45,15 @@ __device__ __forceinline__ float capped(float x, float k, float cap, float two_c
   return (cap - bias) - two_cap * rcp_approx(1.f + fast_exp2(x * k));
 }
 
-template <int HP, int MAXC, int MINB>
-__global__ void __launch_bounds__(kThreads, MINB)
-talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp) {
-  constexpr int HPW = HP / kWarps;
+// HP: heads padded; NW: warps; MAXC: value columns per CTA in units of 16; COMMON: soft cap and bias table present;
+// q_smem: the query rows are staged in shared memory (else their fragments are read from global memory)
+template <int HP, int NW, int MAXC, int MINB, bool COMMON>
+__global__ void __launch_bounds__(NW * 32, MINB)
+talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp, const int q_smem) {
+  constexpr int HPW = HP / NW, kThreads = NW * 32, kTpr = kThreads / BK;    // kTpr: threads that load one key row
   extern __shared__ __align__(128) uint8_t smem[];
-  __shared__ float s_ref[HP * BQ];     // reference maximum (log2 domain) per (head, row)
-  __shared__ float s_cor[HP * BQ];     // factor of this tile for accumulators and sums
+  __shared__ __align__(16) float s_ref[BQ * HP];     // reference maximum (log2 domain) per (row, head)
+  __shared__ float s_cor[BQ * HP];     // factor of this tile for accumulators and sums
   __shared__ int s_flag, s_seq, s_tile;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
   const int H = a.H, G = a.Hkv, Gs = H / G, dk = a.dk;
@@ -97,7 +98,7 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
 
   const int strQ = dk + 8, strK = G * dk + 8, strV = G * dvc + 8;      // elements; odd multiples of 16 bytes
   const uint32_t sQ = smem_u32(smem);
-  const uint32_t sS = sQ + H * BQ * strQ * 2;
+  const uint32_t sS = sQ + (q_smem ? H * BQ * strQ * 2 : 0);
   const uint32_t sK = sS + H * BQ * kSRow * 4;
   const uint32_t sV = sK + BK * strK * 2;
   float* S = reinterpret_cast<float*>(smem + (sS - sQ));
@@ -113,27 +114,27 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
     return static_cast<int64_t>(id) * a.bs + j % a.bs;
   };
   auto load_rows = [&](int t, const void* cache, int d, int d0, int width, uint32_t dst, int stride) {
-    // 32 rows x G heads x width columns (from column d0 of d) of the pool; 8 threads per row
-    const int r = tid >> 3, j = klo + t * BK + r;
+    // 32 rows x G heads x width columns (from column d0 of d) of the pool
+    const int r = tid / kTpr, j = klo + t * BK + r;
     const int64_t row = j < khi ? pool_row(j) : -1;
     const int cpw = width / 8, total = G * cpw;
     const __nv_bfloat16* src = static_cast<const __nv_bfloat16*>(cache) + (row < 0 ? 0 : row) * G * d + d0;
     const int bytes = row >= 0 ? 16 : 0;
     if (width == d) {
-      for (int c = tid & 7; c < total; c += 8) cp_async16(dst + (r * stride + c * 8) * 2, src + c * 8, bytes);
+      for (int c = tid % kTpr; c < total; c += kTpr) cp_async16(dst + (r * stride + c * 8) * 2, src + c * 8, bytes);
     } else {
-      for (int c = tid & 7; c < total; c += 8) {
+      for (int c = tid % kTpr; c < total; c += kTpr) {
         const int hd = c / cpw, cc = c - hd * cpw;
         cp_async16(dst + (r * stride + c * 8) * 2, src + hd * d + cc * 8, bytes);
       }
     }
   };
-  {
+  const __nv_bfloat16* qrow = static_cast<const __nv_bfloat16*>(a.q) + static_cast<int64_t>(q0 + m0) * a.q_stride;
+  if (q_smem) {
     const int cpr = dk / 8, per_row = H * cpr;
     for (int i = tid; i < BQ * per_row; i += kThreads) {
       const int r = i / per_row, c = i - r * per_row, h = c / cpr, cc = c - h * cpr;
-      const __nv_bfloat16* src = static_cast<const __nv_bfloat16*>(a.q) +
-                                 static_cast<int64_t>(q0 + m0 + (r < rows ? r : 0)) * a.q_stride + h * dk + cc * 8;
+      const __nv_bfloat16* src = qrow + static_cast<int64_t>(r < rows ? r : 0) * a.q_stride + h * dk + cc * 8;
       cp_async16(sQ + ((h * BQ + r) * strQ + cc * 8) * 2, src, r < rows ? 16 : 0);
     }
   }
@@ -142,7 +143,7 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
   load_rows(0, a.vc, a.dv, dv0, dvc, sV, strV);
   cp_async_commit();
   for (int i = tid; i < HP * BQ; i += kThreads) {
-    s_ref[i] = -INFINITY;
+    s_ref[i] = i % HP < H ? kNoRef : INFINITY;
     s_cor[i] = 1.f;
   }
   if (tid == 0) s_flag = 0;
@@ -187,7 +188,16 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
                   ldmatrix_x4(b1, sK + ((br + 16) * strK + cur * dk + (2 * ks + bc) * 8) * 2);
                 }
                 uint32_t af[4];
-                ldmatrix_x4(af, sQ + ((h * BQ + ar) * strQ + (2 * ks + ac) * 8) * 2);
+                if (q_smem) {
+                  ldmatrix_x4(af, sQ + ((h * BQ + ar) * strQ + (2 * ks + ac) * 8) * 2);
+                } else {             // rows past the portion repeat its last row: their scores are never used
+                  const __nv_bfloat16* q0p = qrow + static_cast<int64_t>(min(g, rows - 1)) * a.q_stride + h * dk + ks * 16 + tq * 2;
+                  const __nv_bfloat16* q1p = qrow + static_cast<int64_t>(min(g + 8, rows - 1)) * a.q_stride + h * dk + ks * 16 + tq * 2;
+                  af[0] = __ldg(reinterpret_cast<const uint32_t*>(q0p));
+                  af[1] = __ldg(reinterpret_cast<const uint32_t*>(q1p));
+                  af[2] = __ldg(reinterpret_cast<const uint32_t*>(q0p + 8));
+                  af[3] = __ldg(reinterpret_cast<const uint32_t*>(q1p + 8));
+                }
                 const uint32_t f0[2] = {b0[0], b0[1]}, f1[2] = {b0[2], b0[3]}, f2[2] = {b1[0], b1[1]},
                                f3[2] = {b1[2], b1[3]};
                 mma_bf16_16816(s[hh][0], af, f0);
@@ -211,7 +221,7 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
           }
         }
       }
-      for (int i = tid; i < H * BQ; i += kThreads) s_cor[i] = 1.f;
+      for (int i = tid; i < HP * BQ; i += kThreads) s_cor[i] = 1.f;
       if (tid == 0) s_flag = 0;
     }
     __syncthreads();
@@ -220,56 +230,64 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
 
     // ---- mix ----
 #pragma unroll 1
-    for (int r = warp; r < rows; r += kWarps) {
+    for (int r = warp; r < rows; r += NW) {
       const int dist = pos0 + r - (klo + t * BK + lane);
       const bool seen = dist >= 0 && (a.window <= 0 || dist < a.window);
       const int dc = seen ? dist : 0;
       float* Sr = S + r * kSRow + lane;
+      const float* table = a.bias_table + dc;
       float s[HP];
 #pragma unroll
+      for (int h = 0; h < HP; ++h) s[h] = h < H ? Sr[h * BQ * kSRow] : 0.f;
+#pragma unroll
       for (int h = 0; h < HP; ++h) {
-        s[h] = 0.f;
-        if (h < H) {
-          const float bias = a.bias_len > 0 ? __ldg(a.bias_table + h * a.bias_len + dc)
+        if constexpr (COMMON) {
+          const float bias = __ldg(table + min(h, H - 1) * a.bias_len);
+          s[h] = capped(s[h], kx, cap, two_cap, bias);    // a padding head is finite and meets zeros of the mix
+        } else {
+          const float bias = a.bias_len > 0 ? __ldg(table + min(h, H - 1) * a.bias_len)
                                             : mp.r1[h] * logf(1.f + mp.r2[h] * static_cast<float>(dc));
-          const float x = Sr[h * BQ * kSRow];
-          s[h] = cap > 0.f ? capped(x, kx, cap, two_cap, bias) : x * a.scale - bias;
+          s[h] = cap > 0.f ? capped(s[h], kx, cap, two_cap, bias) : s[h] * a.scale - bias;
         }
       }
       __nv_bfloat16* Pr = reinterpret_cast<__nv_bfloat16*>(S + r * kSRow) + lane;
+      const float base = seen ? 0.f : -INFINITY;
       __syncwarp();                            // every lane has read its scores of the row
       // eight mixed heads at a time: few registers stay live beside the accumulators
 #pragma unroll
       for (int hb = 0; hb < HP; hb += 8) {
-        float m[8];
-        bool up = false;
+        float m[8], top = -INFINITY;
 #pragma unroll
-        for (int i = 0; i < 8; ++i) {
-          float acc = 0.f;
+        for (int i = 0; i < 8; ++i) m[i] = base;
 #pragma unroll
-          for (int k = 0; k < HP; ++k) acc = fmaf(mp.t[(hb + i) * HP + k], s[k], acc);
-          m[i] = seen ? acc : -INFINITY;
-          up |= hb + i < H && m[i] > s_ref[(hb + i) * BQ + r] + kSlack;
-        }
-        if (__any_sync(0xffffffffu, up)) {     // some head of this row needs a new reference
+        for (int k = 0; k < HP; ++k)
 #pragma unroll
-          for (int i = 0; i < 8; ++i)
-            if (hb + i < H) {
-              const float mx = warp_max(m[i]), ref = s_ref[(hb + i) * BQ + r];
-              __syncwarp();
-              if (mx > ref + kSlack && lane == 0) {
-                s_ref[(hb + i) * BQ + r] = mx;
-                s_cor[(hb + i) * BQ + r] = fast_exp2(ref - mx);   // ref = -inf: nothing accumulated yet
+          for (int i = 0; i < 8; ++i) m[i] = fmaf(mp.t[(hb + i) * HP + k], s[k], m[i]);
+        float4* ref4 = reinterpret_cast<float4*>(s_ref + r * HP + hb);
+        float4 ra = ref4[0], rb = ref4[1];
+        // a row without a reference yet holds the largest negative float; padding heads hold +inf and stay out
+        top = fmaxf(fmaxf(fmaxf(m[0] - ra.x, m[1] - ra.y), fmaxf(m[2] - ra.z, m[3] - ra.w)),
+                    fmaxf(fmaxf(m[4] - rb.x, m[5] - rb.y), fmaxf(m[6] - rb.z, m[7] - rb.w)));
+        if (__any_sync(0xffffffffu, top > kSlack)) {     // some head of this row needs a new reference
+#pragma unroll
+          for (int i = 0; i < 8; ++i) {
+            const float mx = warp_max(m[i]);
+            if (lane == 0) {
+              const float ref = s_ref[r * HP + hb + i];
+              if (mx > ref + kSlack) {
+                s_ref[r * HP + hb + i] = mx;
+                s_cor[r * HP + hb + i] = fast_exp2(ref - mx);
                 s_flag = 1;
               }
             }
+          }
           __syncwarp();
+          ra = ref4[0], rb = ref4[1];
         }
+        const float ref[8] = {ra.x, ra.y, ra.z, ra.w, rb.x, rb.y, rb.z, rb.w};
 #pragma unroll
         for (int i = 0; i < 8; ++i)
-          if (hb + i < H)
-            Pr[(hb + i) * BQ * kSRow * 2] =
-                __float2bfloat16_rn(seen ? fast_exp2(m[i] - s_ref[(hb + i) * BQ + r]) : 0.f);
+          if (hb + i < H) Pr[(hb + i) * BQ * kSRow * 2] = __float2bfloat16_rn(fast_exp2(m[i] - ref[i]));
       }
     }
     cp_async_wait<1>();
@@ -285,7 +303,7 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
         const int h = warp * HPW + hh;
         if (h < H) {
           if (rescale) {
-            const float c0 = s_cor[h * BQ + g], c1 = s_cor[h * BQ + g + 8];
+            const float c0 = s_cor[g * HP + h], c1 = s_cor[(g + 8) * HP + h];
             l[hh][0] *= c0;
             l[hh][1] *= c1;
 #pragma unroll
@@ -371,8 +389,8 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
   }
 }
 
-template <int HP, int MAXC, int MINB>
-int launch_prefill(const TalkArgs& a, int chunks, size_t smem, cudaStream_t s) {
+template <int HP, int NW, int MAXC, int MINB, bool COMMON>
+int launch_prefill(const TalkArgs& a, int chunks, size_t smem, bool q_smem, cudaStream_t s) {
   MixParam<HP> mp;
   memset(&mp, 0, sizeof(mp));
   for (int h = 0; h < a.H; ++h)
@@ -381,7 +399,7 @@ int launch_prefill(const TalkArgs& a, int chunks, size_t smem, cudaStream_t s) {
     mp.r1[h] = a.r1_host[h];
     mp.r2[h] = a.r2_host[h];
   }
-  auto kern = talking_prefill_kernel<HP, MAXC, MINB>;
+  auto kern = talking_prefill_kernel<HP, NW, MAXC, MINB, COMMON>;
   static size_t configured[64] = {};
   int dev = 0;
   cudaGetDevice(&dev);
@@ -391,8 +409,15 @@ int launch_prefill(const TalkArgs& a, int chunks, size_t smem, cudaStream_t s) {
     if (dev >= 0 && dev < 64) configured[dev] = smem;
   }
   const int64_t tiles = a.rows / BQ + a.n;          // sum over sequences of ceil(q_len / 16) is at most this
-  kern<<<dim3(static_cast<unsigned>(tiles), chunks), kThreads, smem, s>>>(a, mp);
+  kern<<<dim3(static_cast<unsigned>(tiles), chunks), NW * 32, smem, s>>>(a, mp, q_smem ? 1 : 0);
   return launch_result();
+}
+
+template <int HP, int NW, int MAXC, int MINB>
+int launch_prefill(const TalkArgs& a, int chunks, size_t smem, bool q_smem, cudaStream_t s) {
+  if (a.cap > 0.f && a.window > 0 && a.bias_len >= a.window)
+    return launch_prefill<HP, NW, MAXC, MINB, true>(a, chunks, smem, q_smem, s);
+  return launch_prefill<HP, NW, MAXC, MINB, false>(a, chunks, smem, q_smem, s);
 }
 
 }  // namespace
@@ -409,13 +434,18 @@ int talking_prefill_mma_launch(const TalkArgs& a, cudaStream_t s) {
     if (a.dv % (16 * chunks)) continue;
     const int dvc = a.dv / chunks;
     if (dvc / 16 > max_c) continue;
-    const size_t smem = size_t(a.H) * BQ * (a.dk + 8) * 2 + size_t(a.H) * BQ * kSRow * 4 +
-                        size_t(BK) * (a.Hkv * a.dk + 8) * 2 + size_t(BK) * (a.Hkv * dvc + 8) * 2;
+    const size_t q_bytes = size_t(a.H) * BQ * (a.dk + 8) * 2;
+    size_t smem = size_t(a.H) * BQ * kSRow * 4 + size_t(BK) * (a.Hkv * a.dk + 8) * 2 +
+                  size_t(BK) * (a.Hkv * dvc + 8) * 2;
+    const bool q_smem = smem + q_bytes <= 220 * 1024;
+    if (q_smem) smem += q_bytes;
     if (smem > 220 * 1024) continue;
-    const bool two = smem <= 108 * 1024 && dvc / 16 <= max_c / 2;     // two CTAs per SM: half the registers each
-    if (a.H <= 8) return two ? launch_prefill<8, 8, 2>(a, chunks, smem, s) : launch_prefill<8, 16, 1>(a, chunks, smem, s);
-    if (a.H <= 16) return two ? launch_prefill<16, 4, 2>(a, chunks, smem, s) : launch_prefill<16, 8, 1>(a, chunks, smem, s);
-    return launch_prefill<32, 4, 1>(a, chunks, smem, s);
+    const bool two = smem <= 108 * 1024 && dvc / 16 <= 8;             // two CTAs per SM: half the registers each
+    if (a.H <= 8) return two ? launch_prefill<8, 8, 8, 2>(a, chunks, smem, q_smem, s)
+                             : launch_prefill<8, 8, 16, 1>(a, chunks, smem, q_smem, s);
+    if (a.H <= 16) return dvc <= 64 ? launch_prefill<16, 16, 4, 1>(a, chunks, smem, q_smem, s)
+                                    : launch_prefill<16, 16, 8, 1>(a, chunks, smem, q_smem, s);
+    return launch_prefill<32, 16, 4, 1>(a, chunks, smem, q_smem, s);
   }
   return B200_ERR_UNSUPPORTED;
 }

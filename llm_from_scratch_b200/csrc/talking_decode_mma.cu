@@ -1,12 +1,13 @@
 // Talking-heads attention, bf16 tensor-core path for one query token per sequence (mathematics: talking_attention.cu).
 //
-// Bound by reading K and V once.  A CTA of four warps owns one sequence, or one of `splits` equal shares of its
+// Bound by reading K and V once.  A CTA of four or eight warps owns one sequence, or one of `splits` equal shares of its
 // visible keys, with all heads, and walks its keys in tiles of 32 through a ring of (K, V) tiles filled by cp.async:
 //
 //   QK    S^T[key, head] = K q^T per key head (the heads of a group are the N columns of mma.sync m16n8k16); soft
 //         cap and distance bias on the accumulators, fp32 scores of all heads to shared memory
-//   mix   lane = key, warp = every fourth mixed head: the H x H mix, online softmax over the tile (fp32, log2
-//         domain), bf16 weights to shared memory
+//   mix   lane = key, warp = every fourth (eighth) mixed head: the H x H mix, exponentials against a lazy reference
+//         maximum (fp32, log2 domain; it moves only when a score exceeds it by 2^kSlack), bf16 weights to shared
+//         memory; every lane keeps the sums of its own keys
 //   PV    O^T[dv, head] += V^T P^T, fp32 accumulators in registers
 //
 // With more than one share the unnormalised partials (max, sum, O) are merged in fixed order by a second kernel, so
@@ -17,17 +18,22 @@ namespace b200 {
 namespace {
 
 constexpr int BK = 32;
-constexpr int kWarps = 4;
-constexpr int kThreads = kWarps * 32;
 constexpr int kPRow = 40;             // bf16 per weight row: 32 keys + padding (odd multiple of 16 bytes)
 constexpr int kSRow = 33;
 constexpr int kMaxSplits = 32;
+constexpr float kSlack = 30.f;         // log2 of how far a score may exceed the running reference
+constexpr float kNoRef = -3.0e38f;
 constexpr float kLog2e = 1.4426950408889634f;
 
 __device__ __forceinline__ float rcp_approx(float x) {
   float y;
   asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
+}
+
+// cap tanh(x scale / cap) - bias; k = 2 log2(e) scale / cap
+__device__ __forceinline__ float capped(float x, float k, float cap, float two_cap, float bias) {
+  return (cap - bias) - two_cap * rcp_approx(1.f + fast_exp2(x * k));
 }
 
 struct DecodeParts {
@@ -41,13 +47,16 @@ __device__ __forceinline__ float gated(float o, const __nv_bfloat16* gp) {
 }
 
 // HP: heads padded; NT: column tiles of 8 heads per key head; MAXU: row tiles of 16 value columns per warp
-template <int HP, int NT, int MAXU>
-__global__ void __launch_bounds__(kThreads) talking_decode_kernel(const TalkArgs a, const DecodeParts parts) {
+// NW: warps; COMMON: soft cap and bias table present
+template <int HP, int NT, int MAXU, int NW, bool COMMON>
+__global__ void __launch_bounds__(NW * 32) talking_decode_kernel(const TalkArgs a, const DecodeParts parts) {
+  constexpr int kWarps = NW, kThreads = NW * 32, kTpr = kThreads / BK;
   extern __shared__ __align__(128) uint8_t smem[];
   __shared__ float s_talk[HP * HP];     // talk * log2(e), zero-padded
   __shared__ float s_score[HP * kSRow];
   __shared__ __align__(16) __nv_bfloat16 s_p[(HP + 8) * kPRow];   // + rows that pad the last column tile
   __shared__ float s_cor[HP + 8], s_l[HP + 8], s_m[HP + 8];
+  __shared__ int s_flag[2];             // tile parity: some head's reference moved
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
   const int H = a.H, G = a.Hkv, Gs = H / G, dk = a.dk, dv = a.dv, seq = blockIdx.y;
   const int ctx = static_cast<int>(a.ctx_lens[seq]);
@@ -62,7 +71,7 @@ __global__ void __launch_bounds__(kThreads) talking_decode_kernel(const TalkArgs
 
   auto load_tile = [&](int t) {
     const uint32_t kd = sK + (t - t0) % parts.stages * stage_bytes, vd = kd + BK * strK * 2;
-    const int r = tid >> 2, j = klo + t * BK + r;
+    const int r = tid / kTpr, j = klo + t * BK + r;
     int64_t row = -1;
     if (j < ctx) {
       const int blk = j / a.bs;
@@ -73,8 +82,8 @@ __global__ void __launch_bounds__(kThreads) talking_decode_kernel(const TalkArgs
     const int bytes = row >= 0 ? 16 : 0;
     const __nv_bfloat16* kp = static_cast<const __nv_bfloat16*>(a.kc) + (row < 0 ? 0 : row) * G * dk;
     const __nv_bfloat16* vp = static_cast<const __nv_bfloat16*>(a.vc) + (row < 0 ? 0 : row) * G * dv;
-    for (int c = tid & 3; c < G * dk / 8; c += 4) cp_async16(kd + (r * strK + c * 8) * 2, kp + c * 8, bytes);
-    for (int c = tid & 3; c < G * dv / 8; c += 4) cp_async16(vd + (r * strV + c * 8) * 2, vp + c * 8, bytes);
+    for (int c = tid % kTpr; c < G * dk / 8; c += kTpr) cp_async16(kd + (r * strK + c * 8) * 2, kp + c * 8, bytes);
+    for (int c = tid % kTpr; c < G * dv / 8; c += kTpr) cp_async16(vd + (r * strV + c * 8) * 2, vp + c * 8, bytes);
   };
   {
     const __nv_bfloat16* qp = static_cast<const __nv_bfloat16*>(a.q) + static_cast<int64_t>(seq) * a.q_stride;
@@ -98,13 +107,14 @@ __global__ void __launch_bounds__(kThreads) talking_decode_kernel(const TalkArgs
     s_cor[tid] = 1.f;
     s_l[tid] = 0.f;
   }
+  if (tid < 2) s_flag[tid] = 0;
   const float kx = a.cap > 0.f ? 2.f * kLog2e * a.scale / a.cap : 0.f;
 
   constexpr int HW = (HP + kWarps - 1) / kWarps;      // mixed heads per warp
   float m_run[HW], l_run[HW];
 #pragma unroll
   for (int i = 0; i < HW; ++i) {
-    m_run[i] = -INFINITY;
+    m_run[i] = kNoRef;
     l_run[i] = 0.f;
   }
   float o[MAXU][NT][4];
@@ -146,56 +156,83 @@ __global__ void __launch_bounds__(kThreads) talking_decode_kernel(const TalkArgs
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int hg = n * 8 + tq * 2 + (e & 1), key = mt * 16 + g + (e >> 1) * 8;
-          if (hg < Gs) {
-            const int h = c * Gs + hg, dist = max(ctx - 1 - (j0 + key), 0);
-            const float bias = a.bias_len > 0 ? __ldg(a.bias_table + h * a.bias_len + dist)
-                                              : a.r1[h] * logf(1.f + a.r2[h] * static_cast<float>(dist));
-            const float x = s[n][e];
-            s_score[h * kSRow + key] =
-                a.cap > 0.f ? (a.cap - bias) - 2.f * a.cap * rcp_approx(1.f + fast_exp2(x * kx)) : x * a.scale - bias;
-          }
+          if (hg < Gs) s_score[(c * Gs + hg) * kSRow + key] = s[n][e];
         }
+      __syncwarp();
+      // cap and bias of the unit's 16 keys x Gs heads, spread over all lanes
+      for (int i = lane; i < 16 * Gs; i += 32) {
+        const int key = mt * 16 + (i & 15), h = c * Gs + (i >> 4), dist = max(ctx - 1 - (j0 + key), 0);
+        float* sp = s_score + h * kSRow + key;
+        if constexpr (COMMON) {
+          *sp = capped(*sp, kx, a.cap, 2.f * a.cap, __ldg(a.bias_table + h * a.bias_len + dist));
+        } else {
+          const float bias = a.bias_len > 0 ? __ldg(a.bias_table + h * a.bias_len + dist)
+                                            : a.r1[h] * logf(1.f + a.r2[h] * static_cast<float>(dist));
+          *sp = a.cap > 0.f ? capped(*sp, kx, a.cap, 2.f * a.cap, bias) : *sp * a.scale - bias;
+        }
+      }
     }
     __syncthreads();
 
-    // ---- mix, online softmax ----
+    // ---- mix, weights ----
     {
-      const bool seen = j0 + lane < ctx;
+      const float base = j0 + lane < ctx ? 0.f : -INFINITY;
+      if (tid == 0) s_flag[(t + 1) & 1] = 0;      // read by the PV before this tile's first barrier
       float s[HP];
 #pragma unroll
       for (int k = 0; k < HP; ++k) s[k] = s_score[k * kSRow + lane];
+      float m[HW], top = -INFINITY;
+#pragma unroll
+      for (int i = 0; i < HW; ++i) {
+        const float* w = s_talk + (warp + i * kWarps) * HP;
+        m[i] = base;
+#pragma unroll
+        for (int k = 0; k < HP; k += 4) {
+          const float4 x = *reinterpret_cast<const float4*>(w + k);
+          m[i] = fmaf(x.x, s[k], m[i]);
+          m[i] = fmaf(x.y, s[k + 1], m[i]);
+          m[i] = fmaf(x.z, s[k + 2], m[i]);
+          m[i] = fmaf(x.w, s[k + 3], m[i]);
+        }
+        if (warp + i * kWarps < H) top = fmaxf(top, m[i] - m_run[i]);
+      }
+      if (__any_sync(0xffffffffu, top > kSlack)) {
+#pragma unroll
+        for (int i = 0; i < HW; ++i) {
+          const int h = warp + i * kWarps;
+          const float mx = warp_max(m[i]);
+          float cor = 1.f;
+          if (mx > m_run[i] + kSlack && h < H) {
+            cor = fast_exp2(m_run[i] - mx);        // no reference yet: 0
+            m_run[i] = mx;
+          }
+          l_run[i] *= cor;
+          if (lane == 0) s_cor[h] = cor;
+        }
+        if (lane == 0) s_flag[t & 1] = 1;
+      } else if (lane < HW) {
+        s_cor[warp + lane * kWarps] = 1.f;
+      }
 #pragma unroll
       for (int i = 0; i < HW; ++i) {
         const int h = warp + i * kWarps;
         if (h < H) {
-          float m = 0.f;
-#pragma unroll
-          for (int k = 0; k < HP; k += 4) {
-            const float4 w = *reinterpret_cast<const float4*>(s_talk + h * HP + k);
-            m = fmaf(w.x, s[k], m);
-            m = fmaf(w.y, s[k + 1], m);
-            m = fmaf(w.z, s[k + 2], m);
-            m = fmaf(w.w, s[k + 3], m);
-          }
-          if (!seen) m = -INFINITY;
-          const float mn = fmaxf(m_run[i], warp_max(m));      // a tile always holds a visible key
-          const __nv_bfloat16 p = __float2bfloat16_rn(fast_exp2(m - mn));
-          const float cor = fast_exp2(m_run[i] - mn);
-          l_run[i] = l_run[i] * cor + warp_sum(__bfloat162float(p));
-          m_run[i] = mn;
+          const __nv_bfloat16 p = __float2bfloat16_rn(fast_exp2(m[i] - m_run[i]));
+          l_run[i] += __bfloat162float(p);
           s_p[h * kPRow + lane] = p;
-          if (lane == 0) s_cor[h] = cor;
         }
       }
     }
     __syncthreads();
 
     // ---- PV ----
+    const bool rescale = s_flag[t & 1] != 0;
 #pragma unroll
     for (int u = 0; u < MAXU; ++u) {
       const int unit = warp + u * kWarps;
       if (unit < units) {
         const int c = unit / mt_per_head, mt = unit - c * mt_per_head;
+        if (rescale)
 #pragma unroll
         for (int n = 0; n < NT; ++n) {
           const int h = min(c * Gs + n * 8 + tq * 2, HP);       // rows past the heads are padding
@@ -227,8 +264,9 @@ __global__ void __launch_bounds__(kThreads) talking_decode_kernel(const TalkArgs
 #pragma unroll
   for (int i = 0; i < HW; ++i) {
     const int h = warp + i * kWarps;
+    const float l = warp_sum(l_run[i]);
     if (h < H && lane == 0) {
-      s_l[h] = l_run[i];
+      s_l[h] = l;
       s_m[h] = m_run[i];
     }
   }
@@ -274,9 +312,9 @@ __global__ void __launch_bounds__(128) talking_merge_kernel(const TalkArgs a, co
   const int h = static_cast<int>(w - seq * H);
   if (a.ctx_lens[seq] <= 0) return;
   const int64_t p = (seq * n + lane) * H + h;
-  const float m = lane < n ? parts.ml[p * 2] : -INFINITY, l = lane < n ? parts.ml[p * 2 + 1] : 0.f;
+  const float m = lane < n ? parts.ml[p * 2] : kNoRef, l = lane < n ? parts.ml[p * 2 + 1] : 0.f;
   const float mx = warp_max(m);
-  const float f = m == -INFINITY ? 0.f : fast_exp2(m - mx);
+  const float f = m == kNoRef ? 0.f : fast_exp2(m - mx);
   const float inv = 1.f / warp_sum(f * l);
   for (int d0 = 0; d0 < dv; d0 += 32) {
     const int d = d0 + lane;
@@ -293,16 +331,16 @@ __global__ void __launch_bounds__(128) talking_merge_kernel(const TalkArgs a, co
 }
 
 int splits_for(int n, int window) {
-  // enough CTAs for three per SM, shares of at least 64 keys
+  // several CTAs per SM, shares of at least 128 keys
   const int sms = sm_count_cached();
-  int s = (3 * (sms > 0 ? sms : 148) + n - 1) / n;
-  if (window > 0) s = s < (window + 63) / 64 ? s : (window + 63) / 64;
+  int s = (4 * (sms > 0 ? sms : 148) + n - 1) / n;
+  if (window > 0) s = s < (window + 127) / 128 ? s : (window + 127) / 128;
   return s < 1 ? 1 : s > kMaxSplits ? kMaxSplits : s;
 }
 
-template <int HP, int NT, int MAXU>
-int launch_decode(const TalkArgs& a, const DecodeParts& parts, size_t smem, cudaStream_t s) {
-  auto kern = talking_decode_kernel<HP, NT, MAXU>;
+template <int HP, int NT, int MAXU, int NW, bool COMMON>
+int launch_decode_as(const TalkArgs& a, const DecodeParts& parts, size_t smem, cudaStream_t s) {
+  auto kern = talking_decode_kernel<HP, NT, MAXU, NW, COMMON>;
   static size_t configured[64] = {};
   int dev = 0;
   cudaGetDevice(&dev);
@@ -311,16 +349,28 @@ int launch_decode(const TalkArgs& a, const DecodeParts& parts, size_t smem, cuda
       return B200_ERR_LAUNCH;
     if (dev >= 0 && dev < 64) configured[dev] = smem;
   }
-  kern<<<dim3(parts.splits, static_cast<unsigned>(a.rows)), kThreads, smem, s>>>(a, parts);
+  kern<<<dim3(parts.splits, static_cast<unsigned>(a.rows)), NW * 32, smem, s>>>(a, parts);
   int rc = launch_result();
   if (rc != B200_OK || parts.splits == 1) return rc;
   talking_merge_kernel<<<static_cast<unsigned>((a.rows * a.H + 3) / 4), 128, 0, s>>>(a, parts);
   return launch_result();
 }
 
+template <int HP, int NT, int MAXU>
+int launch_decode(const TalkArgs& a, const DecodeParts& parts, size_t smem, cudaStream_t s) {
+  const bool common = a.cap > 0.f && a.window > 0 && a.bias_len >= a.window;
+  if (smem > 76 * 1024) {        // fewer than three CTAs fit an SM: eight warps each
+    constexpr int U = MAXU > 2 ? MAXU / 2 : 1;
+    return common ? launch_decode_as<HP, NT, U, 8, true>(a, parts, smem, s)
+                  : launch_decode_as<HP, NT, U, 8, false>(a, parts, smem, s);
+  }
+  return common ? launch_decode_as<HP, NT, MAXU, 4, true>(a, parts, smem, s)
+                : launch_decode_as<HP, NT, MAXU, 4, false>(a, parts, smem, s);
+}
+
 template <int HP>
 int dispatch_decode(const TalkArgs& a, const DecodeParts& parts, size_t smem, cudaStream_t s) {
-  const int nt = (a.H / a.Hkv + 7) / 8, u = (a.Hkv * a.dv / 16 + kWarps - 1) / kWarps;
+  const int nt = (a.H / a.Hkv + 7) / 8, u = (a.Hkv * a.dv / 16 + 3) / 4;    // row tiles per warp of four
   if (nt == 1) {
     if (u <= 4) return launch_decode<HP, 1, 4>(a, parts, smem, s);
     if (u <= 8) return launch_decode<HP, 1, 8>(a, parts, smem, s);
@@ -355,7 +405,7 @@ int talking_decode_mma_launch(const TalkArgs& a, cudaStream_t s) {
   }
   const size_t q_bytes = size_t(a.H) * (a.dk + 8) * 2;
   const size_t stage = size_t(BK) * (a.Hkv * a.dk + 8 + a.Hkv * a.dv + 8) * 2;
-  parts.stages = q_bytes + 3 * stage <= 100 * 1024 ? 3 : 2;
+  parts.stages = q_bytes + 3 * stage <= 50 * 1024 ? 3 : 2;
   const size_t smem = q_bytes + parts.stages * stage;
   if (smem > 208 * 1024) return B200_ERR_UNSUPPORTED;
   if (a.H <= 8) return dispatch_decode<8>(a, parts, smem, s);
