@@ -209,6 +209,7 @@ struct ScanArgs {
   float* seg_state;          // [segments, H, dk, dv]  pass 1: P, after pass 2: entry state
   float* seg_decay;          // [segments, H, dk]      pass 1: D
   int n, seg_len;
+  bool async;                // 16-byte copies are possible
 };
 
 using f32x2 = unsigned long long;
@@ -287,6 +288,9 @@ __global__ void __launch_bounds__(512, 1) recurrence_scan_kernel(const RecArgs a
   float* sq = sk + kBlockTokens * DK;              // outputs only
   float* sv = sq + (LOCAL ? 0 : kBlockTokens * DK);
   float* so = sv + 2 * kBlockTokens * dv;          // [kBlockTokens, dv], outputs only
+  // rows of the projection as they are, two blocks: [2][kBlockTokens][f | (q) | v]
+  T* raw = reinterpret_cast<T*>(so + (LOCAL ? 0 : kBlockTokens * dv));
+  const int at_q = dk, at_v = LOCAL ? dk : 2 * dk, raw_row = at_v + dv;
   const int tid = threadIdx.x, threads = blockDim.x, rg = tid & (kRowGroups - 1), c0 = (tid / kRowGroups) * C;
   const bool cols = c0 < dv;                       // dv is a multiple of 4: a float4 is in or out as a whole
 
@@ -314,19 +318,47 @@ __global__ void __launch_bounds__(512, 1) recurrence_scan_kernel(const RecArgs a
     }
   }
 
+  auto fetch = [&](int b) {                        // block b of the segment -> raw
+    const int nb = min(kBlockTokens, ntok - b);
+    T* dst = raw + ((b / kBlockTokens) & 1) * kBlockTokens * raw_row;
+    const int64_t tok = info.tok0 + tok_lo + b;
+    constexpr int E = 16 / sizeof(T);
+    const int w = sc.async ? E : 1, ck = dk / w, cv = dv / w, per = (LOCAL ? ck : 2 * ck) + cv;
+    for (int i = tid; i < nb * per; i += threads) {
+      const int t = i / per, c = i - t * per;
+      const int64_t off = (tok + t) * a.stride;
+      const T* src;
+      int to;
+      if (c < ck) {
+        src = static_cast<const T*>(a.f) + off + head * dk + c * w;
+        to = c * w;
+      } else if (!LOCAL && c < 2 * ck) {
+        src = static_cast<const T*>(a.q) + off + head * dk + (c - ck) * w;
+        to = at_q + (c - ck) * w;
+      } else {
+        const int cc = c - (LOCAL ? ck : 2 * ck);
+        src = static_cast<const T*>(a.v) + off + head * dv + cc * w;
+        to = at_v + cc * w;
+      }
+      if (sc.async) cp_async16(smem_u32(dst + t * raw_row + to), src, 16);
+      else dst[t * raw_row + to] = *src;
+    }
+    cp_async_commit();
+  };
+  fetch(0);
   for (int b = 0; b < ntok; b += kBlockTokens) {
     const int nb = min(kBlockTokens, ntok - b);
     const int64_t tok = info.tok0 + tok_lo + b;
+    cp_async_wait<0>();
     __syncthreads();
+    const T* rp = raw + ((b / kBlockTokens) & 1) * kBlockTokens * raw_row;
+    if (b + kBlockTokens < ntok) fetch(b + kBlockTokens);
     for (int i = tid; i < nb * DK; i += threads) {
       const int t = i / DK, d = i % DK;
       float f = 1.f, k = 0.f, q = 0.f;
       if (d < dk) {
-        const int64_t off = (tok + t) * a.stride + head * dk + d;
-        gates(to_float<T>(static_cast<const T*>(a.f)[off]) + a.f_bias[head * dk + d], a.lower[head * dk + d], &f, &k);
-        if (!LOCAL) {
-          q = silu_f(to_float<T>(static_cast<const T*>(a.q)[off]));
-        }
+        gates(to_float<T>(rp[t * raw_row + d]) + __ldg(a.f_bias + head * dk + d), __ldg(a.lower + head * dk + d), &f, &k);
+        if (!LOCAL) q = silu_f(to_float<T>(rp[t * raw_row + at_q + d]));
       }
       sf[i] = f;
       sk[i] = k;
@@ -334,7 +366,7 @@ __global__ void __launch_bounds__(512, 1) recurrence_scan_kernel(const RecArgs a
     }
     for (int i = tid; i < nb * dv; i += threads) {
       const int t = i / dv, d = i - t * dv;
-      const float x = to_float<T>(static_cast<const T*>(a.v)[(tok + t) * a.stride + head * dv + d]);
+      const float x = to_float<T>(rp[t * raw_row + at_v + d]);
       *reinterpret_cast<float2*>(sv + 2 * i) = make_float2(x, x);       // both halves of a packed operand
     }
     __syncthreads();
@@ -492,7 +524,8 @@ int launch_scan(const RecArgs& a, const ScanArgs& sc, int64_t segments, bool cha
   auto local = recurrence_scan_kernel<T, R, C, true>;
   auto full = recurrence_scan_kernel<T, R, C, false>;
   const size_t one = size_t(kBlockTokens) * R * kRowGroups * sizeof(float), v = size_t(kBlockTokens) * a.dv * sizeof(float);
-  const size_t smem_local = 2 * one + 2 * v, smem_full = 3 * one + 3 * v;
+  const size_t smem_local = 2 * one + 2 * v + 2 * kBlockTokens * size_t(a.dk + a.dv) * sizeof(T);
+  const size_t smem_full = 3 * one + 3 * v + 2 * kBlockTokens * size_t(2 * a.dk + a.dv) * sizeof(T);
   if (smem_full > 40 * 1024 &&
       (cudaFuncSetAttribute(local, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem_local)) != cudaSuccess ||
        cudaFuncSetAttribute(full, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem_full)) != cudaSuccess))
@@ -550,6 +583,9 @@ extern "C" int b200_gated_recurrence(const void* q, const void* f, const void* v
     ScanArgs sc{};
     sc.n = num_seqs;
     sc.seg_len = scan_seg_len(total_tokens, num_heads);
+    const int64_t es = dtype == B200_DTYPE_F32 ? 4 : 2;
+    sc.async = dim_k * es % 16 == 0 && dim_v * es % 16 == 0 && token_stride * es % 16 == 0 && aligned16(q) &&
+               aligned16(f) && aligned16(v);
     const int64_t segments = total_tokens / sc.seg_len + num_seqs;
     const bool chained = max_seqlen_q > sc.seg_len;
     if (chained) {

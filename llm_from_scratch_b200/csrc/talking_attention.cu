@@ -185,6 +185,9 @@ extern "C" int b200_talking_attention(const void* q, int64_t q_stride, const voi
   a.bt = block_tables;
   a.bt_stride = bt_stride;
   a.bs = block_size;
+  a.bs_log2 = -1;
+  for (int i = 0; i < 31; ++i)
+    if (block_size == 1 << i) a.bs_log2 = i;
   a.num_blocks = num_blocks;
   a.cu_q = cu_seqlens_q;
   a.cu_k = cu_seqlens_k;

@@ -15,7 +15,7 @@ struct TalkArgs {
   void* out;                 // [rows, H, dv]
   const int32_t* bt;         // [n, bt_stride]
   int64_t bt_stride;
-  int bs;
+  int bs, bs_log2;           // bs_log2: -1 if bs is no power of two
   int64_t num_blocks;
   const int32_t* cu_q;       // [n + 1], or null: row i is the last token of sequence i
   const int32_t* cu_k;

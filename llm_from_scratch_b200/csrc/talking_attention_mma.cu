@@ -45,9 +45,9 @@ __device__ __forceinline__ float capped(float x, float k, float cap, float two_c
   return (cap - bias) - two_cap * rcp_approx(1.f + fast_exp2(x * k));
 }
 
-// HP: heads padded; NW: warps; MAXC: value columns per CTA in units of 16; COMMON: soft cap and bias table present;
-// q_smem: the query rows are staged in shared memory (else their fragments are read from global memory)
-template <int HP, int NW, int MAXC, int MINB, bool COMMON>
+// HP: heads padded; NW: warps; MAXC: value columns per CTA in units of 16; MODE: 0 any constants, 1 soft cap and bias table
+// present, 2 also H == HP; q_smem: the query rows are staged in shared memory (else their fragments are read from global memory)
+template <int HP, int NW, int MAXC, int MINB, int MODE>
 __global__ void __launch_bounds__(NW * 32, MINB)
 talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp, const int q_smem) {
   constexpr int HPW = HP / NW, kThreads = NW * 32, kTpr = kThreads / BK;    // kTpr: threads that load one key row
@@ -56,7 +56,7 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
   __shared__ float s_cor[BQ * HP];     // factor of this tile for accumulators and sums
   __shared__ int s_flag, s_seq, s_tile;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
-  const int H = a.H, G = a.Hkv, Gs = H / G, dk = a.dk;
+  const int H = MODE == 2 ? HP : a.H, G = a.Hkv, Gs = H / G, dk = a.dk;
   const int dvc = a.dv / gridDim.y, dv0 = blockIdx.y * dvc, nc = dvc / 16;
 
   // ---- which (sequence, tile): tiles are numbered sequence by sequence ----
@@ -105,13 +105,13 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
 
   // ---- loads ----
   auto pool_row = [&](int j) -> int64_t {
-    const int blk = j / a.bs;
+    const int blk = a.bs_log2 >= 0 ? j >> a.bs_log2 : j / a.bs;
     const int id = blk < a.bt_stride ? __ldg(a.bt + static_cast<int64_t>(seq) * a.bt_stride + blk) : -1;
     if (id < 0 || id >= a.num_blocks) {
       report(a.status, B200_ERR_BOUNDS);
       return -1;
     }
-    return static_cast<int64_t>(id) * a.bs + j % a.bs;
+    return static_cast<int64_t>(id) * a.bs + (j - blk * a.bs);
   };
   auto load_rows = [&](int t, const void* cache, int d, int d0, int width, uint32_t dst, int stride) {
     // 32 rows x G heads x width columns (from column d0 of d) of the pool
@@ -155,6 +155,15 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
 #pragma unroll
     for (int c = 0; c < 2 * MAXC; ++c) o[hh][c][0] = o[hh][c][1] = o[hh][c][2] = o[hh][c][3] = 0.f;
   }
+  // shared-memory addresses of this warp's fragments; kv: the key head of each of its heads
+  const int ar = (lane & 7) + ((lane >> 3) & 1) * 8, ac = lane >> 4;
+  const int br = (lane & 7) + (lane >> 4) * 8, bc = (lane >> 3) & 1;
+  int kv[HPW];
+#pragma unroll
+  for (int hh = 0; hh < HPW; ++hh) kv[hh] = min(warp * HPW + hh, H - 1) / Gs;
+  const uint32_t adQ = sQ + ((warp * HPW * BQ + ar) * strQ + ac * 8) * 2, stepQ = BQ * strQ * 2;     // per head
+  const uint32_t adK = sK + (br * strK + bc * 8) * 2, adV = sV + (ar * strV + ac * 8) * 2;
+  const uint32_t adP = sS + (warp * HPW * BQ + ar) * kSRow * 4 + ac * 16;
   const float kx = a.cap > 0.f ? 2.f * kLog2e * a.scale / a.cap : 0.f;
   const float cap = a.cap, two_cap = 2.f * a.cap;
   cp_async_wait<1>();
@@ -163,8 +172,6 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
   for (int t = 0; t < ntiles; ++t) {
     // ---- QK ----
     {
-      const int ar = (lane & 7) + ((lane >> 3) & 1) * 8, ac = lane >> 4;
-      const int br = (lane & 7) + (lane >> 4) * 8, bc = (lane >> 3) & 1;
 #pragma unroll
       for (int h0 = 0; h0 < HPW; h0 += 2) {            // two heads at a time share the key fragments of their group
         constexpr int HS = HPW < 2 ? 1 : 2;
@@ -175,21 +182,21 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
           for (int n = 0; n < 4; ++n) s[hh][n][0] = s[hh][n][1] = s[hh][n][2] = s[hh][n][3] = 0.f;
         const int hbase = warp * HPW + h0;
         if (hbase < H) {
+#pragma unroll 4
           for (int ks = 0; ks < dk / 16; ++ks) {
             uint32_t b0[4], b1[4];
-            int cur = -1;
 #pragma unroll
             for (int hh = 0; hh < HS; ++hh) {
               const int h = hbase + hh;
               if (h < H) {
-                if (h / Gs != cur) {
-                  cur = h / Gs;
-                  ldmatrix_x4(b0, sK + (br * strK + cur * dk + (2 * ks + bc) * 8) * 2);
-                  ldmatrix_x4(b1, sK + ((br + 16) * strK + cur * dk + (2 * ks + bc) * 8) * 2);
+                if (hh == 0 || kv[h0 + hh] != kv[h0]) {
+                  const uint32_t at = adK + kv[h0 + hh] * dk * 2 + ks * 32;
+                  ldmatrix_x4(b0, at);
+                  ldmatrix_x4(b1, at + 32 * strK);
                 }
                 uint32_t af[4];
                 if (q_smem) {
-                  ldmatrix_x4(af, sQ + ((h * BQ + ar) * strQ + (2 * ks + ac) * 8) * 2);
+                  ldmatrix_x4(af, adQ + (h0 + hh) * stepQ + ks * 32);
                 } else {             // rows past the portion repeat its last row: their scores are never used
                   const __nv_bfloat16* q0p = qrow + static_cast<int64_t>(min(g, rows - 1)) * a.q_stride + h * dk + ks * 16 + tq * 2;
                   const __nv_bfloat16* q1p = qrow + static_cast<int64_t>(min(g + 8, rows - 1)) * a.q_stride + h * dk + ks * 16 + tq * 2;
@@ -241,11 +248,12 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
       for (int h = 0; h < HP; ++h) s[h] = h < H ? Sr[h * BQ * kSRow] : 0.f;
 #pragma unroll
       for (int h = 0; h < HP; ++h) {
-        if constexpr (COMMON) {
-          const float bias = __ldg(table + min(h, H - 1) * a.bias_len);
+        if constexpr (MODE > 0) {
+          const float bias = __ldg(table);
+          if (h + 1 < H) table += a.bias_len;
           s[h] = capped(s[h], kx, cap, two_cap, bias);    // a padding head is finite and meets zeros of the mix
         } else {
-          const float bias = a.bias_len > 0 ? __ldg(table + min(h, H - 1) * a.bias_len)
+          const float bias = a.bias_len > 0 ? __ldg(a.bias_table + min(h, H - 1) * a.bias_len + dc)
                                             : mp.r1[h] * logf(1.f + mp.r2[h] * static_cast<float>(dc));
           s[h] = cap > 0.f ? capped(s[h], kx, cap, two_cap, bias) : s[h] * a.scale - bias;
         }
@@ -295,7 +303,6 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
 
     // ---- PV ----
     {
-      const int ar = (lane & 7) + ((lane >> 3) & 1) * 8, ac = lane >> 4;
       uint32_t pf[HPW][2][4];
       const bool rescale = s_flag != 0;
 #pragma unroll
@@ -316,7 +323,7 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
           }
 #pragma unroll
           for (int kk = 0; kk < 2; ++kk) {
-            ldmatrix_x4(pf[hh][kk], sS + ((h * BQ + ar) * kSRow) * 4 + (2 * kk + ac) * 16);
+            ldmatrix_x4(pf[hh][kk], adP + hh * (BQ * kSRow * 4) + kk * 32);
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
               const float2 p = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&pf[hh][kk][e]));
@@ -331,15 +338,12 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
         for (int c = 0; c < MAXC; ++c) {
           if (c < nc) {
             uint32_t bf[4];
-            int cur = -1;
 #pragma unroll
             for (int hh = 0; hh < HPW; ++hh) {
               const int h = warp * HPW + hh;
               if (h < H) {
-                if (h / Gs != cur) {
-                  cur = h / Gs;
-                  ldmatrix_x4_trans(bf, sV + ((kk * 16 + ar) * strV + cur * dvc + (2 * c + ac) * 8) * 2);
-                }
+                if (hh == 0 || kv[hh] != kv[hh - 1])
+                  ldmatrix_x4_trans(bf, adV + kv[hh] * dvc * 2 + kk * 32 * strV + c * 32);
                 const uint32_t b0[2] = {bf[0], bf[1]}, b1[2] = {bf[2], bf[3]};
                 mma_bf16_16816(o[hh][2 * c], pf[hh][kk], b0);
                 mma_bf16_16816(o[hh][2 * c + 1], pf[hh][kk], b1);
@@ -389,7 +393,7 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
   }
 }
 
-template <int HP, int NW, int MAXC, int MINB, bool COMMON>
+template <int HP, int NW, int MAXC, int MINB, int MODE>
 int launch_prefill(const TalkArgs& a, int chunks, size_t smem, bool q_smem, cudaStream_t s) {
   MixParam<HP> mp;
   memset(&mp, 0, sizeof(mp));
@@ -399,7 +403,7 @@ int launch_prefill(const TalkArgs& a, int chunks, size_t smem, bool q_smem, cuda
     mp.r1[h] = a.r1_host[h];
     mp.r2[h] = a.r2_host[h];
   }
-  auto kern = talking_prefill_kernel<HP, NW, MAXC, MINB, COMMON>;
+  auto kern = talking_prefill_kernel<HP, NW, MAXC, MINB, MODE>;
   static size_t configured[64] = {};
   int dev = 0;
   cudaGetDevice(&dev);
@@ -416,8 +420,9 @@ int launch_prefill(const TalkArgs& a, int chunks, size_t smem, bool q_smem, cuda
 template <int HP, int NW, int MAXC, int MINB>
 int launch_prefill(const TalkArgs& a, int chunks, size_t smem, bool q_smem, cudaStream_t s) {
   if (a.cap > 0.f && a.window > 0 && a.bias_len >= a.window)
-    return launch_prefill<HP, NW, MAXC, MINB, true>(a, chunks, smem, q_smem, s);
-  return launch_prefill<HP, NW, MAXC, MINB, false>(a, chunks, smem, q_smem, s);
+    return a.H == HP ? launch_prefill<HP, NW, MAXC, MINB, 2>(a, chunks, smem, q_smem, s)
+                     : launch_prefill<HP, NW, MAXC, MINB, 1>(a, chunks, smem, q_smem, s);
+  return launch_prefill<HP, NW, MAXC, MINB, 0>(a, chunks, smem, q_smem, s);
 }
 
 }  // namespace

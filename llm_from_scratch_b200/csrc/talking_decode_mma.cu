@@ -74,10 +74,10 @@ __global__ void __launch_bounds__(NW * 32) talking_decode_kernel(const TalkArgs 
     const int r = tid / kTpr, j = klo + t * BK + r;
     int64_t row = -1;
     if (j < ctx) {
-      const int blk = j / a.bs;
+      const int blk = a.bs_log2 >= 0 ? j >> a.bs_log2 : j / a.bs;
       const int id = blk < a.bt_stride ? __ldg(a.bt + static_cast<int64_t>(seq) * a.bt_stride + blk) : -1;
       if (id < 0 || id >= a.num_blocks) report(a.status, B200_ERR_BOUNDS);
-      else row = static_cast<int64_t>(id) * a.bs + j % a.bs;
+      else row = static_cast<int64_t>(id) * a.bs + (j - blk * a.bs);
     }
     const int bytes = row >= 0 ? 16 : 0;
     const __nv_bfloat16* kp = static_cast<const __nv_bfloat16*>(a.kc) + (row < 0 ? 0 : row) * G * dk;
@@ -123,6 +123,7 @@ __global__ void __launch_bounds__(NW * 32) talking_decode_kernel(const TalkArgs 
 #pragma unroll
     for (int n = 0; n < NT; ++n) o[u][n][0] = o[u][n][1] = o[u][n][2] = o[u][n][3] = 0.f;
   const int mt_per_head = dv / 16, units = G * mt_per_head;
+  const int inv_mt = 65535 / mt_per_head + 1;         // unit / mt_per_head as a multiplication (units < 2^12)
 
   for (int t = t0; t < t1; ++t) {
     if (parts.stages == 3) cp_async_wait<1>();
@@ -231,7 +232,7 @@ __global__ void __launch_bounds__(NW * 32) talking_decode_kernel(const TalkArgs 
     for (int u = 0; u < MAXU; ++u) {
       const int unit = warp + u * kWarps;
       if (unit < units) {
-        const int c = unit / mt_per_head, mt = unit - c * mt_per_head;
+        const int c = (unit * inv_mt) >> 16;
         if (rescale)
 #pragma unroll
         for (int n = 0; n < NT; ++n) {
@@ -247,7 +248,7 @@ __global__ void __launch_bounds__(NW * 32) talking_decode_kernel(const TalkArgs 
           // A = V^T: 16 value columns x 16 keys from rows of keys (transposing load)
           uint32_t af[4];
           const int kr = kk * 16 + (lane & 7) + (lane >> 4) * 8, vc = ((lane >> 3) & 1) * 8;
-          ldmatrix_x4_trans(af, vt + (kr * strV + c * dv + mt * 16 + vc) * 2);
+          ldmatrix_x4_trans(af, vt + (kr * strV + unit * 16 + vc) * 2);
 #pragma unroll
           for (int n = 0; n < NT; ++n) {
             uint32_t bf[2];

@@ -11,7 +11,25 @@ import numpy as np
 import torch
 
 from . import ops
-from .microbench import _time
+
+
+def _time(fn, steps: int, warmup: int) -> float:
+    """Milliseconds per call of ``fn``, ``steps`` calls replayed from one CUDA graph (no host work in between)."""
+    for _ in range(max(warmup, 1)):
+        fn()
+    torch.cuda.synchronize()
+    graph = torch.cuda.CUDAGraph()
+    with torch.cuda.graph(graph):
+        for _ in range(steps):
+            fn()
+    graph.replay()
+    torch.cuda.synchronize()
+    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    e0.record()
+    graph.replay()
+    e1.record()
+    torch.cuda.synchronize()
+    return e0.elapsed_time(e1) / steps
 
 # (width, heads, kv heads, head size, recurrence heads x size, d_ff, window)
 SIZES = {
