@@ -9,8 +9,8 @@
 //        scores of the same row
 //   PV   warp w again holds its heads: O += P V, fp32 accumulators in registers; row sums from the same fragments
 //
-// The three phases are separated by CTA barriers; K of the next tile arrives (cp.async) during mix and PV, V during
-// QK and mix.  Scores are fp32 from the accumulator to the exponential.  The running maximum is lazy: a row keeps
+// A tile takes two barrier intervals: its mix, then its PV together with the next tile's QK (two score buffers).
+// K of the tile after next and V of the next one arrive (cp.async) during the mix.  Scores are fp32 from the accumulator to the exponential.  The running maximum is lazy: a row keeps
 // the reference maximum of an earlier tile until a score exceeds it by 2^kSlack, so the ordinary tile needs no
 // reduction over lanes; the exact maximum only has to keep the exponentials in range.
 #include <string.h>
@@ -22,7 +22,8 @@ namespace {
 
 constexpr int BQ = 16;
 constexpr int BK = 32;
-constexpr int kSRow = 40;            // floats per score row: 32 keys + padding against bank conflicts
+constexpr int kSRow = 36;            // floats per score row: 32 keys + padding (odd multiple of 16 bytes)
+constexpr int kQueryInSmem = 1, kTwoScores = 2;
 constexpr float kSlack = 30.f;       // log2 of how far a score may exceed the row's reference
 
 constexpr float kNoRef = -3.0e38f;   // reference of a row that has seen no key
@@ -49,12 +50,13 @@ __device__ __forceinline__ float capped(float x, float k, float cap, float two_c
 // present, 2 also H == HP; q_smem: the query rows are staged in shared memory (else their fragments are read from global memory)
 template <int HP, int NW, int MAXC, int MINB, int MODE>
 __global__ void __launch_bounds__(NW * 32, MINB)
-talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp, const int q_smem) {
+talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp, const int layout) {
   constexpr int HPW = HP / NW, kThreads = NW * 32, kTpr = kThreads / BK;    // kTpr: threads that load one key row
+  const bool q_smem = layout & kQueryInSmem, two_scores = layout & kTwoScores;
   extern __shared__ __align__(128) uint8_t smem[];
   __shared__ __align__(16) float s_ref[BQ * HP];     // reference maximum (log2 domain) per (row, head)
-  __shared__ float s_cor[BQ * HP];     // factor of this tile for accumulators and sums
-  __shared__ int s_flag, s_seq, s_tile;
+  __shared__ float s_cor[2][BQ * HP];  // by tile parity: factor for accumulators and sums, 1 unless the flag is set
+  __shared__ int s_flag[2], s_seq, s_tile;       // flag (by tile parity): some reference moved
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
   const int H = MODE == 2 ? HP : a.H, G = a.Hkv, Gs = H / G, dk = a.dk;
   const int dvc = a.dv / gridDim.y, dv0 = blockIdx.y * dvc, nc = dvc / 16;
@@ -75,7 +77,8 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
       if (hit) {
         const int src = __ffs(hit) - 1;
         seq = base + src;
-        tile = left - __shfl_sync(0xffffffffu, incl - t, src);
+        // last tile of the sequence first: it sees the most keys
+        tile = __shfl_sync(0xffffffffu, incl, src) - 1 - left;
       } else {
         left -= __shfl_sync(0xffffffffu, incl, 31);
       }
@@ -99,9 +102,10 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
   const int strQ = dk + 8, strK = G * dk + 8, strV = G * dvc + 8;      // elements; odd multiples of 16 bytes
   const uint32_t sQ = smem_u32(smem);
   const uint32_t sS = sQ + (q_smem ? H * BQ * strQ * 2 : 0);
-  const uint32_t sK = sS + H * BQ * kSRow * 4;
+  const uint32_t s_bytes = H * BQ * kSRow * 4;         // one of two score buffers
+  const uint32_t sK = sS + (two_scores ? 2 : 1) * s_bytes;
   const uint32_t sV = sK + BK * strK * 2;
-  float* S = reinterpret_cast<float*>(smem + (sS - sQ));
+  float* S0 = reinterpret_cast<float*>(smem + (sS - sQ));
 
   // ---- loads ----
   auto pool_row = [&](int j) -> int64_t {
@@ -144,9 +148,9 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
   cp_async_commit();
   for (int i = tid; i < HP * BQ; i += kThreads) {
     s_ref[i] = i % HP < H ? kNoRef : INFINITY;
-    s_cor[i] = 1.f;
+    s_cor[0][i] = s_cor[1][i] = 1.f;
   }
-  if (tid == 0) s_flag = 0;
+  if (tid < 2) s_flag[tid] = 0;
 
   float o[HPW][2 * MAXC][4], l[HPW][2];
 #pragma unroll
@@ -169,9 +173,8 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
   cp_async_wait<1>();
   __syncthreads();
 
-  for (int t = 0; t < ntiles; ++t) {
-    // ---- QK ----
-    {
+  // scores of the K tile in shared memory -> S
+  auto qk = [&](float* S) {
 #pragma unroll
       for (int h0 = 0; h0 < HPW; h0 += 2) {            // two heads at a time share the key fragments of their group
         constexpr int HS = HPW < 2 ? 1 : 2;
@@ -228,13 +231,17 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
           }
         }
       }
-      for (int i = tid; i < HP * BQ; i += kThreads) s_cor[i] = 1.f;
-      if (tid == 0) s_flag = 0;
-    }
-    __syncthreads();
-    if (t + 1 < ntiles) load_rows(t + 1, a.kc, dk, 0, dk, sK, strK);
-    cp_async_commit();
+  };
+  qk(S0);
+  cp_async_wait<0>();
+  __syncthreads();
+  if (ntiles > 1) load_rows(1, a.kc, dk, 0, dk, sK, strK);
+  cp_async_commit();
 
+  bool dirty = false;
+  for (int t = 0; t < ntiles; ++t) {
+    const int buf = two_scores ? t & 1 : 0;
+    float* S = S0 + buf * (H * BQ * kSRow);
     // ---- mix ----
 #pragma unroll 1
     for (int r = warp; r < rows; r += NW) {
@@ -284,8 +291,8 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
               const float ref = s_ref[r * HP + hb + i];
               if (mx > ref + kSlack) {
                 s_ref[r * HP + hb + i] = mx;
-                s_cor[r * HP + hb + i] = fast_exp2(ref - mx);
-                s_flag = 1;
+                s_cor[t & 1][r * HP + hb + i] = fast_exp2(ref - mx);
+                s_flag[t & 1] = 1;
               }
             }
           }
@@ -298,19 +305,25 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
           if (hb + i < H) Pr[(hb + i) * BQ * kSRow * 2] = __float2bfloat16_rn(fast_exp2(m[i] - ref[i]));
       }
     }
-    cp_async_wait<1>();
+    cp_async_wait<0>();
     __syncthreads();
 
-    // ---- PV ----
+    // ---- PV of this tile, QK of the next ----
     {
+      const uint32_t pt = adP + buf * s_bytes;
+      const bool rescale = s_flag[t & 1] != 0;
+      // the other parity's flag and factors were last read one tile ago: ready them for the next one
+      if (tid == 0) s_flag[(t + 1) & 1] = 0;
+      if (dirty)
+        for (int i = tid; i < HP * BQ; i += kThreads) s_cor[(t + 1) & 1][i] = 1.f;
+      dirty = rescale;
       uint32_t pf[HPW][2][4];
-      const bool rescale = s_flag != 0;
 #pragma unroll
       for (int hh = 0; hh < HPW; ++hh) {
         const int h = warp * HPW + hh;
         if (h < H) {
           if (rescale) {
-            const float c0 = s_cor[g * HP + h], c1 = s_cor[(g + 8) * HP + h];
+            const float c0 = s_cor[t & 1][g * HP + h], c1 = s_cor[t & 1][(g + 8) * HP + h];
             l[hh][0] *= c0;
             l[hh][1] *= c1;
 #pragma unroll
@@ -323,7 +336,7 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
           }
 #pragma unroll
           for (int kk = 0; kk < 2; ++kk) {
-            ldmatrix_x4(pf[hh][kk], adP + hh * (BQ * kSRow * 4) + kk * 32);
+            ldmatrix_x4(pf[hh][kk], pt + hh * (BQ * kSRow * 4) + kk * 32);
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
               const float2 p = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&pf[hh][kk][e]));
@@ -353,12 +366,13 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
         }
       }
     }
-    cp_async_wait<0>();
+    if (!two_scores) __syncthreads();        // the weights are read, their buffer takes the next scores
+    if (t + 1 < ntiles) qk(S0 + (two_scores ? (t + 1) & 1 : 0) * (H * BQ * kSRow));
     __syncthreads();
     if (t + 1 < ntiles) load_rows(t + 1, a.vc, a.dv, dv0, dvc, sV, strV);
+    if (t + 2 < ntiles) load_rows(t + 2, a.kc, dk, 0, dk, sK, strK);
     cp_async_commit();
   }
-  cp_async_wait<0>();
 
   // ---- normalise, gate, store ----
 #pragma unroll
@@ -394,7 +408,7 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
 }
 
 template <int HP, int NW, int MAXC, int MINB, int MODE>
-int launch_prefill(const TalkArgs& a, int chunks, size_t smem, bool q_smem, cudaStream_t s) {
+int launch_prefill(const TalkArgs& a, int chunks, size_t smem, int layout, cudaStream_t s) {
   MixParam<HP> mp;
   memset(&mp, 0, sizeof(mp));
   for (int h = 0; h < a.H; ++h)
@@ -413,16 +427,16 @@ int launch_prefill(const TalkArgs& a, int chunks, size_t smem, bool q_smem, cuda
     if (dev >= 0 && dev < 64) configured[dev] = smem;
   }
   const int64_t tiles = a.rows / BQ + a.n;          // sum over sequences of ceil(q_len / 16) is at most this
-  kern<<<dim3(static_cast<unsigned>(tiles), chunks), NW * 32, smem, s>>>(a, mp, q_smem ? 1 : 0);
+  kern<<<dim3(static_cast<unsigned>(tiles), chunks), NW * 32, smem, s>>>(a, mp, layout);
   return launch_result();
 }
 
 template <int HP, int NW, int MAXC, int MINB>
-int launch_prefill(const TalkArgs& a, int chunks, size_t smem, bool q_smem, cudaStream_t s) {
+int launch_prefill(const TalkArgs& a, int chunks, size_t smem, int layout, cudaStream_t s) {
   if (a.cap > 0.f && a.window > 0 && a.bias_len >= a.window)
-    return a.H == HP ? launch_prefill<HP, NW, MAXC, MINB, 2>(a, chunks, smem, q_smem, s)
-                     : launch_prefill<HP, NW, MAXC, MINB, 1>(a, chunks, smem, q_smem, s);
-  return launch_prefill<HP, NW, MAXC, MINB, 0>(a, chunks, smem, q_smem, s);
+    return a.H == HP ? launch_prefill<HP, NW, MAXC, MINB, 2>(a, chunks, smem, layout, s)
+                     : launch_prefill<HP, NW, MAXC, MINB, 1>(a, chunks, smem, layout, s);
+  return launch_prefill<HP, NW, MAXC, MINB, 0>(a, chunks, smem, layout, s);
 }
 
 }  // namespace
@@ -440,17 +454,24 @@ int talking_prefill_mma_launch(const TalkArgs& a, cudaStream_t s) {
     const int dvc = a.dv / chunks;
     if (dvc / 16 > max_c) continue;
     const size_t q_bytes = size_t(a.H) * BQ * (a.dk + 8) * 2;
-    size_t smem = size_t(a.H) * BQ * kSRow * 4 + size_t(BK) * (a.Hkv * a.dk + 8) * 2 +
-                  size_t(BK) * (a.Hkv * dvc + 8) * 2;
-    const bool q_smem = smem + q_bytes <= 220 * 1024;
-    if (q_smem) smem += q_bytes;
-    if (smem > 220 * 1024) continue;
+    const size_t s_bytes = size_t(a.H) * BQ * kSRow * 4;
+    const size_t kv = size_t(BK) * (a.Hkv * a.dk + 8) * 2 + size_t(BK) * (a.Hkv * dvc + 8) * 2;
+    size_t smem = 0;
+    int layout = -1;
+    for (int l : {kQueryInSmem | kTwoScores, +kTwoScores, +kQueryInSmem, 0}) {
+      smem = kv + (l & kTwoScores ? 2 : 1) * s_bytes + (l & kQueryInSmem ? q_bytes : 0);
+      if (smem <= 220 * 1024) {
+        layout = l;
+        break;
+      }
+    }
+    if (layout < 0) continue;
     const bool two = smem <= 108 * 1024 && dvc / 16 <= 8;             // two CTAs per SM: half the registers each
-    if (a.H <= 8) return two ? launch_prefill<8, 8, 8, 2>(a, chunks, smem, q_smem, s)
-                             : launch_prefill<8, 8, 16, 1>(a, chunks, smem, q_smem, s);
-    if (a.H <= 16) return dvc <= 64 ? launch_prefill<16, 16, 4, 1>(a, chunks, smem, q_smem, s)
-                                    : launch_prefill<16, 16, 8, 1>(a, chunks, smem, q_smem, s);
-    return launch_prefill<32, 16, 4, 1>(a, chunks, smem, q_smem, s);
+    if (a.H <= 8) return two ? launch_prefill<8, 8, 8, 2>(a, chunks, smem, layout, s)
+                             : launch_prefill<8, 8, 16, 1>(a, chunks, smem, layout, s);
+    if (a.H <= 16) return dvc <= 64 ? launch_prefill<16, 16, 4, 1>(a, chunks, smem, layout, s)
+                                    : launch_prefill<16, 16, 8, 1>(a, chunks, smem, layout, s);
+    return launch_prefill<32, 16, 4, 1>(a, chunks, smem, layout, s);
   }
   return B200_ERR_UNSUPPORTED;
 }

@@ -69,7 +69,8 @@ __global__ void __launch_bounds__(NW * 32) talking_decode_kernel(const TalkArgs 
   const uint32_t sQ = smem_u32(smem), sK = sQ + H * strQ * 2;
   const uint32_t stage_bytes = BK * (strK + strV) * 2;
 
-  auto load_tile = [&](int t) {
+  // which: 1 keys, 2 values, 3 both
+  auto load_tile = [&](int t, int which) {
     const uint32_t kd = sK + (t - t0) % parts.stages * stage_bytes, vd = kd + BK * strK * 2;
     const int r = tid / kTpr, j = klo + t * BK + r;
     int64_t row = -1;
@@ -82,8 +83,10 @@ __global__ void __launch_bounds__(NW * 32) talking_decode_kernel(const TalkArgs 
     const int bytes = row >= 0 ? 16 : 0;
     const __nv_bfloat16* kp = static_cast<const __nv_bfloat16*>(a.kc) + (row < 0 ? 0 : row) * G * dk;
     const __nv_bfloat16* vp = static_cast<const __nv_bfloat16*>(a.vc) + (row < 0 ? 0 : row) * G * dv;
-    for (int c = tid % kTpr; c < G * dk / 8; c += kTpr) cp_async16(kd + (r * strK + c * 8) * 2, kp + c * 8, bytes);
-    for (int c = tid % kTpr; c < G * dv / 8; c += kTpr) cp_async16(vd + (r * strV + c * 8) * 2, vp + c * 8, bytes);
+    if (which & 1)
+      for (int c = tid % kTpr; c < G * dk / 8; c += kTpr) cp_async16(kd + (r * strK + c * 8) * 2, kp + c * 8, bytes);
+    if (which & 2)
+      for (int c = tid % kTpr; c < G * dv / 8; c += kTpr) cp_async16(vd + (r * strV + c * 8) * 2, vp + c * 8, bytes);
   };
   {
     const __nv_bfloat16* qp = static_cast<const __nv_bfloat16*>(a.q) + static_cast<int64_t>(seq) * a.q_stride;
@@ -93,8 +96,16 @@ __global__ void __launch_bounds__(NW * 32) talking_decode_kernel(const TalkArgs 
       cp_async16(sQ + (h * strQ + c * 8) * 2, qp + h * dk + c * 8, 16);
     }
   }
+  // one stage: the next keys arrive during mix and PV, the next values during QK and mix
+  const bool single = parts.stages == 1;
+  if (single) {
+    if (t0 < t1) load_tile(t0, 1);
+    cp_async_commit();
+    if (t0 < t1) load_tile(t0, 2);
+    cp_async_commit();
+  }
   for (int i = 0; i < parts.stages - 1; ++i) {
-    if (t0 + i < t1) load_tile(t0 + i);
+    if (t0 + i < t1) load_tile(t0 + i, 3);
     cp_async_commit();
   }
   for (int i = tid; i < HP * HP; i += kThreads) {
@@ -126,11 +137,13 @@ __global__ void __launch_bounds__(NW * 32) talking_decode_kernel(const TalkArgs 
   const int inv_mt = 65535 / mt_per_head + 1;         // unit / mt_per_head as a multiplication (units < 2^12)
 
   for (int t = t0; t < t1; ++t) {
-    if (parts.stages == 3) cp_async_wait<1>();
-    else cp_async_wait<0>();
+    if (parts.stages == 2) cp_async_wait<0>();
+    else cp_async_wait<1>();
     __syncthreads();
-    if (t + parts.stages - 1 < t1) load_tile(t + parts.stages - 1);
-    cp_async_commit();
+    if (!single) {
+      if (t + parts.stages - 1 < t1) load_tile(t + parts.stages - 1, 3);
+      cp_async_commit();
+    }
     const uint32_t kt = sK + (t - t0) % parts.stages * stage_bytes, vt = kt + BK * strK * 2;
     const int j0 = klo + t * BK;
 
@@ -174,6 +187,10 @@ __global__ void __launch_bounds__(NW * 32) talking_decode_kernel(const TalkArgs 
       }
     }
     __syncthreads();
+    if (single) {
+      if (t + 1 < t1) load_tile(t + 1, 1);
+      cp_async_commit();
+    }
 
     // ---- mix, weights ----
     {
@@ -224,6 +241,7 @@ __global__ void __launch_bounds__(NW * 32) talking_decode_kernel(const TalkArgs 
         }
       }
     }
+    if (single) cp_async_wait<1>();
     __syncthreads();
 
     // ---- PV ----
@@ -259,9 +277,13 @@ __global__ void __launch_bounds__(NW * 32) talking_decode_kernel(const TalkArgs 
         }
       }
     }
+    if (single) {
+      __syncthreads();
+      if (t + 1 < t1) load_tile(t + 1, 2);
+      cp_async_commit();
+    }
   }
   cp_async_wait<0>();
-
 #pragma unroll
   for (int i = 0; i < HW; ++i) {
     const int h = warp + i * kWarps;
@@ -361,7 +383,7 @@ template <int HP, int NT, int MAXU>
 int launch_decode(const TalkArgs& a, const DecodeParts& parts, size_t smem, cudaStream_t s) {
   const bool common = a.cap > 0.f && a.window > 0 && a.bias_len >= a.window;
   if (smem > 76 * 1024) {        // fewer than three CTAs fit an SM: eight warps each
-    constexpr int U = MAXU > 2 ? MAXU / 2 : 1;
+    constexpr int U = MAXU / 2;
     return common ? launch_decode_as<HP, NT, U, 8, true>(a, parts, smem, s)
                   : launch_decode_as<HP, NT, U, 8, false>(a, parts, smem, s);
   }
@@ -407,6 +429,7 @@ int talking_decode_mma_launch(const TalkArgs& a, cudaStream_t s) {
   const size_t q_bytes = size_t(a.H) * (a.dk + 8) * 2;
   const size_t stage = size_t(BK) * (a.Hkv * a.dk + 8 + a.Hkv * a.dv + 8) * 2;
   parts.stages = q_bytes + 3 * stage <= 50 * 1024 ? 3 : 2;
+  if (q_bytes + 2 * stage > 208 * 1024) parts.stages = 1;
   const size_t smem = q_bytes + parts.stages * stage;
   if (smem > 208 * 1024) return B200_ERR_UNSUPPORTED;
   if (a.H <= 8) return dispatch_decode<8>(a, parts, smem, s);
