@@ -35,17 +35,29 @@ def reference(cfg, w, ids):
     return orc.forward(cfg, w, ids)
 
 
-def marked_keys(cfg, w, strength=14.0):
-    """Weights under which a query that repeats token 7 finds the key of the token before... of token 7 alone: one
-    channel of the embedding marks token 7, and the first key / query channel of every head reads that channel,
-    so the score between two marked tokens stands out by far (up to the soft cap)."""
+MARK, SEEK = 7, 8      # the token that marked_keys marks, and the token that looks for it
+
+
+def marked_keys(cfg, w, strength=12.0):
+    """The same weights, but every head's first key channel reads only an embedding channel that is large for token
+    MARK alone, and every head's first query channel one that is large for token SEEK alone: the score of a SEEK
+    query at a MARK key stands out by far, so that whether the query sees the key decides its logits."""
     w = {k: v.clone() for k, v in w.items()}
-    w["embed"][:, 0] = 0
-    w["embed"][7, 0] = 8.0
+    w["embed"][:, :2] = 0
+    w["embed"][MARK, 0] = w["embed"][SEEK, 1] = 8.0
     for i, lay in enumerate(cfg["layers"]):
         c = lay["mixer"]["left"]
-        for name, heads in (("q", c["heads"]), ("k", c["kv_heads"])):
+        for name, heads, channel in (("q", c["heads"], 1), ("k", c["kv_heads"], 0)):
             m = w[f"l{i}.mix.left.{name}"]
-            m[:, 0] = 0
-            m[torch.arange(heads) * c["dim"], 0] = strength ** 0.5
+            first = torch.arange(heads) * c["dim"]
+            m[first] = 0
+            m[first, channel] = strength
+        for name in ("norm1", "ls1", "ls2"):      # the marking channels stay clean
+            if f"l{i}.{name}" in w:
+                w[f"l{i}.{name}"][:2] = 0.0
     return w
+
+
+def plain_tokens(cfg, n, seed):
+    """Tokens without MARK and SEEK."""
+    return [t if t not in (MARK, SEEK) else SEEK + 1 for t in tokens(cfg, n, seed)]
