@@ -218,8 +218,93 @@ __global__ void __launch_bounds__(512) stream_update_kernel(const StreamArgs a) 
   }
 }
 
+// The same boundary when a row is one Pack of four channels per thread (d / 4 threads): every load of the row is
+// issued before the first reduction and nothing is read twice.
+template <typename T, int SC>
+__global__ void __launch_bounds__(1024, 1) stream_update_row_kernel(const StreamArgs a) {
+  constexpr int V = 4;
+  __shared__ float2 scratch[2][32];
+  const int d = a.d, i = threadIdx.x * V, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+  const int64_t row = blockIdx.x;
+  float* xr = a.x + row * SC * d + i;
+  auto sum2 = [&](float p, float q, int use) {           // CTA sums of two values; `use` picks the scratch row
+    p = warp_sum(p);
+    q = warp_sum(q);
+    if (lane == 0) scratch[use][warp] = make_float2(p, q);
+    __syncthreads();
+    float2 t = lane < warps ? scratch[use][lane] : make_float2(0.f, 0.f);
+    return make_float2(warp_sum(t.x), warp_sum(t.y));
+  };
+  Pack<V> x[SC];
+#pragma unroll
+  for (int s = 0; s < SC; ++s) x[s] = load_f<V>(xr + static_cast<int64_t>(s) * d);
+  Pack<V> y = load_t<T, V>(static_cast<const T*>(a.y0) + row * d + i);
+  const Pack<V> nw = load_f<V>(a.norm_w + i);
+  Pack<V> ls;
+#pragma unroll
+  for (int k = 0; k < V; ++k) ls.v[k] = 1.f;
+  if (a.scale != nullptr) ls = load_f<V>(a.scale + i);
+  if (a.y1 != nullptr) {
+    const Pack<V> y1 = load_t<T, V>(static_cast<const T*>(a.y1) + row * d + i);
+    const Pack<V> g0 = load_f<V>(a.w0 + i), g1 = load_f<V>(a.w1 + i);
+    float s0 = 0.f, s1 = 0.f;
+#pragma unroll
+    for (int k = 0; k < V; ++k) {
+      s0 += y.v[k] * y.v[k];
+      s1 += y1.v[k] * y1.v[k];
+    }
+    const float2 t = sum2(s0, s1, 0);
+    const float n0 = 0.5f * rsqrtf(t.x / static_cast<float>(d) + a.join_eps);
+    const float n1 = 0.5f * rsqrtf(t.y / static_cast<float>(d) + a.join_eps);
+#pragma unroll
+    for (int k = 0; k < V; ++k) y.v[k] = y.v[k] * n0 * g0.v[k] + y1.v[k] * n1 * g1.v[k];
+  }
+  Pack<V> u;
+#pragma unroll
+  for (int k = 0; k < V; ++k) {
+    y.v[k] *= ls.v[k];
+    u.v[k] = 0.f;
+  }
+#pragma unroll
+  for (int t = 0; t < SC; ++t) {
+    const float wo = __ldg(a.out + t), wi = a.in ? __ldg(a.in + t) : 1.f;
+    Pack<V> z;
+#pragma unroll
+    for (int k = 0; k < V; ++k) z.v[k] = wo * y.v[k];
+#pragma unroll
+    for (int s = 0; s < SC; ++s) {
+      const float m = __ldg(a.mix + s * SC + t);
+#pragma unroll
+      for (int k = 0; k < V; ++k) z.v[k] += m * x[s].v[k];
+    }
+#pragma unroll
+    for (int k = 0; k < V; ++k) u.v[k] += wi * z.v[k];
+    store_f<V>(xr + static_cast<int64_t>(t) * d, z);
+  }
+  if (a.h == nullptr) return;
+  float ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < V; ++k) ss += u.v[k] * u.v[k];
+  const float inv = rsqrtf(sum2(ss, 0.f, 1).x / static_cast<float>(d) + a.eps);
+#pragma unroll
+  for (int k = 0; k < V; ++k) u.v[k] = u.v[k] * inv * (nw.v[k] + a.plus_one);
+  store_t<T, V>(static_cast<T*>(a.h) + row * d + i, u);
+}
+
+template <typename T>
+int launch_stream_rows(const StreamArgs& a, int64_t rows, cudaStream_t s) {
+  auto kern = stream_update_row_kernel<T, 1>;
+  if (a.S == 2) kern = stream_update_row_kernel<T, 2>;
+  if (a.S == 3) kern = stream_update_row_kernel<T, 3>;
+  if (a.S == 4) kern = stream_update_row_kernel<T, 4>;
+  kern<<<static_cast<unsigned>(rows), a.d / 4, 0, s>>>(a);
+  return launch_result();
+}
+
 template <typename T, int V>
 int launch_streams(const StreamArgs& a, int64_t rows, cudaStream_t s) {
+  if (V == 4 && a.S <= 4 && a.y0 != nullptr && a.norm_w != nullptr && a.d % 128 == 0 && a.d <= 4096)
+    return launch_stream_rows<T>(a, rows, s);
   const size_t smem = static_cast<size_t>(a.d) * sizeof(float);
   int threads = (a.d / V + 31) / 32 * 32;
   threads = threads < 64 ? 64 : threads > 512 ? 512 : threads;

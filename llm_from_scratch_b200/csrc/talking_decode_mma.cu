@@ -54,8 +54,8 @@ __global__ void __launch_bounds__(NW * 32) talking_decode_kernel(const TalkArgs 
   extern __shared__ __align__(128) uint8_t smem[];
   __shared__ float s_talk[HP * HP];     // talk * log2(e), zero-padded
   __shared__ float s_score[HP * kSRow];
-  __shared__ __align__(16) __nv_bfloat16 s_p[(HP + 8) * kPRow];   // + rows that pad the last column tile
-  __shared__ float s_cor[HP + 8], s_l[HP + 8], s_m[HP + 8];
+  __shared__ __align__(16) __nv_bfloat16 s_p[(HP + 8 * NT) * kPRow];   // + rows that pad the last column tile
+  __shared__ float s_cor[HP + 8 * NT], s_l[HP], s_m[HP];
   __shared__ int s_flag[2];             // tile parity: some head's reference moved
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
   const int H = a.H, G = a.Hkv, Gs = H / G, dk = a.dk, dv = a.dv, seq = blockIdx.y;
@@ -66,7 +66,7 @@ __global__ void __launch_bounds__(NW * 32) talking_decode_kernel(const TalkArgs 
   const int t0 = blockIdx.x * per, t1 = min(tiles, t0 + per);
 
   const int strQ = dk + 8, strK = G * dk + 8, strV = G * dv + 8;
-  const uint32_t sQ = smem_u32(smem), sK = sQ + H * strQ * 2;
+  const uint32_t sQ = smem_u32(smem), sK = sQ + (H + 8 * NT) * strQ * 2;      // rows past the heads are padding
   const uint32_t stage_bytes = BK * (strK + strV) * 2;
 
   // which: 1 keys, 2 values, 3 both
@@ -113,11 +113,8 @@ __global__ void __launch_bounds__(NW * 32) talking_decode_kernel(const TalkArgs 
     s_talk[i] = h < H && k < H ? a.talk[h * H + k] * kLog2e : 0.f;
   }
   for (int i = tid; i < HP * kSRow; i += kThreads) s_score[i] = 0.f;
-  for (int i = tid; i < (HP + 8) * kPRow; i += kThreads) s_p[i] = __float2bfloat16_rn(0.f);
-  if (tid < HP + 8) {
-    s_cor[tid] = 1.f;
-    s_l[tid] = 0.f;
-  }
+  for (int i = tid; i < (HP + 8 * NT) * kPRow; i += kThreads) s_p[i] = __float2bfloat16_rn(0.f);
+  if (tid < HP + 8 * NT) s_cor[tid] = 1.f;
   if (tid < 2) s_flag[tid] = 0;
   const float kx = a.cap > 0.f ? 2.f * kLog2e * a.scale / a.cap : 0.f;
 
@@ -134,7 +131,19 @@ __global__ void __launch_bounds__(NW * 32) talking_decode_kernel(const TalkArgs 
 #pragma unroll
     for (int n = 0; n < NT; ++n) o[u][n][0] = o[u][n][1] = o[u][n][2] = o[u][n][3] = 0.f;
   const int mt_per_head = dv / 16, units = G * mt_per_head;
-  const int inv_mt = 65535 / mt_per_head + 1;         // unit / mt_per_head as a multiplication (units < 2^12)
+  // per row tile of this warp: byte offset of its value columns in a V row tile, of its heads' weights, first head
+  uint32_t offV[MAXU], offP[MAXU];
+  int head0[MAXU];
+  {
+    const int kr = (lane & 7) + (lane >> 4) * 8, vc = ((lane >> 3) & 1) * 8;
+#pragma unroll
+    for (int u = 0; u < MAXU; ++u) {
+      const int unit = warp + u * kWarps, c = unit / mt_per_head;
+      offV[u] = (kr * strV + unit * 16 + vc) * 2;
+      head0[u] = c * Gs;
+      offP[u] = smem_u32(s_p) + ((c * Gs + (lane & 7)) * kPRow + ((lane >> 3) & 1) * 8) * 2;
+    }
+  }
 
   for (int t = t0; t < t1; ++t) {
     if (parts.stages == 2) cp_async_wait<0>();
@@ -153,15 +162,16 @@ __global__ void __launch_bounds__(NW * 32) talking_decode_kernel(const TalkArgs 
       float s[NT][4];
 #pragma unroll
       for (int n = 0; n < NT; ++n) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
+      const uint32_t qa = sQ + ((c * Gs + (lane & 7)) * strQ + ((lane >> 3) & 1) * 8) * 2;
       const uint32_t ka = kt + ((mt * 16 + (lane & 15)) * strK + c * dk + (lane >> 4) * 8) * 2;
+#pragma unroll 4
       for (int ks = 0; ks < dk / 16; ++ks) {
         uint32_t af[4];
         ldmatrix_x4(af, ka + ks * 32);
 #pragma unroll
         for (int n = 0; n < NT; ++n) {
           uint32_t bf[2];
-          const int h = min(c * Gs + n * 8 + (lane & 7), H - 1);
-          ldmatrix_x2(bf, sQ + (h * strQ + ks * 16 + ((lane >> 3) & 1) * 8) * 2);
+          ldmatrix_x2(bf, qa + n * 16 * strQ + ks * 32);
           mma_bf16_16816(s[n], af, bf);
         }
       }
@@ -250,28 +260,24 @@ __global__ void __launch_bounds__(NW * 32) talking_decode_kernel(const TalkArgs 
     for (int u = 0; u < MAXU; ++u) {
       const int unit = warp + u * kWarps;
       if (unit < units) {
-        const int c = (unit * inv_mt) >> 16;
         if (rescale)
 #pragma unroll
-        for (int n = 0; n < NT; ++n) {
-          const int h = min(c * Gs + n * 8 + tq * 2, HP);       // rows past the heads are padding
-          const float c0 = s_cor[h], c1 = s_cor[h + 1];
-          o[u][n][0] *= c0;
-          o[u][n][1] *= c1;
-          o[u][n][2] *= c0;
-          o[u][n][3] *= c1;
-        }
+          for (int n = 0; n < NT; ++n) {
+            const float c0 = s_cor[head0[u] + n * 8 + tq * 2], c1 = s_cor[head0[u] + n * 8 + tq * 2 + 1];
+            o[u][n][0] *= c0;
+            o[u][n][1] *= c1;
+            o[u][n][2] *= c0;
+            o[u][n][3] *= c1;
+          }
 #pragma unroll
         for (int kk = 0; kk < 2; ++kk) {
           // A = V^T: 16 value columns x 16 keys from rows of keys (transposing load)
           uint32_t af[4];
-          const int kr = kk * 16 + (lane & 7) + (lane >> 4) * 8, vc = ((lane >> 3) & 1) * 8;
-          ldmatrix_x4_trans(af, vt + (kr * strV + unit * 16 + vc) * 2);
+          ldmatrix_x4_trans(af, vt + offV[u] + kk * 32 * strV);
 #pragma unroll
           for (int n = 0; n < NT; ++n) {
             uint32_t bf[2];
-            const int h = min(c * Gs + n * 8 + (lane & 7), HP + 7);
-            ldmatrix_x2(bf, smem_u32(s_p) + (h * kPRow + kk * 16 + ((lane >> 3) & 1) * 8) * 2);
+            ldmatrix_x2(bf, offP[u] + n * (8 * kPRow * 2) + kk * 32);
             mma_bf16_16816(o[u][n], af, bf);
           }
         }
@@ -402,7 +408,7 @@ int dispatch_decode(const TalkArgs& a, const DecodeParts& parts, size_t smem, cu
   } else if (nt == 2 && HP >= 16) {
     if (u <= 8) return launch_decode<HP, HP >= 16 ? 2 : 1, 8>(a, parts, smem, s);
     if (u <= 16) return launch_decode<HP, HP >= 16 ? 2 : 1, 16>(a, parts, smem, s);
-  } else if (nt <= 4 && HP >= 32) {
+  } else if (nt == 4 && HP >= 32) {
     if (u <= 8) return launch_decode<HP, HP >= 32 ? 4 : 1, 8>(a, parts, smem, s);
   }
   return B200_ERR_UNSUPPORTED;
@@ -426,7 +432,7 @@ int talking_decode_mma_launch(const TalkArgs& a, cudaStream_t s) {
     parts.ml = static_cast<float*>(a.workspace);
     parts.o = parts.ml + static_cast<size_t>(a.rows) * parts.splits * a.H * 2;
   }
-  const size_t q_bytes = size_t(a.H) * (a.dk + 8) * 2;
+  const size_t q_bytes = size_t(a.H + (a.H / a.Hkv + 7) / 8 * 8) * (a.dk + 8) * 2;
   const size_t stage = size_t(BK) * (a.Hkv * a.dk + 8 + a.Hkv * a.dv + 8) * 2;
   parts.stages = q_bytes + 3 * stage <= 50 * 1024 ? 3 : 2;
   if (q_bytes + 2 * stage > 208 * 1024) parts.stages = 1;
