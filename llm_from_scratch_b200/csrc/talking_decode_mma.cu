@@ -49,7 +49,8 @@ __device__ __forceinline__ float gated(float o, const __nv_bfloat16* gp) {
 // HP: heads padded; NT: column tiles of 8 heads per key head; MAXU: row tiles of 16 value columns per warp
 // NW: warps; COMMON: soft cap and bias table present
 template <int HP, int NT, int MAXU, int NW, bool COMMON>
-__global__ void __launch_bounds__(NW * 32) talking_decode_kernel(const TalkArgs a, const DecodeParts parts) {
+__global__ void __launch_bounds__(NW * 32, NW == 8 ? (NT * MAXU <= 4 ? 3 : NT * MAXU <= 8 ? 2 : 1) : 1)
+talking_decode_kernel(const TalkArgs a, const DecodeParts parts) {
   constexpr int kWarps = NW, kThreads = NW * 32, kTpr = kThreads / BK;
   extern __shared__ __align__(128) uint8_t smem[];
   __shared__ float s_talk[HP * HP];     // talk * log2(e), zero-padded
@@ -159,6 +160,19 @@ __global__ void __launch_bounds__(NW * 32) talking_decode_kernel(const TalkArgs 
     // ---- QK, cap, bias ----
     for (int u = warp; u < 2 * G; u += kWarps) {
       const int mt = u & 1, c = u >> 1;
+      // biases of the unit's 16 keys x Gs heads, requested ahead of the products
+      constexpr int NB = 4 * NT;
+      float bias[NB];
+#pragma unroll
+      for (int b = 0; b < NB; ++b) {
+        const int i = lane + b * 32;
+        bias[b] = 0.f;
+        if (i < 16 * Gs) {
+          const int h = c * Gs + (i >> 4), dist = max(ctx - 1 - (j0 + mt * 16 + (i & 15)), 0);
+          if (COMMON || a.bias_len > 0) bias[b] = __ldg(a.bias_table + h * a.bias_len + dist);
+          else bias[b] = a.r1[h] * logf(1.f + a.r2[h] * static_cast<float>(dist));
+        }
+      }
       float s[NT][4];
 #pragma unroll
       for (int n = 0; n < NT; ++n) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
@@ -184,15 +198,12 @@ __global__ void __launch_bounds__(NW * 32) talking_decode_kernel(const TalkArgs 
         }
       __syncwarp();
       // cap and bias of the unit's 16 keys x Gs heads, spread over all lanes
-      for (int i = lane; i < 16 * Gs; i += 32) {
-        const int key = mt * 16 + (i & 15), h = c * Gs + (i >> 4), dist = max(ctx - 1 - (j0 + key), 0);
-        float* sp = s_score + h * kSRow + key;
-        if constexpr (COMMON) {
-          *sp = capped(*sp, kx, a.cap, 2.f * a.cap, __ldg(a.bias_table + h * a.bias_len + dist));
-        } else {
-          const float bias = a.bias_len > 0 ? __ldg(a.bias_table + h * a.bias_len + dist)
-                                            : a.r1[h] * logf(1.f + a.r2[h] * static_cast<float>(dist));
-          *sp = a.cap > 0.f ? capped(*sp, kx, a.cap, 2.f * a.cap, bias) : *sp * a.scale - bias;
+#pragma unroll
+      for (int b = 0; b < NB; ++b) {
+        const int i = lane + b * 32;
+        if (i < 16 * Gs) {
+          float* sp = s_score + (c * Gs + (i >> 4)) * kSRow + mt * 16 + (i & 15);
+          *sp = COMMON || a.cap > 0.f ? capped(*sp, kx, a.cap, 2.f * a.cap, bias[b]) : *sp * a.scale - bias[b];
         }
       }
     }
@@ -388,7 +399,7 @@ int launch_decode_as(const TalkArgs& a, const DecodeParts& parts, size_t smem, c
 template <int HP, int NT, int MAXU>
 int launch_decode(const TalkArgs& a, const DecodeParts& parts, size_t smem, cudaStream_t s) {
   const bool common = a.cap > 0.f && a.window > 0 && a.bias_len >= a.window;
-  if (smem > 76 * 1024) {        // fewer than three CTAs fit an SM: eight warps each
+  if (HP >= 16 || smem > 76 * 1024) {
     constexpr int U = MAXU / 2;
     return common ? launch_decode_as<HP, NT, U, 8, true>(a, parts, smem, s)
                   : launch_decode_as<HP, NT, U, 8, false>(a, parts, smem, s);
@@ -435,7 +446,7 @@ int talking_decode_mma_launch(const TalkArgs& a, cudaStream_t s) {
   const size_t q_bytes = size_t(a.H + (a.H / a.Hkv + 7) / 8 * 8) * (a.dk + 8) * 2;
   const size_t stage = size_t(BK) * (a.Hkv * a.dk + 8 + a.Hkv * a.dv + 8) * 2;
   parts.stages = q_bytes + 3 * stage <= 50 * 1024 ? 3 : 2;
-  if (q_bytes + 2 * stage > 208 * 1024) parts.stages = 1;
+  if (q_bytes + 2 * stage > 76 * 1024) parts.stages = 1;      // other CTAs of the SM hide the loads
   const size_t smem = q_bytes + parts.stages * stage;
   if (smem > 208 * 1024) return B200_ERR_UNSUPPORTED;
   if (a.H <= 8) return dispatch_decode<8>(a, parts, smem, s);
