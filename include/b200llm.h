@@ -513,7 +513,9 @@ int b200_clamped_glu(const void* h, void* act, int64_t rows, int32_t d_ff, float
  * Rows beyond the last sequence are padding.  max_seqlen_q: host bound on rows per sequence.
  * r1, r2 [num_heads] and talk [num_heads, num_heads] fp32 (device); bias_table [num_heads, bias_len] fp32
  * or NULL: r1 ln(1 + r2 distance) for distances 0 .. bias_len - 1, bias_len >= window if given; consts_host: talk,
- * r1, r2 one after the other on the host (NULL: the general kernel runs).  Workspace: b200_talking_attention_workspace_bytes(). */
+ * r1, r2 one after the other on the host (NULL: the general kernel runs).  plan: tile list of b200_prefill_plan for
+ * B200_TALKING_TILE_ROWS rows per tile, or NULL.  Workspace: b200_talking_attention_workspace_bytes(). */
+#define B200_TALKING_TILE_ROWS 16
 size_t b200_talking_attention_workspace_bytes(int32_t num_seqs, int32_t num_heads, int32_t dim_v, int32_t window,
                                               int32_t decode, int32_t dtype);
 int b200_talking_attention(const void* q, int64_t q_stride, const void* gate, int64_t gate_stride, const void* k_cache,
@@ -523,7 +525,8 @@ int b200_talking_attention(const void* q, int64_t q_stride, const void* gate, in
                            int32_t max_seqlen_q, int32_t num_heads, int32_t num_kv_heads, int32_t dim_k, int32_t dim_v,
                            float scale, float softcap, const float* r1, const float* r2, const float* talk,
                            const float* consts_host, const float* bias_table, int32_t bias_len, int32_t window,
-                           void* workspace, size_t workspace_bytes, int32_t dtype, int32_t* status, void* stream);
+                           const int32_t* plan, int32_t plan_tile_rows, int32_t plan_capacity, void* workspace,
+                           size_t workspace_bytes, int32_t dtype, int32_t* status, void* stream);
 
 /* Gated linear recurrence (HGRN2) over per-sequence states: per head
  *   q = silu(q_in), f = lower + (1 - lower) sigmoid(f_in + f_bias), S <- diag(f) S + (1 - f) v^T, o = S^T q,

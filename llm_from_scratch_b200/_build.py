@@ -46,7 +46,7 @@ def _stale(target: Path, deps: list[Path]) -> bool:
 # Sources a model family runs on, where that is not the whole library: ``ensure`` builds a library of just these
 # when the full one is absent.  "api" and "host_path" are the parts every engine uses.
 FAMILY_SOURCES = {
-    "Nabalix": ("api", "host_path", "decode_advance", "sampler", "moe_gemm", "moe_gemm_rows", "store_kvcache", "streams",
+    "Nabalix": ("api", "host_path", "decode_advance", "sampler", "moe_gemm", "moe_gemm_rows", "store_kvcache", "prefill_plan", "streams",
                 "talking_attention", "talking_attention_mma", "talking_decode_mma", "gated_recurrence"),
 }
 

@@ -76,7 +76,7 @@ SIGNATURES = {
     "b200_talking_attention_workspace_bytes": (_sz, [_i32, _i32, _i32, _i32, _i32, _i32]),
     "b200_talking_attention": (_i32, [_vp, _i64, _vp, _i64, _vp, _vp, _vp, _vp, _i64, _i32, _i64, _vp, _vp, _vp, _i32,
                                       _i64, _i32, _i32, _i32, _i32, _i32, _f32, _f32, _vp, _vp, _vp, _vp, _vp, _i32,
-                                      _i32, _vp, _sz, _i32, _vp, _vp]),
+                                      _i32, _vp, _i32, _i32, _vp, _sz, _i32, _vp, _vp]),
     "b200_gated_recurrence_workspace_bytes": (_sz, [_i32, _i64, _i32, _i32, _i32, _i32]),
     "b200_gated_recurrence": (_i32, [_vp, _vp, _vp, _i64, _vp, _vp, _vp, _f32, _vp, _i64, _vp, _vp, _vp, _vp, _i32,
                                      _i64, _i32, _i32, _i32, _i32, _vp, _vp, _sz, _i32, _vp, _vp]),

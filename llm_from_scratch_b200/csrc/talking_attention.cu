@@ -163,7 +163,8 @@ extern "C" int b200_talking_attention(const void* q, int64_t q_stride, const voi
                                       int32_t num_heads, int32_t num_kv_heads, int32_t dim_k, int32_t dim_v,
                                       float scale, float softcap, const float* r1, const float* r2, const float* talk,
                                       const float* consts_host, const float* bias_table, int32_t bias_len,
-                                      int32_t window, void* workspace, size_t workspace_bytes, int32_t dtype,
+                                      int32_t window, const int32_t* plan, int32_t plan_tile_rows,
+                                      int32_t plan_capacity, void* workspace, size_t workspace_bytes, int32_t dtype,
                                       int32_t* status, void* stream) {
   using namespace b200;
   if (num_seqs < 0 || rows < 0 || num_heads <= 0 || num_kv_heads <= 0 || num_heads % num_kv_heads || dim_k <= 0 ||
@@ -205,6 +206,8 @@ extern "C" int b200_talking_attention(const void* q, int64_t q_stride, const voi
   a.talk = talk;
   a.window = window;
   a.max_q = max_seqlen_q;
+  a.plan = cu_seqlens_q && plan_tile_rows == kTalkTileRows && plan_capacity > 0 ? plan : nullptr;
+  a.plan_capacity = plan_capacity;
   a.talk_host = consts_host;
   a.r1_host = consts_host ? consts_host + static_cast<size_t>(num_heads) * num_heads : nullptr;
   a.r2_host = consts_host ? a.r1_host + num_heads : nullptr;

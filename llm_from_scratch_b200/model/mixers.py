@@ -87,7 +87,7 @@ class TalkingHeadsAttention(nn.Module):
         if ctx.is_prefill:
             o = ops.talking_attention(q, g, self.k_cache, self.v_cache, ctx.block_tables, self.consts,
                                       cu_seqlens_q=ctx.cu_seqlens_q, cu_seqlens_k=ctx.cu_seqlens_k,
-                                      max_seqlen_q=ctx.max_seqlen_q)
+                                      max_seqlen_q=ctx.max_seqlen_q, plan=ctx.prefill_plan)
         else:
             o = ops.talking_attention(q, g, self.k_cache, self.v_cache, ctx.block_tables, self.consts,
                                       context_lens=ctx.context_lens)

@@ -123,7 +123,7 @@ class NabalixLM(TokenHead, nn.Module):
         return [m for layer in self.layers for m in (layer.mixer.left, layer.mixer.right)]
 
     def prefill_tile_rows(self) -> int:
-        return 0
+        return ops.TALKING_TILE_ROWS if self.dtype == torch.bfloat16 else 0
 
     def forward(self, input_ids: torch.Tensor, positions: torch.Tensor | None = None) -> torch.Tensor:
         ctx, cfg = get_context(), self.cfg

@@ -794,6 +794,9 @@ def clamped_glu(h: torch.Tensor, limit: float, slope: float) -> torch.Tensor:
     return act
 
 
+TALKING_TILE_ROWS = 16              # B200_TALKING_TILE_ROWS
+
+
 class TalkingHeads:
     """Constants of a talking-heads attention layer on the device: the score scale and cap, the distance bias
     (r1, r2 [H]), the head mix ``talk`` [H, H] (out, in) and the window (0: none).  The bias of every distance
@@ -822,10 +825,11 @@ class TalkingHeads:
 def talking_attention(q: torch.Tensor, gate: torch.Tensor | None, k_cache: torch.Tensor, v_cache: torch.Tensor,
                       block_tables: torch.Tensor, c: TalkingHeads, *, cu_seqlens_q: torch.Tensor | None = None,
                       cu_seqlens_k: torch.Tensor | None = None, context_lens: torch.Tensor | None = None,
-                      max_seqlen_q: int = 1, out: torch.Tensor | None = None, general: bool = False) -> torch.Tensor:
+                      max_seqlen_q: int = 1, plan: "PrefillPlan | None" = None, out: torch.Tensor | None = None,
+                      general: bool = False) -> torch.Tensor:
     """Attention of ``b200_talking_attention`` over the paged pool: q [rows, H * dk], gate [rows, H * dv] (row
     strides free), caches [num_blocks, block_size, Hkv, d*].  Rows are ragged (``cu_seqlens_*``) or one per sequence
-    (``context_lens``).  ``general`` forces the general kernel.  Returns [rows, H, dv]."""
+    (``context_lens``); ``plan``: tile list of the step for ``TALKING_TILE_ROWS`` rows.  ``general`` forces the general kernel.  Returns [rows, H, dv]."""
     dev = _cuda(q, gate, k_cache, v_cache, block_tables, cu_seqlens_q, cu_seqlens_k, context_lens, out)
     rows, H = q.shape[0], c.H
     nb, bs, Hkv, dk = k_cache.shape
@@ -858,7 +862,9 @@ def talking_attention(q: torch.Tensor, gate: torch.Tensor | None, k_cache: torch
         v_cache.data_ptr(), out.data_ptr(), block_tables.data_ptr(), block_tables.stride(0), bs, nb, _ptr(cu_seqlens_q),
         _ptr(cu_seqlens_k), _ptr(context_lens), n, rows, int(max_seqlen_q), H, Hkv, dk, dv, c.scale, c.softcap,
         c.r1.data_ptr(), c.r2.data_ptr(), c.talk.data_ptr(), None if general else c.consts_host.data_ptr(), _ptr(c.table),
-        c.table.shape[1] if c.table is not None else 0, c.window, _ptr(ws), ws.numel() if ws is not None else 0, _dt(q),
+        c.table.shape[1] if c.table is not None else 0, c.window,
+        plan.buffer.data_ptr() if plan is not None else None, plan.tile_rows if plan is not None else 0,
+        plan.capacity if plan is not None else 0, _ptr(ws), ws.numel() if ws is not None else 0, _dt(q),
         status_word(dev).data_ptr(), _stream()), "talking_attention")
     return out
 

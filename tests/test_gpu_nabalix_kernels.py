@@ -133,6 +133,10 @@ def test_talking_attention(H, G, dk, dv, window, bs, dtype, general):
     ops.check_status()
     tol = 1e-5 if dtype == torch.float32 else 1.2e-2
     assert rel(got, want) < tol
+    plan = ops.prefill_plan(cu(qlens), sum(qlens) + 5, 70, ops.TALKING_TILE_ROWS)
+    again = ops.talking_attention(pad(Q), pad(gate.cuda()), kc, vc, bt, c, cu_seqlens_q=cu(qlens), cu_seqlens_k=cu(klens),
+                                  max_seqlen_q=70, plan=plan, general=general)[:sum(qlens)]
+    assert torch.equal(again, got)
     # decode form: the last row of every sequence, plus padding rows of a captured batch
     last = torch.tensor(np.cumsum(qlens) - 1)
     lens = torch.tensor(klens + [0, 0]).cuda()
