@@ -65,6 +65,8 @@ class _Staging:
 _TORCH_DTYPES = {np.dtype(np.int64).str: torch.int64, np.dtype(np.int32).str: torch.int32,
                  np.dtype(np.float32).str: torch.float32}
 
+_NUMPY_DTYPES = {torch.int64: np.int64, torch.int32: np.int32}
+
 
 class ModelRunner:
     def __init__(self, config: dict, model: EngineTransformerLM | None = None):
@@ -121,7 +123,7 @@ class ModelRunner:
             self.max_model_length = self.model_config.context_length or min(self.num_kv_blocks * self.block_size, 1 << 17)
         if not self.enforce_eager:
             self.capture_cudagraph()
-            if self.prefill_tile_rows and not self.mixed_batches and _cfg(config, "prefill_graphs", default=True):
+            if self.prefill_tile_rows and _cfg(config, "prefill_graphs", default=True):
                 self.capture_prefill_graphs()
 
     # ------------------------------------------------------------------ KV pool
@@ -346,12 +348,22 @@ class ModelRunner:
         return logits
 
     # ------------------------------------------------------------------ CUDA graphs for prefill
-    def _prefill_layout(self, tokens: int):
-        """Byte offsets of (cu_seqlens, input_ids, positions, slot_mapping) of a padded prefill batch in
-        the prefill staging buffer: one contiguous run, so a step is one host-to-device copy."""
-        n_cu = self.max_num_seqs + 1
-        o_ids = (n_cu * 4 + 15) & ~15
-        return 0, o_ids, o_ids + tokens * 8, o_ids + 2 * tokens * 8, o_ids + 3 * tokens * 8
+    def _prefill_fields(self, tokens: int):
+        """(name, dtype, shape, byte offset) of a padded prefill batch's inputs in the prefill staging buffer, and
+        its size: one contiguous run, so a step is one host-to-device copy.  Mixed batches also need context
+        lengths, state slots and — last, so that only the rows in use are copied — block tables."""
+        n = self.max_num_seqs
+        fields = [("cu_seqlens_q", torch.int32, (n + 1,)), ("input_ids", torch.int64, (tokens,)),
+                  ("positions", torch.int64, (tokens,)), ("slot_mapping", torch.int64, (tokens,))]
+        if self.mixed_batches:
+            max_blocks = (self.max_model_length + self.block_size - 1) // self.block_size
+            fields += [("cu_seqlens_k", torch.int32, (n + 1,)), ("state_slots", torch.int64, (n,)),
+                       ("block_tables", torch.int32, (n, max_blocks))]
+        out, at = [], 0
+        for name, dtype, shape in fields:
+            out.append((name, dtype, shape, at))
+            at += (int(np.prod(shape)) * dtype.itemsize + 15) & ~15
+        return out, at
 
     @torch.inference_mode()
     def capture_prefill_graphs(self) -> None:
@@ -363,8 +375,8 @@ class ModelRunner:
         buckets = list(range(mult, self.max_num_batched_tokens + 1, mult))
         if not buckets or len(buckets) > 64:
             return
-        dev, tmax, n_cu = self.device, buckets[-1], self.max_num_seqs + 1
-        total = self._prefill_layout(tmax)[-1]
+        dev, tmax = self.device, buckets[-1]
+        total = self._prefill_fields(tmax)[1]
         self.prefill_dev = torch.zeros(total, dtype=torch.uint8, device=dev)
         self.prefill_host = torch.zeros(total, dtype=torch.uint8).pin_memory()
         self.prefill_out = torch.zeros(tmax, self.model_config.d_model, dtype=self.dtype, device=dev)
@@ -372,17 +384,21 @@ class ModelRunner:
         self.prefill_plan_buffer = torch.zeros(plan_entries, dtype=torch.int32, device=dev)
         pool = self.graphs[max(self.graphs)].pool() if self.graphs else None
         for tokens in reversed(buckets):
-            o_cu, o_ids, o_pos, o_slot, _end = self._prefill_layout(tokens)
-            view = lambda off, n, dt: self.prefill_dev[off:off + n * dt.itemsize].view(dt)
-            cu = view(o_cu, n_cu, torch.int32)
-            ids, pos, slots = (view(o, tokens, torch.int64) for o in (o_ids, o_pos, o_slot))
-            slots.fill_(-1)
-            cu.zero_()
+            v = {name: self.prefill_dev[off:off + int(np.prod(shape)) * dt.itemsize].view(dt).view(*shape)
+                 for name, dt, shape, off in self._prefill_fields(tokens)[0]}
+            v["slot_mapping"].fill_(-1)
+            v["cu_seqlens_q"].zero_()
+            if self.mixed_batches:
+                v["cu_seqlens_k"].zero_()
+                v["state_slots"].fill_(-1)
+                v["block_tables"].fill_(-1)
 
             def body():
-                plan = ops.prefill_plan(cu, tokens, tokens, self.prefill_tile_rows, buffer=self.prefill_plan_buffer)
-                set_context(True, cu, cu, tokens, tokens, slots, None, None, pos, plan)
-                self.prefill_out[:tokens] = self.model(ids)
+                plan = ops.prefill_plan(v["cu_seqlens_q"], tokens, tokens, self.prefill_tile_rows,
+                                        buffer=self.prefill_plan_buffer)
+                set_context(True, v["cu_seqlens_q"], v.get("cu_seqlens_k", v["cu_seqlens_q"]), tokens, tokens,
+                            v["slot_mapping"], None, v.get("block_tables"), v["positions"], plan, v.get("state_slots"))
+                self.prefill_out[:tokens] = self.model(v["input_ids"])
 
             body()                                   # warm-up: allocates workspaces, selects GEMM algorithms
             torch.cuda.synchronize()
@@ -391,21 +407,22 @@ class ModelRunner:
                 body()
             if pool is None:
                 pool = g.pool()
-            self.prefill_graphs[tokens] = (g, cu, ids, pos, slots)
+            self.prefill_graphs[tokens] = (g, v)
             torch.cuda.synchronize()
             reset_context()
 
     @torch.inference_mode()
     def _replay_prefill(self, seqs: list[Sequence]):
         """Prefill step from a captured graph: the hidden states of the padded batch (the context is left set for
-        the head), or None when the batch does not fit one (a cached
-        prefix, which needs block tables, or more tokens / sequences than were captured)."""
-        if len(seqs) > self.max_num_seqs:
+        the head), or None when the batch does not fit one (for models without mixed batches a cached
+        prefix, which needs block tables; more tokens / sequences / blocks than were captured)."""
+        n = len(seqs)
+        if n > self.max_num_seqs:
             return None
-        m = md.prepare_prefill(seqs, self.block_size)
-        if m.block_tables is not None:
+        m = md.prepare_prefill(seqs, self.block_size, tables_always=self.mixed_batches)
+        if m.block_tables is not None and not self.mixed_batches:
             return None
-        T, n = len(m.input_ids), len(seqs)
+        T = len(m.input_ids)
         if len(m.slot_mapping) != T:
             raise RuntimeError("slot_mapping and input_ids disagree: Sequence.reference_exact must be off "
                                "when the model runs (it reproduces a reference defect at block multiples)")
@@ -414,22 +431,31 @@ class ModelRunner:
         entry = self.prefill_graphs.get(tokens)
         if entry is None:
             return None
-        g, cu, ids, pos, slots = entry
-        o_cu, o_ids, o_pos, o_slot, end = self._prefill_layout(tokens)
+        g, v = entry
+        fields, end = self._prefill_fields(tokens)
         hb = self.prefill_host.numpy()
-        h_cu = hb[o_cu:o_cu + (self.max_num_seqs + 1) * 4].view(np.int32)
-        h_ids, h_pos, h_slot = (hb[o:o + tokens * 8].view(np.int64) for o in (o_ids, o_pos, o_slot))
-        h_cu[:n + 1] = m.cu_seqlens_q
-        h_cu[n + 1:] = T
-        h_ids[:T] = m.input_ids
-        h_ids[T:] = 0
-        h_pos[:T] = m.positions
-        h_pos[T:] = 0
-        h_slot[:T] = m.slot_mapping
-        h_slot[T:] = -1
+        h = {name: hb[off:off + int(np.prod(shape)) * dt.itemsize].view(_NUMPY_DTYPES[dt]).reshape(shape)
+             for name, dt, shape, off in fields}
+        if self.mixed_batches and m.block_tables.shape[1] > h["block_tables"].shape[1]:
+            return None
+        h["cu_seqlens_q"][:n + 1] = m.cu_seqlens_q
+        h["cu_seqlens_q"][n + 1:] = T
+        for name, values, pad in (("input_ids", m.input_ids, 0), ("positions", m.positions, 0),
+                                  ("slot_mapping", m.slot_mapping, -1)):
+            h[name][:T] = values
+            h[name][T:] = pad
+        if self.mixed_batches:
+            h["cu_seqlens_k"][:n + 1] = m.cu_seqlens_k
+            h["cu_seqlens_k"][n + 1:] = m.cu_seqlens_k[-1]
+            h["state_slots"][:n] = m.state_slots
+            h["state_slots"][n:] = -1
+            h["block_tables"][:n, :m.block_tables.shape[1]] = m.block_tables
+            end = fields[-1][3] + n * h["block_tables"].shape[1] * 4
         self.prefill_dev[:end].copy_(self.prefill_host[:end], non_blocking=True)
         g.replay()
-        set_context(True, cu[:n + 1], cu[:n + 1], m.max_seqlen_q, m.max_seqlen_k, slots, None, None, pos)
+        cu_q = v["cu_seqlens_q"][:n + 1]
+        cu_k = v["cu_seqlens_k"][:n + 1] if self.mixed_batches else cu_q
+        set_context(True, cu_q, cu_k, m.max_seqlen_q, m.max_seqlen_k, v["slot_mapping"], None, None, v["positions"])
         return self.prefill_out[:tokens]
 
     # ------------------------------------------------------------------ CUDA graphs for decode

@@ -59,7 +59,7 @@ def engine_config(model_dir: str, dtype: str, max_tokens: int, block_size: int =
     """Engine configuration whose pools hold ``max_tokens`` tokens of live requests, at most ``max_requests`` of them."""
     cfg = dict(model=model_dir, dtype=dtype, block_size=block_size, max_num_sequences=max_requests,
                max_num_batched_tokens=max_tokens, max_cached_blocks=(max_tokens + block_size - 1) // block_size, eos=-1,
-               device="cuda:0", prefill_token_multiple=64)
+               device="cuda:0", prefill_token_multiple=64, prefill_graphs=False)
     cfg.update(kw)
     return cfg
 

@@ -181,7 +181,8 @@ def agree(streams, cfg, w, prompts, slack):
 
 
 @pytest.mark.parametrize("dtype,slack", [(torch.float32, 3e-4), (torch.bfloat16, 0.12)])
-@pytest.mark.parametrize("kw", [dict(), dict(enforce_eager=True), dict(decode_window=5), dict(max_num_batched_tokens=24),
+@pytest.mark.parametrize("kw", [dict(), dict(prefill_graphs=True), dict(prefill_graphs=True, max_num_batched_tokens=64),
+                                dict(enforce_eager=True), dict(decode_window=5), dict(max_num_batched_tokens=24),
                                 dict(max_num_batched_tokens=40, max_cached_blocks=11)])
 def test_greedy_generation_through_the_scheduler(kw, dtype, slack):
     """``LLMEngine.generate``: more requests than slots; with a small budget prompts are read in portions beside
@@ -191,6 +192,7 @@ def test_greedy_generation_through_the_scheduler(kw, dtype, slack):
     w = fx.weights(cfg, 7)
     prompts = [fx.tokens(cfg, n, 90 + n) for n in (40, 3, 77, 16, 1, 33, 50)]
     eng = make_engine(cfg, w, dtype, max_tokens=1024, max_num_batched_tokens=kw.pop("max_num_batched_tokens", 512), **kw)
+    assert bool(eng.model_runner.prefill_graphs) == ("prefill_graphs" in kw and dtype == torch.bfloat16)
     preempted = []
     original = eng.scheduler.preempt
     eng.scheduler.preempt = lambda s: (preempted.append(s), original(s))
