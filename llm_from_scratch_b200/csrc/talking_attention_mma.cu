@@ -23,6 +23,7 @@ namespace {
 constexpr int BQ = kTalkTileRows;
 constexpr int BK = 32;
 constexpr int kSRow = 36;            // floats per score row: 32 keys + padding (odd multiple of 16 bytes)
+constexpr int kPlane = BQ * kSRow + 4;   // floats per head: heads two apart start eight banks apart
 constexpr int kQueryInSmem = 1, kTwoScores = 2;
 constexpr float kSlack = 30.f;       // log2 of how far a score may exceed the row's reference
 
@@ -33,6 +34,7 @@ template <int HP>
 struct MixParam {
   float t[HP * HP];                  // talk * log2(e), [out][in], zero-padded
   float r1[HP], r2[HP];
+  uint32_t tb[HP * HP / 2];          // talk in bf16 pairs of neighbouring in-heads (tensor-core mix)
 };
 
 __device__ __forceinline__ float rcp_approx(float x) {
@@ -47,7 +49,7 @@ __device__ __forceinline__ float capped(float x, float k, float cap, float two_c
 }
 
 // HP: heads padded; NW: warps; MAXC: value columns per CTA in units of 16; MODE: 0 any constants, 1 soft cap and bias table
-// present, 2 also H == HP; q_smem: the query rows are staged in shared memory (else their fragments are read from global memory)
+// present, 2 also H == HP, 3 as 1 with the mix on tensor cores (a talk matrix of bf16 values); q_smem: the query rows are staged in shared memory (else their fragments are read from global memory)
 template <int HP, int NW, int MAXC, int MINB, int MODE>
 __global__ void __launch_bounds__(NW * 32, MINB)
 talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp, const int layout) {
@@ -56,6 +58,8 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
   extern __shared__ __align__(128) uint8_t smem[];
   __shared__ __align__(16) float s_ref[BQ * HP];     // reference maximum (log2 domain) per (row, head)
   __shared__ float s_cor[2][BQ * HP];  // by tile parity: factor for accumulators and sums, 1 unless the flag is set
+  constexpr int kTalkRow = HP / 2 + 4;           // words per row of the matrix, padded against bank conflicts
+  __shared__ uint32_t s_talk[MODE == 3 ? HP * kTalkRow : 1];
   __shared__ int s_flag[2], s_seq, s_tile;       // flag (by tile parity): some reference moved
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
   const int H = MODE == 2 ? HP : a.H, G = a.Hkv, Gs = H / G, dk = a.dk;
@@ -109,7 +113,7 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
   const int strQ = dk + 8, strK = G * dk + 8, strV = G * dvc + 8;      // elements; odd multiples of 16 bytes
   const uint32_t sQ = smem_u32(smem);
   const uint32_t sS = sQ + (q_smem ? H * BQ * strQ * 2 : 0);
-  const uint32_t s_bytes = H * BQ * kSRow * 4;         // one of two score buffers
+  const uint32_t s_bytes = H * kPlane * 4;         // one of two score buffers
   const uint32_t sK = sS + (two_scores ? 2 : 1) * s_bytes;
   const uint32_t sV = sK + BK * strK * 2;
   float* S0 = reinterpret_cast<float*>(smem + (sS - sQ));
@@ -158,6 +162,8 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
     s_cor[0][i] = s_cor[1][i] = 1.f;
   }
   if (tid < 2) s_flag[tid] = 0;
+  if constexpr (MODE == 3)
+    for (int i = tid; i < HP * HP / 2; i += kThreads) s_talk[i / (HP / 2) * kTalkRow + i % (HP / 2)] = mp.tb[i];
 
   float o[HPW][2 * MAXC][4], l[HPW][2];
 #pragma unroll
@@ -174,12 +180,109 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
   for (int hh = 0; hh < HPW; ++hh) kv[hh] = min(warp * HPW + hh, H - 1) / Gs;
   const uint32_t adQ = sQ + ((warp * HPW * BQ + ar) * strQ + ac * 8) * 2, stepQ = BQ * strQ * 2;     // per head
   const uint32_t adK = sK + (br * strK + bc * 8) * 2, adV = sV + (ar * strV + ac * 8) * 2;
-  const uint32_t adP = sS + (warp * HPW * BQ + ar) * kSRow * 4 + ac * 16;
+  const uint32_t adP = sS + (warp * HPW * kPlane + ar * kSRow) * 4 + ac * 16;
   const float kx = a.cap > 0.f ? 2.f * kLog2e * a.scale / a.cap : 0.f;
   const float cap = a.cap, two_cap = 2.f * a.cap;
   cp_async_wait<1>();
   __syncthreads();
 
+  const float cap_l2 = cap * kLog2e, two_cap_l2 = two_cap * kLog2e;
+  // The mix of one tile on tensor cores: warp = query row, [32 keys x in-heads] x [in-heads x out-heads].  The capped
+  // scores are split into three bf16 parts whose sum is the fp32 value and the matrix is exact in bf16, so that every
+  // product is exact and the sums are fp32.
+  auto mix_mma = [&](float* S, int t) {
+    constexpr int KS = HP / 16, NT = HP / 8;
+#pragma unroll 1
+    for (int r = warp; r < rows; r += NW) {
+      float c[2][NT][4];
+#pragma unroll
+      for (int mt = 0; mt < 2; ++mt) {
+#pragma unroll
+        for (int n = 0; n < NT; ++n) c[mt][n][0] = c[mt][n][1] = c[mt][n][2] = c[mt][n][3] = 0.f;
+        const int key = mt * 16 + g, dist = pos0 + r - (klo + t * BK + key);        // keys g and g + 8 of the row tile
+        const bool seen0 = dist >= 0 && dist < a.window, seen1 = dist >= 8 && dist - 8 < a.window;
+        const float* Sr = S + r * kSRow + key;
+        const float* tab0 = a.bias_table + (seen0 ? dist : 0);
+        const float* tab1 = a.bias_table + (seen1 ? dist - 8 : 0);
+#pragma unroll
+        for (int kk = 0; kk < KS; ++kk) {
+          uint32_t part[3][4];
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {          // fragment register e: keys g + 8 (e & 1), in-heads 2 tq + 8 (e >> 1)
+            float x[2];
+#pragma unroll
+            for (int j = 0; j < 2; ++j) {
+              const int h = min(kk * 16 + (e >> 1) * 8 + tq * 2 + j, H - 1);        // padding meets zeros of the matrix
+              const float bias = __ldg((e & 1 ? tab1 : tab0) + h * a.bias_len);
+              x[j] = fmaf(-kLog2e, bias, cap_l2) - two_cap_l2 * rcp_approx(1.f + fast_exp2(Sr[h * kPlane + (e & 1) * 8] * kx));
+            }
+#pragma unroll
+            for (int q = 0; q < 3; ++q) {
+              part[q][e] = pack_bf16x2(x[0], x[1]);
+              if (q < 2) {
+                x[0] -= __uint_as_float(part[q][e] << 16);
+                x[1] -= __uint_as_float(part[q][e] & 0xffff0000u);
+              }
+            }
+          }
+#pragma unroll
+          for (int n = 0; n < NT; ++n) {
+            const uint32_t* tp = s_talk + (n * 8 + g) * kTalkRow + kk * 8 + tq;
+            const uint32_t bf[2] = {tp[0], tp[4]};
+#pragma unroll
+            for (int q = 0; q < 3; ++q) mma_bf16_16816(c[mt][n], part[q], bf);
+          }
+        }
+#pragma unroll
+        for (int n = 0; n < NT; ++n) {
+          c[mt][n][0] = seen0 ? c[mt][n][0] : -INFINITY;
+          c[mt][n][1] = seen0 ? c[mt][n][1] : -INFINITY;
+          c[mt][n][2] = seen1 ? c[mt][n][2] : -INFINITY;
+          c[mt][n][3] = seen1 ? c[mt][n][3] : -INFINITY;
+        }
+      }
+      float2* refp = reinterpret_cast<float2*>(s_ref + r * HP + tq * 2);
+      float top = -INFINITY;
+#pragma unroll
+      for (int n = 0; n < NT; ++n) {
+        const float2 ref = refp[n * 4];
+#pragma unroll
+        for (int mt = 0; mt < 2; ++mt)
+          top = fmaxf(top, fmaxf(fmaxf(c[mt][n][0], c[mt][n][2]) - ref.x, fmaxf(c[mt][n][1], c[mt][n][3]) - ref.y));
+      }
+      if (__any_sync(0xffffffffu, top > kSlack)) {         // some head of this row needs a new reference
+#pragma unroll
+        for (int n = 0; n < NT; ++n)
+#pragma unroll
+          for (int j = 0; j < 2; ++j) {
+            float mx = fmaxf(fmaxf(c[0][n][j], c[0][n][j + 2]), fmaxf(c[1][n][j], c[1][n][j + 2]));
+            mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 4));
+            mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 8));
+            mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 16));
+            const int at = r * HP + n * 8 + tq * 2 + j;
+            if (g == 0 && mx > s_ref[at] + kSlack) {
+              s_cor[t & 1][at] = fast_exp2(s_ref[at] - mx);
+              s_ref[at] = mx;
+              s_flag[t & 1] = 1;
+            }
+          }
+      }
+      __syncwarp();                              // references are set, every lane has read its scores of the row
+      __nv_bfloat16* Pr = reinterpret_cast<__nv_bfloat16*>(S + r * kSRow) + g;
+#pragma unroll
+      for (int n = 0; n < NT; ++n) {
+        const float2 ref = refp[n * 4];
+        __nv_bfloat16* Ph = Pr + (n * 8 + tq * 2) * (kPlane * 2);
+#pragma unroll
+        for (int mt = 0; mt < 2; ++mt)
+#pragma unroll
+          for (int e = 0; e < 4; ++e)
+            if (HP == H || n * 8 + tq * 2 + (e & 1) < H)
+              Ph[(e & 1) * (kPlane * 2) + mt * 16 + (e >> 1) * 8] =
+                  __float2bfloat16_rn(fast_exp2(c[mt][n][e] - (e & 1 ? ref.y : ref.x)));
+      }
+    }
+  };
   // scores of the K tile in shared memory -> S
   auto qk = [&](float* S) {
 #pragma unroll
@@ -228,7 +331,7 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
           for (int hh = 0; hh < HS; ++hh) {
             const int h = hbase + hh;
             if (h < H) {
-              float* row = S + (h * BQ + g) * kSRow + tq * 2;
+              float* row = S + h * kPlane + g * kSRow + tq * 2;
 #pragma unroll
               for (int n = 0; n < 4; ++n) {
                 *reinterpret_cast<float2*>(row + n * 8) = make_float2(s[hh][n][0], s[hh][n][1]);
@@ -248,8 +351,10 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
   bool dirty = false;
   for (int t = 0; t < ntiles; ++t) {
     const int buf = two_scores ? t & 1 : 0;
-    float* S = S0 + buf * (H * BQ * kSRow);
+    float* S = S0 + buf * (H * kPlane);
     // ---- mix ----
+    if constexpr (MODE == 3) mix_mma(S, t);
+    else
 #pragma unroll 1
     for (int r = warp; r < rows; r += NW) {
       const int dist = pos0 + r - (klo + t * BK + lane);
@@ -259,7 +364,7 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
       const float* table = a.bias_table + dc;
       float s[HP];
 #pragma unroll
-      for (int h = 0; h < HP; ++h) s[h] = h < H ? Sr[h * BQ * kSRow] : 0.f;
+      for (int h = 0; h < HP; ++h) s[h] = h < H ? Sr[h * kPlane] : 0.f;
 #pragma unroll
       for (int h = 0; h < HP; ++h) {
         if constexpr (MODE > 0) {
@@ -309,7 +414,7 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
         const float ref[8] = {ra.x, ra.y, ra.z, ra.w, rb.x, rb.y, rb.z, rb.w};
 #pragma unroll
         for (int i = 0; i < 8; ++i)
-          if (hb + i < H) Pr[(hb + i) * BQ * kSRow * 2] = __float2bfloat16_rn(fast_exp2(m[i] - ref[i]));
+          if (hb + i < H) Pr[(hb + i) * kPlane * 2] = __float2bfloat16_rn(fast_exp2(m[i] - ref[i]));
       }
     }
     cp_async_wait<0>();
@@ -343,7 +448,7 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
           }
 #pragma unroll
           for (int kk = 0; kk < 2; ++kk) {
-            ldmatrix_x4(pf[hh][kk], pt + hh * (BQ * kSRow * 4) + kk * 32);
+            ldmatrix_x4(pf[hh][kk], pt + hh * (kPlane * 4) + kk * 32);
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
               const float2 p = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&pf[hh][kk][e]));
@@ -374,7 +479,7 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
       }
     }
     if (!two_scores) __syncthreads();        // the weights are read, their buffer takes the next scores
-    if (t + 1 < ntiles) qk(S0 + (two_scores ? (t + 1) & 1 : 0) * (H * BQ * kSRow));
+    if (t + 1 < ntiles) qk(S0 + (two_scores ? (t + 1) & 1 : 0) * (H * kPlane));
     __syncthreads();
     if (t + 1 < ntiles) load_rows(t + 1, a.vc, a.dv, dv0, dvc, sV, strV);
     if (t + 2 < ntiles) load_rows(t + 2, a.kc, dk, 0, dk, sK, strK);
@@ -414,6 +519,21 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
   }
 }
 
+// upper half of a float: its bf16 value if it is exact
+inline uint32_t bf16_bits(float x) {
+  uint32_t u;
+  memcpy(&u, &x, 4);
+  return u >> 16;
+}
+inline bool exact_in_bf16(const float* x, int n) {
+  for (int i = 0; i < n; ++i) {
+    uint32_t u;
+    memcpy(&u, x + i, 4);
+    if (u & 0xffffu) return false;
+  }
+  return true;
+}
+
 template <int HP, int NW, int MAXC, int MINB, int MODE>
 int launch_prefill(const TalkArgs& a, int chunks, size_t smem, int layout, cudaStream_t s) {
   MixParam<HP> mp;
@@ -423,6 +543,12 @@ int launch_prefill(const TalkArgs& a, int chunks, size_t smem, int layout, cudaS
   for (int h = 0; h < a.H; ++h) {
     mp.r1[h] = a.r1_host[h];
     mp.r2[h] = a.r2_host[h];
+  }
+  for (int i = 0; i < HP * HP / 2; ++i) {
+    const int h = i / (HP / 2), k = i % (HP / 2) * 2;
+    if (h < a.H)
+      mp.tb[i] = (k < a.H ? bf16_bits(a.talk_host[h * a.H + k]) : 0u) |
+                 (k + 1 < a.H ? bf16_bits(a.talk_host[h * a.H + k + 1]) << 16 : 0u);
   }
   auto kern = talking_prefill_kernel<HP, NW, MAXC, MINB, MODE>;
   static size_t configured[64] = {};
@@ -440,9 +566,15 @@ int launch_prefill(const TalkArgs& a, int chunks, size_t smem, int layout, cudaS
 
 template <int HP, int NW, int MAXC, int MINB>
 int launch_prefill(const TalkArgs& a, int chunks, size_t smem, int layout, cudaStream_t s) {
-  if (a.cap > 0.f && a.window > 0 && a.bias_len >= a.window)
-    return a.H == HP ? launch_prefill<HP, NW, MAXC, MINB, 2>(a, chunks, smem, layout, s)
-                     : launch_prefill<HP, NW, MAXC, MINB, 1>(a, chunks, smem, layout, s);
+  if (a.cap > 0.f && a.window > 0 && a.bias_len >= a.window) {
+    if constexpr (HP >= 16) {
+      if (exact_in_bf16(a.talk_host, a.H * a.H))
+        return launch_prefill<HP, NW, MAXC, MINB, 3>(a, chunks, smem, layout, s);
+    } else if (a.H == HP) {
+      return launch_prefill<HP, NW, MAXC, MINB, 2>(a, chunks, smem, layout, s);
+    }
+    return launch_prefill<HP, NW, MAXC, MINB, 1>(a, chunks, smem, layout, s);
+  }
   return launch_prefill<HP, NW, MAXC, MINB, 0>(a, chunks, smem, layout, s);
 }
 
@@ -461,13 +593,13 @@ int talking_prefill_mma_launch(const TalkArgs& a, cudaStream_t s) {
     const int dvc = a.dv / chunks;
     if (dvc / 16 > max_c) continue;
     const size_t q_bytes = size_t(a.H) * BQ * (a.dk + 8) * 2;
-    const size_t s_bytes = size_t(a.H) * BQ * kSRow * 4;
+    const size_t s_bytes = size_t(a.H) * kPlane * 4;
     const size_t kv = size_t(BK) * (a.Hkv * a.dk + 8) * 2 + size_t(BK) * (a.Hkv * dvc + 8) * 2;
     size_t smem = 0;
     int layout = -1;
     for (int l : {kQueryInSmem | kTwoScores, +kTwoScores, +kQueryInSmem, 0}) {
       smem = kv + (l & kTwoScores ? 2 : 1) * s_bytes + (l & kQueryInSmem ? q_bytes : 0);
-      if (smem <= 220 * 1024) {
+      if (smem <= 216 * 1024) {
         layout = l;
         break;
       }

@@ -67,7 +67,7 @@ def talking_roofline_us(pairs: int, H: int, dk: int, dv: int, tflops: float, sms
             "sfu": pairs * 3 * H / 16 / clk}
 
 
-def kernels(steps: int = 20, warmup: int = 3, sizes=("d1024", "d2048"), hbm_gbs: float = 6547.0,
+def kernels(steps: int = 20, warmup: int = 3, sizes=("d1024", "d2048", "d4096"), hbm_gbs: float = 6547.0,
             tflops: float = 1654.0) -> dict:
     """Every kernel of the family alone: ragged prompts (8 of 1024 tokens), decode at 64 and 256 sequences with
     full windows; beside the prefill / decode attention of the GQA family on the same shapes."""
@@ -82,7 +82,7 @@ def kernels(steps: int = 20, warmup: int = 3, sizes=("d1024", "d2048"), hbm_gbs:
         lens = [1024] * 8
         T, bs, n = sum(lens), 64, len(lens)
         nb = T // bs
-        c = ops.TalkingHeads(D ** -0.5, 30.0, torch.rand(H), torch.rand(H), torch.eye(H) + 0.1 * torch.randn(H, H), W, dev)
+        c = ops.TalkingHeads(D ** -0.5, 30.0, torch.rand(H), torch.rand(H), (torch.eye(H) + 0.1 * torch.randn(H, H)).bfloat16(), W, dev)
         kc, vc = rnd(nb, bs, G, D), rnd(nb, bs, G, D)
         bt = torch.randperm(nb, generator=g, device=dev).int().view(n, -1)
         cu = torch.tensor(np.concatenate([[0], np.cumsum(lens)]), dtype=torch.int32, device=dev)

@@ -82,15 +82,18 @@ class Pool:
 
 
 def head_constants(H, seed):
+    """r1, r2, talk; for some head counts talk is not exact in bf16 (another form of the mix serves it)."""
     g = gen(seed + 77)
+    talk = torch.eye(H) + 0.3 * torch.randn(H, H, generator=g)
     return (torch.rand(H, generator=g).bfloat16().float(), torch.rand(H, generator=g).bfloat16().float(),
-            (torch.eye(H) + 0.3 * torch.randn(H, H, generator=g)).bfloat16().float())
+            talk if H in (12, 28) else talk.bfloat16().float())
 
 
 SHAPES = [  # H, G, dk, dv, window, block size
     (4, 2, 32, 48, 40, 16), (6, 3, 64, 128, 50, 64), (1, 1, 16, 16, 1, 16), (8, 8, 48, 32, 7, 16),
     (16, 4, 64, 64, 100, 16), (12, 2, 128, 128, 64, 32), (24, 4, 64, 32, 33, 16), (32, 2, 32, 64, 70, 16),
-    (5, 1, 80, 96, 0, 16), (3, 3, 20, 24, 10, 16), (16, 16, 32, 32, 0, 64), (9, 3, 256, 256, 90, 16), (16, 1, 64, 64, 48, 16)]
+    (5, 1, 80, 96, 0, 16), (3, 3, 20, 24, 10, 16), (16, 16, 32, 32, 0, 64), (9, 3, 256, 256, 90, 16), (16, 1, 64, 64, 48, 16),
+    (28, 4, 32, 32, 60, 16), (16, 4, 128, 128, 130, 16), (32, 8, 128, 128, 130, 64)]
 
 
 @pytest.mark.parametrize("general", [False, True])
