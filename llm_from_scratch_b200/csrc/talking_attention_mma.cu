@@ -24,6 +24,7 @@ constexpr int BQ = kTalkTileRows;
 constexpr int BK = 32;
 constexpr int kSRow = 36;            // floats per score row: 32 keys + padding (odd multiple of 16 bytes)
 constexpr int kPlane = BQ * kSRow + 4;   // floats per head: heads two apart start eight banks apart
+constexpr int kBiasRow = 52;              // biases of one head for the BQ + BK - 1 distances of a tile, padded
 constexpr int kQueryInSmem = 1, kTwoScores = 2;
 constexpr float kSlack = 30.f;       // log2 of how far a score may exceed the row's reference
 
@@ -116,6 +117,8 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
   const uint32_t s_bytes = H * kPlane * 4;         // one of two score buffers
   const uint32_t sK = sS + (two_scores ? 2 : 1) * s_bytes;
   const uint32_t sV = sK + BK * strK * 2;
+  const uint32_t sB = sV + BK * strV * 2;              // two bias tiles [H][kBiasRow] (MODE > 0)
+  const float* bias0 = reinterpret_cast<const float*>(smem + (sB - sQ));
   float* S0 = reinterpret_cast<float*>(smem + (sS - sQ));
 
   // ---- loads ----
@@ -128,19 +131,37 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
     }
     return static_cast<int64_t>(id) * a.bs + (j - blk * a.bs);
   };
-  auto load_rows = [&](int t, const void* cache, int d, int d0, int width, uint32_t dst, int stride) {
-    // 32 rows x G heads x width columns (from column d0 of d) of the pool
-    const int r = tid / kTpr, j = klo + t * BK + r;
-    const int64_t row = j < khi ? pool_row(j) : -1;
+  // row of the pool this thread's key row of tile t has, -1: none
+  const int my_row = tid / kTpr, my_chunk = tid % kTpr;
+  auto tile_row = [&](int t) -> int64_t {
+    const int j = klo + t * BK + my_row;
+    return j < khi ? pool_row(j) : -1;
+  };
+  // 32 rows x G heads x width columns (from column d0 of d) of the pool; kTpr threads per row
+  auto load_rows = [&](int64_t row, const void* cache, int d, int d0, int width, uint32_t dst, int stride) {
     const int cpw = width / 8, total = G * cpw;
     const __nv_bfloat16* src = static_cast<const __nv_bfloat16*>(cache) + (row < 0 ? 0 : row) * G * d + d0;
     const int bytes = row >= 0 ? 16 : 0;
+    dst += my_row * stride * 2;
     if (width == d) {
-      for (int c = tid % kTpr; c < total; c += kTpr) cp_async16(dst + (r * stride + c * 8) * 2, src + c * 8, bytes);
+#pragma unroll 4
+      for (int c = my_chunk; c < total; c += kTpr) cp_async16(dst + c * 16, src + c * 8, bytes);
     } else {
-      for (int c = tid % kTpr; c < total; c += kTpr) {
+      for (int c = my_chunk; c < total; c += kTpr) {
         const int hd = c / cpw, cc = c - hd * cpw;
-        cp_async16(dst + (r * stride + c * 8) * 2, src + hd * d + cc * 8, bytes);
+        cp_async16(dst + c * 16, src + hd * d + cc * 8, bytes);
+      }
+    }
+  };
+  // biases of tile t: entry i of a head is the distance of row 0 to the tile's last key, plus i
+  auto load_bias = [&](int t) {
+    if constexpr (MODE > 0) {
+      const int dmin = pos0 - (klo + t * BK + BK - 1);
+      const uint32_t dst = sB + (t & 1) * (H * kBiasRow * 4);
+      for (int i = tid; i < H * 48; i += kThreads) {
+        const int h = i / 48, k = i - h * 48, dist = min(max(dmin + k, 0), a.bias_len - 1);
+        asm volatile("cp.async.ca.shared.global [%0], [%1], 4;\n" ::"r"(dst + (h * kBiasRow + k) * 4),
+                     "l"(a.bias_table + h * a.bias_len + dist) : "memory");
       }
     }
   };
@@ -153,9 +174,12 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
       cp_async16(sQ + ((h * BQ + r) * strQ + cc * 8) * 2, src, r < rows ? 16 : 0);
     }
   }
-  load_rows(0, a.kc, dk, 0, dk, sK, strK);
+  int64_t next_row = tile_row(0);
+  load_rows(next_row, a.kc, dk, 0, dk, sK, strK);
   cp_async_commit();
-  load_rows(0, a.vc, a.dv, dv0, dvc, sV, strV);
+  load_rows(next_row, a.vc, a.dv, dv0, dvc, sV, strV);
+  load_bias(0);
+  load_bias(1);
   cp_async_commit();
   for (int i = tid; i < HP * BQ; i += kThreads) {
     s_ref[i] = i % HP < H ? kNoRef : INFINITY;
@@ -202,8 +226,7 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
         const int key = mt * 16 + g, dist = pos0 + r - (klo + t * BK + key);        // keys g and g + 8 of the row tile
         const bool seen0 = dist >= 0 && dist < a.window, seen1 = dist >= 8 && dist - 8 < a.window;
         const float* Sr = S + r * kSRow + key;
-        const float* tab0 = a.bias_table + (seen0 ? dist : 0);
-        const float* tab1 = a.bias_table + (seen1 ? dist - 8 : 0);
+        const float* Br = bias0 + (t & 1) * (H * kBiasRow) + r + BK - 1 - key;
 #pragma unroll
         for (int kk = 0; kk < KS; ++kk) {
           uint32_t part[3][4];
@@ -213,7 +236,7 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
 #pragma unroll
             for (int j = 0; j < 2; ++j) {
               const int h = min(kk * 16 + (e >> 1) * 8 + tq * 2 + j, H - 1);        // padding meets zeros of the matrix
-              const float bias = __ldg((e & 1 ? tab1 : tab0) + h * a.bias_len);
+              const float bias = Br[h * kBiasRow - (e & 1) * 8];
               x[j] = fmaf(-kLog2e, bias, cap_l2) - two_cap_l2 * rcp_approx(1.f + fast_exp2(Sr[h * kPlane + (e & 1) * 8] * kx));
             }
 #pragma unroll
@@ -345,7 +368,10 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
   qk(S0);
   cp_async_wait<0>();
   __syncthreads();
-  if (ntiles > 1) load_rows(1, a.kc, dk, 0, dk, sK, strK);
+  if (ntiles > 1) {
+    next_row = tile_row(1);
+    load_rows(next_row, a.kc, dk, 0, dk, sK, strK);
+  }
   cp_async_commit();
 
   bool dirty = false;
@@ -359,17 +385,16 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
     for (int r = warp; r < rows; r += NW) {
       const int dist = pos0 + r - (klo + t * BK + lane);
       const bool seen = dist >= 0 && (a.window <= 0 || dist < a.window);
-      const int dc = seen ? dist : 0;
+      const int dc = seen ? dist : 0;      // MODE 0
       float* Sr = S + r * kSRow + lane;
-      const float* table = a.bias_table + dc;
+      const float* Br = bias0 + (t & 1) * (H * kBiasRow) + r + BK - 1 - lane;
       float s[HP];
 #pragma unroll
       for (int h = 0; h < HP; ++h) s[h] = h < H ? Sr[h * kPlane] : 0.f;
 #pragma unroll
       for (int h = 0; h < HP; ++h) {
         if constexpr (MODE > 0) {
-          const float bias = __ldg(table);
-          if (h + 1 < H) table += a.bias_len;
+          const float bias = h < H ? Br[h * kBiasRow] : 0.f;
           s[h] = capped(s[h], kx, cap, two_cap, bias);    // a padding head is finite and meets zeros of the mix
         } else {
           const float bias = a.bias_len > 0 ? __ldg(a.bias_table + min(h, H - 1) * a.bias_len + dc)
@@ -481,8 +506,12 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
     if (!two_scores) __syncthreads();        // the weights are read, their buffer takes the next scores
     if (t + 1 < ntiles) qk(S0 + (two_scores ? (t + 1) & 1 : 0) * (H * kPlane));
     __syncthreads();
-    if (t + 1 < ntiles) load_rows(t + 1, a.vc, a.dv, dv0, dvc, sV, strV);
-    if (t + 2 < ntiles) load_rows(t + 2, a.kc, dk, 0, dk, sK, strK);
+    if (t + 1 < ntiles) load_rows(next_row, a.vc, a.dv, dv0, dvc, sV, strV);
+    if (t + 2 < ntiles) {
+      next_row = tile_row(t + 2);
+      load_rows(next_row, a.kc, dk, 0, dk, sK, strK);
+      load_bias(t + 2);
+    }
     cp_async_commit();
   }
 
@@ -594,7 +623,8 @@ int talking_prefill_mma_launch(const TalkArgs& a, cudaStream_t s) {
     if (dvc / 16 > max_c) continue;
     const size_t q_bytes = size_t(a.H) * BQ * (a.dk + 8) * 2;
     const size_t s_bytes = size_t(a.H) * kPlane * 4;
-    const size_t kv = size_t(BK) * (a.Hkv * a.dk + 8) * 2 + size_t(BK) * (a.Hkv * dvc + 8) * 2;
+    const size_t kv = size_t(BK) * (a.Hkv * a.dk + 8) * 2 + size_t(BK) * (a.Hkv * dvc + 8) * 2 +
+                      2 * size_t(a.H) * kBiasRow * 4;      // keys, values, biases
     size_t smem = 0;
     int layout = -1;
     for (int l : {kQueryInSmem | kTwoScores, +kTwoScores, +kQueryInSmem, 0}) {
