@@ -17,7 +17,7 @@
 //   pass 3 (scan)          the outputs from the entry states; the last segment leaves the state in the pool
 //                          A sequence of one segment needs pass 3 only.  A thread keeps R key channels x C value
 //                          columns of the state in registers and walks the tokens; q / f / k / v of 16 tokens at a
-//                          time sit in shared memory as fp32, the 16 threads of a column reduce their part of o by
+//                          time sit in shared memory as fp32, the RG threads of a column reduce their part of o by
 //                          shuffles, and 16 tokens of outputs are normed together.
 #include "common.cuh"
 
@@ -202,7 +202,6 @@ int launch_step(const RecArgs& a, int n, bool vec, cudaStream_t s) {
 // ---------------------------------------------------------------------------------------------
 // Segmented scan
 // ---------------------------------------------------------------------------------------------
-constexpr int kRowGroups = 16;       // threads that share a column group
 constexpr int kBlockTokens = 16;     // tokens staged at a time
 
 struct ScanArgs {
@@ -269,9 +268,10 @@ __device__ __forceinline__ bool find_segment(const RecArgs& a, const ScanArgs& c
   return found[0] >= 0;
 }
 
-template <typename T, int R, int C, bool LOCAL>
+// RG: threads that share a column group
+template <typename T, int R, int C, int RG, bool LOCAL>
 __global__ void __launch_bounds__(512, 1) recurrence_scan_kernel(const RecArgs a, const ScanArgs sc) {
-  constexpr int DK = R * kRowGroups, P = R / 2;
+  constexpr int DK = R * RG, P = R / 2;
   extern __shared__ __align__(16) float sm[];
   const int dk = a.dk, dv = a.dv, head = blockIdx.y, number = blockIdx.x;
   int seq, index;
@@ -291,11 +291,11 @@ __global__ void __launch_bounds__(512, 1) recurrence_scan_kernel(const RecArgs a
   // rows of the projection as they are, two blocks: [2][kBlockTokens][f | (q) | v]
   T* raw = reinterpret_cast<T*>(so + (LOCAL ? 0 : kBlockTokens * dv));
   const int at_q = dk, at_v = LOCAL ? dk : 2 * dk, raw_row = at_v + dv;
-  const int tid = threadIdx.x, threads = blockDim.x, rg = tid & (kRowGroups - 1), c0 = (tid / kRowGroups) * C;
+  const int tid = threadIdx.x, threads = blockDim.x, rg = tid & (RG - 1), c0 = (tid / RG) * C;
   const bool cols = c0 < dv;                       // dv is a multiple of 4: a float4 is in or out as a whole
 
   // pair p of this thread: rows row(p), row(p) + 1
-  auto row = [&](int p) { return (p >> 1) * 64 + rg * 4 + (p & 1) * 2; };
+  auto row = [&](int p) { return (p >> 1) * (4 * RG) + rg * 4 + (p & 1) * 2; };
   f32x2 S[P][C], D[P];
   const int64_t head_state = static_cast<int64_t>(dk) * dv;
   float* pool = a.state + (info.slot * a.H + head) * head_state;
@@ -375,7 +375,7 @@ __global__ void __launch_bounds__(512, 1) recurrence_scan_kernel(const RecArgs a
       f32x2 f[P], k[P], q[P], v[C];
 #pragma unroll
       for (int i = 0; i < P; i += 2) {
-        const int at = t * DK + (i >> 1) * 64 + rg * 4;
+        const int at = t * DK + (i >> 1) * (4 * RG) + rg * 4;
         const ulonglong2 fx = *reinterpret_cast<const ulonglong2*>(sf + at), kx = *reinterpret_cast<const ulonglong2*>(sk + at);
         f[i] = fx.x, f[i + 1] = fx.y, k[i] = kx.x, k[i + 1] = kx.y;
         if (!LOCAL) {
@@ -406,10 +406,10 @@ __global__ void __launch_bounds__(512, 1) recurrence_scan_kernel(const RecArgs a
 #pragma unroll
         for (int p = 0; p < P; ++p) D[p] = mul2(D[p], f[p]);
       } else {
-        // sum over the 16 row groups; every step a lane keeps half of the columns it still has
+        // sum over the row groups; every step a lane keeps half of the columns it still has
         int col = 0;
 #pragma unroll
-        for (int half = C / 2, step = 8; half >= 1; half >>= 1, step >>= 1) {
+        for (int half = C / 2, step = RG / 2; half >= 1; half >>= 1, step >>= 1) {
           const bool up = rg & step;
 #pragma unroll
           for (int c = 0; c < half; ++c) {
@@ -418,7 +418,7 @@ __global__ void __launch_bounds__(512, 1) recurrence_scan_kernel(const RecArgs a
           }
           if (up) col += half;
         }
-        constexpr int kLeft = kRowGroups / C;        // lanes that still share one column
+        constexpr int kLeft = RG / C;        // lanes that still share one column
 #pragma unroll
         for (int step = kLeft / 2; step >= 1; step >>= 1) o[0] += __shfl_xor_sync(0xffffffffu, o[0], step);
         if (cols && (rg & (kLeft - 1)) == 0) so[t * dv + c0 + col] = o[0];
@@ -436,7 +436,7 @@ __global__ void __launch_bounds__(512, 1) recurrence_scan_kernel(const RecArgs a
       }
     }
   }
-  if (LOCAL && tid < kRowGroups) {
+  if (LOCAL && tid < RG) {
     float* dec = sc.seg_decay + (static_cast<int64_t>(number) * a.H + head) * dk;
 #pragma unroll
     for (int p = 0; p < P; ++p) {
@@ -518,12 +518,12 @@ inline int scan_seg_len(int64_t tokens, int H) {
   return want >= 128 ? 128 : want >= 64 ? 64 : 32;
 }
 
-template <typename T, int R, int C>
+template <typename T, int R, int C, int RG>
 int launch_scan(const RecArgs& a, const ScanArgs& sc, int64_t segments, bool chained, cudaStream_t s) {
-  const int groups = (a.dv + C - 1) / C, threads = (groups * kRowGroups + 31) / 32 * 32;
-  auto local = recurrence_scan_kernel<T, R, C, true>;
-  auto full = recurrence_scan_kernel<T, R, C, false>;
-  const size_t one = size_t(kBlockTokens) * R * kRowGroups * sizeof(float), v = size_t(kBlockTokens) * a.dv * sizeof(float);
+  const int groups = (a.dv + C - 1) / C, threads = (groups * RG + 31) / 32 * 32;
+  auto local = recurrence_scan_kernel<T, R, C, RG, true>;
+  auto full = recurrence_scan_kernel<T, R, C, RG, false>;
+  const size_t one = size_t(kBlockTokens) * R * RG * sizeof(float), v = size_t(kBlockTokens) * a.dv * sizeof(float);
   const size_t smem_local = 2 * one + 2 * v + 2 * kBlockTokens * size_t(a.dk + a.dv) * sizeof(T);
   const size_t smem_full = 3 * one + 3 * v + 2 * kBlockTokens * size_t(2 * a.dk + a.dv) * sizeof(T);
   if (smem_full > 40 * 1024 &&
@@ -542,9 +542,9 @@ int launch_scan(const RecArgs& a, const ScanArgs& sc, int64_t segments, bool cha
 
 template <typename T>
 int dispatch_scan(const RecArgs& a, const ScanArgs& sc, int64_t segments, bool chained, cudaStream_t s) {
-  if (a.dk <= 64) return launch_scan<T, 4, 8>(a, sc, segments, chained, s);
-  if (a.dk <= 128) return launch_scan<T, 8, 8>(a, sc, segments, chained, s);
-  return launch_scan<T, 16, 4>(a, sc, segments, chained, s);
+  if (a.dk <= 64) return launch_scan<T, 8, 4, 8>(a, sc, segments, chained, s);
+  if (a.dk <= 128) return launch_scan<T, 8, 8, 16>(a, sc, segments, chained, s);
+  return launch_scan<T, 16, 4, 16>(a, sc, segments, chained, s);
 }
 
 }  // namespace
