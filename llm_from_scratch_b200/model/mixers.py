@@ -124,7 +124,11 @@ class GatedRecurrence(nn.Module):
 
 class ParallelMixer(nn.Module):
     """Two mixers side by side over one input.  Returns both results; their norms and the mean of the two belong
-    to the residual update (``join`` holds the norm weights), which the stream kernel does in one pass."""
+    to the residual update (``join`` holds the norm weights), which the stream kernel does in one pass.
+
+    A decode step runs the right mixer on a second CUDA stream: at decode sizes neither of the two fills the GPU."""
+
+    _side: dict = {}       # second stream per device
 
     def __init__(self, p: Params, d_model: int, left: nn.Module, right: nn.Module):
         super().__init__()
@@ -136,7 +140,19 @@ class ParallelMixer(nn.Module):
 
     def forward(self, h, ctx):
         parts = self.project(h)
-        return self.left(*parts[:self.num_left], ctx), self.right(*parts[self.num_left:], ctx)
+        left, right = parts[:self.num_left], parts[self.num_left:]
+        if ctx.is_prefill:
+            return self.left(*left, ctx), self.right(*right, ctx)
+        main = torch.cuda.current_stream()
+        side = self._side.setdefault(h.device, None) or torch.cuda.Stream(h.device)
+        self._side[h.device] = side
+        side.wait_stream(main)
+        with torch.cuda.stream(side):
+            y1 = self.right(*right, ctx)
+        y = self.left(*left, ctx)
+        main.wait_stream(side)
+        y1.record_stream(main)      # allocated on the side stream, read on this one
+        return y, y1
 
 
 class ClampedGLU(nn.Module):
