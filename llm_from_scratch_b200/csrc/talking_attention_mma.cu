@@ -1,13 +1,14 @@
 // Talking-heads attention, bf16 tensor-core path for ragged prompts and portions (mathematics: talking_attention.cu).
 //
-// The head mix couples all heads of a (query, key) pair, so one CTA owns 16 query rows of one sequence with ALL
+// The head mix couples all heads of a (query, key) pair, so one CTA owns 16 (or 8) query rows of one sequence with ALL
 // heads and walks the visible keys in tiles of 32:
 //
-//   QK   warp w holds heads w*HPW ..: S = Q K^T on mma.sync m16n8k16, fp32 scores to shared memory
-//   mix  warp w owns query rows w and w + 8, lane = key: soft cap, distance bias, the H x H mix with the matrix
-//        as constant-bank operands (it is a kernel parameter), mask, exp2 -> bf16 weights, which overwrite the
-//        scores of the same row
-//   PV   warp w again holds its heads: O += P V, fp32 accumulators in registers; row sums from the same fragments
+//   QK   a warp holds one or two heads: S = Q K^T on mma.sync m16n8k16, fp32 scores to shared memory
+//   mix  a warp owns query rows: soft cap, distance bias, the H x H mix, mask, exp2 -> bf16 weights, which overwrite
+//        the scores of the same row.  The mix runs on tensor cores without losing fp32 accuracy: a score is the sum of
+//        three bf16 values, the matrix is exact in bf16, so all products are exact (more than eight heads); else, and
+//        for matrices that bf16 does not hold, on the FMA pipe with the matrix as constant-bank operands
+//   PV   the warp again holds its heads: O += P V, fp32 accumulators in registers; row sums from the same fragments
 //
 // A tile takes two barrier intervals: its mix, then its PV together with the next tile's QK (two score buffers).
 // K of the tile after next and V of the next one arrive (cp.async) during the mix.  Scores are fp32 from the accumulator to the exponential.  The running maximum is lazy: a row keeps
@@ -20,16 +21,19 @@
 namespace b200 {
 namespace {
 
-constexpr int BQ = kTalkTileRows;
 constexpr int BK = 32;
 constexpr int kSRow = 36;            // floats per score row: 32 keys + padding (odd multiple of 16 bytes)
-constexpr int kPlane = BQ * kSRow + 4;   // floats per head: heads two apart start eight banks apart
+// floats per head of a tile of `rows` queries: heads two apart start eight banks apart
+__host__ __device__ constexpr int plane_floats(int rows) { return rows * kSRow + 4; }
 constexpr int kBiasRow = 52;              // biases of one head for the BQ + BK - 1 distances of a tile, padded
 constexpr int kQueryInSmem = 1, kTwoScores = 2;
 constexpr float kSlack = 30.f;       // log2 of how far a score may exceed the row's reference
 
 constexpr float kNoRef = -3.0e38f;   // reference of a row that has seen no key
 constexpr float kLog2e = 1.4426950408889634f;
+
+// the two warps that share a query row of the mix
+__device__ __forceinline__ void pair_barrier(int row) { asm volatile("bar.sync %0, 64;" ::"r"(row + 1) : "memory"); }
 
 template <int HP>
 struct MixParam {
@@ -51,16 +55,23 @@ __device__ __forceinline__ float capped(float x, float k, float cap, float two_c
 
 // HP: heads padded; NW: warps; MAXC: value columns per CTA in units of 16; MODE: 0 any constants, 1 soft cap and bias table
 // present, 2 also H == HP, 3 as 1 with the mix on tensor cores (a talk matrix of bf16 values); q_smem: the query rows are staged in shared memory (else their fragments are read from global memory)
-template <int HP, int NW, int MAXC, int MINB, int MODE>
+// PAIR: tiles of eight queries, and the sixteen rows of a warp's MMA tile are those of two neighbouring heads that
+// share a key head: half the accumulators per head, so that many or wide heads fit
+template <int HP, int NW, int MAXC, int MINB, int MODE, bool PAIR>
 __global__ void __launch_bounds__(NW * 32, MINB)
 talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp, const int layout) {
-  constexpr int HPW = HP / NW, kThreads = NW * 32, kTpr = kThreads / BK;    // kTpr: threads that load one key row
+  constexpr int BQ = PAIR ? kTalkTileRows / 2 : kTalkTileRows, kPlane = plane_floats(BQ);
+  static_assert(!PAIR || (MODE == 3 && HP == 2 * NW), "a pair of heads per warp");
+  constexpr bool kHalfRow = PAIR && NW == 16;          // two warps share a query row of the mix
+  constexpr int HPW = PAIR ? 1 : HP / NW, kThreads = NW * 32, kTpr = kThreads / BK;    // kTpr: threads that load one key row
   const bool q_smem = layout & kQueryInSmem, two_scores = layout & kTwoScores;
   extern __shared__ __align__(128) uint8_t smem[];
   __shared__ __align__(16) float s_ref[BQ * HP];     // reference maximum (log2 domain) per (row, head)
   __shared__ float s_cor[2][BQ * HP];  // by tile parity: factor for accumulators and sums, 1 unless the flag is set
   constexpr int kTalkRow = HP / 2 + 4;           // words per row of the matrix, padded against bank conflicts
   __shared__ uint32_t s_talk[MODE == 3 ? HP * kTalkRow : 1];
+  __shared__ float s_top[kHalfRow ? 2 * BQ * HP : 1];
+  __shared__ int s_up[kHalfRow ? BQ : 1];
   __shared__ int s_flag[2], s_seq, s_tile;       // flag (by tile parity): some reference moved
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
   const int H = MODE == 2 ? HP : a.H, G = a.Hkv, Gs = H / G, dk = a.dk;
@@ -78,7 +89,7 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
     int left = blockIdx.x, seq = -1, tile = 0;
     for (int base = 0; base < a.n && seq < 0; base += 32) {
       const int s = base + lane;
-      const int t = s < a.n ? (a.cu_q[s + 1] - a.cu_q[s] + BQ - 1) / BQ : 0;
+      const int t = s < a.n ? (a.cu_q[s + 1] - a.cu_q[s] + kTalkTileRows - 1) / kTalkTileRows : 0;
       int incl = t;
 #pragma unroll
       for (int o = 1; o < 32; o <<= 1) {
@@ -105,7 +116,8 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
   if (seq < 0) return;
   const int q0 = a.cu_q[seq], q_len = a.cu_q[seq + 1] - q0;
   const int k_len = a.cu_k[seq + 1] - a.cu_k[seq];
-  const int m0 = s_tile * BQ, rows = min(BQ, q_len - m0);
+  const int m0 = s_tile * kTalkTileRows + (PAIR ? blockIdx.z * BQ : 0), rows = min(BQ, q_len - m0);
+  if (rows <= 0) return;
   const int pos0 = k_len - q_len + m0;                 // position of row 0
   const int klo = a.window > 0 ? max(0, pos0 - a.window + 1) : 0;
   const int khi = pos0 + rows;                         // one past the last visible key
@@ -186,6 +198,7 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
     s_cor[0][i] = s_cor[1][i] = 1.f;
   }
   if (tid < 2) s_flag[tid] = 0;
+  if (kHalfRow && tid < BQ) s_up[tid] = 0;
   if constexpr (MODE == 3)
     for (int i = tid; i < HP * HP / 2; i += kThreads) s_talk[i / (HP / 2) * kTalkRow + i % (HP / 2)] = mp.tb[i];
 
@@ -201,10 +214,11 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
   const int br = (lane & 7) + (lane >> 4) * 8, bc = (lane >> 3) & 1;
   int kv[HPW];
 #pragma unroll
-  for (int hh = 0; hh < HPW; ++hh) kv[hh] = min(warp * HPW + hh, H - 1) / Gs;
-  const uint32_t adQ = sQ + ((warp * HPW * BQ + ar) * strQ + ac * 8) * 2, stepQ = BQ * strQ * 2;     // per head
+  for (int hh = 0; hh < HPW; ++hh) kv[hh] = min(PAIR ? 2 * warp : warp * HPW + hh, H - 1) / Gs;
+  // row of a lane's fragment: ar of one head, or with PAIR row (lane & 7) of head 2 warp + bc
+  const uint32_t adQ = sQ + ((PAIR ? (2 * warp + bc) * BQ + (lane & 7) : warp * HPW * BQ + ar) * strQ + ac * 8) * 2, stepQ = BQ * strQ * 2;     // per head
   const uint32_t adK = sK + (br * strK + bc * 8) * 2, adV = sV + (ar * strV + ac * 8) * 2;
-  const uint32_t adP = sS + (warp * HPW * kPlane + ar * kSRow) * 4 + ac * 16;
+  const uint32_t adP = sS + (PAIR ? (2 * warp + bc) * kPlane + (lane & 7) * kSRow : warp * HPW * kPlane + ar * kSRow) * 4 + ac * 16;
   const float kx = a.cap > 0.f ? 2.f * kLog2e * a.scale / a.cap : 0.f;
   const float cap = a.cap, two_cap = 2.f * a.cap;
   cp_async_wait<1>();
@@ -215,15 +229,16 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
   // scores are split into three bf16 parts whose sum is the fp32 value and the matrix is exact in bf16, so that every
   // product is exact and the sums are fp32.
   auto mix_mma = [&](float* S, int t) {
-    constexpr int KS = HP / 16, NT = HP / 8;
+    constexpr int KS = HP / 16, NT = HP / 8, NM = kHalfRow ? 1 : 2;      // NM: row tiles of 16 keys per warp
+    const int mt0 = kHalfRow ? warp / BQ : 0;
 #pragma unroll 1
-    for (int r = warp; r < rows; r += NW) {
-      float c[2][NT][4];
+    for (int r = kHalfRow ? warp % BQ : warp; r < rows; r += NW) {
+      float c[NM][NT][4];
 #pragma unroll
-      for (int mt = 0; mt < 2; ++mt) {
+      for (int mt = 0; mt < NM; ++mt) {
 #pragma unroll
         for (int n = 0; n < NT; ++n) c[mt][n][0] = c[mt][n][1] = c[mt][n][2] = c[mt][n][3] = 0.f;
-        const int key = mt * 16 + g, dist = pos0 + r - (klo + t * BK + key);        // keys g and g + 8 of the row tile
+        const int key = (mt0 + mt) * 16 + g, dist = pos0 + r - (klo + t * BK + key);        // keys g and g + 8 of the row tile
         const bool seen0 = dist >= 0 && dist < a.window, seen1 = dist >= 8 && dist - 8 < a.window;
         const float* Sr = S + r * kSRow + key;
         const float* Br = bias0 + (t & 1) * (H * kBiasRow) + r + BK - 1 - key;
@@ -270,25 +285,47 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
       for (int n = 0; n < NT; ++n) {
         const float2 ref = refp[n * 4];
 #pragma unroll
-        for (int mt = 0; mt < 2; ++mt)
+        for (int mt = 0; mt < NM; ++mt)
           top = fmaxf(top, fmaxf(fmaxf(c[mt][n][0], c[mt][n][2]) - ref.x, fmaxf(c[mt][n][1], c[mt][n][3]) - ref.y));
       }
-      if (__any_sync(0xffffffffu, top > kSlack)) {         // some head of this row needs a new reference
+      bool up = __any_sync(0xffffffffu, top > kSlack);
+      if constexpr (kHalfRow) {          // both halves of a row use one reference; after this both have read their scores
+        if (up && lane == 0) s_up[r] = 1;
+        pair_barrier(r);
+        up = s_up[r] != 0;
+      }
+      if (up) {                          // some head of this row needs a new reference
 #pragma unroll
         for (int n = 0; n < NT; ++n)
 #pragma unroll
           for (int j = 0; j < 2; ++j) {
-            float mx = fmaxf(fmaxf(c[0][n][j], c[0][n][j + 2]), fmaxf(c[1][n][j], c[1][n][j + 2]));
+            float mx = fmaxf(c[0][n][j], c[0][n][j + 2]);
+            if constexpr (NM == 2) mx = fmaxf(mx, fmaxf(c[NM - 1][n][j], c[NM - 1][n][j + 2]));
             mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 4));
             mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 8));
             mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 16));
             const int at = r * HP + n * 8 + tq * 2 + j;
-            if (g == 0 && mx > s_ref[at] + kSlack) {
+            if constexpr (kHalfRow) {
+              if (g == 0) s_top[mt0 * BQ * HP + at] = mx;
+            } else if (g == 0 && mx > s_ref[at] + kSlack) {
               s_cor[t & 1][at] = fast_exp2(s_ref[at] - mx);
               s_ref[at] = mx;
               s_flag[t & 1] = 1;
             }
           }
+        if constexpr (kHalfRow) {
+          pair_barrier(r);
+          if (mt0 == 0 && lane < HP) {
+            const int at = r * HP + lane;
+            const float mx = fmaxf(s_top[at], s_top[BQ * HP + at]);
+            if (mx > s_ref[at] + kSlack) {
+              s_cor[t & 1][at] = fast_exp2(s_ref[at] - mx);
+              s_ref[at] = mx;
+              s_flag[t & 1] = 1;
+            }
+          }
+          pair_barrier(r);
+        }
       }
       __syncwarp();                              // references are set, every lane has read its scores of the row
       __nv_bfloat16* Pr = reinterpret_cast<__nv_bfloat16*>(S + r * kSRow) + g;
@@ -297,11 +334,11 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
         const float2 ref = refp[n * 4];
         __nv_bfloat16* Ph = Pr + (n * 8 + tq * 2) * (kPlane * 2);
 #pragma unroll
-        for (int mt = 0; mt < 2; ++mt)
+        for (int mt = 0; mt < NM; ++mt)
 #pragma unroll
           for (int e = 0; e < 4; ++e)
             if (HP == H || n * 8 + tq * 2 + (e & 1) < H)
-              Ph[(e & 1) * (kPlane * 2) + mt * 16 + (e >> 1) * 8] =
+              Ph[(e & 1) * (kPlane * 2) + (mt0 + mt) * 16 + (e >> 1) * 8] =
                   __float2bfloat16_rn(fast_exp2(c[mt][n][e] - (e & 1 ? ref.y : ref.x)));
       }
     }
@@ -316,7 +353,7 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
         for (int hh = 0; hh < HS; ++hh)
 #pragma unroll
           for (int n = 0; n < 4; ++n) s[hh][n][0] = s[hh][n][1] = s[hh][n][2] = s[hh][n][3] = 0.f;
-        const int hbase = warp * HPW + h0;
+        const int hbase = PAIR ? 2 * warp : warp * HPW + h0;
         if (hbase < H) {
 #pragma unroll 4
           for (int ks = 0; ks < dk / 16; ++ks) {
@@ -335,7 +372,7 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
                   ldmatrix_x4(af, adQ + (h0 + hh) * stepQ + ks * 32);
                 } else {             // rows past the portion repeat its last row: their scores are never used
                   const __nv_bfloat16* q0p = qrow + static_cast<int64_t>(min(g, rows - 1)) * a.q_stride + h * dk + ks * 16 + tq * 2;
-                  const __nv_bfloat16* q1p = qrow + static_cast<int64_t>(min(g + 8, rows - 1)) * a.q_stride + h * dk + ks * 16 + tq * 2;
+                  const __nv_bfloat16* q1p = qrow + static_cast<int64_t>(min(PAIR ? g : g + 8, rows - 1)) * a.q_stride + (PAIR ? h + 1 : h) * dk + ks * 16 + tq * 2;
                   af[0] = __ldg(reinterpret_cast<const uint32_t*>(q0p));
                   af[1] = __ldg(reinterpret_cast<const uint32_t*>(q1p));
                   af[2] = __ldg(reinterpret_cast<const uint32_t*>(q0p + 8));
@@ -358,7 +395,7 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
 #pragma unroll
               for (int n = 0; n < 4; ++n) {
                 *reinterpret_cast<float2*>(row + n * 8) = make_float2(s[hh][n][0], s[hh][n][1]);
-                *reinterpret_cast<float2*>(row + 8 * kSRow + n * 8) = make_float2(s[hh][n][2], s[hh][n][3]);
+                *reinterpret_cast<float2*>(row + (PAIR ? kPlane : 8 * kSRow) + n * 8) = make_float2(s[hh][n][2], s[hh][n][3]);
               }
             }
           }
@@ -451,16 +488,17 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
       const bool rescale = s_flag[t & 1] != 0;
       // the other parity's flag and factors were last read one tile ago: ready them for the next one
       if (tid == 0) s_flag[(t + 1) & 1] = 0;
+      if (kHalfRow && tid < BQ) s_up[tid] = 0;
       if (dirty)
         for (int i = tid; i < HP * BQ; i += kThreads) s_cor[(t + 1) & 1][i] = 1.f;
       dirty = rescale;
       uint32_t pf[HPW][2][4];
 #pragma unroll
       for (int hh = 0; hh < HPW; ++hh) {
-        const int h = warp * HPW + hh;
+        const int h = PAIR ? 2 * warp : warp * HPW + hh;
         if (h < H) {
           if (rescale) {
-            const float c0 = s_cor[t & 1][g * HP + h], c1 = s_cor[t & 1][(g + 8) * HP + h];
+            const float c0 = s_cor[t & 1][g * HP + h], c1 = s_cor[t & 1][PAIR ? g * HP + h + 1 : (g + 8) * HP + h];
             l[hh][0] *= c0;
             l[hh][1] *= c1;
 #pragma unroll
@@ -490,7 +528,7 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
             uint32_t bf[4];
 #pragma unroll
             for (int hh = 0; hh < HPW; ++hh) {
-              const int h = warp * HPW + hh;
+              const int h = PAIR ? 2 * warp : warp * HPW + hh;
               if (h < H) {
                 if (hh == 0 || kv[hh] != kv[hh - 1])
                   ldmatrix_x4_trans(bf, adV + kv[hh] * dvc * 2 + kk * 32 * strV + c * 32);
@@ -518,14 +556,15 @@ talking_prefill_kernel(const TalkArgs a, const __grid_constant__ MixParam<HP> mp
   // ---- normalise, gate, store ----
 #pragma unroll
   for (int hh = 0; hh < HPW; ++hh) {
-    const int h = warp * HPW + hh;
-    if (h >= H) continue;
+    const int h0 = PAIR ? 2 * warp : warp * HPW + hh;
+    if (h0 >= H) continue;
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
+      const int h = PAIR ? h0 + e : h0;
       float sum = l[hh][e];
       sum += __shfl_xor_sync(0xffffffffu, sum, 1);
       sum += __shfl_xor_sync(0xffffffffu, sum, 2);
-      const int r = g + e * 8;
+      const int r = PAIR ? g : g + e * 8;
       if (r >= rows) continue;
       const float inv = sum > 0.f ? 1.f / sum : 0.f;
       const int64_t row = q0 + m0 + r;
@@ -563,7 +602,7 @@ inline bool exact_in_bf16(const float* x, int n) {
   return true;
 }
 
-template <int HP, int NW, int MAXC, int MINB, int MODE>
+template <int HP, int NW, int MAXC, int MINB, int MODE, bool PAIR = false>
 int launch_prefill(const TalkArgs& a, int chunks, size_t smem, int layout, cudaStream_t s) {
   MixParam<HP> mp;
   memset(&mp, 0, sizeof(mp));
@@ -579,7 +618,7 @@ int launch_prefill(const TalkArgs& a, int chunks, size_t smem, int layout, cudaS
       mp.tb[i] = (k < a.H ? bf16_bits(a.talk_host[h * a.H + k]) : 0u) |
                  (k + 1 < a.H ? bf16_bits(a.talk_host[h * a.H + k + 1]) << 16 : 0u);
   }
-  auto kern = talking_prefill_kernel<HP, NW, MAXC, MINB, MODE>;
+  auto kern = talking_prefill_kernel<HP, NW, MAXC, MINB, MODE, PAIR>;
   static size_t configured[64] = {};
   int dev = 0;
   cudaGetDevice(&dev);
@@ -588,8 +627,8 @@ int launch_prefill(const TalkArgs& a, int chunks, size_t smem, int layout, cudaS
       return B200_ERR_LAUNCH;
     if (dev >= 0 && dev < 64) configured[dev] = smem;
   }
-  const int64_t tiles = a.plan ? a.plan_capacity : a.rows / BQ + a.n;          // sum over sequences of ceil(q_len / 16) is at most this
-  kern<<<dim3(static_cast<unsigned>(tiles), chunks), NW * 32, smem, s>>>(a, mp, layout);
+  const int64_t tiles = a.plan ? a.plan_capacity : a.rows / kTalkTileRows + a.n;          // sum over sequences of ceil(q_len / 16) is at most this
+  kern<<<dim3(static_cast<unsigned>(tiles), chunks, PAIR ? 2 : 1), NW * 32, smem, s>>>(a, mp, layout);
   return launch_result();
 }
 
@@ -617,18 +656,27 @@ int talking_prefill_mma_launch(const TalkArgs& a, cudaStream_t s) {
     return B200_ERR_UNSUPPORTED;
   // value columns per CTA: what the accumulators of a warp's heads hold, and what shared memory leaves room for
   const int max_c = a.H <= 8 ? 16 : a.H <= 16 ? 8 : 4;     // units of 16 columns
+  auto smem_of = [&](int rows, int dvc, int layout) {
+    const size_t kv = size_t(BK) * (a.Hkv * a.dk + 8) * 2 + size_t(BK) * (a.Hkv * dvc + 8) * 2 +
+                      2 * size_t(a.H) * kBiasRow * 4;      // keys, values, biases
+    return kv + (layout & kTwoScores ? 2 : 1) * size_t(a.H) * plane_floats(rows) * 4 +
+           (layout & kQueryInSmem ? size_t(a.H) * rows * (a.dk + 8) * 2 : 0);
+  };
+  const bool tensor_mix = a.cap > 0.f && a.window > 0 && a.bias_len >= a.window && exact_in_bf16(a.talk_host, a.H * a.H);
+  if (tensor_mix && a.H > 16 && (a.H / a.Hkv) % 2 == 0 && a.dv <= 128) {     // many heads: pairs of heads on eight queries
+    for (int l : {kQueryInSmem | kTwoScores, +kTwoScores, +kQueryInSmem, 0}) {
+      const size_t smem = smem_of(kTalkTileRows / 2, a.dv, l);
+      if (smem <= 212 * 1024) return launch_prefill<32, 16, 8, 1, 3, true>(a, 1, smem, l, s);
+    }
+  }
   for (int chunks = 1; chunks <= a.dv / 16; ++chunks) {
     if (a.dv % (16 * chunks)) continue;
     const int dvc = a.dv / chunks;
     if (dvc / 16 > max_c) continue;
-    const size_t q_bytes = size_t(a.H) * BQ * (a.dk + 8) * 2;
-    const size_t s_bytes = size_t(a.H) * kPlane * 4;
-    const size_t kv = size_t(BK) * (a.Hkv * a.dk + 8) * 2 + size_t(BK) * (a.Hkv * dvc + 8) * 2 +
-                      2 * size_t(a.H) * kBiasRow * 4;      // keys, values, biases
     size_t smem = 0;
     int layout = -1;
     for (int l : {kQueryInSmem | kTwoScores, +kTwoScores, +kQueryInSmem, 0}) {
-      smem = kv + (l & kTwoScores ? 2 : 1) * s_bytes + (l & kQueryInSmem ? q_bytes : 0);
+      smem = smem_of(kTalkTileRows, dvc, l);
       if (smem <= 216 * 1024) {
         layout = l;
         break;

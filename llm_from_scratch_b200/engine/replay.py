@@ -51,7 +51,8 @@ class Replay:
             order = [at[id(self.live[rid])] + k for rid, _, w in entries for k in range(len(w))]
             logits = logits[order]
         for rid in end:
-            sched.drop(self.live.pop(rid))
+            if rid in self.live:
+                sched.drop(self.live.pop(rid))
         return logits
 
 
