@@ -11,9 +11,10 @@
 //   PV   the warp again holds its heads: O += P V, fp32 accumulators in registers; row sums from the same fragments
 //
 // A tile takes two barrier intervals: its mix, then its PV together with the next tile's QK (two score buffers).
-// K of the tile after next and V of the next one arrive (cp.async) during the mix.  Scores are fp32 from the accumulator to the exponential.  The running maximum is lazy: a row keeps
-// the reference maximum of an earlier tile until a score exceeds it by 2^kSlack, so the ordinary tile needs no
-// reduction over lanes; the exact maximum only has to keep the exponentials in range.
+// K of the tile after next and V of the next one arrive (cp.async) during the mix.  Scores are fp32 from the
+// accumulator to the exponential.  The running maximum is lazy: a row keeps the reference maximum of an earlier tile
+// until a score exceeds it by 2^kSlack, so the ordinary tile needs no reduction over lanes; the maximum only has to
+// keep the exponentials in range.
 #include <string.h>
 
 #include "talking_attention.cuh"

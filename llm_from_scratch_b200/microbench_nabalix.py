@@ -174,12 +174,16 @@ def throughput(steps: int = 20, warmup: int = 3, sizes=("d1024", "d2048", "d4096
     decoder of the same width, heads, feed-forward and depth."""
     from .engine import SamplingParams, Sequence
     from .engine.llm_engine import LLMEngine
+    from .model import resolve_config
+    from .model.nabalix import init_weights as init_nabalix
     out = {}
     for name in sizes:
         for family, cfg in (("nabalix", nabalix_config(SIZES[name], layers)), ("gqa", gqa_config(SIZES[name], layers))):
             Sequence.counter = itertools.count()
             bs = 64 if family == "nabalix" else 16
-            eng = LLMEngine(dict(model=cfg, dtype=torch.bfloat16, block_size=bs, max_num_sequences=batch,
+            # checkpoints of the family hold bf16 values (the head mix then runs on tensor cores)
+            weights = init_nabalix(resolve_config(cfg), 0, torch.bfloat16) if family == "nabalix" else None
+            eng = LLMEngine(dict(model=cfg, weights=weights, dtype=torch.bfloat16, block_size=bs, max_num_sequences=batch,
                                  max_num_batched_tokens=8 * prompt, max_cached_blocks=(batch + 1) * 2 * prompt // bs, eos=-1,
                                  device="cuda:0", max_model_length=2 * prompt, seed=0))
             rng = np.random.default_rng(0)
