@@ -90,7 +90,7 @@ def head_constants(H, seed):
 
 
 SHAPES = [  # H, G, dk, dv, window, block size
-    (4, 2, 32, 48, 40, 16), (6, 3, 64, 128, 50, 64), (1, 1, 16, 16, 1, 16), (8, 8, 48, 32, 7, 16),
+    (4, 2, 32, 48, 40, 16), (6, 2, 64, 112, 50, 64), (1, 1, 16, 16, 1, 16), (8, 8, 48, 32, 7, 16),
     (16, 4, 64, 64, 100, 16), (12, 2, 128, 128, 64, 32), (24, 4, 64, 32, 33, 16), (32, 2, 32, 64, 70, 16),
     (5, 1, 80, 96, 0, 16), (3, 3, 20, 24, 10, 16), (16, 16, 32, 32, 0, 64), (9, 3, 256, 256, 90, 16), (16, 1, 64, 64, 48, 16),
     (28, 4, 32, 32, 60, 16), (16, 4, 128, 128, 130, 16), (32, 8, 128, 128, 130, 64)]
@@ -180,7 +180,7 @@ def test_talking_attention_without_gate_and_cap_and_with_scores_that_outgrow_the
 
 # --------------------------------------------------------------------------------------- recurrence
 @pytest.mark.parametrize("dtype,tol", [(torch.float32, 2e-5), (torch.bfloat16, 1e-2)])
-@pytest.mark.parametrize("H,dk,dv", [(3, 16, 32), (2, 48, 32), (1, 1, 1), (2, 80, 64), (4, 128, 128), (2, 200, 72), (1, 40, 264),
+@pytest.mark.parametrize("H,dk,dv", [(3, 16, 32), (5, 48, 40), (1, 1, 1), (2, 80, 64), (4, 128, 128), (2, 200, 72), (1, 40, 264),
                                      (2, 33, 30)])
 def test_gated_recurrence_in_portions_and_steps(H, dk, dv, dtype, tol):
     """Unequal sequences in one batch, cut into portions (long ones span several scan segments, one is a single
