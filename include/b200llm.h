@@ -38,7 +38,7 @@
 extern "C" {
 #endif
 
-#define B200_ABI_VERSION 10
+#define B200_ABI_VERSION 11
 
 #define B200_DTYPE_F32 0
 #define B200_DTYPE_BF16 1
@@ -544,6 +544,100 @@ int b200_gated_recurrence(const void* q, const void* f, const void* v, int64_t t
                           const int64_t* context_lens, int32_t num_seqs, int64_t total_tokens, int32_t max_seqlen_q,
                           int32_t num_heads, int32_t dim_k, int32_t dim_v, void* out, void* workspace,
                           size_t workspace_bytes, int32_t dtype, int32_t* status, void* stream);
+
+/* b200_prefill_varlen with an attention sink: exp(sink[h]) (fp32 [num_q_heads], device; NULL: none) joins the softmax
+ * denominator of query head h, without a key, a value or the scale. */
+int b200_prefill_varlen_sink(const void* q, const void* k, const void* v, void* out, int64_t q_token_stride,
+                             int64_t k_token_stride, int64_t v_token_stride, int64_t total_q_tokens,
+                             int64_t total_k_tokens, const int32_t* cu_seqlens_q, const int32_t* cu_seqlens_k,
+                             int32_t num_seqs, int32_t max_seqlen_q, int32_t max_seqlen_k, int32_t num_q_heads,
+                             int32_t num_kv_heads, int32_t head_dim_qk, int32_t head_dim_v, float scale,
+                             const void* k_cache, const void* v_cache, const int32_t* block_tables, int64_t bt_stride,
+                             int32_t block_size, int64_t num_blocks, const int64_t* slot_mapping, const int32_t* plan,
+                             int32_t plan_tile_rows, int32_t plan_capacity, const float* sink, int32_t dtype,
+                             int32_t* status, void* stream);
+
+/* b200_paged_decode_gqa with an attention sink (as above) and value heads of a size of their own.  Workspace:
+ * b200_paged_decode_gqa_workspace_bytes() with head_dim_qk. */
+int b200_paged_decode_sink(const void* q, const void* k_cache, const void* v_cache, void* out,
+                           const int32_t* block_tables, int64_t bt_stride, const int64_t* context_lens, int32_t batch,
+                           int32_t num_q_heads, int32_t num_kv_heads, int32_t head_dim_qk, int32_t head_dim_v,
+                           int32_t block_size, int64_t num_blocks, float scale, const float* sink, void* workspace,
+                           size_t workspace_bytes, int32_t dtype, int32_t* status, void* stream);
+
+/* One sublayer boundary of a decoder that norms the sublayer's output, fp32 residual x [rows, d] in place:
+ *   x <- x + y / sqrt(mean(y^2) + eps) * norm_w,  h = x, or h = x / sqrt(mean(x^2) + eps) * final_w if given.
+ * With embed [vocab, d] / tokens [rows] the residual starts as the embedding row instead.  y, h, embed in dtype. */
+int b200_residual_norm(float* x, const int64_t* tokens, const void* embed, int64_t vocab, const void* y,
+                       const float* norm_w, const float* final_w, float eps, void* h, int64_t rows, int32_t d,
+                       int32_t dtype, int32_t* status, void* stream);
+
+/* Attention prologue with a norm per head: q [T, Hq, dim_k], k [T, Hkv, dim_k], v [T, Hkv, dim_v] are views of one
+ * projection (token stride, heads contiguous).  q and k heads are divided by their root mean square (eps inside) and
+ * multiplied by the fp32 weights [dim_k]; the channel pairs (2i, 2i + 1), i < rot_dims / 2, then turn by
+ * positions[t] * freq[i] (freq fp64, device).  Writes q_out [T, Hq, dim_k], k_out [T, Hkv, dim_k] and, if caches are given,
+ * k and v rows at slot_mapping (< 0: skipped).  dim_k <= 512. */
+int b200_head_norm_rope_store(const void* q, const void* k, const void* v, int64_t token_stride, const float* q_norm_w,
+                              const float* k_norm_w, float eps, const double* freq, int32_t rot_dims,
+                              const int64_t* positions, void* q_out, void* k_out, void* k_cache, void* v_cache,
+                              const int64_t* slot_mapping, int64_t num_slots, int64_t num_tokens, int32_t num_q_heads,
+                              int32_t num_kv_heads, int32_t dim_k, int32_t dim_v, int32_t dtype, int32_t* status,
+                              void* stream);
+
+/* Latent rows without a rotary part: rows_out[t] = rows_in[t] / sqrt(mean + eps) * norm_w [rank], also written to
+ * cache[slot_mapping[t]] (cache NULL: not stored). */
+int b200_latent_norm_store(const void* rows_in, int64_t in_stride, const float* norm_w, float eps, void* rows_out,
+                           void* cache, const int64_t* slot_mapping, int64_t num_slots, int64_t num_tokens, int32_t rank,
+                           int32_t dtype, int32_t* status, void* stream);
+
+/* Packs the cached rows of whole contexts: out row cu_seqlens_k[s] - cu_seqlens_k[0] + j = pool row of position j of
+ * sequence s.  cache [num_blocks, block_size] rows of row_bytes bytes. */
+int b200_gather_rows(const void* cache, int32_t block_size, int64_t num_blocks, int64_t row_bytes,
+                     const int32_t* block_tables, int64_t bt_stride, const int32_t* cu_seqlens_k, int32_t num_seqs,
+                     int32_t max_seqlen_k, void* out, int64_t out_rows, int32_t* status, void* stream);
+
+/* o <- o * sigmoid(gate), element by element, in place; o contiguous [rows, width], gate with a row stride. */
+int b200_sigmoid_gate(void* o, const void* gate, int64_t gate_stride, int64_t rows, int32_t width, int32_t dtype,
+                      void* stream);
+/* x <- max(x, 0)^2 in place. */
+int b200_squared_relu(void* x, int64_t n, int32_t dtype, void* stream);
+/* z <- cap tanh(scale z / cap) in place (cap <= 0: scale z). */
+int b200_softcap_logits(float* logits, int64_t n, float scale, float cap, void* stream);
+
+/* Gated delta rule over per-sequence fp32 states [num_slots, num_heads, dim_k, dim_v]; value head h uses key head
+ * h / (num_heads / num_k_heads).  With q^, k^ of unit length (1e-6 inside the root; q^ also times dim_k^-1/2),
+ * beta = sigmoid(b), g = exp(-exp(a_log) softplus(a_in + dt_bias)):
+ *   S <- g S,  u = beta (v - S^T k^),  S <- S + k^ u^T,  o = S^T q^,
+ *   out = o / sqrt(mean(o^2) + eps) * norm_w [dim_v] * silu(gate)
+ * q, k, v are projections behind a causal convolution per channel over `taps` tokens and silu.
+ *
+ * b200_delta_conv: that convolution for ragged portions; x [tokens, width] (token stride) -> out [tokens, width]; weights
+ * fp32 [taps, width], the last row weighs the current token.  ring fp32 [num_slots, taps, width] keeps the input of
+ * position p in row p mod taps and is moved on.  width a multiple of 4, pointers 16-byte aligned.
+ * b200_delta_rule: ragged portions behind b200_delta_conv (q, k, v with act_stride; b, a_in [T, num_heads] and gate
+ * [T, num_heads * dim_v] with proj_stride).  bf16 with dim_k, dim_v multiples of 16 up to 128 runs the chunked
+ * tensor-core kernels (workspace: b200_delta_rule_workspace_bytes(); without one, tokens go in order).
+ * b200_delta_step: one token per sequence, context_lens[i] long with it (0: skipped), straight from the projections
+ * (one row stride), convolution included; col_q / col_k / col_v: columns of q / k / v in conv_w and the ring.
+ * Slots < 0 are skipped; a sequence whose first token of the call is at position 0 starts from zero. */
+int b200_delta_conv(const void* x, int64_t token_stride, const float* weights, int32_t taps, int32_t width, float* ring,
+                    int64_t num_slots, const int64_t* state_slots, const int32_t* cu_seqlens_q,
+                    const int32_t* cu_seqlens_k, int32_t num_seqs, int64_t total_tokens, void* out, int32_t dtype,
+                    int32_t* status, void* stream);
+size_t b200_delta_rule_workspace_bytes(int32_t num_seqs, int64_t total_tokens, int32_t num_heads, int32_t dim_k,
+                                       int32_t dim_v, int32_t dtype);
+int b200_delta_rule(const void* q, const void* k, const void* v, int64_t act_stride, const void* b, const void* a_in,
+                    const void* gate, int64_t proj_stride, const float* dt_bias, const float* a_log, const float* norm_w,
+                    float eps, float* state, int64_t num_slots, const int64_t* state_slots, const int32_t* cu_seqlens_q,
+                    const int32_t* cu_seqlens_k, int32_t num_seqs, int64_t total_tokens, int32_t num_heads,
+                    int32_t num_k_heads, int32_t dim_k, int32_t dim_v, void* out, void* workspace, size_t workspace_bytes,
+                    int32_t dtype, int32_t* status, void* stream);
+int b200_delta_step(const void* q, const void* k, const void* v, const void* b, const void* a_in, const void* gate,
+                    int64_t proj_stride, const float* conv_w, int32_t taps, int32_t conv_width, int32_t col_q,
+                    int32_t col_k, int32_t col_v, float* conv_ring, const float* dt_bias, const float* a_log,
+                    const float* norm_w, float eps, float* state, int64_t num_slots, const int64_t* state_slots,
+                    const int64_t* context_lens, int32_t num_seqs, int32_t num_heads, int32_t num_k_heads, int32_t dim_k,
+                    int32_t dim_v, void* out, int32_t dtype, int32_t* status, void* stream);
 
 /* ---------------------------------------------------------------------------------------------
  * Diagnostic (no counterpart in the reference, which has no device code): runs the give-up path of the

@@ -80,6 +80,25 @@ SIGNATURES = {
     "b200_gated_recurrence_workspace_bytes": (_sz, [_i32, _i64, _i32, _i32, _i32, _i32]),
     "b200_gated_recurrence": (_i32, [_vp, _vp, _vp, _i64, _vp, _vp, _vp, _f32, _vp, _i64, _vp, _vp, _vp, _vp, _i32,
                                      _i64, _i32, _i32, _i32, _i32, _vp, _vp, _sz, _i32, _vp, _vp]),
+    "b200_prefill_varlen_sink": (_i32, [_vp, _vp, _vp, _vp, _i64, _i64, _i64, _i64, _i64, _vp, _vp, _i32, _i32, _i32, _i32,
+                          _i32, _i32, _i32, _f32, _vp, _vp, _vp, _i64, _i32, _i64, _vp, _vp, _i32, _i32, _vp,
+                          _i32, _vp, _vp]),
+    "b200_paged_decode_sink": (_i32, [_vp, _vp, _vp, _vp, _vp, _i64, _vp, _i32, _i32, _i32, _i32, _i32, _i32, _i64, _f32, _vp,
+                          _vp, _sz, _i32, _vp, _vp]),
+    "b200_residual_norm": (_i32, [_vp, _vp, _vp, _i64, _vp, _vp, _vp, _f32, _vp, _i64, _i32, _i32, _vp, _vp]),
+    "b200_head_norm_rope_store": (_i32, [_vp, _vp, _vp, _i64, _vp, _vp, _f32, _vp, _i32, _vp, _vp, _vp, _vp, _vp, _vp, _i64,
+                          _i64, _i32, _i32, _i32, _i32, _i32, _vp, _vp]),
+    "b200_latent_norm_store": (_i32, [_vp, _i64, _vp, _f32, _vp, _vp, _vp, _i64, _i64, _i32, _i32, _vp, _vp]),
+    "b200_gather_rows": (_i32, [_vp, _i32, _i64, _i64, _vp, _i64, _vp, _i32, _i32, _vp, _i64, _vp, _vp]),
+    "b200_sigmoid_gate": (_i32, [_vp, _vp, _i64, _i64, _i32, _i32, _vp]),
+    "b200_squared_relu": (_i32, [_vp, _i64, _i32, _vp]),
+    "b200_softcap_logits": (_i32, [_vp, _i64, _f32, _f32, _vp]),
+    "b200_delta_conv": (_i32, [_vp, _i64, _vp, _i32, _i32, _vp, _i64, _vp, _vp, _vp, _i32, _i64, _vp, _i32, _vp, _vp]),
+    "b200_delta_rule_workspace_bytes": (_sz, [_i32, _i64, _i32, _i32, _i32, _i32]),
+    "b200_delta_rule": (_i32, [_vp, _vp, _vp, _i64, _vp, _vp, _vp, _i64, _vp, _vp, _vp, _f32, _vp, _i64, _vp, _vp, _vp,
+                          _i32, _i64, _i32, _i32, _i32, _i32, _vp, _vp, _sz, _i32, _vp, _vp]),
+    "b200_delta_step": (_i32, [_vp, _vp, _vp, _vp, _vp, _vp, _i64, _vp, _i32, _i32, _i32, _i32, _i32, _vp, _vp, _vp,
+                          _vp, _f32, _vp, _i64, _vp, _vp, _i32, _i32, _i32, _i32, _i32, _vp, _i32, _vp, _vp]),
     "b200_moe_combine": (_i32, [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i32, _i32, _i32, _vp]),
     "b200_selftest_bounded_wait": (_i32, [_i32, _vp, _vp, _vp]),
     "b200_lm_head_argmax_workspace_bytes": (_sz, [_i32, _i32]),

@@ -115,6 +115,10 @@ __device__ __forceinline__ float fast_exp2(float x) {
   return y;
 }
 
+// What a sink adds to a softmax denominator whose reference maximum (log2 domain) is m: exp(sink) without a key,
+// value or scale.  A sink far above every score overflows to infinity, which turns the row into zeros as it should.
+__device__ __forceinline__ float sink_term(float sink, float m) { return fast_exp2(sink * 1.4426950408889634f - m); }
+
 // Prefill tile list (b200_prefill_plan): int32 header {tile count, rows per tile, capacity, 0} followed
 // by one entry per query tile, (sequence << 16) | tile index, heaviest tiles first.
 constexpr int kPlanHeader = 4;

@@ -19,7 +19,7 @@
 //                          columns of the state in registers and walks the tokens; q / f / k / v of 16 tokens at a
 //                          time sit in shared memory as fp32, the RG threads of a column reduce their part of o by
 //                          shuffles, and 16 tokens of outputs are normed together.
-#include "common.cuh"
+#include "sequences.cuh"
 
 namespace b200 {
 namespace {
@@ -44,24 +44,6 @@ struct RecArgs {
   int32_t* status;
 };
 
-__device__ __forceinline__ float rcp_approx(float x) {
-  float y;
-  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
-
-// sigmoid(z) and sigmoid(-z) from one exponential of -|z|, so that the small one keeps its relative accuracy
-__device__ __forceinline__ void sigmoids(float z, float* s, float* s_neg) {
-  const float t = expf(-fabsf(z)), big = rcp_approx(1.f + t), small = t * big;
-  *s = z >= 0.f ? big : small;
-  *s_neg = z >= 0.f ? small : big;
-}
-__device__ __forceinline__ float silu_f(float x) {
-  float s, n;
-  sigmoids(x, &s, &n);
-  return x * s;
-}
-
 // forget gate and write gate of one channel
 __device__ __forceinline__ void gates(float z, float lower, float* f, float* k) {
   const float open = 1.f - lower;
@@ -69,32 +51,6 @@ __device__ __forceinline__ void gates(float z, float lower, float* f, float* k) 
   sigmoids(z, &s, &n);
   *f = lower + open * s;
   *k = open * n;
-}
-
-// The sequence's token range, first position and state slot; false = nothing to do.
-struct SeqInfo {
-  int64_t tok0;
-  int len;
-  bool fresh;
-  int64_t slot;
-};
-__device__ __forceinline__ bool sequence_info(const RecArgs& a, int s, SeqInfo* r) {
-  if (a.cu_q != nullptr) {
-    r->tok0 = a.cu_q[s];
-    r->len = a.cu_q[s + 1] - a.cu_q[s];
-    r->fresh = (a.cu_k[s + 1] - a.cu_k[s]) <= r->len;
-  } else {
-    const int64_t n = a.ctx_lens[s];
-    r->tok0 = s;
-    r->len = n > 0 ? 1 : 0;
-    r->fresh = n <= 1;
-  }
-  r->slot = a.slots[s];
-  if (r->slot >= a.num_slots) {
-    if (threadIdx.x == 0) report(a.status, B200_ERR_BOUNDS);
-    return false;
-  }
-  return r->len > 0 && r->slot >= 0;
 }
 
 constexpr int kStepThreads = 256;
@@ -233,41 +189,6 @@ __device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
   return r;
 }
 
-// segment number -> (sequence, index within it, first segment number of the sequence); every thread calls it
-__device__ __forceinline__ bool find_segment(const RecArgs& a, const ScanArgs& c, int number, int* seq, int* index) {
-  __shared__ int found[2];
-  if (threadIdx.x < 32) {
-    const int lane = threadIdx.x;
-    int left = number, hit_seq = -1, hit_idx = 0;
-    for (int base = 0; base < c.n && hit_seq < 0; base += 32) {
-      const int s = base + lane;
-      const int t = s < c.n ? (a.cu_q[s + 1] - a.cu_q[s] + c.seg_len - 1) / c.seg_len : 0;
-      int incl = t;
-#pragma unroll
-      for (int o = 1; o < 32; o <<= 1) {
-        const int y = __shfl_up_sync(0xffffffffu, incl, o);
-        if (lane >= o) incl += y;
-      }
-      const unsigned hit = __ballot_sync(0xffffffffu, left < incl);
-      if (hit) {
-        const int src = __ffs(hit) - 1;
-        hit_seq = base + src;
-        hit_idx = left - __shfl_sync(0xffffffffu, incl - t, src);
-      } else {
-        left -= __shfl_sync(0xffffffffu, incl, 31);
-      }
-    }
-    if (lane == 0) {
-      found[0] = hit_seq;
-      found[1] = hit_idx;
-    }
-  }
-  __syncthreads();
-  *seq = found[0];
-  *index = found[1];
-  return found[0] >= 0;
-}
-
 // RG: threads that share a column group
 template <typename T, int R, int C, int RG, bool LOCAL>
 __global__ void __launch_bounds__(512, 1) recurrence_scan_kernel(const RecArgs a, const ScanArgs sc) {
@@ -275,7 +196,7 @@ __global__ void __launch_bounds__(512, 1) recurrence_scan_kernel(const RecArgs a
   extern __shared__ __align__(16) float sm[];
   const int dk = a.dk, dv = a.dv, head = blockIdx.y, number = blockIdx.x;
   int seq, index;
-  if (!find_segment(a, sc, number, &seq, &index)) return;
+  if (!find_segment(a.cu_q, sc.n, sc.seg_len, number, &seq, &index)) return;
   SeqInfo info;
   if (!sequence_info(a, seq, &info)) return;
   const int segments = (info.len + sc.seg_len - 1) / sc.seg_len;
@@ -468,11 +389,9 @@ __global__ void __launch_bounds__(256) recurrence_chain_kernel(const RecArgs a, 
   if (!sequence_info(a, seq, &info)) return;
   const int segments = (info.len + sc.seg_len - 1) / sc.seg_len;
   if (segments <= 1) return;
-  if (threadIdx.x < 32) {                            // number of the sequence's first segment
-    int sum = 0;
-    for (int s = threadIdx.x; s < seq; s += 32) sum += (a.cu_q[s + 1] - a.cu_q[s] + sc.seg_len - 1) / sc.seg_len;
-    for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
-    if (threadIdx.x == 0) s_first = sum;
+  if (threadIdx.x < 32) {
+    const int first = first_segment(a.cu_q, sc.seg_len, seq);
+    if (threadIdx.x == 0) s_first = first;
   }
   __syncthreads();
   const int64_t per_head = static_cast<int64_t>(a.dk) * a.dv;

@@ -24,10 +24,8 @@ struct MlaArgs {
 };
 
 constexpr int kWarps = 4;
-constexpr int kMaxQ = 18;  // (r + dr) <= 576
-constexpr int kMaxV = 16;  // r <= 512
-
-template <typename T>
+// kMaxQ, kMaxV: row elements (r + dr) and latent elements (r) per lane
+template <typename T, int kMaxQ, int kMaxV>
 __global__ void __launch_bounds__(kWarps * 32) mla_decode_simple_kernel(const MlaArgs a) {
   __shared__ float s_m[kWarps], s_l[kWarps];
   __shared__ float s_acc[kWarps][kMaxV * 32];
@@ -147,9 +145,7 @@ extern "C" int b200_mla_decode(const void* q_abs, const void* q_rope, const void
                                          workspace_bytes, status, s);
     if (rc != B200_ERR_UNSUPPORTED) return rc;
   }
-  if (kv_lora_rank + rope_dim > kMaxQ * 32 || kv_lora_rank > kMaxV * 32 ||
-      batch > 2147483647 / 1 || num_heads > 65535)
-    return B200_ERR_UNSUPPORTED;
+  if (kv_lora_rank + rope_dim > 34 * 32 || kv_lora_rank > 32 * 32 || num_heads > 65535) return B200_ERR_UNSUPPORTED;
   MlaArgs a{};
   a.q_abs = q_abs;
   a.q_rope = q_rope;
@@ -167,9 +163,10 @@ extern "C" int b200_mla_decode(const void* q_abs, const void* q_rope, const void
   a.scale_log2 = scale * 1.4426950408889634f;
   a.status = status;
   dim3 grid(batch, num_heads);
-  if (dtype == B200_DTYPE_F32)
-    mla_decode_simple_kernel<float><<<grid, kWarps * 32, 0, s>>>(a);
-  else
-    mla_decode_simple_kernel<__nv_bfloat16><<<grid, kWarps * 32, 0, s>>>(a);
+  const bool wide = kv_lora_rank + rope_dim > 18 * 32 || kv_lora_rank > 16 * 32;
+  auto kern = dtype == B200_DTYPE_F32
+                  ? (wide ? mla_decode_simple_kernel<float, 34, 32> : mla_decode_simple_kernel<float, 18, 16>)
+                  : (wide ? mla_decode_simple_kernel<__nv_bfloat16, 34, 32> : mla_decode_simple_kernel<__nv_bfloat16, 18, 16>);
+  kern<<<grid, kWarps * 32, 0, s>>>(a);
   return launch_result();
 }

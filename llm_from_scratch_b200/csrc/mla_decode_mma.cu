@@ -1,5 +1,5 @@
-// MLA latent-cache decode, bf16, tensor-core path (kv_lora_rank 512, rope_dim 64, <= 16 heads,
-// block size 16).
+// MLA latent-cache decode, bf16, tensor-core path (kv_lora_rank 512 or 256, rope_dim 64 or none, block size 16 or a
+// larger power of two; heads in groups of 16, a group per CTA).  The comments give the numbers of rank 512 with rope_dim 64.
 //
 // Every cached token is one 1152-byte latent row [c (512) | pe (64)] shared by all heads, so a
 // 16-token block is one contiguous 18 KiB segment.  The heads of a sequence are the M = 16 rows
@@ -23,6 +23,8 @@
 //   phase 3  warp w: O[:, 32w..32w+31] += P . c
 #include <cuda.h>
 
+#include <limits.h>
+
 #include "decode_common.cuh"
 #include "umma.cuh"
 
@@ -30,40 +32,44 @@ namespace b200 {
 namespace {
 
 constexpr int kTok = 16;
-constexpr int R = 512, DR = 64, ROW = R + DR;     // latent row, elements
-constexpr int ROWB = ROW * 2;                     // 1152 bytes
-constexpr int CPR = ROWB / 16;                    // 72 chunks per row
-constexpr int BLKB = kTok * ROWB;                 // 18432 bytes per block
 constexpr int GROUP = 4;                          // blocks per group (64 tokens)
 constexpr int GT = GROUP * kTok;                  // 64
 constexpr int kCompute = 512;                     // 16 compute warps: 4 token blocks x 4 k-quarters
 constexpr int kProducers = 32;                    // one warp that only fills the ring (TMA)
 constexpr int kThreads = kCompute + kProducers;
-constexpr int KSTEPS = ROW / 16;                  // 36
-constexpr int QUART_K = KSTEPS / 4;               // 9 k-steps per warp in phase 1
 constexpr int SP_STRIDE = GT + 8;                 // padded row of the partial-S buffer (floats)
-constexpr int SLABS = ROW / 64;                   // 9 slabs of 64 columns (128 bytes) per block
 
-// shared memory map (bytes)
-constexpr int OFF_RING = 0;                                   // 2 groups x 4 blocks
-constexpr int OFF_Q = OFF_RING + 2 * GROUP * BLKB;            // 16 x 1152
-constexpr int OFF_SPART = OFF_Q + 16 * ROWB;                  // [4][16][72] fp32
-constexpr int OFF_P = OFF_SPART + 4 * 16 * SP_STRIDE * 4;     // [16][64] bf16
-constexpr int OFF_STAT = OFF_P + 16 * GT * 2;                 // alpha[16], m[16], l[16] fp32
-constexpr int OFF_SCAN = OFF_STAT + 3 * 16 * 4;               // 34 ints
-constexpr int OFF_BAR = (OFF_SCAN + 34 * 4 + 15) & ~15;        // full[2] mbarriers
-constexpr int SMEM_BYTES = OFF_BAR + 2 * 8 + 8 + 1024;       // + slack to align the ring to 1024 bytes
+// sizes and shared memory map (bytes) of one latent row layout
+template <int R_, int DR_>
+struct Latent {
+  static constexpr int R = R_, DR = DR_, ROW = R + DR;         // latent row, elements
+  static constexpr int ROWB = ROW * 2;                         // 1152 bytes
+  static constexpr int CPR = ROWB / 16;                        // 72 chunks per row
+  static constexpr int BLKB = kTok * ROWB;                     // 18432 bytes per block
+  static constexpr int QUART_K = ROW / 64;                     // 9 k-steps per warp in phase 1
+  static constexpr int SLABS = ROW / 64;                       // 9 slabs of 64 columns (128 bytes) per block
+  static constexpr int NO = R / 128;                           // 8-column tiles of O per warp
+  static constexpr int OFF_RING = 0;                           // 2 groups x 4 blocks
+  static constexpr int OFF_Q = OFF_RING + 2 * GROUP * BLKB;    // 16 x 1152
+  static constexpr int OFF_SPART = OFF_Q + 16 * ROWB;          // [4][16][72] fp32
+  static constexpr int OFF_P = OFF_SPART + 4 * 16 * SP_STRIDE * 4;   // [16][64] bf16
+  static constexpr int OFF_STAT = OFF_P + 16 * GT * 2;         // alpha[16], m[16], l[16] fp32
+  static constexpr int OFF_SCAN = OFF_STAT + 3 * 16 * 4;       // 34 ints
+  static constexpr int OFF_BAR = (OFF_SCAN + 34 * 4 + 15) & ~15;     // full[2] mbarriers
+  static constexpr int SMEM_BYTES = OFF_BAR + 2 * 8 + 8 + 1024;      // + slack to align the ring to 1024 bytes
+};
 
 struct MlaArgs {
-  const __nv_bfloat16* q_abs;   // [B, H, 512]
-  const __nv_bfloat16* q_rope;  // [B, H, 64]
-  const uint8_t* lat;           // [num_blocks, 16, 576] bf16
-  __nv_bfloat16* out;           // [B, H, 512]
+  const __nv_bfloat16* q_abs;   // [B, H, R]
+  const __nv_bfloat16* q_rope;  // [B, H, DR]
+  const uint8_t* lat;           // [num_blocks, 16, ROW] bf16
+  __nv_bfloat16* out;           // [B, H, R]
   const int32_t* bt;
   int64_t bt_stride;
   const int64_t* lens;
   int batch, H;
-  int64_t num_blocks;
+  int sub_log2;                 // a block-table entry is 2^sub_log2 blocks of 16 tokens
+  int64_t num_blocks;           // 16-token blocks of the pool
   float scale_log2;
   float* part_o;
   float* part_ml;
@@ -97,8 +103,13 @@ __device__ __forceinline__ void named_arrive(int id) {
   asm volatile("bar.arrive %0, %1;\n" ::"r"(id), "n"(kThreads) : "memory");
 }
 
+template <int R_, int DR_>
 __global__ void __launch_bounds__(kThreads, 1)
 mla_decode_mma_kernel(const MlaArgs a, const __grid_constant__ CUtensorMap tm_lat) {
+  using Z = Latent<R_, DR_>;
+  constexpr int R = Z::R, DR = Z::DR, ROWB = Z::ROWB, CPR = Z::CPR, BLKB = Z::BLKB, QUART_K = Z::QUART_K, NO = Z::NO;
+  constexpr int OFF_RING = Z::OFF_RING, OFF_Q = Z::OFF_Q, OFF_SPART = Z::OFF_SPART, OFF_P = Z::OFF_P,
+                OFF_STAT = Z::OFF_STAT, OFF_SCAN = Z::OFF_SCAN, OFF_BAR = Z::OFF_BAR;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   const uint32_t sbase = smem_u32(smem);
@@ -109,11 +120,13 @@ mla_decode_mma_kernel(const MlaArgs a, const __grid_constant__ CUtensorMap tm_la
   int* s_scan = reinterpret_cast<int*>(smem + OFF_SCAN);
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
-  const int B = a.batch, H = a.H, p = blockIdx.x;
+  const int B = a.batch, p = blockIdx.x;
+  const int hb = blockIdx.y * 16, H = min(16, a.H - hb);   // this CTA's group of heads
+  const int64_t table_blocks = a.bt_stride << a.sub_log2;
   // the combine kernel is a programmatic dependent: its CTAs may be placed while this grid runs
   asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
 
-  const CtaRange rg = plan_cta_range(a.lens, B, a.bt_stride, kTok, s_scan);
+  const CtaRange rg = plan_cta_range(a.lens, B, table_blocks, kTok, s_scan);
   if (rg.cnt == 0) return;
   auto full_bar = [&](int half) -> uint32_t { return sbase + OFF_BAR + half * 8; };
   // Ring rows that no copy has written (blocks past the end of a group, at first) are read by phase 3
@@ -131,10 +144,16 @@ mla_decode_mma_kernel(const MlaArgs a, const __grid_constant__ CUtensorMap tm_la
 
   auto load_seq = [&](Cursor& c) {
     const int64_t len = a.lens[c.seq];
-    c.nblk = num_kv_blocks(len, a.bt_stride, kTok);
+    c.nblk = num_kv_blocks(len, table_blocks, kTok);
     const int64_t cap = static_cast<int64_t>(c.nblk) * kTok;
     if (len > cap) report(a.status, B200_ERR_BOUNDS);
     c.len = static_cast<int>(len < cap ? len : cap);
+  };
+  // pool block (of 16 tokens) of a sequence's block number blk; an id outside the pool stays outside
+  auto physical = [&](int seq, int blk) -> int {
+    const int id = __ldg(a.bt + static_cast<int64_t>(seq) * a.bt_stride + (blk >> a.sub_log2));
+    if (id >= (INT_MAX >> a.sub_log2)) return INT_MAX;
+    return id < 0 ? id : (id << a.sub_log2) + (blk & ((1 << a.sub_log2) - 1));
   };
   // next group of up to four consecutive blocks of one sequence inside this CTA's range
   auto next_group = [&](Cursor& c, bool with_ids) -> Group {
@@ -146,9 +165,7 @@ mla_decode_mma_kernel(const MlaArgs a, const __grid_constant__ CUtensorMap tm_la
     gr.n = min(GROUP, min(c.nblk - c.blk, c.remaining));
 #pragma unroll
     for (int b = 0; b < GROUP; ++b)
-      gr.ids[b] = (with_ids && b < gr.n)
-                      ? __ldg(a.bt + static_cast<int64_t>(gr.seq) * a.bt_stride + gr.blk0 + b)
-                      : -1;
+      gr.ids[b] = (with_ids && b < gr.n) ? physical(gr.seq, gr.blk0 + b) : -1;
     c.blk += gr.n;
     c.remaining -= gr.n;
     if (c.blk >= c.nblk && c.remaining > 0) {
@@ -212,7 +229,7 @@ mla_decode_mma_kernel(const MlaArgs a, const __grid_constant__ CUtensorMap tm_la
     return;
   }
 
-  float o[4][4];
+  float o[NO][4];
   uint32_t qf[QUART_K][4];
   bool fresh = true, load_q = false;
   int seg_first = 0;
@@ -230,14 +247,14 @@ mla_decode_mma_kernel(const MlaArgs a, const __grid_constant__ CUtensorMap tm_la
         const int r = idx / CPR, c = idx - r * CPR;
         uint4 val = make_uint4(0u, 0u, 0u, 0u);
         if (r < H) {
-          const int64_t row = static_cast<int64_t>(gr.seq) * H + r;
+          const int64_t row = static_cast<int64_t>(gr.seq) * a.H + hb + r;
           val = c < R / 8 ? __ldg(reinterpret_cast<const uint4*>(a.q_abs + row * R) + c)
                           : __ldg(reinterpret_cast<const uint4*>(a.q_rope + row * DR) + (c - R / 8));
         }
         *reinterpret_cast<uint4*>(smem + OFF_Q + r * ROWB + swz72(c, r) * 16) = val;
       }
 #pragma unroll
-      for (int n = 0; n < 4; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
+      for (int n = 0; n < NO; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
       load_q = true;
       if (tid < 16) {
         s_m[tid] = -INFINITY;
@@ -333,11 +350,11 @@ mla_decode_mma_kernel(const MlaArgs a, const __grid_constant__ CUtensorMap tm_la
     }
     compute_sync();
 
-    // ---- phase 3: O[:, 32*warp .. +31] = alpha * O + P . c
+    // ---- phase 3: the R / 16 columns of O of this warp = alpha * O + P . c
     {
       const float al0 = s_alpha[g], al1 = s_alpha[g + 8];
 #pragma unroll
-      for (int n = 0; n < 4; ++n) {
+      for (int n = 0; n < NO; ++n) {
         o[n][0] *= al0;
         o[n][1] *= al0;
         o[n][2] *= al1;
@@ -350,9 +367,9 @@ mla_decode_mma_kernel(const MlaArgs a, const __grid_constant__ CUtensorMap tm_la
         uint32_t pf[4];
         ldmatrix_x4(pf, sP + rp * 128 + (((2 * kk + chp) ^ (rp & 7)) * 16));
 #pragma unroll
-        for (int pr2 = 0; pr2 < 2; ++pr2) {
+        for (int pr2 = 0; pr2 < NO / 2; ++pr2) {
           uint32_t bf[4];
-          const int chunk = 4 * warp + 2 * pr2 + chp;
+          const int chunk = NO * warp + 2 * pr2 + chp;
           ldmatrix_x4_trans(bf, ring + kk * BLKB + lat_off(rp, chunk));
           const uint32_t b0[2] = {bf[0], bf[1]}, b1[2] = {bf[2], bf[3]};
           mma_bf16_16816(o[2 * pr2], pf, b0);
@@ -370,26 +387,26 @@ mla_decode_mma_kernel(const MlaArgs a, const __grid_constant__ CUtensorMap tm_la
       const int h0 = g, h1 = g + 8;
       if (whole) {
         const float i0 = 1.f / s_l[h0], i1 = 1.f / s_l[h1];
-        __nv_bfloat16* ob = a.out + static_cast<int64_t>(gr.seq) * H * R;
+        __nv_bfloat16* ob = a.out + (static_cast<int64_t>(gr.seq) * a.H + hb) * R;
 #pragma unroll
-        for (int n = 0; n < 4; ++n) {
-          const int d = 32 * warp + n * 8 + tq * 2;
+        for (int n = 0; n < NO; ++n) {
+          const int d = NO * 8 * warp + n * 8 + tq * 2;
           if (h0 < H) *reinterpret_cast<uint32_t*>(ob + h0 * R + d) = pack_bf16x2(o[n][0] * i0, o[n][1] * i0);
           if (h1 < H) *reinterpret_cast<uint32_t*>(ob + h1 * R + d) = pack_bf16x2(o[n][2] * i1, o[n][3] * i1);
         }
       } else {
         const int64_t pslot = static_cast<int64_t>(p) * 2 + (seg_first > 0 ? 0 : 1);
-        float* po = a.part_o + pslot * H * R;
+        float* po = a.part_o + (pslot * a.H + hb) * R;
 #pragma unroll
-        for (int n = 0; n < 4; ++n) {
-          const int d = 32 * warp + n * 8 + tq * 2;
+        for (int n = 0; n < NO; ++n) {
+          const int d = NO * 8 * warp + n * 8 + tq * 2;
           if (h0 < H) *reinterpret_cast<float2*>(po + h0 * R + d) = make_float2(o[n][0], o[n][1]);
           if (h1 < H) *reinterpret_cast<float2*>(po + h1 * R + d) = make_float2(o[n][2], o[n][3]);
         }
         if (tid < H)
-          *reinterpret_cast<float2*>(a.part_ml + (pslot * H + tid) * 2) = make_float2(s_m[tid], s_l[tid]);
+          *reinterpret_cast<float2*>(a.part_ml + (pslot * a.H + hb + tid) * 2) = make_float2(s_m[tid], s_l[tid]);
       }
-      if (seq_end && tid == 0) {
+      if (seq_end && tid == 0 && hb == 0) {      // every group of heads cuts the sequences alike
         const int seq_start_flat = flat - gr.blk0;
         a.seq_info[2 * gr.seq] = whole ? -1 : seq_start_flat / rg.per_cta;
         a.seq_info[2 * gr.seq + 1] = whole ? -1 : p;
@@ -401,8 +418,11 @@ mla_decode_mma_kernel(const MlaArgs a, const __grid_constant__ CUtensorMap tm_la
 }
 
 bool mla_fast_shape(int H, int r, int dr, int bs) {
-  return r == R && dr == DR && bs == kTok && H >= 1 && H <= 16;
+  return (r == 512 || r == 256) && (dr == 64 || dr == 0) && bs >= kTok && (bs & (bs - 1)) == 0 && H >= 1 && H <= 128;
 }
+int head_groups(int H) { return (H + 15) / 16; }
+// CTAs per group of heads: one per SM over all groups
+int group_grid(int sms, int H) { return (sms + head_groups(H) - 1) / head_groups(H); }
 
 using EncodeFn = CUresult (*)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*,
                               const cuuint64_t*, const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave,
@@ -430,36 +450,23 @@ size_t mla_decode_mma_workspace(int batch, int H, int r, int dr) {
   if (!mla_fast_shape(H, r, dr, kTok)) return 256;
   int sms = sm_count_cached();
   if (sms <= 0) sms = 148;
-  return decode_workspace_bytes(static_cast<size_t>(sms), batch, H, R);
+  return decode_workspace_bytes(static_cast<size_t>(group_grid(sms, H)), batch, H, r);
 }
 
-int mla_decode_mma_launch(const void* q_abs, const void* q_rope, const void* lat, void* out,
-                          const int32_t* bt, int64_t bt_stride, const int64_t* lens, int batch,
-                          int H, int r, int dr, int bs, int64_t num_blocks, float scale,
-                          void* workspace, size_t workspace_bytes, int32_t* status,
-                          cudaStream_t s) {
-  if (!mla_fast_shape(H, r, dr, bs)) return B200_ERR_UNSUPPORTED;
-  if (!aligned16(q_abs) || !aligned16(q_rope) || !aligned16(lat) || !aligned16(out))
-    return B200_ERR_UNSUPPORTED;
-  if (num_blocks <= 0 || num_blocks * kTok > 2147483647LL) return B200_ERR_UNSUPPORTED;
-  EncodeFn enc = tensor_map_encoder();
-  if (enc == nullptr) return B200_ERR_UNSUPPORTED;
-  const int sms = sm_count_cached();
-  if (sms <= 0) return B200_ERR_NO_DEVICE;
-  const size_t grid = static_cast<size_t>(sms);
-  const size_t need = decode_workspace_bytes(grid, batch, H, R);
-  if (!workspace || workspace_bytes < need) return B200_ERR_WORKSPACE;
-  if (reinterpret_cast<uintptr_t>(workspace) & 255u) return B200_ERR_ALIGN;
-  // The pool seen as (column within a slab: 64, token row: num_blocks * 16, slab: 9) with strides
-  // (2 B, 1152 B, 128 B): one box = one KV block, written slab by slab — [9][16 tokens][128 B] — which is
+namespace {
+template <int R, int DR>
+int launch(MlaArgs a, int64_t grid, EncodeFn enc, cudaStream_t s) {
+  using Z = Latent<R, DR>;
+  // The pool seen as (column within a slab: 64, token row: num_blocks * 16, slab: ROW / 64) with strides
+  // (2 B, ROWB, 128 B): one box = one KV block, written slab by slab — [slabs][16 tokens][128 B] — which is
   // the layout lat_off() addresses, so a block is a single copy instruction.
   CUtensorMap tm;
   {
-    const cuuint64_t dims[3] = {64, static_cast<cuuint64_t>(num_blocks) * kTok, static_cast<cuuint64_t>(SLABS)};
-    const cuuint64_t strides[2] = {static_cast<cuuint64_t>(ROWB), 128};
-    const cuuint32_t box[3] = {64, kTok, static_cast<cuuint32_t>(SLABS)};
+    const cuuint64_t dims[3] = {64, static_cast<cuuint64_t>(a.num_blocks) * kTok, static_cast<cuuint64_t>(Z::SLABS)};
+    const cuuint64_t strides[2] = {static_cast<cuuint64_t>(Z::ROWB), 128};
+    const cuuint32_t box[3] = {64, kTok, static_cast<cuuint32_t>(Z::SLABS)};
     const cuuint32_t estr[3] = {1, 1, 1};
-    if (enc(&tm, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(lat), dims, strides, box, estr,
+    if (enc(&tm, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<uint8_t*>(a.lat), dims, strides, box, estr,
             CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
             CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS)
       return B200_ERR_UNSUPPORTED;
@@ -468,11 +475,34 @@ int mla_decode_mma_launch(const void* q_abs, const void* q_rope, const void* lat
   int dev = 0;
   cudaGetDevice(&dev);
   if (dev >= 0 && dev < 64 && !configured[dev]) {
-    if (cudaFuncSetAttribute(mla_decode_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                             SMEM_BYTES) != cudaSuccess)
+    if (cudaFuncSetAttribute(mla_decode_mma_kernel<R, DR>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                             Z::SMEM_BYTES) != cudaSuccess)
       return B200_ERR_LAUNCH;
     configured[dev] = true;
   }
+  mla_decode_mma_kernel<R, DR>
+      <<<dim3(static_cast<unsigned>(grid), head_groups(a.H)), kThreads, Z::SMEM_BYTES, s>>>(a, tm);
+  return launch_result();
+}
+}  // namespace
+
+int mla_decode_mma_launch(const void* q_abs, const void* q_rope, const void* lat, void* out,
+                          const int32_t* bt, int64_t bt_stride, const int64_t* lens, int batch,
+                          int H, int r, int dr, int bs, int64_t num_blocks, float scale,
+                          void* workspace, size_t workspace_bytes, int32_t* status,
+                          cudaStream_t s) {
+  if (!mla_fast_shape(H, r, dr, bs)) return B200_ERR_UNSUPPORTED;
+  if (!aligned16(q_abs) || (dr > 0 && !aligned16(q_rope)) || !aligned16(lat) || !aligned16(out))
+    return B200_ERR_UNSUPPORTED;
+  if (num_blocks <= 0 || num_blocks * bs > 2147483647LL) return B200_ERR_UNSUPPORTED;
+  EncodeFn enc = tensor_map_encoder();
+  if (enc == nullptr) return B200_ERR_UNSUPPORTED;
+  const int sms = sm_count_cached();
+  if (sms <= 0) return B200_ERR_NO_DEVICE;
+  const size_t grid = static_cast<size_t>(group_grid(sms, H));
+  const size_t need = decode_workspace_bytes(grid, batch, H, r);
+  if (!workspace || workspace_bytes < need) return B200_ERR_WORKSPACE;
+  if (reinterpret_cast<uintptr_t>(workspace) & 255u) return B200_ERR_ALIGN;
   MlaArgs a{};
   a.q_abs = static_cast<const __nv_bfloat16*>(q_abs);
   a.q_rope = static_cast<const __nv_bfloat16*>(q_rope);
@@ -483,17 +513,18 @@ int mla_decode_mma_launch(const void* q_abs, const void* q_rope, const void* lat
   a.lens = lens;
   a.batch = batch;
   a.H = H;
-  a.num_blocks = num_blocks;
+  while ((kTok << a.sub_log2) < bs) ++a.sub_log2;
+  a.num_blocks = num_blocks << a.sub_log2;
   a.scale_log2 = scale * 1.4426950408889634f;
   a.status = status;
   uint8_t* w = static_cast<uint8_t*>(workspace);
   a.part_o = reinterpret_cast<float*>(w);
-  w += align256(grid * 2 * H * R * sizeof(float));
+  w += align256(grid * 2 * H * r * sizeof(float));
   a.part_ml = reinterpret_cast<float*>(w);
   w += align256(grid * 2 * H * 2 * sizeof(float));
   a.seq_info = reinterpret_cast<int32_t*>(w);
-  mla_decode_mma_kernel<<<static_cast<int>(grid), kThreads, SMEM_BYTES, s>>>(a, tm);
-  const int rc = launch_result();
+  const int rc = r == 512 ? (dr ? launch<512, 64>(a, grid, enc, s) : launch<512, 0>(a, grid, enc, s))
+                          : (dr ? launch<256, 64>(a, grid, enc, s) : launch<256, 0>(a, grid, enc, s));
   if (rc != B200_OK) return rc;
   CombineArgs c{};
   c.out = out;
@@ -503,7 +534,7 @@ int mla_decode_mma_launch(const void* q_abs, const void* q_rope, const void* lat
   c.seq_info = a.seq_info;
   c.batch = batch;
   c.H = H;
-  c.D = R;
+  c.D = r;
   return decode_combine_launch(c, s);
 }
 

@@ -1,6 +1,6 @@
 // Paged GQA decode attention.
 //
-// Fast path (bf16, block_size 16, head_dim 32/64/128, group size <= 16, Hkv <= 16)
+// Fast path (bf16, block_size a multiple of 16, head_dim 32/64/128, group size <= 16, Hkv <= 16)
 // ---------------------------------------------------------------------------------------------
 // The work is the flat list of all KV blocks of all sequences, in (sequence, block) order.  It is
 // cut into gridDim.x equal contiguous ranges, one per persistent CTA, so every CTA streams the
@@ -52,15 +52,24 @@ struct DecodeArgs {
   const int32_t* bt;
   int64_t bt_stride;
   const int64_t* lens;
-  int batch, Hq, Hkv, D, bs;
+  int batch, Hq, Hkv, D, Dv, bs;
+  int sub;           // 16-token blocks per block-table entry (fast path)
   int64_t num_blocks;
   float scale_log2;  // softmax scale * log2(e)
   float* part_o;     // [grid][2][Hq][D]   unnormalised partial outputs
   float* part_ml;    // [grid][2][Hq][2]   running max (log2 domain) and sum
   int32_t* seq_info; // [batch][2]         first / last CTA of a split sequence, or -1 (separate merge kernel)
   int32_t* counters; // [batch][Hkv]       arrivals per (sequence, KV head), zero between launches; null = separate merge
+  const float* sink; // [Hq] or null: exp(sink) joins the denominator of its head
   int32_t* status;
 };
+
+// physical 16-token block of a sequence's 16-token block number blk
+__device__ __forceinline__ int64_t physical_block(const DecodeArgs& a, int seq, int blk) {
+  if (a.sub == 1) return a.bt[static_cast<int64_t>(seq) * a.bt_stride + blk];
+  const int id = a.bt[static_cast<int64_t>(seq) * a.bt_stride + blk / a.sub];
+  return id < 0 ? id : static_cast<int64_t>(id) * a.sub + blk % a.sub;
+}
 
 struct Cursor {
   int seq, blk, nblk, len;
@@ -119,6 +128,7 @@ __device__ __forceinline__ void merge_split_sequence(const DecodeArgs& a, int se
       }
     }
     if (active) {
+      if (a.sink != nullptr) L += sink_term(a.sink[head], M);
       const float inv = 1.f / L;
       uint2 packed;
       packed.x = pack_bf16x2(acc.x * inv, acc.y * inv);
@@ -147,11 +157,12 @@ paged_decode_bf16_kernel(const DecodeArgs a) {
   const int B = a.batch;
   const int G = a.Hq / a.Hkv;
   const int p = blockIdx.x, P = gridDim.x;
+  const int64_t table_blocks = a.bt_stride * a.sub;
 
   // ---- plan: total block count, then the (sequence, block) where this CTA's range starts ----
   int local = 0;
   for (int i = threadIdx.x; i < B; i += blockDim.x)
-    local += num_kv_blocks(a.lens[i], a.bt_stride, kTok);
+    local += num_kv_blocks(a.lens[i], table_blocks, kTok);
   int T;
   block_inclusive_scan(local, s_scan, &T);
   if (a.counters == nullptr) {
@@ -175,7 +186,7 @@ paged_decode_bf16_kernel(const DecodeArgs a) {
     int carry = 0;
     for (int base = 0; base < B; base += blockDim.x) {
       const int i = base + threadIdx.x;
-      const int v = i < B ? num_kv_blocks(a.lens[i], a.bt_stride, kTok) : 0;
+      const int v = i < B ? num_kv_blocks(a.lens[i], table_blocks, kTok) : 0;
       int tot;
       const int incl = block_inclusive_scan(v, s_scan, &tot) + carry;
       const int excl = incl - v;
@@ -190,7 +201,7 @@ paged_decode_bf16_kernel(const DecodeArgs a) {
 
   auto load_seq = [&](Cursor& c) {
     const int64_t len = a.lens[c.seq];
-    c.nblk = num_kv_blocks(len, a.bt_stride, kTok);
+    c.nblk = num_kv_blocks(len, table_blocks, kTok);
     const int64_t cap = static_cast<int64_t>(c.nblk) * kTok;
     if (len > cap) report(a.status, B200_ERR_BOUNDS);  // table row too short for the context
     c.len = static_cast<int>(len < cap ? len : cap);
@@ -215,7 +226,7 @@ paged_decode_bf16_kernel(const DecodeArgs a) {
   load_seq(L);
   C.nblk = L.nblk;
   C.len = L.len;
-  int next_id = a.bt[static_cast<int64_t>(L.seq) * a.bt_stride + L.blk];
+  int64_t next_id = physical_block(a, L.seq, L.blk);
 
   const int h = warp;  // KV head of this warp
   const uint32_t ring = smem_u32(smem) + warp * (kStages * 2 * TILEB);
@@ -224,12 +235,11 @@ paged_decode_bf16_kernel(const DecodeArgs a) {
   const uint8_t* vbase = static_cast<const uint8_t*>(a.vc) + static_cast<int64_t>(h) * ROWB;
 
   auto issue = [&](int stage) {
-    const int id = next_id;
+    const int64_t id = next_id;
     const int valid = L.len - L.blk * kTok;  // tokens of this block inside the context
-    const bool ok = static_cast<uint64_t>(static_cast<int64_t>(id)) <
-                    static_cast<uint64_t>(a.num_blocks);
+    const bool ok = static_cast<uint64_t>(id) < static_cast<uint64_t>(a.num_blocks * a.sub);
     if (!ok) report(a.status, B200_ERR_BOUNDS);
-    const int64_t blk_off = ok ? static_cast<int64_t>(id) * kTok * row_stride : 0;
+    const int64_t blk_off = ok ? id * kTok * row_stride : 0;
     const uint32_t kdst = ring + stage * (2 * TILEB), vdst = kdst + TILEB;
 #pragma unroll
     for (int j = 0; j < LOADS; ++j) {
@@ -256,7 +266,7 @@ paged_decode_bf16_kernel(const DecodeArgs a) {
       issue(s);
       if (++issued < cnt) {
         advance(L);
-        next_id = a.bt[static_cast<int64_t>(L.seq) * a.bt_stride + L.blk];
+        next_id = physical_block(a, L.seq, L.blk);
       }
     }
     cp_async_commit();
@@ -267,7 +277,7 @@ paged_decode_bf16_kernel(const DecodeArgs a) {
       issue((j + kStages - 1) % kStages);
       if (++issued < cnt) {
         advance(L);
-        next_id = a.bt[static_cast<int64_t>(L.seq) * a.bt_stride + L.blk];
+        next_id = physical_block(a, L.seq, L.blk);
       }
     }
     cp_async_commit();
@@ -382,6 +392,10 @@ paged_decode_bf16_kernel(const DecodeArgs a) {
         }
         const int head0 = nt * 8 + tq * 2;
         if (whole) {
+          if (a.sink != nullptr) {
+            if (head0 < G) l0 += sink_term(a.sink[h * G + head0], mrow[nt][0]);
+            if (head0 + 1 < G) l1 += sink_term(a.sink[h * G + head0 + 1], mrow[nt][1]);
+          }
           const float i0 = 1.f / l0, i1 = 1.f / l1;
           __nv_bfloat16* op = static_cast<__nv_bfloat16*>(a.out) +
                               (static_cast<int64_t>(C.seq) * a.Hq + h * G) * D;
@@ -493,6 +507,7 @@ paged_decode_combine_kernel(const DecodeArgs a) {
       const float2 ml = *reinterpret_cast<const float2*>(a.part_ml + (slot_of(p) * a.Hq + h) * 2);
       L += exp2f(ml.x - M) * ml.y;
     }
+    if (a.sink != nullptr) L += sink_term(a.sink[h], M);
     s_M[h] = M;
     s_inv[h] = 1.f / L;
   }
@@ -592,11 +607,11 @@ __global__ void __launch_bounds__(kSimpleWarps * 32) paged_decode_simple_kernel(
   __shared__ float s_acc[kSimpleWarps][kSimpleMaxPerLane * 32];
   const int seq = blockIdx.x, head = blockIdx.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int D = a.D, G = a.Hq / a.Hkv, kvh = head / G;
-  T* op = static_cast<T*>(a.out) + (static_cast<int64_t>(seq) * a.Hq + head) * D;
+  const int D = a.D, Dv = a.Dv, G = a.Hq / a.Hkv, kvh = head / G;
+  T* op = static_cast<T*>(a.out) + (static_cast<int64_t>(seq) * a.Hq + head) * Dv;
   int64_t len64 = a.lens[seq];
   if (len64 <= 0) {
-    for (int d = threadIdx.x; d < D; d += blockDim.x) op[d] = from_float<T>(0.f);
+    for (int d = threadIdx.x; d < Dv; d += blockDim.x) op[d] = from_float<T>(0.f);
     return;
   }
   const int64_t cap = a.bt_stride * a.bs;
@@ -622,7 +637,8 @@ __global__ void __launch_bounds__(kSimpleWarps * 32) paged_decode_simple_kernel(
       report(a.status, B200_ERR_BOUNDS);
       continue;
     }
-    const int64_t row = ((static_cast<int64_t>(id) * a.bs + t % a.bs) * a.Hkv + kvh) * D;
+    const int64_t slot = (static_cast<int64_t>(id) * a.bs + t % a.bs) * a.Hkv + kvh;
+    const int64_t row = slot * D, vrow = slot * Dv;
     float dot = 0.f;
 #pragma unroll
     for (int k = 0; k < kSimpleMaxPerLane; ++k) {
@@ -636,7 +652,7 @@ __global__ void __launch_bounds__(kSimpleWarps * 32) paged_decode_simple_kernel(
 #pragma unroll
     for (int k = 0; k < kSimpleMaxPerLane; ++k) {
       const int d = lane + 32 * k;
-      if (d < D) acc[k] = acc[k] * al + pw * to_float<T>(vc[row + d]);
+      if (d < Dv) acc[k] = acc[k] * al + pw * to_float<T>(vc[vrow + d]);
     }
     m = mn;
   }
@@ -655,7 +671,8 @@ __global__ void __launch_bounds__(kSimpleWarps * 32) paged_decode_simple_kernel(
     wgt[w] = s_m[w] == -INFINITY ? 0.f : exp2f(s_m[w] - M);
     Lsum += wgt[w] * s_l[w];
   }
-  for (int d = threadIdx.x; d < D; d += blockDim.x) {
+  if (a.sink != nullptr && M > -INFINITY) Lsum += exp2f(a.sink[head] * 1.4426950408889634f - M);
+  for (int d = threadIdx.x; d < Dv; d += blockDim.x) {
     float v = 0.f;
     for (int w = 0; w < kSimpleWarps; ++w) v += wgt[w] * s_acc[w][d];
     op[d] = from_float<T>(Lsum > 0.f ? v / Lsum : 0.f);
@@ -673,7 +690,7 @@ struct FastPlan {
 FastPlan fast_plan(int Hq, int Hkv, int D, int bs, int dtype) {
   FastPlan pl{};
   pl.ok = false;
-  if (dtype != B200_DTYPE_BF16 || bs != kTok) return pl;
+  if (dtype != B200_DTYPE_BF16 || bs % kTok != 0) return pl;
   if (D != 32 && D != 64 && D != 128) return pl;
   if (Hkv <= 0 || Hkv > kMaxFastThreads / 32 || Hq % Hkv != 0) return pl;
   const int G = Hq / Hkv;
@@ -731,15 +748,13 @@ extern "C" size_t b200_paged_decode_gqa_workspace_bytes(int32_t batch, int32_t n
   return bytes;
 }
 
-extern "C" int b200_paged_decode_gqa(const void* q, const void* k_cache, const void* v_cache,
-                                     void* out, const int32_t* block_tables, int64_t bt_stride,
-                                     const int64_t* context_lens, int32_t batch,
-                                     int32_t num_q_heads, int32_t num_kv_heads, int32_t head_dim,
-                                     int32_t block_size, int64_t num_blocks, float scale,
-                                     void* workspace, size_t workspace_bytes, int32_t dtype,
-                                     int32_t* status, void* stream) {
-  using namespace b200;
-  if (batch < 0 || num_q_heads <= 0 || num_kv_heads <= 0 || head_dim <= 0 || block_size <= 0 ||
+namespace b200 {
+static int paged_decode(const void* q, const void* k_cache, const void* v_cache, void* out, const int32_t* block_tables,
+                        int64_t bt_stride, const int64_t* context_lens, int32_t batch, int32_t num_q_heads,
+                        int32_t num_kv_heads, int32_t head_dim, int32_t head_dim_v, int32_t block_size, int64_t num_blocks,
+                        float scale, const float* sink, void* workspace, size_t workspace_bytes, int32_t dtype,
+                        int32_t* status, void* stream) {
+  if (batch < 0 || num_q_heads <= 0 || num_kv_heads <= 0 || head_dim <= 0 || head_dim_v <= 0 || block_size <= 0 ||
       num_blocks < 0 || bt_stride <= 0)
     return B200_ERR_ARG;
   if (num_q_heads % num_kv_heads != 0) return B200_ERR_ARG;
@@ -761,14 +776,18 @@ extern "C" int b200_paged_decode_gqa(const void* q, const void* k_cache, const v
   a.Hq = num_q_heads;
   a.Hkv = num_kv_heads;
   a.D = head_dim;
+  a.Dv = head_dim_v;
   a.bs = block_size;
+  a.sub = 1;
+  a.sink = sink;
   a.num_blocks = num_blocks;
   a.scale_log2 = scale * 1.4426950408889634f;
   a.status = status;
 
   const FastPlan pl = fast_plan(num_q_heads, num_kv_heads, head_dim, block_size, dtype);
-  const bool fast = pl.ok && aligned16(q) && aligned16(k_cache) && aligned16(v_cache);
+  const bool fast = pl.ok && head_dim_v == head_dim && aligned16(q) && aligned16(k_cache) && aligned16(v_cache);
   if (fast) {
+    a.sub = block_size / kTok;
     const int sms = sm_count_cached();
     if (sms <= 0) return B200_ERR_NO_DEVICE;
     const size_t need = b200_paged_decode_gqa_workspace_bytes(batch, num_q_heads, num_kv_heads,
@@ -808,13 +827,37 @@ extern "C" int b200_paged_decode_gqa(const void* q, const void* k_cache, const v
     return launch_combine(a, batch, s);
   }
 
-  if (head_dim > kSimpleMaxPerLane * 32) return B200_ERR_UNSUPPORTED;
+  if (head_dim > kSimpleMaxPerLane * 32 || head_dim_v > kSimpleMaxPerLane * 32) return B200_ERR_UNSUPPORTED;
   dim3 grid(batch, num_q_heads);
   if (dtype == B200_DTYPE_F32)
     paged_decode_simple_kernel<float><<<grid, kSimpleWarps * 32, 0, s>>>(a);
   else
     paged_decode_simple_kernel<__nv_bfloat16><<<grid, kSimpleWarps * 32, 0, s>>>(a);
   return launch_result();
+}
+}  // namespace b200
+
+extern "C" int b200_paged_decode_gqa(const void* q, const void* k_cache, const void* v_cache,
+                                     void* out, const int32_t* block_tables, int64_t bt_stride,
+                                     const int64_t* context_lens, int32_t batch,
+                                     int32_t num_q_heads, int32_t num_kv_heads, int32_t head_dim,
+                                     int32_t block_size, int64_t num_blocks, float scale,
+                                     void* workspace, size_t workspace_bytes, int32_t dtype,
+                                     int32_t* status, void* stream) {
+  return b200::paged_decode(q, k_cache, v_cache, out, block_tables, bt_stride, context_lens, batch, num_q_heads,
+                            num_kv_heads, head_dim, head_dim, block_size, num_blocks, scale, nullptr, workspace,
+                            workspace_bytes, dtype, status, stream);
+}
+
+extern "C" int b200_paged_decode_sink(const void* q, const void* k_cache, const void* v_cache, void* out,
+                                      const int32_t* block_tables, int64_t bt_stride, const int64_t* context_lens,
+                                      int32_t batch, int32_t num_q_heads, int32_t num_kv_heads, int32_t head_dim_qk,
+                                      int32_t head_dim_v, int32_t block_size, int64_t num_blocks, float scale,
+                                      const float* sink, void* workspace, size_t workspace_bytes, int32_t dtype,
+                                      int32_t* status, void* stream) {
+  return b200::paged_decode(q, k_cache, v_cache, out, block_tables, bt_stride, context_lens, batch, num_q_heads,
+                            num_kv_heads, head_dim_qk, head_dim_v, block_size, num_blocks, scale, sink, workspace,
+                            workspace_bytes, dtype, status, stream);
 }
 
 // ---------------------------------------------------------------------------------------------

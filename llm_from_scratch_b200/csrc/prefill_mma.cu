@@ -41,6 +41,7 @@ struct MmaArgs {
   int64_t bt_stride;
   int bs;
   int64_t num_blocks;
+  const float* sink;     // [Hq] or null
   int32_t* status;
 };
 
@@ -291,6 +292,11 @@ __global__ void __launch_bounds__(kThreads, 2) prefill_mma_kernel(const MmaArgs 
   l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
   l1 += __shfl_xor_sync(0xffffffffu, l1, 1);
   l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
+  if (a.sink != nullptr) {
+    const float sink = a.sink[head];
+    l0 += sink_term(sink, m_r[0]);
+    l1 += sink_term(sink, m_r[1]);
+  }
   const float i0 = l0 > 0.f ? 1.f / l0 : 0.f, i1 = l1 > 0.f ? 1.f / l1 : 0.f;
   const int r0 = warp * 16 + g, r1 = r0 + 8;
   __nv_bfloat16* ob = a.out + (static_cast<int64_t>(q0 + m0) * a.Hq + head) * DV;
@@ -333,7 +339,7 @@ int prefill_mma_launch(const void* q, const void* k, const void* v, void* out, i
                        int Dqk, int Dv, float scale, const void* kc, const void* vc,
                        const int32_t* bt, int64_t bt_stride, int bs, int64_t num_blocks,
                        const int32_t* plan, int plan_tile_rows, int plan_capacity, int32_t* status,
-                       cudaStream_t s, const void* k_tail, int64_t k_tail_stride, int tail) {
+                       cudaStream_t s, const void* k_tail, int64_t k_tail_stride, int tail, const float* sink) {
   const bool paged = bt != nullptr;
   if (tail < 0 || tail % 8 || tail >= Dqk || (tail > 0 && (paged || !k_tail))) return B200_ERR_ARG;
   const bool shape_ok = (Dqk == Dv && (Dqk == 32 || Dqk == 64 || Dqk == 128)) ||
@@ -372,6 +378,7 @@ int prefill_mma_launch(const void* q, const void* k, const void* v, void* out, i
   a.bt_stride = bt_stride;
   a.bs = bs;
   a.num_blocks = num_blocks;
+  a.sink = sink;
   a.status = status;
   if (tail > 0) {   // compiled for MLA's split: 128 per-head columns + 64 shared
     if (Dqk != 192 || tail != 64) return B200_ERR_UNSUPPORTED;

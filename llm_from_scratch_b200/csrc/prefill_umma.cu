@@ -70,6 +70,7 @@ struct UmmaArgs {
   int64_t bt_stride;
   int bs;
   int64_t num_blocks;
+  const float* sink;     // [Hq] or null
   int32_t* status;
 };
 
@@ -406,6 +407,7 @@ prefill_umma_kernel(const UmmaArgs a, const __grid_constant__ CUtensorMap tm_q,
     }
     if (alive && __all_sync(0xffffffffu, umma::mbar_wait(bar(O_FINAL), 0, s_abort))) {
       umma::fence_after_sync();
+      if (a.sink != nullptr) l += sink_term(a.sink[x ? head_b : head_a], m_ref);
       const float inv = l > 0.f ? 1.f / l : 0.f;
       __nv_bfloat16* op = a.out + (static_cast<int64_t>(q0 + qrow) * a.Hq + (x ? head_b : head_a)) * D;
 #pragma unroll 1
@@ -481,7 +483,7 @@ int prefill_umma_launch(const void* q, const void* k, const void* v, void* out, 
                         const int32_t* cu_q, const int32_t* cu_k, int num_seqs, int max_seqlen_q, int Hq, int Hkv, int Dqk, int Dv, float scale,
                         const void* kc, const void* vc, const int32_t* bt, int64_t bt_stride, int bs,
                         int64_t num_blocks, const int32_t* plan, int plan_tile_rows, int plan_capacity,
-                        int32_t* status, cudaStream_t s) {
+                        int32_t* status, cudaStream_t s, const float* sink) {
   const bool paged = bt != nullptr;
   if (Dqk != D || Dv != D || Hkv <= 0 || Hq % Hkv != 0 || ((Hq / Hkv) & 1)) return B200_ERR_UNSUPPORTED;
   if (!(scale > 0.f)) return B200_ERR_UNSUPPORTED;   // the row maximum is taken before scaling
@@ -512,6 +514,7 @@ int prefill_umma_launch(const void* q, const void* k, const void* v, void* out, 
   a.bt_stride = bt_stride;
   a.bs = bs;
   a.num_blocks = num_blocks;
+  a.sink = sink;
   a.status = status;
   static bool configured[64][2] = {};
   int dev = 0;

@@ -74,6 +74,7 @@ struct Args2 {
   int Hq, Hkv, ntiles_max;
   const int32_t* plan;   // tile list for 256-row tiles (see b200_prefill_plan) or null: grid (head, seq, tile rank)
   float scale_log2;
+  const float* sink;     // [Hq] or null
   int32_t* status;
 };
 
@@ -365,6 +366,7 @@ prefill_umma2_kernel(const Args2 a, const __grid_constant__ CUtensorMap tm_q, co
       // the last product: stp / php are the stage and phase of tile nx - 1
       if (alive && __all_sync(0xffffffffu, umma::mbar_wait(pv_done + stp * 16, php, s_abort))) {
         umma::fence_after_sync();
+        if (a.sink != nullptr) l += sink_term(a.sink[head], m_ref);
         const float inv = l > 0.f ? 1.f / l : 0.f;
         __nv_bfloat16* op = a.out + (static_cast<int64_t>(q0 + qrow) * a.Hq + head) * DV;
 #pragma unroll 1
@@ -472,7 +474,7 @@ int prefill_umma2_launch(const void* q, const void* k, const void* v, void* out,
                          int64_t v_stride, int64_t total_q, int64_t total_k, const int32_t* cu_q,
                          const int32_t* cu_k, int num_seqs, int max_seqlen_q, int Hq, int Hkv, int Dqk, int Dv,
                          float scale, const int32_t* plan, int plan_tile_rows, int plan_capacity, int32_t* status,
-                         cudaStream_t s, const void* k_tail, int64_t k_tail_stride, int tail) {
+                         cudaStream_t s, const void* k_tail, int64_t k_tail_stride, int tail, const float* sink) {
   if (prefill_umma2_tile_rows(Hq, Hkv, Dqk, Dv) == 0) return B200_ERR_UNSUPPORTED;
   if (tail != 0 && (tail != 64 || Dqk != 192 || k_tail == nullptr)) return B200_ERR_UNSUPPORTED;
   if (!(scale > 0.f)) return B200_ERR_UNSUPPORTED;   // the row maximum is taken before scaling
@@ -490,6 +492,7 @@ int prefill_umma2_launch(const void* q, const void* k, const void* v, void* out,
   a.ntiles_max = ntiles;
   a.plan = (plan != nullptr && plan_tile_rows == ROWS && plan_capacity > 0 && plan_capacity <= 65535) ? plan : nullptr;
   a.scale_log2 = scale * 1.4426950408889634f;
+  a.sink = sink;
   a.status = status;
   CUtensorMap tq, tk, tkt, tv;
   memset(&tq, 0, sizeof(tq));

@@ -56,6 +56,7 @@ struct Args4 {
   int Hq, Hkv, ntiles_max;
   const int32_t* plan;   // tile list for 128-row tiles (see b200_prefill_plan) or null: grid (head group, seq, tile rank)
   float scale_log2;
+  const float* sink;     // [Hq] or null
   int32_t* status;
 };
 
@@ -308,6 +309,7 @@ prefill_umma4_kernel(const Args4 a, const __grid_constant__ CUtensorMap tm_q, co
       const uint32_t tOx = tmem + x * 128 + 64 + lane_sel;
       if (alive && __all_sync(0xffffffffu, umma::mbar_wait(bar(O_FINAL + x), 0, s_abort))) {
         umma::fence_after_sync();
+        if (a.sink != nullptr) l[pp] += sink_term(a.sink[head0 + x], m_ref[pp]);
         const float inv = l[pp] > 0.f ? 1.f / l[pp] : 0.f;
         __nv_bfloat16* op = a.out + (static_cast<int64_t>(q0 + qrow) * a.Hq + head0 + x) * D;
 #pragma unroll 1
@@ -389,7 +391,7 @@ int prefill_umma4_launch(const void* q, const void* k, const void* v, void* out,
                          int64_t v_stride, int64_t total_q, int64_t total_k, const int32_t* cu_q,
                          const int32_t* cu_k, int num_seqs, int max_seqlen_q, int Hq, int Hkv, int Dqk, int Dv,
                          float scale, const int32_t* plan, int plan_tile_rows, int plan_capacity, int32_t* status,
-                         cudaStream_t s) {
+                         cudaStream_t s, const float* sink) {
   if (prefill_umma4_tile_rows(Hq, Hkv, Dqk, Dv) == 0) return B200_ERR_UNSUPPORTED;
   if (!(scale > 0.f)) return B200_ERR_UNSUPPORTED;   // the row maximum is taken before scaling
   const int ntiles = (max_seqlen_q + BM - 1) / BM;
@@ -405,6 +407,7 @@ int prefill_umma4_launch(const void* q, const void* k, const void* v, void* out,
   a.ntiles_max = ntiles;
   a.plan = (plan != nullptr && plan_tile_rows == BM && plan_capacity > 0 && plan_capacity <= 65535) ? plan : nullptr;
   a.scale_log2 = scale * 1.4426950408889634f;
+  a.sink = sink;
   a.status = status;
   CUtensorMap tq, tk, tv;
   memset(&tq, 0, sizeof(tq));

@@ -25,6 +25,7 @@ struct PrefillArgs {
   int64_t bt_stride;
   int bs;
   int64_t num_blocks;
+  const float* sink;  // [Hq] or null
   int32_t* status;
 };
 
@@ -92,6 +93,7 @@ __global__ void __launch_bounds__(kWarps * 32) prefill_simple_kernel(const Prefi
     m = mn;
   }
   T* op = static_cast<T*>(a.out) + (static_cast<int64_t>(q0 + qi) * a.Hq + head) * a.Dv;
+  if (a.sink != nullptr && nkeys > 0) l += exp2f(a.sink[head] * 1.4426950408889634f - m);
   const float inv = l > 0.f ? 1.f / l : 0.f;
 #pragma unroll
   for (int i = 0; i < kMaxPerLane; ++i) {
@@ -110,7 +112,7 @@ int prefill_mma_launch(const void* q, const void* k, const void* v, void* out, i
                        int Dqk, int Dv, float scale, const void* kc, const void* vc,
                        const int32_t* bt, int64_t bt_stride, int bs, int64_t num_blocks,
                        const int32_t* plan, int plan_tile_rows, int plan_capacity, int32_t* status,
-                       cudaStream_t s, const void* k_tail = nullptr, int64_t k_tail_stride = 0, int tail = 0);
+                       cudaStream_t s, const void* k_tail, int64_t k_tail_stride, int tail, const float* sink);
 
 // tcgen05 path for packed keys/values (prefill_umma2.cu): head dims 128/128 and 192/128, 256 query rows of one head per CTA
 int prefill_umma2_tile_rows(int Hq, int Hkv, int Dqk, int Dv);
@@ -119,12 +121,12 @@ int prefill_umma4_launch(const void* q, const void* k, const void* v, void* out,
                          int64_t v_stride, int64_t total_q, int64_t total_k, const int32_t* cu_q,
                          const int32_t* cu_k, int num_seqs, int max_seqlen_q, int Hq, int Hkv, int Dqk, int Dv,
                          float scale, const int32_t* plan, int plan_tile_rows, int plan_capacity, int32_t* status,
-                         cudaStream_t s);
+                         cudaStream_t s, const float* sink);
 int prefill_umma2_launch(const void* q, const void* k, const void* v, void* out, int64_t q_stride, int64_t k_stride,
                          int64_t v_stride, int64_t total_q, int64_t total_k, const int32_t* cu_q,
                          const int32_t* cu_k, int num_seqs, int max_seqlen_q, int Hq, int Hkv, int Dqk, int Dv,
                          float scale, const int32_t* plan, int plan_tile_rows, int plan_capacity, int32_t* status,
-                         cudaStream_t s, const void* k_tail, int64_t k_tail_stride, int tail);
+                         cudaStream_t s, const void* k_tail, int64_t k_tail_stride, int tail, const float* sink);
 
 // tcgen05 path for a paged prefix (prefill_umma.cu): head_dim 128, even group size, two heads per CTA
 int prefill_umma_launch(const void* q, const void* k, const void* v, void* out, int64_t q_stride,
@@ -133,7 +135,7 @@ int prefill_umma_launch(const void* q, const void* k, const void* v, void* out, 
                         int num_seqs, int max_seqlen_q, int Hq, int Hkv, int Dqk, int Dv, float scale,
                         const void* kc, const void* vc, const int32_t* bt, int64_t bt_stride, int bs,
                         int64_t num_blocks, const int32_t* plan, int plan_tile_rows, int plan_capacity,
-                        int32_t* status, cudaStream_t s);
+                        int32_t* status, cudaStream_t s, const float* sink);
 
 }  // namespace b200
 
@@ -150,7 +152,7 @@ extern "C" int32_t b200_prefill_tile_rows(int32_t num_q_heads, int32_t num_kv_he
   return mma ? 64 : 0;
 }
 
-extern "C" int b200_prefill_varlen(const void* q, const void* k, const void* v, void* out,
+static int prefill_attention(const void* q, const void* k, const void* v, void* out,
                                    int64_t q_token_stride, int64_t k_token_stride,
                                    int64_t v_token_stride, int64_t total_q_tokens,
                                    int64_t total_k_tokens, const int32_t* cu_seqlens_q,
@@ -161,7 +163,7 @@ extern "C" int b200_prefill_varlen(const void* q, const void* k, const void* v, 
                                    const void* v_cache, const int32_t* block_tables,
                                    int64_t bt_stride, int32_t block_size, int64_t num_blocks,
                                    const int64_t* slot_mapping, const int32_t* plan, int32_t plan_tile_rows,
-                                   int32_t plan_capacity, int32_t dtype, int32_t* status, void* stream) {
+                                   int32_t plan_capacity, const float* sink, int32_t dtype, int32_t* status, void* stream) {
   using namespace b200;
   if (num_seqs < 0 || max_seqlen_q < 0 || max_seqlen_k < 0 || num_q_heads <= 0 ||
       num_kv_heads <= 0 || head_dim_qk <= 0 || head_dim_v <= 0)
@@ -199,26 +201,27 @@ extern "C" int b200_prefill_varlen(const void* q, const void* k, const void* v, 
       const int rc2 = prefill_umma2_launch(q, k, v, out, q_token_stride, k_token_stride, v_token_stride,
                                            total_q_tokens, total_k_tokens, cu_seqlens_q, cu_seqlens_k, num_seqs,
                                            max_seqlen_q, num_q_heads, num_kv_heads, head_dim_qk, head_dim_v, scale,
-                                           plan, plan_tile_rows, plan_capacity, status, s, nullptr, 0, 0);
+                                           plan, plan_tile_rows, plan_capacity, status, s, nullptr, 0, 0, sink);
       if (rc2 != B200_ERR_UNSUPPORTED) return rc2;
       // head_dim 64, four query heads of a KV head per CTA
       const int rc4 = prefill_umma4_launch(q, k, v, out, q_token_stride, k_token_stride, v_token_stride,
                                            total_q_tokens, total_k_tokens, cu_seqlens_q, cu_seqlens_k, num_seqs,
                                            max_seqlen_q, num_q_heads, num_kv_heads, head_dim_qk, head_dim_v, scale,
-                                           plan, plan_tile_rows, plan_capacity, status, s);
+                                           plan, plan_tile_rows, plan_capacity, status, s, sink);
       if (rc4 != B200_ERR_UNSUPPORTED) return rc4;
     }
     const int rcu = prefill_umma_launch(q, k, v, out, q_token_stride, k_token_stride, v_token_stride,
                                         total_q_tokens, total_k_tokens, cu_seqlens_q, cu_seqlens_k, num_seqs, max_seqlen_q, num_q_heads,
                                         num_kv_heads, head_dim_qk, head_dim_v, scale, k_cache, v_cache,
                                         block_tables, bt_stride, block_size, num_blocks, plan, plan_tile_rows,
-                                        plan_capacity, status, s);
+                                        plan_capacity, status, s, sink);
     if (rcu != B200_ERR_UNSUPPORTED) return rcu;
     const int rc = prefill_mma_launch(q, k, v, out, q_token_stride, k_token_stride,
                                       v_token_stride, cu_seqlens_q, cu_seqlens_k, num_seqs,
                                       max_seqlen_q, num_q_heads, num_kv_heads, head_dim_qk,
                                       head_dim_v, scale, k_cache, v_cache, block_tables, bt_stride,
-                                      block_size, num_blocks, plan, plan_tile_rows, plan_capacity, status, s);
+                                      block_size, num_blocks, plan, plan_tile_rows, plan_capacity, status, s,
+                                      nullptr, 0, 0, sink);
     if (rc != B200_ERR_UNSUPPORTED) return rc;
   }
 
@@ -246,6 +249,7 @@ extern "C" int b200_prefill_varlen(const void* q, const void* k, const void* v, 
   a.bt_stride = bt_stride;
   a.bs = block_size;
   a.num_blocks = num_blocks;
+  a.sink = sink;
   a.status = status;
   dim3 grid((max_seqlen_q + kWarps - 1) / kWarps, num_q_heads, num_seqs);
   if (dtype == B200_DTYPE_F32)
@@ -253,6 +257,44 @@ extern "C" int b200_prefill_varlen(const void* q, const void* k, const void* v, 
   else
     prefill_simple_kernel<__nv_bfloat16><<<grid, kWarps * 32, 0, s>>>(a);
   return launch_result();
+}
+
+extern "C" int b200_prefill_varlen(const void* q, const void* k, const void* v, void* out,
+                                   int64_t q_token_stride, int64_t k_token_stride,
+                                   int64_t v_token_stride, int64_t total_q_tokens,
+                                   int64_t total_k_tokens, const int32_t* cu_seqlens_q,
+                                   const int32_t* cu_seqlens_k, int32_t num_seqs,
+                                   int32_t max_seqlen_q, int32_t max_seqlen_k,
+                                   int32_t num_q_heads, int32_t num_kv_heads, int32_t head_dim_qk,
+                                   int32_t head_dim_v, float scale, const void* k_cache,
+                                   const void* v_cache, const int32_t* block_tables,
+                                   int64_t bt_stride, int32_t block_size, int64_t num_blocks,
+                                   const int64_t* slot_mapping, const int32_t* plan, int32_t plan_tile_rows,
+                                   int32_t plan_capacity, int32_t dtype, int32_t* status, void* stream) {
+  return prefill_attention(q, k, v, out, q_token_stride, k_token_stride, v_token_stride, total_q_tokens,
+                           total_k_tokens, cu_seqlens_q, cu_seqlens_k, num_seqs, max_seqlen_q, max_seqlen_k,
+                           num_q_heads, num_kv_heads, head_dim_qk, head_dim_v, scale, k_cache, v_cache, block_tables,
+                           bt_stride, block_size, num_blocks, slot_mapping, plan, plan_tile_rows, plan_capacity,
+                           nullptr, dtype, status, stream);
+}
+
+extern "C" int b200_prefill_varlen_sink(const void* q, const void* k, const void* v, void* out,
+                                   int64_t q_token_stride, int64_t k_token_stride,
+                                   int64_t v_token_stride, int64_t total_q_tokens,
+                                   int64_t total_k_tokens, const int32_t* cu_seqlens_q,
+                                   const int32_t* cu_seqlens_k, int32_t num_seqs,
+                                   int32_t max_seqlen_q, int32_t max_seqlen_k,
+                                   int32_t num_q_heads, int32_t num_kv_heads, int32_t head_dim_qk,
+                                   int32_t head_dim_v, float scale, const void* k_cache,
+                                   const void* v_cache, const int32_t* block_tables,
+                                   int64_t bt_stride, int32_t block_size, int64_t num_blocks,
+                                   const int64_t* slot_mapping, const int32_t* plan, int32_t plan_tile_rows,
+                                   int32_t plan_capacity, const float* sink, int32_t dtype, int32_t* status, void* stream) {
+  return prefill_attention(q, k, v, out, q_token_stride, k_token_stride, v_token_stride, total_q_tokens,
+                           total_k_tokens, cu_seqlens_q, cu_seqlens_k, num_seqs, max_seqlen_q, max_seqlen_k,
+                           num_q_heads, num_kv_heads, head_dim_qk, head_dim_v, scale, k_cache, v_cache, block_tables,
+                           bt_stride, block_size, num_blocks, slot_mapping, plan, plan_tile_rows, plan_capacity,
+                           sink, dtype, status, stream);
 }
 
 extern "C" int b200_prefill_varlen_shared_tail(const void* q, const void* k_head, const void* k_tail, const void* v,
@@ -277,10 +319,10 @@ extern "C" int b200_prefill_varlen_shared_tail(const void* q, const void* k_head
                                        total_q_tokens, total_k_tokens, cu_seqlens_q, cu_seqlens_k, num_seqs,
                                        max_seqlen_q, num_heads, num_heads, head_dim_qk, head_dim_v, scale, plan,
                                        plan_tile_rows, plan_capacity, status, static_cast<cudaStream_t>(stream),
-                                       k_tail, k_tail_token_stride, tail_dim);
+                                       k_tail, k_tail_token_stride, tail_dim, nullptr);
   if (rc2 != B200_ERR_UNSUPPORTED) return rc2;
   return prefill_mma_launch(q, k_head, v, out, q_token_stride, k_head_token_stride, v_token_stride, cu_seqlens_q,
                             cu_seqlens_k, num_seqs, max_seqlen_q, num_heads, num_heads, head_dim_qk, head_dim_v,
                             scale, nullptr, nullptr, nullptr, 0, 0, 0, plan, plan_tile_rows, plan_capacity, status,
-                            static_cast<cudaStream_t>(stream), k_tail, k_tail_token_stride, tail_dim);
+                            static_cast<cudaStream_t>(stream), k_tail, k_tail_token_stride, tail_dim, nullptr);
 }

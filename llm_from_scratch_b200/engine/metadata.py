@@ -31,6 +31,27 @@ class StepMetadata:
     last_token_index: Optional[np.ndarray] = None  # int64 [n]  row of each sequence's last token
     state_slots: Optional[np.ndarray] = None    # int64 [n]  recurrent-state slot of every sequence
 
+    def step_parts(self) -> "StepParts":
+        """A ragged step in two parts: the leading sequences that bring one token, and the others."""
+        q, k = np.diff(self.cu_seqlens_q), np.diff(self.cu_seqlens_k)
+        longer = np.nonzero(q != 1)[0]
+        n1 = int(longer[0]) if longer.size else len(q)
+        q, k, single = q[n1:], k[n1:], k[:n1]
+        return StepParts(num_single=n1, single_lens=single.astype(np.int64),
+                         portion_cu_k=np.concatenate([[0], np.cumsum(k)]).astype(np.int32),
+                         max_seqlen_q=int(q.max(initial=0)), max_seqlen_k=int(k.max(initial=0)),
+                         has_prefix=bool((q < k).any()))
+
+
+@dataclass
+class StepParts:
+    num_single: int
+    single_lens: np.ndarray                     # int64 [num_single]  context lengths, the new token included
+    portion_cu_k: np.ndarray                    # int32 [n - num_single + 1]  context offsets of the others, from 0
+    max_seqlen_q: int                           # over the others; 0 = there are none
+    max_seqlen_k: int
+    has_prefix: bool                            # some of their contexts began in an earlier step
+
 
 def block_table_array(s: Sequence) -> np.ndarray:
     """int32 copy of ``s.block_table`` kept on the sequence between steps.  The block manager only ever

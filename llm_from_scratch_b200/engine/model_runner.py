@@ -19,7 +19,7 @@ import torch
 
 from .. import ops
 from ..model import EngineTransformerLM, build_model, init_weights, resolve_config
-from ..utils.context import get_context, reset_context, set_context
+from ..utils.context import Portions, Singles, get_context, reset_context, set_context
 from ..utils.sampler import Sampler
 from . import metadata as md
 from .cache_pool import LayeredCache
@@ -102,6 +102,8 @@ class ModelRunner:
         # models with recurrent state hold a slot per live sequence; models with mixed batches take portions of
         # prompts beside decoded tokens and read every key from the pool
         self.recurrent_state, self.mixed_batches = model.recurrent_state, model.mixed_batches
+        # models that serve the single tokens of a mixed step with their decode kernels (Context.singles / portions)
+        self.splits_steps = getattr(model, "splits_steps", False)
         self.num_state_slots = self.max_num_seqs if self.recurrent_state else 0
         if self.mixed_batches:      # their matrix products accumulate in fp32 from end to end
             torch.backends.cuda.matmul.allow_bf16_reduced_precision_reduction = False
@@ -148,7 +150,8 @@ class ModelRunner:
             util = _cfg(self.config, "gpu_memory_utilization", default=0.5)
             if self.layered_cache is not None:
                 free -= self.num_state_slots * self.layered_cache.slot_bytes()
-            num_blocks = int(free * util) // self.kv_block_bytes()
+            # a model without paged rows still counts its tokens in blocks
+            num_blocks = int(free * util) // max(self.kv_block_bytes(), self.block_size)
         if num_blocks < 1:
             raise RuntimeError("not enough device memory for a single KV block")
         self.num_kv_blocks = int(num_blocks)
@@ -186,6 +189,9 @@ class ModelRunner:
             arrays["input_ids"] = np.concatenate([m.input_ids, np.zeros(pad, dtype=m.input_ids.dtype)])
             arrays["positions"] = np.concatenate([m.positions, np.zeros(pad, dtype=m.positions.dtype)])
             arrays["slot_mapping"] = np.concatenate([m.slot_mapping, np.full(pad, -1, dtype=m.slot_mapping.dtype)])
+        parts = m.step_parts() if self.splits_steps and m.is_prefill else None
+        if parts is not None:
+            arrays["single_lens"], arrays["portion_cu_k"] = parts.single_lens, parts.portion_cu_k
         t = self.staging.upload(arrays)
         plan = None
         if m.is_prefill and self.prefill_tile_rows and m.max_seqlen_q <= 4096 * self.prefill_tile_rows:
@@ -194,7 +200,25 @@ class ModelRunner:
         set_context(m.is_prefill, t.get("cu_seqlens_q"), t.get("cu_seqlens_k"), m.max_seqlen_q, m.max_seqlen_k,
                     t["slot_mapping"], t.get("context_lens"), t.get("block_tables"), t["positions"], plan,
                     t.get("state_slots"))
+        if self.splits_steps:
+            self._set_parts(get_context(), t, parts, len(m.input_ids))
         return t["input_ids"]
+
+    @staticmethod
+    def _set_parts(ctx, t: dict, parts: "md.StepParts | None", num_tokens: int) -> None:
+        """The context's two parts: leading single tokens and the portions behind them (a decode step: singles only)."""
+        slots = ctx.state_slots
+        if parts is None:
+            ctx.singles = Singles(ctx.context_lens.numel(), ctx.context_lens, ctx.block_tables, slots)
+            return
+        n1 = parts.num_single
+        part = lambda x, a, b=None: x[a:b] if x is not None else None
+        if n1:
+            ctx.singles = Singles(n1, t["single_lens"], ctx.block_tables[:n1], part(slots, 0, n1))
+        if parts.max_seqlen_q:
+            ctx.portions = Portions(num_tokens, ctx.cu_seqlens_q[n1:], t["portion_cu_k"], parts.max_seqlen_q,
+                                    parts.max_seqlen_k, int(parts.portion_cu_k[-1]), parts.has_prefix,
+                                    ctx.block_tables[n1:], part(slots, n1))
 
     def prepare_prefill(self, seqs: list[Sequence]) -> torch.Tensor:
         return self._publish(md.prepare_prefill(seqs, self.block_size, tables_always=self.mixed_batches))
@@ -502,6 +526,8 @@ class ModelRunner:
             # a padded row decodes position 0 of an empty context: its output row is never read
             set_context(False, slot_mapping=v["slot_mapping"][:b], context_lens=v["context_lens"][:b],
                         block_tables=v["block_tables"][:b], state_slots=v["state_slots"][:b])
+            if self.splits_steps:
+                self._set_parts(get_context(), {}, None, b)
             positions = (v["context_lens"][:b] - 1).clamp_min(0)
             v["outputs"][:b] = self.model(v["input_ids"][:b], positions)       # warm-up, allocates workspaces
             self.model.greedy_tokens(v["outputs"][:b], out=v["greedy"][:b])

@@ -47,7 +47,7 @@ class FusedProjection(nn.Module):
 
     align = 8
 
-    def __init__(self, parts: list[torch.Tensor]):
+    def __init__(self, parts: list[torch.Tensor], biases: list[torch.Tensor] | None = None):
         super().__init__()
         rows, self.columns, at = [], [], 0
         for w in parts:
@@ -58,10 +58,20 @@ class FusedProjection(nn.Module):
                 rows.append(torch.zeros(pad, w.shape[1], dtype=w.dtype, device=w.device))
             at += w.shape[0] + pad
         self.weight = torch.cat(rows).contiguous()
+        self.bias = None
+        if biases is not None:
+            self.bias = torch.zeros(at, dtype=self.weight.dtype, device=self.weight.device)
+            for (first, n), b in zip(self.columns, biases):
+                self.bias[first:first + n] = b
+
+    def whole(self, x: torch.Tensor) -> torch.Tensor:
+        return F.linear(x, self.weight, self.bias)
+
+    def split(self, y: torch.Tensor) -> list[torch.Tensor]:
+        return [y[:, at:at + n] for at, n in self.columns]
 
     def forward(self, x: torch.Tensor) -> list[torch.Tensor]:
-        y = F.linear(x, self.weight)
-        return [y[:, at:at + n] for at, n in self.columns]
+        return self.split(self.whole(x))
 
 
 class TalkingHeadsAttention(nn.Module):
@@ -179,3 +189,185 @@ class HyperConnection(nn.Module):
         self.read = p.f32(f"hc{q}.in", (streams,))
         self.mix = p.f32(f"hc{q}.mix", (streams, streams))
         self.write = p.f32(f"hc{q}.out", (streams,))
+
+
+# ------------------------------------------------------------------------------------------------
+# mixers that serve the leading single tokens of a step with their decode kernels (Context.singles / portions)
+# ------------------------------------------------------------------------------------------------
+def _step_output(x: torch.Tensor, width: int, ctx) -> torch.Tensor:
+    """Output rows [T, width] of a step for kernels that write the rows of its sequences; padding rows are zero, so that
+    what a later tile loads next to a sequence's last row is finite."""
+    out = torch.empty(x.shape[0], width, dtype=x.dtype, device=x.device)
+    if ctx.portions is not None and ctx.portions.num_tokens < x.shape[0]:
+        out[ctx.portions.num_tokens:].zero_()
+    elif ctx.portions is None and ctx.singles.rows < x.shape[0]:
+        out[ctx.singles.rows:].zero_()
+    return out
+
+
+def _heads(x: torch.Tensor, heads: int, dim: int) -> torch.Tensor:
+    """[T, heads * dim] columns of a projection as [T, heads, dim]; a view, also of strided rows."""
+    return x.unflatten(1, (heads, dim))
+
+
+class GatedDeltaRule(nn.Module):
+    """Gated delta rule behind a short convolution, with an output norm and a silu gate (``b200_delta_rule`` /
+    ``b200_delta_step``); the fp32 state and the convolution's last inputs live in the runner's slot pools."""
+
+    def __init__(self, p: Params, d_model: int, heads: int, kv_heads: int, dim: int, vdim: int, taps: int, eps: float):
+        super().__init__()
+        sizes = {"q": kv_heads * dim, "k": kv_heads * dim, "v": heads * vdim}
+        self.project = FusedProjection([p.lin(n, (w, d_model)) for n, w in sizes.items()]
+                                       + [p.lin("g", (heads * vdim, d_model)), p.lin("b", (heads, d_model)),
+                                          p.lin("a", (heads, d_model))])
+        columns = self.project.columns
+        width = columns[3][0]
+        conv = torch.zeros(taps, width, device=p.device)
+        for (at, n), name in zip(columns, sizes):
+            conv[:, at:at + n] = p.f32(name + ".conv", (n, taps)).t()
+        self.rule = ops.DeltaRule(heads, kv_heads, dim, vdim, tuple(at for at, _ in columns[:3]), conv,
+                                  p.f32("dt_bias", (heads,)), p.f32("A_log", (heads,)), p.f32("norm", (vdim,)), eps)
+        self.w_o = p.lin("o", (d_model, heads * vdim))
+        self.state = self.conv_ring = torch.empty(0)
+
+    def cache_needs(self):
+        c = self.rule
+        return [("slot", "state", (c.heads, c.dim, c.vdim)), ("slot", "conv_ring", (c.taps, c.width))]
+
+    def forward(self, h, ctx, positions):
+        y = self.project.whole(h)
+        _, _, _, g, b, a = self.project.split(y)
+        o = _step_output(y, self.rule.heads * self.rule.vdim, ctx)
+        if ctx.singles is not None:
+            s = ctx.singles
+            ops.delta_step(self.rule, y, b, a, g, self.state, self.conv_ring, s.state_slots, s.context_lens, out=o)
+        if ctx.portions is not None:
+            s = ctx.portions
+            ops.delta_rule(self.rule, y, b, a, g, self.state, self.conv_ring, s.state_slots, s.cu_seqlens_q,
+                           s.cu_seqlens_k, out=o)
+        return F.linear(o, self.w_o)
+
+
+def _portion_attention(q, k, v, k_cache, v_cache, ctx, scale, out, sink=None):
+    """Attention of the step's portions: over the step's own packed keys when every context starts in this step, else
+    over the pool."""
+    s, H, Hkv, dk, dv = ctx.portions, q.shape[1], v.shape[1], q.shape[2], v.shape[2]
+    if s.has_prefix:
+        plan = s.plan(ops.prefill_tile_rows(H, Hkv, dk, dv, q.dtype, paged=True))
+        ops.prefill_varlen(q, None, None, s.cu_seqlens_q, s.cu_seqlens_k, s.max_seqlen_q, s.max_seqlen_k, scale, k_cache,
+                           v_cache, s.block_tables, out=out, plan=plan, sink=sink)
+    else:
+        plan = s.plan(ops.prefill_tile_rows(H, Hkv, dk, dv, q.dtype))
+        ops.prefill_varlen(q, k, v, s.cu_seqlens_q, s.cu_seqlens_q, s.max_seqlen_q, s.max_seqlen_q, scale, out=out, plan=plan,
+                           sink=sink)
+
+
+class SinkAttention(nn.Module):
+    """Grouped-query attention with biased projections, a norm per query / key head, interleaved rotation of the first
+    channels and a learned sink in the softmax denominator."""
+
+    def __init__(self, p: Params, d_model: int, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, rot_dims: int,
+                 rot_base: float, eps: float):
+        super().__init__()
+        self.heads, self.kv_heads, self.dim, self.vdim, self.scale, self.eps = heads, kv_heads, dim, vdim, scale, eps
+        sizes = {"q": heads * dim, "k": kv_heads * dim, "v": kv_heads * vdim}
+        self.project = FusedProjection([p.lin(n, (w, d_model)) for n, w in sizes.items()],
+                                       [p.lin(n + ".b", (w,)) for n, w in sizes.items()])
+        self.q_norm, self.k_norm = p.f32("q.norm", (dim,)), p.f32("k.norm", (dim,))
+        self.sink = p.f32("sink", (heads,))
+        self.freq = ops.rotary_frequencies(rot_base, rot_dims, p.device)
+        self.w_o = p.lin("o", (d_model, heads * vdim))
+        self.k_cache = self.v_cache = torch.empty(0)
+
+    def cache_needs(self):
+        return [("paged", "k_cache", (self.kv_heads, self.dim)), ("paged", "v_cache", (self.kv_heads, self.vdim))]
+
+    def forward(self, h, ctx, positions):
+        q, k, v = self.project(h)
+        T = h.shape[0]
+        q, k = ops.head_norm_rope_store(q, k, v, self.q_norm, self.k_norm, self.eps, self.freq, positions, self.k_cache,
+                                        self.v_cache, ctx.slot_mapping)
+        o = _step_output(h, self.heads * self.vdim, ctx)
+        o3 = o.view(T, self.heads, self.vdim)
+        if ctx.singles is not None:
+            s = ctx.singles
+            ops.paged_decode_gqa(q[:s.rows], self.k_cache, self.v_cache, s.block_tables, s.context_lens, self.scale,
+                                 out=o3[:s.rows], sink=self.sink)
+        if ctx.portions is not None:
+            _portion_attention(q, k, _heads(v, self.kv_heads, self.vdim), self.k_cache, self.v_cache, ctx, self.scale, o3, self.sink)
+        return F.linear(o, self.w_o)
+
+
+class LatentAttention(nn.Module):
+    """Attention over cached latent rows without positions, with an output gate.  Single tokens attend in the absorbed
+    form (queries and results pass through W_uk / W_uv, keys and values are the latent rows themselves); portions expand
+    the rows of their contexts.  ``source``: another layer whose latent rows this one reads instead of its own."""
+
+    def __init__(self, p: Params, d_model: int, heads: int, dim: int, vdim: int, kv_rank: int, scale: float, eps: float,
+                 source: "LatentAttention | None" = None):
+        super().__init__()
+        self.heads, self.dim, self.vdim, self.rank, self.scale, self.eps = heads, dim, vdim, kv_rank, scale, eps
+        parts = [p.lin("q", (heads * dim, d_model)), p.lin("g", (heads * vdim, d_model))]
+        self.source = [source] if source is not None else []         # in a list: not a submodule of this layer
+        if source is None:
+            parts.append(p.lin("dkv", (kv_rank, d_model)))
+            self.norm = p.f32("dkv.norm", (kv_rank,))
+        elif source.source or source.rank != kv_rank:
+            raise ValueError("a layer can share the latent rows of a layer that has its own, of the same rank")
+        self.project = FusedProjection(parts)
+        uk, uv = p.lin("uk", (heads * dim, kv_rank)), p.lin("uv", (heads * vdim, kv_rank))
+        self.expand = FusedProjection([uk, uv])
+        self.w_uk = uk.view(heads, dim, kv_rank)
+        self.w_uv_t = uv.view(heads, vdim, kv_rank).transpose(1, 2)
+        self.w_o = p.lin("o", (d_model, heads * vdim))
+        self.latent_cache = torch.empty(0)
+        self.step_rows = None            # latent rows of the running step's tokens
+        self.context_rows = None         # and of its portions' contexts, when some of those began in an earlier step
+
+    def cache_needs(self):
+        return [] if self.source else [("paged", "latent_cache", (self.rank,))]
+
+    def _absorbed(self, q, s, o):
+        n, H = s.rows, self.heads
+        owner = self.source[0] if self.source else self
+        q_abs = torch.empty(n, H, self.rank, dtype=q.dtype, device=q.device)
+        q3 = _heads(q, H, self.dim)[:n]
+        torch.bmm(q3.transpose(0, 1), self.w_uk, out=q_abs.transpose(0, 1))
+        lat = ops.mla_decode(q_abs, None, owner.latent_cache, s.block_tables, s.context_lens, self.scale)
+        torch.bmm(lat.transpose(0, 1), self.w_uv_t, out=o[:n].view(n, H, self.vdim).transpose(0, 1))
+
+    def _expanded(self, q, ctx, o):
+        s, H = ctx.portions, self.heads
+        owner = self.source[0] if self.source else self
+        rows, cu_k, max_k = owner.step_rows, s.cu_seqlens_q, s.max_seqlen_q
+        if s.has_prefix:
+            if owner.context_rows is None:
+                owner.context_rows = ops.gather_rows(owner.latent_cache, s.block_tables, s.cu_seqlens_k, s.max_seqlen_k, s.total_k)
+            rows, cu_k, max_k = owner.context_rows, s.cu_seqlens_k, s.max_seqlen_k
+        k, v = self.expand(rows)
+        ops.prefill_varlen(_heads(q, H, self.dim), _heads(k, H, self.dim), _heads(v, H, self.vdim), s.cu_seqlens_q, cu_k, s.max_seqlen_q,
+                           max_k, self.scale, out=o.view(-1, H, self.vdim),
+                           plan=s.plan(ops.prefill_tile_rows(H, H, self.dim, self.vdim, q.dtype)))
+
+    def forward(self, h, ctx, positions):
+        q, g, *down = self.project(h)
+        if down:
+            self.step_rows = ops.latent_norm_store(down[0], self.norm, self.eps, self.latent_cache, ctx.slot_mapping)
+            self.context_rows = None
+        o = _step_output(h, self.heads * self.vdim, ctx)
+        if ctx.singles is not None:
+            self._absorbed(q, ctx.singles, o)
+        if ctx.portions is not None:
+            self._expanded(q, ctx, o)
+        return F.linear(ops.sigmoid_gate(o, g), self.w_o)
+
+
+class SquaredReLU(nn.Module):
+    """W_down max(W_up h, 0)^2."""
+
+    def __init__(self, p: Params, d_model: int, d_ff: int):
+        super().__init__()
+        self.w_up, self.w_down = p.lin("up", (d_ff, d_model)), p.lin("down", (d_model, d_ff))
+
+    def forward(self, h, ctx, positions):
+        return F.linear(ops.squared_relu(F.linear(h, self.w_up)), self.w_down)

@@ -151,16 +151,19 @@ def store_rows(rows: torch.Tensor, cache: torch.Tensor, slot_mapping: torch.Tens
 
 def paged_decode_gqa(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                      block_tables: torch.Tensor, context_lens: torch.Tensor, scale: float,
-                     out: torch.Tensor | None = None) -> torch.Tensor:
+                     out: torch.Tensor | None = None, sink: torch.Tensor | None = None) -> torch.Tensor:
     """One query token per sequence over a paged KV pool.
 
-    q: [B, Hq, D]; caches: [num_blocks, block_size, Hkv, D]; block_tables: [B, maxb] int32;
-    context_lens: [B] int64.  Returns out [B, Hq, D].
+    q: [B, Hq, D]; caches: [num_blocks, block_size, Hkv, D] (value heads may have a size of their own);
+    block_tables: [B, maxb] int32; context_lens: [B] int64; ``sink`` fp32 [Hq]: exp(sink) joins the softmax
+    denominator.  Returns out [B, Hq, Dv].
     """
-    dev = _cuda(q, k_cache, v_cache, block_tables, context_lens, out)
+    dev = _cuda(q, k_cache, v_cache, block_tables, context_lens, out, sink)
     B, Hq, D = q.shape
     nb, bs, Hkv, Dc = k_cache.shape
-    if Dc != D or v_cache.shape != k_cache.shape or k_cache.dtype != q.dtype or v_cache.dtype != q.dtype:
+    Dv = v_cache.shape[3]
+    _f32vec("sink", sink, Hq)
+    if Dc != D or v_cache.shape[:3] != k_cache.shape[:3] or k_cache.dtype != q.dtype or v_cache.dtype != q.dtype:
         raise ValueError("cache shape/dtype does not match q")
     if block_tables.dtype != torch.int32 or context_lens.dtype != torch.int64:
         raise ValueError("block_tables must be int32 and context_lens int64")
@@ -171,11 +174,17 @@ def paged_decode_gqa(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
     if not (q.is_contiguous() and k_cache.is_contiguous() and v_cache.is_contiguous()):
         raise ValueError("q and caches must be contiguous")
     if out is None:
-        out = torch.empty_like(q)
-    elif out.shape != q.shape or out.dtype != q.dtype or not out.is_contiguous():
-        raise ValueError("out must match q")
+        out = torch.empty((B, Hq, Dv), dtype=q.dtype, device=q.device)
+    elif out.shape != (B, Hq, Dv) or out.dtype != q.dtype or not out.is_contiguous():
+        raise ValueError("out must be a contiguous [B, Hq, Dv] tensor of q's dtype")
     need = lib.b200_paged_decode_gqa_workspace_bytes(B, Hq, Hkv, D, _dt(q))
     ws = workspace(dev, need, "decode")
+    if sink is not None or Dv != D:
+        check(lib.b200_paged_decode_sink(q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(),
+                                         block_tables.data_ptr(), block_tables.stride(0), context_lens.data_ptr(), B, Hq,
+                                         Hkv, D, Dv, bs, nb, float(scale), _ptr(sink), ws.data_ptr(), ws.numel(), _dt(q),
+                                         status_word(dev).data_ptr(), _stream()), "paged_decode_sink")
+        return out
     check(lib.b200_paged_decode_gqa(q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(),
                                     out.data_ptr(), block_tables.data_ptr(),
                                     block_tables.stride(0), context_lens.data_ptr(), B, Hq, Hkv, D,
@@ -189,8 +198,8 @@ def prefill_varlen(q: torch.Tensor, k: torch.Tensor | None, v: torch.Tensor | No
                    max_seqlen_k: int, scale: float, k_cache: torch.Tensor | None = None,
                    v_cache: torch.Tensor | None = None, block_tables: torch.Tensor | None = None,
                    out: torch.Tensor | None = None, plan: "PrefillPlan | None" = None,
-                   slot_mapping: torch.Tensor | None = None) -> torch.Tensor:
-    """Causal attention over packed ragged sequences.
+                   slot_mapping: torch.Tensor | None = None, sink: torch.Tensor | None = None) -> torch.Tensor:
+    """Causal attention over packed ragged sequences.  ``sink`` (fp32 [Hq]): exp(sink) joins the softmax denominator.
 
     ``slot_mapping`` (int64, one slot per row of k / v): the same call first scatters the new tokens' k / v
     rows into ``k_cache`` / ``v_cache`` (the step's store_kvcache), with or without ``block_tables``.
@@ -255,15 +264,17 @@ def prefill_varlen(q: torch.Tensor, k: torch.Tensor | None, v: torch.Tensor | No
         out = torch.empty((Tq, Hq, Dv), dtype=q.dtype, device=q.device)
     elif out.shape != (Tq, Hq, Dv) or out.dtype != q.dtype or not out.is_contiguous():
         raise ValueError("out must be a contiguous [Tq, Hq, Dv] tensor")
-    check(lib.b200_prefill_varlen(q.data_ptr(), kp, vp, out.data_ptr(), q.stride(0), ks, vs, Tq, total_k,
-                                  cu_seqlens_q.data_ptr(), cu_seqlens_k.data_ptr(), num_seqs,
-                                  int(max_seqlen_q), int(max_seqlen_k), Hq, Hkv, Dqk, Dv,
-                                  float(scale), kcp, vcp, btp, bts, bs, nb,
-                                  slot_mapping.data_ptr() if slot_mapping is not None else None,
-                                  plan.buffer.data_ptr() if plan is not None else None,
-                                  plan.tile_rows if plan is not None else 0,
-                                  plan.capacity if plan is not None else 0, _dt(q),
-                                  status_word(dev).data_ptr(), _stream()), "prefill_varlen")
+    args = (q.data_ptr(), kp, vp, out.data_ptr(), q.stride(0), ks, vs, Tq, total_k, cu_seqlens_q.data_ptr(),
+            cu_seqlens_k.data_ptr(), num_seqs, int(max_seqlen_q), int(max_seqlen_k), Hq, Hkv, Dqk, Dv, float(scale), kcp,
+            vcp, btp, bts, bs, nb, _ptr(slot_mapping), plan.buffer.data_ptr() if plan is not None else None,
+            plan.tile_rows if plan is not None else 0, plan.capacity if plan is not None else 0)
+    tail = (_dt(q), status_word(dev).data_ptr(), _stream())
+    if sink is not None:
+        _cuda(q, sink)
+        _f32vec("sink", sink, Hq)
+        check(lib.b200_prefill_varlen_sink(*args, sink.data_ptr(), *tail), "prefill_varlen_sink")
+    else:
+        check(lib.b200_prefill_varlen(*args, *tail), "prefill_varlen")
     return out
 
 
@@ -313,10 +324,15 @@ class PrefillPlan:
         self.buffer, self.tile_rows, self.capacity = buffer, tile_rows, capacity
 
 
-def prefill_tile_rows(Hq: int, Hkv: int, Dqk: int, Dv: int, dtype: torch.dtype) -> int:
-    """Query rows per tile of the prefill kernel serving this shape; 0 = no tiled kernel (no plan)."""
+def prefill_tile_rows(Hq: int, Hkv: int, Dqk: int, Dv: int, dtype: torch.dtype, paged: bool = False) -> int:
+    """Query rows per tile of the prefill kernel serving this shape with packed (or ``paged``) keys; 0 = no tiled kernel
+    (no plan)."""
     if dtype not in _DTYPES:
         return 0
+    if paged and dtype == torch.bfloat16:
+        if Dqk == Dv == 128 and Hq // Hkv % 2 == 0:
+            return 128                                  # two-head tcgen05 kernel
+        return 64 if (Dqk == Dv and Dqk in (32, 64, 128)) or (Dqk, Dv) == (192, 128) else 0
     return int(lib.b200_prefill_tile_rows(Hq, Hkv, Dqk, Dv, _DTYPES[dtype]))
 
 
@@ -341,33 +357,33 @@ def prefill_plan(cu_seqlens_q: torch.Tensor, total_q_tokens: int, max_seqlen_q: 
     return PrefillPlan(buffer, tile_rows, buffer.numel() - 4)
 
 
-def mla_decode(q_abs: torch.Tensor, q_rope: torch.Tensor, latent_cache: torch.Tensor,
+def mla_decode(q_abs: torch.Tensor, q_rope: torch.Tensor | None, latent_cache: torch.Tensor,
                block_tables: torch.Tensor, context_lens: torch.Tensor, scale: float,
                out: torch.Tensor | None = None) -> torch.Tensor:
     """Absorbed MLA decode over a paged latent pool.
 
-    q_abs: [B, H, r]; q_rope: [B, H, dr]; latent_cache: [num_blocks, block_size, r + dr];
+    q_abs: [B, H, r]; q_rope: [B, H, dr] or None (dr = 0); latent_cache: [num_blocks, block_size, r + dr];
     returns the attention-weighted latent [B, H, r].
     """
     dev = _cuda(q_abs, q_rope, latent_cache, block_tables, context_lens, out)
     B, H, r = q_abs.shape
-    dr = q_rope.shape[2]
+    dr = q_rope.shape[2] if q_rope is not None else 0
     nb, bs, row = latent_cache.shape
-    if row != r + dr or q_rope.shape[:2] != (B, H):
+    if row != r + dr or (q_rope is not None and q_rope.shape[:2] != (B, H)):
         raise ValueError("latent row must be kv_lora_rank + rope_dim wide")
-    if latent_cache.dtype != q_abs.dtype or q_rope.dtype != q_abs.dtype:
+    if latent_cache.dtype != q_abs.dtype or (q_rope is not None and q_rope.dtype != q_abs.dtype):
         raise ValueError("dtype mismatch")
     if block_tables.dtype != torch.int32 or context_lens.dtype != torch.int64:
         raise ValueError("block_tables must be int32 and context_lens int64")
     if block_tables.shape[0] != B or block_tables.stride(1) != 1 or context_lens.numel() != B:
         raise ValueError("metadata batch mismatch")
-    if not (q_abs.is_contiguous() and q_rope.is_contiguous() and latent_cache.is_contiguous()):
+    if not (q_abs.is_contiguous() and (q_rope is None or q_rope.is_contiguous()) and latent_cache.is_contiguous()):
         raise ValueError("inputs must be contiguous")
     if out is None:
         out = torch.empty_like(q_abs)
     need = lib.b200_mla_decode_workspace_bytes(B, H, r, dr, _dt(q_abs))
     ws = workspace(dev, need, "mla")
-    check(lib.b200_mla_decode(q_abs.data_ptr(), q_rope.data_ptr(), latent_cache.data_ptr(),
+    check(lib.b200_mla_decode(q_abs.data_ptr(), _ptr(q_rope), latent_cache.data_ptr(),
                               out.data_ptr(), block_tables.data_ptr(), block_tables.stride(0),
                               context_lens.data_ptr(), B, H, r, dr, bs, nb, float(scale),
                               ws.data_ptr(), ws.numel(), _dt(q_abs), status_word(dev).data_ptr(),
@@ -901,4 +917,217 @@ def gated_recurrence(q: torch.Tensor, f: torch.Tensor, v: torch.Tensor, f_bias: 
         float(eps), state.data_ptr(), slots, state_slots.data_ptr(), _ptr(cu_seqlens_q), _ptr(cu_seqlens_k),
         _ptr(context_lens), n, T, int(max_seqlen_q), H, dk, dv, out.data_ptr(), _ptr(ws),
         ws.numel() if ws is not None else 0, _dt(q), status_word(dev).data_ptr(), _stream()), "gated_recurrence")
+    return out
+
+
+# ------------------------------------------------------------------------------------------------
+# post-norm residual, per-head norms with interleaved rotation, latent rows, gated delta rule
+# ------------------------------------------------------------------------------------------------
+def residual_norm(x: torch.Tensor, eps: float, dtype: torch.dtype, *, tokens: torch.Tensor | None = None,
+                  embed: torch.Tensor | None = None, y: torch.Tensor | None = None, norm_w: torch.Tensor | None = None,
+                  final_w: torch.Tensor | None = None) -> torch.Tensor:
+    """One sublayer boundary with a norm on the sublayer's output (``b200_residual_norm``): x [T, d] fp32 takes the normed
+    ``y`` (or starts as the rows ``tokens`` of ``embed``) in place; returns x, or its norm with ``final_w``, in ``dtype``."""
+    dev = _cuda(x, tokens, embed, y, norm_w, final_w)
+    T, d = x.shape
+    if x.dtype != torch.float32 or not x.is_contiguous():
+        raise ValueError("x must be a contiguous fp32 [T, d] tensor")
+    _f32vec("norm_w", norm_w, d)
+    _f32vec("final_w", final_w, d)
+    if embed is not None:
+        if embed.shape[1] != d or embed.dtype != dtype or not embed.is_contiguous() or tokens is None \
+                or tokens.dtype != torch.int64 or tokens.numel() != T:
+            raise ValueError("embed must be contiguous [vocab, d] in the activation dtype, tokens int64 [T]")
+    elif y is None or norm_w is None or y.shape != (T, d) or y.dtype != dtype or not y.is_contiguous():
+        raise ValueError("y must be contiguous [T, d] in the activation dtype, with its norm weight")
+    h = torch.empty(T, d, dtype=dtype, device=x.device)
+    check(lib.b200_residual_norm(x.data_ptr(), _ptr(tokens) if embed is not None else None, _ptr(embed),
+                                 embed.shape[0] if embed is not None else 0, _ptr(y), _ptr(norm_w), _ptr(final_w), float(eps),
+                                 h.data_ptr(), T, d, _dt(h), status_word(dev).data_ptr(), _stream()), "residual_norm")
+    return h
+
+
+def rotary_frequencies(base: float, dims: int, device) -> torch.Tensor:
+    """base^(-2i / dims), i < dims / 2, in fp64."""
+    i = torch.arange(dims // 2, dtype=torch.float64)
+    return (float(base) ** (-2.0 * i / max(dims, 1))).to(device)
+
+
+def head_norm_rope_store(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, q_norm_w: torch.Tensor, k_norm_w: torch.Tensor,
+                         eps: float, freq: torch.Tensor, positions: torch.Tensor, k_cache: torch.Tensor,
+                         v_cache: torch.Tensor, slot_mapping: torch.Tensor):
+    """Norm of every query / key head, interleaved rotation of its first 2 * freq.numel() channels, scatter of k and v
+    (``b200_head_norm_rope_store``).  q [T, Hq * D], k [T, Hkv * D], v [T, Hkv * Dv] are views of one projection; caches
+    [num_blocks, block_size, Hkv, D*].  Returns (q [T, Hq, D], k [T, Hkv, D])."""
+    dev = _cuda(q, k, v, q_norm_w, k_norm_w, freq, positions, k_cache, v_cache, slot_mapping)
+    T, D = q.shape[0], q_norm_w.numel()
+    nb, bs, Hkv, Dc = k_cache.shape
+    Dv, Hq = v_cache.shape[3], q.shape[1] // D
+    if Dc != D or v_cache.shape[:3] != (nb, bs, Hkv) or not k_cache.is_contiguous() or not v_cache.is_contiguous() \
+            or k_cache.dtype != q.dtype or v_cache.dtype != q.dtype:
+        raise ValueError("caches must be contiguous [num_blocks, block_size, Hkv, d] of q's dtype")
+    if q.shape != (T, Hq * D) or k.shape != (T, Hkv * D) or v.shape != (T, Hkv * Dv) or any(
+            t.stride(1) != 1 or t.stride(0) != q.stride(0) or t.dtype != q.dtype for t in (q, k, v)):
+        raise ValueError("q, k, v must share dtype and row stride")
+    _f32vec("q_norm_w", q_norm_w, D)
+    _f32vec("k_norm_w", k_norm_w, D)
+    if freq.dtype != torch.float64 or not freq.is_contiguous():
+        raise ValueError("freq must be contiguous fp64")
+    for name, t in (("positions", positions), ("slot_mapping", slot_mapping)):
+        if t.dtype != torch.int64 or t.numel() != T or not t.is_contiguous():
+            raise ValueError(f"{name} must be contiguous int64 with one entry per token")
+    qo = torch.empty(T, Hq, D, dtype=q.dtype, device=q.device)
+    ko = torch.empty(T, Hkv, D, dtype=q.dtype, device=q.device)
+    check(lib.b200_head_norm_rope_store(
+        q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), q_norm_w.data_ptr(), k_norm_w.data_ptr(), float(eps),
+        freq.data_ptr(), 2 * freq.numel(), positions.data_ptr(), qo.data_ptr(), ko.data_ptr(), k_cache.data_ptr(),
+        v_cache.data_ptr(), slot_mapping.data_ptr(), nb * bs, T, Hq, Hkv, D, Dv, _dt(q), status_word(dev).data_ptr(),
+        _stream()), "head_norm_rope_store")
+    return qo, ko
+
+
+def latent_norm_store(rows: torch.Tensor, norm_w: torch.Tensor, eps: float, cache: torch.Tensor,
+                      slot_mapping: torch.Tensor) -> torch.Tensor:
+    """RMS norm of latent rows [T, r] (row stride free), written to cache[slot_mapping] and returned [T, r]."""
+    dev = _cuda(rows, norm_w, cache, slot_mapping)
+    T, r = rows.shape
+    _f32vec("norm_w", norm_w, r)
+    if rows.stride(1) != 1 or cache.shape[-1] != r or cache.dtype != rows.dtype or not cache.is_contiguous():
+        raise ValueError("rows/cache shape, dtype or layout mismatch")
+    if slot_mapping.dtype != torch.int64 or slot_mapping.numel() != T or not slot_mapping.is_contiguous():
+        raise ValueError("slot_mapping must be a contiguous int64 tensor with one entry per row")
+    out = torch.empty(T, r, dtype=rows.dtype, device=rows.device)
+    check(lib.b200_latent_norm_store(rows.data_ptr(), rows.stride(0), norm_w.data_ptr(), float(eps), out.data_ptr(),
+                                     cache.data_ptr(), slot_mapping.data_ptr(), cache.numel() // r, T, r, _dt(rows),
+                                     status_word(dev).data_ptr(), _stream()), "latent_norm_store")
+    return out
+
+
+def gather_rows(cache: torch.Tensor, block_tables: torch.Tensor, cu_seqlens_k: torch.Tensor, max_seqlen_k: int,
+                total: int) -> torch.Tensor:
+    """Rows of whole contexts, packed [total, W], from a pool [num_blocks, block_size, W] through the block tables."""
+    dev = _cuda(cache, block_tables, cu_seqlens_k)
+    nb, bs, W = cache.shape
+    n = cu_seqlens_k.numel() - 1
+    if not cache.is_contiguous() or block_tables.dtype != torch.int32 or block_tables.shape[0] < n \
+            or block_tables.stride(1) != 1 or cu_seqlens_k.dtype != torch.int32:
+        raise ValueError("cache must be contiguous, block_tables int32 [n, max_blocks], cu_seqlens_k int32 [n + 1]")
+    out = torch.empty(total, W, dtype=cache.dtype, device=cache.device)
+    check(lib.b200_gather_rows(cache.data_ptr(), bs, nb, W * cache.element_size(), block_tables.data_ptr(),
+                               block_tables.stride(0), cu_seqlens_k.data_ptr(), n, int(max_seqlen_k), out.data_ptr(), total,
+                               status_word(dev).data_ptr(), _stream()), "gather_rows")
+    return out
+
+
+def sigmoid_gate(o: torch.Tensor, gate: torch.Tensor) -> torch.Tensor:
+    """o * sigmoid(gate) in place; o contiguous [T, W], gate [T, W] with a free row stride."""
+    _cuda(o, gate)
+    if o.shape != gate.shape or not o.is_contiguous() or gate.stride(1) != 1 or gate.dtype != o.dtype:
+        raise ValueError("o must be contiguous [T, W] and gate [T, W] of its dtype with contiguous rows")
+    check(lib.b200_sigmoid_gate(o.data_ptr(), gate.data_ptr(), gate.stride(0), o.shape[0], o.shape[1], _dt(o), _stream()),
+          "sigmoid_gate")
+    return o
+
+
+def squared_relu(x: torch.Tensor) -> torch.Tensor:
+    """max(x, 0)^2 in place."""
+    _cuda(x)
+    if not x.is_contiguous():
+        raise ValueError("x must be contiguous")
+    check(lib.b200_squared_relu(x.data_ptr(), x.numel(), _dt(x), _stream()), "squared_relu")
+    return x
+
+
+def softcap_logits(logits: torch.Tensor, scale: float, cap: float) -> torch.Tensor:
+    """cap * tanh(scale * logits / cap) in place on fp32 logits (cap <= 0: scale only)."""
+    _cuda(logits)
+    if logits.dtype != torch.float32 or not logits.is_contiguous():
+        raise ValueError("logits must be contiguous fp32")
+    check(lib.b200_softcap_logits(logits.data_ptr(), logits.numel(), float(scale), float(cap), _stream()), "softcap_logits")
+    return logits
+
+
+class DeltaRule:
+    """Constants of a gated delta rule layer on the device: head layout, convolution weights over the projection columns
+    [q | k | v] (``columns``: first column of each; ``width``: columns in all, weights [taps, width]), gate biases, norm."""
+
+    def __init__(self, heads: int, kv_heads: int, dim: int, vdim: int, columns: tuple[int, int, int], conv_w: torch.Tensor,
+                 dt_bias: torch.Tensor, a_log: torch.Tensor, norm_w: torch.Tensor, eps: float):
+        self.heads, self.kv_heads, self.dim, self.vdim, self.columns, self.eps = heads, kv_heads, dim, vdim, columns, float(eps)
+        self.taps, self.width = conv_w.shape
+        self.conv_w, self.dt_bias, self.a_log, self.norm_w = conv_w, dt_bias, a_log, norm_w
+        for name, t, n in (("conv_w", conv_w, self.taps * self.width), ("dt_bias", dt_bias, heads), ("a_log", a_log, heads),
+                           ("norm_w", norm_w, vdim)):
+            _f32vec(name, t, n)
+
+
+def _delta_inputs(c: DeltaRule, proj: torch.Tensor, b, a, gate, state: torch.Tensor, ring: torch.Tensor,
+                  state_slots: torch.Tensor, n: int) -> None:
+    T = proj.shape[0]
+    H, dk, dv = c.heads, c.dim, c.vdim
+    if proj.shape[1] < c.width or proj.stride(1) != 1 or b.shape != (T, H) or a.shape != (T, H) or gate.shape != (T, H * dv) \
+            or any(t.stride(1) != 1 or t.stride(0) != proj.stride(0) or t.dtype != proj.dtype for t in (b, a, gate)):
+        raise ValueError("proj [T, >= width], b and a [T, heads], gate [T, heads * vdim] must share dtype and row stride")
+    slots = state.shape[0]
+    if state.dtype != torch.float32 or state.shape != (slots, H, dk, dv) or not state.is_contiguous() \
+            or ring.dtype != torch.float32 or ring.shape != (slots, c.taps, c.width) or not ring.is_contiguous():
+        raise ValueError("state must be fp32 [slots, heads, dim, vdim] and the ring fp32 [slots, taps, width]")
+    if state_slots.dtype != torch.int64 or state_slots.numel() < n or not state_slots.is_contiguous():
+        raise ValueError("state_slots must be contiguous int64 with one entry per sequence")
+
+
+def delta_rule(c: DeltaRule, proj: torch.Tensor, b: torch.Tensor, a: torch.Tensor, gate: torch.Tensor, state: torch.Tensor,
+               ring: torch.Tensor, state_slots: torch.Tensor, cu_seqlens_q: torch.Tensor, cu_seqlens_k: torch.Tensor,
+               out: torch.Tensor | None = None, general: bool = False) -> torch.Tensor:
+    """Gated delta rule of ragged portions (``b200_delta_conv`` and ``b200_delta_rule``): proj [T, >= width] with the raw
+    [q | k | v] columns, b, a, gate views with the same row stride; state and convolution ring advance in place.
+    ``general`` forces the token-by-token kernel.  Returns the gated heads [T, heads * vdim]."""
+    dev = _cuda(proj, b, a, gate, state, ring, state_slots, cu_seqlens_q, cu_seqlens_k, out)
+    T, n = proj.shape[0], cu_seqlens_q.numel() - 1
+    _delta_inputs(c, proj, b, a, gate, state, ring, state_slots, n)
+    if cu_seqlens_q.dtype != torch.int32 or cu_seqlens_k.dtype != torch.int32 or cu_seqlens_k.numel() != n + 1:
+        raise ValueError("cu_seqlens must be int32 tensors of the same length")
+    out = _delta_out(c, proj, out)
+    act = torch.empty(T, c.width, dtype=proj.dtype, device=proj.device)
+    check(lib.b200_delta_conv(proj.data_ptr(), proj.stride(0), c.conv_w.data_ptr(), c.taps, c.width, ring.data_ptr(),
+                              ring.shape[0], state_slots.data_ptr(), cu_seqlens_q.data_ptr(), cu_seqlens_k.data_ptr(), n, T,
+                              act.data_ptr(), _dt(proj), status_word(dev).data_ptr(), _stream()), "delta_conv")
+    need = 0 if general else int(lib.b200_delta_rule_workspace_bytes(n, T, c.heads, c.dim, c.vdim, _dt(proj)))
+    ws = workspace(dev, need, "delta") if need else None
+    q, k, v = (act[:, at:] for at in c.columns)
+    check(lib.b200_delta_rule(
+        q.data_ptr(), k.data_ptr(), v.data_ptr(), act.stride(0), b.data_ptr(), a.data_ptr(), gate.data_ptr(), proj.stride(0),
+        c.dt_bias.data_ptr(), c.a_log.data_ptr(), c.norm_w.data_ptr(), c.eps, state.data_ptr(), state.shape[0],
+        state_slots.data_ptr(), cu_seqlens_q.data_ptr(), cu_seqlens_k.data_ptr(), n, T, c.heads, c.kv_heads, c.dim, c.vdim,
+        out.data_ptr(), _ptr(ws), ws.numel() if ws is not None else 0, _dt(proj), status_word(dev).data_ptr(), _stream()),
+        "delta_rule")
+    return out
+
+
+def delta_step(c: DeltaRule, proj: torch.Tensor, b: torch.Tensor, a: torch.Tensor, gate: torch.Tensor, state: torch.Tensor,
+               ring: torch.Tensor, state_slots: torch.Tensor, context_lens: torch.Tensor,
+               out: torch.Tensor | None = None) -> torch.Tensor:
+    """One token per sequence of the gated delta rule, convolution included (``b200_delta_step``); row i of the inputs is
+    sequence i, ``context_lens[i]`` tokens long with it.  Rows beyond ``context_lens`` are left alone."""
+    dev = _cuda(proj, b, a, gate, state, ring, state_slots, context_lens, out)
+    n = context_lens.numel()
+    _delta_inputs(c, proj, b, a, gate, state, ring, state_slots, n)
+    if context_lens.dtype != torch.int64 or n > proj.shape[0] or not context_lens.is_contiguous():
+        raise ValueError("context_lens must be contiguous int64 with at most one entry per row")
+    out = _delta_out(c, proj, out)
+    q, k, v = (proj[:, at:] for at in c.columns)
+    check(lib.b200_delta_step(
+        q.data_ptr(), k.data_ptr(), v.data_ptr(), b.data_ptr(), a.data_ptr(), gate.data_ptr(), proj.stride(0),
+        c.conv_w.data_ptr(), c.taps, c.width, *c.columns, ring.data_ptr(), c.dt_bias.data_ptr(), c.a_log.data_ptr(),
+        c.norm_w.data_ptr(), c.eps, state.data_ptr(), state.shape[0], state_slots.data_ptr(), context_lens.data_ptr(), n,
+        c.heads, c.kv_heads, c.dim, c.vdim, out.data_ptr(), _dt(proj), status_word(dev).data_ptr(), _stream()), "delta_step")
+    return out
+
+
+def _delta_out(c: DeltaRule, proj: torch.Tensor, out: torch.Tensor | None) -> torch.Tensor:
+    shape = (proj.shape[0], c.heads * c.vdim)
+    if out is None:
+        return torch.empty(shape, dtype=proj.dtype, device=proj.device)
+    if out.shape != shape or out.dtype != proj.dtype or not out.is_contiguous():
+        raise ValueError("out must be contiguous [T, heads * vdim] of proj's dtype")
     return out
