@@ -167,51 +167,54 @@ def kernels(steps: int = 20, warmup: int = 3, sizes=("d1024", "d2048", "d4096"),
     return dict(workload="Nabalix kernels alone, bf16", sizes={n: SIZES[n] for n in sizes}, kernels=out)
 
 
+def engine_rates(cfg: dict, weights, block_size: int, steps: int, warmup: int, batch: int, prompt: int) -> dict:
+    """Median wall time of a full prefill step (eight prompts of ``prompt`` tokens) and of a decode step of ``batch``
+    sequences, through an engine of its own."""
+    from .engine import SamplingParams, Sequence
+    from .engine.llm_engine import LLMEngine
+    Sequence.counter = itertools.count()
+    eng = LLMEngine(dict(model=cfg, weights=weights, dtype=torch.bfloat16, block_size=block_size, max_num_sequences=batch,
+                         max_num_batched_tokens=8 * prompt, max_cached_blocks=(batch + 1) * 2 * prompt // block_size, eos=-1,
+                         device="cuda:0", max_model_length=2 * prompt, seed=0))
+    mixed = getattr(eng.model_runner, "mixed_batches", False)
+    rng = np.random.default_rng(0)
+    for _ in range(batch):
+        eng.add_request(rng.integers(0, VOCAB, size=prompt).tolist(),
+                        SamplingParams(temperature=0.0, max_tokens=prompt, ignore_eos=True))
+    times = dict(prefill=[], decode=[])
+    while len(times["decode"]) < steps + warmup:
+        torch.cuda.synchronize()
+        t0 = time.perf_counter()
+        _, n, is_prefill = eng.step()
+        torch.cuda.synchronize()
+        if is_prefill and mixed and n != 8 * prompt:
+            continue                          # prompts finishing beside decoded tokens
+        if not is_prefill and n < batch:
+            continue
+        times["prefill" if is_prefill else "decode"].append(time.perf_counter() - t0)
+    ops.check_status()
+    pre, dec = float(np.median(times["prefill"][2:])), float(np.median(times["decode"][warmup:]))
+    eng.exit()
+    del eng
+    torch.cuda.empty_cache()
+    return dict(prefill_ms=pre * 1e3, prefill_tokens_per_s=8 * prompt / pre, decode_ms=dec * 1e3,
+                decode_tokens_per_s=batch / dec)
+
+
 def throughput(steps: int = 20, warmup: int = 3, sizes=("d1024", "d2048", "d4096"), layers: int = 4, batch: int = 64,
                prompt: int = 1024) -> dict:
     """Prefill and decode throughput through the engine: ``layers`` layers of every size, prompts of ``prompt``
     tokens eight to a step, then ``batch`` sequences decoding from captured graphs; the Nabalix model and the GQA
     decoder of the same width, heads, feed-forward and depth."""
-    from .engine import SamplingParams, Sequence
-    from .engine.llm_engine import LLMEngine
     from .model import resolve_config
     from .model.nabalix import init_weights as init_nabalix
     out = {}
     for name in sizes:
-        for family, cfg in (("nabalix", nabalix_config(SIZES[name], layers)), ("gqa", gqa_config(SIZES[name], layers))):
-            Sequence.counter = itertools.count()
-            bs = 64 if family == "nabalix" else 16
-            # checkpoints of the family hold bf16 values (the head mix then runs on tensor cores)
-            weights = init_nabalix(resolve_config(cfg), 0, torch.bfloat16) if family == "nabalix" else None
-            eng = LLMEngine(dict(model=cfg, weights=weights, dtype=torch.bfloat16, block_size=bs, max_num_sequences=batch,
-                                 max_num_batched_tokens=8 * prompt, max_cached_blocks=(batch + 1) * 2 * prompt // bs, eos=-1,
-                                 device="cuda:0", max_model_length=2 * prompt, seed=0))
-            rng = np.random.default_rng(0)
-            for _ in range(batch):
-                eng.add_request(rng.integers(0, VOCAB, size=prompt).tolist(),
-                                SamplingParams(temperature=0.0, max_tokens=prompt, ignore_eos=True))
-            times = dict(prefill=[], decode=[])
-            tokens = dict(prefill=[], decode=[])
-            while len(times["decode"]) < steps + warmup:
-                torch.cuda.synchronize()
-                t0 = time.perf_counter()
-                _, n, is_prefill = eng.step()
-                torch.cuda.synchronize()
-                kind = "prefill" if is_prefill else "decode"
-                if is_prefill and family == "nabalix" and n != 8 * prompt:
-                    continue                          # prompts finishing beside decoded tokens
-                if not is_prefill and n < batch:
-                    continue
-                times[kind].append(time.perf_counter() - t0)
-                tokens[kind].append(8 * prompt if is_prefill else n)
-            ops.check_status()
-            pre, dec = float(np.median(times["prefill"][2:])), float(np.median(times["decode"][warmup:]))
-            out[f"{name}.{family}"] = dict(prefill_ms=pre * 1e3, prefill_tokens_per_s=8 * prompt / pre, decode_ms=dec * 1e3,
-                                           decode_tokens_per_s=batch / dec)
-            eng.exit()
-            del eng
-            torch.cuda.empty_cache()
-        a, b = out[f"{name}.nabalix"], out[f"{name}.gqa"]
+        cfg = nabalix_config(SIZES[name], layers)
+        # checkpoints of the family hold bf16 values (the head mix then runs on tensor cores)
+        a = engine_rates(cfg, init_nabalix(resolve_config(cfg), 0, torch.bfloat16), 64, steps, warmup, batch, prompt)
+        b = engine_rates(gqa_config(SIZES[name], layers), None, 16, steps, warmup, batch, prompt)
+        out[f"{name}.nabalix"], out[f"{name}.gqa"] = a, b
         out[f"{name}.ratio"] = dict(prefill=a["prefill_tokens_per_s"] / b["prefill_tokens_per_s"],
                                     decode=a["decode_tokens_per_s"] / b["decode_tokens_per_s"])
     return dict(workload=f"engine throughput, {layers} layers, prefill steps of 8 prompts x {prompt} tokens, decode of "

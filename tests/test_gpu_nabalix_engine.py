@@ -1,6 +1,5 @@
 """The Nabalix family through the engine — scheduler, cache pools, state slots, captured graphs, sampler, command
 line — against the plain CPU restatement."""
-import itertools
 import json
 import os
 import subprocess
@@ -11,52 +10,13 @@ import pytest
 import torch
 
 import nabalix_fixtures as fx
+from engine_helpers import agree, error, make_engine, portions, run, write_model
 from oracle import nabalix as orc
 
 pytestmark = pytest.mark.gpu
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 TOL = {torch.float32: 6e-5, torch.bfloat16: 4e-2}
 DTYPES = [torch.float32, torch.bfloat16]
-
-
-def make_engine(cfg, w, dtype, max_tokens=512, block_size=16, **kw):
-    from llm_from_scratch_b200.engine import Sequence
-    from llm_from_scratch_b200.engine.llm_engine import LLMEngine
-    from llm_from_scratch_b200.engine.replay import engine_config
-    Sequence.counter = itertools.count()
-    return LLMEngine(engine_config(cfg, dtype, max_tokens, block_size, weights=w, **kw))
-
-
-def error(got, want):
-    """Worst position: rms over the vocabulary of the centred difference, in units of the logits' own rms."""
-    d = got.double().cpu() - want
-    d = d - d.mean(-1, keepdim=True)
-    return (d.pow(2).mean(-1).sqrt() / want.std()).max().item()
-
-
-def run(eng, steps):
-    """steps: [([(id, tokens)], [ended ids])]; returns {id: logits of every token}."""
-    from llm_from_scratch_b200 import ops
-    from llm_from_scratch_b200.engine.replay import Replay
-    rep, out = Replay(eng), {}
-    for entries, end in steps:
-        y = rep.step([(i, t, range(len(t))) for i, t in entries], end)
-        ops.check_status()
-        for (i, t), part in zip(entries, y.split([len(t) for _, t in entries])):
-            out.setdefault(i, []).append(part.cpu())
-    return {i: torch.cat(v) for i, v in out.items()}
-
-
-def portions(ids, sizes, name="a"):
-    at, steps = 0, []
-    for n in itertools.cycle(sizes):
-        part = ids[at:at + n]
-        if not part:
-            break
-        steps.append(([(name, part)], []))
-        at += n
-    steps[-1] = (steps[-1][0], [name])
-    return steps
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
@@ -172,14 +132,6 @@ def test_long_decoding_behind_a_short_prompt(dtype):
     eng.exit()
 
 
-def agree(streams, cfg, w, prompts, slack):
-    """Greedy streams follow the restatement wherever its two best logits are further apart than ``slack``."""
-    for got, prompt in zip(streams, prompts):
-        logits = orc.forward(cfg, w, list(prompt) + got)[len(prompt) - 1:-1]
-        chosen = logits.gather(1, torch.tensor(got)[:, None])[:, 0]
-        assert (logits.max(-1).values - chosen).max() <= slack * logits.std(), (logits.max(-1).values - chosen).max()
-
-
 @pytest.mark.parametrize("dtype,slack", [(torch.float32, 3e-4), (torch.bfloat16, 0.12)])
 @pytest.mark.parametrize("kw", [dict(), dict(prefill_graphs=True), dict(prefill_graphs=True, max_num_batched_tokens=64),
                                 dict(enforce_eager=True), dict(decode_window=5), dict(max_num_batched_tokens=24),
@@ -198,7 +150,7 @@ def test_greedy_generation_through_the_scheduler(kw, dtype, slack):
     eng.scheduler.preempt = lambda s: (preempted.append(s), original(s))
     out = eng.generate(prompts, SamplingParams(temperature=0.0, max_tokens=25, ignore_eos=True))["token_ids"]
     assert [len(t) for t in out] == [24] * len(prompts)
-    agree(out, cfg, w, prompts, slack)
+    agree(orc, out, cfg, w, prompts, slack)
     assert bool(preempted) == ("max_cached_blocks" in kw)
     assert eng.scheduler.block_manager.num_free_blocks == eng.model_runner.num_kv_blocks
     assert len(eng.scheduler.state_slots.free) == 4
@@ -216,14 +168,6 @@ def test_sampling_with_temperature_and_an_end_token():
     eng.scheduler.eos = first = eng.generate([prompts[0]], SamplingParams(temperature=0.0, max_tokens=4))["token_ids"][0][0]
     assert eng.generate([prompts[0]], SamplingParams(temperature=0.0, max_tokens=20))["token_ids"][0] == [first]
     eng.exit()
-
-
-def write_model(folder, cfg, w):
-    from safetensors.torch import save_file
-    os.makedirs(folder, exist_ok=True)
-    with open(os.path.join(folder, "config.json"), "w") as f:
-        json.dump(cfg, f)
-    save_file({k: v.contiguous() for k, v in w.items()}, os.path.join(folder, "model.safetensors"))
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
@@ -258,4 +202,4 @@ def test_generate_command_line(tmp_path):
                         "float32", "--max-tokens", "9", "--ignore-eos"] + [" ".join(map(str, p)) for p in prompts],
                        capture_output=True, text=True, timeout=300, cwd=ROOT)
     assert r.returncode == 0, r.stderr[-2000:]
-    agree([json.loads(x)["token_ids"] for x in r.stdout.splitlines()], cfg, w, prompts, 3e-4)
+    agree(orc, [json.loads(x)["token_ids"] for x in r.stdout.splitlines()], cfg, w, prompts, 3e-4)
