@@ -340,28 +340,27 @@ __global__ void __launch_bounds__(256, 1) delta_scan_kernel(const ChunkArgs args
       uint32_t h[4], m[4], l[4];
       split_a(S[2 * kk], S[2 * kk + 1], h, m, l);
 #pragma unroll
-      for (int np = 0; np < 4; ++np) {
-        uint32_t bf[4];
-        ldmatrix_x4(bf, st + lay.k + ((np * 16 + r_in) * ROWK + kk * 16 + bh * 8) * 2);
-        {
-          const uint32_t b0[2] = {bf[0], bf[1]}, b1[2] = {bf[2], bf[3]};
-          mma_bf16_16816(D[2 * np], l, b0);
-          mma_bf16_16816(D[2 * np + 1], l, b1);
-          mma_bf16_16816(D[2 * np], m, b0);
-          mma_bf16_16816(D[2 * np + 1], m, b1);
-          mma_bf16_16816(D[2 * np], h, b0);
-          mma_bf16_16816(D[2 * np + 1], h, b1);
+      for (int np = 0; np < 4; np += 2) {
+        uint32_t kf[2][4], qf[2][4];
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+          ldmatrix_x4(kf[u], st + lay.k + (((np + u) * 16 + r_in) * ROWK + kk * 16 + bh * 8) * 2);
+          ldmatrix_x4(qf[u], st + lay.q + (((np + u) * 16 + r_in) * ROWK + kk * 16 + bh * 8) * 2);
         }
-        ldmatrix_x4(bf, st + lay.q + ((np * 16 + r_in) * ROWK + kk * 16 + bh * 8) * 2);
-        {
-          const uint32_t b0[2] = {bf[0], bf[1]}, b1[2] = {bf[2], bf[3]};
-          mma_bf16_16816(O[2 * np], l, b0);
-          mma_bf16_16816(O[2 * np + 1], l, b1);
-          mma_bf16_16816(O[2 * np], m, b0);
-          mma_bf16_16816(O[2 * np + 1], m, b1);
-          mma_bf16_16816(O[2 * np], h, b0);
-          mma_bf16_16816(O[2 * np + 1], h, b1);
-        }
+        auto part = [&](const uint32_t (&p)[4]) {        // eight accumulators between two uses of one
+#pragma unroll
+          for (int u = 0; u < 2; ++u) {
+            const uint32_t k0[2] = {kf[u][0], kf[u][1]}, k1[2] = {kf[u][2], kf[u][3]};
+            const uint32_t q0[2] = {qf[u][0], qf[u][1]}, q1[2] = {qf[u][2], qf[u][3]};
+            mma_bf16_16816(D[2 * (np + u)], p, k0);
+            mma_bf16_16816(D[2 * (np + u) + 1], p, k1);
+            mma_bf16_16816(O[2 * (np + u)], p, q0);
+            mma_bf16_16816(O[2 * (np + u) + 1], p, q1);
+          }
+        };
+        part(l);
+        part(m);
+        part(h);
       }
     }
     // ---- D <- V^T - gamma rk D,  O <- gamma rq O
@@ -397,24 +396,30 @@ __global__ void __launch_bounds__(256, 1) delta_scan_kernel(const ChunkArgs args
         uint32_t h[4], m[4], l[4];
         split_a(in[2 * kk], in[2 * kk + 1], h, m, l);
 #pragma unroll
-        for (int np = kk; np < 4; ++np) {
-          const uint32_t at = base + ((np * 16 + r_in) * ROWP + kk * 16 + bh * 8) * 2;
-          uint32_t bl[4], bm[4], bt[4];
-          ldmatrix_x4(bl, at + 2 * C * ROWP * 2);
-          ldmatrix_x4(bm, at + C * ROWP * 2);
-          ldmatrix_x4(bt, at);
+        for (int n0 = kk & ~1; n0 < 4; n0 += 2) {        // two tiles of 16 rows; the first may lie above the diagonal
+          uint32_t b3[2][3][4];
 #pragma unroll
-          for (int u = 0; u < 2; ++u) {
-            const uint32_t h_b[2] = {bt[2 * u], bt[2 * u + 1]}, m_b[2] = {bm[2 * u], bm[2 * u + 1]},
-                           l_b[2] = {bl[2 * u], bl[2 * u + 1]};
-            float(&c)[4] = acc[2 * np + u];
-            mma_bf16_16816(c, l, h_b);
-            mma_bf16_16816(c, m, m_b);
-            mma_bf16_16816(c, h, l_b);
-            mma_bf16_16816(c, m, h_b);
-            mma_bf16_16816(c, h, m_b);
-            mma_bf16_16816(c, h, h_b);
-          }
+          for (int u = 0; u < 2; ++u)
+            if (n0 + u >= kk) {
+              const uint32_t at = base + (((n0 + u) * 16 + r_in) * ROWP + kk * 16 + bh * 8) * 2;
+#pragma unroll
+              for (int p = 0; p < 3; ++p) ldmatrix_x4(b3[u][p], at + p * C * ROWP * 2);
+            }
+          auto part = [&](const uint32_t (&x)[4], int p) {
+#pragma unroll
+            for (int u = 0; u < 2; ++u)
+              if (n0 + u >= kk) {
+                const uint32_t b0[2] = {b3[u][p][0], b3[u][p][1]}, b1[2] = {b3[u][p][2], b3[u][p][3]};
+                mma_bf16_16816(acc[2 * (n0 + u)], x, b0);
+                mma_bf16_16816(acc[2 * (n0 + u) + 1], x, b1);
+              }
+          };
+          part(l, 0);
+          part(m, 1);
+          part(h, 2);
+          part(m, 0);
+          part(h, 1);
+          part(h, 0);
         }
       }
     };
@@ -439,19 +444,38 @@ __global__ void __launch_bounds__(256, 1) delta_scan_kernel(const ChunkArgs args
       uint32_t h[4], m[4], l[4];
       split_a(U[2 * kk], U[2 * kk + 1], h, m, l);
 #pragma unroll
-      for (int c = 0; c < NK; c += 2) {
-        uint32_t bf[4];
-        ldmatrix_x4_trans(bf, st + lay.k + ((kk * 16 + t_in) * ROWK + (c + th) * 8) * 2);
-        const uint32_t b0[2] = {bf[0], bf[1]}, b1[2] = {bf[2], bf[3]};
-        mma_bf16_16816(S[c], l, b0);
-        mma_bf16_16816(S[c + 1], l, b1);
-        mma_bf16_16816(S[c], m, b0);
-        mma_bf16_16816(S[c + 1], m, b1);
-        mma_bf16_16816(S[c], h, b0);
-        mma_bf16_16816(S[c + 1], h, b1);
+      for (int c = 0; c < NK; c += 8) {
+        uint32_t bf[4][4];
+#pragma unroll
+        for (int u = 0; u < 4; ++u)
+          ldmatrix_x4_trans(bf[u], st + lay.k + ((kk * 16 + t_in) * ROWK + (c + 2 * u + th) * 8) * 2);
+        auto part = [&](const uint32_t (&x)[4]) {
+#pragma unroll
+          for (int u = 0; u < 4; ++u) {
+            const uint32_t b0[2] = {bf[u][0], bf[u][1]}, b1[2] = {bf[u][2], bf[u][3]};
+            mma_bf16_16816(S[c + 2 * u], x, b0);
+            mma_bf16_16816(S[c + 2 * u + 1], x, b1);
+          }
+        };
+        part(l);
+        part(m);
+        part(h);
       }
     }
     // ---- norm over the value columns, output gate
+    // a warp takes the tokens warp, warp + NT / 32, ... in groups of eight; the gates of a group are loaded ahead
+    const int nt = min(C, info.len - j * C), NW = NT / 32, c = lane * 4;
+    const int64_t tok0 = info.tok0 + j * C;
+    const __nv_bfloat16* gp = static_cast<const __nv_bfloat16*>(a.gate) + tok0 * a.proj_stride + head * dv + c;
+    uint2 gate[8];
+    auto load_gates = [&](int t0) {
+#pragma unroll
+      for (int u = 0; u < 8; ++u) {
+        const int t = t0 + u * NW;
+        gate[u] = c < dv && t < nt ? __ldg(reinterpret_cast<const uint2*>(gp + t * a.proj_stride)) : make_uint2(0u, 0u);
+      }
+    };
+    load_gates(warp);
     __syncthreads();                                   // K, Q, V of this stage are done with
     float* so = reinterpret_cast<float*>(stp);
     const int ldo = dv + 4;
@@ -460,22 +484,24 @@ __global__ void __launch_bounds__(256, 1) delta_scan_kernel(const ChunkArgs args
 #pragma unroll
       for (int e = 0; e < 4; ++e) so[(n * 8 + 2 * tq + (e & 1)) * ldo + vr + 8 * (e >> 1)] = O[n][e];
     __syncthreads();
-    const int nt = min(C, info.len - j * C);
-    for (int t = warp; t < nt; t += NT / 32) {
-      const int64_t tok = info.tok0 + j * C + t;
-      const int c = lane * 4;
-      float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (c < dv) o = *reinterpret_cast<const float4*>(so + t * ldo + c);
-      const float inv = rsqrtf(warp_sum(o.x * o.x + o.y * o.y + o.z * o.z + o.w * o.w) / static_cast<float>(dv) + a.eps);
-      if (c < dv) {
-        const uint2 gr = *reinterpret_cast<const uint2*>(static_cast<const __nv_bfloat16*>(a.gate) + tok * a.proj_stride +
-                                                         head * dv + c);
-        const float2 g0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gr.x));
-        const float2 g1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gr.y));
-        const float w0 = __ldg(a.norm_w + c), w1 = __ldg(a.norm_w + c + 1), w2 = __ldg(a.norm_w + c + 2), w3 = __ldg(a.norm_w + c + 3);
-        *reinterpret_cast<uint2*>(static_cast<__nv_bfloat16*>(a.out) + (tok * a.H + head) * dv + c) =
-            make_uint2(pack_bf16x2(o.x * inv * w0 * silu_f(g0.x), o.y * inv * w1 * silu_f(g0.y)),
-                       pack_bf16x2(o.z * inv * w2 * silu_f(g1.x), o.w * inv * w3 * silu_f(g1.y)));
+    float4 w = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (c < dv) w = make_float4(__ldg(a.norm_w + c), __ldg(a.norm_w + c + 1), __ldg(a.norm_w + c + 2), __ldg(a.norm_w + c + 3));
+    for (int t0 = warp; t0 < nt; t0 += 8 * NW) {
+      if (t0 != warp) load_gates(t0);
+#pragma unroll
+      for (int u = 0; u < 8; ++u) {
+        const int t = t0 + u * NW;
+        if (t >= nt) continue;                         // the same for the whole warp
+        float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (c < dv) o = *reinterpret_cast<const float4*>(so + t * ldo + c);
+        const float inv = rsqrtf(warp_sum(o.x * o.x + o.y * o.y + o.z * o.z + o.w * o.w) / static_cast<float>(dv) + a.eps);
+        const float2 g0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gate[u].x));
+        const float2 g1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gate[u].y));
+        using bf16 = __nv_bfloat16;
+        if (c < dv)
+          *reinterpret_cast<uint2*>(static_cast<bf16*>(a.out) + ((tok0 + t) * a.H + head) * dv + c) =
+              make_uint2(pack_bf16x2(o.x * inv * w.x * silu_for<bf16>(g0.x), o.y * inv * w.y * silu_for<bf16>(g0.y)),
+                         pack_bf16x2(o.z * inv * w.z * silu_for<bf16>(g1.x), o.w * inv * w.w * silu_for<bf16>(g1.y)));
       }
     }
   }

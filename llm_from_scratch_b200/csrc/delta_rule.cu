@@ -103,14 +103,14 @@ __global__ void __launch_bounds__(kConvThreads) delta_conv_kernel(const ConvArgs
       float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
       for (int m = 0; m < TAPS; ++m) fma4(y, w[m], h[m]);
-      store4<T>(out + static_cast<int64_t>(t) * a.C, make_float4(silu_f(y.x), silu_f(y.y), silu_f(y.z), silu_f(y.w)));
+      store4<T>(out + static_cast<int64_t>(t) * a.C, make_float4(silu_for<T>(y.x), silu_for<T>(y.y), silu_for<T>(y.z), silu_for<T>(y.w)));
     }
   } else {
     for (int t = lo; t < lo + nt; ++t) {
       float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
       for (int m = 0; m < taps; ++m)
         fma4(y, *reinterpret_cast<const float4*>(a.w + static_cast<int64_t>(m) * a.C + c), input(t - (taps - 1) + m));
-      store4<T>(out + static_cast<int64_t>(t) * a.C, make_float4(silu_f(y.x), silu_f(y.y), silu_f(y.z), silu_f(y.w)));
+      store4<T>(out + static_cast<int64_t>(t) * a.C, make_float4(silu_for<T>(y.x), silu_for<T>(y.y), silu_for<T>(y.z), silu_for<T>(y.w)));
     }
   }
   // The thread that has read the ring is the one that moves it on: the last taps - 1 inputs of the portion.
@@ -146,8 +146,29 @@ __global__ void __launch_bounds__(512) delta_serial_kernel(const DeltaArgs a, in
   float* ring = CONV ? a.conv_ring + info.slot * a.taps * a.conv_width : nullptr;
   const float scale = rsqrtf(static_cast<float>(dk));
   float s[R > 0 ? R : 1][V];
-  for (int t = 0; t < info.len; ++t) {
-    const int64_t tok = info.tok0 + t;
+  auto load_state = [&](int c, bool zero) {
+    if constexpr (R > 0) {
+#pragma unroll
+      for (int i = 0; i < R; ++i) {
+        const int r = rg + i * RG;
+        const float* sp = S + static_cast<int64_t>(r) * dv + c * V;
+        if constexpr (V == 4) {
+          const float4 x = zero || r >= dk ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(sp);
+          s[i][0] = x.x, s[i][1] = x.y, s[i][2] = x.z, s[i][3] = x.w;
+        } else {
+          s[i][0] = zero || r >= dk ? 0.f : *sp;
+        }
+      }
+    }
+  };
+  if (cu < units) load_state(cu, info.fresh);        // in flight while the inputs are gathered
+  const float dt_bias = a.dt_bias[head], a_log = a.a_log[head];
+  const float my_norm = threadIdx.x < dv ? a.norm_w[threadIdx.x] : 0.f;
+  for (int t = 0; t < (CONV ? 1 : info.len); ++t) {
+    const int64_t tok = info.tok0 + t, prow = tok * a.proj_stride + head;
+    const T* gp = static_cast<const T*>(a.gate) + tok * a.proj_stride + head * dv;
+    const T raw_b = static_cast<const T*>(a.b)[prow], raw_a = static_cast<const T*>(a.a)[prow];
+    const T my_gate = threadIdx.x < dv ? gp[threadIdx.x] : from_float<T>(0.f);
     const T* qp = static_cast<const T*>(a.q) + tok * a.act_stride + kh * dk;
     const T* kp = static_cast<const T*>(a.k) + tok * a.act_stride + kh * dk;
     const T* vp = static_cast<const T*>(a.v) + tok * a.act_stride + head * dv;
@@ -164,7 +185,7 @@ __global__ void __launch_bounds__(512) delta_serial_kernel(const DeltaArgs a, in
           if (p >= 0) y += a.conv_w[(a.taps - 1 - m) * a.conv_width + col] * rc[(p % a.taps) * a.conv_width];
         }
         rc[(info.pos0 % a.taps) * a.conv_width] = x;
-        x = to_float<T>(from_float<T>(silu_f(y)));
+        x = to_float<T>(from_float<T>(silu_for<T>(y)));
       }
       sm[i] = x;                  // q | k | v
     }
@@ -179,9 +200,8 @@ __global__ void __launch_bounds__(512) delta_serial_kernel(const DeltaArgs a, in
     }
     const float rq = rsqrtf(warp_sum(qq) + 1e-6f) * scale, rk = rsqrtf(warp_sum(kk) + 1e-6f);
     kq = warp_sum(kq) * rq * rk;
-    const int64_t prow = tok * a.proj_stride + head;
-    const float beta = sigmoid_f(to_float<T>(static_cast<const T*>(a.b)[prow]));
-    const float g = expf(log_decay(to_float<T>(static_cast<const T*>(a.a)[prow]) + a.dt_bias[head], a.a_log[head]));
+    const float beta = sigmoid_f(to_float<T>(raw_b));
+    const float g = expf(log_decay(to_float<T>(raw_a) + dt_bias, a_log));
     const bool zero = info.fresh && t == 0;
     for (int c0 = 0; c0 < units; c0 += CL) {
       const int c = c0 + cu;
@@ -190,19 +210,7 @@ __global__ void __launch_bounds__(512) delta_serial_kernel(const DeltaArgs a, in
       for (int e = 0; e < V; ++e) pk[e] = pq[e] = 0.f;
       if (c < units) {
         if constexpr (R > 0) {
-          if (!resident || t == 0) {
-#pragma unroll
-            for (int i = 0; i < R; ++i) {
-              const int r = rg + i * RG;
-              const float* sp = S + static_cast<int64_t>(r) * dv + c * V;
-              if constexpr (V == 4) {
-                const float4 x = zero || r >= dk ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(sp);
-                s[i][0] = x.x, s[i][1] = x.y, s[i][2] = x.z, s[i][3] = x.w;
-              } else {
-                s[i][0] = zero || r >= dk ? 0.f : *sp;
-              }
-            }
-          }
+          if (t > 0 ? !resident : c0 > 0) load_state(c, zero);
 #pragma unroll
           for (int i = 0; i < R; ++i) {
             const int r = rg + i * RG;
@@ -274,10 +282,10 @@ __global__ void __launch_bounds__(512) delta_serial_kernel(const DeltaArgs a, in
     float ss = 0.f;
     for (int i = lane; i < dv; i += 32) ss += so[i] * so[i];
     const float inv = rsqrtf(warp_sum(ss) / static_cast<float>(dv) + a.eps);
-    const T* gp = static_cast<const T*>(a.gate) + tok * a.proj_stride + head * dv;
     T* op = static_cast<T*>(a.out) + (tok * a.H + head) * dv;
-    for (int i = threadIdx.x; i < dv; i += NT) op[i] = from_float<T>(so[i] * inv * a.norm_w[i] * silu_f(to_float<T>(gp[i])));
-    __syncthreads();
+    if (threadIdx.x < dv) op[threadIdx.x] = from_float<T>(so[threadIdx.x] * inv * my_norm * silu_for<T>(to_float<T>(my_gate)));
+    for (int i = threadIdx.x + NT; i < dv; i += NT) op[i] = from_float<T>(so[i] * inv * a.norm_w[i] * silu_for<T>(to_float<T>(gp[i])));
+    if (!CONV) __syncthreads();
   }
 }
 

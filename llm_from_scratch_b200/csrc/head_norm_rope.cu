@@ -5,6 +5,8 @@
 //
 // in one launch with the scatter of k and v into the paged pool.  Angles are products in double precision reduced
 // modulo 2 pi, so a position of any size keeps fp32 accuracy; a CTA computes them once per token for all heads.
+#include <initializer_list>
+
 #include "common.cuh"
 
 namespace b200 {
@@ -146,8 +148,105 @@ __global__ void __launch_bounds__(kThreads) head_norm_rope_kernel(const HnArgs a
   }
 }
 
+// bf16 heads of 8 * LPH channels (LPH a power of two up to 32): LPH lanes per head, 16 bytes per lane, 32 / LPH heads per warp
+template <int LPH>
+__global__ void __launch_bounds__(kThreads) head_norm_rope_wide_kernel(const HnArgs a) {
+  extern __shared__ float2 cs[];     // [kTokens][half] (cos, sin)
+  constexpr int HPW = 32 / LPH, D = 8 * LPH;
+  const int64_t t0 = static_cast<int64_t>(blockIdx.x) * kTokens;
+  const int nt = static_cast<int>(a.T - t0 < kTokens ? a.T - t0 : kTokens);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, heads = a.Hq + a.Hkv, c = (lane % LPH) * 8;
+  for (int i = threadIdx.x; i < nt * a.half; i += kThreads) {
+    const int t = i / a.half, j = i - t * a.half;
+    double ang = static_cast<double>(a.positions[t0 + t]) * a.freq[j];
+    ang -= 6.283185307179586 * rint(ang * 0.15915494309189535);
+    float s, co;
+    sincosf(static_cast<float>(ang), &s, &co);
+    cs[i] = make_float2(co, s);
+  }
+  const bool turns = c < 2 * a.half;             // whole 8-channel groups turn or pass (half a multiple of four)
+  __syncthreads();
+  union Pack {
+    uint4 u;
+    __nv_bfloat162 p[4];
+  };
+  for (int task = warp * HPW + lane / LPH; task < (nt * heads + HPW - 1) / HPW * HPW; task += kThreads / 32 * HPW) {
+    const bool live = task < nt * heads;
+    const int t = live ? task / heads : 0, h = live ? task - t * heads : 0;
+    const int64_t tok = t0 + t;
+    const bool is_q = h < a.Hq;
+    const int hh = is_q ? h : h - a.Hq;
+    Pack x;
+    x.u = *reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(is_q ? a.q : a.k) + tok * a.stride + hh * D + c);
+    float v[8], ss = 0.f;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float2 f = __bfloat1622float2(x.p[e]);
+      v[2 * e] = f.x;
+      v[2 * e + 1] = f.y;
+      ss += f.x * f.x + f.y * f.y;
+    }
+#pragma unroll
+    for (int o = LPH / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    const float inv = rsqrtf(ss / static_cast<float>(D) + a.eps);
+    const float* w = (is_q ? a.wq : a.wk) + c;
+    const float4 w0 = *reinterpret_cast<const float4*>(w), w1 = *reinterpret_cast<const float4*>(w + 4);
+    const float ww[8] = {w0.x, w0.y, w0.z, w0.w, w1.x, w1.y, w1.z, w1.w};
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      float u = v[2 * e] * inv * ww[2 * e], z = v[2 * e + 1] * inv * ww[2 * e + 1];
+      if (turns) {
+        const float2 r = cs[t * a.half + c / 2 + e];
+        const float nu = u * r.x - z * r.y;
+        z = z * r.x + u * r.y;
+        u = nu;
+      }
+      x.p[e] = __floats2bfloat162_rn(u, z);
+    }
+    if (!live) continue;
+    *reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(is_q ? a.q_out : a.k_out) + (tok * (is_q ? a.Hq : a.Hkv) + hh) * D + c) = x.u;
+    if (!is_q && a.kc != nullptr) {
+      const int64_t slot = a.slots[tok];
+      if (slot >= a.num_slots) report(a.status, B200_ERR_BOUNDS);
+      else if (slot >= 0)
+        *reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(a.kc) + (slot * a.Hkv + hh) * D + c) = x.u;
+    }
+  }
+  if (a.vc != nullptr) {
+    const int per = a.Hkv * a.Dv / 8;
+    for (int i = threadIdx.x; i < nt * per; i += kThreads) {
+      const int t = i / per, j = i - t * per;
+      const int64_t slot = a.slots[t0 + t];
+      if (slot < 0 || slot >= a.num_slots) continue;
+      reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(a.vc) + slot * a.Hkv * a.Dv)[j] =
+          reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(a.v) + (t0 + t) * a.stride)[j];
+    }
+  }
+}
+
+// whether the wide kernel takes the call, and its launch
+bool launch_wide(const HnArgs& a, cudaStream_t s) {
+  const int lph = a.D / 8;
+  if (a.D % 8 || a.Dv % 8 || (lph & (lph - 1)) || lph > 32 || a.half % 4 || a.stride % 8) return false;
+  for (const void* p : {a.q, a.k, a.v, static_cast<const void*>(a.wq), static_cast<const void*>(a.wk),
+                        static_cast<const void*>(a.q_out), static_cast<const void*>(a.k_out), static_cast<const void*>(a.kc),
+                        static_cast<const void*>(a.vc)})
+    if (!aligned16(p)) return false;
+  const unsigned grid = static_cast<unsigned>((a.T + kTokens - 1) / kTokens);
+  const size_t smem = static_cast<size_t>(kTokens) * a.half * sizeof(float2);
+  switch (lph) {
+    case 4: head_norm_rope_wide_kernel<4><<<grid, kThreads, smem, s>>>(a); break;
+    case 8: head_norm_rope_wide_kernel<8><<<grid, kThreads, smem, s>>>(a); break;
+    case 16: head_norm_rope_wide_kernel<16><<<grid, kThreads, smem, s>>>(a); break;
+    case 32: head_norm_rope_wide_kernel<32><<<grid, kThreads, smem, s>>>(a); break;
+    default: return false;
+  }
+  return true;
+}
+
 template <typename T>
 int launch(const HnArgs& a, cudaStream_t s) {
+  if (sizeof(T) == 2 && launch_wide(a, s)) return launch_result();
   const unsigned grid = static_cast<unsigned>((a.T + kTokens - 1) / kTokens);
   const size_t smem = static_cast<size_t>(kTokens) * a.half * sizeof(float2);
   const bool vec = a.D % 4 == 0 && a.D > 64 && a.stride % 4 == 0 && aligned16(a.q) && aligned16(a.k) && aligned16(a.q_out) &&

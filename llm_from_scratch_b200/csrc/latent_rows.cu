@@ -1,6 +1,6 @@
 // Rows of a latent key/value cache without a rotary part: the norm of the down-projection with its scatter into the
 // paged pool, and the gather of whole contexts back out of the pool for the prefill expansion.
-#include "common.cuh"
+#include "sequences.cuh"
 
 namespace b200 {
 namespace {
@@ -99,34 +99,27 @@ __global__ void __launch_bounds__(kWarps * 32) gather_rows_kernel(const GaArgs a
   }
 }
 
-// out = o * sigmoid(g), element by element; o contiguous [T, W], g [T, W] with a row stride
+// out = o * sigmoid(g), element by element; o contiguous [T, W], g [T, W] with a row stride; a CTA per row
 template <typename T, int E>
-__global__ void __launch_bounds__(256) sigmoid_gate_kernel(T* o, const T* g, int64_t g_stride, int64_t units, int per_row) {
+__global__ void __launch_bounds__(256) sigmoid_gate_kernel(T* o, const T* g, int64_t g_stride, int W) {
   union Pack {
     uint4 u;
     T e[16 / sizeof(T)];
   };
-  for (int64_t i = static_cast<int64_t>(blockIdx.x) * blockDim.x + threadIdx.x; i < units;
-       i += static_cast<int64_t>(gridDim.x) * blockDim.x) {
-    const int64_t t = i / per_row;
-    const int c = static_cast<int>(i - t * per_row) * E;
-    auto gated = [](float x, float z) { return x / (1.f + expf(-z)); };
+  o += static_cast<int64_t>(blockIdx.x) * W;
+  g += blockIdx.x * g_stride;
+  for (int c = threadIdx.x * E; c < W; c += blockDim.x * E) {
     if constexpr (E > 1) {
       Pack a, b;
-      a.u = *reinterpret_cast<const uint4*>(o + i * E);
-      b.u = *reinterpret_cast<const uint4*>(g + t * g_stride + c);
+      a.u = *reinterpret_cast<const uint4*>(o + c);
+      b.u = *reinterpret_cast<const uint4*>(g + c);
 #pragma unroll
-      for (int k = 0; k < E; ++k) a.e[k] = from_float<T>(gated(to_float<T>(a.e[k]), to_float<T>(b.e[k])));
-      *reinterpret_cast<uint4*>(o + i * E) = a.u;
+      for (int k = 0; k < E; ++k) a.e[k] = from_float<T>(to_float<T>(a.e[k]) * sigmoid_for<T>(to_float<T>(b.e[k])));
+      *reinterpret_cast<uint4*>(o + c) = a.u;
     } else {
-      o[i] = from_float<T>(gated(to_float<T>(o[i]), to_float<T>(g[t * g_stride + c])));
+      o[c] = from_float<T>(to_float<T>(o[c]) * sigmoid_for<T>(to_float<T>(g[c])));
     }
   }
-}
-
-inline unsigned elementwise_grid(int64_t units) {
-  const int64_t want = (units + 255) / 256;
-  return static_cast<unsigned>(want < 148 * 32 ? want : 148 * 32);
 }
 
 }  // namespace
@@ -189,19 +182,19 @@ extern "C" int b200_sigmoid_gate(void* o, const void* gate, int64_t gate_stride,
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   const int E = dtype == B200_DTYPE_F32 ? 4 : 8;
   const bool vec = width % E == 0 && gate_stride % E == 0 && aligned16(o) && aligned16(gate);
-  const int64_t units = rows * width / (vec ? E : 1);
-  const int per_row = width / (vec ? E : 1);
-  const unsigned grid = elementwise_grid(units);
+  if (rows > 2147483647) return B200_ERR_TOO_LARGE;
+  const int units = (width + (vec ? E : 1) - 1) / (vec ? E : 1), threads = units >= 256 ? 256 : (units + 31) / 32 * 32;
+  const unsigned grid = static_cast<unsigned>(rows);
   if (dtype == B200_DTYPE_F32) {
     auto* p = static_cast<float*>(o);
     auto* g = static_cast<const float*>(gate);
-    if (vec) sigmoid_gate_kernel<float, 4><<<grid, 256, 0, s>>>(p, g, gate_stride, units, per_row);
-    else sigmoid_gate_kernel<float, 1><<<grid, 256, 0, s>>>(p, g, gate_stride, units, per_row);
+    if (vec) sigmoid_gate_kernel<float, 4><<<grid, threads, 0, s>>>(p, g, gate_stride, width);
+    else sigmoid_gate_kernel<float, 1><<<grid, threads, 0, s>>>(p, g, gate_stride, width);
   } else {
     auto* p = static_cast<__nv_bfloat16*>(o);
     auto* g = static_cast<const __nv_bfloat16*>(gate);
-    if (vec) sigmoid_gate_kernel<__nv_bfloat16, 8><<<grid, 256, 0, s>>>(p, g, gate_stride, units, per_row);
-    else sigmoid_gate_kernel<__nv_bfloat16, 1><<<grid, 256, 0, s>>>(p, g, gate_stride, units, per_row);
+    if (vec) sigmoid_gate_kernel<__nv_bfloat16, 8><<<grid, threads, 0, s>>>(p, g, gate_stride, width);
+    else sigmoid_gate_kernel<__nv_bfloat16, 1><<<grid, threads, 0, s>>>(p, g, gate_stride, width);
   }
   return launch_result();
 }

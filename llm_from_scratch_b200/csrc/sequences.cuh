@@ -98,5 +98,12 @@ __device__ __forceinline__ float sigmoid_f(float x) {
   return s;
 }
 __device__ __forceinline__ float silu_f(float x) { return x * sigmoid_f(x); }
+// for values that are rounded to T next: in bf16 on the approximate exponential (relative error below 2^-20)
+template <typename T>
+__device__ __forceinline__ float sigmoid_for(float x) {
+  return sizeof(T) == 2 ? rcp_approx(1.f + fast_exp2(-1.4426950408889634f * x)) : sigmoid_f(x);
+}
+template <typename T>
+__device__ __forceinline__ float silu_for(float x) { return x * sigmoid_for<T>(x); }
 
 }  // namespace b200
