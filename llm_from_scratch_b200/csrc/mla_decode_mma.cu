@@ -103,7 +103,8 @@ __device__ __forceinline__ void named_arrive(int id) {
   asm volatile("bar.arrive %0, %1;\n" ::"r"(id), "n"(kThreads) : "memory");
 }
 
-template <int R_, int DR_>
+// PLAIN: at most 16 heads and 16-token pages, which spares the address arithmetic of the general case
+template <int R_, int DR_, bool PLAIN>
 __global__ void __launch_bounds__(kThreads, 1)
 mla_decode_mma_kernel(const MlaArgs a, const __grid_constant__ CUtensorMap tm_lat) {
   using Z = Latent<R_, DR_>;
@@ -121,8 +122,8 @@ mla_decode_mma_kernel(const MlaArgs a, const __grid_constant__ CUtensorMap tm_la
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
   const int B = a.batch, p = blockIdx.x;
-  const int hb = blockIdx.y * 16, H = min(16, a.H - hb);   // this CTA's group of heads
-  const int64_t table_blocks = a.bt_stride << a.sub_log2;
+  const int hb = PLAIN ? 0 : blockIdx.y * 16, H = PLAIN ? a.H : min(16, a.H - hb);   // this CTA's group of heads
+  const int64_t table_blocks = PLAIN ? a.bt_stride : a.bt_stride << a.sub_log2;
   // the combine kernel is a programmatic dependent: its CTAs may be placed while this grid runs
   asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
 
@@ -151,6 +152,7 @@ mla_decode_mma_kernel(const MlaArgs a, const __grid_constant__ CUtensorMap tm_la
   };
   // pool block (of 16 tokens) of a sequence's block number blk; an id outside the pool stays outside
   auto physical = [&](int seq, int blk) -> int {
+    if (PLAIN) return __ldg(a.bt + static_cast<int64_t>(seq) * a.bt_stride + blk);
     const int id = __ldg(a.bt + static_cast<int64_t>(seq) * a.bt_stride + (blk >> a.sub_log2));
     if (id >= (INT_MAX >> a.sub_log2)) return INT_MAX;
     return id < 0 ? id : (id << a.sub_log2) + (blk & ((1 << a.sub_log2) - 1));
@@ -454,7 +456,7 @@ size_t mla_decode_mma_workspace(int batch, int H, int r, int dr) {
 }
 
 namespace {
-template <int R, int DR>
+template <int R, int DR, bool PLAIN>
 int launch(MlaArgs a, int64_t grid, EncodeFn enc, cudaStream_t s) {
   using Z = Latent<R, DR>;
   // The pool seen as (column within a slab: 64, token row: num_blocks * 16, slab: ROW / 64) with strides
@@ -475,12 +477,12 @@ int launch(MlaArgs a, int64_t grid, EncodeFn enc, cudaStream_t s) {
   int dev = 0;
   cudaGetDevice(&dev);
   if (dev >= 0 && dev < 64 && !configured[dev]) {
-    if (cudaFuncSetAttribute(mla_decode_mma_kernel<R, DR>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    if (cudaFuncSetAttribute(mla_decode_mma_kernel<R, DR, PLAIN>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                              Z::SMEM_BYTES) != cudaSuccess)
       return B200_ERR_LAUNCH;
     configured[dev] = true;
   }
-  mla_decode_mma_kernel<R, DR>
+  mla_decode_mma_kernel<R, DR, PLAIN>
       <<<dim3(static_cast<unsigned>(grid), head_groups(a.H)), kThreads, Z::SMEM_BYTES, s>>>(a, tm);
   return launch_result();
 }
@@ -523,8 +525,10 @@ int mla_decode_mma_launch(const void* q_abs, const void* q_rope, const void* lat
   a.part_ml = reinterpret_cast<float*>(w);
   w += align256(grid * 2 * H * 2 * sizeof(float));
   a.seq_info = reinterpret_cast<int32_t*>(w);
-  const int rc = r == 512 ? (dr ? launch<512, 64>(a, grid, enc, s) : launch<512, 0>(a, grid, enc, s))
-                          : (dr ? launch<256, 64>(a, grid, enc, s) : launch<256, 0>(a, grid, enc, s));
+  const bool plain = H <= 16 && a.sub_log2 == 0;
+  const int rc = r == 512 ? (dr ? (plain ? launch<512, 64, true>(a, grid, enc, s) : launch<512, 64, false>(a, grid, enc, s))
+                                : launch<512, 0, false>(a, grid, enc, s))
+                          : (dr ? launch<256, 64, false>(a, grid, enc, s) : launch<256, 0, false>(a, grid, enc, s));
   if (rc != B200_OK) return rc;
   CombineArgs c{};
   c.out = out;
