@@ -306,8 +306,8 @@ class Delta:
         return y.cpu().split([hi - lo for _, lo, hi in ranges])
 
 
-DELTA_SHAPES = [(4, 2, 64, 64, 4), (2, 2, 128, 128, 4), (3, 1, 48, 32, 2), (6, 2, 32, 112, 3), (2, 1, 80, 16, 5), (3, 3, 20, 12, 1),
-                (2, 1, 33, 7, 4), (1, 1, 256, 256, 4), (1, 1, 16, 16, 4)]
+DELTA_SHAPES = [(4, 2, 64, 64, 4), (2, 2, 128, 128, 4), (2, 1, 128, 64, 4), (3, 1, 64, 128, 2), (3, 1, 48, 32, 2), (6, 2, 32, 112, 3),
+                (2, 1, 80, 16, 5), (3, 3, 20, 12, 1), (2, 1, 33, 7, 4), (1, 1, 256, 256, 4), (1, 1, 16, 16, 4)]
 STATE_TOL = {torch.float32: 3e-5, torch.bfloat16: 3e-5}      # behind equal activations the state is fp32 in either dtype
 
 
