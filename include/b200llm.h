@@ -38,7 +38,7 @@
 extern "C" {
 #endif
 
-#define B200_ABI_VERSION 11
+#define B200_ABI_VERSION 12
 
 #define B200_DTYPE_F32 0
 #define B200_DTYPE_BF16 1
@@ -638,6 +638,99 @@ int b200_delta_step(const void* q, const void* k, const void* v, const void* b, 
                     const float* norm_w, float eps, float* state, int64_t num_slots, const int64_t* state_slots,
                     const int64_t* context_lens, int32_t num_seqs, int32_t num_heads, int32_t num_k_heads, int32_t dim_k,
                     int32_t dim_v, void* out, int32_t dtype, int32_t* status, void* stream);
+
+/* ---------------------------------------------------------------------------------------------
+ * Mechanisms of decoders with parallel gated sublayers, windowed latent attention with sinks, grouped expert routing and
+ * per-layer token inputs (the Meresun family; the reference has no counterpart).  All constants are parameters.
+ * ------------------------------------------------------------------------------------------- */
+
+/* b200_residual_norm with an embedding row that may also join an existing residual, and a norm in equal parts of the row:
+ *   x <- (start ? 0 : x) + y / sqrt(mean(y^2) + eps) * y_norm_w + embed_scale embed[tokens]     (y, embed: NULL = absent)
+ *   h  = x / sqrt(mean over the channel's part of x^2 + eps) * norm_w, `groups` consecutive parts; norm_w NULL: h = x. */
+int b200_residual_group_norm(float* x, const void* y, const float* y_norm_w, const int64_t* tokens, const void* embed,
+                             int64_t vocab, float embed_scale, int32_t start, const float* norm_w, int32_t groups, float eps,
+                             void* h, int64_t rows, int32_t d, int32_t dtype, int32_t* status, void* stream);
+
+/* Parallel sublayers into the fp32 residual x [rows, d], in place: x <- x + y1 sigmoid(gate1) + y2 sigmoid(gate2), h = x in
+ * dtype.  y1, y2 contiguous [rows, d] in dtype, gates with one row stride; y2 NULL: one sublayer.  top_k > 0: y2 holds expert
+ * rows [rows * top_k, d] and row t takes sum_k row_weight[t, k] y2[slot_to_row[t, k]]. */
+int b200_gated_residual(float* x, const void* y1, const void* gate1, const void* y2, const void* gate2, int64_t gate_stride,
+                        const float* row_weight, const int32_t* slot_to_row, int32_t top_k, void* h, int64_t rows, int32_t d,
+                        int32_t dtype, int32_t* status, void* stream);
+
+/* out = c0 N(z) + c1 N(z^2) + c2 N(z^3) + c3 per row of z [rows, width] (row stride), coef fp32 [4] on the device,
+ * N(u) = u / sqrt(mean(u^2) + eps), powers element by element; out contiguous. */
+int b200_poly_norm(const void* z, int64_t row_stride, const float* coef, float eps, void* out, int64_t rows, int32_t width,
+                   int32_t dtype, void* stream);
+
+/* out[t] = gelu_tanh(u[t]) * table[tokens[t], first .. first + width - 1]; u, out [rows, width], table [vocab, table_width]. */
+int b200_gelu_table(const void* u, const void* table, int64_t table_width, int64_t vocab, int32_t first, const int64_t* tokens,
+                    void* out, int64_t rows, int32_t width, int32_t dtype, int32_t* status, void* stream);
+
+/* Latent attention with a rotary part, between the down-projections and the rest, one launch:
+ *   q_out[t]  = q_in[t] / rms * q_norm_w [q_rank]                                            (q_in NULL: no query latent)
+ *   kv_out[t] = [kv_in[t, :kv_rank] / rms * kv_norm_w | rotated kv_in[t, kv_rank:]], also written to cache[slot_mapping[t]]
+ * The channel pairs (2i, 2i + 1), i < rot_dims / 2, of the rotary part (rope_dim wide) turn by positions[t] * freq[i] (freq
+ * fp64); cos and sin are multiplied by `magnitude`.  Inputs with row strides, outputs contiguous. */
+int b200_latent_prologue(const void* q_in, int64_t q_stride, const float* q_norm_w, int32_t q_rank, void* q_out,
+                         const void* kv_in, int64_t kv_stride, const float* kv_norm_w, int32_t kv_rank, int32_t rope_dim,
+                         float eps, const double* freq, int32_t rot_dims, float magnitude, const int64_t* positions,
+                         void* kv_out, void* cache, const int64_t* slot_mapping, int64_t num_slots, int64_t num_tokens,
+                         int32_t dtype, int32_t* status, void* stream);
+
+/* The same rotation on the last rope_dim channels of every head of q [num_tokens, num_heads, head_dim], in place; the rotated
+ * parts of the first tail_rows tokens are also written to tail [tail_rows, num_heads, rope_dim]. */
+int b200_rotate_heads(void* q, int64_t num_tokens, int32_t num_heads, int32_t head_dim, int32_t rope_dim, const double* freq,
+                      int32_t rot_dims, float magnitude, const int64_t* positions, void* tail, int64_t tail_rows, int32_t dtype,
+                      void* stream);
+
+/* b200_gather_rows for the ends of contexts: sequence s is cu_seqlens_full[s + 1] - cu_seqlens_full[s] tokens long and its last
+ * cu_seqlens_k[s + 1] - cu_seqlens_k[s] rows are packed (cu_seqlens_full NULL: whole contexts). */
+int b200_gather_last_rows(const void* cache, int32_t block_size, int64_t num_blocks, int64_t row_bytes,
+                          const int32_t* block_tables, int64_t bt_stride, const int32_t* cu_seqlens_k,
+                          const int32_t* cu_seqlens_full, int32_t num_seqs, int32_t max_seqlen_k, void* out, int64_t out_rows,
+                          int32_t* status, void* stream);
+
+/* Packed ragged causal attention with keys in two parts, a sliding window and a sink: query i of a sequence (at the end of its
+ * k_len keys, bottom-right aligned) sees keys j with 0 <= (k_len - q_len + i) - j < window (window 0: all earlier ones).
+ * k_head [total_k, num_kv_heads, head_dim_qk - tail_dim] and k_tail [total_k, tail_dim], the last columns of every head's key
+ * (tail_dim 0: none); sink as in b200_prefill_varlen_sink.  plan: tile list for b200_prefill_window_tile_rows() rows, or NULL.
+ * bf16: tcgen05 kernels for 192/128 (tail 64 or 0) and 128/128, mma.sync for multiples of eight up to 192/128; else general. */
+int32_t b200_prefill_window_tile_rows(int32_t num_q_heads, int32_t num_kv_heads, int32_t head_dim_qk, int32_t tail_dim,
+                                      int32_t head_dim_v, int32_t dtype);
+int b200_prefill_varlen_window(const void* q, const void* k_head, const void* k_tail, const void* v, void* out,
+                               int64_t q_token_stride, int64_t k_head_token_stride, int64_t k_tail_token_stride,
+                               int64_t v_token_stride, int64_t total_q_tokens, int64_t total_k_tokens,
+                               const int32_t* cu_seqlens_q, const int32_t* cu_seqlens_k, int32_t num_seqs,
+                               int32_t max_seqlen_q, int32_t num_q_heads, int32_t num_kv_heads, int32_t head_dim_qk,
+                               int32_t tail_dim, int32_t head_dim_v, float scale, int32_t window, const float* sink,
+                               const int32_t* plan, int32_t plan_tile_rows, int32_t plan_capacity, int32_t dtype,
+                               int32_t* status, void* stream);
+
+/* b200_mla_decode over the last `window` tokens of every context (0: all) with exp(sink[h]) in the softmax denominator (sink
+ * fp32 [num_heads] or NULL).  Workspace as b200_mla_decode. */
+int b200_mla_decode_window(const void* q_abs, const void* q_rope, const void* latent_cache, void* out_latent,
+                           const int32_t* block_tables, int64_t bt_stride, const int64_t* context_lens, int32_t batch,
+                           int32_t num_heads, int32_t kv_lora_rank, int32_t rope_dim, int32_t block_size, int64_t num_blocks,
+                           float scale, int32_t window, const float* sink, void* workspace, size_t workspace_bytes,
+                           int32_t dtype, int32_t* status, void* stream);
+
+/* Routing with a choice correction and groups: s = sigmoid(logits), c = s + correction (all fp32).  Experts form `groups` equal
+ * groups of neighbours; a group's score is the sum of its two largest c, the `keep` best groups stay, and of their experts the
+ * `top` with the largest c are chosen.  weight [tokens, top] = s of the chosen / (their sum + 1e-20).  sorted_token [tokens *
+ * top] lists the tokens of the rows grouped by expert, expert_offsets [experts] their exclusive ends, slot_to_row [tokens, top]
+ * the row of a token's k-th choice.  At most 512 experts, top 32, 64 groups. */
+size_t b200_moe_group_route_workspace_bytes(int32_t num_tokens, int32_t num_experts, int32_t top);
+int b200_moe_group_route(const float* logits, const float* correction, int32_t num_tokens, int32_t num_experts, int32_t top,
+                         int32_t groups, int32_t keep, int32_t* sorted_token, float* weight, int32_t* expert_offsets,
+                         int32_t* slot_to_row, void* workspace, size_t workspace_bytes, void* stream);
+
+/* b200_moe_grouped_gemm without biases, for any size and also fp32 (general kernel).  glu: w [experts, 2 n_out, k_dim] =
+ * [gate | up] and out = g sigmoid(slope g) (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit).
+ * flags: 0 or B200_MOE_GEMM_EARLY_LAUNCH. */
+int b200_moe_grouped_linear(const void* x, const void* w, void* out, const int32_t* expert_offsets, int64_t num_rows,
+                            int32_t num_experts, int32_t n_out, int32_t k_dim, int32_t glu, float limit, float slope,
+                            int32_t flags, int32_t dtype, int32_t* status, void* stream);
 
 /* ---------------------------------------------------------------------------------------------
  * Diagnostic (no counterpart in the reference, which has no device code): runs the give-up path of the

@@ -46,11 +46,14 @@ def _stale(target: Path, deps: list[Path]) -> bool:
 # Sources a model family runs on, where that is not the whole library: ``ensure`` builds a library of just these
 # when the full one is absent.  "api" and "host_path" are the parts every engine uses.
 FAMILY_SOURCES = {
-    "Nabalix": ("api", "host_path", "decode_advance", "sampler", "moe_gemm", "moe_gemm_rows", "store_kvcache", "prefill_plan", "streams",
+    "Nabalix": ("api", "host_path", "decode_advance", "sampler", "moe_gemm", "moe_gemm_rows", "grouped_linear", "store_kvcache", "prefill_plan", "streams",
                 "talking_attention", "talking_attention_mma", "talking_decode_mma", "gated_recurrence"),
-    "Taminex": ("api", "host_path", "decode_advance", "sampler", "moe_gemm", "moe_gemm_rows", "store_kvcache", "prefill_plan",
+    "Taminex": ("api", "host_path", "decode_advance", "sampler", "moe_gemm", "moe_gemm_rows", "grouped_linear", "store_kvcache", "prefill_plan",
                 "prefill_varlen", "prefill_mma", "prefill_umma", "prefill_umma2", "prefill_umma4", "paged_decode", "mla_decode",
                 "mla_decode_mma", "residual_norm", "head_norm_rope", "latent_rows", "activations", "delta_rule", "delta_chunk"),
+    "Meresun": ("api", "host_path", "decode_advance", "sampler", "moe_gemm", "moe_gemm_rows", "grouped_linear", "moe_group_route",
+                "store_kvcache", "prefill_plan", "prefill_varlen", "prefill_mma", "prefill_umma", "prefill_umma2", "prefill_umma4",
+                "paged_decode", "mla_decode", "mla_decode_mma", "residual_norm", "gated_residual", "latent_rows", "activations"),
 }
 
 

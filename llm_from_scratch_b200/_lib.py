@@ -99,6 +99,23 @@ SIGNATURES = {
                           _i32, _i64, _i32, _i32, _i32, _i32, _vp, _vp, _sz, _i32, _vp, _vp]),
     "b200_delta_step": (_i32, [_vp, _vp, _vp, _vp, _vp, _vp, _i64, _vp, _i32, _i32, _i32, _i32, _i32, _vp, _vp, _vp,
                           _vp, _f32, _vp, _i64, _vp, _vp, _i32, _i32, _i32, _i32, _i32, _vp, _i32, _vp, _vp]),
+    "b200_residual_group_norm": (_i32, [_vp, _vp, _vp, _vp, _vp, _i64, _f32, _i32, _vp, _i32, _f32, _vp, _i64, _i32, _i32,
+                          _vp, _vp]),
+    "b200_gated_residual": (_i32, [_vp, _vp, _vp, _vp, _vp, _i64, _vp, _vp, _i32, _vp, _i64, _i32, _i32, _vp, _vp]),
+    "b200_poly_norm": (_i32, [_vp, _i64, _vp, _f32, _vp, _i64, _i32, _i32, _vp]),
+    "b200_gelu_table": (_i32, [_vp, _vp, _i64, _i64, _i32, _vp, _vp, _i64, _i32, _i32, _vp, _vp]),
+    "b200_latent_prologue": (_i32, [_vp, _i64, _vp, _i32, _vp, _vp, _i64, _vp, _i32, _i32, _f32, _vp, _i32, _f32, _vp, _vp,
+                          _vp, _vp, _i64, _i64, _i32, _vp, _vp]),
+    "b200_rotate_heads": (_i32, [_vp, _i64, _i32, _i32, _i32, _vp, _i32, _f32, _vp, _vp, _i64, _i32, _vp]),
+    "b200_gather_last_rows": (_i32, [_vp, _i32, _i64, _i64, _vp, _i64, _vp, _vp, _i32, _i32, _vp, _i64, _vp, _vp]),
+    "b200_prefill_window_tile_rows": (_i32, [_i32, _i32, _i32, _i32, _i32, _i32]),
+    "b200_prefill_varlen_window": (_i32, [_vp, _vp, _vp, _vp, _vp, _i64, _i64, _i64, _i64, _i64, _i64, _vp, _vp, _i32, _i32,
+                          _i32, _i32, _i32, _i32, _i32, _f32, _i32, _vp, _vp, _i32, _i32, _i32, _vp, _vp]),
+    "b200_mla_decode_window": (_i32, [_vp, _vp, _vp, _vp, _vp, _i64, _vp, _i32, _i32, _i32, _i32, _i32, _i64, _f32, _i32,
+                          _vp, _vp, _sz, _i32, _vp, _vp]),
+    "b200_moe_group_route_workspace_bytes": (_sz, [_i32, _i32, _i32]),
+    "b200_moe_group_route": (_i32, [_vp, _vp, _i32, _i32, _i32, _i32, _i32, _vp, _vp, _vp, _vp, _vp, _sz, _vp]),
+    "b200_moe_grouped_linear": (_i32, [_vp, _vp, _vp, _vp, _i64, _i32, _i32, _i32, _i32, _f32, _f32, _i32, _i32, _vp, _vp]),
     "b200_moe_combine": (_i32, [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i32, _i32, _i32, _vp]),
     "b200_selftest_bounded_wait": (_i32, [_i32, _vp, _vp, _vp]),
     "b200_lm_head_argmax_workspace_bytes": (_sz, [_i32, _i32]),

@@ -119,6 +119,13 @@ __device__ __forceinline__ float fast_exp2(float x) {
 // value or scale.  A sink far above every score overflows to infinity, which turns the row into zeros as it should.
 __device__ __forceinline__ float sink_term(float sink, float m) { return fast_exp2(sink * 1.4426950408889634f - m); }
 
+// Clamped gated linear unit: g sigmoid(slope g) (u + 1), g cut at `limit` above, u at +-limit.
+__device__ __forceinline__ float clamped_glu_f(float g, float u, float limit, float slope) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return g * (u + 1.f) / (1.f + expf(-slope * g));
+}
+
 // Prefill tile list (b200_prefill_plan): int32 header {tile count, rows per tile, capacity, 0} followed
 // by one entry per query tile, (sequence << 16) | tile index, heaviest tiles first.
 constexpr int kPlanHeader = 4;

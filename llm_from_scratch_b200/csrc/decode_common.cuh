@@ -14,6 +14,13 @@ __device__ __forceinline__ int num_kv_blocks(int64_t len, int64_t bt_stride, int
   return static_cast<int>(n < bt_stride ? n : bt_stride);
 }
 
+// First block that the last `window` tokens of a context reach (window <= 0: the whole context).
+__device__ __forceinline__ int first_kv_block(int64_t len, int64_t bt_stride, int bs, int window) {
+  if (window <= 0) return 0;
+  const int64_t cap = bt_stride * bs, n = (len < cap ? len : cap) - window;
+  return n > 0 ? static_cast<int>(n / bs) : 0;
+}
+
 // Inclusive scan over the CTA; `scratch` holds one int per warp.  Every thread must call it.
 __device__ __forceinline__ int block_inclusive_scan(int v, int* scratch, int* total) {
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
@@ -37,16 +44,19 @@ __device__ __forceinline__ int block_inclusive_scan(int v, int* scratch, int* to
 }
 
 // This CTA's share of the flat (sequence, block) list: `cnt` blocks starting at block `start_off`
-// of sequence `start_seq`; `per_cta` is the common range length (the last CTAs may get less or
+// of sequence `start_seq` (counted from the first block its window reaches); `per_cta` is the common range length (the last CTAs may get less or
 // nothing: cnt == 0).  `scratch` is 34 ints of shared memory.  Every thread must call it.
 struct CtaRange {
   int start, cnt, per_cta, start_seq, start_off;
 };
 __device__ __forceinline__ CtaRange plan_cta_range(const int64_t* lens, int batch,
-                                                   int64_t bt_stride, int bs, int* scratch) {
+                                                   int64_t bt_stride, int bs, int* scratch, int window = 0) {
+  auto blocks_of = [&](int i) {
+    const int64_t len = lens[i];
+    return num_kv_blocks(len, bt_stride, bs) - first_kv_block(len, bt_stride, bs, window);
+  };
   int local = 0;
-  for (int i = threadIdx.x; i < batch; i += blockDim.x)
-    local += num_kv_blocks(lens[i], bt_stride, bs);
+  for (int i = threadIdx.x; i < batch; i += blockDim.x) local += blocks_of(i);
   int T;
   block_inclusive_scan(local, scratch, &T);
   CtaRange r;
@@ -59,7 +69,7 @@ __device__ __forceinline__ CtaRange plan_cta_range(const int64_t* lens, int batc
   int carry = 0;
   for (int base = 0; base < batch; base += blockDim.x) {
     const int i = base + threadIdx.x;
-    const int v = i < batch ? num_kv_blocks(lens[i], bt_stride, bs) : 0;
+    const int v = i < batch ? blocks_of(i) : 0;
     int tot;
     const int incl = block_inclusive_scan(v, scratch, &tot) + carry;
     const int excl = incl - v;
@@ -87,6 +97,7 @@ struct CombineArgs {
   const float* part_ml;
   const int32_t* seq_info;
   int batch, H, D;
+  const float* sink;       // [H] or null
 };
 int decode_combine_launch(const CombineArgs& c, cudaStream_t s);
 

@@ -3,11 +3,10 @@
 //   q[h] = rot(rms(q_in[h]) wq),  k[g] = rot(rms(k_in[g]) wk)     rms over the head, fp32
 //   rot: channels (2i, 2i + 1) of the first `rot_dims` turn by position * freq[i], the others pass
 //
-// in one launch with the scatter of k and v into the paged pool.  Angles are products in double precision reduced
-// modulo 2 pi, so a position of any size keeps fp32 accuracy; a CTA computes them once per token for all heads.
+// in one launch with the scatter of k and v into the paged pool.  A CTA computes the angles once per token for all heads.
 #include <initializer_list>
 
-#include "common.cuh"
+#include "rotary.cuh"
 
 namespace b200 {
 namespace {
@@ -72,11 +71,7 @@ __global__ void __launch_bounds__(kThreads) head_norm_rope_kernel(const HnArgs a
   const int nt = static_cast<int>(a.T - t0 < kTokens ? a.T - t0 : kTokens);
   for (int i = threadIdx.x; i < nt * a.half; i += kThreads) {
     const int t = i / a.half, j = i - t * a.half;
-    double ang = static_cast<double>(a.positions[t0 + t]) * a.freq[j];
-    ang -= 6.283185307179586 * rint(ang * 0.15915494309189535);
-    float s, c;
-    sincosf(static_cast<float>(ang), &s, &c);
-    cs[i] = make_float2(c, s);
+    cs[i] = rotary_angle(a.positions[t0 + t], a.freq[j]);
   }
   __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, heads = a.Hq + a.Hkv;
@@ -158,11 +153,7 @@ __global__ void __launch_bounds__(kThreads) head_norm_rope_wide_kernel(const HnA
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, heads = a.Hq + a.Hkv, c = (lane % LPH) * 8;
   for (int i = threadIdx.x; i < nt * a.half; i += kThreads) {
     const int t = i / a.half, j = i - t * a.half;
-    double ang = static_cast<double>(a.positions[t0 + t]) * a.freq[j];
-    ang -= 6.283185307179586 * rint(ang * 0.15915494309189535);
-    float s, co;
-    sincosf(static_cast<float>(ang), &s, &co);
-    cs[i] = make_float2(co, s);
+    cs[i] = rotary_angle(a.positions[t0 + t], a.freq[j]);
   }
   const bool turns = c < 2 * a.half;             // whole 8-channel groups turn or pass (half a multiple of four)
   __syncthreads();

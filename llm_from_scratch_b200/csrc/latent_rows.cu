@@ -1,5 +1,7 @@
-// Rows of a latent key/value cache without a rotary part: the norm of the down-projection with its scatter into the
-// paged pool, and the gather of whole contexts back out of the pool for the prefill expansion.
+// Rows of a latent key/value cache: the norm of the down-projection (with the rotation of a rotary part behind it, and the
+// norm of a query latent beside it) with its scatter into the paged pool, the rotation of the queries' rotary channels, and
+// the gather of contexts, or of the ends of contexts, back out of the pool for the prefill expansion.
+#include "rotary.cuh"
 #include "sequences.cuh"
 
 namespace b200 {
@@ -66,6 +68,166 @@ __global__ void __launch_bounds__(kWarps * 32) latent_norm_kernel(const LnArgs a
   }
 }
 
+struct LpArgs {
+  const void* q_in;          // [T, rq] query latents (row stride free) or null
+  int64_t q_stride;
+  const float* wq;           // [rq]
+  int rq;
+  void* q_out;               // [T, rq]
+  const void* kv_in;         // [T, r + dr]
+  int64_t kv_stride;
+  const float* wkv;          // [r]
+  int r, dr;
+  float eps;
+  const double* freq;        // [half]
+  int half;                  // rotated pairs, the first of the rotary part
+  float magnitude;           // of cos and sin
+  const int64_t* positions;  // [T]
+  void* kv_out;              // [T, r + dr]
+  void* cache;               // [slots, r + dr] or null
+  const int64_t* slots;
+  int64_t num_slots, T;
+  int32_t* status;
+};
+
+// dst (and dst2, if given) = src / rms(src) * w over n elements, by a warp; E elements per access
+template <typename T, int E>
+__device__ __forceinline__ void warp_norm(const T* src, const float* w, int n, float eps, T* dst, T* dst2) {
+  const int lane = threadIdx.x & 31;
+  union Pack {
+    uint4 u;
+    T e[16 / sizeof(T)];
+  };
+  float ss = 0.f;
+  for (int c = lane * E; c < n; c += 32 * E) {
+    Pack p;
+    if constexpr (E > 1) p.u = *reinterpret_cast<const uint4*>(src + c);
+    else p.e[0] = src[c];
+#pragma unroll
+    for (int i = 0; i < E; ++i) ss += to_float<T>(p.e[i]) * to_float<T>(p.e[i]);
+  }
+  const float inv = rsqrtf(warp_sum(ss) / static_cast<float>(n) + eps);
+  for (int c = lane * E; c < n; c += 32 * E) {
+    Pack p;
+    if constexpr (E > 1) p.u = *reinterpret_cast<const uint4*>(src + c);
+    else p.e[0] = src[c];
+#pragma unroll
+    for (int i = 0; i < E; ++i) p.e[i] = from_float<T>(to_float<T>(p.e[i]) * inv * w[c + i]);
+    if constexpr (E > 1) {
+      *reinterpret_cast<uint4*>(dst + c) = p.u;
+      if (dst2) *reinterpret_cast<uint4*>(dst2 + c) = p.u;
+    } else {
+      dst[c] = p.e[0];
+      if (dst2) dst2[c] = p.e[0];
+    }
+  }
+}
+
+// blockIdx.y 0: latent rows; 1: query latents.  A warp per row; EQ / EK elements per access
+template <typename T, int EQ, int EK>
+__global__ void __launch_bounds__(kWarps * 32) latent_prologue_kernel(const LpArgs a) {
+  const int lane = threadIdx.x & 31;
+  const int64_t t = static_cast<int64_t>(blockIdx.x) * kWarps + (threadIdx.x >> 5);
+  if (t >= a.T) return;
+  if (blockIdx.y == 1) {
+    warp_norm<T, EQ>(static_cast<const T*>(a.q_in) + t * a.q_stride, a.wq, a.rq, a.eps, static_cast<T*>(a.q_out) + t * a.rq,
+                     nullptr);
+    return;
+  }
+  const int W = a.r + a.dr;
+  int64_t slot = a.cache ? a.slots[t] : -1;
+  if (slot >= a.num_slots) {
+    if (lane == 0) report(a.status, B200_ERR_BOUNDS);
+    slot = -1;
+  }
+  const T* src = static_cast<const T*>(a.kv_in) + t * a.kv_stride;
+  T* out = static_cast<T*>(a.kv_out) + t * W;
+  T* pool = slot >= 0 ? static_cast<T*>(a.cache) + slot * W : nullptr;
+  warp_norm<T, EK>(src, a.wkv, a.r, a.eps, out, pool);
+  const int64_t pos = a.positions[t];
+  for (int i = lane; 2 * i < a.dr; i += 32) {
+    const int c = a.r + 2 * i;
+    const bool pair = 2 * i + 1 < a.dr;
+    float u = to_float<T>(src[c]), v = pair ? to_float<T>(src[c + 1]) : 0.f;
+    if (i < a.half) {
+      const float2 cs = rotary_angle(pos, a.freq[i]);
+      const float co = cs.x * a.magnitude, si = cs.y * a.magnitude, nu = u * co - v * si;
+      v = v * co + u * si;
+      u = nu;
+    }
+    out[c] = from_float<T>(u);
+    if (pair) out[c + 1] = from_float<T>(v);
+    if (pool) {
+      pool[c] = from_float<T>(u);
+      if (pair) pool[c + 1] = from_float<T>(v);
+    }
+  }
+}
+
+struct RtArgs {
+  void* q;                   // [T, H, D], in place
+  int64_t T;
+  int H, D, dr;              // the last dr channels of a head are its rotary part
+  const double* freq;
+  int half;
+  float magnitude;
+  const int64_t* positions;
+  void* tail;                // [tail_rows, H, dr] or null: a copy of the rotated parts of the first rows
+  int64_t tail_rows;
+};
+
+// kRotTokens tokens per CTA; one pair of channels per thread and trip
+constexpr int kRotTokens = 2;
+template <typename T, bool PAIRS>
+__global__ void __launch_bounds__(256) rotate_heads_kernel(const RtArgs a) {
+  extern __shared__ float2 cs[];     // [kRotTokens][half]
+  const int64_t t0 = static_cast<int64_t>(blockIdx.x) * kRotTokens;
+  const int nt = static_cast<int>(a.T - t0 < kRotTokens ? a.T - t0 : kRotTokens);
+  for (int i = threadIdx.x; i < nt * a.half; i += blockDim.x) {
+    const int t = i / a.half, j = i - t * a.half;
+    const float2 r = rotary_angle(a.positions[t0 + t], a.freq[j]);
+    cs[i] = make_float2(r.x * a.magnitude, r.y * a.magnitude);
+  }
+  __syncthreads();
+  const int pairs = (a.dr + 1) / 2, per = a.H * pairs;
+  for (int i = threadIdx.x; i < nt * per; i += blockDim.x) {
+    const int t = i / per, k = i - t * per, h = k / pairs, j = k - h * pairs;
+    const int64_t tok = t0 + t;
+    T* p = static_cast<T*>(a.q) + (tok * a.H + h) * a.D + (a.D - a.dr) + 2 * j;
+    T* tail = tok < a.tail_rows ? static_cast<T*>(a.tail) + (tok * a.H + h) * a.dr + 2 * j : nullptr;
+    const bool pair = 2 * j + 1 < a.dr;
+    float u, v;
+    if constexpr (PAIRS) {
+      if constexpr (sizeof(T) == 2) {
+        const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p));
+        u = f.x, v = f.y;
+      } else {
+        const float2 f = *reinterpret_cast<const float2*>(p);
+        u = f.x, v = f.y;
+      }
+    } else {
+      u = to_float<T>(p[0]), v = pair ? to_float<T>(p[1]) : 0.f;
+    }
+    if (j < a.half) {
+      const float2 r = cs[t * a.half + j];
+      const float nu = u * r.x - v * r.y;
+      v = v * r.x + u * r.y;
+      u = nu;
+    }
+    auto put = [&](T* d) {
+      if constexpr (PAIRS) {
+        if constexpr (sizeof(T) == 2) *reinterpret_cast<uint32_t*>(d) = pack_bf16x2(u, v);
+        else *reinterpret_cast<float2*>(d) = make_float2(u, v);
+      } else {
+        d[0] = from_float<T>(u);
+        if (pair) d[1] = from_float<T>(v);
+      }
+    };
+    put(p);
+    if (tail) put(tail);
+  }
+}
+
 struct GaArgs {
   const void* cache;         // [num_blocks, bs, W]
   const int32_t* bt;
@@ -73,6 +235,7 @@ struct GaArgs {
   int bs;
   int64_t num_blocks;
   const int32_t* cu_k;       // [n + 1]
+  const int32_t* cu_full;    // [n + 1] or null: whole contexts, of which cu_k counts the last rows
   void* out;                 // [rows, W]
   int64_t rows;
   int W;                     // row width in units
@@ -85,15 +248,16 @@ __global__ void __launch_bounds__(kWarps * 32) gather_rows_kernel(const GaArgs a
   const int s = blockIdx.y, lane = threadIdx.x & 31;
   const int k0 = a.cu_k[s], len = a.cu_k[s + 1] - k0;
   const int64_t base = k0 - a.cu_k[0];
+  const int skip = a.cu_full ? max(a.cu_full[s + 1] - a.cu_full[s] - len, 0) : 0;
   for (int j = blockIdx.x * kWarps + (threadIdx.x >> 5); j < len; j += gridDim.x * kWarps) {
-    const int blk = j / a.bs;
+    const int pos = skip + j, blk = pos / a.bs;
     int64_t id = -1;
     if (blk < a.bt_stride) id = a.bt[s * a.bt_stride + blk];
     if (id < 0 || id >= a.num_blocks || base + j >= a.rows) {
       if (lane == 0) report(a.status, B200_ERR_BOUNDS);
       continue;
     }
-    const U* src = static_cast<const U*>(a.cache) + (id * a.bs + j % a.bs) * a.W;
+    const U* src = static_cast<const U*>(a.cache) + (id * a.bs + pos % a.bs) * a.W;
     U* dst = static_cast<U*>(a.out) + (base + j) * a.W;
     for (int c = lane; c < a.W; c += 32) dst[c] = src[c];
   }
@@ -153,13 +317,21 @@ extern "C" int b200_gather_rows(const void* cache, int32_t block_size, int64_t n
                                 const int32_t* block_tables, int64_t bt_stride, const int32_t* cu_seqlens_k,
                                 int32_t num_seqs, int32_t max_seqlen_k, void* out, int64_t out_rows, int32_t* status,
                                 void* stream) {
+  return b200_gather_last_rows(cache, block_size, num_blocks, row_bytes, block_tables, bt_stride, cu_seqlens_k, nullptr,
+                               num_seqs, max_seqlen_k, out, out_rows, status, stream);
+}
+
+extern "C" int b200_gather_last_rows(const void* cache, int32_t block_size, int64_t num_blocks, int64_t row_bytes,
+                                     const int32_t* block_tables, int64_t bt_stride, const int32_t* cu_seqlens_k,
+                                     const int32_t* cu_seqlens_full, int32_t num_seqs, int32_t max_seqlen_k, void* out,
+                                     int64_t out_rows, int32_t* status, void* stream) {
   using namespace b200;
   if (block_size <= 0 || num_blocks <= 0 || row_bytes <= 0 || bt_stride <= 0 || num_seqs < 0 || max_seqlen_k < 0)
     return B200_ERR_ARG;
   if (num_seqs == 0 || max_seqlen_k == 0) return B200_OK;
   if (!cache || !block_tables || !cu_seqlens_k || !out) return B200_ERR_ARG;
   if (num_seqs > 65535 || row_bytes % 2) return B200_ERR_UNSUPPORTED;
-  GaArgs a{cache, block_tables, bt_stride, block_size, num_blocks, cu_seqlens_k, out, out_rows, 0, status};
+  GaArgs a{cache, block_tables, bt_stride, block_size, num_blocks, cu_seqlens_k, cu_seqlens_full, out, out_rows, 0, status};
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   const dim3 grid((max_seqlen_k + 4 * kWarps - 1) / (4 * kWarps), num_seqs);
   if (row_bytes % 16 == 0 && aligned16(cache) && aligned16(out)) {
@@ -195,6 +367,64 @@ extern "C" int b200_sigmoid_gate(void* o, const void* gate, int64_t gate_stride,
     auto* g = static_cast<const __nv_bfloat16*>(gate);
     if (vec) sigmoid_gate_kernel<__nv_bfloat16, 8><<<grid, threads, 0, s>>>(p, g, gate_stride, width);
     else sigmoid_gate_kernel<__nv_bfloat16, 1><<<grid, threads, 0, s>>>(p, g, gate_stride, width);
+  }
+  return launch_result();
+}
+
+extern "C" int b200_latent_prologue(const void* q_in, int64_t q_stride, const float* q_norm_w, int32_t q_rank, void* q_out,
+                                    const void* kv_in, int64_t kv_stride, const float* kv_norm_w, int32_t kv_rank,
+                                    int32_t rope_dim, float eps, const double* freq, int32_t rot_dims, float magnitude,
+                                    const int64_t* positions, void* kv_out, void* cache, const int64_t* slot_mapping,
+                                    int64_t num_slots, int64_t num_tokens, int32_t dtype, int32_t* status, void* stream) {
+  using namespace b200;
+  if (num_tokens < 0 || kv_rank <= 0 || rope_dim < 0 || rot_dims < 0 || rot_dims % 2 || rot_dims > rope_dim || (q_in && q_rank <= 0))
+    return B200_ERR_ARG;
+  if (dtype != B200_DTYPE_F32 && dtype != B200_DTYPE_BF16) return B200_ERR_UNSUPPORTED;
+  if (num_tokens == 0) return B200_OK;
+  if (!kv_in || !kv_norm_w || !kv_out || !positions || (rot_dims > 0 && !freq) || (q_in && (!q_norm_w || !q_out)) ||
+      (cache && !slot_mapping))
+    return B200_ERR_ARG;
+  if (num_tokens > 2147483647LL * kWarps) return B200_ERR_TOO_LARGE;
+  LpArgs a{q_in, q_stride, q_norm_w, q_rank, q_out, kv_in, kv_stride, kv_norm_w, kv_rank, rope_dim, eps, freq, rot_dims / 2,
+           magnitude, positions, kv_out, cache, slot_mapping, num_slots, num_tokens, status};
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  const dim3 grid(static_cast<unsigned>((num_tokens + kWarps - 1) / kWarps), q_in ? 2 : 1);
+  const int E = dtype == B200_DTYPE_F32 ? 4 : 8;
+  const bool vq = !q_in || (q_rank % E == 0 && q_stride % E == 0 && aligned16(q_in) && aligned16(q_out));
+  const bool vk = kv_rank % E == 0 && (kv_rank + rope_dim) % E == 0 && kv_stride % E == 0 && aligned16(kv_in) && aligned16(kv_out) &&
+                  (!cache || aligned16(cache));
+  if (dtype == B200_DTYPE_F32) {
+    if (vq && vk) latent_prologue_kernel<float, 4, 4><<<grid, kWarps * 32, 0, s>>>(a);
+    else latent_prologue_kernel<float, 1, 1><<<grid, kWarps * 32, 0, s>>>(a);
+  } else {
+    if (vq && vk) latent_prologue_kernel<__nv_bfloat16, 8, 8><<<grid, kWarps * 32, 0, s>>>(a);
+    else latent_prologue_kernel<__nv_bfloat16, 1, 1><<<grid, kWarps * 32, 0, s>>>(a);
+  }
+  return launch_result();
+}
+
+extern "C" int b200_rotate_heads(void* q, int64_t num_tokens, int32_t num_heads, int32_t head_dim, int32_t rope_dim,
+                                 const double* freq, int32_t rot_dims, float magnitude, const int64_t* positions, void* tail,
+                                 int64_t tail_rows, int32_t dtype, void* stream) {
+  using namespace b200;
+  if (num_tokens < 0 || num_heads <= 0 || rope_dim < 0 || rope_dim > head_dim || rot_dims < 0 || rot_dims % 2 ||
+      rot_dims > rope_dim || tail_rows < 0 || tail_rows > num_tokens)
+    return B200_ERR_ARG;
+  if (dtype != B200_DTYPE_F32 && dtype != B200_DTYPE_BF16) return B200_ERR_UNSUPPORTED;
+  if (num_tokens == 0 || rope_dim == 0) return B200_OK;
+  if (!q || !positions || (rot_dims > 0 && !freq) || (tail_rows > 0 && !tail)) return B200_ERR_ARG;
+  if (rot_dims > 4096 || num_tokens > 2147483647LL) return B200_ERR_UNSUPPORTED;
+  RtArgs a{q, num_tokens, num_heads, head_dim, rope_dim, freq, rot_dims / 2, magnitude, positions, tail, tail_rows};
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  const unsigned grid = static_cast<unsigned>((num_tokens + kRotTokens - 1) / kRotTokens);
+  const size_t smem = sizeof(float2) * kRotTokens * (rot_dims / 2);
+  const bool pairs = head_dim % 2 == 0 && rope_dim % 2 == 0 && aligned16(q) && (!tail || aligned16(tail));
+  if (dtype == B200_DTYPE_F32) {
+    if (pairs) rotate_heads_kernel<float, true><<<grid, 256, smem, s>>>(a);
+    else rotate_heads_kernel<float, false><<<grid, 256, smem, s>>>(a);
+  } else {
+    if (pairs) rotate_heads_kernel<__nv_bfloat16, true><<<grid, 256, smem, s>>>(a);
+    else rotate_heads_kernel<__nv_bfloat16, false><<<grid, 256, smem, s>>>(a);
   }
   return launch_result();
 }

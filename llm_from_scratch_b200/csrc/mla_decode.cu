@@ -1,6 +1,7 @@
 // MLA latent-cache decode attention (absorbed form): for every sequence and head
 //   score[t] = (q_abs . c_t + q_rope . pe_t) * scale,  P = softmax(score),  out = sum_t P[t] c_t
-// where the latent pool row of token t is [c_t (kv_lora_rank) | pe_t (rope_dim)].
+// where the latent pool row of token t is [c_t (kv_lora_rank) | pe_t (rope_dim)]; optionally over the last `window` tokens
+// only, and with exp(sink) of the head in the softmax denominator.
 //
 // Generic path: one CTA per (sequence, head), 4 warps striding over the tokens, a lane owning the
 // row elements lane, lane+32, ...; fp32 online softmax, warps merged through shared memory.
@@ -20,6 +21,8 @@ struct MlaArgs {
   int batch, H, r, dr, bs;
   int64_t num_blocks;
   float scale_log2;
+  int window;          // tokens a query sees, itself included; 0: all
+  const float* sink;   // [H] or null
   int32_t* status;
 };
 
@@ -56,7 +59,8 @@ __global__ void __launch_bounds__(kWarps * 32) mla_decode_simple_kernel(const Ml
   for (int i = 0; i < kMaxV; ++i) acc[i] = 0.f;
   float m = -INFINITY, l = 0.f;
   const T* lat = static_cast<const T*>(a.lat);
-  for (int t = warp; t < len; t += kWarps) {
+  const int first = a.window > 0 && len > a.window ? len - a.window : 0;
+  for (int t = first + warp; t < len; t += kWarps) {
     const int id = a.bt[static_cast<int64_t>(seq) * a.bt_stride + t / a.bs];
     if (static_cast<uint64_t>(static_cast<int64_t>(id)) >= static_cast<uint64_t>(a.num_blocks)) {
       report(a.status, B200_ERR_BOUNDS);
@@ -94,6 +98,7 @@ __global__ void __launch_bounds__(kWarps * 32) mla_decode_simple_kernel(const Ml
     wgt[w] = s_m[w] == -INFINITY ? 0.f : exp2f(s_m[w] - M);
     Lsum += wgt[w] * s_l[w];
   }
+  if (a.sink != nullptr && M > -INFINITY) Lsum += exp2f(a.sink[head] * 1.4426950408889634f - M);
   for (int d = threadIdx.x; d < r; d += blockDim.x) {
     float v = 0.f;
     for (int w = 0; w < kWarps; ++w) v += wgt[w] * s_acc[w][d];
@@ -106,8 +111,8 @@ __global__ void __launch_bounds__(kWarps * 32) mla_decode_simple_kernel(const Ml
 // tensor-core path (mla_decode_mma.cu); B200_ERR_UNSUPPORTED when the shape is outside it
 int mla_decode_mma_launch(const void* q_abs, const void* q_rope, const void* lat, void* out,
                           const int32_t* bt, int64_t bt_stride, const int64_t* lens, int batch,
-                          int H, int r, int dr, int bs, int64_t num_blocks, float scale,
-                          void* workspace, size_t workspace_bytes, int32_t* status,
+                          int H, int r, int dr, int bs, int64_t num_blocks, float scale, int window,
+                          const float* sink, void* workspace, size_t workspace_bytes, int32_t* status,
                           cudaStream_t s);
 size_t mla_decode_mma_workspace(int batch, int H, int r, int dr);
 }  // namespace b200
@@ -128,9 +133,20 @@ extern "C" int b200_mla_decode(const void* q_abs, const void* q_rope, const void
                                int64_t num_blocks, float scale, void* workspace,
                                size_t workspace_bytes, int32_t dtype, int32_t* status,
                                void* stream) {
+  return b200_mla_decode_window(q_abs, q_rope, latent_cache, out_latent, block_tables, bt_stride, context_lens, batch,
+                                num_heads, kv_lora_rank, rope_dim, block_size, num_blocks, scale, 0, nullptr, workspace,
+                                workspace_bytes, dtype, status, stream);
+}
+
+extern "C" int b200_mla_decode_window(const void* q_abs, const void* q_rope, const void* latent_cache, void* out_latent,
+                                      const int32_t* block_tables, int64_t bt_stride, const int64_t* context_lens,
+                                      int32_t batch, int32_t num_heads, int32_t kv_lora_rank, int32_t rope_dim,
+                                      int32_t block_size, int64_t num_blocks, float scale, int32_t window,
+                                      const float* sink, void* workspace, size_t workspace_bytes, int32_t dtype,
+                                      int32_t* status, void* stream) {
   using namespace b200;
   if (batch < 0 || num_heads <= 0 || kv_lora_rank <= 0 || rope_dim < 0 || block_size <= 0 ||
-      num_blocks < 0 || bt_stride <= 0)
+      num_blocks < 0 || bt_stride <= 0 || window < 0)
     return B200_ERR_ARG;
   if (dtype != B200_DTYPE_F32 && dtype != B200_DTYPE_BF16) return B200_ERR_UNSUPPORTED;
   if (batch == 0) return B200_OK;
@@ -141,7 +157,7 @@ extern "C" int b200_mla_decode(const void* q_abs, const void* q_rope, const void
   if (dtype == B200_DTYPE_BF16) {
     const int rc = mla_decode_mma_launch(q_abs, q_rope, latent_cache, out_latent, block_tables,
                                          bt_stride, context_lens, batch, num_heads, kv_lora_rank,
-                                         rope_dim, block_size, num_blocks, scale, workspace,
+                                         rope_dim, block_size, num_blocks, scale, window, sink, workspace,
                                          workspace_bytes, status, s);
     if (rc != B200_ERR_UNSUPPORTED) return rc;
   }
@@ -161,6 +177,8 @@ extern "C" int b200_mla_decode(const void* q_abs, const void* q_rope, const void
   a.bs = block_size;
   a.num_blocks = num_blocks;
   a.scale_log2 = scale * 1.4426950408889634f;
+  a.window = window;
+  a.sink = sink;
   a.status = status;
   dim3 grid(batch, num_heads);
   const bool wide = kv_lora_rank + rope_dim > 18 * 32 || kv_lora_rank > 16 * 32;

@@ -71,17 +71,21 @@ struct MlaArgs {
   int sub_log2;                 // a block-table entry is 2^sub_log2 blocks of 16 tokens
   int64_t num_blocks;           // 16-token blocks of the pool
   float scale_log2;
+  int window;                   // tokens a query sees, itself included; 0: all (EDGES kernels)
+  const float* sink;            // [H] or null (EDGES kernels)
   float* part_o;
   float* part_ml;
   int32_t* seq_info;
   int32_t* status;
 };
 
+// Blocks and tokens of a sequence count from the first block its window reaches, block `first` of its table; `lo` tokens of
+// that block lie before the window.
 struct Cursor {
-  int seq, blk, nblk, len, remaining;
+  int seq, blk, nblk, len, remaining, first, lo;
 };
 struct Group {
-  int seq, blk0, n, len, nblk;
+  int seq, blk0, n, len, nblk, lo;
   int ids[4];   // physical block ids, fetched when the group is formed (well before they are used)
 };
 
@@ -103,8 +107,9 @@ __device__ __forceinline__ void named_arrive(int id) {
   asm volatile("bar.arrive %0, %1;\n" ::"r"(id), "n"(kThreads) : "memory");
 }
 
-// PLAIN: at most 16 heads and 16-token pages, which spares the address arithmetic of the general case
-template <int R_, int DR_, bool PLAIN>
+// PLAIN: at most 16 heads and 16-token pages, which spares the address arithmetic of the general case.  EDGES: with a
+// window and sinks, either of which may be absent.
+template <int R_, int DR_, bool PLAIN, bool EDGES>
 __global__ void __launch_bounds__(kThreads, 1)
 mla_decode_mma_kernel(const MlaArgs a, const __grid_constant__ CUtensorMap tm_lat) {
   using Z = Latent<R_, DR_>;
@@ -127,7 +132,7 @@ mla_decode_mma_kernel(const MlaArgs a, const __grid_constant__ CUtensorMap tm_la
   // the combine kernel is a programmatic dependent: its CTAs may be placed while this grid runs
   asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory");
 
-  const CtaRange rg = plan_cta_range(a.lens, B, table_blocks, kTok, s_scan);
+  const CtaRange rg = plan_cta_range(a.lens, B, table_blocks, kTok, s_scan, EDGES ? a.window : 0);
   if (rg.cnt == 0) return;
   auto full_bar = [&](int half) -> uint32_t { return sbase + OFF_BAR + half * 8; };
   // Ring rows that no copy has written (blocks past the end of a group, at first) are read by phase 3
@@ -149,6 +154,13 @@ mla_decode_mma_kernel(const MlaArgs a, const __grid_constant__ CUtensorMap tm_la
     const int64_t cap = static_cast<int64_t>(c.nblk) * kTok;
     if (len > cap) report(a.status, B200_ERR_BOUNDS);
     c.len = static_cast<int>(len < cap ? len : cap);
+    c.first = c.lo = 0;
+    if (EDGES) {
+      c.first = first_kv_block(len, table_blocks, kTok, a.window);
+      c.nblk -= c.first;
+      c.len -= c.first * kTok;
+      if (a.window > 0) c.lo = max(c.len - a.window, 0);
+    }
   };
   // pool block (of 16 tokens) of a sequence's block number blk; an id outside the pool stays outside
   auto physical = [&](int seq, int blk) -> int {
@@ -164,10 +176,11 @@ mla_decode_mma_kernel(const MlaArgs a, const __grid_constant__ CUtensorMap tm_la
     gr.blk0 = c.blk;
     gr.len = c.len;
     gr.nblk = c.nblk;
+    gr.lo = c.lo;
     gr.n = min(GROUP, min(c.nblk - c.blk, c.remaining));
 #pragma unroll
     for (int b = 0; b < GROUP; ++b)
-      gr.ids[b] = (with_ids && b < gr.n) ? physical(gr.seq, gr.blk0 + b) : -1;
+      gr.ids[b] = (with_ids && b < gr.n) ? physical(gr.seq, (EDGES ? c.first : 0) + gr.blk0 + b) : -1;
     c.blk += gr.n;
     c.remaining -= gr.n;
     if (c.blk >= c.nblk && c.remaining > 0) {
@@ -335,9 +348,13 @@ mla_decode_mma_kernel(const MlaArgs a, const __grid_constant__ CUtensorMap tm_la
       }
       x[0] = t0 < valid ? x[0] * a.scale_log2 : -INFINITY;
       x[1] = t0 + 1 < valid ? x[1] * a.scale_log2 : -INFINITY;
+      if (EDGES && gr.blk0 == 0) {                  // tokens of the first block that the window leaves out
+        if (t0 < gr.lo) x[0] = -INFINITY;
+        if (t0 + 1 < gr.lo) x[1] = -INFINITY;
+      }
       const float mx = warp_max(fmaxf(x[0], x[1]));
       const float m_old = s_m[h], l_old = s_l[h];
-      const float m_new = fmaxf(m_old, mx);   // finite: token 0 of every group is valid
+      const float m_new = fmaxf(m_old, mx);   // finite: a token of every group is valid
       const float alpha = fast_exp2(m_old - m_new);
       const float p0 = fast_exp2(x[0] - m_new), p1 = fast_exp2(x[1] - m_new);
       const float sum = warp_sum(p0 + p1);
@@ -388,7 +405,12 @@ mla_decode_mma_kernel(const MlaArgs a, const __grid_constant__ CUtensorMap tm_la
       const bool whole = seq_end && seg_first == 0;
       const int h0 = g, h1 = g + 8;
       if (whole) {
-        const float i0 = 1.f / s_l[h0], i1 = 1.f / s_l[h1];
+        float l0 = s_l[h0], l1 = s_l[h1];
+        if (EDGES && a.sink != nullptr) {
+          if (h0 < H) l0 += sink_term(a.sink[hb + h0], s_m[h0]);
+          if (h1 < H) l1 += sink_term(a.sink[hb + h1], s_m[h1]);
+        }
+        const float i0 = 1.f / l0, i1 = 1.f / l1;
         __nv_bfloat16* ob = a.out + (static_cast<int64_t>(gr.seq) * a.H + hb) * R;
 #pragma unroll
         for (int n = 0; n < NO; ++n) {
@@ -456,7 +478,7 @@ size_t mla_decode_mma_workspace(int batch, int H, int r, int dr) {
 }
 
 namespace {
-template <int R, int DR, bool PLAIN>
+template <int R, int DR, bool PLAIN, bool EDGES>
 int launch(MlaArgs a, int64_t grid, EncodeFn enc, cudaStream_t s) {
   using Z = Latent<R, DR>;
   // The pool seen as (column within a slab: 64, token row: num_blocks * 16, slab: ROW / 64) with strides
@@ -477,12 +499,12 @@ int launch(MlaArgs a, int64_t grid, EncodeFn enc, cudaStream_t s) {
   int dev = 0;
   cudaGetDevice(&dev);
   if (dev >= 0 && dev < 64 && !configured[dev]) {
-    if (cudaFuncSetAttribute(mla_decode_mma_kernel<R, DR, PLAIN>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    if (cudaFuncSetAttribute(mla_decode_mma_kernel<R, DR, PLAIN, EDGES>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                              Z::SMEM_BYTES) != cudaSuccess)
       return B200_ERR_LAUNCH;
     configured[dev] = true;
   }
-  mla_decode_mma_kernel<R, DR, PLAIN>
+  mla_decode_mma_kernel<R, DR, PLAIN, EDGES>
       <<<dim3(static_cast<unsigned>(grid), head_groups(a.H)), kThreads, Z::SMEM_BYTES, s>>>(a, tm);
   return launch_result();
 }
@@ -490,8 +512,8 @@ int launch(MlaArgs a, int64_t grid, EncodeFn enc, cudaStream_t s) {
 
 int mla_decode_mma_launch(const void* q_abs, const void* q_rope, const void* lat, void* out,
                           const int32_t* bt, int64_t bt_stride, const int64_t* lens, int batch,
-                          int H, int r, int dr, int bs, int64_t num_blocks, float scale,
-                          void* workspace, size_t workspace_bytes, int32_t* status,
+                          int H, int r, int dr, int bs, int64_t num_blocks, float scale, int window,
+                          const float* sink, void* workspace, size_t workspace_bytes, int32_t* status,
                           cudaStream_t s) {
   if (!mla_fast_shape(H, r, dr, bs)) return B200_ERR_UNSUPPORTED;
   if (!aligned16(q_abs) || (dr > 0 && !aligned16(q_rope)) || !aligned16(lat) || !aligned16(out))
@@ -518,6 +540,8 @@ int mla_decode_mma_launch(const void* q_abs, const void* q_rope, const void* lat
   while ((kTok << a.sub_log2) < bs) ++a.sub_log2;
   a.num_blocks = num_blocks << a.sub_log2;
   a.scale_log2 = scale * 1.4426950408889634f;
+  a.window = window;
+  a.sink = sink;
   a.status = status;
   uint8_t* w = static_cast<uint8_t*>(workspace);
   a.part_o = reinterpret_cast<float*>(w);
@@ -526,9 +550,14 @@ int mla_decode_mma_launch(const void* q_abs, const void* q_rope, const void* lat
   w += align256(grid * 2 * H * 2 * sizeof(float));
   a.seq_info = reinterpret_cast<int32_t*>(w);
   const bool plain = H <= 16 && a.sub_log2 == 0;
-  const int rc = r == 512 ? (dr ? (plain ? launch<512, 64, true>(a, grid, enc, s) : launch<512, 64, false>(a, grid, enc, s))
-                                : launch<512, 0, false>(a, grid, enc, s))
-                          : (dr ? launch<256, 64, false>(a, grid, enc, s) : launch<256, 0, false>(a, grid, enc, s));
+  int rc;
+  if (window > 0 || sink != nullptr)
+    rc = r == 512 ? (dr ? launch<512, 64, false, true>(a, grid, enc, s) : launch<512, 0, false, true>(a, grid, enc, s))
+                  : (dr ? launch<256, 64, false, true>(a, grid, enc, s) : launch<256, 0, false, true>(a, grid, enc, s));
+  else
+    rc = r == 512 ? (dr ? (plain ? launch<512, 64, true, false>(a, grid, enc, s) : launch<512, 64, false, false>(a, grid, enc, s))
+                        : launch<512, 0, false, false>(a, grid, enc, s))
+                  : (dr ? launch<256, 64, false, false>(a, grid, enc, s) : launch<256, 0, false, false>(a, grid, enc, s));
   if (rc != B200_OK) return rc;
   CombineArgs c{};
   c.out = out;
@@ -539,6 +568,7 @@ int mla_decode_mma_launch(const void* q_abs, const void* q_rope, const void* lat
   c.batch = batch;
   c.H = H;
   c.D = r;
+  c.sink = sink;
   return decode_combine_launch(c, s);
 }
 

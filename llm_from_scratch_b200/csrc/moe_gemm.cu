@@ -6,6 +6,7 @@
 //   mode 0:  out[r, :]  = X[r, :] . W_e^T                      W [E, n_out, K]
 //   mode 1:  act[r, :]  = silu(X[r] . W1_e^T + b1_e) * (X[r] . W3_e^T + b3_e)   W [E, 2*d_ff, K] = [w1 | w3]
 //            (the SwiGLU of mlp.py:61-67; every intermediate rounded to bf16 like the tensor ops)
+//   mode 3:  as mode 1 with a clamped gated unit: g sigmoid(slope g) (u + 1), g = min(X W1^T, limit), u = clamp(X W3^T, +-limit)
 //
 // The operands are swapped with respect to the usual layout: the 128 rows of a WEIGHT tile are the M
 // dimension of the MMA and the (few) token rows are its N dimension (16..NPASS), so a CTA streams
@@ -51,6 +52,7 @@ struct GemmArgs {
   int num_experts;          // routed experts; groups past them are chunks of the dense tail
   int dense_rows;           // rows after the grouped ones that all use weight set `num_experts`
   int rows_single;          // mode 2: the row count of the single group (offsets is not read)
+  float limit, slope;       // mode 3
   unsigned long long* amax_key;   // mode 2: [tiles][rows_single] best (logit, row) key of the tile
 };
 
@@ -121,7 +123,7 @@ moe_gemm_kernel(const GemmArgs a, const __grid_constant__ CUtensorMap tm_w,
   if (rows <= 0) return;                                   // uniform, before any barrier / allocation
   const int npass = (rows + NPASS - 1) / NPASS;
   const int num_k = (a.k_dim + BK - 1) / BK;               // a ragged K tail is zero-filled by TMA
-  const bool swiglu = a.mode == 1;
+  const bool swiglu = a.mode == 1 || a.mode == 3;          // two weight rows per feature
   // first weight row of each 64-row half of the tile, in the [E * rows_per_expert, K] view
   const int w_rows = swiglu ? 2 * a.n_out : a.n_out;
   const int wrow_a = e * w_rows + (swiglu ? tile * 64 : tile * BM);
@@ -367,8 +369,12 @@ moe_gemm_kernel(const GemmArgs a, const __grid_constant__ CUtensorMap tm_w,
                 gv = bf16_round(gv + __bfloat162float(vec ? b1.b[x] : bg[x]));
                 uv = bf16_round(uv + __bfloat162float(vec ? b3.b[x] : bg[a.n_out + x]));
               }
-              const float sv = bf16_round(gv / (1.f + expf(-gv)));
-              o.b[x] = __float2bfloat16(sv * uv);
+              if (a.mode == 3) {
+                o.b[x] = __float2bfloat16(clamped_glu_f(gv, uv, a.limit, a.slope));
+              } else {
+                const float sv = bf16_round(gv / (1.f + expf(-gv)));
+                o.b[x] = __float2bfloat16(sv * uv);
+              }
             }
             if (vec) {
               *reinterpret_cast<uint4*>(dst) = o.u;
@@ -479,8 +485,52 @@ int launch(const GemmArgs& a, const CUtensorMap& tw, const CUtensorMap& tx, dim3
 }  // namespace
 
 int moe_gemm_rows_launch(const void* x, const void* w, const void* bias, void* out, const int32_t* expert_offsets,
-                         int64_t num_rows, int num_experts, int dense_rows, int n_out, int k_dim, int mode,
-                         int32_t* status, cudaStream_t s);
+                         int64_t num_rows, int num_experts, int dense_rows, int n_out, int k_dim, int mode, float limit,
+                         float slope, int32_t* status, cudaStream_t s);
+int grouped_linear_any_launch(const void* x, const void* w, void* out, const int32_t* expert_offsets, int64_t num_rows,
+                              int num_experts, int n_out, int k_dim, bool glu, float limit, float slope, int32_t dtype,
+                              cudaStream_t s);
+
+namespace {
+int grouped_gemm(const void* x, const void* w, const void* bias, void* out, const int32_t* expert_offsets, int64_t num_rows,
+                 int32_t num_experts, int32_t dense_rows, int32_t n_out, int32_t k_dim, int32_t mode, bool early, float limit,
+                 float slope, int32_t* status, void* stream) {
+  if (num_experts > 65535 || num_rows > 2147483647) return B200_ERR_TOO_LARGE;
+  const int64_t w_sets = num_experts + (dense_rows > 0 ? 1 : 0);
+  const bool pairs = mode == 1 || mode == 3;               // two weight rows per output feature
+  const int64_t w_rows = w_sets * (pairs ? 2 : 1) * n_out;
+  if (w_rows > 2147483647) return B200_ERR_TOO_LARGE;
+  CUtensorMap tw, tx;
+  if (!make_map(&tw, w, w_rows, k_dim, pairs ? 64 : BM) || !make_map(&tx, x, num_rows, k_dim, XBOX))
+    return B200_ERR_UNSUPPORTED;
+  GemmArgs a{};
+  a.offsets = expert_offsets;
+  a.n_out = n_out;
+  a.k_dim = k_dim;
+  a.mode = mode;
+  a.out = static_cast<__nv_bfloat16*>(out);
+  a.bias = static_cast<const __nv_bfloat16*>(bias);
+  a.status = status;
+  a.num_experts = num_experts;
+  a.dense_rows = dense_rows;
+  a.limit = limit;
+  a.slope = slope;
+  const int tiles = pairs ? (n_out + 63) / 64 : (n_out + BM - 1) / BM;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  // few rows per expert: deep ring of small stages, two CTAs per SM; otherwise 256 rows per pass
+  const int64_t grouped = num_rows - dense_rows;
+  if (grouped <= 64LL * num_experts) {
+    const dim3 grid(tiles, num_experts + (dense_rows + 63) / 64);
+    return launch<64, 4>(a, tw, tx, grid, early, s);
+  }
+  // many rows per expert: the compute-bound kernel (token rows as the MMA M side, persistent CTAs)
+  const int rc = moe_gemm_rows_launch(x, w, bias, out, expert_offsets, num_rows, num_experts, dense_rows, n_out, k_dim,
+                                      mode, limit, slope, status, s);
+  if (rc != B200_ERR_UNSUPPORTED) return rc;
+  const dim3 grid(tiles, num_experts + (dense_rows + 255) / 256);
+  return launch<256, 4>(a, tw, tx, grid, early, s);
+}
+}  // namespace
 
 }  // namespace b200
 
@@ -498,37 +548,23 @@ extern "C" int b200_moe_grouped_gemm(const void* x, const void* w, const void* b
   if (num_rows == 0) return B200_OK;
   if (!x || !w || !out || !expert_offsets) return B200_ERR_ARG;
   if (k_dim % 8 != 0 || !aligned16(x) || !aligned16(w)) return B200_ERR_ALIGN;   // TMA: 16-byte rows
-  if (num_experts > 65535 || num_rows > 2147483647) return B200_ERR_TOO_LARGE;
-  const int64_t w_sets = num_experts + (dense_rows > 0 ? 1 : 0);
-  const int64_t w_rows = w_sets * (mode == 1 ? 2 : 1) * n_out;
-  if (w_rows > 2147483647) return B200_ERR_TOO_LARGE;
-  CUtensorMap tw, tx;
-  if (!make_map(&tw, w, w_rows, k_dim, mode == 1 ? 64 : BM) || !make_map(&tx, x, num_rows, k_dim, XBOX))
-    return B200_ERR_UNSUPPORTED;
-  GemmArgs a{};
-  a.offsets = expert_offsets;
-  a.n_out = n_out;
-  a.k_dim = k_dim;
-  a.mode = mode;
-  a.out = static_cast<__nv_bfloat16*>(out);
-  a.bias = static_cast<const __nv_bfloat16*>(bias);
-  a.status = status;
-  a.num_experts = num_experts;
-  a.dense_rows = dense_rows;
-  const int tiles = mode == 1 ? (n_out + 63) / 64 : (n_out + BM - 1) / BM;
-  cudaStream_t s = static_cast<cudaStream_t>(stream);
-  // few rows per expert: deep ring of small stages, two CTAs per SM; otherwise 256 rows per pass
-  const int64_t grouped = num_rows - dense_rows;
-  if (grouped <= 64LL * num_experts) {
-    const dim3 grid(tiles, num_experts + (dense_rows + 63) / 64);
-    return launch<64, 4>(a, tw, tx, grid, early, s);
-  }
-  // many rows per expert: the compute-bound kernel (token rows as the MMA M side, persistent CTAs)
-  const int rc = moe_gemm_rows_launch(x, w, bias, out, expert_offsets, num_rows, num_experts, dense_rows, n_out, k_dim,
-                                      mode, status, s);
-  if (rc != B200_ERR_UNSUPPORTED) return rc;
-  const dim3 grid(tiles, num_experts + (dense_rows + 255) / 256);
-  return launch<256, 4>(a, tw, tx, grid, early, s);
+  return grouped_gemm(x, w, bias, out, expert_offsets, num_rows, num_experts, dense_rows, n_out, k_dim, mode, early, 0.f, 0.f,
+                      status, stream);
+}
+
+extern "C" int b200_moe_grouped_linear(const void* x, const void* w, void* out, const int32_t* expert_offsets, int64_t num_rows,
+                                       int32_t num_experts, int32_t n_out, int32_t k_dim, int32_t glu, float limit, float slope,
+                                       int32_t flags, int32_t dtype, int32_t* status, void* stream) {
+  using namespace b200;
+  if (num_rows < 0 || num_experts <= 0 || n_out <= 0 || k_dim <= 0 || (flags & ~B200_MOE_GEMM_EARLY_LAUNCH)) return B200_ERR_ARG;
+  if (dtype != B200_DTYPE_F32 && dtype != B200_DTYPE_BF16) return B200_ERR_UNSUPPORTED;
+  if (num_rows == 0) return B200_OK;
+  if (!x || !w || !out || !expert_offsets) return B200_ERR_ARG;
+  if (dtype == B200_DTYPE_BF16 && k_dim % 8 == 0 && n_out % 8 == 0 && aligned16(x) && aligned16(w) && aligned16(out))
+    return grouped_gemm(x, w, nullptr, out, expert_offsets, num_rows, num_experts, 0, n_out, k_dim, glu ? 3 : 0,
+                        (flags & B200_MOE_GEMM_EARLY_LAUNCH) != 0, limit, slope, status, stream);
+  return grouped_linear_any_launch(x, w, out, expert_offsets, num_rows, num_experts, n_out, k_dim, glu != 0, limit, slope, dtype,
+                                   static_cast<cudaStream_t>(stream));
 }
 
 /* Greedy head: tokens[r] = argmax_v bf16(hidden[r] . W[v] + bias[v]), lowest v among equal maxima. */

@@ -11,6 +11,7 @@
 //   mode 1:  a tile holds 128 rows of w1 and the matching 128 rows of w3 of the same features, so
 //            act[r, f0 .. f0+127] = silu(X[r] . W1^T + b1) * (X[r] . W3^T + b3) is formed in the epilogue and the
 //            [rows, 2 * d_ff] intermediate is never written
+//   mode 3:  as mode 1 with the clamped gated unit of moe_gemm.cu
 //
 // Persistent CTAs (one per SM) walk the list of (group, 256-row tile, column tile) work items, column tile
 // fastest; groups are the experts' row ranges (read from expert_offsets on the device) plus, when
@@ -48,6 +49,7 @@ struct RowsArgs {
   int n_out, k_dim, mode;
   __nv_bfloat16* out;         // [R, n_out]
   const __nv_bfloat16* bias;  // mode 0: [sets, n_out]; mode 1: [sets, 2 * n_out]; or null
+  float limit, slope;         // mode 3
   int32_t* status;
 };
 
@@ -79,7 +81,7 @@ moe_gemm_rows_kernel(const RowsArgs a, const __grid_constant__ CUtensorMap tm_x,
   auto bar = [&](int i) -> uint32_t { return sb + OFF_BAR + i * 8; };
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const bool swiglu = a.mode == 1;
+  const bool swiglu = a.mode == 1 || a.mode == 3;            // two weight rows per feature
   const int groups = a.num_experts + (a.dense_rows > 0 ? 1 : 0);
   const int feat_per_tile = swiglu ? BN / 2 : BN;            // output columns an item produces
   const int n_tiles = (a.n_out + feat_per_tile - 1) / feat_per_tile;
@@ -260,8 +262,12 @@ moe_gemm_rows_kernel(const RowsArgs a, const __grid_constant__ CUtensorMap tm_x,
                 uv = bf16r(uv + __bfloat162float(b3.b[x]));
               }
               // fast exponential and division: their ~1e-6 relative error disappears in the bf16 rounding of silu
-              const float sv = bf16r(__fdividef(gv, 1.f + __expf(-gv)));
-              o.b[x] = __float2bfloat16(sv * uv);
+              if (a.mode == 3) {
+                o.b[x] = __float2bfloat16(clamped_glu_f(gv, uv, a.limit, a.slope));
+              } else {
+                const float sv = bf16r(__fdividef(gv, 1.f + __expf(-gv)));
+                o.b[x] = __float2bfloat16(sv * uv);
+              }
             }
             *reinterpret_cast<uint4*>(orow + c + e8) = o.u;
           }
@@ -338,11 +344,11 @@ bool rows_make_map(CUtensorMap* m, const void* base, int64_t rows, int64_t k) {
 // Launch for the compute-bound regime; B200_ERR_UNSUPPORTED for shapes it does not take (the caller then uses
 // the weight-streaming kernel with several passes).
 int moe_gemm_rows_launch(const void* x, const void* w, const void* bias, void* out, const int32_t* expert_offsets,
-                         int64_t num_rows, int num_experts, int dense_rows, int n_out, int k_dim, int mode,
-                         int32_t* status, cudaStream_t s) {
+                         int64_t num_rows, int num_experts, int dense_rows, int n_out, int k_dim, int mode, float limit,
+                         float slope, int32_t* status, cudaStream_t s) {
   if (n_out % 8 != 0 || k_dim % 8 != 0 || num_experts + 1 >= kMaxGroups) return B200_ERR_UNSUPPORTED;
   const int64_t w_sets = num_experts + (dense_rows > 0 ? 1 : 0);
-  const int64_t w_rows = w_sets * (mode == 1 ? 2 : 1) * n_out;
+  const int64_t w_rows = w_sets * (mode == 1 || mode == 3 ? 2 : 1) * n_out;
   if (w_rows > 2147483647LL || num_rows > 2147483647LL) return B200_ERR_UNSUPPORTED;
   CUtensorMap tx, tw;
   if (!rows_make_map(&tx, x, num_rows, k_dim) || !rows_make_map(&tw, w, w_rows, k_dim)) return B200_ERR_UNSUPPORTED;
@@ -368,9 +374,11 @@ int moe_gemm_rows_launch(const void* x, const void* w, const void* bias, void* o
   a.mode = mode;
   a.out = static_cast<__nv_bfloat16*>(out);
   a.bias = static_cast<const __nv_bfloat16*>(bias);
+  a.limit = limit;
+  a.slope = slope;
   a.status = status;
   // upper bound of the work items, so that small problems do not launch idle CTAs
-  const int64_t feat = mode == 1 ? BN / 2 : BN;
+  const int64_t feat = mode == 1 || mode == 3 ? BN / 2 : BN;
   const int64_t max_items = ((num_rows + BM - 1) / BM + w_sets) * ((n_out + feat - 1) / feat);
   const int grid = static_cast<int>(max_items < sms ? (max_items > 0 ? max_items : 1) : sms);
   moe_gemm_rows_kernel<<<grid, kThreads, SMEM, s>>>(a, tx, tw);

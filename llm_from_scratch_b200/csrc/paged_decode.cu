@@ -589,6 +589,7 @@ int decode_combine_launch(const CombineArgs& c, cudaStream_t s) {
   a.batch = c.batch;
   a.Hq = c.H;
   a.D = c.D;
+  a.sink = c.sink;
   return launch_combine(a, c.batch, s);
 }
 

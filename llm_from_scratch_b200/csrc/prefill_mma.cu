@@ -11,6 +11,9 @@
 // The grid is (query heads, sequences, query tiles) with the tile index reversed, so that the
 // tiles with the most keys are scheduled first and the short tail of a ragged batch fills the
 // gaps; CTAs whose tile lies past the end of their sequence return at once.
+//
+// The general variant serves head sizes that are smaller than the compiled ones (any multiples of eight), a key part shared by
+// all heads of any such width, and a sliding window: the walk starts at the first tile the window of row 0 reaches.
 #include "common.cuh"
 
 namespace b200 {
@@ -42,6 +45,8 @@ struct MmaArgs {
   int bs;
   int64_t num_blocks;
   const float* sink;     // [Hq] or null
+  int dqk, dv, tail;     // general variant: head sizes and width of the shared key part
+  int window;            // general variant: keys a query sees, its own included; 0: all
   int32_t* status;
 };
 
@@ -52,7 +57,7 @@ __device__ __forceinline__ int swz(int c, int row) {
   return c ^ ((row >> 1) & (CPR - 1));
 }
 
-template <int DQK, int DV, bool PAGED, int TAIL = 0>
+template <int DQK, int DV, bool PAGED, int TAIL = 0, bool GENERAL = false>
 __global__ void __launch_bounds__(kThreads, 2) prefill_mma_kernel(const MmaArgs a) {
   extern __shared__ __align__(128) uint8_t smem[];
   constexpr int KQ = DQK / 16;   // k-steps of S
@@ -71,10 +76,17 @@ __global__ void __launch_bounds__(kThreads, 2) prefill_mma_kernel(const MmaArgs 
     tile = a.ntiles_max - 1 - blockIdx.z;
   }
   const int q0 = a.cu_q[seq], q_len = a.cu_q[seq + 1] - q0;
-  const int k0 = a.cu_k[seq], k_len = a.cu_k[seq + 1] - k0;
+  int k0 = a.cu_k[seq], k_len = a.cu_k[seq + 1] - k0;
   const int m0 = tile * BM;
   if (m0 >= q_len) return;
-  const int off = k_len - q_len;                 // keys every new token sees besides its own prefix
+  int off = k_len - q_len;                       // keys every new token sees besides its own prefix
+  if (GENERAL && a.window > 0) {                 // keys count from the first tile that row 0 sees
+    const int skip = max(0, off + m0 - a.window + 1) / BN * BN;
+    k0 += skip;
+    k_len -= skip;
+    off -= skip;
+  }
+  const int dqk = GENERAL ? a.dqk : DQK, dv = GENERAL ? a.dv : DV;
   const int kvh = head / (a.Hq / a.Hkv);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, tq = lane & 3;
   const int rows_q = min(BM, q_len - m0);
@@ -111,6 +123,29 @@ __global__ void __launch_bounds__(kThreads, 2) prefill_mma_kernel(const MmaArgs 
     const int n0 = j * BN;
     const int valid = min(BN, kmax - n0);
     constexpr int CPRK = DQK / 8, CPRV = DV / 8;
+    if constexpr (GENERAL) {
+      const int dh = dqk - a.tail;                 // columns per head, then the tail, then zeros
+#pragma unroll 4
+      for (int i = 0; i < BN * CPRK / kThreads; ++i) {
+        const int idx = threadIdx.x + i * kThreads;
+        const int r = idx / CPRK, c = idx % CPRK;
+        const int64_t row = k0 + n0 + r;
+        const __nv_bfloat16* src = c * 8 < dh ? a.k + row * a.k_stride + static_cast<int64_t>(kvh) * dh + c * 8
+                                              : a.k_tail + row * a.k_tail_stride + (c * 8 - dh);
+        const bool ok = r < valid && c * 8 < dqk;
+        cp_async16(sK + stage * KB + r * (DQK * 2) + swz<DQK>(c, r) * 16, ok ? src : dummy, ok ? 16 : 0);
+      }
+#pragma unroll 4
+      for (int i = 0; i < BN * CPRV / kThreads; ++i) {
+        const int idx = threadIdx.x + i * kThreads;
+        const int r = idx / CPRV, c = idx % CPRV;
+        const bool ok = r < valid && c * 8 < dv;
+        cp_async16(sV + stage * VB + r * (DV * 2) + swz<DV>(c, r) * 16,
+                   ok ? a.v + static_cast<int64_t>(k0 + n0 + r) * a.v_stride + static_cast<int64_t>(kvh) * dv + c * 8 : dummy,
+                   ok ? 16 : 0);
+      }
+      return;
+    }
     if constexpr (TAIL == 0) {
 #pragma unroll
       for (int i = 0; i < BN * CPRK / kThreads; ++i) {
@@ -157,10 +192,10 @@ __global__ void __launch_bounds__(kThreads, 2) prefill_mma_kernel(const MmaArgs 
     for (int i = 0; i < BM * CPR / kThreads; ++i) {
       const int idx = threadIdx.x + i * kThreads;
       const int r = idx / CPR, c = idx % CPR;
-      const bool ok = r < rows_q;
+      const bool ok = r < rows_q && (!GENERAL || c * 8 < dqk);
       const __nv_bfloat16* src =
           a.q + static_cast<int64_t>(q0 + m0 + (ok ? r : 0)) * a.q_stride +
-          static_cast<int64_t>(head) * DQK + c * 8;
+          static_cast<int64_t>(head) * dqk + (ok ? c * 8 : 0);
       cp_async16(sQ + r * (DQK * 2) + swz<DQK>(c, r) * 16, src, ok ? 16 : 0);
     }
   }
@@ -217,7 +252,9 @@ __global__ void __launch_bounds__(kThreads, 2) prefill_mma_kernel(const MmaArgs 
     }
     // ---- scale, causal / length mask, online softmax ----
     const int n0 = j * BN;
-    const bool need_mask = (n0 + BN - 1 > off + m0 + warp * 16) || (n0 + BN > kmax);
+    const bool windowed = GENERAL && a.window > 0;
+    const bool need_mask = (n0 + BN - 1 > off + m0 + warp * 16) || (n0 + BN > kmax) ||
+                           (windowed && n0 <= off + m0 + warp * 16 + 15 - a.window);
     float mx0 = -INFINITY, mx1 = -INFINITY;
 #pragma unroll
     for (int n = 0; n < BN / 8; ++n) {
@@ -230,6 +267,13 @@ __global__ void __launch_bounds__(kThreads, 2) prefill_mma_kernel(const MmaArgs 
         if (key + 1 > lim0) s[n][1] = -INFINITY;
         if (key > lim1) s[n][2] = -INFINITY;
         if (key + 1 > lim1) s[n][3] = -INFINITY;
+        if (windowed) {
+          const int low0 = off + row0 - a.window, low1 = low0 + 8;      // last key before the window
+          if (key <= low0) s[n][0] = -INFINITY;
+          if (key + 1 <= low0) s[n][1] = -INFINITY;
+          if (key <= low1) s[n][2] = -INFINITY;
+          if (key + 1 <= low1) s[n][3] = -INFINITY;
+        }
       }
       mx0 = fmaxf(mx0, fmaxf(s[n][0], s[n][1]));
       mx1 = fmaxf(mx1, fmaxf(s[n][2], s[n][3]));
@@ -299,26 +343,27 @@ __global__ void __launch_bounds__(kThreads, 2) prefill_mma_kernel(const MmaArgs 
   }
   const float i0 = l0 > 0.f ? 1.f / l0 : 0.f, i1 = l1 > 0.f ? 1.f / l1 : 0.f;
   const int r0 = warp * 16 + g, r1 = r0 + 8;
-  __nv_bfloat16* ob = a.out + (static_cast<int64_t>(q0 + m0) * a.Hq + head) * DV;
+  __nv_bfloat16* ob = a.out + (static_cast<int64_t>(q0 + m0) * a.Hq + head) * dv;
 #pragma unroll
   for (int n = 0; n < NV; ++n) {
     const int d = n * 8 + tq * 2;
+    if (GENERAL && d >= dv) continue;
     if (r0 < rows_q)
-      *reinterpret_cast<uint32_t*>(ob + static_cast<int64_t>(r0) * a.Hq * DV + d) =
+      *reinterpret_cast<uint32_t*>(ob + static_cast<int64_t>(r0) * a.Hq * dv + d) =
           pack_bf16x2(o[n][0] * i0, o[n][1] * i0);
     if (r1 < rows_q)
-      *reinterpret_cast<uint32_t*>(ob + static_cast<int64_t>(r1) * a.Hq * DV + d) =
+      *reinterpret_cast<uint32_t*>(ob + static_cast<int64_t>(r1) * a.Hq * dv + d) =
           pack_bf16x2(o[n][2] * i1, o[n][3] * i1);
   }
 }
 
-template <int DQK, int DV, int TAIL = 0>
+template <int DQK, int DV, int TAIL = 0, bool GENERAL = false>
 int launch(const MmaArgs& a, int num_seqs, int plan_capacity, bool paged, cudaStream_t s) {
   constexpr size_t smem = size_t(BM) * DQK * 2 + 2 * size_t(BN) * DQK * 2 + 2 * size_t(BN) * DV * 2;
   static bool configured[64][2] = {};
   int dev = 0;
   cudaGetDevice(&dev);
-  auto kern = paged ? prefill_mma_kernel<DQK, DV, true, 0> : prefill_mma_kernel<DQK, DV, false, TAIL>;
+  auto kern = paged ? prefill_mma_kernel<DQK, DV, !GENERAL, 0, GENERAL> : prefill_mma_kernel<DQK, DV, false, TAIL, GENERAL>;
   if (dev >= 0 && dev < 64 && !configured[dev][paged]) {
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize,
                              static_cast<int>(smem)) != cudaSuccess)
@@ -388,6 +433,50 @@ int prefill_mma_launch(const void* q, const void* k, const void* v, void* out, i
   if (Dqk == 128) return launch<128, 128>(a, num_seqs, plan_capacity, paged, s);
   if (Dqk == 64) return launch<64, 64>(a, num_seqs, plan_capacity, paged, s);
   return launch<32, 32>(a, num_seqs, plan_capacity, paged, s);
+}
+
+// Head sizes up to 192 / 128 in multiples of eight on the next larger compiled ones, packed keys.
+bool prefill_mma_general_shape(int Dqk, int Dv, int tail) {
+  return Dqk <= 192 && Dv <= 128 && Dqk % 8 == 0 && Dv % 8 == 0 && tail % 8 == 0;
+}
+
+int prefill_mma_general_launch(const void* q, const void* k, const void* v, void* out, int64_t q_stride, int64_t k_stride,
+                               int64_t v_stride, const int32_t* cu_q, const int32_t* cu_k, int num_seqs, int max_seqlen_q,
+                               int Hq, int Hkv, int Dqk, int Dv, float scale, const int32_t* plan, int plan_tile_rows,
+                               int plan_capacity, int32_t* status, cudaStream_t s, const void* k_tail, int64_t k_tail_stride,
+                               int tail, const float* sink, int window) {
+  if (!prefill_mma_general_shape(Dqk, Dv, tail)) return B200_ERR_UNSUPPORTED;
+  const int ntiles = (max_seqlen_q + BM - 1) / BM;
+  if (num_seqs > 65535 || ntiles > 65535) return B200_ERR_UNSUPPORTED;
+  auto al = [](const void* p, int64_t stride) { return aligned16(p) && (stride * 2) % 16 == 0; };
+  if (!al(q, q_stride) || !al(k, k_stride) || !al(v, v_stride) || !aligned16(out) || (tail > 0 && !al(k_tail, k_tail_stride)))
+    return B200_ERR_UNSUPPORTED;
+  MmaArgs a{};
+  a.q = static_cast<const __nv_bfloat16*>(q);
+  a.k = static_cast<const __nv_bfloat16*>(k);
+  a.v = static_cast<const __nv_bfloat16*>(v);
+  a.out = static_cast<__nv_bfloat16*>(out);
+  a.q_stride = q_stride;
+  a.k_stride = k_stride;
+  a.v_stride = v_stride;
+  a.k_tail = static_cast<const __nv_bfloat16*>(k_tail);
+  a.k_tail_stride = k_tail_stride;
+  a.cu_q = cu_q;
+  a.cu_k = cu_k;
+  a.Hq = Hq;
+  a.Hkv = Hkv;
+  a.ntiles_max = ntiles;
+  a.plan = (plan != nullptr && plan_tile_rows == BM && plan_capacity > 0 && plan_capacity <= 65535) ? plan : nullptr;
+  a.scale_log2 = scale * 1.4426950408889634f;
+  a.sink = sink;
+  a.dqk = Dqk;
+  a.dv = Dv;
+  a.tail = tail;
+  a.window = window;
+  a.status = status;
+  if (Dqk <= 64 && Dv <= 64) return launch<64, 64, 0, true>(a, num_seqs, plan_capacity, false, s);
+  if (Dqk <= 128) return launch<128, 128, 0, true>(a, num_seqs, plan_capacity, false, s);
+  return launch<192, 128, 0, true>(a, num_seqs, plan_capacity, false, s);
 }
 
 }  // namespace b200

@@ -19,7 +19,8 @@
 // the scores of tile j + 1 into the other buffer before it waits for the probabilities of tile j, so the
 // softmax warps find their next tile ready, and one problem's waits never hold up the other's instructions.
 // K/V tiles go through a ring of NST stages that both problems release.  Rescaling of O is lazy as in
-// prefill_umma.cu and waits for the P.V product before it.  Every wait is bounded; a timeout aborts the CTA
+// prefill_umma.cu and waits for the P.V product before it.  With a sliding window (WINDOW) the walk starts at the first
+// tile that the window of row 0 reaches; problem B meets up to three fully masked tiles there.  Every wait is bounded; a timeout aborts the CTA
 // and is reported.
 //
 // What sets the pace, measured with clock counters in the warps: (1) the special-function unit — the 64
@@ -75,10 +76,11 @@ struct Args2 {
   const int32_t* plan;   // tile list for 256-row tiles (see b200_prefill_plan) or null: grid (head, seq, tile rank)
   float scale_log2;
   const float* sink;     // [Hq] or null
+  int window;            // keys a query sees, its own included (WINDOW kernels)
   int32_t* status;
 };
 
-template <int DQK, int DV, bool TAIL>
+template <int DQK, int DV, bool TAIL, bool WINDOW>
 __global__ void __launch_bounds__(kThreads, 1)
 prefill_umma2_kernel(const Args2 a, const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k,
                      const __grid_constant__ CUtensorMap tm_kt, const __grid_constant__ CUtensorMap tm_v) {
@@ -104,10 +106,16 @@ prefill_umma2_kernel(const Args2 a, const __grid_constant__ CUtensorMap tm_q, co
     tile = a.ntiles_max - 1 - blockIdx.z;
   }
   const int q0 = a.cu_q[seq], q_len = a.cu_q[seq + 1] - q0;
-  const int k0 = a.cu_k[seq], k_len = a.cu_k[seq + 1] - k0;
+  int k0 = a.cu_k[seq], k_len = a.cu_k[seq + 1] - k0;
   const int m0 = tile * ROWS;
   if (m0 >= q_len) return;                       // uniform over the CTA, before any barrier / allocation
-  const int off = k_len - q_len;
+  int off = k_len - q_len;
+  if (WINDOW) {                                  // keys count from the first tile that row 0 sees
+    const int skip = max(0, off + m0 - a.window + 1) / BN * BN;
+    k0 += skip;
+    k_len -= skip;
+    off -= skip;
+  }
   const int kvh = head / (a.Hq / a.Hkv);
   // rows and visible keys of the two problems; B may be empty (the sequence ends inside A)
   int rows[2], kmax[2], nt[2];
@@ -246,6 +254,7 @@ prefill_umma2_kernel(const Args2 a, const __grid_constant__ CUtensorMap tm_q, co
     const uint32_t tS0 = tmem + x * (128 + DV) + lane_sel, tOx = tS0 + 128;
     const int qrow = m0 + x * BM + row;                     // index of the query inside its sequence
     const int lim = min(off + qrow, kmax[x] - 1);           // last visible key
+    const int low = WINDOW ? off + qrow - a.window + 1 : 0; // first visible key (may be negative)
     const int nx = nt[x];
     const uint32_t qk_done = bar(L::QK_DONE + x), pv_done = bar(L::PV_DONE + x);
     const uint32_t my_turn = bar(L::TURN + (x == 0 ? 0 : 4) + (warp & 3));
@@ -263,7 +272,7 @@ prefill_umma2_kernel(const Args2 a, const __grid_constant__ CUtensorMap tm_q, co
       }
       umma::fence_after_sync();
       const int n0 = j * BN;
-      const bool warp_masked = __any_sync(0xffffffffu, n0 + BN - 1 > lim);
+      const bool warp_masked = __any_sync(0xffffffffu, n0 + BN - 1 > lim || (WINDOW && n0 < low));
       // the 64 raw scores of the row stay in registers for both passes
       uint32_t ra[32], rb[32];
       umma::tmem_ld32(tSx, ra);
@@ -272,7 +281,7 @@ prefill_umma2_kernel(const Args2 a, const __grid_constant__ CUtensorMap tm_q, co
       if (warp_masked) {
 #pragma unroll
         for (int e = 0; e < 32; ++e)
-          if (n0 + e > lim) ra[e] = 0xff800000u;            // -inf
+          if (n0 + e > lim || (WINDOW && n0 + e < low)) ra[e] = 0xff800000u;            // -inf
       }
 #pragma unroll
       for (int e = 0; e < 32; e += 2) {
@@ -283,7 +292,7 @@ prefill_umma2_kernel(const Args2 a, const __grid_constant__ CUtensorMap tm_q, co
       if (warp_masked) {
 #pragma unroll
         for (int e = 0; e < 32; ++e)
-          if (n0 + 32 + e > lim) rb[e] = 0xff800000u;
+          if (n0 + 32 + e > lim || (WINDOW && n0 + 32 + e < low)) rb[e] = 0xff800000u;
       }
 #pragma unroll
       for (int e = 0; e < 32; e += 2) {
@@ -436,7 +445,7 @@ bool make_map2(CUtensorMap* m, const void* base, int64_t tokens, int heads, int 
              CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
-template <int DQK, int DV, bool TAIL>
+template <int DQK, int DV, bool TAIL, bool WINDOW>
 int launch2(const Args2& a, const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tkt,
             const CUtensorMap& tv, dim3 grid, cudaStream_t s) {
   using L = Lay<DQK, DV>;
@@ -445,7 +454,7 @@ int launch2(const Args2& a, const CUtensorMap& tq, const CUtensorMap& tk, const 
   int dev = 0;
   cudaGetDevice(&dev);
   if (dev < 0 || dev >= 64) return B200_ERR_UNSUPPORTED;
-  auto kern = prefill_umma2_kernel<DQK, DV, TAIL>;
+  auto kern = prefill_umma2_kernel<DQK, DV, TAIL, WINDOW>;
   if (!configured[dev]) {
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, L::SMEM) != cudaSuccess)
       return B200_ERR_LAUNCH;
@@ -474,7 +483,7 @@ int prefill_umma2_launch(const void* q, const void* k, const void* v, void* out,
                          int64_t v_stride, int64_t total_q, int64_t total_k, const int32_t* cu_q,
                          const int32_t* cu_k, int num_seqs, int max_seqlen_q, int Hq, int Hkv, int Dqk, int Dv,
                          float scale, const int32_t* plan, int plan_tile_rows, int plan_capacity, int32_t* status,
-                         cudaStream_t s, const void* k_tail, int64_t k_tail_stride, int tail, const float* sink) {
+                         cudaStream_t s, const void* k_tail, int64_t k_tail_stride, int tail, const float* sink, int window) {
   if (prefill_umma2_tile_rows(Hq, Hkv, Dqk, Dv) == 0) return B200_ERR_UNSUPPORTED;
   if (tail != 0 && (tail != 64 || Dqk != 192 || k_tail == nullptr)) return B200_ERR_UNSUPPORTED;
   if (!(scale > 0.f)) return B200_ERR_UNSUPPORTED;   // the row maximum is taken before scaling
@@ -493,6 +502,7 @@ int prefill_umma2_launch(const void* q, const void* k, const void* v, void* out,
   a.plan = (plan != nullptr && plan_tile_rows == ROWS && plan_capacity > 0 && plan_capacity <= 65535) ? plan : nullptr;
   a.scale_log2 = scale * 1.4426950408889634f;
   a.sink = sink;
+  a.window = window;
   a.status = status;
   CUtensorMap tq, tk, tkt, tv;
   memset(&tq, 0, sizeof(tq));
@@ -505,11 +515,14 @@ int prefill_umma2_launch(const void* q, const void* k, const void* v, void* out,
   if (tail && !make_map2(&tkt, k_tail, total_k, 1, tail, k_tail_stride, BN)) return B200_ERR_UNSUPPORTED;
   dim3 grid(Hq, num_seqs, ntiles);
   if (a.plan) grid = dim3(Hq, plan_capacity, 1);
-  if (Dqk == 192) {
-    return tail ? launch2<192, 128, true>(a, tq, tk, tkt, tv, grid, s)
-                : launch2<192, 128, false>(a, tq, tk, tkt, tv, grid, s);
+  if (window > 0) {
+    if (Dqk == 128) return launch2<128, 128, false, true>(a, tq, tk, tkt, tv, grid, s);
+    return tail ? launch2<192, 128, true, true>(a, tq, tk, tkt, tv, grid, s)
+                : launch2<192, 128, false, true>(a, tq, tk, tkt, tv, grid, s);
   }
-  return launch2<128, 128, false>(a, tq, tk, tkt, tv, grid, s);
+  if (Dqk == 128) return launch2<128, 128, false, false>(a, tq, tk, tkt, tv, grid, s);
+  return tail ? launch2<192, 128, true, false>(a, tq, tk, tkt, tv, grid, s)
+              : launch2<192, 128, false, false>(a, tq, tk, tkt, tv, grid, s);
 }
 
 }  // namespace b200

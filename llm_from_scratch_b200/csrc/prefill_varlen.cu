@@ -3,7 +3,8 @@
 // Generic path: one warp per (sequence, query token, query head); a lane owns the head-dim
 // elements lane, lane+32, ...; keys are visited in order with an fp32 online softmax.  Keys and
 // values come either from the packed k/v tensors of the step or, when a cached prefix exists,
-// from the paged pool through block_tables (bottom-right aligned causal mask).
+// from the paged pool through block_tables (bottom-right aligned causal mask).  The packed keys may come in two parts, the
+// second shared by all heads, and a query may see only the last `window` keys.
 #include "common.cuh"
 
 namespace b200 {
@@ -26,13 +27,18 @@ struct PrefillArgs {
   int bs;
   int64_t num_blocks;
   const float* sink;  // [Hq] or null
+  const void* k_tail; // [Tk, tail] or null (packed keys): the last `tail` columns of every head's key
+  int64_t k_tail_stride;
+  int tail;
+  int window;         // 0: none
   int32_t* status;
 };
 
 constexpr int kWarps = 4;
-constexpr int kMaxPerLane = 8;  // head dims <= 256
+constexpr int kMaxPerLane = 8;    // head dims <= 256
+constexpr int kWidePerLane = 32;  // head dims <= 1024
 
-template <typename T>
+template <typename T, int kMaxPerLane>
 __global__ void __launch_bounds__(kWarps * 32) prefill_simple_kernel(const PrefillArgs a) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int s = blockIdx.z, head = blockIdx.y;
@@ -52,12 +58,14 @@ __global__ void __launch_bounds__(kWarps * 32) prefill_simple_kernel(const Prefi
     acc[i] = 0.f;
   }
   float m = -INFINITY, l = 0.f;
-  for (int j = 0; j < nkeys; ++j) {
+  const int Dh = a.Dqk - a.tail;
+  for (int j = a.window > 0 ? max(nkeys - a.window, 0) : 0; j < nkeys; ++j) {
     const T* kp;
+    const T* kt = nullptr;
     const T* vp;
     if (a.bt == nullptr) {
-      kp = static_cast<const T*>(a.k) + static_cast<int64_t>(k0 + j) * a.k_stride +
-           static_cast<int64_t>(kvh) * a.Dqk;
+      kp = static_cast<const T*>(a.k) + static_cast<int64_t>(k0 + j) * a.k_stride + static_cast<int64_t>(kvh) * Dh;
+      if (a.tail > 0) kt = static_cast<const T*>(a.k_tail) + static_cast<int64_t>(k0 + j) * a.k_tail_stride;
       vp = static_cast<const T*>(a.v) + static_cast<int64_t>(k0 + j) * a.v_stride +
            static_cast<int64_t>(kvh) * a.Dv;
     } else {
@@ -79,7 +87,8 @@ __global__ void __launch_bounds__(kWarps * 32) prefill_simple_kernel(const Prefi
 #pragma unroll
     for (int i = 0; i < kMaxPerLane; ++i) {
       const int d = lane + 32 * i;
-      if (d < a.Dqk) dot += qv[i] * to_float<T>(kp[d]);
+      if (d < Dh) dot += qv[i] * to_float<T>(kp[d]);
+      else if (d < a.Dqk) dot += qv[i] * to_float<T>(kt[d - Dh]);
     }
     dot = warp_sum(dot) * a.scale_log2;
     const float mn = fmaxf(m, dot);
@@ -126,7 +135,16 @@ int prefill_umma2_launch(const void* q, const void* k, const void* v, void* out,
                          int64_t v_stride, int64_t total_q, int64_t total_k, const int32_t* cu_q,
                          const int32_t* cu_k, int num_seqs, int max_seqlen_q, int Hq, int Hkv, int Dqk, int Dv,
                          float scale, const int32_t* plan, int plan_tile_rows, int plan_capacity, int32_t* status,
-                         cudaStream_t s, const void* k_tail, int64_t k_tail_stride, int tail, const float* sink);
+                         cudaStream_t s, const void* k_tail, int64_t k_tail_stride, int tail, const float* sink,
+                         int window);
+
+// mma.sync path for head sizes below the compiled ones, keys in two parts, a sliding window (prefill_mma.cu); packed keys
+bool prefill_mma_general_shape(int Dqk, int Dv, int tail);
+int prefill_mma_general_launch(const void* q, const void* k, const void* v, void* out, int64_t q_stride, int64_t k_stride,
+                               int64_t v_stride, const int32_t* cu_q, const int32_t* cu_k, int num_seqs, int max_seqlen_q,
+                               int Hq, int Hkv, int Dqk, int Dv, float scale, const int32_t* plan, int plan_tile_rows,
+                               int plan_capacity, int32_t* status, cudaStream_t s, const void* k_tail, int64_t k_tail_stride,
+                               int tail, const float* sink, int window);
 
 // tcgen05 path for a paged prefix (prefill_umma.cu): head_dim 128, even group size, two heads per CTA
 int prefill_umma_launch(const void* q, const void* k, const void* v, void* out, int64_t q_stride,
@@ -151,6 +169,25 @@ extern "C" int32_t b200_prefill_tile_rows(int32_t num_q_heads, int32_t num_kv_he
                    (head_dim_qk == 192 && head_dim_v == 128);
   return mma ? 64 : 0;
 }
+
+namespace b200 {
+namespace {
+int simple_launch(const PrefillArgs& a, int max_seqlen_q, int32_t dtype, cudaStream_t s) {
+  const int widest = a.Dqk > a.Dv ? a.Dqk : a.Dv;
+  if (widest > kWidePerLane * 32 || a.num_seqs > 65535 || a.Hq > 65535) return B200_ERR_UNSUPPORTED;
+  const dim3 grid((max_seqlen_q + kWarps - 1) / kWarps, a.Hq, a.num_seqs);
+  const bool wide = widest > kMaxPerLane * 32;
+  if (dtype == B200_DTYPE_F32) {
+    if (wide) prefill_simple_kernel<float, kWidePerLane><<<grid, kWarps * 32, 0, s>>>(a);
+    else prefill_simple_kernel<float, kMaxPerLane><<<grid, kWarps * 32, 0, s>>>(a);
+  } else {
+    if (wide) prefill_simple_kernel<__nv_bfloat16, kWidePerLane><<<grid, kWarps * 32, 0, s>>>(a);
+    else prefill_simple_kernel<__nv_bfloat16, kMaxPerLane><<<grid, kWarps * 32, 0, s>>>(a);
+  }
+  return launch_result();
+}
+}  // namespace
+}  // namespace b200
 
 static int prefill_attention(const void* q, const void* k, const void* v, void* out,
                                    int64_t q_token_stride, int64_t k_token_stride,
@@ -201,7 +238,7 @@ static int prefill_attention(const void* q, const void* k, const void* v, void* 
       const int rc2 = prefill_umma2_launch(q, k, v, out, q_token_stride, k_token_stride, v_token_stride,
                                            total_q_tokens, total_k_tokens, cu_seqlens_q, cu_seqlens_k, num_seqs,
                                            max_seqlen_q, num_q_heads, num_kv_heads, head_dim_qk, head_dim_v, scale,
-                                           plan, plan_tile_rows, plan_capacity, status, s, nullptr, 0, 0, sink);
+                                           plan, plan_tile_rows, plan_capacity, status, s, nullptr, 0, 0, sink, 0);
       if (rc2 != B200_ERR_UNSUPPORTED) return rc2;
       // head_dim 64, four query heads of a KV head per CTA
       const int rc4 = prefill_umma4_launch(q, k, v, out, q_token_stride, k_token_stride, v_token_stride,
@@ -225,8 +262,6 @@ static int prefill_attention(const void* q, const void* k, const void* v, void* 
     if (rc != B200_ERR_UNSUPPORTED) return rc;
   }
 
-  if (head_dim_qk > kMaxPerLane * 32 || head_dim_v > kMaxPerLane * 32) return B200_ERR_UNSUPPORTED;
-  if (num_seqs > 65535 || num_q_heads > 65535) return B200_ERR_UNSUPPORTED;
   PrefillArgs a{};
   a.q = q;
   a.k = k;
@@ -251,12 +286,7 @@ static int prefill_attention(const void* q, const void* k, const void* v, void* 
   a.num_blocks = num_blocks;
   a.sink = sink;
   a.status = status;
-  dim3 grid((max_seqlen_q + kWarps - 1) / kWarps, num_q_heads, num_seqs);
-  if (dtype == B200_DTYPE_F32)
-    prefill_simple_kernel<float><<<grid, kWarps * 32, 0, s>>>(a);
-  else
-    prefill_simple_kernel<__nv_bfloat16><<<grid, kWarps * 32, 0, s>>>(a);
-  return launch_result();
+  return simple_launch(a, max_seqlen_q, dtype, s);
 }
 
 extern "C" int b200_prefill_varlen(const void* q, const void* k, const void* v, void* out,
@@ -319,10 +349,72 @@ extern "C" int b200_prefill_varlen_shared_tail(const void* q, const void* k_head
                                        total_q_tokens, total_k_tokens, cu_seqlens_q, cu_seqlens_k, num_seqs,
                                        max_seqlen_q, num_heads, num_heads, head_dim_qk, head_dim_v, scale, plan,
                                        plan_tile_rows, plan_capacity, status, static_cast<cudaStream_t>(stream),
-                                       k_tail, k_tail_token_stride, tail_dim, nullptr);
+                                       k_tail, k_tail_token_stride, tail_dim, nullptr, 0);
   if (rc2 != B200_ERR_UNSUPPORTED) return rc2;
   return prefill_mma_launch(q, k_head, v, out, q_token_stride, k_head_token_stride, v_token_stride, cu_seqlens_q,
                             cu_seqlens_k, num_seqs, max_seqlen_q, num_heads, num_heads, head_dim_qk, head_dim_v,
                             scale, nullptr, nullptr, nullptr, 0, 0, 0, plan, plan_tile_rows, plan_capacity, status,
                             static_cast<cudaStream_t>(stream), k_tail, k_tail_token_stride, tail_dim, nullptr);
+}
+
+extern "C" int32_t b200_prefill_window_tile_rows(int32_t num_q_heads, int32_t num_kv_heads, int32_t head_dim_qk,
+                                                 int32_t tail_dim, int32_t head_dim_v, int32_t dtype) {
+  if (dtype != B200_DTYPE_BF16 || num_kv_heads <= 0 || num_q_heads % num_kv_heads != 0) return 0;
+  if (tail_dim == 0 || (tail_dim == 64 && head_dim_qk == 192))
+    if (const int r = b200::prefill_umma2_tile_rows(num_q_heads, num_kv_heads, head_dim_qk, head_dim_v)) return r;
+  return b200::prefill_mma_general_shape(head_dim_qk, head_dim_v, tail_dim) ? 64 : 0;
+}
+
+extern "C" int b200_prefill_varlen_window(const void* q, const void* k_head, const void* k_tail, const void* v, void* out,
+                                          int64_t q_token_stride, int64_t k_head_token_stride, int64_t k_tail_token_stride,
+                                          int64_t v_token_stride, int64_t total_q_tokens, int64_t total_k_tokens,
+                                          const int32_t* cu_seqlens_q, const int32_t* cu_seqlens_k, int32_t num_seqs,
+                                          int32_t max_seqlen_q, int32_t num_q_heads, int32_t num_kv_heads,
+                                          int32_t head_dim_qk, int32_t tail_dim, int32_t head_dim_v, float scale,
+                                          int32_t window, const float* sink, const int32_t* plan, int32_t plan_tile_rows,
+                                          int32_t plan_capacity, int32_t dtype, int32_t* status, void* stream) {
+  using namespace b200;
+  if (num_seqs < 0 || max_seqlen_q < 0 || num_q_heads <= 0 || num_kv_heads <= 0 || num_q_heads % num_kv_heads || head_dim_qk <= 0 ||
+      head_dim_v <= 0 || tail_dim < 0 || tail_dim >= head_dim_qk || window < 0)
+    return B200_ERR_ARG;
+  if (dtype != B200_DTYPE_F32 && dtype != B200_DTYPE_BF16) return B200_ERR_UNSUPPORTED;
+  if (num_seqs == 0 || max_seqlen_q == 0) return B200_OK;
+  if (!q || !k_head || (tail_dim > 0 && !k_tail) || !v || !out || !cu_seqlens_q || !cu_seqlens_k) return B200_ERR_ARG;
+  if (total_q_tokens <= 0 || total_k_tokens <= 0) return B200_ERR_ARG;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (dtype == B200_DTYPE_BF16) {
+    const int rc2 = prefill_umma2_launch(q, k_head, v, out, q_token_stride, k_head_token_stride, v_token_stride, total_q_tokens,
+                                         total_k_tokens, cu_seqlens_q, cu_seqlens_k, num_seqs, max_seqlen_q, num_q_heads,
+                                         num_kv_heads, head_dim_qk, head_dim_v, scale, plan, plan_tile_rows, plan_capacity,
+                                         status, s, k_tail, k_tail_token_stride, tail_dim, sink, window);
+    if (rc2 != B200_ERR_UNSUPPORTED) return rc2;
+    const int rc = prefill_mma_general_launch(q, k_head, v, out, q_token_stride, k_head_token_stride, v_token_stride,
+                                              cu_seqlens_q, cu_seqlens_k, num_seqs, max_seqlen_q, num_q_heads, num_kv_heads,
+                                              head_dim_qk, head_dim_v, scale, plan, plan_tile_rows, plan_capacity, status, s,
+                                              k_tail, k_tail_token_stride, tail_dim, sink, window);
+    if (rc != B200_ERR_UNSUPPORTED) return rc;
+  }
+  PrefillArgs a{};
+  a.q = q;
+  a.k = k_head;
+  a.v = v;
+  a.out = out;
+  a.q_stride = q_token_stride;
+  a.k_stride = k_head_token_stride;
+  a.v_stride = v_token_stride;
+  a.cu_q = cu_seqlens_q;
+  a.cu_k = cu_seqlens_k;
+  a.num_seqs = num_seqs;
+  a.Hq = num_q_heads;
+  a.Hkv = num_kv_heads;
+  a.Dqk = head_dim_qk;
+  a.Dv = head_dim_v;
+  a.scale_log2 = scale * 1.4426950408889634f;
+  a.sink = sink;
+  a.k_tail = k_tail;
+  a.k_tail_stride = k_tail_token_stride;
+  a.tail = tail_dim;
+  a.window = window;
+  a.status = status;
+  return simple_launch(a, max_seqlen_q, dtype, s);
 }

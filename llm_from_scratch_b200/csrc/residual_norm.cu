@@ -1,11 +1,11 @@
-// fp32 residual of a decoder whose layers norm the sublayer's OUTPUT, one launch per sublayer boundary:
+// fp32 residual of a decoder, one launch per boundary between sublayers or layers:
 //
-//   x <- x + y / sqrt(mean(y^2) + eps) * w        y: the sublayer's result, activation dtype
-//   h  = x, rounded to the activation dtype       what the next sublayer reads, or with a final norm
-//   h  = x / sqrt(mean(x^2) + eps) * final_w
+//   x <- x + y / sqrt(mean(y^2) + eps) * w        y: the sublayer's result, activation dtype (optional)
+//   x <- x + scale embed[token]                   (optional; or x starts as that)
+//   h  = x, rounded to the activation dtype       what the next sublayer reads, or with a norm
+//   h  = x / sqrt(mean(x^2) + eps) * norm_w       mean over the row, or over each of `groups` equal parts of it
 //
-// The first boundary starts x from the embedding row instead.  One CTA per token row; with the row in registers every
-// load precedes the first reduction.
+// One CTA per token row; with the row in registers every load precedes the first reduction.
 #include "common.cuh"
 
 namespace b200 {
@@ -14,11 +14,14 @@ namespace {
 struct ResArgs {
   float* x;                  // [T, d]
   const int64_t* tokens;     // [T] with embed, else null
-  const void* embed;         // [vocab, d]
+  const void* embed;         // [vocab, d] or null
   int64_t vocab;
-  const void* y;             // [T, d]
+  float scale;               // of the embedding row
+  int start;                 // x is not read: it begins as zero
+  const void* y;             // [T, d] or null
   const float* w;            // [d]
   const float* final_w;      // [d] or null
+  int groups;                // parts of the final norm, a divisor of d
   float eps;
   void* h;                   // [T, d]
   int d;
@@ -60,30 +63,43 @@ __device__ __forceinline__ int64_t embed_row(const ResArgs& a, int64_t row) {
   return 0;
 }
 
-// N groups of four channels per thread, d a multiple of four
-template <typename T, int N>
+constexpr int kMaxParts = 64;      // groups of the final norm in the register kernel
+
+// N groups of four channels per thread, d a multiple of four; GROUPED: the final norm has a.groups parts, each a multiple of
+// four channels wide
+template <typename T, int N, bool GROUPED>
 __global__ void __launch_bounds__(1024) residual_norm_kernel(const ResArgs a) {
   __shared__ float scratch[2][32];
+  __shared__ float part[GROUPED ? 1024 * N : 1], part_inv[GROUPED ? kMaxParts : 1];
   const int d = a.d, step = blockDim.x * 4, first = threadIdx.x * 4;
   const int64_t row = blockIdx.x;
   float* xr = a.x + row * d;
   T* hr = static_cast<T*>(a.h) + row * d;
   float4 x[N], y[N], w[N], fw[N];
   const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
-  const T* src = a.embed ? static_cast<const T*>(a.embed) + embed_row(a, row) * d : static_cast<const T*>(a.y) + row * d;
+  const T* er = a.embed ? static_cast<const T*>(a.embed) + embed_row(a, row) * d : nullptr;
+  const T* yr = static_cast<const T*>(a.y) + row * d;
 #pragma unroll
   for (int i = 0; i < N; ++i) {
     const int c = first + i * step;
     const bool in = c < d;
-    y[i] = in ? load4<T>(src + c) : zero;
-    x[i] = in && a.embed == nullptr ? *reinterpret_cast<const float4*>(xr + c) : zero;
-    w[i] = in && a.embed == nullptr ? *reinterpret_cast<const float4*>(a.w + c) : zero;
+    x[i] = in && !a.start ? *reinterpret_cast<const float4*>(xr + c) : zero;
+    y[i] = in && a.y ? load4<T>(yr + c) : zero;
+    w[i] = in && a.y ? *reinterpret_cast<const float4*>(a.w + c) : zero;
     fw[i] = in && a.final_w ? *reinterpret_cast<const float4*>(a.final_w + c) : zero;
   }
   if (a.embed != nullptr) {
 #pragma unroll
-    for (int i = 0; i < N; ++i) x[i] = y[i];
-  } else {
+    for (int i = 0; i < N; ++i) {
+      const int c = first + i * step;
+      const float4 e = c < d ? load4<T>(er + c) : zero;
+      x[i].x += a.scale * e.x;
+      x[i].y += a.scale * e.y;
+      x[i].z += a.scale * e.z;
+      x[i].w += a.scale * e.w;
+    }
+  }
+  if (a.y != nullptr) {
     float ss = 0.f;
 #pragma unroll
     for (int i = 0; i < N; ++i) ss += sumsq(y[i]);
@@ -102,13 +118,36 @@ __global__ void __launch_bounds__(1024) residual_norm_kernel(const ResArgs a) {
     if (c < d) *reinterpret_cast<float4*>(xr + c) = x[i];
   }
   if (a.final_w != nullptr) {
-    float ss = 0.f;
+    float inv[N];
+    if constexpr (GROUPED) {
+      const int width = d / a.groups, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
 #pragma unroll
-    for (int i = 0; i < N; ++i) ss += sumsq(x[i]);
-    const float inv = rsqrtf(cta_sum(ss, scratch[1]) / static_cast<float>(d) + a.eps);
+      for (int i = 0; i < N; ++i) {
+        const int c = first + i * step;
+        if (c < d) part[c >> 2] = sumsq(x[i]);
+      }
+      __syncthreads();
+      for (int g = warp; g < a.groups; g += blockDim.x >> 5) {
+        float ss = 0.f;
+        for (int k = lane; k < width >> 2; k += 32) ss += part[g * (width >> 2) + k];
+        ss = warp_sum(ss);
+        if (lane == 0) part_inv[g] = rsqrtf(ss / static_cast<float>(width) + a.eps);
+      }
+      __syncthreads();
+#pragma unroll
+      for (int i = 0; i < N; ++i) inv[i] = part_inv[min((first + i * step) / width, a.groups - 1)];
+    } else {
+      float ss = 0.f;
+#pragma unroll
+      for (int i = 0; i < N; ++i) ss += sumsq(x[i]);
+      inv[0] = rsqrtf(cta_sum(ss, scratch[1]) / static_cast<float>(d) + a.eps);
+#pragma unroll
+      for (int i = 1; i < N; ++i) inv[i] = inv[0];
+    }
 #pragma unroll
     for (int i = 0; i < N; ++i)
-      x[i] = make_float4(x[i].x * inv * fw[i].x, x[i].y * inv * fw[i].y, x[i].z * inv * fw[i].z, x[i].w * inv * fw[i].w);
+      x[i] = make_float4(x[i].x * inv[i] * fw[i].x, x[i].y * inv[i] * fw[i].y, x[i].z * inv[i] * fw[i].z,
+                         x[i].w * inv[i] * fw[i].w);
   }
 #pragma unroll
   for (int i = 0; i < N; ++i) {
@@ -120,39 +159,66 @@ __global__ void __launch_bounds__(1024) residual_norm_kernel(const ResArgs a) {
 // any width
 template <typename T>
 __global__ void __launch_bounds__(256) residual_norm_any_kernel(const ResArgs a) {
-  __shared__ float scratch[2][32];
+  __shared__ float scratch[32];
   const int d = a.d;
   const int64_t row = blockIdx.x;
   float* xr = a.x + row * d;
   T* hr = static_cast<T*>(a.h) + row * d;
-  const T* src = a.embed ? static_cast<const T*>(a.embed) + embed_row(a, row) * d : static_cast<const T*>(a.y) + row * d;
-  float inv = 1.f;
-  if (a.embed == nullptr) {
+  const T* er = a.embed ? static_cast<const T*>(a.embed) + embed_row(a, row) * d : nullptr;
+  const T* yr = a.y ? static_cast<const T*>(a.y) + row * d : nullptr;
+  float inv = 0.f;
+  if (yr != nullptr) {
     float ss = 0.f;
-    for (int c = threadIdx.x; c < d; c += blockDim.x) ss += to_float<T>(src[c]) * to_float<T>(src[c]);
-    inv = rsqrtf(cta_sum(ss, scratch[0]) / static_cast<float>(d) + a.eps);
+    for (int c = threadIdx.x; c < d; c += blockDim.x) ss += to_float<T>(yr[c]) * to_float<T>(yr[c]);
+    inv = rsqrtf(cta_sum(ss, scratch) / static_cast<float>(d) + a.eps);
   }
-  float ss = 0.f;
   for (int c = threadIdx.x; c < d; c += blockDim.x) {
-    const float v = to_float<T>(src[c]);
-    const float x = a.embed ? v : xr[c] + v * inv * a.w[c];
+    float x = a.start ? 0.f : xr[c];
+    if (er != nullptr) x += a.scale * to_float<T>(er[c]);
+    if (yr != nullptr) x += to_float<T>(yr[c]) * inv * a.w[c];
     xr[c] = x;
-    ss += x * x;
     if (a.final_w == nullptr) hr[c] = from_float<T>(x);
   }
-  if (a.final_w != nullptr) {
-    inv = rsqrtf(cta_sum(ss, scratch[1]) / static_cast<float>(d) + a.eps);
-    for (int c = threadIdx.x; c < d; c += blockDim.x) hr[c] = from_float<T>(xr[c] * inv * a.final_w[c]);
+  if (a.final_w == nullptr) return;
+  __syncthreads();
+  const int width = d / a.groups, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  for (int g = warp; g < a.groups; g += blockDim.x >> 5) {     // a warp per part
+    float ss = 0.f;
+    for (int c = g * width + lane; c < (g + 1) * width; c += 32) ss += xr[c] * xr[c];
+    const float r = rsqrtf(warp_sum(ss) / static_cast<float>(width) + a.eps);
+    for (int c = g * width + lane; c < (g + 1) * width; c += 32) hr[c] = from_float<T>(xr[c] * r * a.final_w[c]);
   }
+}
+
+template <typename T, bool GROUPED>
+void launch_vec(const ResArgs& a, unsigned grid, cudaStream_t s) {
+  const int groups = a.d / 4;
+  if (groups <= 1024) residual_norm_kernel<T, 1, GROUPED><<<grid, (groups + 31) / 32 * 32, 0, s>>>(a);
+  else residual_norm_kernel<T, 2, GROUPED><<<grid, (groups + 63) / 64 * 32, 0, s>>>(a);
 }
 
 template <typename T>
 void launch(const ResArgs& a, int64_t rows, bool vec, cudaStream_t s) {
   const unsigned grid = static_cast<unsigned>(rows);
-  const int groups = a.d / 4;
-  if (vec && groups <= 1024) residual_norm_kernel<T, 1><<<grid, (groups + 31) / 32 * 32, 0, s>>>(a);
-  else if (vec && groups <= 2048) residual_norm_kernel<T, 2><<<grid, (groups + 63) / 64 * 32, 0, s>>>(a);
-  else residual_norm_any_kernel<T><<<grid, 256, 0, s>>>(a);
+  const bool grouped = a.final_w && a.groups > 1;
+  if (!vec || a.d / 4 > 2048 || (grouped && (a.d / a.groups % 4 != 0 || a.groups > kMaxParts)))
+    residual_norm_any_kernel<T><<<grid, 256, 0, s>>>(a);
+  else if (grouped) launch_vec<T, true>(a, grid, s);
+  else launch_vec<T, false>(a, grid, s);
+}
+
+int residual_norm(const ResArgs& a, int64_t rows, int32_t dtype, void* stream) {
+  if (rows < 0 || a.d <= 0 || a.groups <= 0 || a.d % a.groups) return B200_ERR_ARG;
+  if (dtype != B200_DTYPE_F32 && dtype != B200_DTYPE_BF16) return B200_ERR_UNSUPPORTED;
+  if (rows == 0) return B200_OK;
+  if (!a.x || !a.h || (a.embed && !a.tokens) || (a.y && !a.w) || (a.start && !a.embed)) return B200_ERR_ARG;
+  if (rows > 2147483647) return B200_ERR_TOO_LARGE;
+  const bool vec = a.d % 4 == 0 && aligned16(a.x) && aligned16(a.h) && (!a.embed || aligned16(a.embed)) &&
+                   (!a.y || (aligned16(a.y) && aligned16(a.w))) && (!a.final_w || aligned16(a.final_w));
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (dtype == B200_DTYPE_F32) launch<float>(a, rows, vec, s);
+  else launch<__nv_bfloat16>(a, rows, vec, s);
+  return launch_result();
 }
 
 }  // namespace
@@ -162,16 +228,16 @@ extern "C" int b200_residual_norm(float* x, const int64_t* tokens, const void* e
                                   const float* norm_w, const float* final_w, float eps, void* h, int64_t rows, int32_t d,
                                   int32_t dtype, int32_t* status, void* stream) {
   using namespace b200;
-  if (rows < 0 || d <= 0) return B200_ERR_ARG;
-  if (dtype != B200_DTYPE_F32 && dtype != B200_DTYPE_BF16) return B200_ERR_UNSUPPORTED;
-  if (rows == 0) return B200_OK;
-  if (!x || !h || (embed ? !tokens : (!y || !norm_w))) return B200_ERR_ARG;
-  if (rows > 2147483647) return B200_ERR_TOO_LARGE;
-  ResArgs a{x, tokens, embed, vocab, y, norm_w, final_w, eps, h, d, status};
-  const bool vec = d % 4 == 0 && aligned16(x) && aligned16(h) && aligned16(embed ? embed : y) &&
-                   (embed || aligned16(norm_w)) && (!final_w || aligned16(final_w));
-  cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (dtype == B200_DTYPE_F32) launch<float>(a, rows, vec, s);
-  else launch<__nv_bfloat16>(a, rows, vec, s);
-  return launch_result();
+  if (rows > 0 && !embed && !y) return B200_ERR_ARG;
+  return residual_norm({x, tokens, embed, vocab, 1.f, embed != nullptr, embed ? nullptr : y, norm_w, final_w, 1, eps, h, d, status},
+                       rows, dtype, stream);
+}
+
+extern "C" int b200_residual_group_norm(float* x, const void* y, const float* y_norm_w, const int64_t* tokens, const void* embed,
+                                        int64_t vocab, float embed_scale, int32_t start, const float* norm_w, int32_t groups,
+                                        float eps, void* h, int64_t rows, int32_t d, int32_t dtype, int32_t* status,
+                                        void* stream) {
+  using namespace b200;
+  return residual_norm({x, tokens, embed, vocab, embed_scale, start != 0, y, y_norm_w, norm_w, groups, eps, h, d, status}, rows,
+                       dtype, stream);
 }

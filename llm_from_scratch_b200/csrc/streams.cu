@@ -326,13 +326,6 @@ int launch_streams(const StreamArgs& a, int64_t rows, cudaStream_t s) {
 // ---------------------------------------------------------------------------------------------
 // Clamped gated linear unit: act = g sigmoid(slope g) (u + 1), g = min(gate, limit), u = clamp(up, +-limit).
 // ---------------------------------------------------------------------------------------------
-template <typename T>
-__device__ __forceinline__ float clamped_glu_one(float g, float u, float limit, float slope) {
-  g = fminf(g, limit);
-  u = fminf(fmaxf(u, -limit), limit);
-  return g * (u + 1.f) / (1.f + expf(-slope * g));
-}
-
 template <typename T, int V>
 __global__ void __launch_bounds__(256) clamped_glu_kernel(const T* __restrict__ h, T* __restrict__ act, int64_t total,
                                                           int F, float limit, float slope) {
@@ -352,11 +345,11 @@ __global__ void __launch_bounds__(256) clamped_glu_kernel(const T* __restrict__ 
       for (int k = 0; k < 4; ++k) {
         const float2 gf = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gw[k]));
         const float2 uf = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&uw[k]));
-        r[k] = pack_bf16x2(clamped_glu_one<T>(gf.x, uf.x, limit, slope), clamped_glu_one<T>(gf.y, uf.y, limit, slope));
+        r[k] = pack_bf16x2(clamped_glu_f(gf.x, uf.x, limit, slope), clamped_glu_f(gf.y, uf.y, limit, slope));
       }
       *reinterpret_cast<uint4*>(o) = make_uint4(r[0], r[1], r[2], r[3]);
     } else {
-      *o = from_float<T>(clamped_glu_one<T>(to_float<T>(g[0]), to_float<T>(g[F]), limit, slope));
+      *o = from_float<T>(clamped_glu_f(to_float<T>(g[0]), to_float<T>(g[F]), limit, slope));
     }
   }
 }

@@ -6,8 +6,10 @@ from . import registry
 from .registry import ModelFamily, build_model, family_of, init_weights, resolve_config
 from .nabalix import NabalixConfig, NabalixLM
 from .taminex import TaminexConfig, TaminexLM
+from .meresun import MeresunConfig, MeresunLM
 
 registry.register(ModelFamily(registry.DEFAULT_FAMILY, ModelConfig, EngineTransformerLM, init_reference_order))
 
 __all__ = ["ModelConfig", "init_reference_order", "EngineTransformerLM", "ModelFamily", "build_model", "family_of",
-           "init_weights", "resolve_config", "NabalixConfig", "NabalixLM", "TaminexConfig", "TaminexLM"]
+           "init_weights", "resolve_config", "NabalixConfig", "NabalixLM", "TaminexConfig", "TaminexLM",
+           "MeresunConfig", "MeresunLM"]

@@ -132,13 +132,31 @@ class GatedRecurrence(nn.Module):
         return F.linear(o, self.w_o)
 
 
+_second_stream: dict = {}       # per device
+
+
+def side_by_side(first, second, ctx, device):
+    """Results of two functions that do not need each other.  A decode step runs the second one on a second CUDA stream: at
+    decode sizes neither of the two fills the GPU.  ``second`` returns a tuple of tensors."""
+    if ctx.is_prefill:
+        return first(), second()
+    main = torch.cuda.current_stream()
+    side = _second_stream.get(device)
+    if side is None:
+        side = _second_stream[device] = torch.cuda.Stream(device)
+    side.wait_stream(main)
+    with torch.cuda.stream(side):
+        y1 = second()
+    y = first()
+    main.wait_stream(side)
+    for t in y1:
+        t.record_stream(main)      # allocated on the side stream, read on this one
+    return y, y1
+
+
 class ParallelMixer(nn.Module):
     """Two mixers side by side over one input.  Returns both results; their norms and the mean of the two belong
-    to the residual update (``join`` holds the norm weights), which the stream kernel does in one pass.
-
-    A decode step runs the right mixer on a second CUDA stream: at decode sizes neither of the two fills the GPU."""
-
-    _side: dict = {}       # second stream per device
+    to the residual update (``join`` holds the norm weights), which the stream kernel does in one pass."""
 
     def __init__(self, p: Params, d_model: int, left: nn.Module, right: nn.Module):
         super().__init__()
@@ -151,17 +169,7 @@ class ParallelMixer(nn.Module):
     def forward(self, h, ctx):
         parts = self.project(h)
         left, right = parts[:self.num_left], parts[self.num_left:]
-        if ctx.is_prefill:
-            return self.left(*left, ctx), self.right(*right, ctx)
-        main = torch.cuda.current_stream()
-        side = self._side.setdefault(h.device, None) or torch.cuda.Stream(h.device)
-        self._side[h.device] = side
-        side.wait_stream(main)
-        with torch.cuda.stream(side):
-            y1 = self.right(*right, ctx)
-        y = self.left(*left, ctx)
-        main.wait_stream(side)
-        y1.record_stream(main)      # allocated on the side stream, read on this one
+        y, (y1,) = side_by_side(lambda: self.left(*left, ctx), lambda: (self.right(*right, ctx),), ctx, h.device)
         return y, y1
 
 
@@ -371,3 +379,159 @@ class SquaredReLU(nn.Module):
 
     def forward(self, h, ctx, positions):
         return F.linear(ops.squared_relu(F.linear(h, self.w_up)), self.w_down)
+
+
+# ------------------------------------------------------------------------------------------------
+# sublayers that run side by side on one normed input, with gates on the way into the residual
+# ------------------------------------------------------------------------------------------------
+class RunCache:
+    """The cache of one run of a mixer whose layer may run several times: what the mixer's ``cache_needs`` lists, as
+    attributes that the runner fills."""
+
+    def __init__(self, mixer: nn.Module):
+        self.mixer = mixer
+
+    def cache_needs(self):
+        return self.mixer.cache_needs()
+
+
+class RotaryLatentAttention(nn.Module):
+    """Latent attention with query latents, a rotary key part shared by the heads, a sliding window (0: none) and a sink.
+    Single tokens attend in the absorbed form over the cached rows [latent | rotated part]; portions expand the rows that
+    their windows reach.  The caller projects (``projections``: query and key / value down-projection)."""
+
+    def __init__(self, p: Params, d_model: int, heads: int, dim: int, rot_dim: int, vdim: int, q_rank: int, kv_rank: int,
+                 scale: float, rotation: ops.Rotation, window: int, eps: float):
+        super().__init__()
+        self.heads, self.dim, self.rot_dim, self.vdim, self.rank = heads, dim, rot_dim, vdim, kv_rank
+        self.scale, self.rotation, self.window, self.eps = scale, rotation, window, eps
+        self.projections = [p.lin("dq", (q_rank, d_model)), p.lin("dkv", (kv_rank + rot_dim, d_model))]
+        self.q_norm, self.kv_norm = p.f32("dq.norm", (q_rank,)), p.f32("dkv.norm", (kv_rank,))
+        self.w_uq = p.lin("uq", (heads * (dim + rot_dim), q_rank))
+        uk, uv = p.lin("uk", (heads * dim, kv_rank)), p.lin("uv", (heads * vdim, kv_rank))
+        self.expand = FusedProjection([uk, uv])
+        self.w_uk = uk.view(heads, dim, kv_rank)
+        self.w_uv_t = uv.view(heads, vdim, kv_rank).transpose(1, 2)
+        self.sink = p.f32("sink", (heads,))
+        self.w_o = p.lin("o", (d_model, heads * vdim))
+
+    def cache_needs(self):
+        return [("paged", "latent_cache", (self.rank + self.rot_dim,))]
+
+    def _absorbed(self, q, q_rot, cache, s, o):
+        n, H = s.rows, self.heads
+        q_abs = torch.empty(n, H, self.rank, dtype=q.dtype, device=q.device)
+        torch.bmm(q[:n, :, :self.dim].transpose(0, 1), self.w_uk, out=q_abs.transpose(0, 1))
+        lat = ops.mla_decode(q_abs, q_rot, cache, s.block_tables, s.context_lens, self.scale, window=self.window, sink=self.sink)
+        torch.bmm(lat.transpose(0, 1), self.w_uv_t, out=o[:n].view(n, H, self.vdim).transpose(0, 1))
+
+    def _expanded(self, q, rows, cache, s, o):
+        H, keys = self.heads, s.keys(self.window)
+        cu_k = s.cu_seqlens_q
+        if keys.has_prefix:
+            cu_k = keys.cu_seqlens_k
+            rows = ops.gather_rows(cache, s.block_tables, cu_k, keys.max_seqlen_k, keys.total_k, s.cu_seqlens_k)
+        k, v = self.expand(rows[:, :self.rank])
+        k_tail = rows[:, self.rank:] if self.rot_dim else None
+        plan = s.plan(ops.prefill_window_tile_rows(H, H, self.dim + self.rot_dim, self.rot_dim, self.vdim, q.dtype))
+        ops.prefill_varlen_window(q, _heads(k, H, self.dim), k_tail, _heads(v, H, self.vdim), s.cu_seqlens_q, cu_k, s.max_seqlen_q,
+                                  self.scale, self.window, self.sink, out=o.view(-1, H, self.vdim), plan=plan)
+
+    def forward(self, dq, dkv, ctx, positions, pools):
+        c_q, rows = ops.latent_prologue(dq, self.q_norm, dkv, self.kv_norm, self.eps, self.rotation, positions,
+                                        pools.latent_cache, ctx.slot_mapping)
+        q = _heads(F.linear(c_q, self.w_uq), self.heads, self.dim + self.rot_dim)
+        singles = ctx.singles.rows if ctx.singles is not None else 0
+        q_rot = ops.rotate_heads(q, self.rot_dim, self.rotation, positions, singles) if self.rot_dim else None
+        o = _step_output(rows, self.heads * self.vdim, ctx)
+        if ctx.singles is not None:
+            self._absorbed(q, q_rot, pools.latent_cache, ctx.singles, o)
+        if ctx.portions is not None:
+            self._expanded(q, rows, pools.latent_cache, ctx.portions, o)
+        return F.linear(o, self.w_o)
+
+
+class PolyNormMLP(nn.Module):
+    """W_down (c0 N(z) + c1 N(z^2) + c2 N(z^3) + c3) with z = W_up h.  The caller projects up (``projections``)."""
+
+    def __init__(self, p: Params, d_model: int, d_ff: int, eps: float):
+        super().__init__()
+        self.eps = eps
+        self.projections = [p.lin("up", (d_ff, d_model))]
+        self.coef = p.f32("act", (4,))
+        self.w_down = p.lin("down", (d_model, d_ff))
+
+    def forward(self, h, up):
+        return (F.linear(ops.poly_norm(up, self.coef, self.eps), self.w_down),)
+
+
+class GroupedMoE(nn.Module):
+    """Clamped GLU experts behind a sigmoid router with a choice correction and groups of experts.  Returns the chosen
+    experts' output rows, their weights and where a token's rows are; the weighted sum belongs to the residual update."""
+
+    # average rows per expert above which bf16 goes to the library's grouped GEMM (see transformer.MoE)
+    own_gemm_max_rows_per_expert = 256
+
+    def __init__(self, p: Params, d_model: int, d_ff: int, experts: int, top: int, groups: int, keep: int, limit: float,
+                 slope: float = 1.702):
+        super().__init__()
+        self.top, self.groups, self.keep, self.limit, self.slope = top, groups, keep, limit, slope
+        self.projections = []
+        self.router = p.lin("router", (experts, d_model))
+        self.correction = p.f32("correction", (experts,))
+        self.w_in = torch.stack([torch.cat([p.lin(f"e{e}.gate", (d_ff, d_model)), p.lin(f"e{e}.up", (d_ff, d_model))])
+                                 for e in range(experts)])
+        self.w_down = torch.stack([p.lin(f"e{e}.down", (d_model, d_ff)) for e in range(experts)])
+        self.library = p.dtype == torch.bfloat16 and d_model % 8 == 0 and d_ff % 8 == 0
+
+    def forward(self, h):
+        z = F.linear(h, self.router) if h.dtype == torch.float32 else torch.mm(h, self.router.t(), out_dtype=torch.float32)
+        tok, weight, offs, slot = ops.moe_group_route(z, self.correction, self.top, self.groups, self.keep)
+        xs = h.index_select(0, tok)
+        if self.library and tok.numel() > self.own_gemm_max_rows_per_expert * self.router.shape[0]:
+            act = ops.clamped_glu(torch._grouped_mm(xs, self.w_in.transpose(1, 2), offs=offs), self.limit, self.slope)
+            return torch._grouped_mm(act, self.w_down.transpose(1, 2), offs=offs), weight, slot
+        act = ops.moe_grouped_linear(xs, self.w_in, offs, glu=(self.limit, self.slope), early_launch=True)
+        return ops.moe_grouped_linear(act, self.w_down, offs, early_launch=True), weight, slot
+
+
+class TokenInput(nn.Module):
+    """proj (gelu(gate x) * e) with e a part of the token's row in a table that all layers share; the norm of the result
+    (``norm``) belongs to the residual update."""
+
+    def __init__(self, p: Params, d_model: int, table: torch.Tensor, first: int, dim: int):
+        super().__init__()
+        self.table, self.first = table, first
+        self.gate, self.proj = p.lin("gate", (dim, d_model)), p.lin("proj", (d_model, dim))
+        self.norm = p.f32("norm", (d_model,))
+
+    def forward(self, x, tokens):
+        return F.linear(ops.gelu_table(F.linear(x, self.gate), self.table, self.first, tokens), self.proj)
+
+
+class GatedSublayers(nn.Module):
+    """A mixer and (optionally) a feed-forward side by side on the same normed input; every result passes a gate
+    sigmoid(W h + b) on its way into the residual.  All linear maps of that input are one GEMM."""
+
+    def __init__(self, p: Params, d_model: int, mixer: nn.Module, mlp: nn.Module | None):
+        super().__init__()
+        self.mixer, self.mlp = mixer, mlp
+        gates = ["rg1"] + (["rg2"] if mlp is not None else [])
+        inner = mixer.projections + (mlp.projections if mlp is not None else [])
+        self.num_mixer, self.num_inner = len(mixer.projections), len(inner)
+        zeros = [torch.zeros(w.shape[0], dtype=w.dtype, device=w.device) for w in inner]
+        self.project = FusedProjection(inner + [p.lin(g, (d_model, d_model)) for g in gates],
+                                       zeros + [p.lin(g + ".b", (d_model,)) for g in gates])
+        mixer.projections = None                       # the fused copy is the one that is kept
+        if mlp is not None:
+            mlp.projections = None
+
+    def forward(self, h, x, ctx, positions, pools):
+        """Adds both sublayers' results to the residual x; returns x in the dtype of h."""
+        parts = self.project(h)
+        into_mixer, into_mlp, gates = parts[:self.num_mixer], parts[self.num_mixer:self.num_inner], parts[self.num_inner:]
+        mix = lambda: self.mixer(*into_mixer, ctx, positions, pools)
+        if self.mlp is None:
+            return ops.gated_residual(x, mix(), gates[0])
+        y, (f, *choice) = side_by_side(mix, lambda: self.mlp(h, *into_mlp), ctx, h.device)
+        return ops.gated_residual(x, y, gates[0], f, gates[1], *choice)

@@ -13,7 +13,6 @@ from dataclasses import dataclass, field
 from typing import Optional
 
 import torch
-import torch.nn.functional as F
 from torch import nn
 
 from .. import ops
@@ -168,10 +167,7 @@ class TaminexLM(TokenHead, nn.Module):
 
     # ------------------------------------------------------------------ head
     def compute_logits(self, hidden: torch.Tensor) -> torch.Tensor:
-        rows = self.logit_rows(hidden).to(self.dtype)
-        z = F.linear(rows, self.w_head) if self.dtype == torch.float32 else \
-            torch.mm(rows, self.w_head.t(), out_dtype=torch.float32)
-        return ops.softcap_logits(z, self.cfg.logit_scale, self.cfg.logit_softcap)
+        return ops.softcap_logits(self.logits_f32(hidden), self.cfg.logit_scale, self.cfg.logit_softcap)
 
     def greedy_tokens(self, hidden: torch.Tensor, out: torch.Tensor | None = None) -> torch.Tensor:
         if self.cfg.logit_scale > 0:        # scale and cap are increasing: the largest logit stays the largest

@@ -449,6 +449,11 @@ class TokenHead:
     def compute_logits(self, hidden: torch.Tensor) -> torch.Tensor:
         return F.linear(self.logit_rows(hidden).to(self.dtype), self.w_head, self.b_head)
 
+    def logits_f32(self, hidden: torch.Tensor) -> torch.Tensor:
+        """Logits of a head without bias in fp32, also in bf16 (fp32 accumulators written as they are)."""
+        rows = self.logit_rows(hidden).to(self.dtype)
+        return F.linear(rows, self.w_head) if self.dtype == torch.float32 else torch.mm(rows, self.w_head.t(), out_dtype=torch.float32)
+
     fused_head_max_rows = 64     # rows up to which the fused head (weights as the MMA M side) beats GEMM + argmax
 
     def greedy_tokens(self, hidden: torch.Tensor, out: torch.Tensor | None = None) -> torch.Tensor:

@@ -6,6 +6,8 @@ the current CUDA stream.  Nothing here computes on the CPU; a CPU tensor is an e
 from __future__ import annotations
 
 import array
+import math
+from dataclasses import dataclass
 
 import torch
 
@@ -359,14 +361,16 @@ def prefill_plan(cu_seqlens_q: torch.Tensor, total_q_tokens: int, max_seqlen_q: 
 
 def mla_decode(q_abs: torch.Tensor, q_rope: torch.Tensor | None, latent_cache: torch.Tensor,
                block_tables: torch.Tensor, context_lens: torch.Tensor, scale: float,
-               out: torch.Tensor | None = None) -> torch.Tensor:
+               out: torch.Tensor | None = None, window: int = 0, sink: torch.Tensor | None = None) -> torch.Tensor:
     """Absorbed MLA decode over a paged latent pool.
 
     q_abs: [B, H, r]; q_rope: [B, H, dr] or None (dr = 0); latent_cache: [num_blocks, block_size, r + dr];
-    returns the attention-weighted latent [B, H, r].
+    returns the attention-weighted latent [B, H, r].  ``window`` > 0: over the last ``window`` tokens only; ``sink``
+    fp32 [H]: exp(sink) joins the softmax denominator.
     """
-    dev = _cuda(q_abs, q_rope, latent_cache, block_tables, context_lens, out)
+    dev = _cuda(q_abs, q_rope, latent_cache, block_tables, context_lens, out, sink)
     B, H, r = q_abs.shape
+    _f32vec("sink", sink, H)
     dr = q_rope.shape[2] if q_rope is not None else 0
     nb, bs, row = latent_cache.shape
     if row != r + dr or (q_rope is not None and q_rope.shape[:2] != (B, H)):
@@ -383,11 +387,13 @@ def mla_decode(q_abs: torch.Tensor, q_rope: torch.Tensor | None, latent_cache: t
         out = torch.empty_like(q_abs)
     need = lib.b200_mla_decode_workspace_bytes(B, H, r, dr, _dt(q_abs))
     ws = workspace(dev, need, "mla")
-    check(lib.b200_mla_decode(q_abs.data_ptr(), _ptr(q_rope), latent_cache.data_ptr(),
-                              out.data_ptr(), block_tables.data_ptr(), block_tables.stride(0),
-                              context_lens.data_ptr(), B, H, r, dr, bs, nb, float(scale),
-                              ws.data_ptr(), ws.numel(), _dt(q_abs), status_word(dev).data_ptr(),
-                              _stream()), "mla_decode")
+    args = (q_abs.data_ptr(), _ptr(q_rope), latent_cache.data_ptr(), out.data_ptr(), block_tables.data_ptr(),
+            block_tables.stride(0), context_lens.data_ptr(), B, H, r, dr, bs, nb, float(scale))
+    tail = (ws.data_ptr(), ws.numel(), _dt(q_abs), status_word(dev).data_ptr(), _stream())
+    if window or sink is not None:
+        check(lib.b200_mla_decode_window(*args, int(window), _ptr(sink), *tail), "mla_decode_window")
+    else:
+        check(lib.b200_mla_decode(*args, *tail), "mla_decode")
     return out
 
 
@@ -947,10 +953,40 @@ def residual_norm(x: torch.Tensor, eps: float, dtype: torch.dtype, *, tokens: to
     return h
 
 
-def rotary_frequencies(base: float, dims: int, device) -> torch.Tensor:
-    """base^(-2i / dims), i < dims / 2, in fp64."""
+@dataclass(frozen=True)
+class YarnScaling:
+    """YaRN stretching of rotary frequencies: pairs that turn fewer than ``slow`` times within ``original`` positions turn
+    ``factor`` times slower, those that turn more than ``fast`` times as they are, those between on a linear ramp."""
+    factor: float
+    original: float
+    fast: float
+    slow: float
+
+    @property
+    def magnitude(self) -> float:
+        """What cos and sin are multiplied by."""
+        return 0.1 * math.log(self.factor) + 1.0
+
+    def pair(self, turns: float, base: float, dims: int) -> float:
+        """Index (real) of the pair that turns ``turns`` times within ``original`` positions."""
+        return dims * math.log(self.original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
+
+    def ramp(self, base: float, dims: int) -> torch.Tensor:
+        """How far every pair is stretched, 0 to 1."""
+        first = max(math.floor(self.pair(self.fast, base, dims)), 0)
+        last = min(math.ceil(self.pair(self.slow, base, dims)), dims - 1)
+        i = torch.arange(dims // 2, dtype=torch.float64)
+        return ((i - first) / max(last - first, 0.001)).clamp(0.0, 1.0)
+
+
+def rotary_frequencies(base: float, dims: int, device, scaling: YarnScaling | None = None) -> torch.Tensor:
+    """base^(-2i / dims), i < dims / 2, in fp64, stretched by ``scaling``."""
     i = torch.arange(dims // 2, dtype=torch.float64)
-    return (float(base) ** (-2.0 * i / max(dims, 1))).to(device)
+    freq = float(base) ** (-2.0 * i / max(dims, 1))
+    if scaling is not None and dims:
+        ramp = scaling.ramp(float(base), dims)
+        freq = freq / scaling.factor * ramp + freq * (1.0 - ramp)
+    return freq.to(device)
 
 
 def head_norm_rope_store(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, q_norm_w: torch.Tensor, k_norm_w: torch.Tensor,
@@ -1004,18 +1040,22 @@ def latent_norm_store(rows: torch.Tensor, norm_w: torch.Tensor, eps: float, cach
 
 
 def gather_rows(cache: torch.Tensor, block_tables: torch.Tensor, cu_seqlens_k: torch.Tensor, max_seqlen_k: int,
-                total: int) -> torch.Tensor:
-    """Rows of whole contexts, packed [total, W], from a pool [num_blocks, block_size, W] through the block tables."""
-    dev = _cuda(cache, block_tables, cu_seqlens_k)
+                total: int, cu_seqlens_full: torch.Tensor | None = None) -> torch.Tensor:
+    """Rows of whole contexts, packed [total, W], from a pool [num_blocks, block_size, W] through the block tables.  With
+    ``cu_seqlens_full`` (the contexts' own offsets) ``cu_seqlens_k`` counts the last rows of every context."""
+    dev = _cuda(cache, block_tables, cu_seqlens_k, cu_seqlens_full)
     nb, bs, W = cache.shape
     n = cu_seqlens_k.numel() - 1
     if not cache.is_contiguous() or block_tables.dtype != torch.int32 or block_tables.shape[0] < n \
             or block_tables.stride(1) != 1 or cu_seqlens_k.dtype != torch.int32:
         raise ValueError("cache must be contiguous, block_tables int32 [n, max_blocks], cu_seqlens_k int32 [n + 1]")
     out = torch.empty(total, W, dtype=cache.dtype, device=cache.device)
-    check(lib.b200_gather_rows(cache.data_ptr(), bs, nb, W * cache.element_size(), block_tables.data_ptr(),
-                               block_tables.stride(0), cu_seqlens_k.data_ptr(), n, int(max_seqlen_k), out.data_ptr(), total,
-                               status_word(dev).data_ptr(), _stream()), "gather_rows")
+    if cu_seqlens_full is not None and (cu_seqlens_full.dtype != torch.int32 or cu_seqlens_full.numel() != n + 1):
+        raise ValueError("cu_seqlens_full must be int32 [n + 1]")
+    check(lib.b200_gather_last_rows(cache.data_ptr(), bs, nb, W * cache.element_size(), block_tables.data_ptr(),
+                                    block_tables.stride(0), cu_seqlens_k.data_ptr(), _ptr(cu_seqlens_full), n,
+                                    int(max_seqlen_k), out.data_ptr(), total, status_word(dev).data_ptr(), _stream()),
+          "gather_rows")
     return out
 
 
@@ -1130,4 +1170,219 @@ def _delta_out(c: DeltaRule, proj: torch.Tensor, out: torch.Tensor | None) -> to
         return torch.empty(shape, dtype=proj.dtype, device=proj.device)
     if out.shape != shape or out.dtype != proj.dtype or not out.is_contiguous():
         raise ValueError("out must be contiguous [T, heads * vdim] of proj's dtype")
+    return out
+
+
+# ------------------------------------------------------------------------------------------------
+# parallel gated sublayers, windowed latent attention, grouped expert routing, token inputs
+# ------------------------------------------------------------------------------------------------
+def _tokens(name: str, t: torch.Tensor, n: int) -> None:
+    if t.dtype != torch.int64 or t.numel() != n or not t.is_contiguous():
+        raise ValueError(f"{name} must be contiguous int64 with one entry per token")
+
+
+def residual_group_norm(x: torch.Tensor, norm_w: torch.Tensor, groups: int, eps: float, dtype: torch.dtype, *,
+                        y: torch.Tensor | None = None, y_norm_w: torch.Tensor | None = None,
+                        tokens: torch.Tensor | None = None, embed: torch.Tensor | None = None, embed_scale: float = 1.0,
+                        start: bool = False) -> torch.Tensor:
+    """One layer boundary (``b200_residual_group_norm``): x [T, d] fp32 takes the normed ``y`` and the scaled embedding rows
+    (either may be absent; ``start``: x begins as zero) in place; returns its norm in ``groups`` parts, in ``dtype``."""
+    dev = _cuda(x, norm_w, y, y_norm_w, tokens, embed)
+    T, d = x.shape
+    if x.dtype != torch.float32 or not x.is_contiguous():
+        raise ValueError("x must be a contiguous fp32 [T, d] tensor")
+    _f32vec("norm_w", norm_w, d)
+    _f32vec("y_norm_w", y_norm_w, d)
+    if y is not None and (y_norm_w is None or y.shape != (T, d) or y.dtype != dtype or not y.is_contiguous()):
+        raise ValueError("y must be contiguous [T, d] in the activation dtype, with its norm weight")
+    if embed is not None:
+        if embed.shape[1] != d or embed.dtype != dtype or not embed.is_contiguous() or tokens is None:
+            raise ValueError("embed must be contiguous [vocab, d] in the activation dtype, with tokens")
+        _tokens("tokens", tokens, T)
+    h = torch.empty(T, d, dtype=dtype, device=x.device)
+    check(lib.b200_residual_group_norm(
+        x.data_ptr(), _ptr(y), _ptr(y_norm_w), _ptr(tokens) if embed is not None else None, _ptr(embed),
+        embed.shape[0] if embed is not None else 0, float(embed_scale), 1 if start else 0, norm_w.data_ptr(), int(groups),
+        float(eps), h.data_ptr(), T, d, _dt(h), status_word(dev).data_ptr(), _stream()), "residual_group_norm")
+    return h
+
+
+def gated_residual(x: torch.Tensor, y1: torch.Tensor, gate1: torch.Tensor, y2: torch.Tensor | None = None,
+                   gate2: torch.Tensor | None = None, row_weight: torch.Tensor | None = None,
+                   slot_to_row: torch.Tensor | None = None) -> torch.Tensor:
+    """x [T, d] fp32 <- x + y1 sigmoid(gate1) + y2 sigmoid(gate2) in place; gates [T, d] are views of one projection.  With
+    ``row_weight`` / ``slot_to_row`` [T, top] y2 holds expert rows [T * top, d].  Returns x in the dtype of y1."""
+    dev = _cuda(x, y1, gate1, y2, gate2, row_weight, slot_to_row)
+    T, d = x.shape
+    top = slot_to_row.shape[1] if slot_to_row is not None else 0
+    if x.dtype != torch.float32 or not x.is_contiguous() or y1.shape != (T, d) or not y1.is_contiguous():
+        raise ValueError("x must be contiguous fp32 [T, d], y1 contiguous [T, d]")
+    for g in (gate1, gate2):
+        if g is not None and (g.shape != (T, d) or g.dtype != y1.dtype or g.stride(1) != 1 or g.stride(0) != gate1.stride(0)):
+            raise ValueError("gates must be [T, d] in the dtype of y1 with one row stride")
+    if y2 is not None and (gate2 is None or y2.shape != ((T * top) if top else T, d) or y2.dtype != y1.dtype
+                           or not y2.is_contiguous()):
+        raise ValueError("y2 must be contiguous [T, d] (or [T * top, d]) in the dtype of y1, with its gate")
+    if top and (row_weight is None or row_weight.dtype != torch.float32 or row_weight.shape != (T, top)
+                or slot_to_row.dtype != torch.int32 or not row_weight.is_contiguous() or not slot_to_row.is_contiguous()):
+        raise ValueError("row_weight must be fp32 and slot_to_row int32, both contiguous [T, top]")
+    h = torch.empty(T, d, dtype=y1.dtype, device=x.device)
+    check(lib.b200_gated_residual(x.data_ptr(), y1.data_ptr(), gate1.data_ptr(), _ptr(y2), _ptr(gate2), gate1.stride(0),
+                                  _ptr(row_weight), _ptr(slot_to_row), top, h.data_ptr(), T, d, _dt(h),
+                                  status_word(dev).data_ptr(), _stream()), "gated_residual")
+    return h
+
+
+def poly_norm(z: torch.Tensor, coef: torch.Tensor, eps: float) -> torch.Tensor:
+    """c0 N(z) + c1 N(z^2) + c2 N(z^3) + c3 per row of z [T, W] (row stride free), N a division by the root mean square."""
+    _cuda(z, coef)
+    _f32vec("coef", coef, 4)
+    if z.stride(1) != 1:
+        raise ValueError("rows must be contiguous")
+    out = torch.empty(z.shape, dtype=z.dtype, device=z.device)
+    check(lib.b200_poly_norm(z.data_ptr(), z.stride(0), coef.data_ptr(), float(eps), out.data_ptr(), z.shape[0], z.shape[1],
+                             _dt(z), _stream()), "poly_norm")
+    return out
+
+
+def gelu_table(u: torch.Tensor, table: torch.Tensor, first: int, tokens: torch.Tensor) -> torch.Tensor:
+    """gelu_tanh(u[t]) * table[tokens[t], first : first + W] for u [T, W], table [vocab, >= first + W]."""
+    dev = _cuda(u, table, tokens)
+    T, W = u.shape
+    if not u.is_contiguous() or not table.is_contiguous() or table.dtype != u.dtype or first + W > table.shape[1]:
+        raise ValueError("u and table must be contiguous, of one dtype, the table wide enough")
+    _tokens("tokens", tokens, T)
+    out = torch.empty_like(u)
+    check(lib.b200_gelu_table(u.data_ptr(), table.data_ptr(), table.shape[1], table.shape[0], int(first), tokens.data_ptr(),
+                              out.data_ptr(), T, W, _dt(u), status_word(dev).data_ptr(), _stream()), "gelu_table")
+    return out
+
+
+class Rotation:
+    """Interleaved rotation of the first 2 * freq.numel() channels of a rotary part; cos and sin times ``magnitude``."""
+
+    def __init__(self, base: float, dims: int, device, scaling: YarnScaling | None = None):
+        self.dims = dims
+        self.freq = rotary_frequencies(base, dims, device, scaling)
+        self.magnitude = scaling.magnitude if scaling is not None else 1.0
+
+
+def latent_prologue(q_in: torch.Tensor | None, q_norm_w: torch.Tensor | None, kv_in: torch.Tensor, kv_norm_w: torch.Tensor,
+                    eps: float, rotation: Rotation, positions: torch.Tensor, cache: torch.Tensor, slot_mapping: torch.Tensor):
+    """Norm of query latents [T, rq] and of latent rows [T, r | dr], whose last dr channels are rotated instead; the rows are
+    also written to cache[slot_mapping] (``b200_latent_prologue``).  Inputs with free row strides.  Returns both."""
+    dev = _cuda(q_in, q_norm_w, kv_in, kv_norm_w, rotation.freq, positions, cache, slot_mapping)
+    T, W = kv_in.shape
+    r = kv_norm_w.numel()
+    _f32vec("kv_norm_w", kv_norm_w, r)
+    if r > W or rotation.dims > W - r or kv_in.stride(1) != 1 or cache.shape[-1] != W or cache.dtype != kv_in.dtype \
+            or not cache.is_contiguous():
+        raise ValueError("latent rows / cache shape, dtype or layout mismatch")
+    for name, t in (("positions", positions), ("slot_mapping", slot_mapping)):
+        _tokens(name, t, T)
+    q_out, rq = None, 0
+    if q_in is not None:
+        rq = q_in.shape[1]
+        if q_in.shape[0] != T or q_in.stride(1) != 1 or q_in.dtype != kv_in.dtype:
+            raise ValueError("query latents must be [T, rq] in the dtype of the latent rows")
+        _f32vec("q_norm_w", q_norm_w, rq)
+        q_out = torch.empty(T, rq, dtype=kv_in.dtype, device=kv_in.device)
+    kv_out = torch.empty(T, W, dtype=kv_in.dtype, device=kv_in.device)
+    check(lib.b200_latent_prologue(
+        _ptr(q_in), q_in.stride(0) if q_in is not None else 0, _ptr(q_norm_w), rq, _ptr(q_out), kv_in.data_ptr(),
+        kv_in.stride(0), kv_norm_w.data_ptr(), r, W - r, float(eps), rotation.freq.data_ptr(), rotation.dims,
+        rotation.magnitude, positions.data_ptr(), kv_out.data_ptr(), cache.data_ptr(), slot_mapping.data_ptr(),
+        cache.numel() // W, T, _dt(kv_in), status_word(dev).data_ptr(), _stream()), "latent_prologue")
+    return q_out, kv_out
+
+
+def rotate_heads(q: torch.Tensor, rope_dim: int, rotation: Rotation, positions: torch.Tensor, tail_rows: int = 0):
+    """Rotates the last ``rope_dim`` channels of every head of q [T, H, D] in place; returns a contiguous copy of the rotated
+    parts of the first ``tail_rows`` tokens [tail_rows, H, rope_dim] (None for none)."""
+    _cuda(q, rotation.freq, positions)
+    T, H, D = q.shape
+    if not q.is_contiguous() or rope_dim > D or rotation.dims > rope_dim or tail_rows > T:
+        raise ValueError("q must be contiguous [T, H, D] with the rotary part inside the head")
+    _tokens("positions", positions, T)
+    tail = torch.empty(tail_rows, H, rope_dim, dtype=q.dtype, device=q.device) if tail_rows else None
+    check(lib.b200_rotate_heads(q.data_ptr(), T, H, D, rope_dim, rotation.freq.data_ptr(), rotation.dims, rotation.magnitude,
+                                positions.data_ptr(), _ptr(tail), tail_rows, _dt(q), _stream()), "rotate_heads")
+    return tail
+
+
+def prefill_window_tile_rows(Hq: int, Hkv: int, Dqk: int, tail: int, Dv: int, dtype: torch.dtype) -> int:
+    """Query rows per tile of the kernel behind ``prefill_varlen_window``; 0 = no tiled kernel."""
+    return int(lib.b200_prefill_window_tile_rows(Hq, Hkv, Dqk, tail, Dv, _DTYPES[dtype])) if dtype in _DTYPES else 0
+
+
+def prefill_varlen_window(q: torch.Tensor, k_head: torch.Tensor, k_tail: torch.Tensor | None, v: torch.Tensor,
+                          cu_seqlens_q: torch.Tensor, cu_seqlens_k: torch.Tensor, max_seqlen_q: int, scale: float,
+                          window: int = 0, sink: torch.Tensor | None = None, out: torch.Tensor | None = None,
+                          plan: "PrefillPlan | None" = None) -> torch.Tensor:
+    """Causal attention over packed keys [Tk, Hkv, Dqk - tail] with a part [Tk, tail] shared by the heads behind them (or
+    None), a sliding window (0: none) and a sink (``b200_prefill_varlen_window``).  q [Tq, Hq, Dqk], v [Tk, Hkv, Dv]; token
+    strides free, heads contiguous.  Contexts may start in the middle: only their ends count.  Returns [Tq, Hq, Dv]."""
+    dev = _cuda(q, k_head, k_tail, v, cu_seqlens_q, cu_seqlens_k, sink, out)
+    Tq, Hq, Dqk = q.shape
+    Tk, Hkv, Dv = v.shape
+    tail = k_tail.shape[1] if k_tail is not None else 0
+    if cu_seqlens_q.dtype != torch.int32 or cu_seqlens_k.dtype != torch.int32 or cu_seqlens_q.numel() != cu_seqlens_k.numel():
+        raise ValueError("cu_seqlens must be int32 tensors of the same length")
+    if k_head.shape != (Tk, Hkv, Dqk - tail) or (tail and k_tail.shape[0] != Tk) \
+            or any(t is not None and t.dtype != q.dtype for t in (k_head, k_tail, v)):
+        raise ValueError("k_head must be [Tk, Hkv, Dqk - tail], k_tail [Tk, tail], v [Tk, Hkv, Dv] in the dtype of q")
+    for t, D in ((q, Dqk), (k_head, Dqk - tail), (v, Dv)):
+        if t.stride(2) != 1 or (t.shape[1] > 1 and t.stride(1) != D):
+            raise ValueError("heads must be contiguous")
+    if tail and k_tail.stride(1) != 1:
+        raise ValueError("k_tail rows must be contiguous")
+    _f32vec("sink", sink, Hq)
+    if out is None:
+        out = torch.empty((Tq, Hq, Dv), dtype=q.dtype, device=q.device)
+    elif out.shape != (Tq, Hq, Dv) or out.dtype != q.dtype or not out.is_contiguous():
+        raise ValueError("out must be a contiguous [Tq, Hq, Dv] tensor")
+    check(lib.b200_prefill_varlen_window(
+        q.data_ptr(), k_head.data_ptr(), _ptr(k_tail), v.data_ptr(), out.data_ptr(), q.stride(0), k_head.stride(0),
+        k_tail.stride(0) if tail else 0, v.stride(0), Tq, Tk, cu_seqlens_q.data_ptr(), cu_seqlens_k.data_ptr(),
+        cu_seqlens_q.numel() - 1, int(max_seqlen_q), Hq, Hkv, Dqk, tail, Dv, float(scale), int(window), _ptr(sink),
+        plan.buffer.data_ptr() if plan is not None else None, plan.tile_rows if plan is not None else 0,
+        plan.capacity if plan is not None else 0, _dt(q), status_word(dev).data_ptr(), _stream()), "prefill_varlen_window")
+    return out
+
+
+def moe_group_route(logits: torch.Tensor, correction: torch.Tensor, top: int, groups: int = 1, keep: int = 1):
+    """Grouped choice of ``top`` experts per token from fp32 logits [T, E] (``b200_moe_group_route``).  Returns (sorted_token
+    [T * top], weight fp32 [T, top], expert_offsets [E], slot_to_row [T, top])."""
+    dev = _cuda(logits, correction)
+    T, E = logits.shape
+    if logits.dtype != torch.float32 or not logits.is_contiguous():
+        raise ValueError("logits must be contiguous fp32 [T, E]")
+    _f32vec("correction", correction, E)
+    tok = torch.empty(T * top, dtype=torch.int32, device=dev)
+    w = torch.empty(T, top, dtype=torch.float32, device=dev)
+    offs = torch.empty(E, dtype=torch.int32, device=dev)
+    slot = torch.empty(T, top, dtype=torch.int32, device=dev)
+    ws = workspace(dev, int(lib.b200_moe_group_route_workspace_bytes(T, E, top)), "moe_group_route")
+    check(lib.b200_moe_group_route(logits.data_ptr(), correction.data_ptr(), T, E, int(top), int(groups), int(keep),
+                                   tok.data_ptr(), w.data_ptr(), offs.data_ptr(), slot.data_ptr(), ws.data_ptr(), ws.numel(),
+                                   _stream()), "moe_group_route")
+    return tok, w, offs, slot
+
+
+def moe_grouped_linear(x: torch.Tensor, w: torch.Tensor, expert_offsets: torch.Tensor,
+                       glu: tuple[float, float] | None = None, early_launch: bool = False) -> torch.Tensor:
+    """Rows of x [R, k] grouped by expert times the expert's weight w [E, n, k] -> [R, n], any size, bf16 or fp32.  ``glu``
+    (limit, slope): w is [E, 2 n, k] = [gate | up] and the clamped gated unit of the two comes back [R, n]."""
+    dev = _cuda(x, w, expert_offsets)
+    (R, k), (E, n, k2) = x.shape, w.shape
+    if x.dtype != w.dtype or k != k2 or not x.is_contiguous() or not w.is_contiguous() or expert_offsets.dtype != torch.int32 \
+            or expert_offsets.numel() != E or (glu is not None and n % 2):
+        raise ValueError("x [R, k] and w [E, n, k] must be contiguous, of one dtype; expert_offsets int32 [E]")
+    n_out = n // 2 if glu is not None else n
+    limit, slope = glu if glu is not None else (0.0, 0.0)
+    out = torch.empty(R, n_out, dtype=x.dtype, device=dev)
+    check(lib.b200_moe_grouped_linear(x.data_ptr(), w.data_ptr(), out.data_ptr(), expert_offsets.data_ptr(), R, E, n_out, k,
+                                      0 if glu is None else 1, float(limit), float(slope),
+                                      MOE_GEMM_EARLY_LAUNCH if early_launch else 0, _dt(x), status_word(dev).data_ptr(),
+                                      _stream()), "moe_grouped_linear")
     return out

@@ -40,6 +40,15 @@ class Singles:
 
 
 @dataclass
+class KeyRange:
+    """The keys that the portions of a step reach: the ends of their contexts, packed."""
+    cu_seqlens_k: torch.Tensor                    # int32 [n + 1], starts at 0
+    max_seqlen_k: int
+    total_k: int
+    has_prefix: bool                              # some of them came in an earlier step
+
+
+@dataclass
 class Portions:
     """The other sequences of a mixed step: prompts and portions of prompts, ragged, behind the singles' rows."""
     num_tokens: int                               # rows of the step that belong to a sequence, singles included
@@ -51,7 +60,14 @@ class Portions:
     has_prefix: bool                              # some context is longer than its portion
     block_tables: torch.Tensor                    # int32 [n, max_blocks]
     state_slots: Optional[torch.Tensor]           # int64 [n]
+    ranges: dict = field(default_factory=dict)    # window -> KeyRange, for the windows the model's layers have
     plans: dict = field(default_factory=dict)     # tile lists by rows per tile, built when a layer asks
+
+    def keys(self, window: int = 0) -> KeyRange:
+        """What a layer with this sliding window needs of the contexts (0: all of them)."""
+        if window in self.ranges:
+            return self.ranges[window]
+        return KeyRange(self.cu_seqlens_k, self.max_seqlen_k, self.total_k, self.has_prefix)
 
     def plan(self, tile_rows: int):
         if tile_rows <= 0:
