@@ -116,7 +116,8 @@ def clamped_glu(gate, up, limit, slope=1.702):
 
 
 def route(h, w_router, correction, groups, keep, top):
-    """Per token the chosen experts (a set, ascending) and their weights."""
+    """Per token the chosen experts (a set, ascending), their weights, and the margin of the choice: how far the last kept
+    group is from the next, and the last chosen expert from the next one allowed, whichever is closer."""
     s = torch.sigmoid(h @ w_router.T)
     out = []
     for t in range(h.shape[0]):
@@ -125,15 +126,23 @@ def route(h, w_router, correction, groups, keep, top):
         score = [sum(sorted(choice[g * size:(g + 1) * size])[-2:]) for g in range(groups)]
         best = sorted(range(groups), key=lambda g: -score[g])[:keep]
         allowed = [e for e in range(len(choice)) if e // size in best]
-        chosen = sorted(sorted(allowed, key=lambda e: -choice[e])[:top])
-        out.append((chosen, s[t, chosen] / (s[t, chosen].sum() + 1e-20)))
+        ranked = sorted(allowed, key=lambda e: -choice[e])
+        chosen = sorted(ranked[:top])
+        gaps = [choice[ranked[top - 1]] - choice[ranked[top]]] if top < len(ranked) else []
+        if keep < groups:
+            order = sorted(score, reverse=True)
+            gaps.append(order[keep - 1] - order[keep])
+        out.append((chosen, s[t, chosen] / (s[t, chosen].sum() + 1e-20), min(gaps, default=math.inf)))
     return out
 
 
-def moe_mlp(h, w, c):
+def moe_mlp(h, w, c, margins=None):
     r, rows = c["router"], []
     g = r.get("groups") or {"count": 1, "keep": 1}
-    for x, (chosen, weights) in zip(h, route(h, w["router"], w["correction"], g["count"], g["keep"], r["top"])):
+    choices = route(h, w["router"], w["correction"], g["count"], g["keep"], r["top"])
+    if margins is not None:
+        margins.append([m for _, _, m in choices])
+    for x, (chosen, weights, _) in zip(h, choices):
         y = torch.zeros_like(x)
         for e, p in zip(chosen, weights):
             act = clamped_glu(w[f"e{e}.gate"] @ x, w[f"e{e}.up"] @ x, c["expert"]["limit"])
@@ -174,8 +183,9 @@ def _sub(w, prefix):
     return {k[len(prefix):]: v for k, v in w.items() if k.startswith(prefix)}
 
 
-def forward(config, weights, tokens, dtype=torch.float64, collect=None):
-    """Logits [n, vocab] of one sequence; ``collect`` (a list) receives the residual after every layer run."""
+def forward(config, weights, tokens, dtype=torch.float64, collect=None, margins=None):
+    """Logits [n, vocab] of one sequence; ``collect`` (a list) receives the residual after every layer run, ``margins`` the
+    margins of every routing, per token."""
     w = {k: v.to(dtype) if v.is_floating_point() else v for k, v in weights.items()}
     eps, groups = config["norm"]["eps"], config["norm"].get("groups", 1)
     ids = torch.as_tensor(tokens, dtype=torch.long)
@@ -191,7 +201,7 @@ def forward(config, weights, tokens, dtype=torch.float64, collect=None):
         mlp = layer.get("mlp")
         if mlp is not None:
             m = _sub(lw, "mlp.")
-            f = dense_mlp(h, m, eps) if mlp["kind"] == "dense" else moe_mlp(h, m, mlp)
+            f = dense_mlp(h, m, eps) if mlp["kind"] == "dense" else moe_mlp(h, m, mlp, margins)
             y = y + f * residual_gate(h, lw["rg2"], lw["rg2.b"])
         x = token_input(x + y, side[:, i * dim:(i + 1) * dim], lw, eps)
         if collect is not None:
