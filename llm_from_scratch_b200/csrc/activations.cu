@@ -1,6 +1,6 @@
 // Activations of feed-forwards and heads: squared ReLU, the polynomial of normed powers, a tanh GELU that scales rows of a
 // token table, and the scale and soft cap of logits.
-#include "common.cuh"
+#include "sequences.cuh"
 
 namespace b200 {
 namespace {
@@ -106,24 +106,57 @@ void poly_norm(const void* z, int64_t stride, const float* coef, float eps, void
   else poly_norm_kernel<T, E, 0><<<grid, 512, 0, s>>>(zp, stride, coef, eps, op, W);
 }
 
-// out[t] = gelu_tanh(u[t]) * table[tokens[t], first .. first + W - 1]
-template <typename T>
+// out[t] = gelu_tanh(u[t]) * table[tokens[t], first .. first + W - 1]; E elements per access.
+// gelu_tanh(z) = z sigmoid(2 sqrt(2 / pi) (z + 0.044715 z^3))
+template <typename T, int E>
 __global__ void __launch_bounds__(256) gelu_table_kernel(const T* u, const T* table, int64_t table_width, int64_t vocab, int first,
                                                          const int64_t* tokens, T* out, int64_t rows, int W, int32_t* status) {
-  const int64_t total = rows * W;
+  const int units = W / E;
+  const int64_t total = rows * units;
+  union Pack {
+    uint4 u;
+    T e[16 / sizeof(T)];
+  };
   for (int64_t i = static_cast<int64_t>(blockIdx.x) * blockDim.x + threadIdx.x; i < total;
        i += static_cast<int64_t>(gridDim.x) * blockDim.x) {
-    const int64_t t = i / W;
-    const int c = static_cast<int>(i - t * W);
+    const int64_t t = i / units;
+    const int c = static_cast<int>(i - t * units) * E;
     int64_t tok = tokens[t];
     if (tok < 0 || tok >= vocab) {
       report(status, B200_ERR_BOUNDS);
       tok = 0;
     }
-    const float z = to_float<T>(u[i]);
-    const float g = 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
-    out[i] = from_float<T>(g * to_float<T>(table[tok * table_width + first + c]));
+    const T* up = u + t * W + c;
+    const T* tp = table + tok * table_width + first + c;
+    Pack z, e;
+    if constexpr (E > 1) {
+      z.u = *reinterpret_cast<const uint4*>(up);
+      e.u = *reinterpret_cast<const uint4*>(tp);
+    } else {
+      z.e[0] = up[0];
+      e.e[0] = tp[0];
+    }
+#pragma unroll
+    for (int k = 0; k < E; ++k) {
+      const float v = to_float<T>(z.e[k]);
+      z.e[k] = from_float<T>(v * sigmoid_for<T>(1.5957691216057308f * (v + 0.044715f * v * v * v)) * to_float<T>(e.e[k]));
+    }
+    if constexpr (E > 1) *reinterpret_cast<uint4*>(out + t * W + c) = z.u;
+    else out[t * W + c] = z.e[0];
   }
+}
+
+template <typename T>
+void gelu_table(const void* u, const void* table, int64_t table_width, int64_t vocab, int first, const int64_t* tokens, void* out,
+                int64_t rows, int W, int32_t* status, cudaStream_t s) {
+  constexpr int E = 16 / sizeof(T);
+  const bool vec = W % E == 0 && table_width % E == 0 && first % E == 0 && aligned16(u) && aligned16(table) && aligned16(out);
+  const int64_t blocks = (rows * (W / (vec ? E : 1)) + 255) / 256;
+  const unsigned grid = static_cast<unsigned>(blocks < 148 * 32 ? blocks : 148 * 32);
+  const T* up = static_cast<const T*>(u);
+  const T* tp = static_cast<const T*>(table);
+  if (vec) gelu_table_kernel<T, E><<<grid, 256, 0, s>>>(up, tp, table_width, vocab, first, tokens, static_cast<T*>(out), rows, W, status);
+  else gelu_table_kernel<T, 1><<<grid, 256, 0, s>>>(up, tp, table_width, vocab, first, tokens, static_cast<T*>(out), rows, W, status);
 }
 
 __global__ void __launch_bounds__(256) softcap_kernel(float* z, int64_t n, float scale, float cap, float inv_cap) {
@@ -198,13 +231,7 @@ extern "C" int b200_gelu_table(const void* u, const void* table, int64_t table_w
   if (rows == 0) return B200_OK;
   if (!u || !table || !tokens || !out) return B200_ERR_ARG;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  const unsigned grid = elementwise_grid(rows * width);
-  if (dtype == B200_DTYPE_F32)
-    gelu_table_kernel<float><<<grid, 256, 0, s>>>(static_cast<const float*>(u), static_cast<const float*>(table), table_width,
-                                                  vocab, first, tokens, static_cast<float*>(out), rows, width, status);
-  else
-    gelu_table_kernel<__nv_bfloat16><<<grid, 256, 0, s>>>(
-        static_cast<const __nv_bfloat16*>(u), static_cast<const __nv_bfloat16*>(table), table_width, vocab, first, tokens,
-        static_cast<__nv_bfloat16*>(out), rows, width, status);
+  if (dtype == B200_DTYPE_F32) gelu_table<float>(u, table, table_width, vocab, first, tokens, out, rows, width, status, s);
+  else gelu_table<__nv_bfloat16>(u, table, table_width, vocab, first, tokens, out, rows, width, status, s);
   return launch_result();
 }

@@ -126,6 +126,13 @@ __device__ __forceinline__ float clamped_glu_f(float g, float u, float limit, fl
   return g * (u + 1.f) / (1.f + expf(-slope * g));
 }
 
+// The same for results that are rounded to bf16 next: approximate exponential and division (relative error about 1e-6).
+__device__ __forceinline__ float clamped_glu_bf16(float g, float u, float limit, float slope) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return __fdividef(g * (u + 1.f), 1.f + fminf(__expf(-slope * g), 1e30f));
+}
+
 // Prefill tile list (b200_prefill_plan): int32 header {tile count, rows per tile, capacity, 0} followed
 // by one entry per query tile, (sequence << 16) | tile index, heaviest tiles first.
 constexpr int kPlanHeader = 4;

@@ -90,7 +90,9 @@ struct LpArgs {
   int32_t* status;
 };
 
-// dst (and dst2, if given) = src / rms(src) * w over n elements, by a warp; E elements per access
+// dst (and dst2, if given) = src / rms(src) * w over n elements, by a warp; E elements per access.  Rows of up to kKeep
+// accesses per lane stay in registers between the two passes.
+constexpr int kKeep = 4;
 template <typename T, int E>
 __device__ __forceinline__ void warp_norm(const T* src, const float* w, int n, float eps, T* dst, T* dst2) {
   const int lane = threadIdx.x & 31;
@@ -98,29 +100,48 @@ __device__ __forceinline__ void warp_norm(const T* src, const float* w, int n, f
     uint4 u;
     T e[16 / sizeof(T)];
   };
-  float ss = 0.f;
-  for (int c = lane * E; c < n; c += 32 * E) {
+  auto load = [&](int c) {
     Pack p;
     if constexpr (E > 1) p.u = *reinterpret_cast<const uint4*>(src + c);
     else p.e[0] = src[c];
+    return p;
+  };
+  Pack keep[kKeep];
+  float ss = 0.f;
+  auto add = [&](const Pack& p) {
 #pragma unroll
     for (int i = 0; i < E; ++i) ss += to_float<T>(p.e[i]) * to_float<T>(p.e[i]);
-  }
-  const float inv = rsqrtf(warp_sum(ss) / static_cast<float>(n) + eps);
-  for (int c = lane * E; c < n; c += 32 * E) {
-    Pack p;
-    if constexpr (E > 1) p.u = *reinterpret_cast<const uint4*>(src + c);
-    else p.e[0] = src[c];
+  };
 #pragma unroll
-    for (int i = 0; i < E; ++i) p.e[i] = from_float<T>(to_float<T>(p.e[i]) * inv * w[c + i]);
+  for (int k = 0; k < kKeep; ++k)
+    if ((k * 32 + lane) * E < n) keep[k] = load((k * 32 + lane) * E);
+#pragma unroll
+  for (int k = 0; k < kKeep; ++k)
+    if ((k * 32 + lane) * E < n) add(keep[k]);
+  for (int c = (kKeep * 32 + lane) * E; c < n; c += 32 * E) add(load(c));
+  const float inv = rsqrtf(warp_sum(ss) / static_cast<float>(n) + eps);
+  auto put = [&](int c, Pack p) {
     if constexpr (E > 1) {
+#pragma unroll
+      for (int i = 0; i < E; i += 4) {
+        const float4 wv = *reinterpret_cast<const float4*>(w + c + i);
+        p.e[i] = from_float<T>(to_float<T>(p.e[i]) * inv * wv.x);
+        p.e[i + 1] = from_float<T>(to_float<T>(p.e[i + 1]) * inv * wv.y);
+        p.e[i + 2] = from_float<T>(to_float<T>(p.e[i + 2]) * inv * wv.z);
+        p.e[i + 3] = from_float<T>(to_float<T>(p.e[i + 3]) * inv * wv.w);
+      }
       *reinterpret_cast<uint4*>(dst + c) = p.u;
       if (dst2) *reinterpret_cast<uint4*>(dst2 + c) = p.u;
     } else {
+      p.e[0] = from_float<T>(to_float<T>(p.e[0]) * inv * w[c]);
       dst[c] = p.e[0];
       if (dst2) dst2[c] = p.e[0];
     }
-  }
+  };
+#pragma unroll
+  for (int k = 0; k < kKeep; ++k)
+    if ((k * 32 + lane) * E < n) put((k * 32 + lane) * E, keep[k]);
+  for (int c = (kKeep * 32 + lane) * E; c < n; c += 32 * E) put(c, load(c));
 }
 
 // blockIdx.y 0: latent rows; 1: query latents.  A warp per row; EQ / EK elements per access
@@ -143,7 +164,6 @@ __global__ void __launch_bounds__(kWarps * 32) latent_prologue_kernel(const LpAr
   const T* src = static_cast<const T*>(a.kv_in) + t * a.kv_stride;
   T* out = static_cast<T*>(a.kv_out) + t * W;
   T* pool = slot >= 0 ? static_cast<T*>(a.cache) + slot * W : nullptr;
-  warp_norm<T, EK>(src, a.wkv, a.r, a.eps, out, pool);
   const int64_t pos = a.positions[t];
   for (int i = lane; 2 * i < a.dr; i += 32) {
     const int c = a.r + 2 * i;
@@ -162,6 +182,7 @@ __global__ void __launch_bounds__(kWarps * 32) latent_prologue_kernel(const LpAr
       if (pair) pool[c + 1] = from_float<T>(v);
     }
   }
+  warp_norm<T, EK>(src, a.wkv, a.r, a.eps, out, pool);
 }
 
 struct RtArgs {
@@ -174,57 +195,65 @@ struct RtArgs {
   const int64_t* positions;
   void* tail;                // [tail_rows, H, dr] or null: a copy of the rotated parts of the first rows
   int64_t tail_rows;
+  int per_cta;               // tokens
 };
 
-// kRotTokens tokens per CTA; one pair of channels per thread and trip
-constexpr int kRotTokens = 2;
-template <typename T, bool PAIRS>
+// per_cta tokens per CTA; V consecutive channels (whole pairs, 16 bytes) per thread and trip, or one pair
+template <typename T, int V>
 __global__ void __launch_bounds__(256) rotate_heads_kernel(const RtArgs a) {
-  extern __shared__ float2 cs[];     // [kRotTokens][half]
-  const int64_t t0 = static_cast<int64_t>(blockIdx.x) * kRotTokens;
-  const int nt = static_cast<int>(a.T - t0 < kRotTokens ? a.T - t0 : kRotTokens);
+  extern __shared__ float2 cs[];     // [per_cta][half]
+  const int64_t t0 = static_cast<int64_t>(blockIdx.x) * a.per_cta;
+  const int nt = static_cast<int>(a.T - t0 < a.per_cta ? a.T - t0 : a.per_cta);
   for (int i = threadIdx.x; i < nt * a.half; i += blockDim.x) {
     const int t = i / a.half, j = i - t * a.half;
     const float2 r = rotary_angle(a.positions[t0 + t], a.freq[j]);
     cs[i] = make_float2(r.x * a.magnitude, r.y * a.magnitude);
   }
   __syncthreads();
-  const int pairs = (a.dr + 1) / 2, per = a.H * pairs;
+  constexpr int W = V > 2 ? V : 2;
+  const int units = (a.dr + W - 1) / W, per = a.H * units;
   for (int i = threadIdx.x; i < nt * per; i += blockDim.x) {
-    const int t = i / per, k = i - t * per, h = k / pairs, j = k - h * pairs;
+    const int t = i / per, k = i - t * per, h = k / units, c = (k - h * units) * W;
     const int64_t tok = t0 + t;
-    T* p = static_cast<T*>(a.q) + (tok * a.H + h) * a.D + (a.D - a.dr) + 2 * j;
-    T* tail = tok < a.tail_rows ? static_cast<T*>(a.tail) + (tok * a.H + h) * a.dr + 2 * j : nullptr;
-    const bool pair = 2 * j + 1 < a.dr;
-    float u, v;
-    if constexpr (PAIRS) {
-      if constexpr (sizeof(T) == 2) {
-        const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p));
-        u = f.x, v = f.y;
-      } else {
-        const float2 f = *reinterpret_cast<const float2*>(p);
-        u = f.x, v = f.y;
-      }
+    T* p = static_cast<T*>(a.q) + (tok * a.H + h) * a.D + (a.D - a.dr) + c;
+    T* tail = tok < a.tail_rows ? static_cast<T*>(a.tail) + (tok * a.H + h) * a.dr + c : nullptr;
+    float x[W];
+    union {
+      uint4 u;
+      T e[16 / sizeof(T)];
+    } pack;
+    const bool pair = c + 1 < a.dr;
+    if constexpr (V > 2) {
+      pack.u = *reinterpret_cast<const uint4*>(p);
+#pragma unroll
+      for (int e = 0; e < W; ++e) x[e] = to_float<T>(pack.e[e]);
     } else {
-      u = to_float<T>(p[0]), v = pair ? to_float<T>(p[1]) : 0.f;
+      x[0] = to_float<T>(p[0]);
+      x[1] = pair ? to_float<T>(p[1]) : 0.f;
     }
-    if (j < a.half) {
-      const float2 r = cs[t * a.half + j];
-      const float nu = u * r.x - v * r.y;
-      v = v * r.x + u * r.y;
-      u = nu;
-    }
-    auto put = [&](T* d) {
-      if constexpr (PAIRS) {
-        if constexpr (sizeof(T) == 2) *reinterpret_cast<uint32_t*>(d) = pack_bf16x2(u, v);
-        else *reinterpret_cast<float2*>(d) = make_float2(u, v);
-      } else {
-        d[0] = from_float<T>(u);
-        if (pair) d[1] = from_float<T>(v);
+#pragma unroll
+    for (int e = 0; e < W; e += 2) {
+      const int j = (c + e) >> 1;
+      if (j < a.half) {
+        const float2 r = cs[t * a.half + j];
+        const float u = x[e], v = x[e + 1];
+        x[e] = u * r.x - v * r.y;
+        x[e + 1] = v * r.x + u * r.y;
       }
-    };
-    put(p);
-    if (tail) put(tail);
+    }
+    if constexpr (V > 2) {
+#pragma unroll
+      for (int e = 0; e < W; ++e) pack.e[e] = from_float<T>(x[e]);
+      *reinterpret_cast<uint4*>(p) = pack.u;
+      if (tail) *reinterpret_cast<uint4*>(tail) = pack.u;
+    } else {
+      p[0] = from_float<T>(x[0]);
+      if (pair) p[1] = from_float<T>(x[1]);
+      if (tail) {
+        tail[0] = from_float<T>(x[0]);
+        if (pair) tail[1] = from_float<T>(x[1]);
+      }
+    }
   }
 }
 
@@ -390,9 +419,9 @@ extern "C" int b200_latent_prologue(const void* q_in, int64_t q_stride, const fl
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   const dim3 grid(static_cast<unsigned>((num_tokens + kWarps - 1) / kWarps), q_in ? 2 : 1);
   const int E = dtype == B200_DTYPE_F32 ? 4 : 8;
-  const bool vq = !q_in || (q_rank % E == 0 && q_stride % E == 0 && aligned16(q_in) && aligned16(q_out));
+  const bool vq = !q_in || (q_rank % E == 0 && q_stride % E == 0 && aligned16(q_in) && aligned16(q_out) && aligned16(q_norm_w));
   const bool vk = kv_rank % E == 0 && (kv_rank + rope_dim) % E == 0 && kv_stride % E == 0 && aligned16(kv_in) && aligned16(kv_out) &&
-                  (!cache || aligned16(cache));
+                  aligned16(kv_norm_w) && (!cache || aligned16(cache));
   if (dtype == B200_DTYPE_F32) {
     if (vq && vk) latent_prologue_kernel<float, 4, 4><<<grid, kWarps * 32, 0, s>>>(a);
     else latent_prologue_kernel<float, 1, 1><<<grid, kWarps * 32, 0, s>>>(a);
@@ -413,18 +442,21 @@ extern "C" int b200_rotate_heads(void* q, int64_t num_tokens, int32_t num_heads,
   if (dtype != B200_DTYPE_F32 && dtype != B200_DTYPE_BF16) return B200_ERR_UNSUPPORTED;
   if (num_tokens == 0 || rope_dim == 0) return B200_OK;
   if (!q || !positions || (rot_dims > 0 && !freq) || (tail_rows > 0 && !tail)) return B200_ERR_ARG;
-  if (rot_dims > 4096 || num_tokens > 2147483647LL) return B200_ERR_UNSUPPORTED;
-  RtArgs a{q, num_tokens, num_heads, head_dim, rope_dim, freq, rot_dims / 2, magnitude, positions, tail, tail_rows};
+  if (rot_dims > 2048 || num_tokens > 2147483647LL) return B200_ERR_UNSUPPORTED;
+  RtArgs a{q, num_tokens, num_heads, head_dim, rope_dim, freq, rot_dims / 2, magnitude, positions, tail, tail_rows, 1};
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  const unsigned grid = static_cast<unsigned>((num_tokens + kRotTokens - 1) / kRotTokens);
-  const size_t smem = sizeof(float2) * kRotTokens * (rot_dims / 2);
-  const bool pairs = head_dim % 2 == 0 && rope_dim % 2 == 0 && aligned16(q) && (!tail || aligned16(tail));
+  // a few tokens per CTA share its threads for their angles; small steps spread over the SMs instead
+  a.per_cta = num_tokens >= 4096 ? 4 : num_tokens >= 512 ? 2 : 1;
+  const unsigned grid = static_cast<unsigned>((num_tokens + a.per_cta - 1) / a.per_cta);
+  const size_t smem = sizeof(float2) * a.per_cta * (rot_dims / 2);
+  const int E = dtype == B200_DTYPE_F32 ? 4 : 8;
+  const bool vec = head_dim % E == 0 && rope_dim % E == 0 && aligned16(q) && (!tail || aligned16(tail));
   if (dtype == B200_DTYPE_F32) {
-    if (pairs) rotate_heads_kernel<float, true><<<grid, 256, smem, s>>>(a);
-    else rotate_heads_kernel<float, false><<<grid, 256, smem, s>>>(a);
+    if (vec) rotate_heads_kernel<float, 4><<<grid, 256, smem, s>>>(a);
+    else rotate_heads_kernel<float, 2><<<grid, 256, smem, s>>>(a);
   } else {
-    if (pairs) rotate_heads_kernel<__nv_bfloat16, true><<<grid, 256, smem, s>>>(a);
-    else rotate_heads_kernel<__nv_bfloat16, false><<<grid, 256, smem, s>>>(a);
+    if (vec) rotate_heads_kernel<__nv_bfloat16, 8><<<grid, 256, smem, s>>>(a);
+    else rotate_heads_kernel<__nv_bfloat16, 2><<<grid, 256, smem, s>>>(a);
   }
   return launch_result();
 }

@@ -370,7 +370,7 @@ moe_gemm_kernel(const GemmArgs a, const __grid_constant__ CUtensorMap tm_w,
                 uv = bf16_round(uv + __bfloat162float(vec ? b3.b[x] : bg[a.n_out + x]));
               }
               if (a.mode == 3) {
-                o.b[x] = __float2bfloat16(clamped_glu_f(gv, uv, a.limit, a.slope));
+                o.b[x] = __float2bfloat16(clamped_glu_bf16(gv, uv, a.limit, a.slope));
               } else {
                 const float sv = bf16_round(gv / (1.f + expf(-gv)));
                 o.b[x] = __float2bfloat16(sv * uv);

@@ -263,7 +263,7 @@ moe_gemm_rows_kernel(const RowsArgs a, const __grid_constant__ CUtensorMap tm_x,
               }
               // fast exponential and division: their ~1e-6 relative error disappears in the bf16 rounding of silu
               if (a.mode == 3) {
-                o.b[x] = __float2bfloat16(clamped_glu_f(gv, uv, a.limit, a.slope));
+                o.b[x] = __float2bfloat16(clamped_glu_bf16(gv, uv, a.limit, a.slope));
               } else {
                 const float sv = bf16r(__fdividef(gv, 1.f + __expf(-gv)));
                 o.b[x] = __float2bfloat16(sv * uv);

@@ -20,7 +20,8 @@
 // softmax warps find their next tile ready, and one problem's waits never hold up the other's instructions.
 // K/V tiles go through a ring of NST stages that both problems release.  Rescaling of O is lazy as in
 // prefill_umma.cu and waits for the P.V product before it.  With a sliding window (WINDOW) the walk starts at the first
-// tile that the window of row 0 reaches; problem B meets up to three fully masked tiles there.  Every wait is bounded; a timeout aborts the CTA
+// tile that the window of row 0 reaches; problem B passes over the first tiles, which none of its rows sees: its issuing
+// thread and its softmax warps take the same turns at every barrier there, without products.  Every wait is bounded; a timeout aborts the CTA
 // and is reported.
 //
 // What sets the pace, measured with clock counters in the warps: (1) the special-function unit — the 64
@@ -129,6 +130,8 @@ prefill_umma2_kernel(const Args2 a, const __grid_constant__ CUtensorMap tm_q, co
     nt[x] = rows[x] > 0 ? (km + BN - 1) / BN : 0;
   }
   const bool has_b = rows[1] > 0;
+  // first tile a row of B sees: at most two behind A's, which A always walks (the window moves by 128 keys)
+  const int first_b = WINDOW ? max(0, off + m0 + BM - a.window + 1) / BN : 0;
   const int n = max(nt[0], nt[1]);               // KV tiles walked by the CTA; >= 1
 
   if (tid == 0) {
@@ -207,7 +210,12 @@ prefill_umma2_kernel(const Args2 a, const __grid_constant__ CUtensorMap tm_q, co
       const uint64_t kd = umma::smem_desc(sb + L::OFF_KV, 0, 1024);
       const uint64_t vd = umma::smem_desc(sb + L::OFF_KV + L::K_BYTES, K_SLAB, 1024);
       const uint32_t tSx = tmem + x * (128 + DV), tOx = tSx + 128;
-      auto qk = [&](int st, int buf) {       // S[buf] = Q . K^T of the tile in stage st, contraction in steps of 16
+      const int j0 = WINDOW && x == 1 ? first_b : 0;
+      auto qk = [&](int st, int buf, int j) {       // S[buf] = Q . K^T of tile j in stage st, contraction in steps of 16
+        if (WINDOW && j < j0) {
+          umma::mbar_arrive(bar(L::QK_DONE + x) + st * 16);
+          return;
+        }
         const uint32_t so = st * (L::STAGE >> 4);
 #pragma unroll
         for (int ks = 0; ks < DQK / 16; ++ks)
@@ -219,7 +227,7 @@ prefill_umma2_kernel(const Args2 a, const __grid_constant__ CUtensorMap tm_q, co
       if (!ok) give_up();
       if (ok) {
         umma::fence_after_sync();
-        qk(0, 0);
+        qk(0, 0, 0);
       }
       int st = 0, ph = 0;                      // stage and phase of tile j
       for (int j = 0; ok && j < nx; ++j) {
@@ -231,16 +239,22 @@ prefill_umma2_kernel(const Args2 a, const __grid_constant__ CUtensorMap tm_q, co
         if (j + 1 < nx) {
           WAIT_OR_ABORT(L::K_FULL + st1, ph1)
           umma::fence_after_sync();
-          qk(st1, (j + 1) & 1);
+          qk(st1, (j + 1) & 1, j + 1);
         }
         WAIT_OR_ABORT(L::P_READY + 2 * x + (j & 1), (j >> 1) & 1)
         WAIT_OR_ABORT(L::V_FULL + st, ph)
         umma::fence_after_sync();
+        if (WINDOW && j < j0) {
+          umma::mbar_arrive(bar(L::PV_DONE + x) + st * 16);
+          st = st1;
+          ph = ph1;
+          continue;
+        }
         const uint32_t so = st * (L::STAGE >> 4);
 #pragma unroll
         for (int ks = 0; ks < BN / 16; ++ks)        // O += P[j & 1] . V_j : contraction over the 64 keys
           umma::mma_ts(tOx, tSx + (j & 1) * 64 + ks * 8, umma::desc_advance(vd, so + ks * (2048 >> 4)), idesc_pv,
-                       !(j == 0 && ks == 0));
+                       !(j == j0 && ks == 0));
         umma::commit(bar(L::PV_DONE + x) + st * 16);
         st = st1;
         ph = ph1;
@@ -259,6 +273,7 @@ prefill_umma2_kernel(const Args2 a, const __grid_constant__ CUtensorMap tm_q, co
     const uint32_t qk_done = bar(L::QK_DONE + x), pv_done = bar(L::PV_DONE + x);
     const uint32_t my_turn = bar(L::TURN + (x == 0 ? 0 : 4) + (warp & 3));
     const uint32_t their_turn = bar(L::TURN + (x == 0 ? 4 : 0) + (warp & 3));
+    const int j0 = WINDOW && x == 1 ? first_b : 0;          // first tile with products
     float m_ref = -INFINITY, l = 0.f;
     bool alive = true;
     int st = 0, ph = 0, stp = 0, php = 0;                   // stage and phase of tile j and of tile j - 1
@@ -271,6 +286,22 @@ prefill_umma2_kernel(const Args2 a, const __grid_constant__ CUtensorMap tm_q, co
         break;
       }
       umma::fence_after_sync();
+      if (WINDOW && j < j0) {                                 // problem B only: every tile here is one of A's
+        if (!__all_sync(0xffffffffu, umma::mbar_wait(my_turn, j & 1, s_abort))) {
+          give_up();
+          alive = false;
+          break;
+        }
+        umma::mbar_arrive(their_turn);
+        umma::mbar_arrive(bar(L::P_READY + 2 * x + (j & 1)));
+        stp = st;
+        php = ph;
+        if (++st == NST) {
+          st = 0;
+          ph ^= 1;
+        }
+        continue;
+      }
       const int n0 = j * BN;
       const bool warp_masked = __any_sync(0xffffffffu, n0 + BN - 1 > lim || (WINDOW && n0 < low));
       // the 64 raw scores of the row stay in registers for both passes
@@ -306,7 +337,7 @@ prefill_umma2_kernel(const Args2 a, const __grid_constant__ CUtensorMap tm_q, co
         const float m_new = need ? mx : m_ref;
         const float alpha = (m_ref == -INFINITY) ? (need ? 0.f : 1.f) : fast_exp2(m_ref - m_new);
         l *= alpha;
-        if (j > 0) {
+        if (j > j0) {
           // O still receives P(j-1).V(j-1): the scores of this tile were issued ahead of that product
           if (!__all_sync(0xffffffffu, umma::mbar_wait(pv_done + stp * 16, php, s_abort))) {
             give_up();

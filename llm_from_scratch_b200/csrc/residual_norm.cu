@@ -64,13 +64,14 @@ __device__ __forceinline__ int64_t embed_row(const ResArgs& a, int64_t row) {
 }
 
 constexpr int kMaxParts = 64;      // groups of the final norm in the register kernel
+enum Parts { kWhole, kWarps, kAny };
 
-// N groups of four channels per thread, d a multiple of four; GROUPED: the final norm has a.groups parts, each a multiple of
-// four channels wide
-template <typename T, int N, bool GROUPED>
+// N groups of four channels per thread, d a multiple of four.  PARTS: the final norm is one part, or a.groups parts of which
+// each is whole warps wide (a multiple of 128 channels: one barrier) or any multiple of four channels wide
+template <typename T, int N, Parts PARTS>
 __global__ void __launch_bounds__(1024) residual_norm_kernel(const ResArgs a) {
   __shared__ float scratch[2][32];
-  __shared__ float part[GROUPED ? 1024 * N : 1], part_inv[GROUPED ? kMaxParts : 1];
+  __shared__ float part[PARTS == kAny ? 1024 * N : 32 * N], part_inv[PARTS == kAny ? kMaxParts : 1];
   const int d = a.d, step = blockDim.x * 4, first = threadIdx.x * 4;
   const int64_t row = blockIdx.x;
   float* xr = a.x + row * d;
@@ -119,7 +120,22 @@ __global__ void __launch_bounds__(1024) residual_norm_kernel(const ResArgs a) {
   }
   if (a.final_w != nullptr) {
     float inv[N];
-    if constexpr (GROUPED) {
+    if constexpr (PARTS == kWarps) {
+      const int width = d / a.groups, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+#pragma unroll
+      for (int i = 0; i < N; ++i) {
+        const float ss = warp_sum(sumsq(x[i]));
+        if (lane == 0) part[i * nw + warp] = ss;              // of channels (i * nw + warp) * 128 ...
+      }
+      __syncthreads();
+#pragma unroll
+      for (int i = 0; i < N; ++i) {
+        const int per = width >> 7, first_warp = (i * nw + warp) / per * per;
+        float ss = 0.f;
+        for (int k = lane; k < per; k += 32) ss += first_warp + k < N * nw ? part[first_warp + k] : 0.f;
+        inv[i] = rsqrtf(warp_sum(ss) / static_cast<float>(width) + a.eps);
+      }
+    } else if constexpr (PARTS == kAny) {
       const int width = d / a.groups, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
 #pragma unroll
       for (int i = 0; i < N; ++i) {
@@ -190,11 +206,11 @@ __global__ void __launch_bounds__(256) residual_norm_any_kernel(const ResArgs a)
   }
 }
 
-template <typename T, bool GROUPED>
+template <typename T, Parts PARTS>
 void launch_vec(const ResArgs& a, unsigned grid, cudaStream_t s) {
   const int groups = a.d / 4;
-  if (groups <= 1024) residual_norm_kernel<T, 1, GROUPED><<<grid, (groups + 31) / 32 * 32, 0, s>>>(a);
-  else residual_norm_kernel<T, 2, GROUPED><<<grid, (groups + 63) / 64 * 32, 0, s>>>(a);
+  if (groups <= 1024) residual_norm_kernel<T, 1, PARTS><<<grid, (groups + 31) / 32 * 32, 0, s>>>(a);
+  else residual_norm_kernel<T, 2, PARTS><<<grid, (groups + 63) / 64 * 32, 0, s>>>(a);
 }
 
 template <typename T>
@@ -203,8 +219,9 @@ void launch(const ResArgs& a, int64_t rows, bool vec, cudaStream_t s) {
   const bool grouped = a.final_w && a.groups > 1;
   if (!vec || a.d / 4 > 2048 || (grouped && (a.d / a.groups % 4 != 0 || a.groups > kMaxParts)))
     residual_norm_any_kernel<T><<<grid, 256, 0, s>>>(a);
-  else if (grouped) launch_vec<T, true>(a, grid, s);
-  else launch_vec<T, false>(a, grid, s);
+  else if (!grouped) launch_vec<T, kWhole>(a, grid, s);
+  else if (a.d / a.groups % 128 == 0) launch_vec<T, kWarps>(a, grid, s);
+  else launch_vec<T, kAny>(a, grid, s);
 }
 
 int residual_norm(const ResArgs& a, int64_t rows, int32_t dtype, void* stream) {

@@ -127,7 +127,10 @@ class ModelRunner:
             self.max_model_length = self.model_config.context_length or min(self.num_kv_blocks * self.block_size, 1 << 17)
         if not self.enforce_eager:
             self.capture_cudagraph()
-            if self.prefill_tile_rows and _cfg(config, "prefill_graphs", default=True):
+            # a model with steps in two parts may have its steps of whole prompts captured (no single tokens, every
+            # context inside the step); its layers ask for the tile lists themselves
+            self.captures_prompts = self.splits_steps and getattr(model, "captures_prompts", False)
+            if (self.prefill_tile_rows or self.captures_prompts) and _cfg(config, "prefill_graphs", default=True):
                 self.capture_prefill_graphs()
 
     # ------------------------------------------------------------------ KV pool
@@ -411,7 +414,7 @@ class ModelRunner:
         self.prefill_host = torch.zeros(total, dtype=torch.uint8).pin_memory()
         self.prefill_out = torch.zeros(tmax, self.model_config.d_model, dtype=self.dtype, device=dev)
         plan_entries = ops.lib.b200_prefill_plan_bytes(tmax, self.max_num_seqs, self.prefill_tile_rows) // 4
-        self.prefill_plan_buffer = torch.zeros(plan_entries, dtype=torch.int32, device=dev)
+        self.prefill_plan_buffer = torch.zeros(max(plan_entries, 1), dtype=torch.int32, device=dev)
         pool = self.graphs[max(self.graphs)].pool() if self.graphs else None
         for tokens in reversed(buckets):
             v = {name: self.prefill_dev[off:off + int(np.prod(shape)) * dt.itemsize].view(dt).view(*shape)
@@ -428,6 +431,9 @@ class ModelRunner:
                                         buffer=self.prefill_plan_buffer)
                 set_context(True, v["cu_seqlens_q"], v.get("cu_seqlens_k", v["cu_seqlens_q"]), tokens, tokens,
                             v["slot_mapping"], None, v.get("block_tables"), v["positions"], plan, v.get("state_slots"))
+                if self.captures_prompts:
+                    get_context().portions = Portions(tokens, v["cu_seqlens_q"], v["cu_seqlens_k"], tokens, tokens, tokens, False,
+                                                      v["block_tables"], v["state_slots"], captured=True)
                 self.prefill_out[:tokens] = self.model(v["input_ids"])
 
             body()                                   # warm-up: allocates workspaces, selects GEMM algorithms
@@ -445,13 +451,18 @@ class ModelRunner:
     def _replay_prefill(self, seqs: list[Sequence]):
         """Prefill step from a captured graph: the hidden states of the padded batch (the context is left set for
         the head), or None when the batch does not fit one (for models without mixed batches a cached
-        prefix, which needs block tables; more tokens / sequences / blocks than were captured)."""
+        prefix, which needs block tables; for models with steps in two parts single tokens or a prefix; more tokens /
+        sequences / blocks than were captured)."""
         n = len(seqs)
         if n > self.max_num_seqs:
             return None
         m = md.prepare_prefill(seqs, self.block_size, tables_always=self.mixed_batches)
         if m.block_tables is not None and not self.mixed_batches:
             return None
+        if self.splits_steps:
+            parts = m.step_parts()
+            if parts.num_single or parts.has_prefix:
+                return None
         T = len(m.input_ids)
         if len(m.slot_mapping) != T:
             raise RuntimeError("slot_mapping and input_ids disagree: Sequence.reference_exact must be off "

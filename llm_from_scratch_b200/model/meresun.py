@@ -171,6 +171,8 @@ class MeresunLM(TokenHead, nn.Module):
         self.runs = [(self.layers[i], RunCache(self.layers[i].sublayers.mixer), again) for i, again in cfg.layer_runs()]
         self.final_norm = p.f32("final.norm", (cfg.d_model,))
         self.w_head, self.b_head = p.lin("head", (cfg.vocab_size, cfg.d_model)), None
+        # steps of whole prompts can be captured: every layer's attention then takes its grid from a tile list
+        self.captures_prompts = all(layer.sublayers.mixer.tile_rows(dtype) for layer in self.layers)
         self.attention_windows = sorted({c.window for c in cfg.layers if c.window})
 
     def cache_owners(self):

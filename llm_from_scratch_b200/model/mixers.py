@@ -206,7 +206,9 @@ def _step_output(x: torch.Tensor, width: int, ctx) -> torch.Tensor:
     """Output rows [T, width] of a step for kernels that write the rows of its sequences; padding rows are zero, so that
     what a later tile loads next to a sequence's last row is finite."""
     out = torch.empty(x.shape[0], width, dtype=x.dtype, device=x.device)
-    if ctx.portions is not None and ctx.portions.num_tokens < x.shape[0]:
+    if ctx.portions is not None and ctx.portions.captured:
+        out.zero_()
+    elif ctx.portions is not None and ctx.portions.num_tokens < x.shape[0]:
         out[ctx.portions.num_tokens:].zero_()
     elif ctx.portions is None and ctx.singles.rows < x.shape[0]:
         out[ctx.singles.rows:].zero_()
@@ -418,6 +420,10 @@ class RotaryLatentAttention(nn.Module):
     def cache_needs(self):
         return [("paged", "latent_cache", (self.rank + self.rot_dim,))]
 
+    def tile_rows(self, dtype) -> int:
+        """Query rows per tile of the kernel that serves this layer's portions; 0: a general one without tile lists."""
+        return ops.prefill_window_tile_rows(self.heads, self.heads, self.dim + self.rot_dim, self.rot_dim, self.vdim, dtype)
+
     def _absorbed(self, q, q_rot, cache, s, o):
         n, H = s.rows, self.heads
         q_abs = torch.empty(n, H, self.rank, dtype=q.dtype, device=q.device)
@@ -433,7 +439,7 @@ class RotaryLatentAttention(nn.Module):
             rows = ops.gather_rows(cache, s.block_tables, cu_k, keys.max_seqlen_k, keys.total_k, s.cu_seqlens_k)
         k, v = self.expand(rows[:, :self.rank])
         k_tail = rows[:, self.rank:] if self.rot_dim else None
-        plan = s.plan(ops.prefill_window_tile_rows(H, H, self.dim + self.rot_dim, self.rot_dim, self.vdim, q.dtype))
+        plan = s.plan(self.tile_rows(q.dtype))
         ops.prefill_varlen_window(q, _heads(k, H, self.dim), k_tail, _heads(v, H, self.vdim), s.cu_seqlens_q, cu_k, s.max_seqlen_q,
                                   self.scale, self.window, self.sink, out=o.view(-1, H, self.vdim), plan=plan)
 

@@ -51,7 +51,8 @@ class KeyRange:
 @dataclass
 class Portions:
     """The other sequences of a mixed step: prompts and portions of prompts, ragged, behind the singles' rows."""
-    num_tokens: int                               # rows of the step that belong to a sequence, singles included
+    num_tokens: int                               # rows of the step that belong to a sequence, singles included (a bound
+                                                  # in captured steps)
     cu_seqlens_q: torch.Tensor                    # int32 [n + 1], rows of the step
     cu_seqlens_k: torch.Tensor                    # int32 [n + 1], starts at 0
     max_seqlen_q: int
@@ -60,6 +61,7 @@ class Portions:
     has_prefix: bool                              # some context is longer than its portion
     block_tables: torch.Tensor                    # int32 [n, max_blocks]
     state_slots: Optional[torch.Tensor]           # int64 [n]
+    captured: bool = False                        # part of a CUDA graph: lengths differ from replay to replay
     ranges: dict = field(default_factory=dict)    # window -> KeyRange, for the windows the model's layers have
     plans: dict = field(default_factory=dict)     # tile lists by rows per tile, built when a layer asks
 

@@ -215,6 +215,26 @@ def test_greedy_generation_through_the_scheduler(kw, dtype, slack):
     eng.exit()
 
 
+@pytest.mark.parametrize("dtype,slack", [(torch.float32, 3e-4), (torch.bfloat16, 0.15)])
+def test_captured_steps_of_whole_prompts(dtype, slack):
+    """Steps of new prompts replay a graph in bf16 (padded batches of unlike lengths, windows, experts); steps with single
+    tokens or with the rest of a prompt do not.  The general fp32 kernels are never captured."""
+    from llm_from_scratch_b200.engine import SamplingParams
+    cfg = fx.config()
+    w = fx.weights(cfg, 7)
+    prompts = [fx.tokens(cfg, n, 90 + n) for n in (40, 3, 77, 130, 2, 33, 50, 200)]
+    eng = make_engine(cfg, w, dtype, max_tokens=2048, max_num_batched_tokens=256, prefill_graphs=True)
+    runner, replayed = eng.model_runner, []
+    original = runner._replay_prefill
+    runner._replay_prefill = lambda seqs: (lambda h: (replayed.append(h is not None), h)[1])(original(seqs))
+    out = eng.generate(prompts, SamplingParams(temperature=0.0, max_tokens=13, ignore_eos=True))["token_ids"]
+    agree(orc, out, cfg, w, prompts, slack)
+    assert bool(runner.prefill_graphs) == (dtype == torch.bfloat16)
+    if dtype == torch.bfloat16:
+        assert True in replayed and False in replayed
+    eng.exit()
+
+
 def test_sampling_with_temperature_and_an_end_token():
     from llm_from_scratch_b200.engine import SamplingParams
     cfg = fx.config()
