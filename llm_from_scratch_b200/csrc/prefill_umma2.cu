@@ -309,10 +309,20 @@ prefill_umma2_kernel(const Args2 a, const __grid_constant__ CUtensorMap tm_q, co
       umma::tmem_ld32(tSx, ra);
       umma::tmem_ld32_issue(tSx + 32, rb);
       float mx0 = -INFINITY, mx1 = -INFINITY;
+      uint64_t seen = 0;                                      // WINDOW: bit e set: the row sees key n0 + e
       if (warp_masked) {
+        if constexpr (WINDOW) {
+          const int hi = lim - n0, lo = low - n0;
+          seen = (hi >= 63 ? ~0ull : hi < 0 ? 0ull : (2ull << hi) - 1ull) & (lo <= 0 ? ~0ull : lo > 63 ? 0ull : ~0ull << lo);
+          const uint32_t m = static_cast<uint32_t>(seen);
 #pragma unroll
-        for (int e = 0; e < 32; ++e)
-          if (n0 + e > lim || (WINDOW && n0 + e < low)) ra[e] = 0xff800000u;            // -inf
+          for (int e = 0; e < 32; ++e)
+            if (!(m & (1u << e))) ra[e] = 0xff800000u;        // -inf
+        } else {
+#pragma unroll
+          for (int e = 0; e < 32; ++e)
+            if (n0 + e > lim) ra[e] = 0xff800000u;            // -inf
+        }
       }
 #pragma unroll
       for (int e = 0; e < 32; e += 2) {
@@ -321,9 +331,10 @@ prefill_umma2_kernel(const Args2 a, const __grid_constant__ CUtensorMap tm_q, co
       }
       umma::tmem_ld32_wait(rb);
       if (warp_masked) {
+        const uint32_t m = static_cast<uint32_t>(seen >> 32);
 #pragma unroll
         for (int e = 0; e < 32; ++e)
-          if (n0 + 32 + e > lim || (WINDOW && n0 + 32 + e < low)) rb[e] = 0xff800000u;
+          if (WINDOW ? !(m & (1u << e)) : n0 + 32 + e > lim) rb[e] = 0xff800000u;
       }
 #pragma unroll
       for (int e = 0; e < 32; e += 2) {

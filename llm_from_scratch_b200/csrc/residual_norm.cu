@@ -5,7 +5,8 @@
 //   h  = x, rounded to the activation dtype       what the next sublayer reads, or with a norm
 //   h  = x / sqrt(mean(x^2) + eps) * norm_w       mean over the row, or over each of `groups` equal parts of it
 //
-// One CTA per token row; with the row in registers every load precedes the first reduction.
+// One CTA per token row; the row stays in registers, and its loads precede the first reduction.  Weights are read where they
+// are used: every CTA of an SM reads the same ones, and without them two CTAs of the widest rows fit an SM.
 #include "common.cuh"
 
 namespace b200 {
@@ -69,14 +70,14 @@ enum Parts { kWhole, kWarps, kAny };
 // N groups of four channels per thread, d a multiple of four.  PARTS: the final norm is one part, or a.groups parts of which
 // each is whole warps wide (a multiple of 128 channels: one barrier) or any multiple of four channels wide
 template <typename T, int N, Parts PARTS>
-__global__ void __launch_bounds__(1024) residual_norm_kernel(const ResArgs a) {
+__global__ void __launch_bounds__(1024, N == 1 ? 2 : 1) residual_norm_kernel(const ResArgs a) {
   __shared__ float scratch[2][32];
   __shared__ float part[PARTS == kAny ? 1024 * N : 32 * N], part_inv[PARTS == kAny ? kMaxParts : 1];
   const int d = a.d, step = blockDim.x * 4, first = threadIdx.x * 4;
   const int64_t row = blockIdx.x;
   float* xr = a.x + row * d;
   T* hr = static_cast<T*>(a.h) + row * d;
-  float4 x[N], y[N], w[N], fw[N];
+  float4 x[N], y[N];
   const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
   const T* er = a.embed ? static_cast<const T*>(a.embed) + embed_row(a, row) * d : nullptr;
   const T* yr = static_cast<const T*>(a.y) + row * d;
@@ -86,8 +87,6 @@ __global__ void __launch_bounds__(1024) residual_norm_kernel(const ResArgs a) {
     const bool in = c < d;
     x[i] = in && !a.start ? *reinterpret_cast<const float4*>(xr + c) : zero;
     y[i] = in && a.y ? load4<T>(yr + c) : zero;
-    w[i] = in && a.y ? *reinterpret_cast<const float4*>(a.w + c) : zero;
-    fw[i] = in && a.final_w ? *reinterpret_cast<const float4*>(a.final_w + c) : zero;
   }
   if (a.embed != nullptr) {
 #pragma unroll
@@ -107,10 +106,12 @@ __global__ void __launch_bounds__(1024) residual_norm_kernel(const ResArgs a) {
     const float inv = rsqrtf(cta_sum(ss, scratch[0]) / static_cast<float>(d) + a.eps);
 #pragma unroll
     for (int i = 0; i < N; ++i) {
-      x[i].x += y[i].x * inv * w[i].x;
-      x[i].y += y[i].y * inv * w[i].y;
-      x[i].z += y[i].z * inv * w[i].z;
-      x[i].w += y[i].w * inv * w[i].w;
+      const int c = first + i * step;
+      const float4 w = c < d ? *reinterpret_cast<const float4*>(a.w + c) : zero;
+      x[i].x += y[i].x * inv * w.x;
+      x[i].y += y[i].y * inv * w.y;
+      x[i].z += y[i].z * inv * w.z;
+      x[i].w += y[i].w * inv * w.w;
     }
   }
 #pragma unroll
@@ -161,9 +162,11 @@ __global__ void __launch_bounds__(1024) residual_norm_kernel(const ResArgs a) {
       for (int i = 1; i < N; ++i) inv[i] = inv[0];
     }
 #pragma unroll
-    for (int i = 0; i < N; ++i)
-      x[i] = make_float4(x[i].x * inv[i] * fw[i].x, x[i].y * inv[i] * fw[i].y, x[i].z * inv[i] * fw[i].z,
-                         x[i].w * inv[i] * fw[i].w);
+    for (int i = 0; i < N; ++i) {
+      const int c = first + i * step;
+      const float4 w = c < d ? *reinterpret_cast<const float4*>(a.final_w + c) : zero;
+      x[i] = make_float4(x[i].x * inv[i] * w.x, x[i].y * inv[i] * w.y, x[i].z * inv[i] * w.z, x[i].w * inv[i] * w.w);
+    }
   }
 #pragma unroll
   for (int i = 0; i < N; ++i) {
