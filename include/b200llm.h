@@ -685,7 +685,8 @@ int b200_rotate_heads(void* q, int64_t num_tokens, int32_t num_heads, int32_t he
                       void* stream);
 
 /* b200_gather_rows for the ends of contexts: sequence s is cu_seqlens_full[s + 1] - cu_seqlens_full[s] tokens long and its last
- * cu_seqlens_k[s + 1] - cu_seqlens_k[s] rows are packed (cu_seqlens_full NULL: whole contexts). */
+ * cu_seqlens_k[s + 1] - cu_seqlens_k[s] rows are packed (cu_seqlens_full NULL: whole contexts).  Rows of out (out_rows of them)
+ * behind the last packed one become zero. */
 int b200_gather_last_rows(const void* cache, int32_t block_size, int64_t num_blocks, int64_t row_bytes,
                           const int32_t* block_tables, int64_t bt_stride, const int32_t* cu_seqlens_k,
                           const int32_t* cu_seqlens_full, int32_t num_seqs, int32_t max_seqlen_k, void* out, int64_t out_rows,

@@ -268,13 +268,19 @@ struct GaArgs {
   void* out;                 // [rows, W]
   int64_t rows;
   int W;                     // row width in units
+  int n;                     // sequences
   int32_t* status;
 };
 
-// rows of sequence blockIdx.y, a warp per row; U is the copy unit
+// rows of sequence blockIdx.y, a warp per row; U is the copy unit.  blockIdx.y == n: zeros behind the last row
 template <typename U>
 __global__ void __launch_bounds__(kWarps * 32) gather_rows_kernel(const GaArgs a) {
   const int s = blockIdx.y, lane = threadIdx.x & 31;
+  if (s == a.n) {
+    for (int64_t j = a.cu_k[s] - a.cu_k[0] + blockIdx.x * kWarps + (threadIdx.x >> 5); j < a.rows; j += gridDim.x * kWarps)
+      for (int c = lane; c < a.W; c += 32) static_cast<U*>(a.out)[j * a.W + c] = U{};
+    return;
+  }
   const int k0 = a.cu_k[s], len = a.cu_k[s + 1] - k0;
   const int64_t base = k0 - a.cu_k[0];
   const int skip = a.cu_full ? max(a.cu_full[s + 1] - a.cu_full[s] - len, 0) : 0;
@@ -359,10 +365,10 @@ extern "C" int b200_gather_last_rows(const void* cache, int32_t block_size, int6
     return B200_ERR_ARG;
   if (num_seqs == 0 || max_seqlen_k == 0) return B200_OK;
   if (!cache || !block_tables || !cu_seqlens_k || !out) return B200_ERR_ARG;
-  if (num_seqs > 65535 || row_bytes % 2) return B200_ERR_UNSUPPORTED;
-  GaArgs a{cache, block_tables, bt_stride, block_size, num_blocks, cu_seqlens_k, cu_seqlens_full, out, out_rows, 0, status};
+  if (num_seqs >= 65535 || row_bytes % 2) return B200_ERR_UNSUPPORTED;
+  GaArgs a{cache, block_tables, bt_stride, block_size, num_blocks, cu_seqlens_k, cu_seqlens_full, out, out_rows, 0, num_seqs, status};
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  const dim3 grid((max_seqlen_k + 4 * kWarps - 1) / (4 * kWarps), num_seqs);
+  const dim3 grid((max_seqlen_k + 4 * kWarps - 1) / (4 * kWarps), num_seqs + 1);
   if (row_bytes % 16 == 0 && aligned16(cache) && aligned16(out)) {
     a.W = static_cast<int>(row_bytes / 16);
     gather_rows_kernel<uint4><<<grid, kWarps * 32, 0, s>>>(a);

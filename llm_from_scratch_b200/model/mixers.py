@@ -424,19 +424,27 @@ class RotaryLatentAttention(nn.Module):
         """Query rows per tile of the kernel that serves this layer's portions; 0: a general one without tile lists."""
         return ops.prefill_window_tile_rows(self.heads, self.heads, self.dim + self.rot_dim, self.rot_dim, self.vdim, dtype)
 
-    def _absorbed(self, q, q_rot, cache, s, o):
-        n, H = s.rows, self.heads
-        q_abs = torch.empty(n, H, self.rank, dtype=q.dtype, device=q.device)
-        torch.bmm(q[:n, :, :self.dim].transpose(0, 1), self.w_uk, out=q_abs.transpose(0, 1))
-        lat = ops.mla_decode(q_abs, q_rot, cache, s.block_tables, s.context_lens, self.scale, window=self.window, sink=self.sink)
-        torch.bmm(lat.transpose(0, 1), self.w_uv_t, out=o[:n].view(n, H, self.vdim).transpose(0, 1))
+    row_multiple = 8      # single tokens of mixed steps: the batched products meet few distinct sizes (cf. prefill_token_multiple)
+    key_multiple = 256    # the same for the rows of contexts that are expanded
+
+    def _absorbed(self, q, q_rot, cache, ctx, o):
+        s, H = ctx.singles, self.heads
+        n = m = s.rows
+        if ctx.portions is not None and -(-n // self.row_multiple) * self.row_multiple <= ctx.portions.num_tokens:
+            m = -(-n // self.row_multiple) * self.row_multiple     # rows n .. m - 1 are of portions, which write them later
+        q_abs, lat = (torch.empty(m, H, self.rank, dtype=q.dtype, device=q.device) for _ in range(2))
+        torch.bmm(q[:m, :, :self.dim].transpose(0, 1), self.w_uk, out=q_abs.transpose(0, 1))
+        ops.mla_decode(q_abs[:n], q_rot, cache, s.block_tables, s.context_lens, self.scale, out=lat[:n], window=self.window,
+                       sink=self.sink)
+        torch.bmm(lat.transpose(0, 1), self.w_uv_t, out=o[:m].view(m, H, self.vdim).transpose(0, 1))
 
     def _expanded(self, q, rows, cache, s, o):
         H, keys = self.heads, s.keys(self.window)
         cu_k = s.cu_seqlens_q
         if keys.has_prefix:
             cu_k = keys.cu_seqlens_k
-            rows = ops.gather_rows(cache, s.block_tables, cu_k, keys.max_seqlen_k, keys.total_k, s.cu_seqlens_k)
+            rows = ops.gather_rows(cache, s.block_tables, cu_k, keys.max_seqlen_k, keys.total_k, s.cu_seqlens_k,
+                                   self.key_multiple)
         k, v = self.expand(rows[:, :self.rank])
         k_tail = rows[:, self.rank:] if self.rot_dim else None
         plan = s.plan(self.tile_rows(q.dtype))
@@ -451,7 +459,7 @@ class RotaryLatentAttention(nn.Module):
         q_rot = ops.rotate_heads(q, self.rot_dim, self.rotation, positions, singles) if self.rot_dim else None
         o = _step_output(rows, self.heads * self.vdim, ctx)
         if ctx.singles is not None:
-            self._absorbed(q, q_rot, pools.latent_cache, ctx.singles, o)
+            self._absorbed(q, q_rot, pools.latent_cache, ctx, o)
         if ctx.portions is not None:
             self._expanded(q, rows, pools.latent_cache, ctx.portions, o)
         return F.linear(o, self.w_o)

@@ -47,7 +47,8 @@ def _cuda(*ts: torch.Tensor | None) -> torch.device:
 
 
 def _stream() -> int:
-    return torch.cuda.current_stream().cuda_stream
+    """The current stream's handle, without building a stream object (an eager step asks for it once per launch)."""
+    return torch._C._cuda_getCurrentRawStream(torch._C._cuda_getDevice())
 
 
 def status_word(device: torch.device) -> torch.Tensor:
@@ -1040,15 +1041,17 @@ def latent_norm_store(rows: torch.Tensor, norm_w: torch.Tensor, eps: float, cach
 
 
 def gather_rows(cache: torch.Tensor, block_tables: torch.Tensor, cu_seqlens_k: torch.Tensor, max_seqlen_k: int,
-                total: int, cu_seqlens_full: torch.Tensor | None = None) -> torch.Tensor:
+                total: int, cu_seqlens_full: torch.Tensor | None = None, multiple: int = 1) -> torch.Tensor:
     """Rows of whole contexts, packed [total, W], from a pool [num_blocks, block_size, W] through the block tables.  With
-    ``cu_seqlens_full`` (the contexts' own offsets) ``cu_seqlens_k`` counts the last rows of every context."""
+    ``cu_seqlens_full`` (the contexts' own offsets) ``cu_seqlens_k`` counts the last rows of every context.  ``multiple``:
+    the result is padded with zero rows to a multiple of this many."""
     dev = _cuda(cache, block_tables, cu_seqlens_k, cu_seqlens_full)
     nb, bs, W = cache.shape
     n = cu_seqlens_k.numel() - 1
     if not cache.is_contiguous() or block_tables.dtype != torch.int32 or block_tables.shape[0] < n \
             or block_tables.stride(1) != 1 or cu_seqlens_k.dtype != torch.int32:
         raise ValueError("cache must be contiguous, block_tables int32 [n, max_blocks], cu_seqlens_k int32 [n + 1]")
+    total = -(-total // multiple) * multiple
     out = torch.empty(total, W, dtype=cache.dtype, device=cache.device)
     if cu_seqlens_full is not None and (cu_seqlens_full.dtype != torch.int32 or cu_seqlens_full.numel() != n + 1):
         raise ValueError("cu_seqlens_full must be int32 [n + 1]")

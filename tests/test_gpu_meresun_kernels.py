@@ -180,6 +180,9 @@ def test_gather_the_ends_of_contexts(W):
     got = ops.gather_rows(pool.cuda(), bt.cuda(), cu(ends).cuda(), max(ends), sum(ends), cu(lens).cuda())
     ops.check_status()
     assert torch.equal(got.cpu(), want)
+    torch.full((192, W), float("nan"), device="cuda")                  # what freed memory may hold
+    got = ops.gather_rows(pool.cuda(), bt.cuda(), cu(ends).cuda(), max(ends), sum(ends), cu(lens).cuda(), 64).cpu()
+    assert got.shape == (128, W) and torch.equal(got[:sum(ends)], want) and not got[sum(ends):].any()
 
 
 # ------------------------------------------------------------------------------------- windowed attention
