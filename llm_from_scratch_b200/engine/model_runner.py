@@ -226,8 +226,8 @@ class ModelRunner:
             ctx.portions = Portions(num_tokens, ctx.cu_seqlens_q[n1:], t["portion_cu_k"], parts.max_seqlen_q,
                                     parts.max_seqlen_k, int(parts.portion_cu_k[-1]), parts.has_prefix,
                                     ctx.block_tables[n1:], part(slots, n1),
-                                    {w: KeyRange(t[f"portion_cu_k.{w}"], r.max_seqlen_k, int(r.cu_k[-1]), r.has_prefix)
-                                     for w, r in parts.ranges.items()})
+                                    ranges={w: KeyRange(t[f"portion_cu_k.{w}"], r.max_seqlen_k, int(r.cu_k[-1]), r.has_prefix)
+                                            for w, r in parts.ranges.items()})
 
     def prepare_prefill(self, seqs: list[Sequence]) -> torch.Tensor:
         return self._publish(md.prepare_prefill(seqs, self.block_size, tables_always=self.mixed_batches))

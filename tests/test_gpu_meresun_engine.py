@@ -61,6 +61,19 @@ def test_whole_prompts_portions_and_single_tokens_give_the_same_logits(dtype):
     eng.exit()
 
 
+def test_portions_gather_only_what_their_windows_reach(monkeypatch):
+    from llm_from_scratch_b200 import ops
+    cfg = fx.config([fx.layer(fx.dense(), window=20), fx.layer(fx.dense(), window=0), fx.layer(fx.dense(), window=90)], loop=None)
+    w, ids = fx.weights(cfg, 1), fx.tokens(cfg, 120, 3)
+    want, totals = reference(cfg, w, ids, torch.float32), []
+    plain = ops.gather_rows
+    monkeypatch.setattr(ops, "gather_rows", lambda *a, **k: (totals.append(a[4]), plain(*a, **k))[1])
+    eng = make_engine(cfg, w, torch.float32)
+    assert error(run(eng, portions(ids, [60, 10, 50]))["a"], want) < TOL[torch.float32]
+    assert totals == [29, 70, 70, 69, 120, 120]
+    eng.exit()
+
+
 VARIANTS = {
     "ones": fx.config([fx.layer(fx.moe(ff=8, experts=1, top=1, groups=(1, 1)), heads=1, dim=8, rot_dim=8, vdim=8, q_rank=8, kv_rank=8,
                                 window=1)], vocab=17, width=24, groups=1, side=5, loop=None),
