@@ -38,7 +38,7 @@
 extern "C" {
 #endif
 
-#define B200_ABI_VERSION 12
+#define B200_ABI_VERSION 13
 
 #define B200_DTYPE_F32 0
 #define B200_DTYPE_BF16 1
@@ -726,12 +726,82 @@ int b200_moe_group_route(const float* logits, const float* correction, int32_t n
                          int32_t groups, int32_t keep, int32_t* sorted_token, float* weight, int32_t* expert_offsets,
                          int32_t* slot_to_row, void* workspace, size_t workspace_bytes, void* stream);
 
-/* b200_moe_grouped_gemm without biases, for any size and also fp32 (general kernel).  glu: w [experts, 2 n_out, k_dim] =
- * [gate | up] and out = g sigmoid(slope g) (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit).
+/* b200_moe_grouped_gemm without biases, for any size and also fp32 (general kernel).  act: what follows the linear map —
+ * nothing; the clamped GLU: w [experts, 2 n_out, k_dim] = [gate | up] and out = g sigmoid(slope g) (u + 1) with g =
+ * min(gate, limit), u = clamp(up, -limit, limit); the squared ReLU max(., 0)^2 (of the fp32 sums).  limit and slope count for
+ * the GLU only.
  * flags: 0 or B200_MOE_GEMM_EARLY_LAUNCH. */
+#define B200_EXPERT_LINEAR 0
+#define B200_EXPERT_CLAMPED_GLU 1
+#define B200_EXPERT_SQUARED_RELU 2
 int b200_moe_grouped_linear(const void* x, const void* w, void* out, const int32_t* expert_offsets, int64_t num_rows,
-                            int32_t num_experts, int32_t n_out, int32_t k_dim, int32_t glu, float limit, float slope,
+                            int32_t num_experts, int32_t n_out, int32_t k_dim, int32_t act, float limit, float slope,
                             int32_t flags, int32_t dtype, int32_t* status, void* stream);
+
+/* ---------------------------------------------------------------------------------------------
+ * Mechanisms of decoders with token shift, short convolutions in front of attention, sigmoid attention inside chunks and a
+ * softmax over the chosen experts (the Sodonex family; the reference has no counterpart).  All constants are parameters.
+ *
+ * State slots: with cu_seqlens_q / cu_seqlens_k (int32 [num_seqs + 1]) a step holds ragged portions, the last tokens of contexts
+ * of cu_seqlens_k lengths, and rows behind the last sequence are padding; with cu_seqlens_q NULL row i is sequence i with
+ * context_lens[i] tokens (0: padding).  state_slots int64 [num_seqs], -1: no state.  A sequence at position 0 ignores what its
+ * slot holds; every call moves the state on.
+ * ------------------------------------------------------------------------------------------- */
+
+/* One boundary between sublayers: x' = x + gain y / sqrt(mean(y^2) + eps), or embed_scale embed[tokens] where embed is given
+ * (y NULL: x' = x).  top > 0: y holds expert rows [rows * top, d] and row t takes sum_k row_weight[t, k] y[slot_to_row[t, k]].
+ * x' goes to x_out (NULL: nowhere; x_out == x is allowed without shift), and h [rows, d] in dtype is one of
+ *   x' + (before - x') shift    shift fp32 [d]; before = the previous token's x', from state [num_slots, d] at a portion's start
+ *   final_gain x' / sqrt(mean(x'^2) + eps)    final_norm
+ *   x'                                        otherwise */
+int b200_shift_residual(const float* x, float* x_out, const int64_t* tokens, const void* embed, int64_t vocab, float embed_scale,
+                        const void* y, const float* row_weight, const int32_t* slot_to_row, int32_t top, float gain,
+                        const float* shift, float* state, int64_t num_slots, const int64_t* state_slots,
+                        const int32_t* cu_seqlens_q, const int32_t* cu_seqlens_k, const int64_t* context_lens, int32_t num_seqs,
+                        int32_t final_norm, float final_gain, float eps, void* h, int64_t rows, int32_t d, int32_t dtype,
+                        int32_t* status, void* stream);
+
+/* Attention prologue: causal convolution of `taps` taps on every channel of q [T, Hq * D] and k [T, Hkv * D] (one token stride;
+ * weights [taps, channels], the last row weighs the current token), v = the convolved k, RMS norm of the whole convolved q and of
+ * the whole convolved k, rotation of the first rot_dims channels of every head (channel i with i + rot_dims / 2, by positions[t] *
+ * freq[i], freq fp64).  q_out [T, Hq, D]; k_out, v_out [T, Hkv, D] (NULL: not wanted); k and v also go to the pools at
+ * slot_mapping[t] (negative: not stored).  ring [num_slots, taps - 1, (Hq + Hkv) * D] keeps the last inputs of every sequence. */
+int b200_conv_norm_rope_store(const void* q, const void* k, int64_t token_stride, const float* conv_q, const float* conv_k,
+                              int32_t taps, float* ring, int64_t num_slots, const int64_t* state_slots,
+                              const int32_t* cu_seqlens_q, const int32_t* cu_seqlens_k, const int64_t* context_lens,
+                              int32_t num_seqs, const float* q_norm_w, const float* k_norm_w, float eps, const double* freq,
+                              int32_t rot_dims, const int64_t* positions, void* q_out, void* k_out, void* v_out, void* k_cache,
+                              void* v_cache, const int64_t* slot_mapping, int64_t pool_slots, int64_t num_tokens,
+                              int32_t num_q_heads, int32_t num_kv_heads, int32_t head_dim, int32_t dtype, int32_t* status,
+                              void* stream);
+
+/* Packed ragged causal attention with weights sigmoid(scale q.k + bias[head]) that are summed as they are.  Query i of a sequence
+ * (at the end of its k_len keys) has index n = k_len - q_len + i and sees the keys j <= n with j / chunk = n / chunk (chunk 0:
+ * all): packed contexts start at a multiple of the chunk.  out[t, h] is multiplied by sigmoid(gate[t, h]) (gate NULL: not).
+ * plan: tile list for b200_sigmoid_attention_tile_rows() rows, or NULL.  bf16: tcgen05 kernel for 128/128 and 64/64, mma.sync for
+ * multiples of eight up to 192/128; else general. */
+int32_t b200_sigmoid_attention_tile_rows(int32_t num_q_heads, int32_t num_kv_heads, int32_t head_dim_qk, int32_t head_dim_v,
+                                         int32_t dtype);
+int b200_sigmoid_attention(const void* q, const void* k, const void* v, void* out, int64_t q_token_stride, int64_t k_token_stride,
+                           int64_t v_token_stride, int64_t total_q_tokens, int64_t total_k_tokens, const int32_t* cu_seqlens_q,
+                           const int32_t* cu_seqlens_k, int32_t num_seqs, int32_t max_seqlen_q, int32_t num_q_heads,
+                           int32_t num_kv_heads, int32_t head_dim_qk, int32_t head_dim_v, float scale, const float* bias,
+                           int32_t chunk, const void* gate, int64_t gate_token_stride, const int32_t* plan,
+                           int32_t plan_tile_rows, int32_t plan_capacity, int32_t dtype, int32_t* status, void* stream);
+
+/* The same for one token per sequence over the paged pools: the last token of context_lens[i] sees its own chunk.  Workspace as
+ * b200_paged_decode_gqa. */
+int b200_sigmoid_decode(const void* q, const void* k_cache, const void* v_cache, void* out, const int32_t* block_tables,
+                        int64_t bt_stride, const int64_t* context_lens, int32_t batch, int32_t num_q_heads, int32_t num_kv_heads,
+                        int32_t head_dim_qk, int32_t head_dim_v, int32_t block_size, int64_t num_blocks, float scale,
+                        const float* bias, int32_t chunk, const void* gate, int64_t gate_token_stride, void* workspace,
+                        size_t workspace_bytes, int32_t dtype, int32_t* status, void* stream);
+
+/* b200_moe_group_route without groups, on z = logits + bias: the `top` largest z are chosen (equal ones: the lower index), their
+ * weights are the softmax of z over the chosen.  Workspace as b200_moe_group_route. */
+int b200_moe_softmax_route(const float* logits, const float* bias, int32_t num_tokens, int32_t num_experts, int32_t top,
+                           int32_t* sorted_token, float* weight, int32_t* expert_offsets, int32_t* slot_to_row, void* workspace,
+                           size_t workspace_bytes, void* stream);
 
 /* ---------------------------------------------------------------------------------------------
  * Diagnostic (no counterpart in the reference, which has no device code): runs the give-up path of the

@@ -54,6 +54,9 @@ FAMILY_SOURCES = {
     "Meresun": ("api", "host_path", "decode_advance", "sampler", "moe_gemm", "moe_gemm_rows", "grouped_linear", "moe_group_route",
                 "store_kvcache", "prefill_plan", "prefill_varlen", "prefill_mma", "prefill_umma", "prefill_umma2", "prefill_umma4",
                 "paged_decode", "mla_decode", "mla_decode_mma", "residual_norm", "gated_residual", "latent_rows", "activations"),
+    "Sodonex": ("api", "host_path", "decode_advance", "sampler", "moe_gemm", "moe_gemm_rows", "grouped_linear", "moe_group_route",
+                "store_kvcache", "prefill_plan", "prefill_varlen", "prefill_mma", "prefill_umma", "prefill_umma2", "prefill_umma4",
+                "paged_decode", "latent_rows", "activations", "shift_residual", "conv_norm_rope"),
 }
 
 

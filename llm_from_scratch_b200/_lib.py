@@ -115,6 +115,16 @@ SIGNATURES = {
                           _vp, _vp, _sz, _i32, _vp, _vp]),
     "b200_moe_group_route_workspace_bytes": (_sz, [_i32, _i32, _i32]),
     "b200_moe_group_route": (_i32, [_vp, _vp, _i32, _i32, _i32, _i32, _i32, _vp, _vp, _vp, _vp, _vp, _sz, _vp]),
+    "b200_moe_softmax_route": (_i32, [_vp, _vp, _i32, _i32, _i32, _vp, _vp, _vp, _vp, _vp, _sz, _vp]),
+    "b200_shift_residual": (_i32, [_vp, _vp, _vp, _vp, _i64, _f32, _vp, _vp, _vp, _i32, _f32, _vp, _vp, _i64, _vp, _vp, _vp, _vp,
+                                   _i32, _i32, _f32, _f32, _vp, _i64, _i32, _i32, _vp, _vp]),
+    "b200_conv_norm_rope_store": (_i32, [_vp, _vp, _i64, _vp, _vp, _i32, _vp, _i64, _vp, _vp, _vp, _vp, _i32, _vp, _vp, _f32, _vp,
+                                         _i32, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i64, _i32, _i32, _i32, _i32, _vp, _vp]),
+    "b200_sigmoid_attention_tile_rows": (_i32, [_i32, _i32, _i32, _i32, _i32]),
+    "b200_sigmoid_attention": (_i32, [_vp, _vp, _vp, _vp, _i64, _i64, _i64, _i64, _i64, _vp, _vp, _i32, _i32, _i32, _i32, _i32,
+                                      _i32, _f32, _vp, _i32, _vp, _i64, _vp, _i32, _i32, _i32, _vp, _vp]),
+    "b200_sigmoid_decode": (_i32, [_vp, _vp, _vp, _vp, _vp, _i64, _vp, _i32, _i32, _i32, _i32, _i32, _i32, _i64, _f32, _vp, _i32,
+                                   _vp, _i64, _vp, _sz, _i32, _vp, _vp]),
     "b200_moe_grouped_linear": (_i32, [_vp, _vp, _vp, _vp, _i64, _i32, _i32, _i32, _i32, _f32, _f32, _i32, _i32, _vp, _vp]),
     "b200_moe_combine": (_i32, [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i32, _i32, _i32, _vp]),
     "b200_selftest_bounded_wait": (_i32, [_i32, _vp, _vp, _vp]),

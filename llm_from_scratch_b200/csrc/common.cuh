@@ -133,6 +133,11 @@ __device__ __forceinline__ float clamped_glu_bf16(float g, float u, float limit,
   return __fdividef(g * (u + 1.f), 1.f + fminf(__expf(-slope * g), 1e30f));
 }
 
+__device__ __forceinline__ float squared_relu_f(float x) {
+  x = fmaxf(x, 0.f);
+  return x * x;
+}
+
 // Prefill tile list (b200_prefill_plan): int32 header {tile count, rows per tile, capacity, 0} followed
 // by one entry per query tile, (sequence << 16) | tile index, heaviest tiles first.
 constexpr int kPlanHeader = 4;

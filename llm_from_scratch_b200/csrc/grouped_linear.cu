@@ -1,6 +1,6 @@
 // Linear maps of rows grouped by expert for every size and both dtypes (fp32 arithmetic): what the tensor-core grouped GEMMs do
 // not take.  out[r] = X[r] . W_e^T with W [E, n_out, k], or with `glu` the clamped gated unit of the two halves of
-// W [E, 2 n_out, k] = [gate | up].  Expert e owns rows [offsets[e-1], offsets[e]).
+// W [E, 2 n_out, k] = [gate | up], or max(., 0)^2 of the plain map.  Expert e owns rows [offsets[e-1], offsets[e]).
 #include "common.cuh"
 
 namespace b200 {
@@ -19,8 +19,9 @@ struct GlArgs {
 };
 
 // One CTA per 64 rows of an expert and 64 output columns; 4 x 4 results per thread
-template <typename T, bool GLU>
+template <typename T, int ACT>
 __global__ void __launch_bounds__(256) grouped_linear_kernel(const GlArgs a) {
+  constexpr bool GLU = ACT == B200_EXPERT_CLAMPED_GLU;
   constexpr int P = GLU ? 2 : 1;
   __shared__ float sx[TK][TM + 4], sw[P][TK][TN + 4];
   // the row tile: experts in order, ceil(rows / 64) tiles each
@@ -79,29 +80,30 @@ __global__ void __launch_bounds__(256) grouped_linear_kernel(const GlArgs a) {
       const int n = n0 + tx * 4 + j;
       if (n >= a.n_out) continue;
       if constexpr (GLU) o[n] = from_float<T>(clamped_glu_f(acc[0][i][j], acc[P - 1][i][j], a.limit, a.slope));
-      else o[n] = from_float<T>(acc[0][i][j]);
+      else o[n] = from_float<T>(ACT == B200_EXPERT_SQUARED_RELU ? squared_relu_f(acc[0][i][j]) : acc[0][i][j]);
     }
   }
 }
 
 template <typename T>
-void launch(const GlArgs& a, dim3 grid, bool glu, cudaStream_t s) {
-  if (glu) grouped_linear_kernel<T, true><<<grid, 256, 0, s>>>(a);
-  else grouped_linear_kernel<T, false><<<grid, 256, 0, s>>>(a);
+void launch(const GlArgs& a, dim3 grid, int act, cudaStream_t s) {
+  if (act == B200_EXPERT_CLAMPED_GLU) grouped_linear_kernel<T, B200_EXPERT_CLAMPED_GLU><<<grid, 256, 0, s>>>(a);
+  else if (act == B200_EXPERT_SQUARED_RELU) grouped_linear_kernel<T, B200_EXPERT_SQUARED_RELU><<<grid, 256, 0, s>>>(a);
+  else grouped_linear_kernel<T, B200_EXPERT_LINEAR><<<grid, 256, 0, s>>>(a);
 }
 
 }  // namespace
 
 int grouped_linear_any_launch(const void* x, const void* w, void* out, const int32_t* expert_offsets, int64_t num_rows,
-                              int num_experts, int n_out, int k_dim, bool glu, float limit, float slope, int32_t dtype,
+                              int num_experts, int n_out, int k_dim, int act, float limit, float slope, int32_t dtype,
                               cudaStream_t s) {
   const int64_t row_tiles = (num_rows + TM - 1) / TM + num_experts;      // at most this many
   const int col_tiles = (n_out + TN - 1) / TN;
   if (row_tiles > 65535) return B200_ERR_TOO_LARGE;
   GlArgs a{x, w, out, expert_offsets, num_experts, n_out, k_dim, num_rows, limit, slope};
   const dim3 grid(col_tiles, static_cast<unsigned>(row_tiles));
-  if (dtype == B200_DTYPE_F32) launch<float>(a, grid, glu, s);
-  else launch<__nv_bfloat16>(a, grid, glu, s);
+  if (dtype == B200_DTYPE_F32) launch<float>(a, grid, act, s);
+  else launch<__nv_bfloat16>(a, grid, act, s);
   return launch_result();
 }
 

@@ -6,6 +6,7 @@
 //   mode 0:  out[r, :]  = X[r, :] . W_e^T                      W [E, n_out, K]
 //   mode 1:  act[r, :]  = silu(X[r] . W1_e^T + b1_e) * (X[r] . W3_e^T + b3_e)   W [E, 2*d_ff, K] = [w1 | w3]
 //            (the SwiGLU of mlp.py:61-67; every intermediate rounded to bf16 like the tensor ops)
+//   mode 4:  as mode 0 without a bias, act[r, :] = max(X[r, :] . W_e^T, 0)^2 of the fp32 accumulators
 //   mode 3:  as mode 1 with a clamped gated unit: g sigmoid(slope g) (u + 1), g = min(X W1^T, limit), u = clamp(X W3^T, +-limit)
 //
 // The operands are swapped with respect to the usual layout: the 128 rows of a WEIGHT tile are the M
@@ -330,14 +331,14 @@ moe_gemm_kernel(const GemmArgs a, const __grid_constant__ CUtensorMap tm_w,
               if (bp) bb.u = *reinterpret_cast<const uint4*>(bp);
 #pragma unroll
               for (int x = 0; x < 8; ++x) {
-                float y = bf16_round(v[x]);
+                float y = a.mode == 4 ? squared_relu_f(v[x]) : bf16_round(v[x]);
                 if (bp) y += __bfloat162float(bb.b[x]);
                 o.b[x] = __float2bfloat16(y);
               }
               *reinterpret_cast<uint4*>(dst) = o.u;
             } else {
               for (int x = 0; x < 8 && f + x < a.n_out; ++x) {
-                float y = bf16_round(v[x]);
+                float y = a.mode == 4 ? squared_relu_f(v[x]) : bf16_round(v[x]);
                 if (bp) y += __bfloat162float(bp[x]);
                 dst[x] = __float2bfloat16(y);
               }
@@ -488,7 +489,7 @@ int moe_gemm_rows_launch(const void* x, const void* w, const void* bias, void* o
                          int64_t num_rows, int num_experts, int dense_rows, int n_out, int k_dim, int mode, float limit,
                          float slope, int32_t* status, cudaStream_t s);
 int grouped_linear_any_launch(const void* x, const void* w, void* out, const int32_t* expert_offsets, int64_t num_rows,
-                              int num_experts, int n_out, int k_dim, bool glu, float limit, float slope, int32_t dtype,
+                              int num_experts, int n_out, int k_dim, int act, float limit, float slope, int32_t dtype,
                               cudaStream_t s);
 
 namespace {
@@ -553,17 +554,20 @@ extern "C" int b200_moe_grouped_gemm(const void* x, const void* w, const void* b
 }
 
 extern "C" int b200_moe_grouped_linear(const void* x, const void* w, void* out, const int32_t* expert_offsets, int64_t num_rows,
-                                       int32_t num_experts, int32_t n_out, int32_t k_dim, int32_t glu, float limit, float slope,
+                                       int32_t num_experts, int32_t n_out, int32_t k_dim, int32_t act, float limit, float slope,
                                        int32_t flags, int32_t dtype, int32_t* status, void* stream) {
   using namespace b200;
-  if (num_rows < 0 || num_experts <= 0 || n_out <= 0 || k_dim <= 0 || (flags & ~B200_MOE_GEMM_EARLY_LAUNCH)) return B200_ERR_ARG;
+  if (num_rows < 0 || num_experts <= 0 || n_out <= 0 || k_dim <= 0 || act < B200_EXPERT_LINEAR ||
+      act > B200_EXPERT_SQUARED_RELU || (flags & ~B200_MOE_GEMM_EARLY_LAUNCH))
+    return B200_ERR_ARG;
   if (dtype != B200_DTYPE_F32 && dtype != B200_DTYPE_BF16) return B200_ERR_UNSUPPORTED;
   if (num_rows == 0) return B200_OK;
   if (!x || !w || !out || !expert_offsets) return B200_ERR_ARG;
   if (dtype == B200_DTYPE_BF16 && k_dim % 8 == 0 && n_out % 8 == 0 && aligned16(x) && aligned16(w) && aligned16(out))
-    return grouped_gemm(x, w, nullptr, out, expert_offsets, num_rows, num_experts, 0, n_out, k_dim, glu ? 3 : 0,
+    return grouped_gemm(x, w, nullptr, out, expert_offsets, num_rows, num_experts, 0, n_out, k_dim,
+                        act == B200_EXPERT_CLAMPED_GLU ? 3 : act == B200_EXPERT_SQUARED_RELU ? 4 : 0,
                         (flags & B200_MOE_GEMM_EARLY_LAUNCH) != 0, limit, slope, status, stream);
-  return grouped_linear_any_launch(x, w, out, expert_offsets, num_rows, num_experts, n_out, k_dim, glu != 0, limit, slope, dtype,
+  return grouped_linear_any_launch(x, w, out, expert_offsets, num_rows, num_experts, n_out, k_dim, act, limit, slope, dtype,
                                    static_cast<cudaStream_t>(stream));
 }
 

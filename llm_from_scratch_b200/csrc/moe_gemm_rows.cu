@@ -287,7 +287,8 @@ moe_gemm_rows_kernel(const RowsArgs a, const __grid_constant__ CUtensorMap tm_x,
             if (bp) bb.u = __ldg(reinterpret_cast<const uint4*>(bp + c + e8));
 #pragma unroll
             for (int x = 0; x < 8; ++x) {
-              float y = bf16r(__uint_as_float(r[e8 + x]));
+              const float acc_x = __uint_as_float(r[e8 + x]);
+              float y = a.mode == 4 ? squared_relu_f(acc_x) : bf16r(acc_x);
               if (bp) y += __bfloat162float(bb.b[x]);
               o.b[x] = __float2bfloat16(y);
             }

@@ -4,9 +4,13 @@
 //   the `top` experts with the largest c inside the `keep` groups with the largest scores
 //   weight of a chosen expert = s / (sum of the chosen s + 1e-20)
 //
+// or, with SOFT, c = logits + correction and the weights are the softmax of c over the chosen experts.
+//
 // All fp32; equal scores go to the lower index.  A warp per token, the experts of a lane in registers.  Up to kSingle tokens one
 // CTA selects and sorts in the same launch; above, a first launch leaves the chosen experts and every CTA's counts, a second
 // one places the rows.  Rows of one expert are in no particular order: nothing computed from a row depends on its place.
+#include <type_traits>
+
 #include "common.cuh"
 
 namespace b200 {
@@ -30,7 +34,7 @@ struct GrArgs {
 
 // Writes the token's experts and weights, in order of choice.  EPL: experts per lane, expert e in lane e % 32; `choice`
 // [E] and `score` [kMaxGroups] are the warp's.
-template <int EPL>
+template <int EPL, bool SOFT>
 __device__ __forceinline__ void select_experts(const GrArgs& a, int t, float* choice, float* score) {
   const int lane = threadIdx.x & 31, size = a.E / a.groups;
   float s[EPL], c[EPL];
@@ -38,8 +42,9 @@ __device__ __forceinline__ void select_experts(const GrArgs& a, int t, float* ch
   for (int i = 0; i < EPL; ++i) {
     const int e = lane + 32 * i;
     const float z = e < a.E ? a.logits[static_cast<int64_t>(t) * a.E + e] : 0.f;
-    s[i] = 1.f / (1.f + expf(-z));
+    s[i] = SOFT ? z : 1.f / (1.f + expf(-z));
     c[i] = e < a.E ? s[i] + a.correction[e] : -INFINITY;
+    if (SOFT) s[i] = c[i];
   }
   if (a.groups > 1) {
 #pragma unroll
@@ -74,7 +79,7 @@ __device__ __forceinline__ void select_experts(const GrArgs& a, int t, float* ch
   }
   unsigned taken = 0;                                  // bit i: this lane's expert i is chosen
   int my_expert = 0;                                   // lane k keeps choice k
-  float my_score = 0.f, sum = 0.f;
+  float my_score = 0.f, sum = 0.f, largest = 0.f;      // SOFT: the first choice has the largest score
   for (int k = 0; k < a.K; ++k) {
     float best = -INFINITY;
     int at = kMaxExperts;
@@ -103,6 +108,10 @@ __device__ __forceinline__ void select_experts(const GrArgs& a, int t, float* ch
         sc = s[i];
       }
     sc = __shfl_sync(0xffffffffu, sc, at & 31);
+    if (SOFT) {
+      if (k == 0) largest = sc;
+      sc = expf(sc - largest);
+    }
     if (lane == k) {
       my_expert = at;
       my_score = sc;
@@ -111,7 +120,7 @@ __device__ __forceinline__ void select_experts(const GrArgs& a, int t, float* ch
   }
   if (lane < a.K) {
     a.expert[static_cast<int64_t>(t) * a.K + lane] = my_expert;
-    a.weight[static_cast<int64_t>(t) * a.K + lane] = my_score / (sum + 1e-20f);
+    a.weight[static_cast<int64_t>(t) * a.K + lane] = my_score / (SOFT ? sum : sum + 1e-20f);
   }
 }
 
@@ -146,7 +155,7 @@ __device__ __forceinline__ void place_rows(const GrArgs& a, int t0, int t1, int3
   }
 }
 
-template <int EPL, bool SINGLE>
+template <int EPL, bool SINGLE, bool SOFT>
 __global__ void __launch_bounds__((SINGLE ? kSingleWarps : kWarps) * 32) group_select_kernel(const GrArgs a) {
   constexpr int W = SINGLE ? kSingleWarps : kWarps;
   extern __shared__ float choices[];                   // [W][E] with groups
@@ -154,7 +163,7 @@ __global__ void __launch_bounds__((SINGLE ? kSingleWarps : kWarps) * 32) group_s
   __shared__ int32_t count[EPL * 32], cursor[SINGLE ? EPL * 32 : 1];
   const int warp = threadIdx.x >> 5, t0 = blockIdx.x * a.per_cta, t1 = min(t0 + a.per_cta, a.T);
   for (int e = threadIdx.x; e < EPL * 32; e += blockDim.x) count[e] = 0;
-  for (int t = t0 + warp; t < t1; t += W) select_experts<EPL>(a, t, choices + warp * a.E, scores[warp]);
+  for (int t = t0 + warp; t < t1; t += W) select_experts<EPL, SOFT>(a, t, choices + warp * a.E, scores[warp]);
   __syncthreads();                                     // the CTA's choices are written, and visible to it
   for (int i = t0 * a.K + threadIdx.x; i < t1 * a.K; i += blockDim.x) atomicAdd(&count[a.expert[i]], 1);
   __syncthreads();
@@ -184,13 +193,13 @@ __global__ void __launch_bounds__(kWarps * 32) group_place_kernel(const GrArgs a
   place_rows(a, t0, min(t0 + a.per_cta, a.T), cursor);
 }
 
-template <int EPL>
+template <int EPL, bool SOFT>
 void launch(const GrArgs& a, int ctas, bool single, cudaStream_t s) {
   const size_t per_warp = a.groups > 1 ? a.E * sizeof(float) : 0;
   if (single) {
-    group_select_kernel<EPL, true><<<1, kSingleWarps * 32, kSingleWarps * per_warp, s>>>(a);
+    group_select_kernel<EPL, true, SOFT><<<1, kSingleWarps * 32, kSingleWarps * per_warp, s>>>(a);
   } else {
-    group_select_kernel<EPL, false><<<ctas, kWarps * 32, kWarps * per_warp, s>>>(a);
+    group_select_kernel<EPL, false, SOFT><<<ctas, kWarps * 32, kWarps * per_warp, s>>>(a);
     group_place_kernel<<<ctas, kWarps * 32, 0, s>>>(a);
   }
 }
@@ -203,11 +212,11 @@ extern "C" size_t b200_moe_group_route_workspace_bytes(int32_t num_tokens, int32
   return (static_cast<size_t>(num_tokens) * top + static_cast<size_t>(b200::kMaxCtas) * num_experts) * sizeof(int32_t);
 }
 
-extern "C" int b200_moe_group_route(const float* logits, const float* correction, int32_t num_tokens, int32_t num_experts,
-                                    int32_t top, int32_t groups, int32_t keep, int32_t* sorted_token, float* weight,
-                                    int32_t* expert_offsets, int32_t* slot_to_row, void* workspace, size_t workspace_bytes,
-                                    void* stream) {
-  using namespace b200;
+namespace b200 {
+namespace {
+int route(const float* logits, const float* correction, int32_t num_tokens, int32_t num_experts, int32_t top, int32_t groups,
+          int32_t keep, bool soft, int32_t* sorted_token, float* weight, int32_t* expert_offsets, int32_t* slot_to_row,
+          void* workspace, size_t workspace_bytes, void* stream) {
   if (num_tokens < 0 || num_experts <= 0 || top <= 0 || groups <= 0 || num_experts % groups || keep <= 0 || keep > groups ||
       top > keep * (num_experts / groups))
     return B200_ERR_ARG;
@@ -226,10 +235,31 @@ extern "C" int b200_moe_group_route(const float* logits, const float* correction
     ctas = (num_tokens + a.per_cta - 1) / a.per_cta;
   }
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (num_experts <= 32) launch<1>(a, ctas, single, s);
-  else if (num_experts <= 64) launch<2>(a, ctas, single, s);
-  else if (num_experts <= 128) launch<4>(a, ctas, single, s);
-  else if (num_experts <= 256) launch<8>(a, ctas, single, s);
-  else launch<16>(a, ctas, single, s);
+  auto go = [&](auto epl) {
+    if (soft) launch<decltype(epl)::value, true>(a, ctas, single, s);
+    else launch<decltype(epl)::value, false>(a, ctas, single, s);
+  };
+  if (num_experts <= 32) go(std::integral_constant<int, 1>());
+  else if (num_experts <= 64) go(std::integral_constant<int, 2>());
+  else if (num_experts <= 128) go(std::integral_constant<int, 4>());
+  else if (num_experts <= 256) go(std::integral_constant<int, 8>());
+  else go(std::integral_constant<int, 16>());
   return launch_result();
+}
+}  // namespace
+}  // namespace b200
+
+extern "C" int b200_moe_group_route(const float* logits, const float* correction, int32_t num_tokens, int32_t num_experts,
+                                    int32_t top, int32_t groups, int32_t keep, int32_t* sorted_token, float* weight,
+                                    int32_t* expert_offsets, int32_t* slot_to_row, void* workspace, size_t workspace_bytes,
+                                    void* stream) {
+  return b200::route(logits, correction, num_tokens, num_experts, top, groups, keep, false, sorted_token, weight, expert_offsets,
+                     slot_to_row, workspace, workspace_bytes, stream);
+}
+
+extern "C" int b200_moe_softmax_route(const float* logits, const float* bias, int32_t num_tokens, int32_t num_experts, int32_t top,
+                                      int32_t* sorted_token, float* weight, int32_t* expert_offsets, int32_t* slot_to_row,
+                                      void* workspace, size_t workspace_bytes, void* stream) {
+  return b200::route(logits, bias, num_tokens, num_experts, top, 1, 1, true, sorted_token, weight, expert_offsets, slot_to_row,
+                     workspace, workspace_bytes, stream);
 }

@@ -29,9 +29,13 @@
 //
 // Generic path (any dtype / head_dim <= 256 / block size): one CTA per (sequence, query head),
 // fp32 FMA arithmetic.  It is the path the fp32 engine configuration uses.
+//
+// SIGM variants of both: the weights are sigmoid(scale q.k + bias[head]) and are not normalised, only the keys of the last
+// token's chunk of positions are listed and read, pieces of a cut sequence just add up, and a row leaves through its gate.
 #include <limits.h>
 
 #include "decode_common.cuh"
+#include "sequences.cuh"
 
 namespace b200 {
 namespace {
@@ -62,7 +66,21 @@ struct DecodeArgs {
   int32_t* counters; // [batch][Hkv]       arrivals per (sequence, KV head), zero between launches; null = separate merge
   const float* sink; // [Hq] or null: exp(sink) joins the denominator of its head
   int32_t* status;
+  const float* bias; // [Hq], SIGM kernels (null: softmax)
+  int chunk;         // positions per chunk, SIGM kernels
+  const void* gate;  // [batch, Hq] or null, SIGM kernels
+  int64_t gate_stride;
 };
+
+// what a finished row of the SIGM kernels is multiplied by
+template <typename T>
+__device__ __forceinline__ float gate_of(const DecodeArgs& a, int seq, int head) {
+  return a.gate ? sigmoid_f(to_float<T>(static_cast<const T*>(a.gate)[seq * a.gate_stride + head])) : 1.f;
+}
+// first position of the chunk of a context's last token
+__device__ __forceinline__ int64_t chunk_start(const DecodeArgs& a, int64_t len) {
+  return len > 0 ? (len - 1) / a.chunk * a.chunk : 0;
+}
 
 // physical 16-token block of a sequence's 16-token block number blk
 __device__ __forceinline__ int64_t physical_block(const DecodeArgs& a, int seq, int blk) {
@@ -71,8 +89,9 @@ __device__ __forceinline__ int64_t physical_block(const DecodeArgs& a, int seq, 
   return id < 0 ? id : static_cast<int64_t>(id) * a.sub + blk % a.sub;
 }
 
+// nblk blocks from block `first` on hold keys that count; blk runs from 0
 struct Cursor {
-  int seq, blk, nblk, len;
+  int seq, blk, nblk, len, first;
 };
 
 template <int D>
@@ -87,7 +106,7 @@ __device__ __forceinline__ int swizzle_chunk(int c, int t) {
 // fp32 columns per lane, 32 / (D / 4) heads per pass; the lanes of a head share the search for its maximum,
 // and the weighted sum takes four pieces per trip so that their loads are in flight together.  Loads bypass
 // L1: other SMs wrote the data.
-template <int D>
+template <int D, bool SIGM>
 __device__ __forceinline__ void merge_split_sequence(const DecodeArgs& a, int seq, int h, int G, int first,
                                                      int np, int lane) {
   constexpr int LPH = D / 4;    // lanes per head
@@ -129,7 +148,7 @@ __device__ __forceinline__ void merge_split_sequence(const DecodeArgs& a, int se
     }
     if (active) {
       if (a.sink != nullptr) L += sink_term(a.sink[head], M);
-      const float inv = 1.f / L;
+      const float inv = SIGM ? gate_of<__nv_bfloat16>(a, seq, head) : 1.f / L;
       uint2 packed;
       packed.x = pack_bf16x2(acc.x * inv, acc.y * inv);
       packed.y = pack_bf16x2(acc.z * inv, acc.w * inv);
@@ -139,7 +158,7 @@ __device__ __forceinline__ void merge_split_sequence(const DecodeArgs& a, int se
   }
 }
 
-template <int D, int NT>
+template <int D, int NT, bool SIGM>
 __global__ void __launch_bounds__(kMaxFastThreads)
 paged_decode_bf16_kernel(const DecodeArgs a) {
   extern __shared__ __align__(128) uint8_t smem[];
@@ -158,11 +177,15 @@ paged_decode_bf16_kernel(const DecodeArgs a) {
   const int G = a.Hq / a.Hkv;
   const int p = blockIdx.x, P = gridDim.x;
   const int64_t table_blocks = a.bt_stride * a.sub;
+  // blocks ahead of the chunk of a context's last token, and blocks from there on
+  auto skipped = [&](int64_t len) -> int {
+    return SIGM ? static_cast<int>(min(chunk_start(a, len) / kTok, table_blocks)) : 0;
+  };
+  auto listed = [&](int64_t len) -> int { return num_kv_blocks(len, table_blocks, kTok) - skipped(len); };
 
   // ---- plan: total block count, then the (sequence, block) where this CTA's range starts ----
   int local = 0;
-  for (int i = threadIdx.x; i < B; i += blockDim.x)
-    local += num_kv_blocks(a.lens[i], table_blocks, kTok);
+  for (int i = threadIdx.x; i < B; i += blockDim.x) local += listed(a.lens[i]);
   int T;
   block_inclusive_scan(local, s_scan, &T);
   if (a.counters == nullptr) {
@@ -186,7 +209,7 @@ paged_decode_bf16_kernel(const DecodeArgs a) {
     int carry = 0;
     for (int base = 0; base < B; base += blockDim.x) {
       const int i = base + threadIdx.x;
-      const int v = i < B ? num_kv_blocks(a.lens[i], table_blocks, kTok) : 0;
+      const int v = i < B ? listed(a.lens[i]) : 0;
       int tot;
       const int incl = block_inclusive_scan(v, s_scan, &tot) + carry;
       const int excl = incl - v;
@@ -201,8 +224,9 @@ paged_decode_bf16_kernel(const DecodeArgs a) {
 
   auto load_seq = [&](Cursor& c) {
     const int64_t len = a.lens[c.seq];
-    c.nblk = num_kv_blocks(len, table_blocks, kTok);
-    const int64_t cap = static_cast<int64_t>(c.nblk) * kTok;
+    c.first = skipped(len);
+    c.nblk = listed(len);
+    const int64_t cap = static_cast<int64_t>(c.first + c.nblk) * kTok;
     if (len > cap) report(a.status, B200_ERR_BOUNDS);  // table row too short for the context
     c.len = static_cast<int>(len < cap ? len : cap);
   };
@@ -226,7 +250,8 @@ paged_decode_bf16_kernel(const DecodeArgs a) {
   load_seq(L);
   C.nblk = L.nblk;
   C.len = L.len;
-  int64_t next_id = physical_block(a, L.seq, L.blk);
+  C.first = L.first;
+  int64_t next_id = physical_block(a, L.seq, L.first + L.blk);
 
   const int h = warp;  // KV head of this warp
   const uint32_t ring = smem_u32(smem) + warp * (kStages * 2 * TILEB);
@@ -236,7 +261,7 @@ paged_decode_bf16_kernel(const DecodeArgs a) {
 
   auto issue = [&](int stage) {
     const int64_t id = next_id;
-    const int valid = L.len - L.blk * kTok;  // tokens of this block inside the context
+    const int valid = L.len - (L.first + L.blk) * kTok;  // tokens of this block inside the context
     const bool ok = static_cast<uint64_t>(id) < static_cast<uint64_t>(a.num_blocks * a.sub);
     if (!ok) report(a.status, B200_ERR_BOUNDS);
     const int64_t blk_off = ok ? id * kTok * row_stride : 0;
@@ -255,6 +280,16 @@ paged_decode_bf16_kernel(const DecodeArgs a) {
 
   float o[NT][KS][4];
   float mrow[NT][2], lrow[NT][2];
+  float bias[NT][2];             // SIGM: of this thread's two heads, as the exponent takes them
+  if constexpr (SIGM) {
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int head = nt * 8 + tq * 2 + e;
+        bias[nt][e] = head < G ? -1.4426950408889634f * a.bias[h * G + head] : 0.f;
+      }
+  }
   uint32_t qf[NT][KS][2];
   int seg_first = 0;
   bool fresh = true;
@@ -266,7 +301,7 @@ paged_decode_bf16_kernel(const DecodeArgs a) {
       issue(s);
       if (++issued < cnt) {
         advance(L);
-        next_id = physical_block(a, L.seq, L.blk);
+        next_id = physical_block(a, L.seq, L.first + L.blk);
       }
     }
     cp_async_commit();
@@ -277,7 +312,7 @@ paged_decode_bf16_kernel(const DecodeArgs a) {
       issue((j + kStages - 1) % kStages);
       if (++issued < cnt) {
         advance(L);
-        next_id = physical_block(a, L.seq, L.blk);
+        next_id = physical_block(a, L.seq, L.first + L.blk);
       }
     }
     cp_async_commit();
@@ -290,7 +325,7 @@ paged_decode_bf16_kernel(const DecodeArgs a) {
 #pragma unroll
       for (int nt = 0; nt < NT; ++nt) {
         const int head = nt * 8 + g;
-        mrow[nt][0] = mrow[nt][1] = -INFINITY;
+        mrow[nt][0] = mrow[nt][1] = SIGM ? 0.f : -INFINITY;
         lrow[nt][0] = lrow[nt][1] = 0.f;
 #pragma unroll
         for (int ks = 0; ks < KS; ++ks) {
@@ -312,7 +347,7 @@ paged_decode_bf16_kernel(const DecodeArgs a) {
     __syncwarp();
 
     const uint32_t kt = ring + (j % kStages) * (2 * TILEB), vt = kt + TILEB;
-    const int valid = C.len - C.blk * kTok;
+    const int valid = C.len - (C.first + C.blk) * kTok;
 
     // ---- S^T[token, head] = K . Q^T ----
     float s[NT][4];
@@ -332,6 +367,19 @@ paged_decode_bf16_kernel(const DecodeArgs a) {
 
     // ---- online softmax over the token axis (rows g and g+8 of the tile) ----
     uint32_t pb[NT][2];
+    if constexpr (SIGM) {
+      const int low = static_cast<int>(chunk_start(a, C.len)) - (C.first + C.blk) * kTok;   // first token that counts
+      const bool in0 = g < valid && g >= low, in1 = g + 8 < valid && g + 8 >= low;
+#pragma unroll
+      for (int nt = 0; nt < NT; ++nt) {
+        const float b0 = bias[nt][0], b1 = bias[nt][1];
+        auto weight = [&](float x, float b) { return rcp_approx(1.f + fast_exp2(fmaf(x, -a.scale_log2, b))); };
+        const float p0 = in0 ? weight(s[nt][0], b0) : 0.f, p1 = in0 ? weight(s[nt][1], b1) : 0.f;
+        const float p2 = in1 ? weight(s[nt][2], b0) : 0.f, p3 = in1 ? weight(s[nt][3], b1) : 0.f;
+        pb[nt][0] = movmatrix_trans(pack_bf16x2(p0, p1));
+        pb[nt][1] = movmatrix_trans(pack_bf16x2(p2, p3));
+      }
+    } else {
 #pragma unroll
     for (int nt = 0; nt < NT; ++nt) {
       float x0 = s[nt][0] * a.scale_log2, x1 = s[nt][1] * a.scale_log2;
@@ -361,6 +409,7 @@ paged_decode_bf16_kernel(const DecodeArgs a) {
         o[nt][mt][2] *= al0;
         o[nt][mt][3] *= al1;
       }
+    }
     }
 
     // ---- O^T[d, head] += V^T . P^T ----
@@ -396,7 +445,11 @@ paged_decode_bf16_kernel(const DecodeArgs a) {
             if (head0 < G) l0 += sink_term(a.sink[h * G + head0], mrow[nt][0]);
             if (head0 + 1 < G) l1 += sink_term(a.sink[h * G + head0 + 1], mrow[nt][1]);
           }
-          const float i0 = 1.f / l0, i1 = 1.f / l1;
+          float i0 = 1.f / l0, i1 = 1.f / l1;
+          if constexpr (SIGM) {
+            i0 = head0 < G ? gate_of<__nv_bfloat16>(a, C.seq, h * G + head0) : 0.f;
+            i1 = head0 + 1 < G ? gate_of<__nv_bfloat16>(a, C.seq, h * G + head0 + 1) : 0.f;
+          }
           __nv_bfloat16* op = static_cast<__nv_bfloat16*>(a.out) +
                               (static_cast<int64_t>(C.seq) * a.Hq + h * G) * D;
 #pragma unroll
@@ -459,7 +512,7 @@ paged_decode_bf16_kernel(const DecodeArgs a) {
         arrived = __shfl_sync(0xffffffffu, arrived, 0);
         if (arrived == np - 1) {
           __threadfence();
-          merge_split_sequence<D>(a, C.seq, h, G, first, np, lane);
+          merge_split_sequence<D, SIGM>(a, C.seq, h, G, first, np, lane);
           if (lane == 0) *cnt = 0;   // ready for the next launch
         }
       }
@@ -509,7 +562,7 @@ paged_decode_combine_kernel(const DecodeArgs a) {
     }
     if (a.sink != nullptr) L += sink_term(a.sink[h], M);
     s_M[h] = M;
-    s_inv[h] = 1.f / L;
+    s_inv[h] = a.bias != nullptr ? gate_of<__nv_bfloat16>(a, i, h) : 1.f / L;     // SIGM: M is 0
   }
   __syncthreads();
   constexpr int kVec = 4;
@@ -602,7 +655,7 @@ namespace {
 constexpr int kSimpleWarps = 4;
 constexpr int kSimpleMaxPerLane = 8;  // head_dim <= 256
 
-template <typename T>
+template <typename T, bool SIGM>
 __global__ void __launch_bounds__(kSimpleWarps * 32) paged_decode_simple_kernel(const DecodeArgs a) {
   __shared__ float s_m[kSimpleWarps], s_l[kSimpleWarps];
   __shared__ float s_acc[kSimpleWarps][kSimpleMaxPerLane * 32];
@@ -632,7 +685,7 @@ __global__ void __launch_bounds__(kSimpleWarps * 32) paged_decode_simple_kernel(
   float m = -INFINITY, l = 0.f;
   const T* kc = static_cast<const T*>(a.kc);
   const T* vc = static_cast<const T*>(a.vc);
-  for (int t = warp; t < len; t += kSimpleWarps) {
+  for (int t = (SIGM ? static_cast<int>(chunk_start(a, len)) : 0) + warp; t < len; t += kSimpleWarps) {
     const int id = a.bt[static_cast<int64_t>(seq) * a.bt_stride + t / a.bs];
     if (static_cast<uint64_t>(static_cast<int64_t>(id)) >= static_cast<uint64_t>(a.num_blocks)) {
       report(a.status, B200_ERR_BOUNDS);
@@ -646,7 +699,17 @@ __global__ void __launch_bounds__(kSimpleWarps * 32) paged_decode_simple_kernel(
       const int d = lane + 32 * k;
       if (d < D) dot += qv[k] * to_float<T>(kc[row + d]);
     }
-    dot = warp_sum(dot) * a.scale_log2;
+    dot = warp_sum(dot);
+    if constexpr (SIGM) {
+      const float p = sigmoid_f(dot * a.scale_log2 + a.bias[head]);
+#pragma unroll
+      for (int k = 0; k < kSimpleMaxPerLane; ++k) {
+        const int d = lane + 32 * k;
+        if (d < Dv) acc[k] += p * to_float<T>(vc[vrow + d]);
+      }
+      continue;
+    }
+    dot *= a.scale_log2;
     const float mn = fmaxf(m, dot);
     const float al = exp2f(m - mn), pw = exp2f(dot - mn);
     l = l * al + pw;
@@ -664,6 +727,15 @@ __global__ void __launch_bounds__(kSimpleWarps * 32) paged_decode_simple_kernel(
 #pragma unroll
   for (int k = 0; k < kSimpleMaxPerLane; ++k) s_acc[warp][lane + 32 * k] = acc[k];
   __syncthreads();
+  if constexpr (SIGM) {
+    const float gate = gate_of<T>(a, seq, head);
+    for (int d = threadIdx.x; d < Dv; d += blockDim.x) {
+      float v = 0.f;
+      for (int w = 0; w < kSimpleWarps; ++w) v += s_acc[w][d];
+      op[d] = from_float<T>(v * gate);
+    }
+    return;
+  }
   float M = -INFINITY;
   for (int w = 0; w < kSimpleWarps; ++w) M = fmaxf(M, s_m[w]);
   float Lsum = 0.f;
@@ -711,7 +783,7 @@ FastPlan fast_plan(int Hq, int Hkv, int D, int bs, int dtype) {
   return pl;
 }
 
-template <int D, int NT>
+template <int D, int NT, bool SIGM>
 int launch_fast(const DecodeArgs& a, const FastPlan& pl, int grid, cudaStream_t s) {
   // per-device "shared-memory limit raised" flags: written without a lock; two host threads racing here both
   // make the same idempotent cudaFuncSetAttribute call and both store true
@@ -719,13 +791,13 @@ int launch_fast(const DecodeArgs& a, const FastPlan& pl, int grid, cudaStream_t 
   int dev = 0;
   cudaGetDevice(&dev);
   if (dev >= 0 && dev < 64 && !configured[dev]) {
-    if (cudaFuncSetAttribute(paged_decode_bf16_kernel<D, NT>,
+    if (cudaFuncSetAttribute(paged_decode_bf16_kernel<D, NT, SIGM>,
                              cudaFuncAttributeMaxDynamicSharedMemorySize,
                              220 * 1024) != cudaSuccess)
       return B200_ERR_LAUNCH;
     configured[dev] = true;
   }
-  paged_decode_bf16_kernel<D, NT><<<grid, pl.threads, pl.smem, s>>>(a);
+  paged_decode_bf16_kernel<D, NT, SIGM><<<grid, pl.threads, pl.smem, s>>>(a);
   return launch_result();
 }
 
@@ -750,11 +822,22 @@ extern "C" size_t b200_paged_decode_gqa_workspace_bytes(int32_t batch, int32_t n
 }
 
 namespace b200 {
+namespace {
+// what the sigmoid form has in addition
+struct SigmoidForm {
+  const float* bias;
+  int chunk;
+  const void* gate;
+  int64_t gate_stride;
+};
+}  // namespace
+
+template <bool SIGM = false>
 static int paged_decode(const void* q, const void* k_cache, const void* v_cache, void* out, const int32_t* block_tables,
                         int64_t bt_stride, const int64_t* context_lens, int32_t batch, int32_t num_q_heads,
                         int32_t num_kv_heads, int32_t head_dim, int32_t head_dim_v, int32_t block_size, int64_t num_blocks,
                         float scale, const float* sink, void* workspace, size_t workspace_bytes, int32_t dtype,
-                        int32_t* status, void* stream) {
+                        int32_t* status, void* stream, const SigmoidForm& form = {}) {
   if (batch < 0 || num_q_heads <= 0 || num_kv_heads <= 0 || head_dim <= 0 || head_dim_v <= 0 || block_size <= 0 ||
       num_blocks < 0 || bt_stride <= 0)
     return B200_ERR_ARG;
@@ -784,6 +867,12 @@ static int paged_decode(const void* q, const void* k_cache, const void* v_cache,
   a.num_blocks = num_blocks;
   a.scale_log2 = scale * 1.4426950408889634f;
   a.status = status;
+  if constexpr (SIGM) {
+    a.bias = form.bias;
+    a.chunk = form.chunk > 0 ? form.chunk : 2147483647;
+    a.gate = form.gate;
+    a.gate_stride = form.gate_stride;
+  }
 
   const FastPlan pl = fast_plan(num_q_heads, num_kv_heads, head_dim, block_size, dtype);
   const bool fast = pl.ok && head_dim_v == head_dim && aligned16(q) && aligned16(k_cache) && aligned16(v_cache);
@@ -819,21 +908,22 @@ static int paged_decode(const void* q, const void* k_cache, const void* v_cache,
     int rc;
     const int gi = static_cast<int>(grid);
     if (head_dim == 128)
-      rc = pl.nt == 1 ? launch_fast<128, 1>(a, pl, gi, s) : launch_fast<128, 2>(a, pl, gi, s);
+      rc = pl.nt == 1 ? launch_fast<128, 1, SIGM>(a, pl, gi, s) : launch_fast<128, 2, SIGM>(a, pl, gi, s);
     else if (head_dim == 64)
-      rc = pl.nt == 1 ? launch_fast<64, 1>(a, pl, gi, s) : launch_fast<64, 2>(a, pl, gi, s);
+      rc = pl.nt == 1 ? launch_fast<64, 1, SIGM>(a, pl, gi, s) : launch_fast<64, 2, SIGM>(a, pl, gi, s);
     else
-      rc = pl.nt == 1 ? launch_fast<32, 1>(a, pl, gi, s) : launch_fast<32, 2>(a, pl, gi, s);
+      rc = pl.nt == 1 ? launch_fast<32, 1, SIGM>(a, pl, gi, s) : launch_fast<32, 2, SIGM>(a, pl, gi, s);
     if (rc != B200_OK || fused_merge) return rc;
     return launch_combine(a, batch, s);
   }
 
   if (head_dim > kSimpleMaxPerLane * 32 || head_dim_v > kSimpleMaxPerLane * 32) return B200_ERR_UNSUPPORTED;
+  if (SIGM) a.scale_log2 = scale;      // the sigmoid of the generic kernel takes natural exponents
   dim3 grid(batch, num_q_heads);
   if (dtype == B200_DTYPE_F32)
-    paged_decode_simple_kernel<float><<<grid, kSimpleWarps * 32, 0, s>>>(a);
+    paged_decode_simple_kernel<float, SIGM><<<grid, kSimpleWarps * 32, 0, s>>>(a);
   else
-    paged_decode_simple_kernel<__nv_bfloat16><<<grid, kSimpleWarps * 32, 0, s>>>(a);
+    paged_decode_simple_kernel<__nv_bfloat16, SIGM><<<grid, kSimpleWarps * 32, 0, s>>>(a);
   return launch_result();
 }
 }  // namespace b200
@@ -859,6 +949,18 @@ extern "C" int b200_paged_decode_sink(const void* q, const void* k_cache, const 
   return b200::paged_decode(q, k_cache, v_cache, out, block_tables, bt_stride, context_lens, batch, num_q_heads,
                             num_kv_heads, head_dim_qk, head_dim_v, block_size, num_blocks, scale, sink, workspace,
                             workspace_bytes, dtype, status, stream);
+}
+
+extern "C" int b200_sigmoid_decode(const void* q, const void* k_cache, const void* v_cache, void* out,
+                                   const int32_t* block_tables, int64_t bt_stride, const int64_t* context_lens, int32_t batch,
+                                   int32_t num_q_heads, int32_t num_kv_heads, int32_t head_dim_qk, int32_t head_dim_v,
+                                   int32_t block_size, int64_t num_blocks, float scale, const float* bias, int32_t chunk,
+                                   const void* gate, int64_t gate_token_stride, void* workspace, size_t workspace_bytes,
+                                   int32_t dtype, int32_t* status, void* stream) {
+  if (!bias || chunk < 0) return B200_ERR_ARG;
+  return b200::paged_decode<true>(q, k_cache, v_cache, out, block_tables, bt_stride, context_lens, batch, num_q_heads,
+                                  num_kv_heads, head_dim_qk, head_dim_v, block_size, num_blocks, scale, nullptr, workspace,
+                                  workspace_bytes, dtype, status, stream, {bias, chunk, gate, gate_token_stride});
 }
 
 // ---------------------------------------------------------------------------------------------

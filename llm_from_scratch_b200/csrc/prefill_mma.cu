@@ -13,8 +13,9 @@
 // gaps; CTAs whose tile lies past the end of their sequence return at once.
 //
 // The general variant serves head sizes that are smaller than the compiled ones (any multiples of eight), a key part shared by
-// all heads of any such width, and a sliding window: the walk starts at the first tile the window of row 0 reaches.
-#include "common.cuh"
+// all heads of any such width, and a sliding window: the walk starts at the first tile the window of row 0 reaches.  With SIGM
+// the weights are sigmoid(scale q.k + bias[head]), the visible keys those of the query's chunk, and rows leave through a gate.
+#include "sequences.cuh"
 
 namespace b200 {
 namespace {
@@ -47,6 +48,10 @@ struct MmaArgs {
   const float* sink;     // [Hq] or null
   int dqk, dv, tail;     // general variant: head sizes and width of the shared key part
   int window;            // general variant: keys a query sees, its own included; 0: all
+  const float* bias;     // SIGM: [Hq], added to the scores
+  int chunk;             // SIGM: positions per chunk, counted from the first key
+  const __nv_bfloat16* gate;   // SIGM: [tokens, Hq] or null
+  int64_t gate_stride;
   int32_t* status;
 };
 
@@ -57,7 +62,7 @@ __device__ __forceinline__ int swz(int c, int row) {
   return c ^ ((row >> 1) & (CPR - 1));
 }
 
-template <int DQK, int DV, bool PAGED, int TAIL = 0, bool GENERAL = false>
+template <int DQK, int DV, bool PAGED, int TAIL = 0, bool GENERAL = false, bool SIGM = false>
 __global__ void __launch_bounds__(kThreads, 2) prefill_mma_kernel(const MmaArgs a) {
   extern __shared__ __align__(128) uint8_t smem[];
   constexpr int KQ = DQK / 16;   // k-steps of S
@@ -80,8 +85,12 @@ __global__ void __launch_bounds__(kThreads, 2) prefill_mma_kernel(const MmaArgs 
   const int m0 = tile * BM;
   if (m0 >= q_len) return;
   int off = k_len - q_len;                       // keys every new token sees besides its own prefix
-  if (GENERAL && a.window > 0) {                 // keys count from the first tile that row 0 sees
-    const int skip = max(0, off + m0 - a.window + 1) / BN * BN;
+  int skip = 0;                                  // keys ahead of the walk
+  const bool cut = SIGM || (GENERAL && a.window > 0);
+  // first key that the query sees whose own key is number i, in keys of the walk (may be negative)
+  auto first_key = [&](int i) -> int { return SIGM ? (i + skip) / a.chunk * a.chunk - skip : i - a.window + 1; };
+  if (cut) {                                     // keys count from the first tile that row 0 sees
+    skip = max(0, first_key(off + m0)) / BN * BN;
     k0 += skip;
     k_len -= skip;
     off -= skip;
@@ -220,6 +229,10 @@ __global__ void __launch_bounds__(kThreads, 2) prefill_mma_kernel(const MmaArgs 
   for (int n = 0; n < NV; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
   float m_r[2] = {-INFINITY, -INFINITY}, l_r[2] = {0.f, 0.f};
   const int row0 = m0 + warp * 16 + g;  // query index (within the sequence) of c0/c1; +8 for c2/c3
+  // first visible keys of these rows, and the largest of the warp's rows
+  const int low0 = cut ? first_key(off + row0) : 0, low1 = cut ? first_key(off + row0 + 8) : 0;
+  const int low_max = cut ? first_key(off + m0 + warp * 16 + 15) : 0;
+  const float nbias = SIGM ? -1.4426950408889634f * a.bias[head] : 0.f;
 
   for (int j = 0; j < ntiles; ++j) {
     const int stage = j & 1;
@@ -252,9 +265,26 @@ __global__ void __launch_bounds__(kThreads, 2) prefill_mma_kernel(const MmaArgs 
     }
     // ---- scale, causal / length mask, online softmax ----
     const int n0 = j * BN;
-    const bool windowed = GENERAL && a.window > 0;
     const bool need_mask = (n0 + BN - 1 > off + m0 + warp * 16) || (n0 + BN > kmax) ||
-                           (windowed && n0 <= off + m0 + warp * 16 + 15 - a.window);
+                           (cut && n0 < low_max);
+    uint32_t pf[BN / 16][4];
+    if constexpr (SIGM) {
+      const int lim0 = min(off + row0, kmax - 1), lim1 = min(off + row0 + 8, kmax - 1);
+#pragma unroll
+      for (int n = 0; n < BN / 8; ++n) {
+        float p[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          p[e] = rcp_approx(1.f + fast_exp2(fmaf(s[n][e], -a.scale_log2, nbias)));
+          if (need_mask) {
+            const int key = n0 + n * 8 + tq * 2 + (e & 1);
+            if (key > (e < 2 ? lim0 : lim1) || key < (e < 2 ? low0 : low1)) p[e] = 0.f;
+          }
+        }
+        pf[n >> 1][(n & 1) * 2] = pack_bf16x2(p[0], p[1]);
+        pf[n >> 1][(n & 1) * 2 + 1] = pack_bf16x2(p[2], p[3]);
+      }
+    } else {
     float mx0 = -INFINITY, mx1 = -INFINITY;
 #pragma unroll
     for (int n = 0; n < BN / 8; ++n) {
@@ -267,12 +297,11 @@ __global__ void __launch_bounds__(kThreads, 2) prefill_mma_kernel(const MmaArgs 
         if (key + 1 > lim0) s[n][1] = -INFINITY;
         if (key > lim1) s[n][2] = -INFINITY;
         if (key + 1 > lim1) s[n][3] = -INFINITY;
-        if (windowed) {
-          const int low0 = off + row0 - a.window, low1 = low0 + 8;      // last key before the window
-          if (key <= low0) s[n][0] = -INFINITY;
-          if (key + 1 <= low0) s[n][1] = -INFINITY;
-          if (key <= low1) s[n][2] = -INFINITY;
-          if (key + 1 <= low1) s[n][3] = -INFINITY;
+        if (cut) {
+          if (key < low0) s[n][0] = -INFINITY;
+          if (key + 1 < low0) s[n][1] = -INFINITY;
+          if (key < low1) s[n][2] = -INFINITY;
+          if (key + 1 < low1) s[n][3] = -INFINITY;
         }
       }
       mx0 = fmaxf(mx0, fmaxf(s[n][0], s[n][1]));
@@ -289,7 +318,6 @@ __global__ void __launch_bounds__(kThreads, 2) prefill_mma_kernel(const MmaArgs 
     m_r[0] = mn0;
     m_r[1] = mn1;
     float ls0 = 0.f, ls1 = 0.f;
-    uint32_t pf[BN / 16][4];
 #pragma unroll
     for (int n = 0; n < BN / 8; ++n) {
       const float p0 = fast_exp2(s[n][0] - sub0), p1 = fast_exp2(s[n][1] - sub0);
@@ -307,6 +335,7 @@ __global__ void __launch_bounds__(kThreads, 2) prefill_mma_kernel(const MmaArgs 
       o[n][1] *= al0;
       o[n][2] *= al1;
       o[n][3] *= al1;
+    }
     }
     // ---- O += P V ----
     {
@@ -341,8 +370,16 @@ __global__ void __launch_bounds__(kThreads, 2) prefill_mma_kernel(const MmaArgs 
     l0 += sink_term(sink, m_r[0]);
     l1 += sink_term(sink, m_r[1]);
   }
-  const float i0 = l0 > 0.f ? 1.f / l0 : 0.f, i1 = l1 > 0.f ? 1.f / l1 : 0.f;
+  float i0 = l0 > 0.f ? 1.f / l0 : 0.f, i1 = l1 > 0.f ? 1.f / l1 : 0.f;
   const int r0 = warp * 16 + g, r1 = r0 + 8;
+  if constexpr (SIGM) {
+    auto gate = [&](int r) {
+      return a.gate != nullptr && r < rows_q
+                 ? sigmoid_f(__bfloat162float(a.gate[static_cast<int64_t>(q0 + m0 + r) * a.gate_stride + head])) : 1.f;
+    };
+    i0 = gate(r0);
+    i1 = gate(r1);
+  }
   __nv_bfloat16* ob = a.out + (static_cast<int64_t>(q0 + m0) * a.Hq + head) * dv;
 #pragma unroll
   for (int n = 0; n < NV; ++n) {
@@ -357,13 +394,13 @@ __global__ void __launch_bounds__(kThreads, 2) prefill_mma_kernel(const MmaArgs 
   }
 }
 
-template <int DQK, int DV, int TAIL = 0, bool GENERAL = false>
+template <int DQK, int DV, int TAIL = 0, bool GENERAL = false, bool SIGM = false>
 int launch(const MmaArgs& a, int num_seqs, int plan_capacity, bool paged, cudaStream_t s) {
   constexpr size_t smem = size_t(BM) * DQK * 2 + 2 * size_t(BN) * DQK * 2 + 2 * size_t(BN) * DV * 2;
   static bool configured[64][2] = {};
   int dev = 0;
   cudaGetDevice(&dev);
-  auto kern = paged ? prefill_mma_kernel<DQK, DV, !GENERAL, 0, GENERAL> : prefill_mma_kernel<DQK, DV, false, TAIL, GENERAL>;
+  auto kern = paged ? prefill_mma_kernel<DQK, DV, !GENERAL, 0, GENERAL, SIGM> : prefill_mma_kernel<DQK, DV, false, TAIL, GENERAL, SIGM>;
   if (dev >= 0 && dev < 64 && !configured[dev][paged]) {
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize,
                              static_cast<int>(smem)) != cudaSuccess)
@@ -477,6 +514,44 @@ int prefill_mma_general_launch(const void* q, const void* k, const void* v, void
   if (Dqk <= 64 && Dv <= 64) return launch<64, 64, 0, true>(a, num_seqs, plan_capacity, false, s);
   if (Dqk <= 128) return launch<128, 128, 0, true>(a, num_seqs, plan_capacity, false, s);
   return launch<192, 128, 0, true>(a, num_seqs, plan_capacity, false, s);
+}
+
+// Sigmoid weights inside chunks of positions, with an output gate; packed keys.
+int prefill_mma_sigmoid_launch(const void* q, const void* k, const void* v, void* out, int64_t q_stride, int64_t k_stride,
+                               int64_t v_stride, const int32_t* cu_q, const int32_t* cu_k, int num_seqs, int max_seqlen_q,
+                               int Hq, int Hkv, int Dqk, int Dv, float scale, const float* bias, int chunk, const void* gate,
+                               int64_t gate_stride, const int32_t* plan, int plan_tile_rows, int plan_capacity, int32_t* status,
+                               cudaStream_t s) {
+  if (!prefill_mma_general_shape(Dqk, Dv, 0)) return B200_ERR_UNSUPPORTED;
+  const int ntiles = (max_seqlen_q + BM - 1) / BM;
+  if (num_seqs > 65535 || ntiles > 65535) return B200_ERR_UNSUPPORTED;
+  auto al = [](const void* p, int64_t stride) { return aligned16(p) && (stride * 2) % 16 == 0; };
+  if (!al(q, q_stride) || !al(k, k_stride) || !al(v, v_stride) || !aligned16(out)) return B200_ERR_UNSUPPORTED;
+  MmaArgs a{};
+  a.q = static_cast<const __nv_bfloat16*>(q);
+  a.k = static_cast<const __nv_bfloat16*>(k);
+  a.v = static_cast<const __nv_bfloat16*>(v);
+  a.out = static_cast<__nv_bfloat16*>(out);
+  a.q_stride = q_stride;
+  a.k_stride = k_stride;
+  a.v_stride = v_stride;
+  a.cu_q = cu_q;
+  a.cu_k = cu_k;
+  a.Hq = Hq;
+  a.Hkv = Hkv;
+  a.ntiles_max = ntiles;
+  a.plan = (plan != nullptr && plan_tile_rows == BM && plan_capacity > 0 && plan_capacity <= 65535) ? plan : nullptr;
+  a.scale_log2 = scale * 1.4426950408889634f;
+  a.bias = bias;
+  a.chunk = chunk > 0 ? chunk : 2147483647;
+  a.gate = static_cast<const __nv_bfloat16*>(gate);
+  a.gate_stride = gate_stride;
+  a.dqk = Dqk;
+  a.dv = Dv;
+  a.status = status;
+  if (Dqk <= 64 && Dv <= 64) return launch<64, 64, 0, true, true>(a, num_seqs, plan_capacity, false, s);
+  if (Dqk <= 128) return launch<128, 128, 0, true, true>(a, num_seqs, plan_capacity, false, s);
+  return launch<192, 128, 0, true, true>(a, num_seqs, plan_capacity, false, s);
 }
 
 }  // namespace b200

@@ -24,6 +24,11 @@
 // thread and its softmax warps take the same turns at every barrier there, without products.  Every wait is bounded; a timeout aborts the CTA
 // and is reported.
 //
+// With SIGM the weights are sigmoid(scale q.k + bias[head]) instead of a softmax: no maximum, no sum and no rescaling of O; a
+// query sees the keys of its own chunk of positions (the walk starts and ends as with a window, whose first key is here the
+// chunk's), and the epilogue multiplies every row by the sigmoid of its gate.  Two exponentials share one reciprocal:
+// with a = 1 + 2^x, b = 1 + 2^y and r = 1 / (a b), 1 / a = r b and 1 / b = r a (x, y cut at 60: weights below 2^-60 do not count).
+//
 // What sets the pace, measured with clock counters in the warps: (1) the special-function unit — the 64
 // exponentials of a row tile occupy it for 512 clocks per warp, and the A and B warps of a scheduler, left
 // alone, run in step, share it during their exponentials (1,200 clocks each) and leave it idle during their
@@ -35,7 +40,7 @@
 // product into O).
 #include <cuda.h>
 
-#include "common.cuh"
+#include "sequences.cuh"
 #include "umma.cuh"
 
 namespace b200 {
@@ -78,15 +83,20 @@ struct Args2 {
   float scale_log2;
   const float* sink;     // [Hq] or null
   int window;            // keys a query sees, its own included (WINDOW kernels)
+  const float* bias;     // [Hq], added to the scores (SIGM kernels)
+  int chunk;             // positions per chunk, counted from the first key (SIGM kernels)
+  const __nv_bfloat16* gate;   // [tokens, Hq] or null (SIGM kernels)
+  int64_t gate_stride;
   int32_t* status;
 };
 
-template <int DQK, int DV, bool TAIL, bool WINDOW>
+template <int DQK, int DV, bool TAIL, bool WINDOW, bool SIGM>
 __global__ void __launch_bounds__(kThreads, 1)
 prefill_umma2_kernel(const Args2 a, const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k,
                      const __grid_constant__ CUtensorMap tm_kt, const __grid_constant__ CUtensorMap tm_v) {
   using L = Lay<DQK, DV>;
   constexpr int NST = L::NST;
+  constexpr bool CUT = WINDOW || SIGM;           // contexts have a first visible key
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   const uint32_t sb = smem_u32(smem);
@@ -111,8 +121,13 @@ prefill_umma2_kernel(const Args2 a, const __grid_constant__ CUtensorMap tm_q, co
   const int m0 = tile * ROWS;
   if (m0 >= q_len) return;                       // uniform over the CTA, before any barrier / allocation
   int off = k_len - q_len;
-  if (WINDOW) {                                  // keys count from the first tile that row 0 sees
-    const int skip = max(0, off + m0 - a.window + 1) / BN * BN;
+  int skip = 0;                                  // keys ahead of the walk
+  // first key that the query sees whose own key is number i, in keys of the walk (may be negative)
+  auto first_key = [&](int i) -> int {
+    return SIGM ? (i + skip) / a.chunk * a.chunk - skip : i - a.window + 1;
+  };
+  if (CUT) {                                     // keys count from the first tile that row 0 sees
+    skip = max(0, first_key(off + m0)) / BN * BN;
     k0 += skip;
     k_len -= skip;
     off -= skip;
@@ -130,8 +145,9 @@ prefill_umma2_kernel(const Args2 a, const __grid_constant__ CUtensorMap tm_q, co
     nt[x] = rows[x] > 0 ? (km + BN - 1) / BN : 0;
   }
   const bool has_b = rows[1] > 0;
-  // first tile a row of B sees: at most two behind A's, which A always walks (the window moves by 128 keys)
-  const int first_b = WINDOW ? max(0, off + m0 + BM - a.window + 1) / BN : 0;
+  // first tile a row of B sees: the tiles before it are all of A's (a window moves by 128 keys; a chunk that starts with B
+  // starts where A ends)
+  const int first_b = CUT ? max(0, first_key(off + m0 + BM)) / BN : 0;
   const int n = max(nt[0], nt[1]);               // KV tiles walked by the CTA; >= 1
 
   if (tid == 0) {
@@ -210,9 +226,9 @@ prefill_umma2_kernel(const Args2 a, const __grid_constant__ CUtensorMap tm_q, co
       const uint64_t kd = umma::smem_desc(sb + L::OFF_KV, 0, 1024);
       const uint64_t vd = umma::smem_desc(sb + L::OFF_KV + L::K_BYTES, K_SLAB, 1024);
       const uint32_t tSx = tmem + x * (128 + DV), tOx = tSx + 128;
-      const int j0 = WINDOW && x == 1 ? first_b : 0;
+      const int j0 = CUT && x == 1 ? first_b : 0;
       auto qk = [&](int st, int buf, int j) {       // S[buf] = Q . K^T of tile j in stage st, contraction in steps of 16
-        if (WINDOW && j < j0) {
+        if (CUT && j < j0) {
           umma::mbar_arrive(bar(L::QK_DONE + x) + st * 16);
           return;
         }
@@ -244,7 +260,7 @@ prefill_umma2_kernel(const Args2 a, const __grid_constant__ CUtensorMap tm_q, co
         WAIT_OR_ABORT(L::P_READY + 2 * x + (j & 1), (j >> 1) & 1)
         WAIT_OR_ABORT(L::V_FULL + st, ph)
         umma::fence_after_sync();
-        if (WINDOW && j < j0) {
+        if (CUT && j < j0) {
           umma::mbar_arrive(bar(L::PV_DONE + x) + st * 16);
           st = st1;
           ph = ph1;
@@ -268,13 +284,14 @@ prefill_umma2_kernel(const Args2 a, const __grid_constant__ CUtensorMap tm_q, co
     const uint32_t tS0 = tmem + x * (128 + DV) + lane_sel, tOx = tS0 + 128;
     const int qrow = m0 + x * BM + row;                     // index of the query inside its sequence
     const int lim = min(off + qrow, kmax[x] - 1);           // last visible key
-    const int low = WINDOW ? off + qrow - a.window + 1 : 0; // first visible key (may be negative)
+    const int low = CUT ? first_key(off + qrow) : 0;        // first visible key (may be negative)
     const int nx = nt[x];
     const uint32_t qk_done = bar(L::QK_DONE + x), pv_done = bar(L::PV_DONE + x);
     const uint32_t my_turn = bar(L::TURN + (x == 0 ? 0 : 4) + (warp & 3));
     const uint32_t their_turn = bar(L::TURN + (x == 0 ? 4 : 0) + (warp & 3));
-    const int j0 = WINDOW && x == 1 ? first_b : 0;          // first tile with products
+    const int j0 = CUT && x == 1 ? first_b : 0;             // first tile with products
     float m_ref = -INFINITY, l = 0.f;
+    const float nbias = SIGM ? -1.4426950408889634f * a.bias[head] : 0.f;
     bool alive = true;
     int st = 0, ph = 0, stp = 0, php = 0;                   // stage and phase of tile j and of tile j - 1
     for (int j = 0; j < nx; ++j) {
@@ -286,7 +303,7 @@ prefill_umma2_kernel(const Args2 a, const __grid_constant__ CUtensorMap tm_q, co
         break;
       }
       umma::fence_after_sync();
-      if (WINDOW && j < j0) {                                 // problem B only: every tile here is one of A's
+      if (CUT && j < j0) {                                    // problem B only: every tile here is one of A's
         if (!__all_sync(0xffffffffu, umma::mbar_wait(my_turn, j & 1, s_abort))) {
           give_up();
           alive = false;
@@ -303,13 +320,61 @@ prefill_umma2_kernel(const Args2 a, const __grid_constant__ CUtensorMap tm_q, co
         continue;
       }
       const int n0 = j * BN;
-      const bool warp_masked = __any_sync(0xffffffffu, n0 + BN - 1 > lim || (WINDOW && n0 < low));
+      const bool warp_masked = __any_sync(0xffffffffu, n0 + BN - 1 > lim || (CUT && n0 < low));
       // the 64 raw scores of the row stay in registers for both passes
       uint32_t ra[32], rb[32];
       umma::tmem_ld32(tSx, ra);
       umma::tmem_ld32_issue(tSx + 32, rb);
       float mx0 = -INFINITY, mx1 = -INFINITY;
-      uint64_t seen = 0;                                      // WINDOW: bit e set: the row sees key n0 + e
+      uint64_t seen = 0;                                      // CUT: bit e set: the row sees key n0 + e
+      if constexpr (SIGM) {
+        if (warp_masked) {
+          const int hi = lim - n0, lo = low - n0;
+          seen = (hi >= 63 ? ~0ull : hi < 0 ? 0ull : (2ull << hi) - 1ull) & (lo <= 0 ? ~0ull : lo > 63 ? 0ull : ~0ull << lo);
+        }
+        if (x == 0 ? (has_b && j >= 1) : (j < nt[0])) {       // turns as below
+          if (!__all_sync(0xffffffffu, umma::mbar_wait(my_turn, (x == 0 ? j - 1 : j) & 1, s_abort))) {
+            give_up();
+            alive = false;
+            break;
+          }
+        }
+        const uint64_t nscale2 = umma::pack_f32x2(-a.scale_log2, -a.scale_log2), nbias2 = umma::pack_f32x2(nbias, nbias);
+        const uint64_t one2 = umma::pack_f32x2(1.f, 1.f);
+        auto weigh = [&](const uint32_t (&r)[32], int c, uint32_t m) {
+          uint32_t pk[16];
+#pragma unroll
+          for (int e = 0; e < 32; e += 2) {
+            float s0, s1, d0, d1;
+            umma::unpack_f32x2(
+                umma::fma_f32x2(umma::pack_f32x2(__uint_as_float(r[e]), __uint_as_float(r[e + 1])), nscale2, nbias2), s0, s1);
+            umma::unpack_f32x2(umma::add_f32x2(umma::pack_f32x2(fast_exp2(fminf(s0, 60.f)), fast_exp2(fminf(s1, 60.f))), one2),
+                               d0, d1);
+            const float rc = rcp_approx(d0 * d1);
+            float p0 = rc * d1, p1 = rc * d0;
+            if (warp_masked) {
+              if (!(m & (1u << e))) p0 = 0.f;
+              if (!(m & (2u << e))) p1 = 0.f;
+            }
+            pk[e >> 1] = pack_bf16x2(p0, p1);
+          }
+          umma::tmem_st16(tSx + c * 16, pk);
+        };
+        weigh(ra, 0, static_cast<uint32_t>(seen));
+        umma::tmem_ld32_wait(rb);
+        weigh(rb, 1, static_cast<uint32_t>(seen >> 32));
+        umma::mbar_arrive(their_turn);
+        umma::tmem_wait_st();
+        umma::fence_before_sync();
+        umma::mbar_arrive(bar(L::P_READY + 2 * x + (j & 1)));
+        stp = st;
+        php = ph;
+        if (++st == NST) {
+          st = 0;
+          ph ^= 1;
+        }
+        continue;
+      }
       if (warp_masked) {
         if constexpr (WINDOW) {
           const int hi = lim - n0, lo = low - n0;
@@ -418,7 +483,12 @@ prefill_umma2_kernel(const Args2 a, const __grid_constant__ CUtensorMap tm_q, co
       if (alive && __all_sync(0xffffffffu, umma::mbar_wait(pv_done + stp * 16, php, s_abort))) {
         umma::fence_after_sync();
         if (a.sink != nullptr) l += sink_term(a.sink[head], m_ref);
-        const float inv = l > 0.f ? 1.f / l : 0.f;
+        float inv = l > 0.f ? 1.f / l : 0.f;
+        if constexpr (SIGM) {
+          inv = 1.f;
+          if (a.gate != nullptr && row < rows[x])
+            inv = sigmoid_f(__bfloat162float(a.gate[static_cast<int64_t>(q0 + qrow) * a.gate_stride + head]));
+        }
         __nv_bfloat16* op = a.out + (static_cast<int64_t>(q0 + qrow) * a.Hq + head) * DV;
 #pragma unroll 1
         for (int c = 0; c < DV / 32; ++c) {
@@ -487,7 +557,7 @@ bool make_map2(CUtensorMap* m, const void* base, int64_t tokens, int heads, int 
              CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
-template <int DQK, int DV, bool TAIL, bool WINDOW>
+template <int DQK, int DV, bool TAIL, bool WINDOW, bool SIGM = false>
 int launch2(const Args2& a, const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tkt,
             const CUtensorMap& tv, dim3 grid, cudaStream_t s) {
   using L = Lay<DQK, DV>;
@@ -496,7 +566,7 @@ int launch2(const Args2& a, const CUtensorMap& tq, const CUtensorMap& tk, const 
   int dev = 0;
   cudaGetDevice(&dev);
   if (dev < 0 || dev >= 64) return B200_ERR_UNSUPPORTED;
-  auto kern = prefill_umma2_kernel<DQK, DV, TAIL, WINDOW>;
+  auto kern = prefill_umma2_kernel<DQK, DV, TAIL, WINDOW, SIGM>;
   if (!configured[dev]) {
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, L::SMEM) != cudaSuccess)
       return B200_ERR_LAUNCH;
@@ -565,6 +635,49 @@ int prefill_umma2_launch(const void* q, const void* k, const void* v, void* out,
   if (Dqk == 128) return launch2<128, 128, false, false>(a, tq, tk, tkt, tv, grid, s);
   return tail ? launch2<192, 128, true, false>(a, tq, tk, tkt, tv, grid, s)
               : launch2<192, 128, false, false>(a, tq, tk, tkt, tv, grid, s);
+}
+
+// Sigmoid weights inside chunks of positions, with an output gate; head sizes 128 and 64.
+int prefill_umma2_sigmoid_tile_rows(int Hq, int Hkv, int Dqk, int Dv) {
+  return Hkv > 0 && Hq % Hkv == 0 && Dqk == Dv && (Dqk == 128 || Dqk == 64) ? ROWS : 0;
+}
+
+int prefill_umma2_sigmoid_launch(const void* q, const void* k, const void* v, void* out, int64_t q_stride, int64_t k_stride,
+                                 int64_t v_stride, int64_t total_q, int64_t total_k, const int32_t* cu_q, const int32_t* cu_k,
+                                 int num_seqs, int max_seqlen_q, int Hq, int Hkv, int Dqk, int Dv, float scale, const float* bias,
+                                 int chunk, const void* gate, int64_t gate_stride, const int32_t* plan, int plan_tile_rows,
+                                 int plan_capacity, int32_t* status, cudaStream_t s) {
+  if (prefill_umma2_sigmoid_tile_rows(Hq, Hkv, Dqk, Dv) == 0) return B200_ERR_UNSUPPORTED;
+  const int ntiles = (max_seqlen_q + ROWS - 1) / ROWS;
+  if (num_seqs > 65535 || ntiles > 65535 || Hq > 65535) return B200_ERR_UNSUPPORTED;
+  auto al = [](const void* p, int64_t stride) { return p != nullptr && aligned16(p) && (stride * 2) % 16 == 0; };
+  if (!al(q, q_stride) || !al(k, k_stride) || !al(v, v_stride) || !aligned16(out)) return B200_ERR_UNSUPPORTED;
+  Args2 a{};
+  a.out = static_cast<__nv_bfloat16*>(out);
+  a.cu_q = cu_q;
+  a.cu_k = cu_k;
+  a.Hq = Hq;
+  a.Hkv = Hkv;
+  a.ntiles_max = ntiles;
+  a.plan = (plan != nullptr && plan_tile_rows == ROWS && plan_capacity > 0 && plan_capacity <= 65535) ? plan : nullptr;
+  a.scale_log2 = scale * 1.4426950408889634f;
+  a.bias = bias;
+  a.chunk = chunk > 0 ? chunk : 2147483647;
+  a.gate = static_cast<const __nv_bfloat16*>(gate);
+  a.gate_stride = gate_stride;
+  a.status = status;
+  CUtensorMap tq, tk, tkt, tv;
+  memset(&tq, 0, sizeof(tq));
+  memset(&tk, 0, sizeof(tk));
+  memset(&tkt, 0, sizeof(tkt));
+  memset(&tv, 0, sizeof(tv));
+  if (!make_map2(&tq, q, total_q, Hq, Dqk, q_stride, BM) || !make_map2(&tk, k, total_k, Hkv, Dqk, k_stride, BN) ||
+      !make_map2(&tv, v, total_k, Hkv, Dv, v_stride, BN))
+    return B200_ERR_UNSUPPORTED;
+  dim3 grid(Hq, num_seqs, ntiles);
+  if (a.plan) grid = dim3(Hq, plan_capacity, 1);
+  return Dqk == 128 ? launch2<128, 128, false, false, true>(a, tq, tk, tkt, tv, grid, s)
+                    : launch2<64, 64, false, false, true>(a, tq, tk, tkt, tv, grid, s);
 }
 
 }  // namespace b200

@@ -4,8 +4,9 @@
 // elements lane, lane+32, ...; keys are visited in order with an fp32 online softmax.  Keys and
 // values come either from the packed k/v tensors of the step or, when a cached prefix exists,
 // from the paged pool through block_tables (bottom-right aligned causal mask).  The packed keys may come in two parts, the
-// second shared by all heads, and a query may see only the last `window` keys.
-#include "common.cuh"
+// second shared by all heads, and a query may see only the last `window` keys.  SIGM: the weights are sigmoid(scale q.k +
+// bias[head]), summed as they are over the keys of the query's chunk of positions, and rows leave through a gate.
+#include "sequences.cuh"
 
 namespace b200 {
 namespace {
@@ -32,13 +33,17 @@ struct PrefillArgs {
   int tail;
   int window;         // 0: none
   int32_t* status;
+  const float* bias;  // SIGM: [Hq]
+  int chunk;          // SIGM: positions per chunk, counted from the first key
+  const void* gate;   // SIGM: [tokens, Hq] or null
+  int64_t gate_stride;
 };
 
 constexpr int kWarps = 4;
 constexpr int kMaxPerLane = 8;    // head dims <= 256
 constexpr int kWidePerLane = 32;  // head dims <= 1024
 
-template <typename T, int kMaxPerLane>
+template <typename T, int kMaxPerLane, bool SIGM>
 __global__ void __launch_bounds__(kWarps * 32) prefill_simple_kernel(const PrefillArgs a) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int s = blockIdx.z, head = blockIdx.y;
@@ -59,7 +64,8 @@ __global__ void __launch_bounds__(kWarps * 32) prefill_simple_kernel(const Prefi
   }
   float m = -INFINITY, l = 0.f;
   const int Dh = a.Dqk - a.tail;
-  for (int j = a.window > 0 ? max(nkeys - a.window, 0) : 0; j < nkeys; ++j) {
+  const int first = SIGM ? (nkeys - 1) / a.chunk * a.chunk : a.window > 0 ? max(nkeys - a.window, 0) : 0;
+  for (int j = first; j < nkeys; ++j) {
     const T* kp;
     const T* kt = nullptr;
     const T* vp;
@@ -90,7 +96,17 @@ __global__ void __launch_bounds__(kWarps * 32) prefill_simple_kernel(const Prefi
       if (d < Dh) dot += qv[i] * to_float<T>(kp[d]);
       else if (d < a.Dqk) dot += qv[i] * to_float<T>(kt[d - Dh]);
     }
-    dot = warp_sum(dot) * a.scale_log2;
+    dot = warp_sum(dot);
+    if constexpr (SIGM) {
+      const float p = sigmoid_f(dot * a.scale_log2 + a.bias[head]);
+#pragma unroll
+      for (int i = 0; i < kMaxPerLane; ++i) {
+        const int d = lane + 32 * i;
+        if (d < a.Dv) acc[i] += p * to_float<T>(vp[d]);
+      }
+      continue;
+    }
+    dot *= a.scale_log2;
     const float mn = fmaxf(m, dot);
     const float al = exp2f(m - mn), pw = exp2f(dot - mn);
     l = l * al + pw;
@@ -103,7 +119,9 @@ __global__ void __launch_bounds__(kWarps * 32) prefill_simple_kernel(const Prefi
   }
   T* op = static_cast<T*>(a.out) + (static_cast<int64_t>(q0 + qi) * a.Hq + head) * a.Dv;
   if (a.sink != nullptr && nkeys > 0) l += exp2f(a.sink[head] * 1.4426950408889634f - m);
-  const float inv = l > 0.f ? 1.f / l : 0.f;
+  float inv = l > 0.f ? 1.f / l : 0.f;
+  if constexpr (SIGM)
+    inv = a.gate ? sigmoid_f(to_float<T>(static_cast<const T*>(a.gate)[static_cast<int64_t>(q0 + qi) * a.gate_stride + head])) : 1.f;
 #pragma unroll
   for (int i = 0; i < kMaxPerLane; ++i) {
     const int d = lane + 32 * i;
@@ -146,6 +164,19 @@ int prefill_mma_general_launch(const void* q, const void* k, const void* v, void
                                int plan_capacity, int32_t* status, cudaStream_t s, const void* k_tail, int64_t k_tail_stride,
                                int tail, const float* sink, int window);
 
+// sigmoid weights inside chunks: tcgen05 at head sizes 128 and 64 (prefill_umma2.cu), mma.sync at the general ones (prefill_mma.cu)
+int prefill_umma2_sigmoid_tile_rows(int Hq, int Hkv, int Dqk, int Dv);
+int prefill_umma2_sigmoid_launch(const void* q, const void* k, const void* v, void* out, int64_t q_stride, int64_t k_stride,
+                                 int64_t v_stride, int64_t total_q, int64_t total_k, const int32_t* cu_q, const int32_t* cu_k,
+                                 int num_seqs, int max_seqlen_q, int Hq, int Hkv, int Dqk, int Dv, float scale, const float* bias,
+                                 int chunk, const void* gate, int64_t gate_stride, const int32_t* plan, int plan_tile_rows,
+                                 int plan_capacity, int32_t* status, cudaStream_t s);
+int prefill_mma_sigmoid_launch(const void* q, const void* k, const void* v, void* out, int64_t q_stride, int64_t k_stride,
+                               int64_t v_stride, const int32_t* cu_q, const int32_t* cu_k, int num_seqs, int max_seqlen_q,
+                               int Hq, int Hkv, int Dqk, int Dv, float scale, const float* bias, int chunk, const void* gate,
+                               int64_t gate_stride, const int32_t* plan, int plan_tile_rows, int plan_capacity, int32_t* status,
+                               cudaStream_t s);
+
 // tcgen05 path for a paged prefix (prefill_umma.cu): head_dim 128, even group size, two heads per CTA
 int prefill_umma_launch(const void* q, const void* k, const void* v, void* out, int64_t q_stride,
                         int64_t k_stride, int64_t v_stride, int64_t total_q, int64_t total_k,
@@ -172,17 +203,18 @@ extern "C" int32_t b200_prefill_tile_rows(int32_t num_q_heads, int32_t num_kv_he
 
 namespace b200 {
 namespace {
+template <bool SIGM = false>
 int simple_launch(const PrefillArgs& a, int max_seqlen_q, int32_t dtype, cudaStream_t s) {
   const int widest = a.Dqk > a.Dv ? a.Dqk : a.Dv;
   if (widest > kWidePerLane * 32 || a.num_seqs > 65535 || a.Hq > 65535) return B200_ERR_UNSUPPORTED;
   const dim3 grid((max_seqlen_q + kWarps - 1) / kWarps, a.Hq, a.num_seqs);
   const bool wide = widest > kMaxPerLane * 32;
   if (dtype == B200_DTYPE_F32) {
-    if (wide) prefill_simple_kernel<float, kWidePerLane><<<grid, kWarps * 32, 0, s>>>(a);
-    else prefill_simple_kernel<float, kMaxPerLane><<<grid, kWarps * 32, 0, s>>>(a);
+    if (wide) prefill_simple_kernel<float, kWidePerLane, SIGM><<<grid, kWarps * 32, 0, s>>>(a);
+    else prefill_simple_kernel<float, kMaxPerLane, SIGM><<<grid, kWarps * 32, 0, s>>>(a);
   } else {
-    if (wide) prefill_simple_kernel<__nv_bfloat16, kWidePerLane><<<grid, kWarps * 32, 0, s>>>(a);
-    else prefill_simple_kernel<__nv_bfloat16, kMaxPerLane><<<grid, kWarps * 32, 0, s>>>(a);
+    if (wide) prefill_simple_kernel<__nv_bfloat16, kWidePerLane, SIGM><<<grid, kWarps * 32, 0, s>>>(a);
+    else prefill_simple_kernel<__nv_bfloat16, kMaxPerLane, SIGM><<<grid, kWarps * 32, 0, s>>>(a);
   }
   return launch_result();
 }
@@ -417,4 +449,63 @@ extern "C" int b200_prefill_varlen_window(const void* q, const void* k_head, con
   a.window = window;
   a.status = status;
   return simple_launch(a, max_seqlen_q, dtype, s);
+}
+
+extern "C" int32_t b200_sigmoid_attention_tile_rows(int32_t num_q_heads, int32_t num_kv_heads, int32_t head_dim_qk,
+                                                    int32_t head_dim_v, int32_t dtype) {
+  if (dtype != B200_DTYPE_BF16 || num_kv_heads <= 0 || num_q_heads % num_kv_heads != 0) return 0;
+  if (const int r = b200::prefill_umma2_sigmoid_tile_rows(num_q_heads, num_kv_heads, head_dim_qk, head_dim_v)) return r;
+  return b200::prefill_mma_general_shape(head_dim_qk, head_dim_v, 0) ? 64 : 0;
+}
+
+extern "C" int b200_sigmoid_attention(const void* q, const void* k, const void* v, void* out, int64_t q_token_stride,
+                                      int64_t k_token_stride, int64_t v_token_stride, int64_t total_q_tokens,
+                                      int64_t total_k_tokens, const int32_t* cu_seqlens_q, const int32_t* cu_seqlens_k,
+                                      int32_t num_seqs, int32_t max_seqlen_q, int32_t num_q_heads, int32_t num_kv_heads,
+                                      int32_t head_dim_qk, int32_t head_dim_v, float scale, const float* bias, int32_t chunk,
+                                      const void* gate, int64_t gate_token_stride, const int32_t* plan, int32_t plan_tile_rows,
+                                      int32_t plan_capacity, int32_t dtype, int32_t* status, void* stream) {
+  using namespace b200;
+  if (num_seqs < 0 || max_seqlen_q < 0 || num_q_heads <= 0 || num_kv_heads <= 0 || num_q_heads % num_kv_heads || head_dim_qk <= 0 ||
+      head_dim_v <= 0 || chunk < 0)
+    return B200_ERR_ARG;
+  if (dtype != B200_DTYPE_F32 && dtype != B200_DTYPE_BF16) return B200_ERR_UNSUPPORTED;
+  if (num_seqs == 0 || max_seqlen_q == 0) return B200_OK;
+  if (!q || !k || !v || !out || !cu_seqlens_q || !cu_seqlens_k || !bias) return B200_ERR_ARG;
+  if (total_q_tokens <= 0 || total_k_tokens <= 0) return B200_ERR_ARG;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (dtype == B200_DTYPE_BF16) {
+    const int rc2 = prefill_umma2_sigmoid_launch(q, k, v, out, q_token_stride, k_token_stride, v_token_stride, total_q_tokens,
+                                                 total_k_tokens, cu_seqlens_q, cu_seqlens_k, num_seqs, max_seqlen_q, num_q_heads,
+                                                 num_kv_heads, head_dim_qk, head_dim_v, scale, bias, chunk, gate,
+                                                 gate_token_stride, plan, plan_tile_rows, plan_capacity, status, s);
+    if (rc2 != B200_ERR_UNSUPPORTED) return rc2;
+    const int rc = prefill_mma_sigmoid_launch(q, k, v, out, q_token_stride, k_token_stride, v_token_stride, cu_seqlens_q,
+                                              cu_seqlens_k, num_seqs, max_seqlen_q, num_q_heads, num_kv_heads, head_dim_qk,
+                                              head_dim_v, scale, bias, chunk, gate, gate_token_stride, plan, plan_tile_rows,
+                                              plan_capacity, status, s);
+    if (rc != B200_ERR_UNSUPPORTED) return rc;
+  }
+  PrefillArgs a{};
+  a.q = q;
+  a.k = k;
+  a.v = v;
+  a.out = out;
+  a.q_stride = q_token_stride;
+  a.k_stride = k_token_stride;
+  a.v_stride = v_token_stride;
+  a.cu_q = cu_seqlens_q;
+  a.cu_k = cu_seqlens_k;
+  a.num_seqs = num_seqs;
+  a.Hq = num_q_heads;
+  a.Hkv = num_kv_heads;
+  a.Dqk = head_dim_qk;
+  a.Dv = head_dim_v;
+  a.scale_log2 = scale;       // the sigmoid takes natural exponents
+  a.bias = bias;
+  a.chunk = chunk > 0 ? chunk : 2147483647;
+  a.gate = gate;
+  a.gate_stride = gate_token_stride;
+  a.status = status;
+  return simple_launch<true>(a, max_seqlen_q, dtype, s);
 }

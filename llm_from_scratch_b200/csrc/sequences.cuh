@@ -36,7 +36,7 @@ __device__ __forceinline__ bool sequence_info(const Args& a, int s, SeqInfo* r) 
 }
 
 // Segment number -> (sequence, index within it) when every sequence of n is cut into segments of seg_len tokens;
-// false: no such segment.  Every thread of the CTA calls it.
+// false: no such segment (index: how many segments behind the last one).  Every thread of the CTA calls it.
 __device__ __forceinline__ bool find_segment(const int32_t* cu_q, int n, int seg_len, int number, int* seq, int* index) {
   __shared__ int found[2];
   if (threadIdx.x < 32) {
@@ -62,13 +62,59 @@ __device__ __forceinline__ bool find_segment(const int32_t* cu_q, int n, int seg
     }
     if (lane == 0) {
       found[0] = hit_seq;
-      found[1] = hit_idx;
+      found[1] = hit_seq < 0 ? left : hit_idx;
     }
   }
   __syncthreads();
   *seq = found[0];
   *index = found[1];
   return found[0] >= 0;
+}
+
+// The tokens of one segment, for kernels that also serve the padding rows behind the last sequence: those form segments of
+// their own, in no sequence.
+struct Segment {
+  int64_t first;     // row of its first token
+  int count;
+  int index;         // segments of the sequence before it
+  int len;           // tokens of the sequence in this step
+  int64_t pos0;      // position of the sequence's first token in this step
+  int64_t slot;      // of its state, -1: none
+};
+// The CTA's segment; false: it has none.  ``Args`` as for sequence_info, with n sequences over T rows.  With ctx_lens row i is
+// sequence i, one token; else the grid holds T / seg_len + n + 1 CTAs.  Every thread of the CTA calls it.
+template <typename Args>
+__device__ __forceinline__ bool segment_of(const Args& a, int seg_len, Segment* r) {
+  if (a.cu_q == nullptr) {
+    r->first = blockIdx.x;
+    r->count = r->len = 1;
+    r->index = 0;
+    r->pos0 = a.ctx_lens ? max(a.ctx_lens[blockIdx.x] - 1, static_cast<int64_t>(0)) : 0;
+    r->slot = a.ctx_lens && a.slots && a.ctx_lens[blockIdx.x] > 0 ? a.slots[blockIdx.x] : -1;
+  } else {
+    int seq;
+    if (find_segment(a.cu_q, a.n, seg_len, blockIdx.x, &seq, &r->index)) {
+      const int q0 = a.cu_q[seq];
+      r->len = a.cu_q[seq + 1] - q0;
+      r->first = q0 + static_cast<int64_t>(r->index) * seg_len;
+      r->count = min(seg_len, r->len - r->index * seg_len);
+      r->pos0 = (a.cu_k[seq + 1] - a.cu_k[seq]) - r->len;
+      r->slot = a.slots ? a.slots[seq] : -1;
+    } else {
+      r->first = a.cu_q[a.n] + static_cast<int64_t>(r->index) * seg_len;
+      if (r->first >= a.T) return false;
+      r->count = static_cast<int>(a.T - r->first < seg_len ? a.T - r->first : seg_len);
+      r->len = r->count;
+      r->index = 0;
+      r->pos0 = 0;
+      r->slot = -1;
+    }
+  }
+  if (r->slot >= a.num_slots) {
+    if (threadIdx.x == 0) report(a.status, B200_ERR_BOUNDS);
+    r->slot = -1;
+  }
+  return true;
 }
 
 // Number of the first segment of sequence seq.  Threads of warp 0 call it.

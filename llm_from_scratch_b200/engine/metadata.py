@@ -31,9 +31,9 @@ class StepMetadata:
     last_token_index: Optional[np.ndarray] = None  # int64 [n]  row of each sequence's last token
     state_slots: Optional[np.ndarray] = None    # int64 [n]  recurrent-state slot of every sequence
 
-    def step_parts(self, windows: tuple = ()) -> "StepParts":
+    def step_parts(self, windows: tuple = (), chunks: tuple = ()) -> "StepParts":
         """A ragged step in two parts: the leading sequences that bring one token, and the others.  ``windows``: sliding
-        windows for which the ends of the others' contexts are worked out."""
+        windows, and ``chunks``: chunk sizes for which the ends of the others' contexts are worked out."""
         q, k = np.diff(self.cu_seqlens_q), np.diff(self.cu_seqlens_k)
         longer = np.nonzero(q != 1)[0]
         n1 = int(longer[0]) if longer.size else len(q)
@@ -41,12 +41,14 @@ class StepMetadata:
         return StepParts(num_single=n1, single_lens=single.astype(np.int64),
                          portion_cu_k=np.concatenate([[0], np.cumsum(k)]).astype(np.int32),
                          max_seqlen_q=int(q.max(initial=0)), max_seqlen_k=int(k.max(initial=0)),
-                         has_prefix=bool((q < k).any()), ranges={w: KeyRangeArrays.of(q, np.minimum(k, q + w - 1)) for w in windows})
+                         has_prefix=bool((q < k).any()), ranges={w: KeyRangeArrays.of(q, np.minimum(k, q + w - 1)) for w in windows},
+                         chunk_ranges={c: KeyRangeArrays.of(q, k - (k - q) // c * c) for c in chunks})
 
 
 @dataclass
 class KeyRangeArrays:
-    """The last keys of every context, as many as a window reaches from the portion's first token."""
+    """The last keys of every context: as many as a window reaches from the portion's first token, or from the start of that
+    token's chunk on."""
     cu_k: np.ndarray                            # int32 [n + 1]
     max_seqlen_k: int
     has_prefix: bool
@@ -65,6 +67,7 @@ class StepParts:
     max_seqlen_k: int
     has_prefix: bool                            # some of their contexts began in an earlier step
     ranges: dict = field(default_factory=dict)  # window -> KeyRangeArrays
+    chunk_ranges: dict = field(default_factory=dict)  # chunk size -> KeyRangeArrays
 
 
 def block_table_array(s: Sequence) -> np.ndarray:

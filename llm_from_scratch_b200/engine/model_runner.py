@@ -106,6 +106,7 @@ class ModelRunner:
         self.splits_steps = getattr(model, "splits_steps", False)
         # sliding windows of its layers: portions then need only the ends of their contexts
         self.attention_windows = tuple(getattr(model, "attention_windows", ()))
+        self.attention_chunks = tuple(getattr(model, "attention_chunks", ()))     # the same for chunks of positions
         self.num_state_slots = self.max_num_seqs if self.recurrent_state else 0
         if self.mixed_batches:      # their matrix products accumulate in fp32 from end to end
             torch.backends.cuda.matmul.allow_bf16_reduced_precision_reduction = False
@@ -194,11 +195,13 @@ class ModelRunner:
             arrays["input_ids"] = np.concatenate([m.input_ids, np.zeros(pad, dtype=m.input_ids.dtype)])
             arrays["positions"] = np.concatenate([m.positions, np.zeros(pad, dtype=m.positions.dtype)])
             arrays["slot_mapping"] = np.concatenate([m.slot_mapping, np.full(pad, -1, dtype=m.slot_mapping.dtype)])
-        parts = m.step_parts(self.attention_windows) if self.splits_steps and m.is_prefill else None
+        parts = m.step_parts(self.attention_windows, self.attention_chunks) if self.splits_steps and m.is_prefill else None
         if parts is not None:
             arrays["single_lens"], arrays["portion_cu_k"] = parts.single_lens, parts.portion_cu_k
             for w, r in parts.ranges.items():
                 arrays[f"portion_cu_k.{w}"] = r.cu_k
+            for c, r in parts.chunk_ranges.items():
+                arrays[f"portion_cu_k.chunk{c}"] = r.cu_k
         t = self.staging.upload(arrays)
         plan = None
         if m.is_prefill and self.prefill_tile_rows and m.max_seqlen_q <= 4096 * self.prefill_tile_rows:
@@ -223,11 +226,12 @@ class ModelRunner:
         if n1:
             ctx.singles = Singles(n1, t["single_lens"], ctx.block_tables[:n1], part(slots, 0, n1))
         if parts.max_seqlen_q:
+            key_range = lambda name, r: KeyRange(t[f"portion_cu_k.{name}"], r.max_seqlen_k, int(r.cu_k[-1]), r.has_prefix)
             ctx.portions = Portions(num_tokens, ctx.cu_seqlens_q[n1:], t["portion_cu_k"], parts.max_seqlen_q,
                                     parts.max_seqlen_k, int(parts.portion_cu_k[-1]), parts.has_prefix,
                                     ctx.block_tables[n1:], part(slots, n1),
-                                    ranges={w: KeyRange(t[f"portion_cu_k.{w}"], r.max_seqlen_k, int(r.cu_k[-1]), r.has_prefix)
-                                            for w, r in parts.ranges.items()})
+                                    ranges={w: key_range(w, r) for w, r in parts.ranges.items()},
+                                    chunk_ranges={c: key_range(f"chunk{c}", r) for c, r in parts.chunk_ranges.items()})
 
     def prepare_prefill(self, seqs: list[Sequence]) -> torch.Tensor:
         return self._publish(md.prepare_prefill(seqs, self.block_size, tables_always=self.mixed_batches))

@@ -7,9 +7,10 @@ from .registry import ModelFamily, build_model, family_of, init_weights, resolve
 from .nabalix import NabalixConfig, NabalixLM
 from .taminex import TaminexConfig, TaminexLM
 from .meresun import MeresunConfig, MeresunLM
+from .sodonex import SodonexConfig, SodonexLM
 
 registry.register(ModelFamily(registry.DEFAULT_FAMILY, ModelConfig, EngineTransformerLM, init_reference_order))
 
 __all__ = ["ModelConfig", "init_reference_order", "EngineTransformerLM", "ModelFamily", "build_model", "family_of",
            "init_weights", "resolve_config", "NabalixConfig", "NabalixLM", "TaminexConfig", "TaminexLM",
-           "MeresunConfig", "MeresunLM"]
+           "MeresunConfig", "MeresunLM", "SodonexConfig", "SodonexLM"]

@@ -479,34 +479,67 @@ class PolyNormMLP(nn.Module):
         return (F.linear(ops.poly_norm(up, self.coef, self.eps), self.w_down),)
 
 
-class GroupedMoE(nn.Module):
-    """Clamped GLU experts behind a sigmoid router with a choice correction and groups of experts.  Returns the chosen
-    experts' output rows, their weights and where a token's rows are; the weighted sum belongs to the residual update."""
+class RoutedExperts(nn.Module):
+    """Feed-forwards of which a router picks some per token.  Returns the chosen experts' output rows, their weights and where
+    a token's rows are; the weighted sum belongs to the residual update.  A kind of experts says how it routes (``route``), what
+    its first map does (``first``) and the same activation behind a plain product (``activation``)."""
 
     # average rows per expert above which bf16 goes to the library's grouped GEMM (see transformer.MoE)
     own_gemm_max_rows_per_expert = 256
 
-    def __init__(self, p: Params, d_model: int, d_ff: int, experts: int, top: int, groups: int, keep: int, limit: float,
-                 slope: float = 1.702):
+    def __init__(self, p: Params, d_model: int, d_ff: int, experts: int, maps_in: tuple[str, ...]):
         super().__init__()
-        self.top, self.groups, self.keep, self.limit, self.slope = top, groups, keep, limit, slope
-        self.projections = []
         self.router = p.lin("router", (experts, d_model))
-        self.correction = p.f32("correction", (experts,))
-        self.w_in = torch.stack([torch.cat([p.lin(f"e{e}.gate", (d_ff, d_model)), p.lin(f"e{e}.up", (d_ff, d_model))])
-                                 for e in range(experts)])
+        self.w_in = torch.stack([torch.cat([p.lin(f"e{e}.{m}", (d_ff, d_model)) for m in maps_in]) for e in range(experts)])
         self.w_down = torch.stack([p.lin(f"e{e}.down", (d_model, d_ff)) for e in range(experts)])
         self.library = p.dtype == torch.bfloat16 and d_model % 8 == 0 and d_ff % 8 == 0
 
     def forward(self, h):
         z = F.linear(h, self.router) if h.dtype == torch.float32 else torch.mm(h, self.router.t(), out_dtype=torch.float32)
-        tok, weight, offs, slot = ops.moe_group_route(z, self.correction, self.top, self.groups, self.keep)
+        tok, weight, offs, slot = self.route(z)
         xs = h.index_select(0, tok)
         if self.library and tok.numel() > self.own_gemm_max_rows_per_expert * self.router.shape[0]:
-            act = ops.clamped_glu(torch._grouped_mm(xs, self.w_in.transpose(1, 2), offs=offs), self.limit, self.slope)
+            act = self.activation(torch._grouped_mm(xs, self.w_in.transpose(1, 2), offs=offs))
             return torch._grouped_mm(act, self.w_down.transpose(1, 2), offs=offs), weight, slot
-        act = ops.moe_grouped_linear(xs, self.w_in, offs, glu=(self.limit, self.slope), early_launch=True)
-        return ops.moe_grouped_linear(act, self.w_down, offs, early_launch=True), weight, slot
+        return ops.moe_grouped_linear(self.first(xs, offs), self.w_down, offs, early_launch=True), weight, slot
+
+
+class GroupedMoE(RoutedExperts):
+    """Clamped GLU experts behind a sigmoid router with a choice correction and groups of experts."""
+
+    def __init__(self, p: Params, d_model: int, d_ff: int, experts: int, top: int, groups: int, keep: int, limit: float,
+                 slope: float = 1.702):
+        super().__init__(p, d_model, d_ff, experts, ("gate", "up"))
+        self.top, self.groups, self.keep, self.limit, self.slope = top, groups, keep, limit, slope
+        self.projections = []
+        self.correction = p.f32("correction", (experts,))
+
+    def route(self, z):
+        return ops.moe_group_route(z, self.correction, self.top, self.groups, self.keep)
+
+    def first(self, xs, offs):
+        return ops.moe_grouped_linear(xs, self.w_in, offs, glu=(self.limit, self.slope), early_launch=True)
+
+    def activation(self, h):
+        return ops.clamped_glu(h, self.limit, self.slope)
+
+
+class SoftmaxMoE(RoutedExperts):
+    """Squared-ReLU experts behind a router with a bias; the weights are the softmax over the chosen logits."""
+
+    def __init__(self, p: Params, d_model: int, d_ff: int, experts: int, top: int):
+        super().__init__(p, d_model, d_ff, experts, ("up",))
+        self.top = top
+        self.router_bias = p.f32("router.b", (experts,))
+
+    def route(self, z):
+        return ops.moe_softmax_route(z, self.router_bias, self.top)
+
+    def first(self, xs, offs):
+        return ops.moe_grouped_linear(xs, self.w_in, offs, squared_relu=True, early_launch=True)
+
+    def activation(self, h):
+        return ops.squared_relu(h)
 
 
 class TokenInput(nn.Module):
@@ -549,3 +582,77 @@ class GatedSublayers(nn.Module):
             return ops.gated_residual(x, mix(), gates[0])
         y, (f, *choice) = side_by_side(mix, lambda: self.mlp(h, *into_mlp), ctx, h.device)
         return ops.gated_residual(x, y, gates[0], f, gates[1], *choice)
+
+
+# ------------------------------------------------------------------------------------------------
+# tokens that look at the ones just before them: shifted inputs, convolved queries and keys
+# ------------------------------------------------------------------------------------------------
+class TokenShift(nn.Module):
+    """Mixes what a mixer reads with the previous token's, channel by channel; the residual kernel does it on the way
+    (``ops.shift_residual``), the last token of every sequence lives in the runner's slot pool."""
+
+    def __init__(self, p: Params, d_model: int):
+        super().__init__()
+        self.weight = p.f32("shift", (d_model,))
+        self.state = torch.empty(0)
+
+    def cache_needs(self):
+        return [("slot", "state", (self.weight.numel(),))]
+
+
+class SigmoidAttention(nn.Module):
+    """Grouped-query attention whose weights are sigmoid(scale q.k + bias of the head), summed without a normalisation over the
+    keys of the query's chunk of positions (0: no chunks).  Queries and keys pass a short causal convolution, then a norm over
+    the whole projection and a rotation of channel halves; the values are the convolved keys.  A gate per head follows."""
+
+    def __init__(self, p: Params, d_model: int, heads: int, kv_heads: int, dim: int, taps: int, scale: float, rot_dims: int,
+                 rot_base: float, chunk: int, eps: float):
+        super().__init__()
+        self.heads, self.kv_heads, self.dim, self.taps = heads, kv_heads, dim, taps
+        self.scale, self.chunk, self.eps = scale, chunk, eps
+        sizes = {"q": heads * dim, "k": kv_heads * dim}
+        gate = p.lin("g", (heads, d_model))
+        self.project = FusedProjection([p.lin(n, (w, d_model)) for n, w in sizes.items()] + [gate],
+                                       [p.lin(n + ".b", (w,)) for n, w in sizes.items()] + [gate.new_zeros(heads)])
+        self.conv_q, self.conv_k = (p.f32(n + ".conv", (w, taps)).t().contiguous() for n, w in sizes.items())
+        self.q_norm, self.k_norm = (p.f32(n + ".norm", (w,)) for n, w in sizes.items())
+        self.bias = p.f32("pb", (heads,))
+        self.freq = ops.rotary_frequencies(rot_base, rot_dims, p.device)
+        self.w_o, self.b_o = p.lin("o", (d_model, heads * dim)), p.lin("o.b", (d_model,))
+        self.k_cache = self.v_cache = torch.empty(0)
+        self.conv_ring = None                              # one tap: nothing is carried over
+
+    def cache_needs(self):
+        row = (self.kv_heads, self.dim)
+        needs = [("paged", "k_cache", row), ("paged", "v_cache", row)]
+        if self.taps > 1:
+            needs.append(("slot", "conv_ring", (self.taps - 1, (self.heads + self.kv_heads) * self.dim)))
+        return needs
+
+    def tile_rows(self, dtype) -> int:
+        """Query rows per tile of the kernel that serves this layer's portions; 0: a general one without tile lists."""
+        return ops.sigmoid_attention_tile_rows(self.heads, self.kv_heads, self.dim, self.dim, dtype)
+
+    def _portions(self, q, k, v, gate, s, out):
+        keys, cu_k = s.keys(chunk=self.chunk), s.cu_seqlens_q
+        if keys.has_prefix:
+            cu_k = keys.cu_seqlens_k
+            k, v = (ops.gather_rows(c.flatten(2), s.block_tables, cu_k, keys.max_seqlen_k, keys.total_k,
+                                    s.cu_seqlens_k).unflatten(1, (self.kv_heads, self.dim)) for c in (self.k_cache, self.v_cache))
+        ops.sigmoid_attention(q, k, v, s.cu_seqlens_q, cu_k, s.max_seqlen_q, self.scale, self.bias, self.chunk, gate, out=out,
+                              plan=s.plan(self.tile_rows(q.dtype)))
+
+    def forward(self, h, ctx, positions, rows):
+        q, k, gate = self.project(h)
+        q, k, v = ops.conv_norm_rope_store(q, k, self.conv_q, self.conv_k, self.conv_ring, rows, self.q_norm, self.k_norm, self.eps,
+                                           self.freq, positions, self.k_cache, self.v_cache, ctx.slot_mapping,
+                                           packed=ctx.portions is not None)
+        o = _step_output(h, self.heads * self.dim, ctx)
+        o3 = o.view(-1, self.heads, self.dim)
+        if ctx.singles is not None:
+            s = ctx.singles
+            ops.sigmoid_decode(q[:s.rows], self.k_cache, self.v_cache, s.block_tables, s.context_lens, self.scale, self.bias,
+                               self.chunk, gate[:s.rows], out=o3[:s.rows])
+        if ctx.portions is not None:
+            self._portions(q, k, v, gate, ctx.portions, o3)
+        return F.linear(o, self.w_o, self.b_o)

@@ -1373,19 +1373,226 @@ def moe_group_route(logits: torch.Tensor, correction: torch.Tensor, top: int, gr
 
 
 def moe_grouped_linear(x: torch.Tensor, w: torch.Tensor, expert_offsets: torch.Tensor,
-                       glu: tuple[float, float] | None = None, early_launch: bool = False) -> torch.Tensor:
+                       glu: tuple[float, float] | None = None, early_launch: bool = False,
+                       squared_relu: bool = False) -> torch.Tensor:
     """Rows of x [R, k] grouped by expert times the expert's weight w [E, n, k] -> [R, n], any size, bf16 or fp32.  ``glu``
-    (limit, slope): w is [E, 2 n, k] = [gate | up] and the clamped gated unit of the two comes back [R, n]."""
+    (limit, slope): w is [E, 2 n, k] = [gate | up] and the clamped gated unit of the two comes back [R, n]; ``squared_relu``:
+    max(., 0)^2 of the result."""
     dev = _cuda(x, w, expert_offsets)
     (R, k), (E, n, k2) = x.shape, w.shape
     if x.dtype != w.dtype or k != k2 or not x.is_contiguous() or not w.is_contiguous() or expert_offsets.dtype != torch.int32 \
-            or expert_offsets.numel() != E or (glu is not None and n % 2):
+            or expert_offsets.numel() != E or (glu is not None and (n % 2 or squared_relu)):
         raise ValueError("x [R, k] and w [E, n, k] must be contiguous, of one dtype; expert_offsets int32 [E]")
     n_out = n // 2 if glu is not None else n
     limit, slope = glu if glu is not None else (0.0, 0.0)
     out = torch.empty(R, n_out, dtype=x.dtype, device=dev)
     check(lib.b200_moe_grouped_linear(x.data_ptr(), w.data_ptr(), out.data_ptr(), expert_offsets.data_ptr(), R, E, n_out, k,
-                                      0 if glu is None else 1, float(limit), float(slope),
+                                      1 if glu is not None else 2 if squared_relu else 0, float(limit), float(slope),
                                       MOE_GEMM_EARLY_LAUNCH if early_launch else 0, _dt(x), status_word(dev).data_ptr(),
                                       _stream()), "moe_grouped_linear")
     return out
+
+
+# ------------------------------------------------------------------------------------------------
+# token shift, convolved queries and keys, sigmoid attention in chunks, softmax over the chosen experts
+# ------------------------------------------------------------------------------------------------
+@dataclass
+class StepRows:
+    """Which sequence the rows of a step belong to, for kernels that carry state from token to token: ragged portions
+    (``cu_seqlens_q`` / ``cu_seqlens_k``), or row i = sequence i with ``context_lens`` tokens."""
+    state_slots: torch.Tensor                     # int64 [n], -1 = no state
+    cu_seqlens_q: torch.Tensor | None = None      # int32 [n + 1]
+    cu_seqlens_k: torch.Tensor | None = None
+    context_lens: torch.Tensor | None = None      # int64 [n]
+
+    @classmethod
+    def of(cls, ctx) -> "StepRows":
+        if ctx.is_prefill:
+            return cls(ctx.state_slots, ctx.cu_seqlens_q, ctx.cu_seqlens_k)
+        return cls(ctx.state_slots, context_lens=ctx.context_lens)
+
+    def check(self, T: int) -> int:
+        """Number of sequences."""
+        ragged = self.cu_seqlens_q is not None
+        n = self.cu_seqlens_q.numel() - 1 if ragged else T
+        if self.state_slots.dtype != torch.int64 or self.state_slots.numel() < n or not self.state_slots.is_contiguous():
+            raise ValueError("state_slots must be contiguous int64 with one entry per sequence")
+        if ragged:
+            if self.cu_seqlens_q.dtype != torch.int32 or self.cu_seqlens_k is None or self.cu_seqlens_k.dtype != torch.int32 \
+                    or self.cu_seqlens_k.numel() != n + 1:
+                raise ValueError("cu_seqlens must be int32 tensors of the same length")
+        elif self.context_lens is None or self.context_lens.dtype != torch.int64 or self.context_lens.numel() != T \
+                or not self.context_lens.is_contiguous():
+            raise ValueError("context_lens must be contiguous int64 with one entry per row")
+        return n
+
+
+def shift_residual(x: torch.Tensor | None, eps: float, dtype: torch.dtype, *, x_out: torch.Tensor | None = None,
+                   tokens: torch.Tensor | None = None, embed: torch.Tensor | None = None, embed_scale: float = 1.0,
+                   y: torch.Tensor | None = None, gain: float = 1.0, row_weight: torch.Tensor | None = None,
+                   slot_to_row: torch.Tensor | None = None, shift: torch.Tensor | None = None,
+                   state: torch.Tensor | None = None, rows: StepRows | None = None,
+                   final_gain: float | None = None) -> torch.Tensor:
+    """One boundary of a residual x [T, d] fp32 (``b200_shift_residual``): x' = x + gain y / rms(y), with y dense [T, d] or
+    the expert rows [T * top, d] behind ``slot_to_row`` / ``row_weight`` [T, top], or x' = the scaled embedding rows.  x' goes to
+    ``x_out``.  Returns x' in ``dtype``, mixed with the previous token's (``shift`` [d], ``state`` [slots, d], ``rows``), or
+    normed with one number (``final_gain``)."""
+    dev = _cuda(x, x_out, tokens, embed, y, row_weight, slot_to_row, shift, state)
+    T, d = (tokens.numel(), embed.shape[1]) if embed is not None else x.shape
+    for name, t in (("x", x if embed is None else None), ("x_out", x_out)):
+        if t is not None and (t.dtype != torch.float32 or t.shape != (T, d) or not t.is_contiguous()):
+            raise ValueError(f"{name} must be a contiguous fp32 [T, d] tensor")
+    if embed is not None:
+        if embed.dtype != dtype or not embed.is_contiguous():
+            raise ValueError("embed must be contiguous [vocab, d] in the activation dtype")
+        _tokens("tokens", tokens, T)
+    top = slot_to_row.shape[1] if slot_to_row is not None else 0
+    if y is not None and (y.shape != ((T * top) if top else T, d) or y.dtype != dtype or not y.is_contiguous()):
+        raise ValueError("y must be contiguous [T, d] (or [T * top, d]) in the activation dtype")
+    if top and (y is None or row_weight is None or row_weight.dtype != torch.float32 or row_weight.shape != (T, top)
+                or slot_to_row.dtype != torch.int32 or not row_weight.is_contiguous() or not slot_to_row.is_contiguous()):
+        raise ValueError("row_weight must be fp32 and slot_to_row int32, both contiguous [T, top]")
+    n = 0
+    if shift is not None:
+        _f32vec("shift", shift, d)
+        if state is None or state.dtype != torch.float32 or state.dim() != 2 or state.shape[1] != d or not state.is_contiguous():
+            raise ValueError("state must be contiguous fp32 [slots, d]")
+        if x is not None and x_out is not None and x.data_ptr() == x_out.data_ptr() and embed is None:
+            raise ValueError("with a shift the residual cannot be updated in place")
+        n = rows.check(T)
+    h = torch.empty(T, d, dtype=dtype, device=dev)
+    check(lib.b200_shift_residual(
+        _ptr(x), _ptr(x_out), _ptr(tokens) if embed is not None else None, _ptr(embed), embed.shape[0] if embed is not None else 0,
+        float(embed_scale), _ptr(y), _ptr(row_weight), _ptr(slot_to_row), top, float(gain), _ptr(shift), _ptr(state),
+        state.shape[0] if state is not None else 0, rows.state_slots.data_ptr() if shift is not None else None,
+        _ptr(rows.cu_seqlens_q) if shift is not None else None, _ptr(rows.cu_seqlens_k) if shift is not None else None,
+        _ptr(rows.context_lens) if shift is not None else None, n, 1 if final_gain is not None else 0, float(final_gain or 0.0),
+        float(eps), h.data_ptr(), T, d, _dt(h), status_word(dev).data_ptr(), _stream()), "shift_residual")
+    return h
+
+
+def conv_norm_rope_store(q: torch.Tensor, k: torch.Tensor, conv_q: torch.Tensor, conv_k: torch.Tensor,
+                         ring: torch.Tensor | None, rows: StepRows, q_norm_w: torch.Tensor, k_norm_w: torch.Tensor, eps: float,
+                         freq: torch.Tensor, positions: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
+                         slot_mapping: torch.Tensor, packed: bool = True):
+    """Short convolution of q [T, Hq * D] and k [T, Hkv * D] (views of one projection; weights [taps, channels]), values = the
+    convolved keys, norms over the whole projections, rotation of channel halves, scatter into the pools [num_blocks,
+    block_size, Hkv, D] (``b200_conv_norm_rope_store``).  ``ring`` [slots, taps - 1, channels of q and k] carries the last inputs.
+    Returns q [T, Hq, D] and, with ``packed``, k and v [T, Hkv, D] (else None)."""
+    dev = _cuda(q, k, conv_q, conv_k, ring, q_norm_w, k_norm_w, freq, positions, k_cache, v_cache, slot_mapping)
+    nb, bs, Hkv, D = k_cache.shape
+    T, taps = q.shape[0], conv_q.shape[0]
+    Cq, Ck = q.shape[1], Hkv * D
+    if Cq % D or k.shape != (T, Ck) or any(t.stride(1) != 1 or t.stride(0) != q.stride(0) or t.dtype != q.dtype for t in (q, k)):
+        raise ValueError("q [T, Hq * D] and k [T, Hkv * D] must share dtype and row stride")
+    if v_cache.shape != k_cache.shape or any(not c.is_contiguous() or c.dtype != q.dtype for c in (k_cache, v_cache)):
+        raise ValueError("caches must be contiguous [num_blocks, block_size, Hkv, D] of q's dtype")
+    _f32vec("conv_q", conv_q, taps * Cq)
+    _f32vec("conv_k", conv_k, taps * Ck)
+    _f32vec("q_norm_w", q_norm_w, Cq)
+    _f32vec("k_norm_w", k_norm_w, Ck)
+    if taps > 1 and (ring is None or ring.dtype != torch.float32 or ring.shape[1:] != (taps - 1, Cq + Ck) or not ring.is_contiguous()):
+        raise ValueError("ring must be contiguous fp32 [slots, taps - 1, channels]")
+    if freq.dtype != torch.float64 or not freq.is_contiguous():
+        raise ValueError("freq must be contiguous fp64")
+    for name, t in (("positions", positions), ("slot_mapping", slot_mapping)):
+        _tokens(name, t, T)
+    n = rows.check(T)
+    qo = torch.empty(T, Cq // D, D, dtype=q.dtype, device=dev)
+    ko, vo = (torch.empty(T, Hkv, D, dtype=q.dtype, device=dev) for _ in range(2)) if packed else (None, None)
+    check(lib.b200_conv_norm_rope_store(
+        q.data_ptr(), k.data_ptr(), q.stride(0), conv_q.data_ptr(), conv_k.data_ptr(), taps, _ptr(ring) if taps > 1 else None,
+        ring.shape[0] if taps > 1 else 0, rows.state_slots.data_ptr(), _ptr(rows.cu_seqlens_q), _ptr(rows.cu_seqlens_k),
+        _ptr(rows.context_lens), n, q_norm_w.data_ptr(), k_norm_w.data_ptr(), float(eps), freq.data_ptr(), 2 * freq.numel(),
+        positions.data_ptr(), qo.data_ptr(), _ptr(ko), _ptr(vo), k_cache.data_ptr(), v_cache.data_ptr(), slot_mapping.data_ptr(),
+        nb * bs, T, Cq // D, Hkv, D, _dt(q), status_word(dev).data_ptr(), _stream()), "conv_norm_rope_store")
+    return qo, ko, vo
+
+
+def sigmoid_attention_tile_rows(Hq: int, Hkv: int, Dqk: int, Dv: int, dtype: torch.dtype) -> int:
+    """Query rows per tile of the kernel behind ``sigmoid_attention``; 0 = no tiled kernel."""
+    return int(lib.b200_sigmoid_attention_tile_rows(Hq, Hkv, Dqk, Dv, _DTYPES[dtype])) if dtype in _DTYPES else 0
+
+
+def _gate_rows(gate: torch.Tensor | None, rows: int, heads: int, dtype: torch.dtype) -> None:
+    if gate is not None and (gate.shape != (rows, heads) or gate.dtype != dtype or (heads > 1 and gate.stride(1) != 1)):
+        raise ValueError("gate must be [tokens, heads] in the dtype of q with contiguous rows")
+
+
+def sigmoid_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, cu_seqlens_q: torch.Tensor, cu_seqlens_k: torch.Tensor,
+                      max_seqlen_q: int, scale: float, bias: torch.Tensor, chunk: int = 0, gate: torch.Tensor | None = None,
+                      out: torch.Tensor | None = None, plan: "PrefillPlan | None" = None) -> torch.Tensor:
+    """Causal attention over packed keys with weights sigmoid(scale q.k + bias[head]), not normalised, inside chunks of
+    positions (0: none), every head's row times sigmoid(gate) (``b200_sigmoid_attention``).  q [Tq, Hq, Dqk], k [Tk, Hkv, Dqk],
+    v [Tk, Hkv, Dv]; packed contexts start where a chunk starts.  Returns [Tq, Hq, Dv]."""
+    dev = _cuda(q, k, v, cu_seqlens_q, cu_seqlens_k, bias, gate, out)
+    Tq, Hq, Dqk = q.shape
+    Tk, Hkv, Dv = v.shape
+    if cu_seqlens_q.dtype != torch.int32 or cu_seqlens_k.dtype != torch.int32 or cu_seqlens_q.numel() != cu_seqlens_k.numel():
+        raise ValueError("cu_seqlens must be int32 tensors of the same length")
+    if k.shape != (Tk, Hkv, Dqk) or k.dtype != q.dtype or v.dtype != q.dtype:
+        raise ValueError("k must be [Tk, Hkv, Dqk] and v [Tk, Hkv, Dv] in the dtype of q")
+    for t, D in ((q, Dqk), (k, Dqk), (v, Dv)):
+        if t.stride(2) != 1 or (t.shape[1] > 1 and t.stride(1) != D):
+            raise ValueError("heads must be contiguous")
+    _f32vec("bias", bias, Hq)
+    _gate_rows(gate, Tq, Hq, q.dtype)
+    if out is None:
+        out = torch.empty((Tq, Hq, Dv), dtype=q.dtype, device=q.device)
+    elif out.shape != (Tq, Hq, Dv) or out.dtype != q.dtype or not out.is_contiguous():
+        raise ValueError("out must be a contiguous [Tq, Hq, Dv] tensor")
+    check(lib.b200_sigmoid_attention(
+        q.data_ptr(), k.data_ptr(), v.data_ptr(), out.data_ptr(), q.stride(0), k.stride(0), v.stride(0), Tq, Tk,
+        cu_seqlens_q.data_ptr(), cu_seqlens_k.data_ptr(), cu_seqlens_q.numel() - 1, int(max_seqlen_q), Hq, Hkv, Dqk, Dv,
+        float(scale), bias.data_ptr(), int(chunk), _ptr(gate), gate.stride(0) if gate is not None else 0,
+        plan.buffer.data_ptr() if plan is not None else None, plan.tile_rows if plan is not None else 0,
+        plan.capacity if plan is not None else 0, _dt(q), status_word(dev).data_ptr(), _stream()), "sigmoid_attention")
+    return out
+
+
+def sigmoid_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, block_tables: torch.Tensor,
+                   context_lens: torch.Tensor, scale: float, bias: torch.Tensor, chunk: int = 0, gate: torch.Tensor | None = None,
+                   out: torch.Tensor | None = None) -> torch.Tensor:
+    """``sigmoid_attention`` of one token per sequence over the paged pools (``b200_sigmoid_decode``): q [B, Hq, D], caches
+    [num_blocks, block_size, Hkv, D*].  Returns [B, Hq, Dv]."""
+    dev = _cuda(q, k_cache, v_cache, block_tables, context_lens, bias, gate, out)
+    B, Hq, D = q.shape
+    nb, bs, Hkv, Dc = k_cache.shape
+    Dv = v_cache.shape[3]
+    if Dc != D or v_cache.shape[:3] != k_cache.shape[:3] or k_cache.dtype != q.dtype or v_cache.dtype != q.dtype \
+            or not (q.is_contiguous() and k_cache.is_contiguous() and v_cache.is_contiguous()):
+        raise ValueError("q and caches must be contiguous, of one dtype and head size")
+    if block_tables.dtype != torch.int32 or block_tables.dim() != 2 or block_tables.shape[0] != B or block_tables.stride(1) != 1 \
+            or context_lens.dtype != torch.int64 or context_lens.numel() != B or not context_lens.is_contiguous():
+        raise ValueError("block_tables must be int32 [B, maxb] and context_lens int64 [B]")
+    _f32vec("bias", bias, Hq)
+    _gate_rows(gate, B, Hq, q.dtype)
+    if out is None:
+        out = torch.empty((B, Hq, Dv), dtype=q.dtype, device=q.device)
+    elif out.shape != (B, Hq, Dv) or out.dtype != q.dtype or not out.is_contiguous():
+        raise ValueError("out must be a contiguous [B, Hq, Dv] tensor of q's dtype")
+    ws = workspace(dev, lib.b200_paged_decode_gqa_workspace_bytes(B, Hq, Hkv, D, _dt(q)), "decode")
+    check(lib.b200_sigmoid_decode(
+        q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(), block_tables.data_ptr(), block_tables.stride(0),
+        context_lens.data_ptr(), B, Hq, Hkv, D, Dv, bs, nb, float(scale), bias.data_ptr(), int(chunk), _ptr(gate),
+        gate.stride(0) if gate is not None else 0, ws.data_ptr(), ws.numel(), _dt(q), status_word(dev).data_ptr(), _stream()),
+        "sigmoid_decode")
+    return out
+
+
+def moe_softmax_route(logits: torch.Tensor, bias: torch.Tensor, top: int):
+    """The ``top`` experts with the largest logits + bias per token, weights = softmax over those alone; fp32 logits [T, E]
+    (``b200_moe_softmax_route``).  Returns what ``moe_group_route`` returns."""
+    dev = _cuda(logits, bias)
+    T, E = logits.shape
+    if logits.dtype != torch.float32 or not logits.is_contiguous():
+        raise ValueError("logits must be contiguous fp32 [T, E]")
+    _f32vec("bias", bias, E)
+    tok = torch.empty(T * top, dtype=torch.int32, device=dev)
+    w = torch.empty(T, top, dtype=torch.float32, device=dev)
+    offs = torch.empty(E, dtype=torch.int32, device=dev)
+    slot = torch.empty(T, top, dtype=torch.int32, device=dev)
+    ws = workspace(dev, int(lib.b200_moe_group_route_workspace_bytes(T, E, top)), "moe_group_route")
+    check(lib.b200_moe_softmax_route(logits.data_ptr(), bias.data_ptr(), T, E, int(top), tok.data_ptr(), w.data_ptr(),
+                                     offs.data_ptr(), slot.data_ptr(), ws.data_ptr(), ws.numel(), _stream()), "moe_softmax_route")
+    return tok, w, offs, slot

@@ -63,10 +63,13 @@ class Portions:
     state_slots: Optional[torch.Tensor]           # int64 [n]
     captured: bool = False                        # part of a CUDA graph: lengths differ from replay to replay
     ranges: dict = field(default_factory=dict)    # window -> KeyRange, for the windows the model's layers have
+    chunk_ranges: dict = field(default_factory=dict)   # the same by chunk size, for layers that attend inside chunks
     plans: dict = field(default_factory=dict)     # tile lists by rows per tile, built when a layer asks
 
-    def keys(self, window: int = 0) -> KeyRange:
-        """What a layer with this sliding window needs of the contexts (0: all of them)."""
+    def keys(self, window: int = 0, chunk: int = 0) -> KeyRange:
+        """What a layer with this sliding window, or with chunks of this size, needs of the contexts (0: all of them)."""
+        if chunk in self.chunk_ranges:
+            return self.chunk_ranges[chunk]
         if window in self.ranges:
             return self.ranges[window]
         return KeyRange(self.cu_seqlens_k, self.max_seqlen_k, self.total_k, self.has_prefix)
