@@ -388,6 +388,7 @@ extern "C" int b200_conv_norm_rope_store(
     return B200_ERR_ARG;
   if (cu_seqlens_q ? !cu_seqlens_k : !context_lens || num_seqs != num_tokens) return B200_ERR_ARG;
   if (num_tokens > 2147483647 - num_seqs) return B200_ERR_TOO_LARGE;
+  if (taps == 1) state_slots = nullptr;      // no state
   CnArgs a{q, k, token_stride, conv_q, conv_k, taps, ring, state_slots, num_slots, cu_seqlens_q, cu_seqlens_k, context_lens,
            num_seqs, q_norm_w, k_norm_w, eps, freq, rot_dims / 2, positions, q_out, k_out, v_out, k_cache, v_cache, slot_mapping,
            pool_slots, num_tokens, num_q_heads * head_dim, num_kv_heads * head_dim, head_dim,
