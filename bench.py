@@ -284,7 +284,7 @@ def main():
     ap.add_argument("--no-engine", action="store_true", help="skip the engine job (profiling runs)")
     ap.add_argument("--workload", default="decode", choices=["decode", "mla_decode", "prefill", "prefill64", "mla_prefill", "store", "moe_experts", "lm_head", "engine", "engine_mla", "engine_step",
                                                                  "nabalix", "nabalix_kernels", "taminex", "taminex_kernels",
-                                                                 "meresun", "meresun_kernels"],
+                                                                 "meresun", "meresun_kernels", "sodonex", "sodonex_kernels"],
                     help="decode = the benchmark (paged GQA decode); the others time a secondary kernel on "
                          "its benchmark shape and print a short JSON line (single GPU, no reference arm)")
     ap.add_argument("--rate", type=float, default=0.0, help="engine workload: Poisson arrival rate (req/s); 0 = offline")
@@ -299,7 +299,7 @@ def main():
     if args.workload != "decode":
         from llm_from_scratch_b200 import microbench
         torch.cuda.set_device(int(os.environ.get("LOCAL_RANK", "0")))
-        if args.workload.startswith(("nabalix", "taminex", "meresun")):
+        if args.workload.startswith(("nabalix", "taminex", "meresun", "sodonex")):
             import importlib
             family, _, part = args.workload.partition("_")
             fn = getattr(importlib.import_module(f"llm_from_scratch_b200.microbench_{family}"), part or "throughput")
@@ -314,7 +314,7 @@ def main():
         if args.batch != BATCH:   # profiling cases: fewer sequences / tokens
             key = {"mla_decode": "batch", "engine": "batch", "prefill": "total", "store": "tokens",
                    "moe_experts": "tokens", "engine_mla": "batch", "mla_prefill": "seqs", "engine_step": "batch",
-                   "prefill64": "seqs", "lm_head": "rows", "nabalix": "batch", "taminex": "batch", "meresun": "batch"}[args.workload]
+                   "prefill64": "seqs", "lm_head": "rows", "nabalix": "batch", "taminex": "batch", "meresun": "batch", "sodonex": "batch"}[args.workload]
             kw[key] = args.batch
         res = fn(**kw)
         if not res:       # a non-zero rank of a multi-replica engine run

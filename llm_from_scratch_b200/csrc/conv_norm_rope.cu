@@ -49,7 +49,7 @@ struct CnArgs {
   int32_t* status;
 };
 
-constexpr int kSegment = 16;
+constexpr int kSegment = 16, kMaxSegment = 64;
 
 // slot in the pool of a token, -1: none
 __device__ __forceinline__ int64_t pool_slot(const CnArgs& a, int64_t tok) {
@@ -69,169 +69,191 @@ __device__ __forceinline__ void angles(const CnArgs& a, const Segment& g, float2
   }
 }
 
-// ---- eight channels per thread (bf16) ----
-union Pack8 {
-  uint4 u;
-  __nv_bfloat162 p[4];
-};
-__device__ __forceinline__ void unpack8(uint4 u, float (&v)[8]) {
-  Pack8 k;
-  k.u = u;
+// ---- eight channels per thread (bf16), as four packed fp32 pairs ----
+__device__ __forceinline__ void load_pairs(const float* p, f32x2 (&v)[4]) {
+  const ulonglong2 a = *reinterpret_cast<const ulonglong2*>(p), b = *reinterpret_cast<const ulonglong2*>(p + 4);
+  v[0] = a.x, v[1] = a.y, v[2] = b.x, v[3] = b.y;
+}
+__device__ __forceinline__ void store_pairs(float* p, const f32x2 (&v)[4]) {
+  *reinterpret_cast<ulonglong2*>(p) = make_ulonglong2(v[0], v[1]);
+  *reinterpret_cast<ulonglong2*>(p + 4) = make_ulonglong2(v[2], v[3]);
+}
+__device__ __forceinline__ void unpack_pairs(uint4 u, f32x2 (&v)[4]) {
+  const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+  for (int e = 0; e < 4; ++e) v[e] = pack2(__uint_as_float(w[e] << 16), __uint_as_float(w[e] & 0xffff0000u));
+}
+__device__ __forceinline__ uint4 round_pairs(const f32x2 (&v)[4]) {
+  uint32_t w[4];
 #pragma unroll
   for (int e = 0; e < 4; ++e) {
-    const float2 f = __bfloat1622float2(k.p[e]);
-    v[2 * e] = f.x;
-    v[2 * e + 1] = f.y;
+    const float2 f = unpack2(v[e]);
+    w[e] = pack_bf16x2(f.x, f.y);
   }
-}
-__device__ __forceinline__ uint4 pack8(const float (&v)[8]) {
-  return make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]), pack_bf16x2(v[6], v[7]));
-}
-__device__ __forceinline__ void load8(const float* p, float (&v)[8]) {
-  const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
-  v[0] = a.x, v[1] = a.y, v[2] = a.z, v[3] = a.w, v[4] = b.x, v[5] = b.y, v[6] = b.z, v[7] = b.w;
-}
-__device__ __forceinline__ void store8(float* p, const float (&v)[8]) {
-  *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
-  *reinterpret_cast<float4*>(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
+  return make_uint4(w[0], w[1], w[2], w[3]);
 }
 
-// B tokens per round: their sums share a barrier.  half a multiple of eight, so that a thread's partner channels are one thread's.
-template <int TAPS, int B, int THREADS>
-__global__ void __launch_bounds__(THREADS) conv_norm_rope_kernel(const CnArgs a) {
+// Shared-memory rows that threads read in pieces of eight floats are kept as two planes of four, so that neighbouring threads'
+// 16-byte accesses lie side by side.
+__device__ __forceinline__ void load_planes(const float* p, int plane, f32x2 (&v)[4]) {
+  const ulonglong2 a = *reinterpret_cast<const ulonglong2*>(p), b = *reinterpret_cast<const ulonglong2*>(p + plane);
+  v[0] = a.x, v[1] = a.y, v[2] = b.x, v[3] = b.y;
+}
+
+// half a multiple of eight, so that a thread's partner channels are one thread's.  SHFL: that thread is in the same warp; else
+// the values pass through shared memory.
+template <int TAPS, bool SHFL, int THREADS>
+__global__ void __launch_bounds__(THREADS, 640 / THREADS > 0 ? 640 / THREADS : 1) conv_norm_rope_kernel(const CnArgs a) {
   extern __shared__ float4 smem4[];
-  __shared__ __align__(16) float sums[2][B][2][32];                         // squares of every warp's channels of q and k
+  __shared__ float sums[2][2][32];                                          // squares of every warp's channels of q and k
+  __shared__ int64_t s_slot[kMaxSegment];
   Segment g;
   if (!segment_of(a, a.seg_len, &g)) return;
   const int C = a.Cq + a.Ck, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
-  float* swap = reinterpret_cast<float*>(smem4);                            // [2][B][C] convolved values, for the partners
-  float2* cs = reinterpret_cast<float2*>(swap + 2 * B * C);                 // [seg_len][half]
+  float* cos_t = reinterpret_cast<float*>(smem4);                           // [seg_len][2 planes][half / 2]
+  float* sin_t = cos_t + a.seg_len * a.half;
+  float* swap = sin_t + a.seg_len * a.half;                                 // [2][2 planes][C / 2] weighted values, for the partners
   const int c = threadIdx.x * 8;                                            // channel of [q | k]
   const bool in = c < C, is_k = c >= a.Cq;
-  const int cc = is_k ? c - a.Cq : c;                                       // channel of q or k
+  const int cc = is_k ? c - a.Cq : c, width = is_k ? a.Ck : a.Cq;           // channel of q or k
   const int ch = cc % a.D;                                                  // and of the head
   const int partner = ch < a.half ? a.half : ch < 2 * a.half ? -a.half : 0;
-  const __nv_bfloat16* src = static_cast<const __nv_bfloat16*>(is_k ? a.k : a.q) + cc;
-  float w[TAPS][8];
-  uint4 hist[TAPS];                                                         // hist[m]: input TAPS - 1 - m tokens back
+  const bool mixed = a.Cq % 256 != 0;                                       // a warp holds channels of both
+  const __nv_bfloat16* src = static_cast<const __nv_bfloat16*>(is_k ? a.k : a.q) + g.first * a.stride + cc;
+  auto input = [&](int t) {                                                 // loads run two tokens ahead
+    return in && t < g.count ? *reinterpret_cast<const uint4*>(src + t * a.stride) : make_uint4(0, 0, 0, 0);
+  };
+  uint4 next = input(0), after = input(1);
+  f32x2 w[TAPS][4];
+  uint4 hist[TAPS - 1];                                                     // hist[m]: input TAPS - 1 - m tokens back
 #pragma unroll
-  for (int m = 0; m < TAPS; ++m) {
-    hist[m] = make_uint4(0, 0, 0, 0);
+  for (int m = 0; m < TAPS; ++m)
 #pragma unroll
-    for (int e = 0; e < 8; ++e) w[m][e] = 0.f;
-  }
+    for (int e = 0; e < 4; ++e) w[m][e] = 0;
+#pragma unroll
+  for (int m = 0; m < TAPS - 1; ++m) hist[m] = make_uint4(0, 0, 0, 0);
   if (in) {
 #pragma unroll
-    for (int m = 0; m < TAPS; ++m) load8(is_k ? a.wk + static_cast<int64_t>(m) * a.Ck + cc : a.wq + static_cast<int64_t>(m) * a.Cq + cc, w[m]);
-    // the inputs before the segment: hist[1 ..] become hist[0 ..] when the first token arrives
+    for (int m = 0; m < TAPS; ++m) load_pairs((is_k ? a.wk : a.wq) + static_cast<int64_t>(m) * width + cc, w[m]);
 #pragma unroll
-    for (int m = 1; m < TAPS; ++m) {
-      const int back = TAPS - m;                                            // tokens before the segment's first
+    for (int m = 0; m < TAPS - 1; ++m) {
+      const int back = TAPS - 1 - m;                                        // tokens before the segment's first
       if (g.index > 0) {
-        hist[m] = *reinterpret_cast<const uint4*>(src + (g.first - back) * a.stride);
+        hist[m] = *reinterpret_cast<const uint4*>(src - back * a.stride);
       } else if (g.slot >= 0 && g.pos0 - back >= 0) {
-        float v[8];
-        load8(a.ring + (g.slot * (TAPS - 1) + (g.pos0 - back) % (TAPS - 1)) * C + c, v);
-        hist[m] = pack8(v);                                                 // the state holds rounded values
+        f32x2 v[4];
+        load_pairs(a.ring + (g.slot * (TAPS - 1) + (g.pos0 - back) % (TAPS - 1)) * C + c, v);
+        hist[m] = round_pairs(v);                                           // the state holds rounded values
       }
     }
     if (g.index == 0 && g.slot >= 0) {
       for (int m = 0; m < min(TAPS - 1, g.len); ++m) {
         const int t = g.len - 1 - m;
-        float v[8];
-        unpack8(*reinterpret_cast<const uint4*>(src + (g.first + t) * a.stride), v);
-        store8(a.ring + (g.slot * (TAPS - 1) + (g.pos0 + t) % (TAPS - 1)) * C + c, v);
+        f32x2 v[4];
+        unpack_pairs(*reinterpret_cast<const uint4*>(src + t * a.stride), v);
+        store_pairs(a.ring + (g.slot * (TAPS - 1) + (g.pos0 + t) % (TAPS - 1)) * C + c, v);
       }
     }
   }
-  for (int i = threadIdx.x; i < 4 * B * 32; i += blockDim.x)
-    if ((i & 31) >= nw) (&sums[0][0][0][0])[i] = 0.f;
-  angles(a, g, cs);
-  uint4 next[B];
+  for (int i = threadIdx.x; i < 4 * 32; i += blockDim.x)
+    if ((i & 31) >= nw) (&sums[0][0][0])[i] = 0.f;
+  for (int t = threadIdx.x; t < g.count; t += blockDim.x) s_slot[t] = pool_slot(a, g.first + t);
+  for (int i = threadIdx.x; i < g.count * a.half; i += blockDim.x) {
+    const int t = i / a.half, j = i - t * a.half;
+    const float2 r = rotary_angle(a.positions[g.first + t], a.freq[j]);
+    const int at = t * a.half + (j >> 2 & 1) * (a.half / 2) + (j >> 3) * 4 + (j & 3);
+    cos_t[at] = r.x;
+    sin_t[at] = r.y;
+  }
+  const float per = 1.f / static_cast<float>(width);
+  const float* norm = (is_k ? a.nk : a.nq) + cc;
+  const f32x2 sign = pack2(partner < 0 ? -1.f : 1.f, partner < 0 ? -1.f : 1.f);
+  const int angle = (partner > 0 ? ch : ch - a.half) / 2, to = threadIdx.x * 4 + partner / 2, other = lane + partner / 8;
+  for (int t = 0; t < g.count; ++t) {
+    const uint4 cur = next;
+    next = after;
+    after = input(t + 2);
+    f32x2 y[4], z[4];
 #pragma unroll
-  for (int b = 0; b < B; ++b)
-    next[b] = in && b < g.count ? *reinterpret_cast<const uint4*>(src + (g.first + b) * a.stride) : make_uint4(0, 0, 0, 0);
-  for (int t0 = 0, round = 0; t0 < g.count; t0 += B, ++round) {
-    float y[B][8];
-    float* ex = swap + (round & 1) * B * C;
+    for (int e = 0; e < 4; ++e) y[e] = 0;
 #pragma unroll
-    for (int b = 0; b < B; ++b) {
+    for (int m = 0; m < TAPS; ++m) {
+      f32x2 v[4];
+      unpack_pairs(m < TAPS - 1 ? hist[m] : cur, v);
 #pragma unroll
-      for (int m = 0; m + 1 < TAPS; ++m) hist[m] = hist[m + 1];
-      hist[TAPS - 1] = next[b];
-#pragma unroll
-      for (int e = 0; e < 8; ++e) y[b][e] = 0.f;
-#pragma unroll
-      for (int m = 0; m < TAPS; ++m) {
-        float v[8];
-        unpack8(hist[m], v);
-#pragma unroll
-        for (int e = 0; e < 8; ++e) y[b][e] = fmaf(w[m][e], v[e], y[b][e]);
-      }
+      for (int e = 0; e < 4; ++e) y[e] = fma2(w[m][e], v[e], y[e]);
     }
 #pragma unroll
-    for (int b = 0; b < B; ++b)
-      if (in && t0 + B + b < g.count) next[b] = *reinterpret_cast<const uint4*>(src + (g.first + t0 + B + b) * a.stride);
+    for (int m = 0; m < TAPS - 1; ++m) hist[m] = m + 1 < TAPS - 1 ? hist[m + 1 < TAPS - 1 ? m + 1 : 0] : cur;
+    f32x2 sq = 0;
 #pragma unroll
-    for (int b = 0; b < B; ++b) {
-      float ss = 0.f;
-#pragma unroll
-      for (int e = 0; e < 8; ++e) ss += y[b][e] * y[b][e];
-      if (in && partner != 0) store8(ex + b * C + c, y[b]);
-      const float sk = warp_sum(is_k ? ss : 0.f), sq = warp_sum(is_k ? 0.f : ss);
+    for (int e = 0; e < 4; ++e) sq = fma2(y[e], y[e], sq);
+    const float2 f = unpack2(sq);
+    float* part = sums[t & 1][0];
+    if (mixed) {
+      const float sq_q = warp_sum(is_k ? 0.f : f.x + f.y), sq_k = warp_sum(is_k ? f.x + f.y : 0.f);
       if (lane == 0) {
-        sums[round & 1][b][0][warp] = sq;
-        sums[round & 1][b][1][warp] = sk;
+        part[warp] = sq_q;
+        part[32 + warp] = sq_k;
       }
+    } else {
+      const float sum = warp_sum(f.x + f.y);
+      if (lane == 0) {
+        part[is_k * 32 + warp] = sum;
+        part[!is_k * 32 + warp] = 0.f;
+      }
+    }
+    uint4 raw = make_uint4(0, 0, 0, 0);
+    if (is_k) raw = round_pairs(y);
+    if (in) {
+      f32x2 weight[4];
+      load_pairs(norm, weight);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) y[e] = mul2(y[e], weight[e]);
+    }
+#pragma unroll
+    for (int e = 0; e < 4; ++e) z[e] = mul2(y[e], sign);                  // the upper half's values enter with a minus
+    float* ex = swap + (t & 1) * C;
+    if constexpr (SHFL) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) z[e] = __shfl_sync(0xffffffffu, z[e], other);
+    } else if (partner != 0 && in) {
+      *reinterpret_cast<ulonglong2*>(ex + threadIdx.x * 4) = make_ulonglong2(z[0], z[1]);
+      *reinterpret_cast<ulonglong2*>(ex + C / 2 + threadIdx.x * 4) = make_ulonglong2(z[2], z[3]);
     }
     __syncthreads();
-    if (!in) {
+    float total = warp_sum(part[(mixed ? 0 : is_k) * 32 + lane]);
+    if (mixed) {
+      const float total_k = warp_sum(part[32 + lane]);
+      if (is_k) total = total_k;
+    }
+    if (!in) continue;
+    const float r = rsqrtf(total * per + a.eps);
+    const f32x2 inv = pack2(r, r);
+    if (partner != 0) {
+      f32x2 cs[4], sn[4];
+      if constexpr (!SHFL) load_planes(ex + to, C / 2, z);
+      load_planes(cos_t + t * a.half + angle, a.half / 2, cs);
+      load_planes(sin_t + t * a.half + angle, a.half / 2, sn);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) y[e] = fma2(z[e], sn[e], mul2(y[e], cs[e]));
+    }
+#pragma unroll
+    for (int e = 0; e < 4; ++e) y[e] = mul2(y[e], inv);
+    const uint4 o = round_pairs(y);
+    const int64_t at = (g.first + t) * width + cc;
+    if (!is_k) {
+      *reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(a.q_out) + at) = o;
       continue;
     }
-    float nw8[8], np8[8];
-    const float* norm = is_k ? a.nk : a.nq;
-    load8(norm + cc, nw8);
-    if (partner != 0) load8(norm + cc + partner, np8);
-#pragma unroll
-    for (int b = 0; b < B; ++b) {
-      const int t = t0 + b;
-      if (t >= g.count) break;
-      float total = 0.f;
-      for (int i = 0; i < nw; i += 4) {
-        const float4 p = *reinterpret_cast<const float4*>(&sums[round & 1][b][is_k][i]);
-        total += (p.x + p.y) + (p.z + p.w);
-      }
-      const float inv = rsqrtf(total / static_cast<float>(is_k ? a.Ck : a.Cq) + a.eps);
-      const int64_t tok = g.first + t;
-      const uint4 raw = pack8(y[b]);
-      float o[8];
-#pragma unroll
-      for (int e = 0; e < 8; ++e) o[e] = y[b][e] * inv * nw8[e];
-      if (partner != 0) {
-        float z[8];
-        load8(ex + b * C + c + partner, z);
-        const float sign = partner > 0 ? -1.f : 1.f;
-        const float2* angle = cs + t * a.half + (partner > 0 ? ch : ch - a.half);
-#pragma unroll
-        for (int e = 0; e < 8; ++e) {
-          const float2 r = angle[e];
-          o[e] = o[e] * r.x + sign * (z[e] * inv * np8[e]) * r.y;
-        }
-      }
-      const uint4 out = pack8(o);
-      if (!is_k) {
-        *reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(a.q_out) + tok * a.Cq + cc) = out;
-        continue;
-      }
-      if (a.k_out != nullptr) {
-        *reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(a.k_out) + tok * a.Ck + cc) = out;
-        *reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(a.v_out) + tok * a.Ck + cc) = raw;
-      }
-      const int64_t slot = pool_slot(a, tok);
-      if (slot >= 0) {
-        *reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(a.kc) + slot * a.Ck + cc) = out;
-        *reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(a.vc) + slot * a.Ck + cc) = raw;
-      }
+    if (a.k_out != nullptr) {
+      *reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(a.k_out) + at) = o;
+      *reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(a.v_out) + at) = raw;
+    }
+    const int64_t slot = s_slot[t];
+    if (slot >= 0) {
+      *reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(a.kc) + slot * a.Ck + cc) = o;
+      *reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(a.vc) + slot * a.Ck + cc) = raw;
     }
   }
 }
@@ -334,25 +356,32 @@ bool allow_shared(Kernel kern, bool* configured) {
   return true;
 }
 
-template <int TAPS, int B, int THREADS>
+template <int TAPS, bool SHFL, int THREADS>
 int launch_wide(const CnArgs& a, unsigned grid, int threads, cudaStream_t s) {
-  const size_t smem = static_cast<size_t>(2 * B) * (a.Cq + a.Ck) * sizeof(float) + static_cast<size_t>(a.seg_len) * a.half * sizeof(float2);
+  const size_t smem = (static_cast<size_t>(2 * a.seg_len) * a.half + (SHFL ? 0 : 2 * (a.Cq + a.Ck))) * sizeof(float);
   if (smem > kMaxShared) return B200_ERR_UNSUPPORTED;
-  auto kern = conv_norm_rope_kernel<TAPS, B, THREADS>;
+  auto kern = conv_norm_rope_kernel<TAPS, SHFL, THREADS>;
   static bool configured[64] = {};
   if (smem > 40 * 1024 && !allow_shared(kern, configured)) return B200_ERR_LAUNCH;
   kern<<<grid, threads, smem, s>>>(a);
   return launch_result();
 }
 
-template <int B, int THREADS>
-int launch_taps(const CnArgs& a, unsigned grid, int threads, cudaStream_t s) {
-  switch (a.taps) {
-    case 2: return launch_wide<2, B, THREADS>(a, grid, threads, s);
-    case 3: return launch_wide<3, B, THREADS>(a, grid, threads, s);
-    case 4: return launch_wide<4, B, THREADS>(a, grid, threads, s);
-    default: return B200_ERR_UNSUPPORTED;
+template <int TAPS>
+int launch_taps(CnArgs a, cudaStream_t s) {
+  const int threads = ((a.Cq + a.Ck) / 8 + 31) / 32 * 32;
+  unsigned grid = static_cast<unsigned>(a.T);
+  if (a.cu_q != nullptr) {
+    // one wave: a CTA's start (weights, angles, inputs before its segment) costs as much as a few tokens
+    const int64_t ctas = static_cast<int64_t>(sm_count_cached()) * (threads > 640 ? 1 : 640 / threads);
+    const int64_t fit = ctas > a.n ? (a.T + ctas - a.n - 1) / (ctas - a.n) : kMaxSegment;
+    a.seg_len = static_cast<int>(fit < 4 ? 4 : fit < kMaxSegment ? fit : kMaxSegment);
+    grid = static_cast<unsigned>(a.T / a.seg_len + a.n + 1);
   }
+  const bool shfl = 32 % (a.D / 8) == 0;          // a head lies inside one warp
+  if (threads <= 320) return shfl ? launch_wide<TAPS, true, 320>(a, grid, threads, s) : launch_wide<TAPS, false, 320>(a, grid, threads, s);
+  if (threads <= 640) return shfl ? launch_wide<TAPS, true, 640>(a, grid, threads, s) : launch_wide<TAPS, false, 640>(a, grid, threads, s);
+  return shfl ? launch_wide<TAPS, true, 1024>(a, grid, threads, s) : launch_wide<TAPS, false, 1024>(a, grid, threads, s);
 }
 
 template <typename T>
@@ -404,9 +433,8 @@ extern "C" int b200_conv_norm_rope_store(
                         static_cast<const void*>(v_cache)})
     wide = wide && aligned16(p);
   if (wide) {
-    const int threads = ((a.Cq + a.Ck) / 8 + 31) / 32 * 32;
-    const int rc = threads > 640   ? launch_taps<1, 1024>(a, grid, threads, s)
-                   : cu_seqlens_q ? launch_taps<2, 640>(a, grid, threads, s) : launch_taps<1, 640>(a, grid, threads, s);
+    const int rc = taps == 2 ? launch_taps<2>(a, s) : taps == 3 ? launch_taps<3>(a, s)
+                   : taps == 4 ? launch_taps<4>(a, s) : B200_ERR_UNSUPPORTED;
     if (rc != B200_ERR_UNSUPPORTED) return rc;
   }
   return launch_any<__nv_bfloat16>(a, grid, s);

@@ -9,8 +9,9 @@
 //   h  = x', rounded to the activation dtype
 //
 // x' goes to a buffer of its own: with a shift a CTA also needs the row before its first one, and works it out once more from x
-// and y, which the row's own CTA must not have overwritten.  A CTA owns up to R rows of one sequence.  The CTA that reads a
-// sequence's state is the one that moves it on: it works out the sequence's last row, if that is not its own.
+// and y, which the row's own CTA must not have overwritten.  A CTA walks up to `rows` rows of one sequence in order, the next
+// row's loads in flight while it reduces and writes the current one; the row before stays in registers.  The CTA that reads a
+// sequence's state is the one that moves it on: it also works out the sequence's last row, if that is not its own.
 #include <initializer_list>
 
 #include "sequences.cuh"
@@ -44,7 +45,10 @@ struct ShArgs {
   int64_t T;
   int d;
   int32_t* status;
+  int rows;                  // rows per CTA, at most kMaxRows
 };
+
+constexpr int kMaxRows = 8;
 
 // V channels in fp32
 template <typename T, int V>
@@ -125,169 +129,198 @@ __device__ __forceinline__ void load_x(const ShArgs& a, int64_t row, int c, floa
   for (int i = 0; i < V; ++i) x[i] *= a.scale;
 }
 
-// Sums over the CTA of N values per thread; scratch [N][32].
-template <int N>
-__device__ __forceinline__ void cta_sums(float (&v)[N], float (*scratch)[32]) {
+// Sum over the CTA; scratch is of this use alone until the next barrier but one.
+__device__ __forceinline__ float cta_sum(float v, float* scratch) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
-#pragma unroll
-  for (int j = 0; j < N; ++j) v[j] = warp_sum(v[j]);
-  if (lane == 0) {
-#pragma unroll
-    for (int j = 0; j < N; ++j) scratch[j][warp] = v[j];
-  }
+  v = warp_sum(v);
+  if (lane == 0) scratch[warp] = v;
   __syncthreads();
-#pragma unroll
-  for (int j = 0; j < N; ++j) v[j] = warp_sum(lane < nw ? scratch[j][lane] : 0.f);
+  return warp_sum(lane < nw ? scratch[lane] : 0.f);
 }
 
 // The rows of a CTA: own ones first .. first + count - 1, and at most one more row that is worked out and not written: the row
-// before them, or the sequence's last one for its state.
+// before them (halo), or the sequence's last one for its state (tail).
 struct Work {
   Segment g;
-  int64_t extra;             // row or -1
-  bool halo;                 // extra is the row before
-  bool from_state, save;
+  bool halo, tail, from_state, save;
+  // rows in the order of the walk
+  __device__ __forceinline__ int steps() const { return g.count + halo + tail; }
+  __device__ __forceinline__ int64_t row(int i) const {
+    return tail && i == g.count ? g.first + g.len - 1 : g.first + i - halo;
+  }
+  __device__ __forceinline__ bool own(int i) const { return i >= halo && i < g.count + halo; }
 };
 template <bool SHIFT>
 __device__ __forceinline__ bool work_of(const ShArgs& a, int rows, Work* w) {
-  w->extra = -1;
-  w->halo = w->from_state = w->save = false;
+  w->halo = w->tail = w->from_state = w->save = false;
   if constexpr (SHIFT) {
     if (!segment_of(a, rows, &w->g)) return false;
     const Segment& g = w->g;
-    if (g.index > 0) {
-      w->halo = true;
-      w->extra = g.first - 1;
-    } else {
-      w->save = g.slot >= 0;
-      w->from_state = w->save && g.pos0 > 0;
-      if (w->save && g.len > g.count) w->extra = g.first + g.len - 1;
-    }
+    w->halo = g.index > 0;
+    w->save = g.index == 0 && g.slot >= 0;
+    w->from_state = w->save && g.pos0 > 0;
+    w->tail = w->save && g.len > g.count;
   } else {
     w->g.first = static_cast<int64_t>(blockIdx.x) * rows;
     w->g.count = static_cast<int>(a.T - w->g.first < rows ? a.T - w->g.first : rows);
-    w->g.slot = -1;
   }
   return true;
 }
 
-// V channels per thread, all of a row in one pass
-template <typename T, int V, int R, bool SHIFT>
-__global__ void __launch_bounds__(R > 1 ? 512 : 1024) shift_residual_kernel(const ShArgs a) {
-  constexpr int N = SHIFT ? R + 1 : R;                 // row R: the extra one
-  __shared__ float scratch[2][N][32];
+// What is loaded of a row ahead of its turn: x, and y as it lies in memory (TOP > 0: one piece per expert).
+template <typename T, int V, int TOP>
+struct Ahead {
+  float x[V];
+  uint4 y[TOP > 0 ? TOP : 1];
+};
+
+// V channels per thread (16 bytes of T), a row in one pass.  TOP: 0: y holds one row per token, else at most TOP expert rows
+template <typename T, int TOP, bool SHIFT>
+__global__ void __launch_bounds__(1024) shift_residual_kernel(const ShArgs a) {
+  constexpr int V = 16 / sizeof(T);
+  __shared__ float scratch[2][32], scratch_norm[2][32];
+  __shared__ int s_from[(kMaxRows + 1) * (TOP > 0 ? TOP : 1)];
+  __shared__ float s_weight[(kMaxRows + 1) * (TOP > 0 ? TOP : 1)];
   Work w;
-  if (!work_of<SHIFT>(a, R, &w)) return;
-  const int c = threadIdx.x * V;
+  if (!work_of<SHIFT>(a, a.rows, &w)) return;
+  const int c = threadIdx.x * V, steps = w.steps();
   const bool in = c < a.d;
-  float x[N][V], y[N][V], ss[N];
-  auto row = [&](int j) -> int64_t { return j < R ? (j < w.g.count ? w.g.first + j : -1) : w.extra; };
-#pragma unroll
-  for (int j = 0; j < N; ++j) {
-    ss[j] = 0.f;
-#pragma unroll
-    for (int i = 0; i < V; ++i) x[j][i] = y[j][i] = 0.f;
-    if (!in || row(j) < 0) continue;
-    load_x<T, V>(a, row(j), c, x[j]);
-    if (a.y != nullptr) load_y<T, V>(a, row(j), c, y[j]);
+  if constexpr (TOP > 0) {
+    for (int i = threadIdx.x; i < steps * TOP; i += blockDim.x) {
+      const int k = i % TOP;
+      int from = -1;
+      float weight = 0.f;
+      if (k < a.top) {
+        const int64_t at = w.row(i / TOP) * a.top + k;
+        from = a.row_of[at];
+        weight = a.weight[at];
+        if (from < 0 || from >= a.T * a.top) {
+          report(a.status, B200_ERR_BOUNDS);
+          from = -1;
+        }
+      }
+      s_from[i] = from;
+      s_weight[i] = weight;
+    }
+    __syncthreads();
   }
-  float carried[V], mix[V];
+  auto fetch = [&](int i, Ahead<T, V, TOP>& r) {
+    if (!in) return;
+    const int64_t row = w.row(i);
+    load_x<T, V>(a, row, c, r.x);
+    if constexpr (TOP > 0) {
+#pragma unroll
+      for (int k = 0; k < TOP; ++k) {
+        const int from = s_from[i * TOP + k];
+        r.y[k] = from < 0 ? make_uint4(0, 0, 0, 0)
+                          : *reinterpret_cast<const uint4*>(static_cast<const T*>(a.y) + static_cast<int64_t>(from) * a.d + c);
+      }
+    } else if (a.y != nullptr) {
+      r.y[0] = *reinterpret_cast<const uint4*>(static_cast<const T*>(a.y) + row * a.d + c);
+    }
+  };
+  auto unpack = [&](uint4 u, float (&v)[V]) {
+    union {
+      uint4 u;
+      T e[V];
+    } k;
+    k.u = u;
+#pragma unroll
+    for (int i = 0; i < V; ++i) v[i] = to_float<T>(k.e[i]);
+  };
+  float before[V];
   if constexpr (SHIFT) {
 #pragma unroll
-    for (int i = 0; i < V; ++i) carried[i] = mix[i] = 0.f;
-    if (in) {
-      load_row<float, V>(a.shift + c, mix);
-      if (w.from_state) load_row<float, V>(a.state + w.g.slot * a.d + c, carried);
+    for (int i = 0; i < V; ++i) before[i] = 0.f;
+    if (in && w.from_state) load_row<float, V>(a.state + w.g.slot * a.d + c, before);
+  }
+  Ahead<T, V, TOP> next;
+#pragma unroll
+  for (int i = 0; i < V; ++i) next.x[i] = 0.f;
+#pragma unroll
+  for (int k = 0; k < (TOP > 0 ? TOP : 1); ++k) next.y[k] = make_uint4(0, 0, 0, 0);
+  fetch(0, next);
+  for (int i = 0; i < steps; ++i) {
+    float x[V], y[V];
+    if constexpr (TOP > 0) {
+#pragma unroll
+      for (int e = 0; e < V; ++e) y[e] = 0.f;
+#pragma unroll
+      for (int k = 0; k < TOP; ++k) {
+        float r[V];
+        unpack(next.y[k], r);
+        const float f = s_weight[i * TOP + k];
+#pragma unroll
+        for (int e = 0; e < V; ++e) y[e] = fmaf(f, r[e], y[e]);
+      }
+    } else {
+      unpack(next.y[0], y);
+    }
+#pragma unroll
+    for (int e = 0; e < V; ++e) x[e] = next.x[e];
+    if (i + 1 < steps) fetch(i + 1, next);
+    if (a.y != nullptr) {
+      float ss = 0.f;
+#pragma unroll
+      for (int e = 0; e < V; ++e) ss += y[e] * y[e];
+      const float f = a.gain * rsqrtf(cta_sum(ss, scratch[i & 1]) / static_cast<float>(a.d) + a.eps);
+#pragma unroll
+      for (int e = 0; e < V; ++e) x[e] += f * y[e];
+    }
+    const int64_t row = w.row(i);
+    T* h = static_cast<T*>(a.h) + row * a.d + c;
+    const bool own = w.own(i);
+    if (own && in && a.x_out != nullptr) store_row<float, V>(a.x_out + row * a.d + c, x);
+    if constexpr (SHIFT) {
+      if (own && in) {
+        float mix[V];
+        load_row<float, V>(a.shift + c, mix);
+#pragma unroll
+        for (int e = 0; e < V; ++e) mix[e] = x[e] + (before[e] - x[e]) * mix[e];
+        store_row<T, V>(h, mix);
+      }
+#pragma unroll
+      for (int e = 0; e < V; ++e) before[e] = x[e];
+    } else {
+      if (a.norm) {
+        float ss = 0.f;
+#pragma unroll
+        for (int e = 0; e < V; ++e) ss += x[e] * x[e];
+        const float f = a.final_gain * rsqrtf(cta_sum(ss, scratch_norm[i & 1]) / static_cast<float>(a.d) + a.eps);
+#pragma unroll
+        for (int e = 0; e < V; ++e) x[e] *= f;
+      }
+      if (in) store_row<T, V>(h, x);
     }
   }
-  if (a.y != nullptr) {
-#pragma unroll
-    for (int j = 0; j < N; ++j)
-#pragma unroll
-      for (int i = 0; i < V; ++i) ss[j] += y[j][i] * y[j][i];
-    cta_sums<N>(ss, scratch[0]);
-#pragma unroll
-    for (int j = 0; j < N; ++j) {
-      const float f = a.gain * rsqrtf(ss[j] / static_cast<float>(a.d) + a.eps);
-#pragma unroll
-      for (int i = 0; i < V; ++i) x[j][i] += f * y[j][i];
-    }
-  }
-  if (a.x_out != nullptr && in) {
-#pragma unroll
-    for (int j = 0; j < R; ++j)
-      if (j < w.g.count) store_row<float, V>(a.x_out + row(j) * a.d + c, x[j]);
-  }
-  T* h = static_cast<T*>(a.h) + c;
   if constexpr (SHIFT) {
-    if (!in) return;
-    if (w.halo) {
-#pragma unroll
-      for (int i = 0; i < V; ++i) carried[i] = x[R][i];
-    }
-#pragma unroll
-    for (int j = 0; j < R; ++j) {
-      if (j >= w.g.count) break;
-      float o[V];
-#pragma unroll
-      for (int i = 0; i < V; ++i) {
-        o[i] = x[j][i] + (carried[i] - x[j][i]) * mix[i];
-        carried[i] = x[j][i];
-      }
-      store_row<T, V>(h + row(j) * a.d, o);
-    }
-    if (w.save) {
-      if (w.extra >= 0) {
-#pragma unroll
-        for (int i = 0; i < V; ++i) carried[i] = x[R][i];
-      }
-      store_row<float, V>(a.state + w.g.slot * a.d + c, carried);
-    }
-  } else {
-    if (a.norm) {
-#pragma unroll
-      for (int j = 0; j < N; ++j) {
-        ss[j] = 0.f;
-#pragma unroll
-        for (int i = 0; i < V; ++i) ss[j] += x[j][i] * x[j][i];
-      }
-      cta_sums<N>(ss, scratch[1]);
-#pragma unroll
-      for (int j = 0; j < N; ++j) {
-        const float f = a.final_gain * rsqrtf(ss[j] / static_cast<float>(a.d) + a.eps);
-#pragma unroll
-        for (int i = 0; i < V; ++i) x[j][i] *= f;
-      }
-    }
-    if (!in) return;
-#pragma unroll
-    for (int j = 0; j < R; ++j)
-      if (j < w.g.count) store_row<T, V>(h + row(j) * a.d, x[j]);
+    if (w.save && in) store_row<float, V>(a.state + w.g.slot * a.d + c, before);      // the last row of the walk is the sequence's
   }
 }
 
 // any width, a row per CTA
 template <typename T, bool SHIFT>
 __global__ void __launch_bounds__(256) shift_residual_any_kernel(const ShArgs a) {
-  __shared__ float scratch[2][2][32];
+  __shared__ float scratch[3][32];
   Work w;
   if (!work_of<SHIFT>(a, 1, &w)) return;
-  const int64_t row = w.g.first;
-  float ss[2] = {0.f, 0.f};
+  const int64_t row = w.g.first, extra = w.halo ? row - 1 : w.tail ? row + w.g.len - 1 : -1;
+  float s0 = 0.f, s1 = 0.f;
   if (a.y != nullptr) {
     for (int c = threadIdx.x; c < a.d; c += blockDim.x) {
       float y[1];
       load_y<T, 1>(a, row, c, y);
-      ss[0] += y[0] * y[0];
-      if (w.extra >= 0) {
-        load_y<T, 1>(a, w.extra, c, y);
-        ss[1] += y[0] * y[0];
+      s0 += y[0] * y[0];
+      if (extra >= 0) {
+        load_y<T, 1>(a, extra, c, y);
+        s1 += y[0] * y[0];
       }
     }
-    cta_sums<2>(ss, scratch[0]);
+    s0 = cta_sum(s0, scratch[0]);
+    s1 = cta_sum(s1, scratch[1]);
   }
-  const float f0 = a.gain * rsqrtf(ss[0] / static_cast<float>(a.d) + a.eps);
-  const float f1 = a.gain * rsqrtf(ss[1] / static_cast<float>(a.d) + a.eps);
+  const float f0 = a.gain * rsqrtf(s0 / static_cast<float>(a.d) + a.eps);
+  const float f1 = a.gain * rsqrtf(s1 / static_cast<float>(a.d) + a.eps);
   auto value = [&](int64_t r, int c, float f) -> float {
     float x[1], y[1] = {0.f};
     load_x<T, 1>(a, r, c, x);
@@ -295,44 +328,47 @@ __global__ void __launch_bounds__(256) shift_residual_any_kernel(const ShArgs a)
     return x[0] + f * y[0];
   };
   T* h = static_cast<T*>(a.h) + row * a.d;
-  float sq[2] = {0.f, 0.f};
+  float sq = 0.f;
   for (int c = threadIdx.x; c < a.d; c += blockDim.x) {
     const float x = value(row, c, f0);
-    if (a.x_out != nullptr) a.x_out[row * a.d + c] = x;
+    sq += x * x;
     if constexpr (SHIFT) {
-      const float extra = w.extra >= 0 ? value(w.extra, c, f1) : 0.f;
-      const float before = w.halo ? extra : w.from_state ? a.state[w.g.slot * a.d + c] : 0.f;
+      const float other = extra >= 0 ? value(extra, c, f1) : 0.f;
+      const float before = w.halo ? other : w.from_state ? a.state[w.g.slot * a.d + c] : 0.f;
       h[c] = from_float<T>(x + (before - x) * a.shift[c]);
-      if (w.save) a.state[w.g.slot * a.d + c] = w.extra >= 0 ? extra : x;
-    } else {
-      sq[0] += x * x;
-      if (!a.norm) h[c] = from_float<T>(x);
+      if (w.save) a.state[w.g.slot * a.d + c] = w.tail ? other : x;
+      if (a.x_out != nullptr) a.x_out[row * a.d + c] = x;
+    } else if (!a.norm) {
+      h[c] = from_float<T>(x);
+      if (a.x_out != nullptr) a.x_out[row * a.d + c] = x;
     }
   }
   if constexpr (!SHIFT) {
     if (!a.norm) return;
-    cta_sums<2>(sq, scratch[1]);
-    const float f = a.final_gain * rsqrtf(sq[0] / static_cast<float>(a.d) + a.eps);
-    for (int c = threadIdx.x; c < a.d; c += blockDim.x) h[c] = from_float<T>(value(row, c, f0) * f);
+    const float f = a.final_gain * rsqrtf(cta_sum(sq, scratch[2]) / static_cast<float>(a.d) + a.eps);
+    for (int c = threadIdx.x; c < a.d; c += blockDim.x) {
+      const float x = value(row, c, f0);
+      if (a.x_out != nullptr) a.x_out[row * a.d + c] = x;
+      h[c] = from_float<T>(x * f);
+    }
   }
 }
 
-constexpr int kRows = 4;             // rows per CTA of prompts
-constexpr int64_t kManyRows = 2048;  // below, a CTA per row fills the GPU better
-
 template <typename T, bool SHIFT>
-void launch(const ShArgs& a, bool vec, cudaStream_t s) {
+void launch(ShArgs a, bool vec, cudaStream_t s) {
   constexpr int V = 16 / sizeof(T);
   const int threads = (a.d / V + 31) / 32 * 32;
   const bool one_each = SHIFT && a.cu_q == nullptr;
-  auto grid = [&](int rows) {
-    if (one_each) return static_cast<unsigned>(a.T);
-    if (SHIFT) return static_cast<unsigned>(a.T / rows + a.n + 1);
-    return static_cast<unsigned>((a.T + rows - 1) / rows);
-  };
-  if (!vec || threads > 1024) shift_residual_any_kernel<T, SHIFT><<<grid(1), 256, 0, s>>>(a);
-  else if (a.T >= kManyRows && threads <= 512 && !one_each) shift_residual_kernel<T, V, kRows, SHIFT><<<grid(kRows), threads, 0, s>>>(a);
-  else shift_residual_kernel<T, V, 1, SHIFT><<<grid(1), threads, 0, s>>>(a);
+  // long walks save rows that are worked out twice and keep loads in flight; short ones fill the GPU with few rows
+  a.rows = one_each ? 1 : a.T >= 148 * 16 ? kMaxRows : a.T >= 148 * 4 ? 2 : 1;
+  const bool any = !vec || threads > 1024 || a.top > 8;
+  if (any) a.rows = 1;
+  const unsigned grid = static_cast<unsigned>(one_each ? a.T : SHIFT ? a.T / a.rows + a.n + 1 : (a.T + a.rows - 1) / a.rows);
+  if (any) shift_residual_any_kernel<T, SHIFT><<<grid, 256, 0, s>>>(a);
+  else if (a.top == 0) shift_residual_kernel<T, 0, SHIFT><<<grid, threads, 0, s>>>(a);
+  else if (a.top <= 2) shift_residual_kernel<T, 2, SHIFT><<<grid, threads, 0, s>>>(a);
+  else if (a.top <= 4) shift_residual_kernel<T, 4, SHIFT><<<grid, threads, 0, s>>>(a);
+  else shift_residual_kernel<T, 8, SHIFT><<<grid, threads, 0, s>>>(a);
 }
 
 }  // namespace
@@ -356,7 +392,7 @@ extern "C" int b200_shift_residual(const float* x, float* x_out, const int64_t* 
   }
   if (rows > 2147483647 - num_seqs) return B200_ERR_TOO_LARGE;
   ShArgs a{x, x_out, tokens, embed, vocab, embed_scale, y, row_weight, slot_to_row, top, gain, shift, state, state_slots,
-           num_slots, cu_seqlens_q, cu_seqlens_k, context_lens, num_seqs, final_norm, final_gain, eps, h, rows, d, status};
+           num_slots, cu_seqlens_q, cu_seqlens_k, context_lens, num_seqs, final_norm, final_gain, eps, h, rows, d, status, 1};
   const int V = dtype == B200_DTYPE_F32 ? 4 : 8;
   bool vec = d % V == 0;
   for (const void* p : {static_cast<const void*>(x), static_cast<const void*>(x_out), embed, y, static_cast<const void*>(shift),

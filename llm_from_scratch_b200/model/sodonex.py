@@ -98,6 +98,13 @@ class SodonexConfig:
         return out
 
 
+def _number(p: Params, name: str) -> float:
+    t = p.raw(name)
+    if t.numel() != 1:
+        raise ValueError(f"{p.prefix + name} must be a single number, not {tuple(t.shape)}")
+    return float(t)
+
+
 class SodonexBlock(nn.Module):
     def __init__(self, p: Params, cfg: SodonexConfig, c: SodonexLayer):
         super().__init__()
@@ -106,11 +113,11 @@ class SodonexBlock(nn.Module):
         self.mixer = SigmoidAttention(p.at("mix."), d, c.heads, c.kv_heads, c.dim, c.conv, c.scale, c.rot_dims, c.rot_base, c.chunk,
                                       cfg.eps)
         # what the sublayers' normed results are multiplied by on their way into the residual
-        self.gain1 = cfg.residual_mult * float(p.raw("norm1", ()))
+        self.gain1 = cfg.residual_mult * _number(p, "norm1")
         self.mlp, self.gain2 = None, 0.0
         if c.experts:
             self.mlp = SoftmaxMoE(p.at("mlp."), d, c.d_ff, c.experts, c.top)
-            self.gain2 = cfg.residual_mult * float(p.raw("norm2", ()))
+            self.gain2 = cfg.residual_mult * _number(p, "norm2")
 
 
 class SodonexLM(TokenHead, nn.Module):
@@ -127,7 +134,7 @@ class SodonexLM(TokenHead, nn.Module):
         p = Params(weights, self.device, dtype)
         self.embed = p.lin("embed", (cfg.vocab_size, cfg.d_model))
         self.layers = nn.ModuleList([SodonexBlock(p.at(f"l{i}."), cfg, c) for i, c in enumerate(cfg.layers)])
-        self.final_gain = float(p.raw("final.norm", ()))
+        self.final_gain = _number(p, "final.norm")
         self.w_head, self.b_head = p.lin("head", (cfg.vocab_size, cfg.d_model)), None
         # steps of whole prompts can be captured: every layer's attention then takes its grid from a tile list
         self.captures_prompts = all(layer.mixer.tile_rows(dtype) for layer in self.layers)
