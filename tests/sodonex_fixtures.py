@@ -47,7 +47,7 @@ def weights(cfg, seed=0, dtype=torch.bfloat16):
         if lay["mlp"]:
             n = lay["mlp"]["router"]["experts"]
             r = w[f"l{i}.mlp.router"]
-            r *= 0.04
+            r *= 0.04 / max(cfg["embedding"]["scale"], 1.0)
             r[:, first:first + E] = 0
             r[torch.arange(n), first + torch.randperm(E, generator=g)[:n]] = 1.0
             w[f"l{i}.mlp.router.b"] *= 0.1
